@@ -92,15 +92,29 @@ class Config:
         if model_package.is_package(path):
             self._package_root = path
             path, self._manifest = model_package.resolve_package(path, provider)
+        self._dir = path
+        if not os.path.exists(os.path.join(path, "genai_config.json")):
+            # a checkpoint that is a model directory as it is (config.json + weights): its genai_config.json is made in memory
+            from .models import stack_checkpoint
+            cfg = stack_checkpoint.read_stack_config(path)
+            if cfg is not None:
+                self._c = native.Config.from_json(json.dumps(stack_checkpoint.genai_config_of(cfg, provider or "cuda")), overlay)
+                self._model_data = {}
+                return
         self._c = native.Config(path, overlay)
         self._model_data: Dict[str, bytes] = {}
+
+    @property
+    def config_path(self) -> str:
+        """The model directory."""
+        return self._dir
 
     @property
     def tokenizer_path(self) -> str:
         """Directory of the tokenizer files: the model directory, a relative `model.tokenizer_dir` under it, or a shared
         asset of the package (`sha256:<hex>[/tail]`)."""
         from . import model_package
-        return model_package.resolve_asset(self._c.config_path, self._c.tokenizer_dir, self._package_root, self._manifest)
+        return model_package.resolve_asset(self.config_path, self._c.tokenizer_dir, self._package_root, self._manifest)
 
     def __getattr__(self, name):
         return getattr(self._c, name)
@@ -165,7 +179,11 @@ class Model:
         from .models import marian, transducer
         if self.type not in LLM_TYPES + VLM_TYPES + ALM_TYPES + [marian.MODEL_TYPE] + list(transducer.MODEL_TYPES):
             raise RuntimeError(f"Unsupported model type: {self.type}")
-        self.dtype = torch.bfloat16 if want_cuda else torch.float32
+        # "compute_dtype": "float32" of the cuda provider: 32-bit weights, activations and products (declared stacks)
+        want = next((dict(o).get("compute_dtype", "bfloat16") for p, o in c.decoder["provider_options"] if p == "cuda"), "bfloat16")
+        if want not in ("bfloat16", "float32"):
+            raise RuntimeError(f"compute_dtype={want} is not supported (bfloat16 or float32)")
+        self.dtype = torch.bfloat16 if want_cuda and want == "bfloat16" else torch.float32
         from .models.loader import load_decoder
         t_load = time.perf_counter()
         with _Trace("model", "load"):
@@ -400,7 +418,7 @@ class SequenceState:
                        block_table=self.block_table[rows_used].contiguous() if len(rows_used) != self.rows else self.block_table,
                        logits_rows=None if want_all_logits else i32(last),
                        max_q_len=max(len(t) for t in row_tokens if t), max_kv_len=max(self.kv_len), inputs_embeds=inputs_embeds,
-                       min_q_len=min(len(t) for t in row_tokens if t),
+                       min_q_len=min(len(t) for t in row_tokens if t), host_lens=[(p, len(row_tokens[r])) for p, r in zip(past, rows_used)],
                        state_slots=i32(rows_used) if self.decoder.arch.has_linear_layers else None,
                        **self._cross_fields(rows_used))
         if mrope:
@@ -563,8 +581,9 @@ class SequenceState:
             ar = torch.arange(bs, device=dev)
             s_idx, d_idx = (src[:, None] * bs + ar).reshape(-1), (dst[:, None] * bs + ar).reshape(-1)
             self.kv.full[:, :, d_idx] = self.kv.full[:, :, s_idx]
-            if self.kv.conv is not None:
-                self.kv.conv[:, d_idx] = self.kv.conv[:, s_idx]
+            for pool in (self.kv.conv, self.kv.latent):
+                if pool is not None:
+                    pool[:, d_idx] = pool[:, s_idx]
             self._moves = []
         if self._tbl_dirty:
             self.block_table.copy_(torch.from_numpy(self._tbl))

@@ -32,6 +32,9 @@ C_API_SO = os.path.join(C_API_DIR, "libogb200_genai.so")
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v"]
+# Sources compiled without --use_fast_math: recurrences, 32-bit models and the norms of an fp32 residual stream keep IEEE division,
+# square roots and denormals.
+PRECISE_SOURCES = {"gemm_simt.cu", "latent_attention.cu", "layer_ops.cu", "linear_attention.cu"}
 
 
 def _newer(sources, target) -> bool:
@@ -86,7 +89,8 @@ def build_kernels(force=False, verbose=False) -> str:
     def compile_one(src):
         obj = os.path.join(BUILD_DIR, "csrc", os.path.basename(src) + ".o")
         if force or _newer([src] + hdrs, obj):
-            logs.append((src, _run([nvcc, *NVCC_FLAGS, "-I" + CSRC_DIR, "-c", src, "-o", obj], verbose)))
+            flags = [f for f in NVCC_FLAGS if f != "--use_fast_math"] if os.path.basename(src) in PRECISE_SOURCES else NVCC_FLAGS
+            logs.append((src, _run([nvcc, *flags, "-I" + CSRC_DIR, "-c", src, "-o", obj], verbose)))
         return obj
 
     with ThreadPoolExecutor(max_workers=8) as ex:

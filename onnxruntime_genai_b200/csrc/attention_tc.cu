@@ -27,6 +27,12 @@
 // word; the producers and the issuer leave their loops, the softmax warps keep walking theirs without waiting (they share a
 // named barrier per warp pair, which has no time limit, so none of them may leave early), the producer waits (bounded) for
 // copies in flight, TMEM is freed and the kernel returns.
+// The latent form (LAT) serves long prompts of latent-attention layers: keys and values of the request's visible positions were
+// expanded into dense matrices beforehand ([rows, H * dim] and [rows, H * vdim] column ranges of one product, and the rotated key
+// part that all heads share as columns of the gathered latents), so a row of K is put together from two tensor maps (the head's
+// unrotated part, then the shared rotated part, each padded to 64 columns that meet zeros in Q), and key position j of request b
+// is dense row row_base[b] + j - first_kv[b] instead of a block-table lookup.  Every head has keys of its own: one CTA = (request,
+// head, 128 tokens).
 // The cache must hold finite values in every slot of a block that is in use (PagedKVCache allocates zeros): keys past the end
 // of a request inside its last 16-key group are masked (P = 0) but still multiplied.
 #include <cstdlib>
@@ -47,6 +53,13 @@ constexpr int TCA_REGS_SOFTMAX = 224, TCA_REGS_OTHER = 40;   // after setmaxnreg
 constexpr float TCA_LOG2E = 1.4426950408889634f;
 constexpr float TCA_RESCALE_GAP = 8.f;   // log2 units
 
+// Latent form: where a request's expanded rows start, and how a head's columns are laid out (see LAT above).
+struct TcLatent {
+  const int32_t *row_base, *first_kv;      // per request of the batch; row_base < 0: the request is not served here
+  int dim, rot, vdim;                      // a query head is (dim | rot) columns of q
+  int kr_col;                              // column of the shared rotated part in its matrix
+};
+
 struct TcAttnParams {
   const __nv_bfloat16* q; int q_stride;
   const int32_t* cu_seqlens; const int32_t* past_lens;
@@ -56,22 +69,26 @@ struct TcAttnParams {
   float scale, softcap;
   int window, B, Hq, Hkv, min_rows;
   int* status;
+  TcLatent lat;
 };
 
-template <int D, int BN>
+template <int DK, int DV, int BN>
 struct TcaCfg {
-  static constexpr int HALVES = D / 64;
-  static constexpr int Q_BYTES = TCA_BM * D * 2;
-  static constexpr int KV_TILE = BN * D * 2;                 // one K (or V) tile
+  static constexpr int K_HALVES = DK / 64, V_HALVES = DV / 64;
+  static constexpr int Q_BYTES = TCA_BM * DK * 2;
+  static constexpr int K_TILE = BN * DK * 2, V_TILE = BN * DV * 2;
   // K and V tiles have rings of their own: a K tile is free as soon as its Q K^T is done (one tile period earlier than the
   // V tile of the same keys), and the loads must run two to three tile periods ahead of their use to hide their latency.
   static constexpr int BUDGET = 227 * 1024 - 1024 - 1536 - Q_BYTES;      // 1 KiB of alignment slack, static shared memory
-  static constexpr int RING = BUDGET / KV_TILE >= 8 ? 8 : BUDGET / KV_TILE;
-  static constexpr int K_STAGES = (RING + 1) / 2, V_STAGES = RING / 2;
-  static constexpr int SMEM = 1024 + Q_BYTES + (K_STAGES + V_STAGES) * KV_TILE;
+  static constexpr int PAIRS = BUDGET / (K_TILE + V_TILE) >= 4 ? 4 : BUDGET / (K_TILE + V_TILE);
+  static constexpr int V_STAGES = PAIRS;
+  static constexpr int K_STAGES = PAIRS < 4 && BUDGET - PAIRS * (K_TILE + V_TILE) >= K_TILE ? PAIRS + 1 : PAIRS;
+  static_assert(PAIRS >= 2, "the rings need two stages each");
+  static constexpr int SMEM = 1024 + Q_BYTES + K_STAGES * K_TILE + V_STAGES * V_TILE;
   static constexpr int S_BUFS = 3;
   static constexpr int S_COLS = BN, O_COL = S_BUFS * BN;
-  static constexpr int COLS_USED = S_BUFS * BN + D;
+  static constexpr int COLS_USED = S_BUFS * BN + DV;
+  static_assert(COLS_USED <= 512, "scores and output must fit in tensor memory");
   static constexpr int TMEM_COLS = COLS_USED <= 128 ? 128 : (COLS_USED <= 256 ? 256 : 512);
   static constexpr int CTAS_PER_SM = 1;
 };
@@ -107,16 +124,19 @@ __device__ __forceinline__ void umma_f16_ta(uint32_t tmem_d, uint32_t tmem_a, ui
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
-template <int D, int BN>
-__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<D, BN>::CTAS_PER_SM)
-attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, TcAttnParams p) {
-  using Cfg = TcaCfg<D, BN>;
-  constexpr int HALVES = Cfg::HALVES, KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
+// DK: width of the staged query and key rows; DV: width of the value rows; LAT: the latent form, whose first NOPE of the DK columns
+// are the unrotated part.
+template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK>
+__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN>::CTAS_PER_SM)
+attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_r,
+                    TcAttnParams p) {
+  using Cfg = TcaCfg<DK, DV, BN>;
+  constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ __align__(128) uint8_t smem_dyn[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;                                  // [HALVES][128 rows][128 B]
   uint8_t* sK = sQ + Cfg::Q_BYTES;                     // [KS][HALVES][BN keys][128 B]
-  uint8_t* sV = sK + KS * Cfg::KV_TILE;                // [VS][HALVES][BN keys][128 B]
+  uint8_t* sV = sK + KS * Cfg::K_TILE;                 // [VS][HALVES][BN keys][128 B]
   __shared__ uint64_t k_full[KS], k_empty[KS], v_full[VS], v_empty[VS], s_full[Cfg::S_BUFS], p_full[Cfg::S_BUFS], o_done[Cfg::S_BUFS], q_full;
   __shared__ uint32_t tmem_slot;
   __shared__ int abort_flag;
@@ -135,6 +155,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   // the tail of the grid is made of short CTAs
   const int row0 = int(gridDim.x - 1 - blockIdx.x) * TCA_BM;
   if (rows < p.min_rows || row0 >= rows) return;      // before anything is allocated
+  if (LAT && p.lat.row_base[b] < 0) return;
   const int past = p.past_lens[b];
   const bool full = p.window < 0;
   const int32_t* table = p.block_table + size_t(b) * p.table_cols;
@@ -143,6 +164,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   int kv_lo = 0;
   if (p.window > 0) kv_lo = max(0, past + row0 / G - p.window + 1);
   const int tile_begin = kv_lo / BN;
+  const int lat_row0 = LAT ? p.lat.row_base[b] - p.lat.first_kv[b] : 0;      // dense row of key position 0 (may be negative)
+  const int lat_first = LAT ? p.lat.first_kv[b] : 0;                          // positions before it were not expanded (never visible)
   const int n_tiles = kv_hi > kv_lo ? (kv_hi + BN - 1) / BN - tile_begin : 0;
 
   if (tid == 0) {
@@ -179,22 +202,37 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     uint64_t* empty = is_k ? k_empty : v_empty;
     uint8_t* ring = is_k ? sK : sV;
     const int NS = is_k ? KS : VS;
+    const int tile_bytes = is_k ? Cfg::K_TILE : Cfg::V_TILE;
     if (lane == 0) tma_prefetch_desc(tmap);
     const int last_group = max(0, (kv_hi - 1) / 16 * 16);
     int issued = 0;
     for (int it = 0; it < n_tiles; ++it) {
       const int st = it % NS;
       if (it >= NS && !mbar_wait_bounded(&empty[st], ((it / NS) - 1) & 1, abort_p)) { if (lane == 0) fail(OGB_ERR_WAIT_TMA); break; }
-      if (lane == 0) mbar_expect_tx(&full[st], Cfg::KV_TILE);
+      if (lane == 0) mbar_expect_tx(&full[st], tile_bytes);
       __syncwarp();
       // Key groups past the end of the range re-read the last valid group (their scores are masked), so every stage
       // receives the same byte count.
       if (lane < BN / 16) {
-        const int j0 = min((tile_begin + it) * BN + lane * 16, last_group);
-        const int slot0 = table[j0 / p.block_size] * p.block_size + j0 % p.block_size;
-        uint8_t* dst = ring + st * Cfg::KV_TILE + lane * 16 * 128;
+        int j0 = min((tile_begin + it) * BN + lane * 16, last_group);
+        uint8_t* dst = ring + st * tile_bytes + lane * 16 * 128;
+        if constexpr (LAT) {
+          j0 = max(j0, lat_first);                     // (key groups ahead of the first expanded row are masked as well)
+          if (is_k) {
 #pragma unroll
-        for (int h = 0; h < HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh * D + h * 64, slot0);
+            for (int h = 0; h < Cfg::K_HALVES; ++h) {
+              if (h < NOPE / 64) tma_load_2d(dst + h * (BN * 128), &tmap_k, &full[st], kvh * p.lat.dim + h * 64, lat_row0 + j0);
+              else tma_load_2d(dst + h * (BN * 128), &tmap_r, &full[st], p.lat.kr_col + (h - NOPE / 64) * 64, lat_row0 + j0);
+            }
+          } else {
+#pragma unroll
+            for (int h = 0; h < Cfg::V_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), &tmap_v, &full[st], kvh * p.lat.vdim + h * 64, lat_row0 + j0);
+          }
+        } else {
+          const int slot0 = table[j0 / p.block_size] * p.block_size + j0 % p.block_size;
+#pragma unroll
+          for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh * DK + h * 64, slot0);
+        }
       }
       issued = it + 1;
     }
@@ -208,7 +246,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   } else if (warp == TCA_MMA_WARP) {
     // ------------------------------------------------------------------------------ MMA issuer
     constexpr uint32_t idesc_qk = umma_idesc_f16(TCA_BM, BN, 1);
-    constexpr uint32_t idesc_pv = umma_idesc_f16(TCA_BM, D, 1) | (1u << 16);     // B operand MN-major
+    constexpr uint32_t idesc_pv = umma_idesc_f16(TCA_BM, DV, 1) | (1u << 16);    // B operand MN-major
     const uint32_t q_addr = smem_u32(sQ), k_ring = smem_u32(sK), v_ring = smem_u32(sV);
     constexpr uint32_t lbo = BN * 128, sbo = 1024;       // between the 64-dim halves of V; between 8-key groups
     bool ok = mbar_wait_bounded(&q_full, 0, abort_p);
@@ -218,9 +256,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       if (!mbar_wait_bounded(&k_full[st], (it / KS) & 1, abort_p)) return false;
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t k_addr = k_ring + st * Cfg::KV_TILE;
+        const uint32_t k_addr = k_ring + st * Cfg::K_TILE;
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
           const uint64_t da = umma_desc_sw128(q_addr + (ks >> 2) * (TCA_BM * 128) + (ks & 3) * 32);
           const uint64_t db = umma_desc_sw128(k_addr + (ks >> 2) * (BN * 128) + (ks & 3) * 32);
           umma_f16(tmem_base + (it % Cfg::S_BUFS) * Cfg::S_COLS, da, db, idesc_qk, ks > 0);
@@ -242,7 +280,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       if (!mbar_wait_bounded(&v_full[st], (it / VS) & 1, abort_p)) { if (lane == 0) fail(OGB_ERR_WAIT_TMA); ok = false; break; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t v_addr = v_ring + st * Cfg::KV_TILE;
+        const uint32_t v_addr = v_ring + st * Cfg::V_TILE;
 #pragma unroll
         for (int ks = 0; ks < BN / 16; ++ks) {
           const uint64_t db = umma_desc_sw128_mn(v_addr + ks * 16 * 128, lbo, sbo);
@@ -260,7 +298,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     // ------------------------------------------------------------------------------ softmax warps
     asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(TCA_REGS_SOFTMAX));
     constexpr int HC = BN / 2;                 // key columns per thread and tile
-    constexpr int OC = D / 2;                  // output columns per thread
+    constexpr int OC = DV / 2;                 // output columns per thread
     const int quarter = warp & 3, half = warp >> 2;
     const int r = quarter * 32 + lane;
     const int gr = row0 + r;
@@ -273,12 +311,16 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     // still arrives at every barrier its partner arrives at.
     auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory"); };
     {
-      const __nv_bfloat16* src = p.q + size_t(tok0 + tq) * p.q_stride + size_t(hq) * D;
+      const __nv_bfloat16* src = p.q + size_t(tok0 + tq) * p.q_stride + size_t(hq) * (LAT ? p.lat.dim + p.lat.rot : DK);
 #pragma unroll
-      for (int cc = 0; cc < D / 16; ++cc) {
-        const int c = half * (D / 16) + cc;
+      for (int cc = 0; cc < DK / 16; ++cc) {
+        const int c = half * (DK / 16) + cc;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (valid) v = *reinterpret_cast<const uint4*>(src + c * 8);
+        if constexpr (LAT) {
+          // columns past a part's own width are zeros: what K holds there (other heads' columns) does not count
+          const int col = c * 8 < NOPE ? c * 8 : c * 8 - NOPE, width = c * 8 < NOPE ? p.lat.dim : p.lat.rot;
+          if (valid && col < width) v = *reinterpret_cast<const uint4*>(src + (c * 8 < NOPE ? col : p.lat.dim + col));
+        } else if (valid) v = *reinterpret_cast<const uint4*>(src + c * 8);
         *reinterpret_cast<uint4*>(sQ + (c >> 3) * (TCA_BM * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
       }
       fence_proxy_async_smem();
@@ -411,7 +453,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
         l = l * scale_o + exp2f(sk - mm);
       }
       const float inv = l > 0.f ? scale_o / l : 0.f;
-      __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * D + half * OC;
+      __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * (LAT ? p.lat.vdim : DV) + half * OC;
 #pragma unroll
       for (int c = 0; c < OC / 16; ++c) {
         uint32_t v[16];
@@ -432,8 +474,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           hi.y = pack_bf16x2(__uint_as_float(v[10]) * inv, __uint_as_float(v[11]) * inv);
           hi.z = pack_bf16x2(__uint_as_float(v[12]) * inv, __uint_as_float(v[13]) * inv);
           hi.w = pack_bf16x2(__uint_as_float(v[14]) * inv, __uint_as_float(v[15]) * inv);
-          *reinterpret_cast<uint4*>(po + c * 16) = lo;
-          *reinterpret_cast<uint4*>(po + c * 16 + 8) = hi;
+          if (!LAT || half * OC + c * 16 < p.lat.vdim) *reinterpret_cast<uint4*>(po + c * 16) = lo;
+          if (!LAT || half * OC + c * 16 + 8 < p.lat.vdim) *reinterpret_cast<uint4*>(po + c * 16 + 8) = hi;
         }
       }
     }
@@ -443,10 +485,21 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   if (warp == TCA_K_WARP) tmem_dealloc(tmem_base, Cfg::TMEM_COLS);
 }
 
+template <int NOPE, int ROT, int DV, int BN>
+static int LaunchTcLatent(const TcAttnParams& p, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr, int max_q_len, cudaStream_t stream) {
+  using Cfg = TcaCfg<NOPE + ROT, DV, BN>;
+  auto kern = attention_tc_kernel<NOPE + ROT, DV, BN, true, NOPE>;
+  static bool configured[OGB_MAX_DEVICES] = {};
+  if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
+  dim3 grid((max_q_len + TCA_BM - 1) / TCA_BM, p.Hkv, p.B);
+  launch_pdl(kern, grid, dim3(TCA_THREADS), Cfg::SMEM, stream, mk, mv, mr, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 template <int D, int BN>
 static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
-  using Cfg = TcaCfg<D, BN>;
-  auto kern = attention_tc_kernel<D, BN>;
+  using Cfg = TcaCfg<D, D, BN>;
+  auto kern = attention_tc_kernel<D, D, BN>;
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
   CUtensorMap mk, mv;
@@ -456,7 +509,7 @@ static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_ca
   if (!MakeMapBf16(&mv, v_cache, cache_slots, p.Hkv * D, p.Hkv * D, 16)) return -2;
   const int G = p.Hq / p.Hkv;
   dim3 grid((max_q_len * G + TCA_BM - 1) / TCA_BM, p.Hkv, p.B);
-  launch_pdl(kern, grid, dim3(TCA_THREADS), Cfg::SMEM, stream, mk, mv, p);
+  launch_pdl(kern, grid, dim3(TCA_THREADS), Cfg::SMEM, stream, mk, mv, mv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -478,7 +531,7 @@ OGB_API int ogb_attention_tc(const void* q, int q_stride, const void* k_cache, c
   if (!ogb_attention_tc_supported(D, block_size, 16, cache_slots)) return -5;
   if (Hkv <= 0 || Hq % Hkv || (q_stride % 8) || (out_stride % 8)) return -1;
   if (((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out)) & 15) != 0) return -1;
-  TcAttnParams p;
+  TcAttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
   p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.block_table = block_table; p.table_cols = table_cols; p.block_size = block_size;
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;
@@ -488,4 +541,47 @@ OGB_API int ogb_attention_tc(const void* q, int q_stride, const void* k_cache, c
   // 128 keys per tile (measured on B200 against 64: 457 vs 429 TFLOP/s at 4096 tokens, head_dim 128)
   if (D == 128) return LaunchTc<128, 128>(p, k_cache, v_cache, max_q_len, cache_slots, stream);
   return LaunchTc<64, 128>(p, k_cache, v_cache, max_q_len, cache_slots, stream);
+}
+
+// 1 when the latent form can serve these sizes: 16-byte pieces everywhere, unrotated part up to 192 columns, rotated part up to 64,
+// values up to 128.
+OGB_API int ogb_attention_tc_latent_supported(int dim, int rot, int vdim) {
+  return dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && dim > 0 && dim <= 192 && rot > 0 && rot <= 64 && vdim > 0 && vdim <= 128;
+}
+
+// Long prompts of a latent-attention layer.  q: row t holds H heads of (dim | rot) rotated queries; kv [rows, >= H * (dim + vdim)]: the
+// expanded keys (head-major columns) then values; kr [rows, >= kr_col + rot]: the shared rotated key part from column kr_col on.
+// row_base / first_kv [B]: dense row of each request's first expanded position (a multiple of 16) and that position; row_base < 0
+// leaves the request out.  Output row t: H heads of vdim columns.
+OGB_API int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldkv, const void* kr, int ldkr, int kr_col, int rows,
+                                    const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* row_base, const int32_t* first_kv, void* out,
+                                    int out_stride, float scale, int window, int B, int max_q_len, int H, int dim, int rot, int vdim, int* status,
+                                    void* stream_) {
+  if (B <= 0 || max_q_len <= 0 || rows <= 0) return 0;
+  if (!ogb_attention_tc_latent_supported(dim, rot, vdim)) return -5;
+  if ((q_stride % 8) || (out_stride % 8) || (ldkv % 8) || (ldkr % 8) || (kr_col % 8)) return -1;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kr) | reinterpret_cast<uintptr_t>(out)) & 15) return -1;
+  TcAttnParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
+  p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.block_size = 16;
+  p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;
+  p.scale = scale; p.window = window; p.B = B; p.Hq = H; p.Hkv = H; p.min_rows = 1; p.status = status;
+  p.lat.row_base = row_base; p.lat.first_kv = first_kv; p.lat.dim = dim; p.lat.rot = rot; p.lat.vdim = vdim; p.lat.kr_col = kr_col;
+  CUtensorMap mk, mv, mr;
+  const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(kv);
+  if ((H * dim) % 8) return -1;
+  if (!MakeMapBf16(&mk, base, rows, H * dim, ldkv, 16) || !MakeMapBf16(&mv, base + size_t(H) * dim, rows, H * vdim, ldkv, 16) ||
+      !MakeMapBf16(&mr, kr, rows, kr_col + rot, ldkr, 16))
+    return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream_);
+  // tiles of 128 keys where two stages of both rings fit beside the query tile, else 64
+  const int nope = (dim + 63) / 64;
+  if (vdim <= 64) {
+    if (nope == 1) return LaunchTcLatent<64, 64, 64, 128>(p, mk, mv, mr, max_q_len, s);
+    if (nope == 2) return LaunchTcLatent<128, 64, 64, 128>(p, mk, mv, mr, max_q_len, s);
+    return LaunchTcLatent<192, 64, 64, 64>(p, mk, mv, mr, max_q_len, s);
+  }
+  if (nope == 1) return LaunchTcLatent<64, 64, 128, 128>(p, mk, mv, mr, max_q_len, s);
+  if (nope == 2) return LaunchTcLatent<128, 64, 128, 128>(p, mk, mv, mr, max_q_len, s);
+  return LaunchTcLatent<192, 64, 128, 64>(p, mk, mv, mr, max_q_len, s);
 }

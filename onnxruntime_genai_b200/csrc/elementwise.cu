@@ -314,7 +314,7 @@ struct ShortConvParams {
   const uint4* bcx; int bcx_stride;       // [T, 3C] bf16, stride in elements
   const __nv_bfloat16* weight;            // [C, L]
   const __nv_bfloat16* bias;              // [C] or null
-  uint4* cache;                           // [slots, C]
+  uint4* cache; int cache_vecs;           // [slots, C] rows, a row stride of cache_vecs 16-byte pieces
   const int32_t* slots; const int32_t* positions; const int32_t* cu_seqlens; const int32_t* past_lens;
   const int32_t* block_table; int table_cols, block_size;
   uint4* out;                             // [T, C]
@@ -362,13 +362,13 @@ __global__ void __launch_bounds__(256) short_conv_kernel(ShortConvParams p) {
         if (k == 0) mine = e;
       } else {
         const int blk = table[q / p.block_size];
-        e = p.cache[(size_t(blk) * p.block_size + q % p.block_size) * nvec + v];
+        e = p.cache[(size_t(blk) * p.block_size + q % p.block_size) * p.cache_vecs + v];
       }
       const __nv_bfloat16* ee = reinterpret_cast<const __nv_bfloat16*>(&e);
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] += bf2f(p.weight[size_t(v * 8 + j) * p.L + (p.L - 1 - k)]) * bf2f(ee[j]);
     }
-    if (slot >= 0) p.cache[size_t(slot) * nvec + v] = mine;
+    if (slot >= 0) p.cache[size_t(slot) * p.cache_vecs + v] = mine;
     uint4 o;
     __nv_bfloat16* oe = reinterpret_cast<__nv_bfloat16*>(&o);
     if (!p.plain) {
@@ -566,34 +566,34 @@ OGB_API int ogb_act(const void* x, void* out, long long n, int act, void* stream
 
 static int LaunchShortConv(const void* bcx, int bcx_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                            const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
-                           int table_cols, int block_size, void* out, int T, int B, int C, int L, int plain, int silu, void* stream);
+                           int table_cols, int block_size, void* out, int T, int B, int C, int L, int cache_stride, int plain, int silu, void* stream);
 
 OGB_API int ogb_short_conv(const void* bcx, int bcx_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                            const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
                            int table_cols, int block_size, void* out, int T, int B, int C, int L, void* stream) {
   return LaunchShortConv(bcx, bcx_stride, weight, bias, cache, slots, positions, cu_seqlens, past_lens, block_table, table_cols, block_size, out,
-                         T, B, C, L, 0, 0, stream);
+                         T, B, C, L, C, 0, 0, stream);
 }
 
 // The causal depthwise convolution without gates (x [T, C] with a row stride, e.g. a slice of a wider projection), optional SiLU:
 // the CausalConvWithState op of the gated-delta-net and Mamba-2 layers over the same paged window.
 OGB_API int ogb_causal_conv(const void* x, int x_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                             const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
-                            int table_cols, int block_size, void* out, int T, int B, int C, int L, int silu, void* stream) {
+                            int table_cols, int block_size, void* out, int T, int B, int C, int L, int cache_stride, int silu, void* stream) {
   if (reinterpret_cast<uintptr_t>(x) & 15) return -1;
   return LaunchShortConv(x, x_stride, weight, bias, cache, slots, positions, cu_seqlens, past_lens, block_table, table_cols, block_size, out,
-                         T, B, C, L, 1, silu, stream);
+                         T, B, C, L, cache_stride, 1, silu, stream);
 }
 
 static int LaunchShortConv(const void* bcx, int bcx_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                            const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
-                           int table_cols, int block_size, void* out, int T, int B, int C, int L, int plain, int silu, void* stream) {
+                           int table_cols, int block_size, void* out, int T, int B, int C, int L, int cache_stride, int plain, int silu, void* stream) {
   if (T <= 0) return 0;
-  if (B <= 0 || (C % 8) || (bcx_stride % 8) || L < 1 || L > 16 || block_size <= 0) return -1;
+  if (B <= 0 || (C % 8) || (bcx_stride % 8) || (cache_stride % 8) || L < 1 || L > 16 || block_size <= 0) return -1;
   ShortConvParams p;
   p.bcx = static_cast<const uint4*>(bcx); p.bcx_stride = bcx_stride;
   p.weight = static_cast<const __nv_bfloat16*>(weight); p.bias = static_cast<const __nv_bfloat16*>(bias);
-  p.cache = static_cast<uint4*>(cache); p.slots = slots; p.positions = positions; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens;
+  p.cache = static_cast<uint4*>(cache); p.cache_vecs = cache_stride / 8; p.slots = slots; p.positions = positions; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens;
   p.block_table = block_table; p.table_cols = table_cols; p.block_size = block_size; p.out = static_cast<uint4*>(out);
   p.T = T; p.B = B; p.C = C; p.L = L; p.plain = plain; p.silu = silu;
   const int threads = min(256, max(32, (C / 8 + 31) / 32 * 32));

@@ -59,6 +59,11 @@ struct GroupParams {
   const int* num_tiles;     // device scalar: tiles in use; CTAs beyond it return at once
 };
 
+// A batch of products that share A's rows (per-head projections): problem z multiplies the K columns of A that start at
+// z * a_cols with weight rows [z * N, (z + 1) * N) and writes C + z * c_cols.  K columns past a problem's own may hold other
+// problems' values: the weight map ends at K, so they meet zeros.  m_tiles > 0 switches it on (blockIdx.y = z * m_tiles + tile).
+struct BatchParams { int m_tiles, a_cols, c_cols; };
+
 // Rotary embedding + KV-cache append fused into the epilogue of a QKV projection (positions == nullptr: off).  Output
 // columns are [Hq query heads | Hkv key heads | Hkv value heads] of D each; the rotation pairs element i with i + rot / 2
 // (the non-interleaved form); keys and values go to row `slots[m]` of the caches [slots, Hkv, D] (slot < 0: nowhere).
@@ -80,12 +85,15 @@ struct GemmParams {
   int out_fp32;         // 0 bf16, 1 fp32, 2 fp16 output
   int act_pair;         // tiles hold 64 gate rows + 64 up rows, output has N/2 columns: 1 = silu(gate)*up,
                         // 2 = clamped SwiGLU: g = min(gate, limit), u = clamp(up, +-limit), g*sigmoid(alpha*g)*(u+1)
+                        // 3 = max(gate, 0)*up
   float act_alpha, act_limit;
-  const __nv_bfloat16* residual;
+  const void* residual;
   int ldr;
+  int res_fp32;         // the residual rows are fp32 (an fp32 residual stream), else bf16
   const __nv_bfloat16* bias;
   int* status;
   int pdl;
+  BatchParams bat;
   CommParams comm;
   int comm_epilogue;    // 1: the epilogue runs the fused all-reduce / reduce-scatter (and the call closes an epoch)
   int ag_rows;          // > 0: all-gather -> GEMM: the activations are not read through the tensor map but assembled from the
@@ -240,14 +248,24 @@ __device__ __forceinline__ uint32_t comm_open_call(const CommParams& c, unsigned
 // every inlined copy of this routine (three output types, vector and tail forms) costs instruction-cache misses.
 struct StoreArgs {
   void* C;
-  const __nv_bfloat16* residual;
+  const void* residual;
   int ldc, ldr, out_kind, n_out;    // out_kind: 0 bf16, 1 fp32, 2 fp16
+  int res_fp32;
 };
 static __device__ __noinline__ void epi_store8(const StoreArgs a, int m, int col, float4 lo, float4 hi) {
   float v[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
   const bool full = col + 8 <= a.n_out;
-  if (a.residual) {
-    const __nv_bfloat16* r = a.residual + size_t(m) * a.ldr + col;
+  if (a.residual && a.res_fp32) {
+    const float* r = static_cast<const float*>(a.residual) + size_t(m) * a.ldr + col;
+    if (full && (reinterpret_cast<uintptr_t>(r) & 15) == 0) {
+      const float4 x = *reinterpret_cast<const float4*>(r), y = *reinterpret_cast<const float4*>(r + 4);
+      v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w; v[4] += y.x; v[5] += y.y; v[6] += y.z; v[7] += y.w;
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) if (col + j < a.n_out) v[j] += r[j];
+    }
+  } else if (a.residual) {
+    const __nv_bfloat16* r = static_cast<const __nv_bfloat16*>(a.residual) + size_t(m) * a.ldr + col;
     if (full && (reinterpret_cast<uintptr_t>(r) & 15) == 0) {
       const uint4 q = *reinterpret_cast<const uint4*>(r);
       const float2 x0 = unpack_bf16x2(q.x), x1 = unpack_bf16x2(q.y), x2 = unpack_bf16x2(q.z), x3 = unpack_bf16x2(q.w);
@@ -344,7 +362,12 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, uint8_t* smem
     const int n_out = p.act_pair ? p.N / 2 : p.N;    // output columns of the whole problem
     const int col0 = n_tile * (p.act_pair ? 64 : 128);
     const uint32_t part_addr = smem_u32(part);
-    const StoreArgs sa{p.C, p.residual, p.ldc, p.ldr, p.out_fp32, n_out};
+    void* C = p.C;
+    if (p.bat.m_tiles > 0) {
+      const size_t off = size_t(blockIdx.y / p.bat.m_tiles) * p.bat.c_cols;
+      C = p.out_fp32 == 1 ? static_cast<void*>(static_cast<float*>(C) + off) : static_cast<void*>(static_cast<__nv_bfloat16*>(C) + off);
+    }
+    const StoreArgs sa{C, p.residual, p.ldc, p.ldr, p.out_fp32, n_out, p.res_fp32};
 
     // sum over the split-K cluster of 8 accumulators of token column mc, weight rows n_local.., scaled by the folded norm
     auto reduce8 = [&](int mc, int n_local, float scale, float (&v)[8]) {
@@ -407,6 +430,9 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, uint8_t* smem
         if (p.act_pair == 1) {
 #pragma unroll
           for (int j = 0; j < 8; ++j) v[j] = silu(v[j]) * u[j];
+        } else if (p.act_pair == 3) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[j] = fmaxf(v[j], 0.f) * u[j];
         } else {
 #pragma unroll
           for (int j = 0; j < 8; ++j) {

@@ -1,0 +1,86 @@
+// Linear layers outside the tensor cores: true fp32 products of the 32-bit models (fp32 operands, fp32 multiply-adds, no reduced
+// precision mode), and bf16 products whose sizes or addresses TMA cannot take (strides that are not multiples of 16 bytes).
+//   C[m, z * c_cols + n] = sum_k A[m, z * a_cols + k] * W[z * N + n, k]   (+ residual[m, n], fp32)
+// One CTA = a 64 x 64 output tile, 16 columns of K at a time through shared memory, 4 x 4 outputs per thread.
+#include "common.cuh"
+#include "kernels.h"
+
+namespace ogb {
+
+struct SimtGemmParams {
+  const void* A; const void* W; void* C; const float* residual;
+  int lda, a_cols, ldw, ldc, c_cols, ldr;
+  int M, N, K;
+};
+
+template <typename T> __device__ __forceinline__ float ld_f32(const T* p);
+template <> __device__ __forceinline__ float ld_f32<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ld_f32<__nv_bfloat16>(const __nv_bfloat16* p) { return bf2f(*p); }
+
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256) gemm_simt_kernel(SimtGemmParams p) {
+  constexpr int BM = 64, BN = 64, BK = 16;
+  __shared__ float sA[BK][BM + 4], sW[BK][BN + 4];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int z = blockIdx.z, m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
+  const T* A = static_cast<const T*>(p.A) + size_t(z) * p.a_cols;
+  const T* W = static_cast<const T*>(p.W) + size_t(z) * p.N * p.ldw;
+  const int tid = threadIdx.x, tx = tid % 16, ty = tid / 16;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < p.K; k0 += BK) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int idx = tid + i * 256, r = idx / BK, k = idx % BK;
+      sA[k][r] = (m0 + r < p.M && k0 + k < p.K) ? ld_f32(A + size_t(m0 + r) * p.lda + k0 + k) : 0.f;
+      sW[k][r] = (n0 + r < p.N && k0 + k < p.K) ? ld_f32(W + size_t(n0 + r) * p.ldw + k0 + k) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < BK; ++k) {
+      float a[4], w[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { a[i] = sA[k][ty * 4 + i]; w[i] = sW[k][tx * 4 + i]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], w[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= p.M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= p.N) continue;
+      float v = acc[i][j];
+      if (p.residual) v += p.residual[size_t(m) * p.ldr + n];
+      TO* dst = static_cast<TO*>(p.C) + size_t(m) * p.ldc + size_t(z) * p.c_cols + n;
+      if constexpr (sizeof(TO) == 4) *dst = v; else *dst = f2bf(v);
+    }
+  }
+}
+
+}  // namespace ogb
+
+using namespace ogb;
+
+// in_fp32 / out_fp32: element types of A and W / of C (else bf16).  residual (fp32, may be C itself) only with batch == 1.
+OGB_API int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K,
+                          int batch, const float* residual, int ldr, int in_fp32, int out_fp32, void* stream_) {
+  if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
+  if (residual && batch != 1) return -1;
+  if (M > 64 * 65535 || batch > 65535) return -1;
+  SimtGemmParams p{A, W, C, residual, lda, a_cols, ldw, ldc, c_cols, ldr, M, N, K};
+  const dim3 grid((N + 63) / 64, (M + 63) / 64, batch);
+  auto s = static_cast<cudaStream_t>(stream_);
+  bool ok;
+  if (in_fp32) ok = out_fp32 ? launch_pdl(gemm_simt_kernel<float, float>, grid, dim3(256), 0, s, p)
+                             : launch_pdl(gemm_simt_kernel<float, __nv_bfloat16>, grid, dim3(256), 0, s, p);
+  else ok = out_fp32 ? launch_pdl(gemm_simt_kernel<__nv_bfloat16, float>, grid, dim3(256), 0, s, p)
+                     : launch_pdl(gemm_simt_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(256), 0, s, p);
+  return ok ? 0 : -4;
+}

@@ -63,12 +63,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
   float* ssq = reinterpret_cast<float*>(smem + Cfg::SSQ_OFFSET);   // [BT] sums of squares of the activation rows (folded norm)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n_tile = blockIdx.x, m_tile = blockIdx.y, split = blockIdx.z;
+  const int n_tile = blockIdx.x, split = blockIdx.z;
+  const int batch = p.bat.m_tiles > 0 ? blockIdx.y / p.bat.m_tiles : 0;        // problem of a batched launch
+  const int m_tile = blockIdx.y - batch * p.bat.m_tiles;
+  const int a_col0 = batch * p.bat.a_cols;
   const int kb0 = split * p.kb_per_split;
   const int num_kb = min(p.kb_per_split, p.total_kb - kb0);
   // Grouped mode: the tile list is written by the kernel before this one, so nothing is read ahead of it.
   const bool grouped = p.grp.tile_expert != nullptr;
-  int row0 = m_tile * BT, rows = min(BT, p.M - row0), w_row0 = 0;
+  int row0 = m_tile * BT, rows = min(BT, p.M - row0), w_row0 = batch * p.N;
   if (grouped) {
     if (p.pdl) pdl_wait();
     if (m_tile >= *p.grp.num_tiles) return;   // uniform over the CTA and over its split-K cluster
@@ -113,7 +116,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
       };
       auto load_a = [&](int i) {
         if (gather) return;   // assembled by warps 2..5 below
-        tma_load_2d(stage_a(i % STAGES), &tmap_a, &full_bar[i % STAGES], (kb0 + i) * GEMM_BLOCK_K, row0);
+        tma_load_2d(stage_a(i % STAGES), &tmap_a, &full_bar[i % STAGES], a_col0 + (kb0 + i) * GEMM_BLOCK_K, row0);
       };
       // Weights are never written by an earlier kernel of the stream: fill the pipeline with them
       // before waiting for the producer of the activations.
@@ -534,6 +537,9 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const
             if (p.act_pair == 1) {
 #pragma unroll
               for (int q = 0; q < 8; ++q) v[q] = silu(v[q]) * u[q];
+            } else if (p.act_pair == 3) {
+#pragma unroll
+              for (int q = 0; q < 8; ++q) v[q] = fmaxf(v[q], 0.f) * u[q];
             } else {
 #pragma unroll
               for (int q = 0; q < 8; ++q) {
@@ -545,9 +551,19 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const
           }
           const int col = col0 + oc * 8;
           if (col >= n_out) continue;
-          if (p.residual) {
+          if (p.residual && p.res_fp32) {
+            const float* r = static_cast<const float*>(p.residual) + size_t(m) * p.ldr + col;
+            if (col + 8 <= n_out && (reinterpret_cast<uintptr_t>(r) & 15) == 0) {
+              const float4 x = *reinterpret_cast<const float4*>(r), y = *reinterpret_cast<const float4*>(r + 4);
+              v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w; v[4] += y.x; v[5] += y.y; v[6] += y.z; v[7] += y.w;
+            } else {
 #pragma unroll
-            for (int q = 0; q < 8; ++q) if (col + q < n_out) v[q] += bf2f(p.residual[size_t(m) * p.ldr + col + q]);
+              for (int q = 0; q < 8; ++q) if (col + q < n_out) v[q] += r[q];
+            }
+          } else if (p.residual) {
+            const __nv_bfloat16* r = static_cast<const __nv_bfloat16*>(p.residual) + size_t(m) * p.ldr + col;
+#pragma unroll
+            for (int q = 0; q < 8; ++q) if (col + q < n_out) v[q] += bf2f(r[q]);
           }
           if (p.out_fp32) {
             float* dst = reinterpret_cast<float*>(p.C) + size_t(m) * p.ldc + col;
@@ -730,7 +746,8 @@ OGB_API long long ogb_comm_capacity(int device) {
 // flags bit 0: fp32 output; bit 1: paired silu(gate)*up epilogue (N = 2 * output columns, rows
 // interleaved in blocks of 64); bit 2: fused all-reduce over the registered symmetric buffers; bit 3: fused
 // reduce-scatter by token rows instead (rank r ends up with rows [r * ceil(M / world), ...) of the sum, written as
-// rows 0.. of C; residual, if given, is that slice too); bit 4: activations gathered from the ranks' pushes.
+// rows 0.. of C; residual, if given, is that slice too); bit 4: activations gathered from the ranks' pushes; bit 5: the residual
+// is fp32; bit 6: the paired activation is max(gate, 0) * up.
 OGB_API int ogb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
                           const void* bias, const void* residual, int ldr, int flags, int splits, int device, int* status,
                           int sm_count, void* stream_) {
@@ -771,8 +788,9 @@ OGB_API int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, 
   GemmParams p = {};
   p.M = M; p.N = N; p.K = K;
   p.splits = splits; p.kb_per_split = kb_per; p.total_kb = total_kb;
-  p.C = C; p.ldc = ldc; p.out_fp32 = out_fp32; p.act_pair = act_pair;
-  p.residual = static_cast<const __nv_bfloat16*>(residual); p.ldr = ldr;
+  p.C = C; p.ldc = ldc; p.out_fp32 = out_fp32; p.act_pair = act_pair ? ((flags >> 6) & 1 ? 3 : 1) : 0;
+  p.residual = residual; p.ldr = ldr; p.res_fp32 = (flags >> 5) & 1;
+  if ((p.res_fp32 || p.act_pair == 3) && fused_ar) return -1;      // the reductions carry bf16 rows
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.status = status;
   p.pdl = pdl_enabled;
@@ -828,6 +846,39 @@ OGB_API int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, 
   if (persistent && !extras && auto_split && bt == 256 && splits == 1 && !p.comm_epilogue && p.ag_rows == 0 && n_tiles * m_tiles >= sm_count)
     return LaunchPersistent(tw, ta, p, n_tiles, m_tiles, sm_count, stream);
   dim3 grid(n_tiles, m_tiles, splits);
+  switch (bt) {
+    case 16: return Launch<16>(tw, ta, p, grid, stream);
+    case 32: return Launch<32>(tw, ta, p, grid, stream);
+    case 64: return Launch<64>(tw, ta, p, grid, stream);
+    case 128: return Launch<128>(tw, ta, p, grid, stream);
+    case 256: return Launch<256>(tw, ta, p, grid, stream);
+  }
+  return -5;
+}
+
+// A batch of `batch` products over the same M rows of A (per-head projections): C[:, z * c_cols + n] = sum_k A[:, z * a_cols + k] *
+// W[z * N + n, k], k < K.  A [M, a_width] bf16 (a_cols a multiple of 8, every column finite), W [batch * N, K] bf16, C bf16.
+OGB_API int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M,
+                                  int N, int K, int batch, int* status, void* stream_) {
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
+  if ((a_cols % 8) || (lda % 8) || (ldw % 8)) return -1;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -1;
+  static const int pdl_enabled = [] { const char* e = getenv("OGB_PDL"); return (e && e[0] == '0') ? 0 : 1; }();
+  const int bt = ogb_gemm_token_tile(M, 0);
+  CUtensorMap tw, ta;
+  if (!MakeMap(&tw, W, batch * N, K, ldw, GEMM_BLOCK_N)) return -2;
+  if (!MakeMap(&ta, A, M, a_width, lda, bt)) return -2;
+  GemmParams p = {};
+  p.M = M; p.N = N; p.K = K;
+  p.total_kb = (K + GEMM_BLOCK_K - 1) / GEMM_BLOCK_K;
+  p.splits = 1; p.kb_per_split = p.total_kb;
+  p.C = C; p.ldc = ldc;
+  p.status = status;
+  p.pdl = pdl_enabled;
+  p.bat.m_tiles = (M + bt - 1) / bt; p.bat.a_cols = a_cols; p.bat.c_cols = c_cols;
+  if ((long long)p.bat.m_tiles * batch > 65535) return -1;
+  dim3 grid((N + GEMM_BLOCK_N - 1) / GEMM_BLOCK_N, p.bat.m_tiles * batch, 1);
   switch (bt) {
     case 16: return Launch<16>(tw, ta, p, grid, stream);
     case 32: return Launch<32>(tw, ta, p, grid, stream);

@@ -382,7 +382,7 @@ gemv_w4_kernel(const __nv_bfloat16* __restrict__ A, int lda, const uint8_t* __re
           if (m >= p.M) break;
           float v = total(m, tid);
           if (pair) v = silu(v) * total(m, tid + 64);
-          if (p.residual) v += bf2f(p.residual[size_t(m) * p.ldr + col]);
+          if (p.residual) v += bf2f(static_cast<const __nv_bfloat16*>(p.residual)[size_t(m) * p.ldr + col]);
           if (p.out_fp32) reinterpret_cast<float*>(p.C)[size_t(m) * p.ldc + col] = v;
           else reinterpret_cast<__nv_bfloat16*>(p.C)[size_t(m) * p.ldc + col] = f2bf(v);
         }

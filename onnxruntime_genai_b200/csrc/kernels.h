@@ -27,7 +27,8 @@ int ogb_comm_has_nvls(int device);
 int ogb_comm_set_options(int use_nvls, long long two_shot_bytes, int p2p_two_hop);   // negative (-2 for the last): leave unchanged
 long long ogb_comm_capacity(int device);
 // flags: bit 0 fp32 output, bit 1 paired silu(gate)*up epilogue, bit 2 fused tensor-parallel all-reduce,
-// bit 3 fused reduce-scatter by token rows (sequence-parallel form)
+// bit 3 fused reduce-scatter by token rows (sequence-parallel form), bit 5 the residual is fp32, bit 6 the paired activation is
+// max(gate, 0) * up
 int ogb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, const void* bias,
                   const void* residual, int ldr, int flags, int splits, int device, int* status, int sm_count, void* stream);
 
@@ -45,6 +46,48 @@ typedef struct OgbGemmFused {
 int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, const void* bias,
                         const void* residual, int ldr, int flags, int splits, int device, int* status, int sm_count, void* stream,
                         const OgbGemmFused* fused);
+
+// Per-head products over the same rows of A: C[:, z * c_cols + n] = sum_k A[:, z * a_cols + k] * W[z * N + n, k]
+int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N,
+                          int K, int batch, int* status, void* stream);
+
+// ---- gemm_simt.cu: fp32 products and bf16 products TMA cannot address
+int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K, int batch,
+                  const float* residual, int ldr, int in_fp32, int out_fp32, void* stream);
+
+// ---- layer_ops.cu: fp32 residual stream
+int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, int T, int H, int vocab, float scale, void* stream);
+int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const float* b, void* out, int out_fp32, int n_rows, int H, float eps,
+                    int layernorm, void* stream);
+int ogb_act_mul_rows(const void* x, int ldx, void* out, int ldo, int T, int I, int act, int fp32, void* stream);
+int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const void* bias, void* cache, int ldcache, const int32_t* slots,
+                         const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols,
+                         int block_size, void* out, int T, int B, int C, int L, int silu, int fp32, void* stream);
+
+// ---- attention_tc.cu, latent form (long prompts over expanded keys and values)
+int ogb_attention_tc_latent_supported(int dim, int rot, int vdim);
+int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldkv, const void* kr, int ldkr, int kr_col, int rows,
+                            const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* row_base, const int32_t* first_kv, void* out,
+                            int out_stride, float scale, int window, int B, int max_q_len, int H, int dim, int rot, int vdim, int* status,
+                            void* stream);
+
+// ---- latent_attention.cu: attention over a paged cache of latent rows [c (R) | rotated key (rot)]
+typedef struct OgbLatentShape { int H, dim, rot, vdim, R, rot_dims; } OgbLatentShape;
+int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const float* norm_w, float eps, const int32_t* positions, const float* cos,
+                    const float* sin, int max_pos, const int32_t* slots, void* cache, int ldcache, int T, int fp32, void* stream);
+int ogb_latent_mma_supported(const OgbLatentShape* sh);
+int ogb_latent_rows_per_tile(int H, int max_q_len);
+long long ogb_latent_scratch_bytes(int total_rows, int R, int splits);
+int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
+                         const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
+                         void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
+                         long long scratch_bytes, void* stream);
+int ogb_latent_attention_simt(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
+                              const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
+                              void* out, float scale, int window, int B, int T, int skip_q_len, int fp32, void* stream);
+int ogb_latent_gather(const void* cache, int ldcache, const int32_t* block_table, int table_cols, int block_size, const int32_t* row_base,
+                      const int32_t* first_kv, const int32_t* kv_len, const int32_t* req, int n_req, int rows, int width, void* out, int ldo,
+                      void* stream);
 
 // Grouped expert GEMM over token rows sorted by expert (tile list from ogb_moe_sort); act_kind 1 = silu(gate)*up,
 // 2 = clamped SwiGLU(alpha, limit); flags as above (bit 2 unused).
@@ -97,7 +140,7 @@ int ogb_act_mul(const void* x, void* out, int T, int I, int act, void* stream);
 int ogb_act(const void* x, void* out, long long n, int act, void* stream);
 int ogb_causal_conv(const void* x, int x_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                     const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
-                    int table_cols, int block_size, void* out, int T, int B, int C, int L, int silu, void* stream);
+                    int table_cols, int block_size, void* out, int T, int B, int C, int L, int cache_stride, int silu, void* stream);
 int ogb_short_conv(const void* bcx, int bcx_stride, const void* weight, const void* bias, void* cache, const int32_t* slots,
                    const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table,
                    int table_cols, int block_size, void* out, int T, int B, int C, int L, void* stream);
@@ -112,12 +155,13 @@ int ogb_gather_rows_f16(const void* in, const int32_t* rows, void* out, int n_ro
 
 // ---- linear_attention.cu: gated delta rule over packed sequences; state [slots, Hv, dk, dv] fp32 updated in place
 int ogb_gated_delta_fused(const void* conv, long long conv_stride, long long q_off, long long k_off, long long v_off, const void* ba,
-                          long long ba_stride, long long b_off, long long a_off, const float* neg_exp_a, const float* dt_bias, float q_scale,
-                          float* state, const int32_t* slots, const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk,
-                          int Hv, int dk, int dv, void* stream);
-int ogb_gdn_gate_norm(const void* o, const void* z, long long z_stride, const float* w, float eps, void* out, int T, int Hv, int dv, void* stream);
+                          long long ba_stride, long long b_off, long long a_off, const float* neg_exp_a, const float* dt_bias,
+                          float q_scale, float l2_eps, float* state, long long slot_stride, const int32_t* slots, const int32_t* cu_seqlens,
+                          const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, int max_q_len, int fp32, void* stream);
+int ogb_gdn_gate_norm(const void* o, const void* z, long long z_stride, const float* w, float eps, void* out, long long out_stride, int T, int Hv,
+                      int dv, int fp32, void* stream);
 int ogb_gated_delta(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state, const int32_t* slots,
-                    const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, void* stream);
+                    const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, int max_q_len, void* stream);
 int ogb_mamba2_scan_fused(const void* conv, long long conv_stride, const void* dt_raw, long long dt_stride, const float* dt_bias, const float* neg_a,
                           const float* Dv, float* state, const int32_t* slots, const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B,
                           int heads, int groups, int P, int N, void* stream);

@@ -1,0 +1,539 @@
+// Latent attention over a paged cache.  A token's cache row is its normalised latent c (R values) followed by one rotated key part
+// (rot values) that all heads share; per-head keys and values are linear maps of c.  With the key map folded into the query
+// (qlat[t, h] = W_uk[h]^T q[t, h], made by a per-head product beforehand) a head's score against cached position j is
+//     (qlat[t, h] . c_j + q_rot[t, h] . k_rot_j) * scale
+// and its result before the value map is sum_j p_j c_j: every head of a token reads the same rows, once, for scores and values.
+// Kernels:
+//   latent_prep_kernel   RMS norm of the latent and rotation of the key part into the cache; rotation of the queries' rotary parts.
+//   latent_mma_kernel    decode steps and short portions: one CTA = (request, up to 64 (token, head) rows, key split); tiles of 64
+//                        cache rows through cp.async double buffering serve as K (all columns) and as V (the first R columns) of
+//                        warp-level MMAs.  Like paged_attention_kernel (attention.cu) it is bound by the cache stream and its rows are
+//                        few; long prompts take the tensor-memory kernel (attention_tc.cu) on expanded keys and values instead.
+//   latent_simt_kernel   the same op in plain fp32 arithmetic for fp32 models and for sizes the other kernels cannot address.
+//   latent_gather_kernel cached rows of some requests into a dense matrix (input of the key / value expansion of long prompts).
+// A query at position p sees keys (p - window, p] (window > 0) or [0, p].  Built without fast-math.
+#include <cstdlib>
+#include "common.cuh"
+#include "kernels.h"
+
+namespace ogb {
+
+constexpr float LAT_LOG2E = 1.4426950408889634f;
+
+template <typename T> __device__ __forceinline__ float lat_f32(T v);
+template <> __device__ __forceinline__ float lat_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float lat_f32<__nv_bfloat16>(__nv_bfloat16 v) { return bf2f(v); }
+template <typename T> __device__ __forceinline__ T lat_from(float v);
+template <> __device__ __forceinline__ float lat_from<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 lat_from<__nv_bfloat16>(float v) { return f2bf(v); }
+
+// ------------------------------------------------------------------------------------ norm + rotation + append
+// proj row t: [H heads of (dim | rot)] queries, R latent values, rot shared key values.  One CTA per token.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ proj, int ldp, OgbLatentShape sh, const float* __restrict__ norm_w, float eps,
+                                                          const int32_t* __restrict__ positions, const float* __restrict__ cosc,
+                                                          const float* __restrict__ sinc, int max_pos, const int32_t* __restrict__ slots,
+                                                          T* __restrict__ cache, int ldcache) {
+  __shared__ float part[4];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  T* row = proj + size_t(t) * ldp;
+  const T* down = row + sh.H * (sh.dim + sh.rot);
+  const int pos = min(max(positions[t], 0), max_pos - 1), slot = slots[t];
+  const int half = sh.rot_dims / 2;
+  const float *cs = cosc + size_t(pos) * half, *sn = sinc + size_t(pos) * half;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < sh.R; i += 128) { const float v = lat_f32(down[i]); ss += v * v; }
+  ss = warp_sum(ss);
+  if (lane == 0) part[warp] = ss;
+  __syncthreads();
+  if (slot >= 0) {
+    const float inv = 1.f / sqrtf((part[0] + part[1] + part[2] + part[3]) / sh.R + eps);
+    T* dst = cache + size_t(slot) * ldcache;
+    for (int i = threadIdx.x; i < sh.R; i += 128) dst[i] = lat_from<T>(lat_f32(down[i]) * inv * norm_w[i]);
+    for (int i = threadIdx.x; i < sh.rot; i += 128) {
+      float v = lat_f32(down[sh.R + i]);
+      if (i < half) v = v * cs[i] - lat_f32(down[sh.R + i + half]) * sn[i];
+      else if (i < 2 * half) v = v * cs[i - half] + lat_f32(down[sh.R + i - half]) * sn[i - half];
+      dst[sh.R + i] = lat_from<T>(v);
+    }
+  }
+  for (int idx = threadIdx.x; idx < sh.H * half; idx += 128) {
+    const int h = idx / half, i = idx - h * half;
+    T* q = row + h * (sh.dim + sh.rot) + sh.dim;
+    const float u = lat_f32(q[i]), v = lat_f32(q[i + half]);
+    q[i] = lat_from<T>(u * cs[i] - v * sn[i]);
+    q[i + half] = lat_from<T>(v * cs[i] + u * sn[i]);
+  }
+}
+
+// ------------------------------------------------------------------------------------ warp-MMA kernel
+struct LatentParams {
+  const __nv_bfloat16* qlat;      // [T, H, R]
+  const __nv_bfloat16* proj;      // rotary query parts at row t, column h * (dim + rot) + dim
+  int ldp, dim;
+  const __nv_bfloat16* cache; int ldcache;
+  const int32_t *cu, *past, *table; int table_cols, block_size;
+  __nv_bfloat16* out;             // [T, H, R]
+  float* part_o; float* part_ml;
+  float scale;
+  int window, B, H, R, rot, kp, pitch, splits, total_rows, skip_q_len;
+};
+
+constexpr int LAT_BN = 64, LAT_THREADS = 256, LAT_PP = LAT_BN + 8;   // keys per tile; pitch of a P row
+
+template <int MT>
+__host__ __device__ constexpr int lat_smem_bytes(int pitch) {
+  return MT * 16 * pitch * 2 + 2 * LAT_BN * pitch * 2 + MT * 16 * LAT_PP * 2 + 8 * MT * 16 * 4 + 64;
+}
+
+template <int MT, int NTW>
+__global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p) {
+  constexpr int BM = MT * 16, KG = 8 / MT;             // rows; key groups (warps of one row block)
+  extern __shared__ __align__(128) uint8_t smem[];
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* sK = sQ + BM * p.pitch;               // [2][64][pitch]
+  __nv_bfloat16* sP = sK + 2 * LAT_BN * p.pitch;       // [BM][LAT_PP]
+  float* wred = reinterpret_cast<float*>(sP + BM * LAT_PP);   // [KG][BM] row maxima / sums of the key groups
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int mt = warp % MT, kg = warp / MT;
+  const int b = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+  const int H = p.H, tok0 = p.cu[b], q_len = p.cu[b + 1] - tok0, rows = q_len * H;
+  const int row0 = blockIdx.x * BM;
+  if (row0 >= rows || (p.skip_q_len > 0 && q_len >= p.skip_q_len)) return;
+  const int past = p.past[b];
+  const int32_t* table = p.table + size_t(b) * p.table_cols;
+  // this tile's keys, then the part of them this split owns
+  const int kv_hi = past + min(q_len - 1, (row0 + BM - 1) / H) + 1;
+  const int kv_lo = p.window > 0 ? max(0, past + row0 / H - p.window + 1) : 0;
+  const int per = ((kv_hi - kv_lo + LAT_BN - 1) / LAT_BN + p.splits - 1) / p.splits * LAT_BN;
+  const int lo = kv_lo + split * per, hi = min(kv_hi, lo + per);
+  if (p.splits > 1 && lo >= hi) {
+    for (int r = tid; r < BM; r += LAT_THREADS)
+      if (row0 + r < rows) {
+        float* pm = p.part_ml + (size_t(split) * p.total_rows + size_t(tok0) * H + row0 + r) * 2;
+        pm[0] = -INFINITY; pm[1] = 0.f;
+      }
+    return;
+  }
+  const int n_tiles = (hi - lo + LAT_BN - 1) / LAT_BN;
+  const int kc = (p.R + p.rot) / 8, rc = p.R / 8;      // 16-byte chunks of a cache row; of its latent
+  auto load = [&](int it) {                            // a warp copies 8 rows of the tile; rows past the range become zeros
+    const int j = lo + it * LAT_BN + warp * 8 + (lane & 7);
+    int slot = -1;
+    if (j < hi) slot = table[j / p.block_size] * p.block_size + j % p.block_size;
+    __nv_bfloat16* dst = sK + ((it & 1) * LAT_BN + warp * 8) * p.pitch;
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int sl = __shfl_sync(0xffffffffu, slot, r);
+      const __nv_bfloat16* src = p.cache + (sl >= 0 ? size_t(sl) * p.ldcache : 0);
+      for (int c = lane; c < kc; c += 32) cp_async16(dst + r * p.pitch + c * 8, src + c * 8, sl >= 0);
+    }
+  };
+  // queries: latent part from qlat, rotary part from the projection
+  for (int idx = tid; idx < BM * kc; idx += LAT_THREADS) {
+    const int r = idx / kc, c = idx - r * kc, gr = row0 + r;
+    const bool ok = gr < rows;
+    const __nv_bfloat16* src = p.qlat;
+    if (ok) {
+      const size_t tr = size_t(tok0) * H + gr;
+      src = c < rc ? p.qlat + tr * p.R + c * 8 : p.proj + (tr / H) * p.ldp + size_t(gr % H) * (p.dim + p.rot) + p.dim + (c - rc) * 8;
+    }
+    cp_async16(sQ + r * p.pitch + c * 8, src, ok);
+  }
+  if (kc * 8 < p.kp) {                                 // columns between the row's end and the next multiple of 16 are zeros
+    for (int r = tid; r < BM; r += LAT_THREADS) *reinterpret_cast<uint4*>(sQ + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
+    for (int r = tid; r < 2 * LAT_BN; r += LAT_THREADS) *reinterpret_cast<uint4*>(sK + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
+  }
+  if (n_tiles > 0) load(0);
+  cp_async_commit();
+
+  const int r_lo = mt * 16 + g, r_hi = r_lo + 8;       // score rows of this thread
+  const bool v_lo = row0 + r_lo < rows, v_hi = row0 + r_hi < rows;
+  const int q_lo = past + (row0 + r_lo) / H, q_hi = past + (row0 + r_hi) / H;
+  const float sc2 = p.scale * LAT_LOG2E;
+  const int ksteps = p.kp / 16, c0 = warp * NTW * 8;   // output columns [c0, c0 + 8 * NTW) of every row
+  float o[MT][NTW][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NTW; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
+  float mx[MT][2], l_lo = 0.f, l_hi = 0.f;             // running maxima of rows (16 m + g, + 8); sums over this thread's own keys
+#pragma unroll
+  for (int m = 0; m < MT; ++m) mx[m][0] = mx[m][1] = -INFINITY;
+
+  for (int it = 0; it < n_tiles; ++it) {
+    cp_async_wait<0>();
+    __syncthreads();                                   // tile it has landed; every warp is done with tile it - 1
+    if (it + 1 < n_tiles) load(it + 1);
+    cp_async_commit();
+    const __nv_bfloat16* tk = sK + (it & 1) * LAT_BN * p.pitch;
+    // ---- scores of 16 rows x 8 * MT keys
+    float s[MT][4];
+#pragma unroll
+    for (int n = 0; n < MT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+    const __nv_bfloat16* qa = sQ + (mt * 16 + (lane & 15)) * p.pitch + (lane >> 4) * 8;
+    if constexpr (MT == 1) {
+      float s2[4] = {0.f, 0.f, 0.f, 0.f};
+      const __nv_bfloat16* ka = tk + (kg * 8 + (lane & 7)) * p.pitch + (lane >> 3) * 8;
+#pragma unroll 2
+      for (int ks = 0; ks < ksteps; ks += 2) {
+        uint32_t qf[4], kb[4];
+        ldmatrix_x4(kb, ka + ks * 16);
+        ldmatrix_x4(qf, qa + ks * 16);
+        mma_bf16_16816(s[0], qf, kb[0], kb[1]);
+        if (ks + 1 < ksteps) {
+          ldmatrix_x4(qf, qa + ks * 16 + 16);
+          mma_bf16_16816(s2, qf, kb[2], kb[3]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[0][e] += s2[e];
+    } else {
+      const __nv_bfloat16* ka = tk + (kg * 8 * MT + (lane >> 4) * 8 + (lane & 7)) * p.pitch + ((lane >> 3) & 1) * 8;
+#pragma unroll 2
+      for (int ks = 0; ks < ksteps; ++ks) {
+        uint32_t qf[4];
+        ldmatrix_x4(qf, qa + ks * 16);
+#pragma unroll
+        for (int np = 0; np < MT / 2; ++np) {
+          uint32_t kb[4];
+          ldmatrix_x4(kb, ka + np * 16 * p.pitch + ks * 16);
+          mma_bf16_16816(s[np * 2], qf, kb[0], kb[1]);
+          mma_bf16_16816(s[np * 2 + 1], qf, kb[2], kb[3]);
+        }
+      }
+    }
+    const int jb = lo + it * LAT_BN + kg * 8 * MT + t4 * 2;
+    float mlo = -INFINITY, mhi = -INFINITY;
+#pragma unroll
+    for (int n = 0; n < MT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = jb + n * 8 + (e & 1), qp = e >= 2 ? q_hi : q_lo;
+        const bool ok = (e >= 2 ? v_hi : v_lo) && j < hi && j <= qp && (p.window <= 0 || j > qp - p.window);
+        s[n][e] = ok ? s[n][e] * sc2 : -INFINITY;
+        if (e >= 2) mhi = fmaxf(mhi, s[n][e]); else mlo = fmaxf(mlo, s[n][e]);
+      }
+    mlo = fmaxf(mlo, __shfl_xor_sync(0xffffffffu, mlo, 1)); mlo = fmaxf(mlo, __shfl_xor_sync(0xffffffffu, mlo, 2));
+    mhi = fmaxf(mhi, __shfl_xor_sync(0xffffffffu, mhi, 1)); mhi = fmaxf(mhi, __shfl_xor_sync(0xffffffffu, mhi, 2));
+    if (t4 == 0) { wred[kg * BM + r_lo] = mlo; wred[kg * BM + r_hi] = mhi; }
+    __syncthreads();
+    // ---- new maxima of all rows (every warp holds output columns of all of them), P of the own rows
+    float al[MT][2];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float n = mx[m][e];
+#pragma unroll
+        for (int k = 0; k < KG; ++k) n = fmaxf(n, wred[k * BM + m * 16 + g + e * 8]);
+        al[m][e] = n == -INFINITY ? 1.f : exp2f(mx[m][e] - n);
+        mx[m][e] = n;
+      }
+    float a_lo = 0.f, a_hi = 0.f, n_lo = 0.f, n_hi = 0.f;
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+      if (m == mt) { a_lo = al[m][0]; a_hi = al[m][1]; n_lo = mx[m][0] == -INFINITY ? 0.f : mx[m][0]; n_hi = mx[m][1] == -INFINITY ? 0.f : mx[m][1]; }
+    l_lo *= a_lo; l_hi *= a_hi;
+#pragma unroll
+    for (int n = 0; n < MT; ++n) {
+      const float p0 = exp2f(s[n][0] - n_lo), p1 = exp2f(s[n][1] - n_lo), p2 = exp2f(s[n][2] - n_hi), p3 = exp2f(s[n][3] - n_hi);
+      l_lo += p0 + p1; l_hi += p2 + p3;
+      const int kcol = kg * 8 * MT + n * 8 + t4 * 2;
+      *reinterpret_cast<uint32_t*>(sP + r_lo * LAT_PP + kcol) = pack_bf16x2(p0, p1);
+      *reinterpret_cast<uint32_t*>(sP + r_hi * LAT_PP + kcol) = pack_bf16x2(p2, p3);
+    }
+    __syncthreads();
+    // ---- O = O * alpha + P C
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < NTW; ++n) { o[m][n][0] *= al[m][0]; o[m][n][1] *= al[m][0]; o[m][n][2] *= al[m][1]; o[m][n][3] *= al[m][1]; }
+#pragma unroll
+    for (int kk = 0; kk < LAT_BN / 16; ++kk) {
+      uint32_t pa[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) ldmatrix_x4(pa[m], sP + (m * 16 + (lane & 15)) * LAT_PP + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int np = 0; np < NTW / 2; ++np) {
+        if (c0 + np * 16 >= p.R) break;
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, tk + (kk * 16 + (lane & 15)) * p.pitch + c0 + np * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16_16816(o[m][np * 2], pa[m], vb[0], vb[1]);
+          mma_bf16_16816(o[m][np * 2 + 1], pa[m], vb[2], vb[3]);
+        }
+      }
+    }
+  }
+  cp_async_wait<0>();
+  // row sums: the quad's threads, then the key groups
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  __syncthreads();
+  if (t4 == 0) { wred[kg * BM + r_lo] = l_lo; wred[kg * BM + r_hi] = l_hi; }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = m * 16 + g + e * 8;
+      if (row0 + r >= rows) continue;
+      float l = 0.f;
+#pragma unroll
+      for (int k = 0; k < KG; ++k) l += wred[k * BM + r];
+      const size_t orow = size_t(tok0) * H + row0 + r;
+      if (p.splits > 1) {
+        float* po = p.part_o + (size_t(split) * p.total_rows + orow) * p.R;
+#pragma unroll
+        for (int n = 0; n < NTW; ++n)
+          if (c0 + n * 8 < p.R) *reinterpret_cast<float2*>(po + c0 + n * 8 + t4 * 2) = make_float2(o[m][n][e * 2], o[m][n][e * 2 + 1]);
+        if (warp == 0 && t4 == 0) {
+          float* pm = p.part_ml + (size_t(split) * p.total_rows + orow) * 2;
+          pm[0] = mx[m][e]; pm[1] = l;
+        }
+      } else {
+        const float inv = l > 0.f ? 1.f / l : 0.f;
+        __nv_bfloat16* po = p.out + orow * p.R;
+#pragma unroll
+        for (int n = 0; n < NTW; ++n)
+          if (c0 + n * 8 < p.R) *reinterpret_cast<uint32_t*>(po + c0 + n * 8 + t4 * 2) = pack_bf16x2(o[m][n][e * 2] * inv, o[m][n][e * 2 + 1] * inv);
+      }
+    }
+}
+
+// One CTA per (token, head) row: merges the split partials.
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                             __nv_bfloat16* __restrict__ out, int total_rows, int R, int splits) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x;
+  float M = -INFINITY;
+  for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[(size_t(s) * total_rows + row) * 2]);
+  float L = 0.f;
+  for (int s = 0; s < splits; ++s) {
+    const float* ml = part_ml + (size_t(s) * total_rows + row) * 2;
+    if (ml[0] != -INFINITY) L += exp2f(ml[0] - M) * ml[1];
+  }
+  const float inv = L > 0.f ? 1.f / L : 0.f;
+  for (int c = threadIdx.x * 4; c < R; c += 512) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < splits; ++s) {
+      const float m = part_ml[(size_t(s) * total_rows + row) * 2];
+      if (m == -INFINITY) continue;
+      const float w = exp2f(m - M);
+      const float4 v = *reinterpret_cast<const float4*>(part_o + (size_t(s) * total_rows + row) * R + c);
+      a.x += w * v.x; a.y += w * v.y; a.z += w * v.z; a.w += w * v.w;
+    }
+    *reinterpret_cast<uint2*>(out + size_t(row) * R + c) = make_uint2(pack_bf16x2(a.x * inv, a.y * inv), pack_bf16x2(a.z * inv, a.w * inv));
+  }
+}
+
+// ------------------------------------------------------------------------------------ plain kernel
+constexpr int LAT_SIMT_COLS = 16;                      // latent columns per thread (R <= 2048)
+template <typename T>
+__global__ void __launch_bounds__(128) latent_simt_kernel(const T* __restrict__ qlat, const T* __restrict__ proj, int ldp, OgbLatentShape sh,
+                                                          const T* __restrict__ cache, int ldcache, const int32_t* __restrict__ cu,
+                                                          const int32_t* __restrict__ past_lens, const int32_t* __restrict__ tables, int table_cols,
+                                                          int block_size, T* __restrict__ out, float scale, int window, int B, int skip_q_len) {
+  extern __shared__ float sq[];                        // [R + rot] query, then 32 scores
+  float* ssc = sq + sh.R + sh.rot;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  int rlo = 0, rhi = B - 1;
+  while (rlo < rhi) {
+    const int mid = (rlo + rhi + 1) >> 1;
+    if (cu[mid] <= t) rlo = mid; else rhi = mid - 1;
+  }
+  const int b = rlo, q_len = cu[b + 1] - cu[b];
+  if (t >= cu[b + 1] || (skip_q_len > 0 && q_len >= skip_q_len)) return;
+  const int pos = past_lens[b] + t - cu[b], n = sh.R + sh.rot;
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int32_t* table = tables + size_t(b) * table_cols;
+  for (int i = threadIdx.x; i < n; i += 128)
+    sq[i] = lat_f32(i < sh.R ? qlat[(size_t(t) * sh.H + h) * sh.R + i] : proj[size_t(t) * ldp + size_t(h) * (sh.dim + sh.rot) + sh.dim + i - sh.R]);
+  float acc[LAT_SIMT_COLS];
+#pragma unroll
+  for (int c = 0; c < LAT_SIMT_COLS; ++c) acc[c] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  auto row_of = [&](int j) { return cache + (size_t(table[j / block_size]) * block_size + j % block_size) * ldcache; };
+  for (int j0 = lo; j0 <= pos; j0 += 32) {
+    __syncthreads();
+    for (int k = warp; k < 32; k += 4) {
+      const int j = j0 + k;
+      float d = 0.f;
+      if (j <= pos) {
+        const T* row = row_of(j);
+        for (int i = lane; i < n; i += 32) d = fmaf(sq[i], lat_f32(row[i]), d);
+      }
+      d = warp_sum(d);
+      if (lane == 0) ssc[k] = j <= pos ? d * scale : -INFINITY;
+    }
+    __syncthreads();
+    float mn = m;
+    for (int k = 0; k < 32; ++k) mn = fmaxf(mn, ssc[k]);
+    const float al = expf(m - mn);                     // m = -inf at first: 0
+    l *= al;
+#pragma unroll
+    for (int c = 0; c < LAT_SIMT_COLS; ++c) acc[c] *= al;
+    for (int k = 0; k < 32 && j0 + k <= pos; ++k) {
+      const float pr = expf(ssc[k] - mn);
+      l += pr;
+      const T* row = row_of(j0 + k);
+#pragma unroll
+      for (int c = 0; c < LAT_SIMT_COLS; ++c) {
+        const int i = c * 128 + threadIdx.x;
+        if (i < sh.R) acc[c] = fmaf(pr, lat_f32(row[i]), acc[c]);
+      }
+    }
+    m = mn;
+  }
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int c = 0; c < LAT_SIMT_COLS; ++c) {
+    const int i = c * 128 + threadIdx.x;
+    if (i < sh.R) out[(size_t(t) * sh.H + h) * sh.R + i] = lat_from<T>(acc[c] * inv);
+  }
+}
+
+// ------------------------------------------------------------------------------------ gather
+// Dense row i holds cached position first_kv[k] + i - row_base[k] of request req[k], k the last with row_base[k] <= i; rows past
+// kv_len[k] are zeros (a request's rows are padded to a multiple of 16).
+__global__ void latent_gather_kernel(const uint4* __restrict__ cache, int ldvec, const int32_t* __restrict__ tables, int table_cols, int block_size,
+                                     const int32_t* __restrict__ row_base, const int32_t* __restrict__ first_kv, const int32_t* __restrict__ kv_len,
+                                     const int32_t* __restrict__ req, int n_req, int rows, int nvec, uint4* __restrict__ out, int ldo) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (i >= rows) return;
+  int lo = 0, hi = n_req - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (row_base[mid] <= i) lo = mid; else hi = mid - 1;
+  }
+  const int j = first_kv[lo] + i - row_base[lo];
+  const bool ok = j < kv_len[lo];
+  const uint4* src = cache;
+  if (ok) src += (size_t(tables[size_t(req[lo]) * table_cols + j / block_size]) * block_size + j % block_size) * ldvec;
+  for (int c = lane; c < nvec; c += 32) out[size_t(i) * ldo + c] = ok ? src[c] : make_uint4(0, 0, 0, 0);
+}
+
+template <int MT, int NTW>
+static int LaunchLatentMma(const LatentParams& p, int max_q_len, cudaStream_t s) {
+  auto kern = latent_mma_kernel<MT, NTW>;
+  static bool configured[OGB_MAX_DEVICES] = {};
+  if (!set_max_dyn_smem(kern, 227 * 1024, configured)) return -3;
+  const dim3 grid((max_q_len * p.H + MT * 16 - 1) / (MT * 16), 1, p.B * p.splits);
+  if (!launch_pdl(kern, grid, dim3(LAT_THREADS), lat_smem_bytes<MT>(p.pitch), s, p)) return -4;
+  if (p.splits > 1 && !launch_pdl(latent_combine_kernel, dim3(p.total_rows), dim3(128), 0, s, static_cast<const float*>(p.part_o),
+                                  static_cast<const float*>(p.part_ml), p.out, p.total_rows, p.R, p.splits))
+    return -4;
+  return 0;
+}
+template <int MT>
+static int LaunchLatentMt(const LatentParams& p, int max_q_len, cudaStream_t s) {
+  if (p.R <= 128) return LaunchLatentMma<MT, 2>(p, max_q_len, s);
+  if (p.R <= 256) return LaunchLatentMma<MT, 4>(p, max_q_len, s);
+  return LaunchLatentMma<MT, 8>(p, max_q_len, s);
+}
+
+static int lat_pitch(const OgbLatentShape* sh) { return (sh->R + sh->rot + 15) / 16 * 16 + 8; }     // an odd number of 16-byte chunks
+
+}  // namespace ogb
+
+using namespace ogb;
+
+OGB_API int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const float* norm_w, float eps, const int32_t* positions, const float* cos,
+                            const float* sin, int max_pos, const int32_t* slots, void* cache, int ldcache, int T, int fp32, void* stream) {
+  if (T <= 0) return 0;
+  if (sh->rot_dims < 0 || sh->rot_dims > sh->rot || (sh->rot_dims & 1) || (sh->rot_dims > 0 && (!cos || !sin || max_pos <= 0))) return -1;
+  if (sh->R + sh->rot > ldcache) return -1;
+  auto s = static_cast<cudaStream_t>(stream);
+  using Hf = __nv_bfloat16;
+  return (fp32 ? launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), 0, s, static_cast<float*>(proj), ldp, *sh, norm_w, eps, positions, cos, sin,
+                            max_pos, slots, static_cast<float*>(cache), ldcache)
+               : launch_pdl(latent_prep_kernel<Hf>, dim3(T), dim3(128), 0, s, static_cast<Hf*>(proj), ldp, *sh, norm_w, eps, positions, cos, sin, max_pos,
+                            slots, static_cast<Hf*>(cache), ldcache)) ? 0 : -4;
+}
+
+// 1 when the warp-MMA kernel can address these sizes (16-byte pieces everywhere, the tile fits in shared memory).
+OGB_API int ogb_latent_mma_supported(const OgbLatentShape* sh) {
+  return sh->R % 8 == 0 && sh->rot % 8 == 0 && sh->dim % 8 == 0 && sh->R >= 8 && sh->R <= 512 && lat_smem_bytes<1>(lat_pitch(sh)) <= 227 * 1024;
+}
+
+// Rows of (token, head) a CTA takes for requests of at most max_q_len tokens.
+OGB_API int ogb_latent_rows_per_tile(int H, int max_q_len) {
+  const int rows = H * max_q_len;
+  return rows <= 16 ? 16 : (rows <= 32 ? 32 : 64);
+}
+
+OGB_API long long ogb_latent_scratch_bytes(int total_rows, int R, int splits) {
+  return splits <= 1 ? 0 : (long long)splits * total_rows * (R + 2) * 4;
+}
+
+// bf16.  skip_q_len > 0: requests with at least that many tokens are left to another kernel (their rows of `out` are unspecified).
+OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
+                                 const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
+                                 void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
+                                 long long scratch_bytes, void* stream) {
+  if (B <= 0 || T <= 0 || max_q_len <= 0) return 0;
+  if (!ogb_latent_mma_supported(sh)) return -5;
+  if ((ldp % 8) || (ldcache % 8) || block_size <= 0) return -1;
+  if ((reinterpret_cast<uintptr_t>(qlat) | reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) return -1;
+  if (splits < 1) splits = 1;
+  const int rows = T * sh->H;
+  if (ogb_latent_scratch_bytes(rows, sh->R, splits) > scratch_bytes || (long long)B * splits > 65535) return -2;
+  LatentParams p;
+  p.qlat = static_cast<const __nv_bfloat16*>(qlat); p.proj = static_cast<const __nv_bfloat16*>(proj); p.ldp = ldp; p.dim = sh->dim;
+  p.cache = static_cast<const __nv_bfloat16*>(cache); p.ldcache = ldcache;
+  p.cu = cu_seqlens; p.past = past_lens; p.table = block_table; p.table_cols = table_cols; p.block_size = block_size;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.part_o = static_cast<float*>(scratch);
+  p.part_ml = p.part_o ? p.part_o + size_t(splits) * rows * sh->R : nullptr;
+  p.scale = scale; p.window = window; p.B = B; p.H = sh->H; p.R = sh->R; p.rot = sh->rot;
+  p.kp = (sh->R + sh->rot + 15) / 16 * 16; p.pitch = lat_pitch(sh);
+  p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len;
+  auto s = static_cast<cudaStream_t>(stream);
+  int bm = ogb_latent_rows_per_tile(sh->H, skip_q_len > 0 && skip_q_len - 1 < max_q_len ? skip_q_len - 1 : max_q_len);
+  if (bm == 64 && lat_smem_bytes<4>(p.pitch) > 227 * 1024) bm = 32;
+  if (bm == 32 && lat_smem_bytes<2>(p.pitch) > 227 * 1024) bm = 16;
+  if (skip_q_len > 0 && max_q_len > skip_q_len - 1) max_q_len = skip_q_len - 1;
+  if (max_q_len <= 0) return 0;
+  if (bm == 16) return LaunchLatentMt<1>(p, max_q_len, s);
+  if (bm == 32) return LaunchLatentMt<2>(p, max_q_len, s);
+  return LaunchLatentMt<4>(p, max_q_len, s);
+}
+
+OGB_API int ogb_latent_attention_simt(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
+                                      const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
+                                      void* out, float scale, int window, int B, int T, int skip_q_len, int fp32, void* stream) {
+  if (B <= 0 || T <= 0) return 0;
+  if (sh->R > 128 * LAT_SIMT_COLS || sh->H > 65535 || block_size <= 0) return -5;
+  const int smem = (sh->R + sh->rot + 32) * 4;
+  if (smem > 48 * 1024) return -5;
+  auto s = static_cast<cudaStream_t>(stream);
+  using Hf = __nv_bfloat16;
+  return (fp32 ? launch_pdl(latent_simt_kernel<float>, dim3(T, sh->H), dim3(128), smem, s, static_cast<const float*>(qlat), static_cast<const float*>(proj),
+                            ldp, *sh, static_cast<const float*>(cache), ldcache, cu_seqlens, past_lens, block_table, table_cols, block_size,
+                            static_cast<float*>(out), scale, window, B, skip_q_len)
+               : launch_pdl(latent_simt_kernel<Hf>, dim3(T, sh->H), dim3(128), smem, s, static_cast<const Hf*>(qlat), static_cast<const Hf*>(proj), ldp, *sh,
+                            static_cast<const Hf*>(cache), ldcache, cu_seqlens, past_lens, block_table, table_cols, block_size, static_cast<Hf*>(out), scale,
+                            window, B, skip_q_len)) ? 0 : -4;
+}
+
+// width, ldcache, ldo in bf16 elements, multiples of 8
+OGB_API int ogb_latent_gather(const void* cache, int ldcache, const int32_t* block_table, int table_cols, int block_size, const int32_t* row_base,
+                              const int32_t* first_kv, const int32_t* kv_len, const int32_t* req, int n_req, int rows, int width, void* out, int ldo,
+                              void* stream) {
+  if (rows <= 0 || n_req <= 0) return 0;
+  if ((width % 8) || (ldcache % 8) || (ldo % 8) || block_size <= 0) return -1;
+  return launch_pdl(latent_gather_kernel, dim3((rows + 7) / 8), dim3(256), 0, static_cast<cudaStream_t>(stream), static_cast<const uint4*>(cache),
+                    ldcache / 8, block_table, table_cols, block_size, row_base, first_kv, kv_len, req, n_req, rows, width / 8, static_cast<uint4*>(out),
+                    ldo / 8) ? 0 : -4;
+}

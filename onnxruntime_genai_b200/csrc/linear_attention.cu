@@ -2,61 +2,98 @@
 // with update_rule "gated_delta" that the reference's builder emits for Qwen3-Next / Qwen3.5 style hybrids
 // (src/python/py/models/builders/base.py:3419-3452, qwen.py:1842-1860; state handling src/models/recurrent_state.h:12-66).
 //
-// One CTA = (request, value head, 32 columns of the head's state S [dk, dv]).  The tile lives in registers: a thread keeps 16 to 64
-// rows of one column (the rows of a column are split over up to 8 threads); CTAs are small so that several share an SM and their
-// load / update / store phases overlap.  The
-// per-token update needs no shared-memory traffic for S: with k_t, q_t broadcast from shared memory,
+// Two kernels over the same state pool (fp32, [slots][value heads][dk][dv] with a slot stride), for bf16 and fp32 activations and any
+// dk / dv (rows and columns past the sizes are zeros):
+//   gated_delta_kernel        decode-shaped steps.  One CTA = (request, value head, 32 columns of the head's state S [dk, dv]); a thread
+//                             keeps 16 to 64 rows of one column, the lanes of a warp are neighbouring columns (the state streams in
+//                             full lines), the row splits of a column meet in shared memory.
+//   gated_delta_chunk_kernel  prompts.  The lanes of a warp are 8 columns x 4 row splits, so that the two dot products of a token are
+//                             finished by two shuffles and the token loop has no barrier; the keys and queries of a chunk of tokens
+//                             are normalised into shared memory by all warps beforehand.
+// Per token, with k_t, q_t of the head:
 //     S[:, j] *= exp(g);   mem = sum_i S[i, j] k[i];   delta = (v[j] - mem) * beta;   S[i, j] += k[i] * delta;   o[j] = sum_i S[i, j] q[i]
 // Tokens of a request are walked in order inside the kernel (a decode step is one token, a prompt chunk many); the state is read
-// from / written to the request's slot of the fp32 pool once per launch.  A request whose past length is 0 starts from zero.
+// from / written to the request's slot once per launch.  A request whose past length is 0 starts from zero.
+// This file is built without fast-math: the recurrence and all that feeds it is plain fp32.
 #include "common.cuh"
 #include "kernels.h"
 
 namespace ogb {
 
+template <typename T> __device__ __forceinline__ float act_f32(T v);
+template <> __device__ __forceinline__ float act_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ float act_f32<__nv_bfloat16>(__nv_bfloat16 v) { return bf2f(v); }
+template <typename T> __device__ __forceinline__ T act_from(float v);
+template <> __device__ __forceinline__ float act_from<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 act_from<__nv_bfloat16>(float v) { return f2bf(v); }
+
+template <typename T>
 struct GdnParams {
-  const __nv_bfloat16 *q, *k, *v;     // rows of token t at q + t * tok_stride (+ head offsets): separate tensors or slices of one projection
+  const T *q, *k, *v;                 // rows of token t at q + t * tok_stride (+ head offsets): separate tensors or slices of one projection
   long long tok_stride_qk, tok_stride_v;
   const float *g, *beta;              // [T, Hv] log-decay and write strength ...
-  const __nv_bfloat16 *b_raw, *a_raw; // ... or (g == null) their raw projections [T, Hv] with a row stride: beta = sigmoid(b),
+  const T *b_raw, *a_raw;             // ... or (g == null) their raw projections [T, Hv] with a row stride: beta = sigmoid(b),
   long long ba_stride;                //     g = neg_exp_a[h] * softplus(a + dt_bias[h])
   const float *neg_exp_a, *dt_bias;
   int l2norm;                         // q and k are L2-normalised per head here (q then scaled by q_scale)
   float q_scale;
+  float l2_eps;                       // > 0: unit vectors are x / sqrt(sum(x^2) + l2_eps); 0: x / max(sqrt(sum(x^2)), 1e-6)
   float* state;
+  long long slot_stride;              // floats between the states of consecutive slots
   const int32_t *slots, *cu_seqlens, *past_lens;
-  __nv_bfloat16* out;
+  T* out;
   int Hk, Hv, dv, dk;
 };
 
-template <int NPT>
-__global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams p) {
+__device__ __forceinline__ float inv_length(float sumsq, float l2_eps) {
+  return l2_eps > 0.f ? 1.f / sqrtf(sumsq + l2_eps) : 1.f / fmaxf(sqrtf(sumsq), 1e-6f);
+}
+
+// decay exp(g) and write strength beta of token t, value head h
+template <typename T>
+__device__ __forceinline__ void gdn_gates(const GdnParams<T>& p, int t, int h, float& decay, float& beta) {
+  if (p.g) {
+    decay = expf(p.g[size_t(t) * p.Hv + h]);
+    beta = p.beta[size_t(t) * p.Hv + h];
+  } else {
+    const float ar = act_f32(p.a_raw[size_t(t) * p.ba_stride + h]) + p.dt_bias[h];
+    const float soft = ar > 20.f ? ar : log1pf(expf(ar));
+    decay = expf(p.neg_exp_a[h] * soft);
+    beta = 1.f / (1.f + expf(-act_f32(p.b_raw[size_t(t) * p.ba_stride + h])));
+  }
+}
+
+constexpr int GDN_MAX_DK = 1024, GDN_MAX_SPLITS = 16;
+
+template <typename T, int NPT>
+__global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams<T> p) {
   // thread (j, sp): column j of the state, rows [sp * NPT, (sp + 1) * NPT); the two dot products of a token (with k, then with q)
   // are summed over the splits through shared memory
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y;
   const int Hk = p.Hk, Hv = p.Hv, dv = p.dv, dk = p.dk;
-  const int splits = dk / NPT, CT = blockDim.x / splits;      // CT columns per CTA (blockIdx.z walks the column tiles)
-  const int jj = threadIdx.x % CT, j = blockIdx.z * CT + jj, sp = threadIdx.x / CT, n0 = sp * NPT;
+  const int splits = blockDim.x / 32;                         // 32 columns per CTA (blockIdx.z walks the column tiles)
+  const int jj = threadIdx.x % 32, j = blockIdx.z * 32 + jj, sp = threadIdx.x / 32, n0 = sp * NPT;
   const int hk = h / (Hv / Hk);
   const int t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
   if (t0 >= t1) return;
-  __shared__ float sk[256], sq[256];
-  __shared__ float sM[8][128], sO[8][128];
+  __shared__ float sk[GDN_MAX_DK], sq[GDN_MAX_DK];
+  __shared__ float sM[GDN_MAX_SPLITS][32], sO[GDN_MAX_SPLITS][32];
   __shared__ float sNorm[2][16];
-  float* S = p.state + ((size_t(p.slots[b]) * Hv + h) * dk + n0) * dv;
+  float* S = p.state + size_t(p.slots[b]) * p.slot_stride + (size_t(h) * dk + n0) * dv;
   float col[NPT];
   const bool live = j < dv;
   const bool fresh = p.past_lens[b] == 0;
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh) ? S[size_t(i) * dv + j] : 0.f;
+  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh && n0 + i < dk) ? S[size_t(i) * dv + j] : 0.f;
+  for (int i = dk + threadIdx.x; i < splits * NPT; i += blockDim.x) { sk[i] = 0.f; sq[i] = 0.f; }
   for (int t = t0; t < t1; ++t) {
     __syncthreads();
     float ssk = 0.f, ssq = 0.f;
     for (int i = threadIdx.x; i < dk; i += blockDim.x) {
-      const float kv_ = bf2f(p.k[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]);
-      const float qv_ = bf2f(p.q[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]);
+      const float kv_ = act_f32(p.k[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]);
+      const float qv_ = act_f32(p.q[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]);
       sk[i] = kv_; sq[i] = qv_;
       ssk += kv_ * kv_; ssq += qv_ * qv_;
     }
@@ -68,20 +105,12 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams p) {
     __syncthreads();
     if (p.l2norm) {
       float tk = 0.f, tq = 0.f;
-      for (int w = 0; w < int(blockDim.x >> 5); ++w) { tk += sNorm[0][w]; tq += sNorm[1][w]; }
-      rk = 1.f / fmaxf(sqrtf(tk), 1e-6f);
-      rq = p.q_scale / fmaxf(sqrtf(tq), 1e-6f);
+      for (int w = 0; w < splits; ++w) { tk += sNorm[0][w]; tq += sNorm[1][w]; }
+      rk = inv_length(tk, p.l2_eps);
+      rq = p.q_scale * inv_length(tq, p.l2_eps);
     }
     float decay, bt;
-    if (p.g) {
-      decay = __expf(p.g[size_t(t) * Hv + h]);
-      bt = p.beta[size_t(t) * Hv + h];
-    } else {
-      const float ar = bf2f(p.a_raw[size_t(t) * p.ba_stride + h]) + p.dt_bias[h];
-      const float soft = ar > 20.f ? ar : log1pf(__expf(ar));
-      decay = __expf(p.neg_exp_a[h] * soft);
-      bt = 1.f / (1.f + __expf(-bf2f(p.b_raw[size_t(t) * p.ba_stride + h])));
-    }
+    gdn_gates(p, t, h, decay, bt);
     float mem = 0.f;
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
@@ -94,7 +123,7 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams p) {
       mem = 0.f;
       for (int s2 = 0; s2 < splits; ++s2) mem += sM[s2][jj];
     }
-    const float vj = live ? bf2f(p.v[size_t(t) * p.tok_stride_v + size_t(h) * dv + j]) : 0.f;
+    const float vj = live ? act_f32(p.v[size_t(t) * p.tok_stride_v + size_t(h) * dv + j]) : 0.f;
     const float delta = (vj - mem * rk) * bt * rk;       // the normalised key is rk * sk: once in the read, once in the write
     float o = 0.f;
 #pragma unroll
@@ -108,34 +137,136 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams p) {
       if (sp == 0)
         for (int s2 = 1; s2 < splits; ++s2) o += sO[s2][jj];
     }
-    if (live && sp == 0) p.out[(size_t(t) * Hv + h) * dv + j] = f2bf(o * rq);
+    if (live && sp == 0) p.out[(size_t(t) * Hv + h) * dv + j] = act_from<T>(o * rq);
   }
   if (live) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) S[size_t(i) * dv + j] = col[i];
+    for (int i = 0; i < NPT; ++i) if (n0 + i < dk) S[size_t(i) * dv + j] = col[i];
+  }
+}
+
+// NPT rows per thread, 4 * NPT >= dk.  Row of thread split sp, register i: (i / 4) * 16 + sp * 4 + i % 4, so that a thread's rows come
+// as groups of four and the four splits of a warp read neighbouring 16-byte words of a key.  CH tokens per chunk.
+template <typename T, int NPT, int CH>
+__global__ void __launch_bounds__(128) gated_delta_chunk_kernel(GdnParams<T> p) {
+  constexpr int DKP = NPT * 4;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.x, h = blockIdx.y;
+  const int Hv = p.Hv, dv = p.dv, dk = p.dk;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sp = lane & 3;
+  const int jj = warp * 8 + (lane >> 2), j = blockIdx.z * 32 + jj;
+  const int hk = h / (Hv / p.Hk);
+  const int t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
+  if (t0 >= t1) return;
+  __shared__ __align__(16) float sk[CH][DKP];
+  __shared__ __align__(16) float sq[CH][DKP];
+  __shared__ float sv[CH][32], sgate[2][CH];
+  const bool live = j < dv, fresh = p.past_lens[b] == 0;
+  float* S = p.state + size_t(p.slots[b]) * p.slot_stride + size_t(h) * dk * dv;
+  auto row_of = [&](int i) { return (i >> 2) * 16 + sp * 4 + (i & 3); };
+  float col[NPT];
+#pragma unroll
+  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh && row_of(i) < dk) ? S[size_t(row_of(i)) * dv + j] : 0.f;
+
+  // a chunk's raw keys / queries / values on their way from global memory: held in registers while the previous chunk is computed
+  constexpr int PER = DKP / 32, TW = CH / 4;               // elements per lane of a row, rows per warp
+  float rk[TW][PER], rq[TW][PER], rv[TW], ga, gb;
+  auto fetch = [&](int c0) {
+#pragma unroll
+    for (int w = 0; w < TW; ++w) {
+      const int t = c0 + w * 4 + warp;
+#pragma unroll
+      for (int e = 0; e < PER; ++e) {
+        const int i = e * 32 + lane;
+        const bool ok = t < t1 && i < dk;
+        rk[w][e] = ok ? act_f32(p.k[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]) : 0.f;
+        rq[w][e] = ok ? act_f32(p.q[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]) : 0.f;
+      }
+      const int jc = blockIdx.z * 32 + lane;
+      rv[w] = (t < t1 && jc < dv) ? act_f32(p.v[size_t(t) * p.tok_stride_v + size_t(h) * dv + jc]) : 0.f;
+    }
+    ga = gb = 0.f;
+    if (threadIdx.x < CH && c0 + int(threadIdx.x) < t1) gdn_gates(p, c0 + threadIdx.x, h, ga, gb);
+  };
+  fetch(t0);
+  for (int c0 = t0; c0 < t1; c0 += CH) {
+    __syncthreads();                                       // the previous chunk is no longer read
+#pragma unroll
+    for (int w = 0; w < TW; ++w) {
+      float ssk = 0.f, ssq = 0.f;
+#pragma unroll
+      for (int e = 0; e < PER; ++e) { ssk += rk[w][e] * rk[w][e]; ssq += rq[w][e] * rq[w][e]; }
+      float nk = 1.f, nq = 1.f;
+      if (p.l2norm) {
+        nk = inv_length(warp_sum(ssk), p.l2_eps);
+        nq = p.q_scale * inv_length(warp_sum(ssq), p.l2_eps);
+      }
+      const int tt = w * 4 + warp;
+#pragma unroll
+      for (int e = 0; e < PER; ++e) { sk[tt][e * 32 + lane] = rk[w][e] * nk; sq[tt][e * 32 + lane] = rq[w][e] * nq; }
+      sv[tt][lane] = rv[w];
+    }
+    if (threadIdx.x < CH) { sgate[0][threadIdx.x] = ga; sgate[1][threadIdx.x] = gb; }
+    __syncthreads();
+    if (c0 + CH < t1) fetch(c0 + CH);
+    const int n = min(CH, t1 - c0);
+    for (int tt = 0; tt < n; ++tt) {
+      const float decay = sgate[0][tt], bt = sgate[1][tt], vj = sv[tt][jj];
+      const float4* k4 = reinterpret_cast<const float4*>(sk[tt]) + sp;
+      const float4* q4 = reinterpret_cast<const float4*>(sq[tt]) + sp;
+      float m4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < NPT / 4; ++i) {
+        const float4 kk = k4[i * 4];
+        col[4 * i] *= decay; col[4 * i + 1] *= decay; col[4 * i + 2] *= decay; col[4 * i + 3] *= decay;
+        m4[0] = fmaf(col[4 * i], kk.x, m4[0]); m4[1] = fmaf(col[4 * i + 1], kk.y, m4[1]);
+        m4[2] = fmaf(col[4 * i + 2], kk.z, m4[2]); m4[3] = fmaf(col[4 * i + 3], kk.w, m4[3]);
+      }
+      float mem = (m4[0] + m4[1]) + (m4[2] + m4[3]);
+      mem += __shfl_xor_sync(0xffffffffu, mem, 1);
+      mem += __shfl_xor_sync(0xffffffffu, mem, 2);
+      const float delta = (vj - mem) * bt;
+      float o4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < NPT / 4; ++i) {
+        const float4 kk = k4[i * 4], qq = q4[i * 4];
+        col[4 * i] = fmaf(kk.x, delta, col[4 * i]); col[4 * i + 1] = fmaf(kk.y, delta, col[4 * i + 1]);
+        col[4 * i + 2] = fmaf(kk.z, delta, col[4 * i + 2]); col[4 * i + 3] = fmaf(kk.w, delta, col[4 * i + 3]);
+        o4[0] = fmaf(col[4 * i], qq.x, o4[0]); o4[1] = fmaf(col[4 * i + 1], qq.y, o4[1]);
+        o4[2] = fmaf(col[4 * i + 2], qq.z, o4[2]); o4[3] = fmaf(col[4 * i + 3], qq.w, o4[3]);
+      }
+      float o = (o4[0] + o4[1]) + (o4[2] + o4[3]);
+      o += __shfl_xor_sync(0xffffffffu, o, 1);
+      o += __shfl_xor_sync(0xffffffffu, o, 2);
+      if (live && sp == 0) p.out[(size_t(c0 + tt) * Hv + h) * dv + j] = act_from<T>(o);
+    }
+  }
+  if (live) {
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) if (row_of(i) < dk) S[size_t(row_of(i)) * dv + j] = col[i];
   }
 }
 
 // Output gate of a gated-delta-net layer: per value head, RMS norm of the recurrence output times its weight, times silu of the gate
-// projection z (a column slice of the layer's input projection).  One warp per (token, head).
-__global__ void gdn_gate_norm_kernel(const __nv_bfloat16* __restrict__ o, const __nv_bfloat16* __restrict__ z, long long z_stride,
-                                     const float* __restrict__ w, float eps, __nv_bfloat16* __restrict__ out, int rows, int Hv, int dv) {
+// projection z (a column slice of the layer's input projection).  One warp per (token, head); out rows have a stride of their own.
+template <typename T>
+__global__ void gdn_gate_norm_kernel(const T* __restrict__ o, const T* __restrict__ z, long long z_stride, const float* __restrict__ w, float eps,
+                                     T* __restrict__ out, long long out_stride, int rows, int Hv, int dv) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= rows) return;
   const int t = row / Hv, h = row % Hv;
-  const __nv_bfloat16* src = o + size_t(row) * dv;
-  float x[8];
+  const T* src = o + size_t(row) * dv;
   float ss = 0.f;
-  int n = 0;
-  for (int e = lane; e < dv; e += 32, ++n) { x[n] = bf2f(src[e]); ss += x[n] * x[n]; }
+  for (int e = lane; e < dv; e += 32) { const float x = act_f32(src[e]); ss += x * x; }
   ss = warp_sum(ss);
-  const float inv = rsqrtf(ss / dv + eps);
-  n = 0;
-  for (int e = lane; e < dv; e += 32, ++n) {
-    const float zz = bf2f(z[size_t(t) * z_stride + size_t(h) * dv + e]);
-    out[size_t(row) * dv + e] = f2bf(x[n] * inv * w[e] * (zz / (1.f + __expf(-zz))));
+  const float inv = 1.f / sqrtf(ss / dv + eps);
+  T* dst = out + size_t(t) * out_stride + size_t(h) * dv;
+  for (int e = lane; e < dv; e += 32) {
+    const float zz = act_f32(z[size_t(t) * z_stride + size_t(h) * dv + e]);
+    dst[e] = act_from<T>(act_f32(src[e]) * inv * w[e] * (zz / (1.f + expf(-zz))));
   }
 }
 
@@ -143,68 +274,96 @@ __global__ void gdn_gate_norm_kernel(const __nv_bfloat16* __restrict__ o, const 
 
 using namespace ogb;
 
-static int LaunchGatedDelta(GdnParams p, int B, void* stream) {
+template <typename T, int NPT>
+static bool LaunchGdnDecode(const GdnParams<T>& p, int B, int splits, cudaStream_t s) {
+  return launch_pdl(gated_delta_kernel<T, NPT>, dim3(B, p.Hv, (p.dv + 31) / 32), dim3(32 * splits), 0, s, p);
+}
+template <typename T, int NPT, int CH>
+static bool LaunchGdnChunk(const GdnParams<T>& p, int B, cudaStream_t s) {
+  return launch_pdl(gated_delta_chunk_kernel<T, NPT, CH>, dim3(B, p.Hv, (p.dv + 31) / 32), dim3(128), 0, s, p);
+}
+
+// max_q_len: the most tokens a request of the launch feeds (1: the decode kernel; 0: unknown, treated as a prompt)
+template <typename T>
+static int LaunchGatedDelta(const GdnParams<T>& p, int B, int max_q_len, void* stream) {
   if (B <= 0) return 0;
   const int dk = p.dk, dv = p.dv;
-  if (p.Hk <= 0 || p.Hv % p.Hk || dv > 128 || dv <= 0) return -1;
-  if (dk < 16 || dk > 256 || (dk & (dk - 1))) return -5;
-  // a CTA takes 32 columns of the head's state (all of them when dv is not a multiple of 32): small CTAs, several per SM, so that
-  // the load, update and store phases of different CTAs overlap
-  const int Pp = (dv % 32 == 0) ? 32 : (dv + 31) / 32 * 32;
-  const int ztiles = (dv % 32 == 0) ? dv / 32 : 1;
-  int npt = dk < 32 ? dk : 32;      // measured at Qwen3.5 shapes: 32 rows per thread 51 us, 16 rows 63 us, 64 rows 54 us (64 requests)
-  if (Pp * (dk / npt) > 512) npt = 64;
-  const int splits = dk / npt;
-  if (splits > 8 || Pp * splits > 512) return -5;
-  dim3 grid(B, p.Hv, ztiles), block(Pp * splits);
+  if (p.Hk <= 0 || p.Hv % p.Hk || dv <= 0 || dk <= 0) return -1;
+  if (dk > GDN_MAX_DK) return -5;
   auto s = static_cast<cudaStream_t>(stream);
   bool ok;
-  switch (npt) {
-    case 16: ok = launch_pdl(gated_delta_kernel<16>, grid, block, 0, s, p); break;
-    case 32: ok = launch_pdl(gated_delta_kernel<32>, grid, block, 0, s, p); break;
-    case 64: ok = launch_pdl(gated_delta_kernel<64>, grid, block, 0, s, p); break;
-    default: return -5;
+  if (max_q_len != 1 && dk <= 256) {
+    if (dk <= 32) ok = LaunchGdnChunk<T, 8, 32>(p, B, s);
+    else if (dk <= 64) ok = LaunchGdnChunk<T, 16, 32>(p, B, s);
+    else if (dk <= 128) ok = LaunchGdnChunk<T, 32, 32>(p, B, s);
+    else ok = LaunchGdnChunk<T, 64, 16>(p, B, s);
+    return ok ? 0 : -4;
   }
+  // measured at Qwen3.5 shapes: 32 rows per thread 51 us, 16 rows 63 us, 64 rows 54 us (64 requests)
+  if (dk <= 16) ok = LaunchGdnDecode<T, 16>(p, B, 1, s);
+  else if (dk <= 32 * GDN_MAX_SPLITS) ok = LaunchGdnDecode<T, 32>(p, B, (dk + 31) / 32, s);
+  else ok = LaunchGdnDecode<T, 64>(p, B, (dk + 63) / 64, s);
   return ok ? 0 : -4;
 }
 
 OGB_API int ogb_gated_delta(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state, const int32_t* slots,
-                            const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, void* stream) {
-  GdnParams p{};
-  p.q = static_cast<const __nv_bfloat16*>(q); p.k = static_cast<const __nv_bfloat16*>(k); p.v = static_cast<const __nv_bfloat16*>(v);
+                            const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, int max_q_len,
+                            void* stream) {
+  using T = __nv_bfloat16;
+  GdnParams<T> p{};
+  p.q = static_cast<const T*>(q); p.k = static_cast<const T*>(k); p.v = static_cast<const T*>(v);
   p.tok_stride_qk = static_cast<long long>(Hk) * dk; p.tok_stride_v = static_cast<long long>(Hv) * dv;
   p.g = g; p.beta = beta; p.l2norm = 0; p.q_scale = 1.f;
-  p.state = state; p.slots = slots; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.out = static_cast<__nv_bfloat16*>(out);
+  p.state = state; p.slot_stride = static_cast<long long>(Hv) * dk * dv;
+  p.slots = slots; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.out = static_cast<T*>(out);
   p.Hk = Hk; p.Hv = Hv; p.dv = dv; p.dk = dk;
-  return LaunchGatedDelta(p, B, stream);
+  return LaunchGatedDelta(p, B, max_q_len, stream);
+}
+
+template <typename T>
+static int GatedDeltaFused(const void* conv, long long conv_stride, long long q_off, long long k_off, long long v_off, const void* ba,
+                           long long ba_stride, long long b_off, long long a_off, const float* neg_exp_a, const float* dt_bias, float q_scale,
+                           float l2_eps, float* state, long long slot_stride, const int32_t* slots, const int32_t* cu_seqlens,
+                           const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv, int max_q_len, void* stream) {
+  GdnParams<T> p{};
+  auto c = static_cast<const T*>(conv);
+  auto r = static_cast<const T*>(ba);
+  p.q = c + q_off; p.k = c + k_off; p.v = c + v_off; p.tok_stride_qk = conv_stride; p.tok_stride_v = conv_stride;
+  p.g = nullptr; p.beta = nullptr; p.b_raw = r + b_off; p.a_raw = r + a_off; p.ba_stride = ba_stride;
+  p.neg_exp_a = neg_exp_a; p.dt_bias = dt_bias; p.l2norm = 1; p.q_scale = q_scale; p.l2_eps = l2_eps;
+  p.state = state; p.slot_stride = slot_stride > 0 ? slot_stride : static_cast<long long>(Hv) * dk * dv;
+  p.slots = slots; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.out = static_cast<T*>(out);
+  p.Hk = Hk; p.Hv = Hv; p.dv = dv; p.dk = dk;
+  return LaunchGatedDelta(p, B, max_q_len, stream);
 }
 
 // The recurrence fed straight from the layer's tensors: q / k / v are column ranges of the convolved projection `conv` [T, row
 // stride] (q at q_off, k at k_off, v at v_off), normalised here; the decay and the write strength come from the raw b / a
-// projections (column ranges of `ba`, row stride ba_stride) with the layer's -exp(A_log) and dt_bias.
+// projections (column ranges of `ba`, row stride ba_stride) with the layer's -exp(A_log) and dt_bias.  l2_eps, slot_stride and
+// max_q_len as in GdnParams / LaunchGatedDelta (slot_stride 0: dense); fp32: element type of conv, ba and out (else bf16).
 OGB_API int ogb_gated_delta_fused(const void* conv, long long conv_stride, long long q_off, long long k_off, long long v_off, const void* ba,
                                   long long ba_stride, long long b_off, long long a_off, const float* neg_exp_a, const float* dt_bias,
-                                  float q_scale, float* state, const int32_t* slots, const int32_t* cu_seqlens, const int32_t* past_lens,
-                                  void* out, int B, int Hk, int Hv, int dk, int dv, void* stream) {
-  GdnParams p{};
-  auto c = static_cast<const __nv_bfloat16*>(conv);
-  auto r = static_cast<const __nv_bfloat16*>(ba);
-  p.q = c + q_off; p.k = c + k_off; p.v = c + v_off; p.tok_stride_qk = conv_stride; p.tok_stride_v = conv_stride;
-  p.g = nullptr; p.beta = nullptr; p.b_raw = r + b_off; p.a_raw = r + a_off; p.ba_stride = ba_stride;
-  p.neg_exp_a = neg_exp_a; p.dt_bias = dt_bias; p.l2norm = 1; p.q_scale = q_scale;
-  p.state = state; p.slots = slots; p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.out = static_cast<__nv_bfloat16*>(out);
-  p.Hk = Hk; p.Hv = Hv; p.dv = dv; p.dk = dk;
-  return LaunchGatedDelta(p, B, stream);
+                                  float q_scale, float l2_eps, float* state, long long slot_stride, const int32_t* slots,
+                                  const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int B, int Hk, int Hv, int dk, int dv,
+                                  int max_q_len, int fp32, void* stream) {
+  return fp32 ? GatedDeltaFused<float>(conv, conv_stride, q_off, k_off, v_off, ba, ba_stride, b_off, a_off, neg_exp_a, dt_bias, q_scale, l2_eps,
+                                       state, slot_stride, slots, cu_seqlens, past_lens, out, B, Hk, Hv, dk, dv, max_q_len, stream)
+              : GatedDeltaFused<__nv_bfloat16>(conv, conv_stride, q_off, k_off, v_off, ba, ba_stride, b_off, a_off, neg_exp_a, dt_bias, q_scale,
+                                               l2_eps, state, slot_stride, slots, cu_seqlens, past_lens, out, B, Hk, Hv, dk, dv, max_q_len, stream);
 }
 
-OGB_API int ogb_gdn_gate_norm(const void* o, const void* z, long long z_stride, const float* w, float eps, void* out, int T, int Hv, int dv,
-                              void* stream) {
+OGB_API int ogb_gdn_gate_norm(const void* o, const void* z, long long z_stride, const float* w, float eps, void* out, long long out_stride, int T,
+                              int Hv, int dv, int fp32, void* stream) {
   if (T <= 0) return 0;
-  if (dv <= 0 || dv > 256) return -1;
+  if (dv <= 0) return -1;
   const int rows = T * Hv;
-  return launch_pdl(gdn_gate_norm_kernel, dim3((rows + 7) / 8), dim3(256), 0, static_cast<cudaStream_t>(stream),
-                    static_cast<const __nv_bfloat16*>(o), static_cast<const __nv_bfloat16*>(z), z_stride, w, eps,
-                    static_cast<__nv_bfloat16*>(out), rows, Hv, dv) ? 0 : -4;
+  const dim3 grid((rows + 7) / 8), block(256);
+  auto s = static_cast<cudaStream_t>(stream);
+  using H = __nv_bfloat16;
+  return (fp32 ? launch_pdl(gdn_gate_norm_kernel<float>, grid, block, 0, s, static_cast<const float*>(o), static_cast<const float*>(z), z_stride, w, eps,
+                            static_cast<float*>(out), out_stride, rows, Hv, dv)
+               : launch_pdl(gdn_gate_norm_kernel<H>, grid, block, 0, s, static_cast<const H*>(o), static_cast<const H*>(z), z_stride, w, eps,
+                            static_cast<H*>(out), out_stride, rows, Hv, dv)) ? 0 : -4;
 }
 
 // ---------------------------------------------------------------------------------------------- Mamba-2 selective scan

@@ -54,6 +54,7 @@ class Request:
         self._engine = None
         self._opaque = None
         self._adapter: Optional[str] = None
+        self.given_tokens = False     # the caller feeds every token (Engine.run_given), nothing is sampled
         self.t_added = self.t_first = None
 
     # tokens ------------------------------------------------------------------------------------
@@ -121,6 +122,7 @@ class Request:
         o.repetition_penalty, o.no_repeat_ngram_size = float(s["repetition_penalty"]), int(s["no_repeat_ngram_size"])
         o.random_seed, o.chunk_size = int(s["random_seed"]), int(s.get("chunk_size") or 0)
         o.num_beams, o.batch_size = int(s["num_beams"]), int(s["batch_size"])
+        o.given_tokens = self.given_tokens
         if self.params.guidance_type and self.params.guidance_ff_tokens:
             raise RuntimeError("Engine requests do not support guidance ff_tokens")
         return o
@@ -241,7 +243,9 @@ class ModelExecutor:
             b *= 2
         return b
 
-    def forward(self, plan) -> torch.Tensor:
+    def forward(self, plan, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Enqueues the planned step; fp32 logits of every request's last token, or (rows: int32, on the device) of those rows of
+        the packed step."""
         B, T = len(plan.entries), plan.token_count
         st = self.staging
         lora = self.lora_of(plan) if self.lora_of is not None else None
@@ -254,7 +258,7 @@ class ModelExecutor:
             graph, logits = g
             graph.replay()
             self.last_key = key
-            return logits[:B]
+            return logits[:B] if rows is None else logits[rows.long()]      # one token per request: packed row = request
         st.upload()
         s = self._step_inputs(T, B, st.table_cols, plan.max_query_len, plan.max_kv_len)
         if plan.max_query_len > 1:
@@ -265,6 +269,10 @@ class ModelExecutor:
                     break
                 nd += 1
             s.num_decode = nd
+            if self.decoder.arch.latent_row:
+                s.host_lens = [(e.processed_before, e.num_tokens) for e in plan.entries]
+        if rows is not None:
+            s.logits_rows = rows
         if lora is not None:
             s.lora_ids, s.lora_names = lora
         if self.state_slots_of is not None:
@@ -668,6 +676,54 @@ class Engine:
         self._need_first.discard(request._native.id)
         if self.spec is not None:
             self.spec.forget(request._native.id)
+
+    def run_given(self, entries) -> List[torch.Tensor]:
+        """One step over given tokens (scoring, replay of recorded token streams): entries are (request, token ids, want), `want` the
+        places among these ids whose next-token logits are returned.  A request is admitted with its first ids (it must be new) and
+        goes on from its cache and state with later ones; nothing is sampled.  The step holds exactly these tokens, all entries as one
+        batch.  Returns fp32 logits [len(want), vocab] per entry, on the model's device.  remove_request gives a request's blocks
+        and state back."""
+        self._drain()
+        if self.core.has_pending_requests():
+            raise RuntimeError("run_given: the engine has generating requests in progress")
+        for rq, ids, want in entries:
+            ids = np.asarray(ids, dtype=np.int32).reshape(-1)
+            if any(w < 0 or w >= ids.size for w in want):
+                raise RuntimeError("run_given: `want` names places outside the given tokens")
+            if rq._native is None:
+                rq.given_tokens = True
+                rq.add_tokens(ids)
+                self.add_request(rq)
+            elif not rq.given_tokens:
+                raise RuntimeError("run_given: the request is a generating one")
+            else:
+                rq.continue_with(ids)
+        plan = self.core.plan()
+        self.last_outcome = plan.outcome
+        at = {e.request.id: e for e in plan.entries}
+        whole = plan.outcome == StepOutcome.Planned and all(
+            rq._native.id in at and at[rq._native.id].num_tokens == np.size(ids) for rq, ids, _ in entries) and len(at) == len(entries)
+        if not whole:
+            if plan.outcome == StepOutcome.Planned:
+                self.core.abort(FailureKind.CapacityExceeded, "run_given")
+            raise RuntimeError("run_given: the step does not fit the engine's cache, batch or max_scheduled_tokens")
+        st = self.staging
+        try:
+            st.flip()
+            self.core.pack(st.addr, st.max_tokens, st.max_batch, st.table_cols)
+            rows = [at[rq._native.id].packed_offset + w for rq, _, want in entries for w in want]
+            with torch.no_grad():
+                logits = self.executor.forward(plan, torch.tensor(rows, dtype=torch.int32, device=self.model.device))
+                if logits.is_cuda:
+                    torch.cuda.current_stream().synchronize()      # the pinned inputs of the next step may be packed now
+        except Exception as e:
+            self._fail(e)
+            raise
+        self.last_outcome = self.core.commit(np.zeros(len(plan.entries), dtype=np.int32))
+        self.step_count += 1
+        for rq, _, _ in entries:
+            self._need_first.discard(rq._native.id)
+        return list(torch.split(logits, [len(want) for _, _, want in entries]))
 
     def has_pending_requests(self) -> bool:
         return self.core.has_pending_requests()

@@ -17,7 +17,7 @@ LLM_TYPES = [
     "chatglm", "decoder", "ernie4_5", "gemma", "gemma2", "gemma3_text", "gptoss", "gpt_oss", "granite", "hunyuan", "hunyuandensev1", "hunyuan_v1_dense",
     "internlm2", "llama", "mistral", "nemotron", "olmo", "olmo2", "exaone4", "phi", "phi3", "phimoe", "qwen2", "qwen3",
     "smollm3", "lfm2", "gpt2", "helium", "mixtral", "qwen2_moe", "qwen3_moe", "granitemoe", "olmoe", "qwen2_vl", "qwen2_5_vl", "qwen3_vl",
-    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared",      # hybrids of gated-delta-net (linear attention) and full-attention layers
+    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar",      # hybrids of gated-delta-net (linear attention) and full-attention layers
 ]
 
 
@@ -25,6 +25,52 @@ LLM_TYPES = [
 # at the image-token positions (reference: src/models/model_type.h:20-26 lists the VLM / ALM families).
 VLM_TYPES = ["phi3v", "gemma3", "mistral3", "llava", "fara"]
 ALM_TYPES = ["whisper"]
+
+
+@dataclass
+class RotarySpec:
+    """Rotary positions of one layer: the first `dims` entries of a vector turn in pairs (i, i + dims / 2) with the frequencies
+    base^(-2 i / dims); scaling: None or the YaRN parameters {factor, original, fast, slow}."""
+    dims: int
+    base: float
+    scaling: Optional[Dict[str, float]] = None
+
+    def key(self):
+        return (self.dims, self.base, tuple(sorted((self.scaling or {}).items())))
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a stack whose configuration lists its layers one by one (every layer has sizes of its own).  kind:
+      "linear_attention"  gated delta rule: `kv_heads` query / key heads of `dim`, `heads` value heads of `vdim`, convolution of `conv` taps;
+      "latent_attention"  `heads` heads of `dim` unrotated + `rot_dim` rotated query / key dimensions and `vdim` value dimensions over a
+                          latent of `kv_rank` values per token; window 0: every earlier token is visible."""
+    kind: str
+    heads: int
+    dim: int
+    vdim: int
+    kv_heads: int = 0
+    conv: int = 0
+    kv_rank: int = 0
+    rot_dim: int = 0
+    scale: float = 1.0
+    window: int = 0
+    rotary: Optional[RotarySpec] = None
+    ff: int = 0                       # width of the gated feed-forward (0: the layer has none)
+    weights_of: Optional[int] = None  # layer whose weights this one uses (cache and state are its own)
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim if self.kind == "linear_attention" else 0
+
+    @property
+    def state_elems(self) -> int:
+        return self.heads * self.dim * self.vdim if self.kind == "linear_attention" else 0
+
+    @property
+    def latent_row(self) -> int:
+        """Values a token keeps in the latent cache (rounded up to whole 16-byte pieces of 16-bit values)."""
+        return (self.kv_rank + self.rot_dim + 7) // 8 * 8 if self.kind == "latent_attention" else 0
 
 
 @dataclass
@@ -81,6 +127,10 @@ class ArchConfig:
     mamba_state_size: int = 0
     mamba_n_groups: int = 1
     mamba_conv_kernel: int = 4
+    # Declared stacks: one entry per layer (see LayerSpec); layer_types then mirrors the entries' kinds.  Such stacks keep an fp32
+    # residual stream and join both sub-layers of a block in one output projection (parallel_block).
+    layer_specs: Optional[List[LayerSpec]] = None
+    delta_l2_eps: float = 0.0        # gated delta rule: > 0 makes unit vectors x / sqrt(sum(x^2) + eps) instead of x / max(|x|, 1e-6)
     # Multimodal RoPE (Qwen2-VL): rotary pairs per position component (temporal, height, width); None: ordinary RoPE
     mrope_section: Optional[List[int]] = None
     mrope_interleaved: bool = False  # qwen3_vl: the three position components alternate over the rotary pairs
@@ -180,15 +230,35 @@ class ArchConfig:
     def mamba_conv_dim(self) -> int:
         return self.mamba_intermediate + 2 * self.mamba_n_groups * self.mamba_state_size
 
+    def is_latent_layer(self, layer: int) -> bool:
+        return self.layer_types is not None and self.layer_types[layer] == "latent_attention"
+
+    def delta_sizes(self, layer: int):
+        """(key heads, value heads, key dim, value dim) of a gated-delta-net layer."""
+        if self.layer_specs is not None:
+            sp = self.layer_specs[layer]
+            return sp.kv_heads, sp.heads, sp.dim, sp.vdim
+        return self.linear_num_key_heads, self.linear_num_value_heads, self.linear_key_head_dim, self.linear_value_head_dim
+
+    @property
+    def latent_row(self) -> int:
+        """Values per token of the latent cache rows (the widest layer's)."""
+        return max((sp.latent_row for sp in self.layer_specs), default=0) if self.layer_specs is not None else 0
+
     @property
     def recurrent_state_shape(self):
-        """Per request and layer: gated delta net [value heads, key dim, value dim]; Mamba-2 [heads, state size, head dim]."""
+        """Per request and layer: gated delta net [value heads, key dim, value dim]; Mamba-2 [heads, state size, head dim]; stacks whose
+        layers differ: the largest layer's element count (a layer's state fills the front of its slot)."""
+        if self.layer_specs is not None:
+            return ((max(sp.state_elems for sp in self.layer_specs) + 3) // 4 * 4,)
         if self.has_mamba_layers:
             return (self.mamba_num_heads, self.mamba_state_size, self.mamba_head_dim)
         return (self.linear_num_value_heads, self.linear_key_head_dim, self.linear_value_head_dim)
 
     @property
     def recurrent_conv_dim(self) -> int:
+        if self.layer_specs is not None:      # rows of whole 16-byte pieces
+            return (max(sp.conv_channels for sp in self.layer_specs) + 7) // 8 * 8
         return self.mamba_conv_dim if self.has_mamba_layers else self.linear_conv_dim
 
     @property
@@ -207,6 +277,8 @@ class ArchConfig:
         """Channels of the paged convolution-input cache of a layer (0: the layer keeps none)."""
         if self.is_conv_layer(layer):
             return self.hidden_size
+        if self.layer_specs is not None:
+            return self.layer_specs[layer].conv_channels
         if self.is_linear_layer(layer):
             return self.linear_conv_dim
         if self.is_mamba_layer(layer):
@@ -225,6 +297,89 @@ class ArchConfig:
 
     def to_dict(self) -> Dict[str, Any]:
         return asdict(self)
+
+
+# Designs whose config.json lists the layers one by one ("architecture", "layers": [{"type", "mixer", "mlp"}, ...], "norm", "vocab",
+# "width"): what a design fixes for all its models.
+STACK_DESIGNS: Dict[str, Dict[str, Any]] = {
+    # parallel blocks under one layer norm (weight and bias); gated delta rule and latent attention; ReLU-gated feed-forward
+    "Luzatar": dict(model_type="luzatar", layernorm=True, parallel_block=True, activation="relu", delta_l2_eps=1e-6),
+}
+_STACK_MIXERS = {"delta": "linear_attention", "latent_attention": "latent_attention"}
+
+
+def is_stack_config(cfg: Dict[str, Any]) -> bool:
+    return isinstance(cfg, dict) and cfg.get("architecture") in STACK_DESIGNS and isinstance(cfg.get("layers"), list)
+
+
+def _stack_layer(i: int, e: Dict[str, Any]) -> LayerSpec:
+    kind = _STACK_MIXERS.get(e.get("type"))
+    if kind is None:
+        raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
+    m, mlp = e["mixer"], e.get("mlp")
+    if mlp and mlp.get("kind", "dense") != "dense":
+        raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+    sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), ff=int(mlp["ff"]) if mlp else 0,
+                   weights_of=None if e.get("weights_of") is None else int(e["weights_of"]))
+    if kind == "linear_attention":
+        sp.kv_heads, sp.conv = int(m["kv_heads"]), int(m["conv"])
+        if sp.heads % sp.kv_heads:
+            raise ValueError(f"layer {i}: {sp.heads} heads do not divide over {sp.kv_heads} key heads")
+    else:
+        sp.kv_rank, sp.rot_dim, sp.scale = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"])
+        sp.window = int((m.get("mask") or {}).get("size") or 0)
+        if m.get("rot"):
+            sc = m["rot"].get("scaling")
+            sp.rotary = RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"]), {k: float(v) for k, v in sc.items()} if sc else None)
+            if sp.rotary.dims > sp.rot_dim or sp.rotary.dims % 2:
+                raise ValueError(f"layer {i}: {sp.rotary.dims} rotary dimensions do not fit the rotated part of {sp.rot_dim}")
+    return sp
+
+
+def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
+    """config.json of a declared stack -> ArchConfig."""
+    specs = [_stack_layer(i, e) for i, e in enumerate(cfg["layers"])]
+    for i, sp in enumerate(specs):
+        if sp.weights_of is not None and not (0 <= sp.weights_of < len(specs) and specs[sp.weights_of].weights_of is None and
+                                              specs[sp.weights_of].kind == sp.kind and sp.weights_of != i):
+            raise ValueError(f"layer {i}: weights_of {sp.weights_of} does not name a layer of its kind with weights of its own")
+    lat = [sp for sp in specs if sp.kind == "latent_attention"]
+    # longest sequence the rotary scaling was made for, and at least 32768 positions (recurrent and windowed layers have no limit)
+    span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in lat if sp.rotary and sp.rotary.scaling]
+    eos = cfg.get("eos_token_id")
+    return ArchConfig(vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=max(sp.heads for sp in specs),
+                      num_kv_heads=1, head_dim=max((sp.kv_rank + sp.rot_dim for sp in lat), default=specs[0].dim),
+                      intermediate_size=max(sp.ff for sp in specs), context_length=int(cfg.get("context_length") or max([32768] + span)),
+                      norm_eps=float(cfg["norm"]["eps"]), layer_specs=specs, layer_types=[sp.kind for sp in specs], no_rope=not lat,
+                      bos_token_id=int(cfg.get("bos_token_id", 0)), eos_token_id=-1 if eos is None else eos, pad_token_id=int(cfg.get("pad_token_id", 0)),
+                      **STACK_DESIGNS[cfg["architecture"]])
+
+
+def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
+    """Names and shapes of a declared stack's checkpoint tensors."""
+    W = arch.hidden_size
+    out: Dict[str, tuple] = {"embed": (arch.vocab_size, W), "final.norm": (W,), "head": (arch.vocab_size, W)}
+    if arch.layernorm:
+        out["final.norm.b"] = (W,)
+    for i, sp in enumerate(arch.layer_specs):
+        if sp.weights_of is not None:
+            continue
+        p, m = f"l{i}.", f"l{i}.mix."
+        out[p + "norm1"] = (W,)
+        if arch.layernorm:
+            out[p + "norm1.b"] = (W,)
+        if sp.kind == "linear_attention":
+            kd, vd = sp.kv_heads * sp.dim, sp.heads * sp.vdim
+            for n, c in (("q", kd), ("k", kd), ("v", vd)):
+                out[m + n], out[m + n + ".conv"] = (c, W), (c, sp.conv)
+            out.update({m + "b": (sp.heads, W), m + "a": (sp.heads, W), m + "A_log": (sp.heads,), m + "dt_bias": (sp.heads,), m + "norm": (sp.vdim,),
+                        m + "g": (vd, W), m + "o": (W, vd)})
+        else:
+            out.update({m + "q": (sp.heads * (sp.dim + sp.rot_dim), W), m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
+                        m + "uk": (sp.heads * sp.dim, sp.kv_rank), m + "uv": (sp.heads * sp.vdim, sp.kv_rank), m + "o": (W, sp.heads * sp.vdim)})
+        if sp.ff:
+            out.update({p + "mlp.gate": (sp.ff, W), p + "mlp.up": (sp.ff, W), p + "mlp.down": (W, sp.ff)})
+    return out
 
 
 def from_hf_config(cfg: Dict[str, Any]) -> ArchConfig:
@@ -488,6 +643,29 @@ def from_hf_config(cfg: Dict[str, Any]) -> ArchConfig:
 
 
 # --------------------------------------------------------------------------------------------- RoPE caches
+def yarn_frequencies(inv_freq, rot: int, base: float, factor: float, original: float, fast: float, slow: float, last: int):
+    """YaRN: pairs that turn fewer than `slow` times over the original context are slowed down by `factor`, pairs that turn more than
+    `fast` times keep their frequency, a linear ramp over the pair index lies between (its upper end is capped at `last`)."""
+    def corr(num_rot):
+        return (rot * math.log(original / (num_rot * 2 * math.pi))) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(corr(fast)), 0), min(math.ceil(corr(slow)), last)
+    ramp = np.clip((np.arange(rot // 2, dtype=np.float64) - lo) / max(hi - lo, 1e-3), 0, 1)
+    return inv_freq / factor * ramp + inv_freq * (1.0 - ramp)
+
+
+def rotary_tables(spec: RotarySpec, n: int):
+    """cos / sin [n, dims / 2] fp32 of a layer's rotary positions (angles in float64; YaRN multiplies both by 0.1 ln(factor) + 1)."""
+    inv_freq = spec.base ** (-np.arange(0, spec.dims, 2, dtype=np.float64) / spec.dims)
+    amp = 1.0
+    if spec.scaling:
+        sc = spec.scaling
+        inv_freq = yarn_frequencies(inv_freq, spec.dims, spec.base, sc["factor"], sc["original"], sc["fast"], sc["slow"], spec.dims - 1)
+        amp = 0.1 * math.log(sc["factor"]) + 1.0
+    ang = np.outer(np.arange(n, dtype=np.float64), inv_freq)
+    return (np.cos(ang) * amp).astype(np.float32), (np.sin(ang) * amp).astype(np.float32)
+
+
 def rope_caches(arch: ArchConfig, max_positions: Optional[int] = None, local: bool = False):
     """cos/sin caches of shape [positions, rotary_dim/2] (fp32), with the frequency rescaling the
     reference's exporter applies (default, linear, llama3, yarn; src/python/py/models/builders/
@@ -518,13 +696,7 @@ def rope_caches(arch: ArchConfig, max_positions: Optional[int] = None, local: bo
         old = float(sc.get("original_max_position_embeddings", arch.context_length / factor))
         beta_fast, beta_slow = float(sc.get("beta_fast", 32)), float(sc.get("beta_slow", 1))
 
-        def corr(num_rot):
-            return (rot * math.log(old / (num_rot * 2 * math.pi))) / (2 * math.log(arch.rope_theta))
-
-        lo, hi = max(math.floor(corr(beta_fast)), 0), min(math.ceil(corr(beta_slow)), rot // 2 - 1)
-        ramp = np.clip((np.arange(rot // 2, dtype=np.float64) - lo) / max(hi - lo, 1e-3), 0, 1)
-        mask = 1.0 - ramp
-        inv_freq = inv_freq / factor * (1 - mask) + inv_freq * mask
+        inv_freq = yarn_frequencies(inv_freq, rot, arch.rope_theta, factor, old, beta_fast, beta_slow, rot // 2 - 1)
         attn_factor = float(sc.get("attention_factor") or (0.1 * math.log(factor) + 1.0))
     t = np.arange(n, dtype=np.float64)
     freqs = np.outer(t, inv_freq)

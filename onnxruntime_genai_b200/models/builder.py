@@ -33,7 +33,7 @@ import numpy as np
 import torch
 
 from ..utils import onnx_proto as op
-from .arch import PRESETS, ArchConfig, from_hf_config, longrope_caches, rope_caches
+from .arch import PRESETS, ArchConfig, from_hf_config, is_stack_config, longrope_caches, rope_caches
 
 _ONNX_DT = {"fp32": op.FLOAT, "fp16": op.FLOAT16, "bf16": op.BFLOAT16}
 _TORCH_DT = {"fp32": torch.float32, "fp16": torch.float16, "bf16": torch.bfloat16}
@@ -1509,6 +1509,29 @@ def _split_packed_qkv(sd: Dict[str, torch.Tensor], arch: ArchConfig) -> None:
         sd[base + "q_proj.weight"], sd[base + "k_proj.weight"], sd[base + "v_proj.weight"] = q, kk, vv
 
 
+def export_stack(model_dir: str, raw_cfg: dict, output_dir: str, precision: str, execution_provider: str, extra: dict) -> str:
+    """A declared stack (config.json that lists its layers): the weights stay as they are, a genai_config.json is written beside them.
+    random_weights / synthetic_weights: weights drawn on the device at load (`seed`)."""
+    from . import stack_checkpoint as sc
+    if precision not in ("bf16", "fp32"):
+        raise ValueError("declared stacks are exported in bf16 or fp32")
+    synthetic = bool(int(extra.get("synthetic_weights", extra.get("random_weights", 0))))
+    filename = "model.synthetic.json" if synthetic else sc.WEIGHTS
+    os.makedirs(output_dir, exist_ok=True)
+    same = os.path.abspath(model_dir) == os.path.abspath(output_dir)
+    for fn in ("config.json", "tokenizer.json", "tokenizer_config.json", "special_tokens_map.json", "chat_template.jinja") + (() if synthetic else (filename,)):
+        if not same and os.path.exists(os.path.join(model_dir, fn)):
+            shutil.copy(os.path.join(model_dir, fn), os.path.join(output_dir, fn))
+    if synthetic:
+        with open(os.path.join(output_dir, filename), "w") as f:
+            json.dump({"seed": int(extra.get("seed", 0)), "std": float(extra.get("std", 0.02))}, f)
+    doc = sc.genai_config_of(raw_cfg, execution_provider, precision, filename, int(extra.get("paged_block_size", 16)), int(extra.get("max_batch_size", 64)),
+                             int(extra["context_length"]) if "context_length" in extra else None)
+    with open(os.path.join(output_dir, "genai_config.json"), "w") as f:
+        json.dump(doc, f, indent=2)
+    return output_dir
+
+
 def create_model(model_name_or_dir: str, output_dir: str, precision: str, execution_provider: str, extra_options: Optional[dict] = None):
     extra = dict(extra_options or {})
     state_dict = None
@@ -1523,6 +1546,8 @@ def create_model(model_name_or_dir: str, output_dir: str, precision: str, execut
     else:
         with open(os.path.join(model_name_or_dir, "config.json")) as f:
             raw_cfg = json.load(f)
+        if is_stack_config(raw_cfg):
+            return export_stack(model_name_or_dir, raw_cfg, output_dir, precision, execution_provider, extra)
         if (raw_cfg.get("architectures") or [""])[0] == "WhisperForConditionalGeneration" or raw_cfg.get("model_type") == "whisper":
             # encoder-decoder speech checkpoint: decoder.onnx + encoder.onnx + the log-mel front end's configuration
             arch, enc, dsd, esd = whisper_from_hf(raw_cfg, load_hf_state_dict(model_name_or_dir))
@@ -1599,7 +1624,7 @@ def create_model(model_name_or_dir: str, output_dir: str, precision: str, execut
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description="Export a model directory (genai_config.json + ONNX + external data)")
-    ap.add_argument("-m", "--model_name", required=True, help="Hugging Face model directory or a preset: " + ", ".join(PRESETS))
+    ap.add_argument("-m", "--model_name", required=True, help="Hugging Face model directory, the directory of a declared stack, or a preset: " + ", ".join(PRESETS))
     ap.add_argument("-o", "--output", required=True)
     ap.add_argument("-p", "--precision", required=True, choices=["int4", "bf16", "fp16", "fp32"])
     ap.add_argument("-e", "--execution_provider", default="cuda", choices=["cpu", "cuda"])

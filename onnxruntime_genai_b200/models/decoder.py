@@ -16,6 +16,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
+import numpy as np
 import torch
 
 from .. import ops
@@ -50,6 +51,8 @@ class StepInputs:
     return_hidden: bool = False
     lora_ids: Optional[torch.Tensor] = None      # [T] int32: index of each token's adapter in `lora_names` (len(lora_names) = none)
     lora_names: Optional[tuple] = None           # adapters present in this step (a batch may mix several and none)
+    host_lens: Optional[list] = None             # [(past length, tokens)] of every request, where the host knows them (latent layers: plans long prompts)
+    latent_plans: Optional[dict] = None          # made by the forward: expansion plan of the long requests per window
     state_slots: Optional[torch.Tensor] = None   # [B] int32 slot of each request in the recurrent-state pool (linear-attention layers)
 
 
@@ -71,12 +74,19 @@ class PagedKVCache:
         self.num_window_blocks = num_window_blocks
         hk = kv_heads if kv_heads is not None else arch.num_kv_heads
         conv = [arch.conv_state_channels(i) > 0 for i in range(arch.num_layers)]
+        # Latent-attention layers: one row per token (normalised latent, shared rotated key) in the same paged slots.
+        self.latent_index = {i: j for j, i in enumerate(i for i in range(arch.num_layers) if arch.is_latent_layer(i))}
+        self.latent = (torch.zeros(len(self.latent_index), num_blocks * block_size, arch.latent_row, dtype=dtype, device=device)
+                       if self.latent_index else None)
+        if self.latent is not None and kv_bits != 16:
+            raise RuntimeError("KV cache quantization is not available for latent-attention layers")
+        conv = [c or i in self.latent_index for i, c in enumerate(conv)]        # layers without key / value rows
         self.windowed = [num_window_blocks > 0 and arch.layer_window(i) > 0 and not conv[i] for i in range(arch.num_layers)]
         n_full = sum(1 for w, c in zip(self.windowed, conv) if not w and not c)
         n_win = sum(1 for w in self.windowed if w)
         # Hybrid models: the gated input (b * x) of every position of every convolution layer, in the same paged slots as
         # the keys and values - rewinding, beam reordering and block sharing need nothing layer-specific.
-        self.conv_index = {i: j for j, i in enumerate(i for i, c in enumerate(conv) if c)}
+        self.conv_index = {i: j for j, i in enumerate(i for i in range(arch.num_layers) if arch.conv_state_channels(i) > 0)}
         cc = conv_channels if conv_channels is not None else arch.hidden_size
         if arch.has_linear_layers:
             cc = arch.recurrent_conv_dim
@@ -88,7 +98,7 @@ class PagedKVCache:
         self.state = None
         self.state_slots = 0
         row, kdt = (arch.head_dim + 16, torch.int8) if kv_bits == 8 else (arch.head_dim, dtype)
-        self.full = torch.zeros(max(n_full, 1), 2, num_blocks * block_size, hk, row, dtype=kdt, device=device)
+        self.full = torch.zeros(max(n_full, 0 if arch.layer_specs is not None else 1), 2, num_blocks * block_size, hk, row, dtype=kdt, device=device)
         self.win = (torch.zeros(n_win, 2, num_window_blocks * block_size, hk, row, dtype=kdt, device=device)
                     if n_win else None)
         self._index = []
@@ -107,7 +117,10 @@ class PagedKVCache:
         return pool[j, 0], pool[j, 1], win
 
     def conv_layer(self, i: int) -> torch.Tensor:
-        return self.conv[self.conv_index[i]]
+        return self.conv[self.conv_index[i]][:, :self.arch.conv_state_channels(i)]
+
+    def latent_layer(self, i: int) -> torch.Tensor:
+        return self.latent[self.latent_index[i]]
 
     def ensure_state_slots(self, n: int) -> None:
         """At least n request slots in the recurrent-state pool (grown by copying; states of live slots are kept)."""
@@ -120,7 +133,12 @@ class PagedKVCache:
         self.state, self.state_slots = new, n
 
     def state_layer(self, i: int) -> torch.Tensor:
-        return self.state[self.lin_index[i]]
+        """[slots, heads, ...] state of one layer; slots may be further apart than a state is long (stacks whose layers differ)."""
+        st = self.state[self.lin_index[i]]
+        if self.arch.layer_specs is None:
+            return st
+        sp = self.arch.layer_specs[i]
+        return st[:, :sp.state_elems].view(st.shape[0], sp.heads, sp.dim, sp.vdim)
 
     @staticmethod
     def bytes_per_block(arch: ArchConfig, block_size: int, dtype, kv_heads: Optional[int] = None, conv_channels: Optional[int] = None,
@@ -130,7 +148,8 @@ class PagedKVCache:
         cc = arch.recurrent_conv_dim if arch.has_linear_layers else (conv_channels if conv_channels is not None else arch.hidden_size)
         es = torch.empty((), dtype=dtype).element_size()
         kv_row = arch.head_dim + 16 if kv_bits == 8 else arch.head_dim * es
-        return ((arch.num_layers - n_conv) * 2 * hk * kv_row + n_conv * cc * es) * block_size
+        n_lat = sum(1 for i in range(arch.num_layers) if arch.is_latent_layer(i))
+        return ((arch.num_layers - n_conv - n_lat) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row) * es) * block_size
 
 
 class CrossKVCache:
@@ -201,6 +220,16 @@ class LayerWeights:
     lin_neg_exp_a: Optional[torch.Tensor] = None
     lin_norm_w: Optional[torch.Tensor] = None
     lin_out_w: Optional[torch.Tensor] = None
+    lat_in_w: Optional[torch.Tensor] = None    # latent attention: stacked [queries (heads x (dim | rot)) | latent | shared rotated key] projection
+    lat_norm_w: Optional[torch.Tensor] = None  # RMS weight of the latent (fp32)
+    lat_uk_t: Optional[torch.Tensor] = None    # per head the transposed key map [heads * kv_rank, dim]: folds keys into the query
+    lat_uv: Optional[torch.Tensor] = None      # value map [heads * vdim, kv_rank]
+    lat_ukv: Optional[torch.Tensor] = None     # [key map; value map]: expands cached latents for long prompts
+    rope_cos: Optional[torch.Tensor] = None    # rotary tables of this layer
+    rope_sin: Optional[torch.Tensor] = None
+    join_w: Optional[torch.Tensor] = None      # parallel blocks on an fp32 stream: [mixer output map | down] over [mixer output (padded) | feed-forward]
+    mix_cols: int = 0                          # columns of the mixer output in the joined input, and where the feed-forward starts
+    mlp_col: int = 0
     cross_ln_w: Optional[torch.Tensor] = None  # encoder-decoder cross-attention (whisper)
     cross_ln_b: Optional[torch.Tensor] = None
     cross_q_w: Optional[torch.Tensor] = None
@@ -348,29 +377,43 @@ class DecoderModel:
                             max_kv_len=s.max_kv_len, out=out)
         return out
 
-    def _linear_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor) -> torch.Tensor:
+    @staticmethod
+    def _wide_linear(x, w):
+        """x @ w.T with rows of whole 16-byte pieces, so that column ranges of the result can be read in vectors."""
+        N = w.shape[0]
+        if not x.is_cuda:
+            return ops.linear(x, w)
+        out = torch.empty(x.shape[0], (N + 7) // 8 * 8, dtype=x.dtype, device=x.device)[:, :N]
+        return ops.linear(x, w, out=out)
+
+    def _linear_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out=None) -> torch.Tensor:
         """A gated-delta-net layer (reference graph: builders/qwen.py:1776-1867).  The causal convolution reads the projected
         q / k / v rows of the last K - 1 positions from the paged cache (the short-convolution kernel of the hybrid models with
-        unit gates), so rewinding and block copies need no convolution state; the recurrent state lives in the request's slot."""
+        unit gates), so rewinding and block copies need no convolution state; the recurrent state lives in the request's slot.
+        out: the layer's value heads are left there (a column range), their output projection is the caller's."""
         a = self.arch
         if s.state_slots is None:
             raise RuntimeError("this model has linear-attention layers: the caller must provide StepInputs.state_slots")
         T = x.shape[0]
-        cd, vd, nk, nv, hk, hv = a.linear_conv_dim, a.linear_value_dim, a.linear_num_key_heads, a.linear_num_value_heads, a.linear_key_head_dim, a.linear_value_head_dim
-        proj = self._linear(x, lw.lin_in_w)
+        nk, nv, hk, hv = a.delta_sizes(li)
+        vd, kd = nv * hv, nk * hk
+        cd = 2 * kd + vd
+        proj = self._wide_linear(x, lw.lin_in_w)
         qkv, z, b_, a_ = proj[:, :cd], proj[:, cd:cd + vd], proj[:, cd + vd:cd + vd + nv], proj[:, cd + vd + nv:]
         conv = ops.causal_conv(qkv, lw.lin_conv_w, None, kv.conv_layer(li), s.slot_mapping, s.positions, s.cu_seqlens, s.past_lens,
                                s.block_table, kv.block_size, silu=True)
-        if (conv.is_cuda and conv.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16 and hv <= 128 and hk in (16, 32, 64, 128, 256) and
-                lw.lin_norm_w.dtype == torch.float32):
+        if conv.is_cuda:
             # normalisation, gates, recurrence and the gated output norm in two kernels
             o = ops.gated_delta_layer(conv, proj, cd, vd, nk, nv, hk, hv, lw.lin_neg_exp_a, lw.lin_dt_bias, lw.lin_norm_w, a.norm_eps,
-                                      kv.state_layer(li), s.state_slots, s.cu_seqlens, s.past_lens)
-            return self._row_parallel(o, lw.lin_out_w, None, None)
+                                      kv.state_layer(li), s.state_slots, s.cu_seqlens, s.past_lens, s.max_q_len, a.delta_l2_eps, out)
+            return o if out is not None else self._row_parallel(o, lw.lin_out_w, None, None)
         conv = conv.float()
-        kd = nk * hk
-        q = torch.nn.functional.normalize(conv[:, :kd].view(T, nk, hk), dim=-1, eps=1e-6) * (hk ** -0.5)
-        k = torch.nn.functional.normalize(conv[:, kd:2 * kd].view(T, nk, hk), dim=-1, eps=1e-6)
+        q, k = conv[:, :kd].view(T, nk, hk), conv[:, kd:2 * kd].view(T, nk, hk)
+        if a.delta_l2_eps > 0:
+            q, k = (t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + a.delta_l2_eps) for t in (q, k))
+        else:
+            q, k = (torch.nn.functional.normalize(t, dim=-1, eps=1e-6) for t in (q, k))
+        q = q * (hk ** -0.5)
         v = conv[:, 2 * kd:].view(T, nv, hv)
         beta = torch.sigmoid(b_.float())
         g = lw.lin_neg_exp_a * torch.nn.functional.softplus(a_.float() + lw.lin_dt_bias)
@@ -378,7 +421,64 @@ class DecoderModel:
                             s.state_slots, s.cu_seqlens, s.past_lens).float()
         o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + a.norm_eps) * lw.lin_norm_w          # RMS norm per value head
         o = (o.view(T, vd) * torch.nn.functional.silu(z.float())).to(x.dtype)
-        return self._row_parallel(o, lw.lin_out_w, None, None)
+        return out.copy_(o) if out is not None else self._row_parallel(o, lw.lin_out_w, None, None)
+
+    def _latent_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """A latent-attention layer: writes the value heads of every token to `out` [T, heads * vdim] (a column range).  Decode steps and
+        short portions attend over the cached latents with the key map folded into the queries; requests that feed many tokens expand
+        the latents they can see to keys and values and run on the tensor-memory kernel."""
+        sp = self.arch.layer_specs[li]
+        T = x.shape[0]
+        shape = ops.latent_shape(sp.heads, sp.dim, sp.rot_dim, sp.vdim, sp.kv_rank, sp.rotary.dims if sp.rotary else 0)
+        cache = kv.latent_layer(li)
+        proj = self._wide_linear(x, lw.lat_in_w)
+        ops.latent_prep(proj, shape, lw.lat_norm_w, self.arch.norm_eps, s.positions, lw.rope_cos, lw.rope_sin, s.slot_mapping, cache)
+        plan = None
+        if s.host_lens is not None and s.max_q_len >= ops.LATENT_LONG_TOKENS and ops.latent_long_supported(shape, proj, cache, kv.block_size):
+            if s.latent_plans is None:
+                s.latent_plans = {}
+            plan = s.latent_plans.get(sp.window)
+            if plan is None:
+                plan = s.latent_plans[sp.window] = ops.LatentPlan(s.host_lens, sp.window, x.device)
+        n_short = T
+        if plan is not None:
+            # tokens up to the last one of a short request (the scheduler puts the decoding requests first)
+            ends = np.cumsum([n for _, n in s.host_lens])
+            n_short = max([int(e) for e, (_, n) in zip(ends, s.host_lens) if n < ops.LATENT_LONG_TOKENS], default=0)
+        if n_short > 0:
+            qlat = ops.head_project(proj[:n_short], lw.lat_uk_t, sp.heads, sp.dim + sp.rot_dim)
+            olat = ops.latent_attention(qlat, proj, shape, cache, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale, sp.window,
+                                        s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0)
+            ops.head_project(olat, lw.lat_uv, sp.heads, sp.kv_rank, out=out[:n_short])
+        if plan is not None and plan.rows > 0:
+            ops.latent_attention_long(proj, shape, lw.lat_ukv, cache, plan, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale,
+                                      sp.window, out)
+        return out
+
+    def _forward_stream(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
+        """Parallel blocks on an fp32 residual stream (declared stacks): per layer one norm, the mixer and the gated feed-forward side by
+        side into the column ranges of one matrix, and one output projection of both whose epilogue adds to the stream in fp32."""
+        a = self.arch
+        if self.tp.size > 1:
+            raise RuntimeError("declared stacks run on one GPU")
+        if s.lora_ids is not None or self.active_adapter is not None:
+            raise RuntimeError("LoRA adapters are not available for declared stacks")
+        h = s.inputs_embeds.float().clone() if s.inputs_embeds is not None else ops.embedding_stream(s.input_ids, self.embed, a.embed_scale)
+        T = h.shape[0]
+        for li, lw in enumerate(self.layers):
+            x = ops.norm_stream(h, lw.ln1_w, a.norm_eps, lw.ln1_b, a.layernorm, self.dtype)
+            K = lw.join_w.shape[1]
+            used = (lw.mlp_col == lw.mix_cols or lw.gate_up_w is None) and K == lw.mix_cols + (a.layer_specs[li].ff)
+            y = (torch.empty if used else torch.zeros)(T, K, dtype=self.dtype, device=h.device)      # padding columns meet zero weights: finite
+            mixer = self._linear_attention if lw.lin_in_w is not None else self._latent_attention
+            mixer(s, kv, li, lw, x, out=y[:, :lw.mix_cols])
+            if lw.gate_up_w is not None:
+                ops.gate_up_act(x, lw.gate_up_w, None, a.activation, out=y[:, lw.mlp_col:lw.mlp_col + a.layer_specs[li].ff],
+                                interleaved=lw.gate_up_interleaved)
+            h = ops.linear(y, lw.join_w, residual=h, out=h, out_fp32=True)
+        x = ops.norm_stream(h, self.final_norm_w, a.norm_eps, self.final_norm_b, a.layernorm, self.dtype, rows=s.logits_rows)
+        self.last_hidden = x
+        return ops.linear(x, self.lm_head_w, out_fp32=True)
 
     def _mamba(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor) -> torch.Tensor:
         """A Mamba-2 layer (GraniteMoeHybrid).  Like the gated-delta-net layers, the causal convolution reads the projected
@@ -599,6 +699,8 @@ class DecoderModel:
                 finally:
                     self._dumping = False
         a = self.arch
+        if a.layer_specs is not None:
+            return self._forward_stream(s, kv)
         if self._sp_ok(s):
             return self._forward_sp(s, kv)
         if self._fused_step_ok(s):
@@ -738,7 +840,9 @@ class DecoderModel:
         for t in (self.embed, self.final_norm_w, self.final_norm_b, self.lm_head_w, self.lm_head_b, self.cos, self.sin):
             if t is not None:
                 yield t
+        seen = set()
         for lw in self.layers:
             for v in vars(lw).values():
-                if isinstance(v, torch.Tensor):
+                if isinstance(v, torch.Tensor) and id(v) not in seen:      # layers may share weights
+                    seen.add(id(v))
                     yield v

@@ -316,6 +316,11 @@ def _vec(g: GraphView, name: str, dtype, device, sl: Optional[slice] = None) -> 
 
 def load_decoder(model_dir: str, cfg, device, dtype, tp=None, decoder: Optional[dict] = None) -> DecoderModel:
     d = decoder or cfg.decoder
+    if d["filename"].endswith((".safetensors", ".synthetic.json")):      # a declared stack: config.json + safetensors instead of a graph
+        from .stack_checkpoint import load_stack_decoder
+        return load_stack_decoder(model_dir, d["filename"], cfg.context_length, device, dtype, tp)
+    if torch.device(device).type == "cuda" and dtype != torch.bfloat16:
+        raise NotImplementedError("graph checkpoints run in bfloat16 on CUDA devices")
     g = GraphView(os.path.join(model_dir, d["filename"]))
     arch = arch_from_checkpoint(cfg, g, d)
     g.set_arch_shapes(arch)

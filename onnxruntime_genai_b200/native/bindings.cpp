@@ -334,6 +334,7 @@ PYBIND11_MODULE(_og_native, m) {
       .def_readwrite("no_repeat_ngram_size", &RequestOptions::no_repeat_ngram_size)
       .def_readwrite("random_seed", &RequestOptions::random_seed).def_readwrite("chunk_size", &RequestOptions::chunk_size)
       .def_readwrite("num_beams", &RequestOptions::num_beams).def_readwrite("batch_size", &RequestOptions::batch_size)
+      .def_readwrite("given_tokens", &RequestOptions::given_tokens)
       .def("resolve", [](const RequestOptions& o) { auto a = o.Resolve(); return py::make_tuple(a.top_k, a.top_p, a.temperature); });
 
   py::class_<Request, std::shared_ptr<Request>>(m, "Request")

@@ -115,7 +115,7 @@ void Request::ContinueWith(const int32_t* ids, size_t n, int new_max_length) {
   if (int(tokens_.size() + n) >= opt_.max_length)
     throw std::runtime_error("continue_with: max_length (cumulative across turns) would be exceeded");
   tokens_.insert(tokens_.end(), ids, ids + n);
-  prefill_ = true;
+  prefill_ = !(opt_.given_tokens && Pending() == 1 && processed_ > 0);
   status_ = RequestStatus::kAssigned;
 }
 
@@ -406,6 +406,10 @@ StepOutcome EngineCore::Commit(const int32_t* tokens, size_t n) {
     metrics_.tokens_scheduled += uint64_t(e.num_tokens);
     if (!e.samples) continue;
     r.prefill_ = false;
+    if (r.opt_.given_tokens) {      // nothing is sampled: the turn ends with its last given token
+      r.status_ = RequestStatus::kTurnComplete;
+      continue;
+    }
     const int32_t tok = tokens[i];
     // A sampled end-of-sequence token is part of the sequence and of the stream the caller reads, as in the reference
     // engine (src/engine/request.cpp CommitStep pushes whatever the search appended, and GreedySearch_Cpu appends the

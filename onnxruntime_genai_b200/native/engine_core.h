@@ -73,6 +73,9 @@ struct RequestOptions {
   int chunk_size{0};  // 0 = no per-request prefill cap
   int num_beams{1};
   int batch_size{1};
+  // Given tokens only: the request's tokens are fed portion by portion (AddTokens, then ContinueWith), nothing is sampled or appended;
+  // once a portion has been run the turn is complete until the next one arrives.
+  bool given_tokens{false};
   SamplingArgs Resolve() const;
 };
 
@@ -92,6 +95,7 @@ class Request {
   uint64_t Seed() const { return seed_; }
 
   void AddTokens(const int32_t* ids, size_t n);      // only while Unassigned
+  // A given-tokens request that continues with one token is planned like a decoding request.
   void ContinueWith(const int32_t* ids, size_t n, int new_max_length = 0);   // only while TurnComplete; > 0: the limit from now on
   // Speculative decoding: stages up to n proposed continuation tokens behind the pending token of a decoding request.  The
   // next step then feeds [pending token, drafts...] (1 + n rows whose logits verify the proposal) and is closed with

@@ -129,6 +129,35 @@ def embedding(ids: torch.Tensor, table, scale: float = 1.0) -> torch.Tensor:
     return out
 
 
+def embedding_stream(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """Embedding rows as the start of an fp32 residual stream (bf16 or fp32 table, any width)."""
+    _check_index("embedding_stream", "ids", ids, table.shape[0])
+    if not table.is_cuda:
+        return ref.embedding(ids, table).float() * scale
+    assert ids.dtype == torch.int32 and table.is_contiguous() and table.dtype in (torch.bfloat16, torch.float32)
+    T, H = ids.numel(), table.shape[1]
+    out = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    _lib.check(_lib.lib().ogb_embedding_stream(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), T, H, table.shape[0], float(scale),
+                                              _stream()), "embedding_stream")
+    return out
+
+
+def norm_stream(x, weight, eps, bias=None, layernorm=False, dtype=torch.bfloat16, rows=None):
+    """Norm of the rows of an fp32 residual stream [T, H] (of the rows listed in `rows`, int32, when given) as `dtype`; weight and bias
+    are fp32."""
+    if rows is not None:
+        _check_index("norm_stream", "rows", rows, x.shape[0])
+    if not x.is_cuda:
+        h = x if rows is None else x[rows.long()]
+        return ref.norm(h.float(), weight, eps, None, bias, layernorm)[0].to(dtype)
+    assert x.dtype == torch.float32 and x.is_contiguous() and weight.dtype == torch.float32 and (bias is None or bias.dtype == torch.float32)
+    n, H = (x.shape[0] if rows is None else rows.numel()), x.shape[1]
+    out = torch.empty(n, H, dtype=dtype, device=x.device)
+    _lib.check(_lib.lib().ogb_norm_stream(_ptr(x), _ptr(rows), _ptr(weight), _ptr(bias), _ptr(out), int(dtype == torch.float32), n, H, float(eps),
+                                         int(layernorm), _stream()), "norm_stream")
+    return out
+
+
 # ------------------------------------------------------------------------------------------ norm
 def norm(x, weight, eps, residual=None, bias=None, layernorm=False, out=None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
     """Returns (normalised, new_residual).  With `residual`, normalises x + residual and returns the
@@ -170,7 +199,7 @@ def norm_moe_combine(pending: PendingCombine, weight, eps, residual, bias=None, 
 
 
 # ------------------------------------------------------------------------------------------ GEMM
-GEMM_FP32_OUT, GEMM_ACT_PAIR, GEMM_ALLREDUCE, GEMM_REDUCE_SCATTER, GEMM_GATHERED_A = 1, 2, 4, 8, 16
+GEMM_FP32_OUT, GEMM_ACT_PAIR, GEMM_ALLREDUCE, GEMM_REDUCE_SCATTER, GEMM_GATHERED_A, GEMM_FP32_RESIDUAL, GEMM_PAIR_RELU = 1, 2, 4, 8, 16, 32, 64
 
 
 FUSED_MAX_TOKENS = 128     # the decode-step fusions (folded norm, rotary + cache append) run in the decode-sized GEMM kernel
@@ -219,6 +248,37 @@ def _gemm_w4(x, w, out, bias, residual, flags, splits):
     return out
 
 
+def _tma_ok(x, w) -> bool:
+    """TMA can address both operands of a bf16 product: 16-byte row strides and addresses."""
+    return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0
+
+
+def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None):
+    """The fp32 / unaligned form of a product (csrc/gemm_simt.cu)."""
+    assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and out.dtype in (torch.float32, torch.bfloat16)
+    _lib.check(_lib.lib().ogb_gemm_simt(_ptr(x), x.stride(0), int(a_cols), _ptr(w), w.stride(0), _ptr(out), out.stride(0), int(c_cols), x.shape[0],
+                                       w.shape[0] // batch, K or x.shape[1], int(batch), _ptr(residual), residual.stride(0) if residual is not None else 0,
+                                       int(x.dtype == torch.float32), int(out.dtype == torch.float32), _stream()), "gemm_simt")
+    return out
+
+
+def head_project(x, w, heads: int, a_cols: int, out=None):
+    """Per-head products over the same token rows: out[:, h * N + n] = sum_k x[:, h * a_cols + k] * w[h * N + n, k] with
+    w [heads * N, K]; x may be wider than the heads need.  Returns [T, heads * N] (or writes `out`, which may be a column range)."""
+    K, N = w.shape[1], w.shape[0] // heads
+    if out is None:
+        out = torch.empty(x.shape[0], heads * N, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        out.copy_(ref.head_project(x, w, heads, a_cols))
+        return out
+    if x.dtype == torch.float32 or a_cols % 8 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8 or (x.data_ptr() | w.data_ptr()) % 16:
+        return _gemm_simt(x, w, out, batch=heads, a_cols=a_cols, c_cols=N, K=K)
+    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    _lib.check(_lib.lib().ogb_gemm_bf16_batched(_ptr(x), x.stride(0), x.shape[1], int(a_cols), _ptr(w), w.stride(0), _ptr(out), out.stride(0), N,
+                                               x.shape[0], N, K, heads, workspace(x.device).status, _stream()), "gemm_bf16_batched")
+    return out
+
+
 def linear(x, w, bias=None, residual=None, out_fp32=False, out=None, splits=0, all_reduce=False, reduce_scatter=None, norm_eps=0.0):
     """y = x @ w.T (+bias) (+residual).  x [T, K] bf16, w [N, K] bf16 (K contiguous).  With all_reduce the
     partial products of the tensor-parallel ranks are summed inside the kernel over NVLink peer memory.
@@ -237,9 +297,17 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, out=None, splits=0, a
             out = torch.empty(x.shape[0], w.N, dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
         return _gemm_w4(x, w, out, bias, residual, GEMM_FP32_OUT if out_fp32 else 0, splits)
     if not x.is_cuda:
-        return ref.linear(x, w, bias, residual, out_fp32, norm_eps)
-    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
-    assert x.stride(-1) == 1 and w.stride(-1) == 1
+        y = ref.linear(x, w, bias, residual, out_fp32, norm_eps)
+        return y if out is None else out.copy_(y)
+    assert x.dtype == w.dtype and x.stride(-1) == 1 and w.stride(-1) == 1
+    if x.dtype == torch.float32 or (bias is None and norm_eps == 0 and not all_reduce and reduce_scatter is None and not _tma_ok(x, w) and
+                                    (residual is None or residual.dtype == torch.float32)):
+        # 32-bit models, and bf16 shapes TMA cannot address
+        assert bias is None and norm_eps == 0 and not all_reduce and reduce_scatter is None
+        if out is None:
+            out = torch.empty(x.shape[0], w.shape[0], dtype=torch.float32 if out_fp32 else x.dtype, device=x.device)
+        return _gemm_simt(x, w, out, residual)
+    assert x.dtype == torch.bfloat16
     fused = None
     if norm_eps > 0:
         if x.shape[0] > FUSED_MAX_TOKENS:
@@ -254,6 +322,8 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, out=None, splits=0, a
     if out is None:
         out = torch.empty(rows_out, w.shape[0], dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
     flags = (GEMM_FP32_OUT if out_fp32 else 0) | (GEMM_ALLREDUCE if all_reduce else 0) | (GEMM_REDUCE_SCATTER if reduce_scatter else 0)
+    if residual is not None and residual.dtype == torch.float32:
+        flags |= GEMM_FP32_RESIDUAL       # an fp32 residual stream, updated in place by the epilogue when `out` is the residual itself
     return _gemm(x, w, out, bias, residual, flags, splits, fused)
 
 
@@ -333,22 +403,32 @@ def gate_up_act(x, w, bias=None, act="silu", out=None, splits=0, interleaved=Fal
             y = y.view(-1, inter // 64, 2, 64).transpose(1, 2).reshape(-1, 2 * inter)
         return act_mul(y.contiguous(), act)
     if not x.is_cuda:
-        return ref.gate_up_act(x, w, bias, act, interleaved)
+        y = ref.gate_up_act(x, w, bias, act, interleaved)
+        return y if out is None else out.copy_(y)
     inter = w.shape[0] // 2
-    if act != "silu" or not interleaved or inter % 64:
+    if act not in ("silu", "relu") or not interleaved or inter % 64 or x.dtype != torch.bfloat16 or not _tma_ok(x, w):
         y = linear(x, w, bias)
         if interleaved:
             y = y.view(-1, inter // 64, 2, 64).transpose(1, 2).reshape(-1, 2 * inter)
-        return act_mul(y.contiguous(), act)
+        return act_mul(y.contiguous(), act, out)
     if out is None:
         out = torch.empty(x.shape[0], inter, dtype=torch.bfloat16, device=x.device)
-    return _gemm(x, w, out, bias, None, GEMM_ACT_PAIR, splits, fused)
+    return _gemm(x, w, out, bias, None, GEMM_ACT_PAIR | (GEMM_PAIR_RELU if act == "relu" else 0), splits, fused)
 
 
-def act_mul(x, act="silu"):
+def act_mul(x, act="silu", out=None):
+    """act(x[:, :I]) * x[:, I:2I]; `out` may be a column range of a wider matrix."""
     if not x.is_cuda:
-        return ref.act_mul(x, act)
+        y = ref.act_mul(x, act)
+        return y if out is None else out.copy_(y)
     T, two_i = x.shape
+    if out is not None or x.dtype != torch.bfloat16 or act not in ("silu", "gelu", "gelu_tanh"):
+        if out is None:
+            out = torch.empty(T, two_i // 2, dtype=x.dtype, device=x.device)
+        assert x.stride(1) == 1 and out.stride(1) == 1 and out.dtype == x.dtype
+        _lib.check(_lib.lib().ogb_act_mul_rows(_ptr(x), x.stride(0), _ptr(out), out.stride(0), T, two_i // 2, _ACT[act], int(x.dtype == torch.float32),
+                                              _stream()), "act_mul_rows")
+        return out
     out = torch.empty(T, two_i // 2, dtype=x.dtype, device=x.device)
     _lib.check(_lib.lib().ogb_act_mul(_ptr(x), _ptr(out), T, two_i // 2, _ACT[act], _stream()), "act_mul")
     return out
@@ -372,23 +452,30 @@ def short_conv(bcx, weight, bias, cache, slots, positions, cu_seqlens, past_lens
 def causal_conv(x, weight, bias, cache, slots, positions, cu_seqlens, past_lens, block_table, block_size: int, silu: bool = True):
     """Causal depthwise convolution (no gates) of the recurrent layer kinds over packed sequences, with the window of earlier
     positions read from the paged `cache` [slots, C] that this step's rows are appended to; optional SiLU.  x [T, C] may be a
-    column slice of a wider tensor.  Returns [T, C] in x's dtype."""
-    if not x.is_cuda or x.dtype != torch.bfloat16 or x.stride(1) != 1 or (x.stride(0) % 8) or (x.data_ptr() % 16):
+    column slice of a wider tensor, `cache` a column range of wider rows.  Returns [T, C] in x's dtype."""
+    if not x.is_cuda:
         ones = torch.ones_like(x)
         y = short_conv(torch.cat([ones, ones, x], dim=1).contiguous(), weight, bias, cache, slots, positions, cu_seqlens, past_lens, block_table, block_size)
         return torch.nn.functional.silu(y.float()).to(x.dtype) if silu else y
     T, C = x.shape[0], weight.shape[0]
-    assert weight.is_contiguous() and cache.is_contiguous() and block_table.stride(1) == 1
+    assert weight.is_contiguous() and cache.stride(1) == 1 and block_table.stride(1) == 1 and x.stride(1) == 1
+    assert weight.dtype == x.dtype and cache.dtype == x.dtype
     out = torch.empty(T, C, dtype=x.dtype, device=x.device)
-    _lib.check(_lib.lib().ogb_causal_conv(_ptr(x), x.stride(0), _ptr(weight), _ptr(bias), _ptr(cache), _ptr(slots), _ptr(positions),
-                                         _ptr(cu_seqlens), _ptr(past_lens), _ptr(block_table), block_table.stride(0), int(block_size),
-                                         _ptr(out), T, past_lens.shape[0], C, weight.shape[1], int(silu), _stream()), "causal_conv")
+    args = (_ptr(slots), _ptr(positions), _ptr(cu_seqlens), _ptr(past_lens), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), T,
+            past_lens.shape[0], C, weight.shape[1])
+    if x.dtype == torch.float32 or C % 8 or x.stride(0) % 8 or cache.stride(0) % 8 or (x.data_ptr() | cache.data_ptr()) % 16 or weight.shape[1] > 16:
+        _lib.check(_lib.lib().ogb_causal_conv_rows(_ptr(x), x.stride(0), _ptr(weight), _ptr(bias), _ptr(cache), cache.stride(0), *args, int(silu),
+                                                  int(x.dtype == torch.float32), _stream()), "causal_conv_rows")
+        return out
+    _lib.check(_lib.lib().ogb_causal_conv(_ptr(x), x.stride(0), _ptr(weight), _ptr(bias), _ptr(cache), *args, cache.stride(0), int(silu), _stream()),
+               "causal_conv")
     return out
 
 
-def gated_delta(q, k, v, g, beta, state, slots, cu_seqlens, past_lens):
+def gated_delta(q, k, v, g, beta, state, slots, cu_seqlens, past_lens, max_q_len: int = 0):
     """Gated-delta-rule recurrence of a linear-attention layer over packed sequences (see ops/reference.py::gated_delta).
-    state [slots, Hv, dk, dv] fp32 is updated in place."""
+    state [slots, Hv, dk, dv] fp32 is updated in place.  max_q_len: most tokens of one request (1 selects the decode kernel, 0: not
+    known)."""
     if not q.is_cuda:
         return ref.gated_delta(q, k, v, g, beta, state, slots, cu_seqlens, past_lens)
     T, Hk, dk = q.shape
@@ -399,28 +486,33 @@ def gated_delta(q, k, v, g, beta, state, slots, cu_seqlens, past_lens):
     out = torch.empty(T, Hv, dv, dtype=torch.bfloat16, device=q.device)
     B = past_lens.shape[0]
     _lib.check(_lib.lib().ogb_gated_delta(_ptr(q), _ptr(k), _ptr(v), _ptr(gf), _ptr(bf), _ptr(state), _ptr(slots), _ptr(cu_seqlens), _ptr(past_lens),
-                                          _ptr(out), B, Hk, Hv, dk, dv, _stream()), "gated_delta")
+                                          _ptr(out), B, Hk, Hv, dk, dv, int(max_q_len), _stream()), "gated_delta")
     return out
 
 
-def gated_delta_layer(conv, proj, cd, vd, Hk, Hv, dk, dv, neg_exp_a, dt_bias, norm_w, norm_eps, state, slots, cu_seqlens, past_lens):
-    """The part of a gated-delta-net layer between its convolution and its output projection, as two kernels on bf16 CUDA tensors:
-    conv [T, cd] = silu(conv1d([q | k | v])), proj [T, cd + vd + 2 Hv] = the input projection [qkv | z | b | a].  q and k are
+def gated_delta_layer(conv, proj, cd, vd, Hk, Hv, dk, dv, neg_exp_a, dt_bias, norm_w, norm_eps, state, slots, cu_seqlens, past_lens,
+                      max_q_len: int = 0, l2_eps: float = 0.0, out=None):
+    """The part of a gated-delta-net layer between its convolution and its output projection, as two kernels on CUDA tensors (bf16 or
+    fp32): conv [T, cd] = silu(conv1d([q | k | v])), proj [T, cd + vd + 2 Hv] = the input projection [qkv | z | b | a].  q and k are
     L2-normalised per head (q also scaled by dk^-0.5), beta = sigmoid(b), log-decay = neg_exp_a * softplus(a + dt_bias), the
     recurrence updates `state` in place, and the result is RMS-normalised per value head, weighted and gated by silu(z).
-    Returns [T, Hv * dv]."""
+    l2_eps > 0: unit vectors are x / sqrt(sum(x^2) + l2_eps), else x / max(|x|, 1e-6).  state [slots, Hv * dk * dv (or more)]: a slot's
+    state is dense, slots may be further apart.  Returns [T, Hv * dv] (`out`: a matrix, or a column range, to write it to)."""
     T = conv.shape[0]
-    assert conv.is_cuda and conv.dtype == torch.bfloat16 and proj.dtype == torch.bfloat16 and conv.stride(1) == 1 and proj.stride(1) == 1
-    kd = Hk * dk
-    o = torch.empty(T, Hv, dv, dtype=torch.bfloat16, device=conv.device)
+    assert conv.is_cuda and conv.dtype == proj.dtype and conv.dtype in (torch.bfloat16, torch.float32) and conv.stride(1) == 1 and proj.stride(1) == 1
+    assert state.dtype == torch.float32 and state[0].numel() >= Hv * dk * dv and state[0].is_contiguous()
+    kd, f32 = Hk * dk, int(conv.dtype == torch.float32)
+    o = torch.empty(T, Hv, dv, dtype=conv.dtype, device=conv.device)
     B = past_lens.shape[0]
     _lib.check(_lib.lib().ogb_gated_delta_fused(_ptr(conv), conv.stride(0), 0, kd, 2 * kd, _ptr(proj), proj.stride(0), cd + vd, cd + vd + Hv,
-                                                _ptr(neg_exp_a), _ptr(dt_bias), float(dk) ** -0.5, _ptr(state), _ptr(slots), _ptr(cu_seqlens),
-                                                _ptr(past_lens), _ptr(o), B, Hk, Hv, dk, dv, _stream()), "gated_delta_fused")
-    out = torch.empty(T, Hv * dv, dtype=torch.bfloat16, device=conv.device)
+                                                _ptr(neg_exp_a), _ptr(dt_bias), float(dk) ** -0.5, float(l2_eps), _ptr(state), state.stride(0),
+                                                _ptr(slots), _ptr(cu_seqlens), _ptr(past_lens), _ptr(o), B, Hk, Hv, dk, dv, int(max_q_len), f32,
+                                                _stream()), "gated_delta_fused")
+    if out is None:
+        out = torch.empty(T, Hv * dv, dtype=conv.dtype, device=conv.device)
     z = proj[:, cd:cd + vd]
-    _lib.check(_lib.lib().ogb_gdn_gate_norm(_ptr(o), _ptr(z), proj.stride(0), _ptr(norm_w), float(norm_eps), _ptr(out), T, Hv, dv, _stream()),
-               "gdn_gate_norm")
+    _lib.check(_lib.lib().ogb_gdn_gate_norm(_ptr(o), _ptr(z), proj.stride(0), _ptr(norm_w), float(norm_eps), _ptr(out), out.stride(0), T, Hv, dv, f32,
+                                            _stream()), "gdn_gate_norm")
     return out
 
 
@@ -733,6 +825,124 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
     _lib.check(rc, "paged_attention")
     if splits > 1:
         _lib.LAUNCH_COUNT += 1  # the combine kernel
+    return out
+
+
+# ------------------------------------------------------------------------------------------ latent attention
+LATENT_LONG_TOKENS = 64      # requests that feed at least this many tokens attend on expanded keys and values (tensor-memory kernel)
+
+
+def latent_shape(heads, dim, rot, vdim, kv_rank, rot_dims):
+    return _lib.LatentShape(H=heads, dim=dim, rot=rot, vdim=vdim, R=kv_rank, rot_dims=rot_dims)
+
+
+def _sh(shape):
+    import ctypes
+    return ctypes.byref(shape)
+
+
+def latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache):
+    """In place: rotates the rotary part of every query head of proj ([H heads of (dim | rot)] then [latent | shared rotary key]), and
+    writes the RMS-normalised latent and the rotated key of each token to its row of `cache` [slots, >= kv_rank + rot] (slot < 0: to no
+    row).  cos / sin [positions, rot_dims / 2] fp32, or None for a layer that does not rotate."""
+    _check_index("latent_prep", "slots", slots[:proj.shape[0]], cache.shape[0], -1)
+    if cos is not None:
+        _check_index("latent_prep", "positions", positions[:proj.shape[0]], cos.shape[0])
+    if not proj.is_cuda:
+        return ref.latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache)
+    assert proj.stride(1) == 1 and cache.stride(1) == 1 and cache.dtype == proj.dtype and norm_w.dtype == torch.float32
+    _lib.check(_lib.lib().ogb_latent_prep(_ptr(proj), proj.stride(0), _sh(shape), _ptr(norm_w), float(eps), _ptr(positions), _ptr(cos), _ptr(sin),
+                                         cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(cache), cache.stride(0), proj.shape[0],
+                                         int(proj.dtype == torch.float32), _stream()), "latent_prep")
+    return proj
+
+
+def choose_latent_splits(batch: int, row_tiles: int, max_kv_len: int, window: int, sm_count: int = 148) -> int:
+    """Key splits of a latent-attention launch: about one CTA per SM, each with at least two tiles of 64 keys."""
+    span = max_kv_len if window <= 0 else min(max_kv_len, window + 64)
+    return max(1, min(sm_count // max(1, batch * row_tiles), span // 128, 32))
+
+
+def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0, max_q_len=1, max_kv_len=1,
+                     skip_q_len=0, splits=None):
+    """Attention of every head over the shared latent rows: qlat [T, H * kv_rank] (queries with the key map folded in), the rotated
+    query parts in proj.  window > 0: position p sees (p - window, p].  skip_q_len > 0: requests with at least that many tokens are
+    not computed (their rows are unspecified).  Returns [T, H * kv_rank]."""
+    _check_index("latent_attention", "block_table", block_table, cache.shape[0] // block_size, -1)
+    if not qlat.is_cuda:
+        return ref.latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window)
+    T, B, H, R = qlat.shape[0], past_lens.shape[0], shape.H, shape.R
+    out = torch.empty_like(qlat)
+    L = _lib.lib()
+    f32 = qlat.dtype == torch.float32
+    if (f32 or not L.ogb_latent_mma_supported(_sh(shape)) or proj.stride(0) % 8 or cache.stride(0) % 8 or
+            (qlat.data_ptr() | proj.data_ptr() | cache.data_ptr()) % 16):
+        _lib.check(L.ogb_latent_attention_simt(_ptr(qlat), _ptr(proj), proj.stride(0), _sh(shape), _ptr(cache), cache.stride(0), _ptr(cu_seqlens),
+                                               _ptr(past_lens), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale),
+                                               int(window), B, T, int(skip_q_len), int(f32), _stream()), "latent_attention_simt")
+        return out
+    q_len = min(max_q_len, skip_q_len - 1) if skip_q_len > 0 else max_q_len
+    if splits is None:
+        bm = L.ogb_latent_rows_per_tile(H, q_len)
+        splits = choose_latent_splits(B, -(-H * q_len // bm), max_kv_len, window)
+    need = L.ogb_latent_scratch_bytes(T * H, R, splits)
+    scratch = workspace(qlat.device).attn_scratch(need) if splits > 1 else None
+    _lib.check(L.ogb_latent_attention(_ptr(qlat), _ptr(proj), proj.stride(0), _sh(shape), _ptr(cache), cache.stride(0), _ptr(cu_seqlens), _ptr(past_lens),
+                                      _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale), int(window), B, T,
+                                      int(max_q_len), int(skip_q_len), int(splits), _ptr(scratch), scratch.numel() if scratch is not None else 0,
+                                      _stream()), "latent_attention")
+    if splits > 1:
+        _lib.LAUNCH_COUNT += 1      # the combine kernel
+    return out
+
+
+def latent_long_supported(shape, proj, cache, block_size: int) -> bool:
+    return (proj.is_cuda and proj.dtype == torch.bfloat16 and bool(_lib.lib().ogb_attention_tc_latent_supported(shape.dim, shape.rot, shape.vdim)) and
+            shape.R % 8 == 0 and proj.stride(0) % 8 == 0 and cache.stride(0) % 8 == 0)
+
+
+class LatentPlan:
+    """Where the long requests of a step put their expanded keys: per request a run of dense rows (a multiple of 16) for the cached
+    positions its tokens can see."""
+    __slots__ = ("rows", "row_base", "first_kv", "g_base", "g_first", "g_len", "g_req", "n_req", "max_q_len")
+
+    def __init__(self, lens, window: int, device, min_tokens: int = LATENT_LONG_TOKENS):
+        B = len(lens)
+        base, first = np.full(B, -1, dtype=np.int32), np.zeros(B, dtype=np.int32)
+        compact, rows, self.max_q_len = [], 0, 0
+        for b, (past, n) in enumerate(lens):
+            if n < min_tokens:
+                continue
+            lo = max(0, past - window + 1) // 16 * 16 if window > 0 else 0
+            base[b], first[b] = rows, lo
+            compact.append((rows, lo, past + n, b))
+            rows += (past + n - lo + 15) // 16 * 16
+            self.max_q_len = max(self.max_q_len, n)
+        self.rows, self.n_req = rows, len(compact)
+        if rows == 0:
+            return
+        flat = np.concatenate([base, first, np.asarray(compact, dtype=np.int32).T.reshape(-1)]).astype(np.int32)
+        host = torch.from_numpy(flat)
+        dev = host.pin_memory().to(device, non_blocking=True) if torch.device(device).type == "cuda" else host
+        k = self.n_req
+        self.row_base, self.first_kv = dev[:B], dev[B:2 * B]
+        self.g_base, self.g_first, self.g_len, self.g_req = (dev[2 * B + i * k:2 * B + (i + 1) * k] for i in range(4))
+
+
+def latent_attention_long(proj, shape, w_ukv, cache, plan: LatentPlan, cu_seqlens, past_lens, block_table, block_size, scale, window, out):
+    """The long requests of a step (plan): their visible latents are gathered, expanded to per-head keys and values by one product with
+    w_ukv [H * (dim + vdim), kv_rank], and attended on the tensor cores.  Writes the requests' rows of out [T, >= H * vdim]."""
+    L = _lib.lib()
+    width = shape.R + shape.rot
+    lat = torch.empty(plan.rows, width, dtype=torch.bfloat16, device=proj.device)
+    _lib.check(L.ogb_latent_gather(_ptr(cache), cache.stride(0), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(plan.g_base),
+                                   _ptr(plan.g_first), _ptr(plan.g_len), _ptr(plan.g_req), plan.n_req, plan.rows, width, _ptr(lat), width, _stream()),
+               "latent_gather")
+    kv = linear(lat[:, :shape.R], w_ukv)
+    _lib.check(L.ogb_attention_tc_latent(_ptr(proj), proj.stride(0), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), shape.R, plan.rows,
+                                         _ptr(cu_seqlens), _ptr(past_lens), _ptr(plan.row_base), _ptr(plan.first_kv), _ptr(out), out.stride(0),
+                                         float(scale), int(window), past_lens.shape[0], plan.max_q_len, shape.H, shape.dim, shape.rot, shape.vdim,
+                                         workspace(proj.device).status, _stream()), "attention_tc_latent")
     return out
 
 

@@ -24,6 +24,13 @@ class GemmFused(ctypes.Structure):
                 ("Hq", c_int), ("Hkv", c_int), ("D", c_int), ("rot", c_int), ("max_pos", c_int)]
 
 
+class LatentShape(ctypes.Structure):
+    """OgbLatentShape of csrc/kernels.h: sizes of a latent-attention layer."""
+    _fields_ = [(n, c_int) for n in ("H", "dim", "rot", "vdim", "R", "rot_dims")]
+
+
+_LS = ctypes.POINTER(LatentShape)
+
 _SIGS = {
     "ogb_runtime_init": (c_int, [c_int]),
     "ogb_status_device_ptr": (_P, [c_int]),
@@ -63,7 +70,24 @@ _SIGS = {
     "ogb_embedding_q4": (c_int, [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, _P]),
     "ogb_act_mul": (c_int, [_P, _P, c_int, c_int, c_int, _P]),
     "ogb_act": (c_int, [_P, _P, c_longlong, c_int, _P]),
-    "ogb_causal_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_causal_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_causal_conv_rows": (c_int, [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P]),
+    "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_int, _P]),
+    "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, c_int, c_int, c_int, c_float, _P]),
+    "ogb_norm_stream": (c_int, [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P]),
+    "ogb_act_mul_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_latent_prep": (c_int, [_P, c_int, _LS, _P, c_float, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P]),
+    "ogb_latent_mma_supported": (c_int, [_LS]),
+    "ogb_latent_rows_per_tile": (c_int, [c_int, c_int]),
+    "ogb_latent_scratch_bytes": (c_longlong, [c_int, c_int, c_int]),
+    "ogb_latent_attention": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
+                                     _P, c_longlong, _P]),
+    "ogb_latent_attention_simt": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_latent_gather": (c_int, [_P, c_int, _P, c_int, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P, c_int, _P]),
+    "ogb_attention_tc_latent_supported": (c_int, [c_int, c_int, c_int]),
+    "ogb_attention_tc_latent": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_float, c_int, c_int, c_int, c_int,
+                                        c_int, c_int, c_int, _P, _P]),
     "ogb_short_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P]),
     "ogb_decode_advance": (c_int, [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
     "ogb_logits_edit": (c_int, [_P, c_int, _P, _P, _P, _P, c_int, _P]),
@@ -82,9 +106,9 @@ _SIGS = {
     "ogb_paged_attention_kv8": (c_int, [_P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P, c_float, c_float, c_int, c_int,
                                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, c_int, _P, _P, _P]),
     "ogb_gated_delta_fused": (c_int, [_P, c_longlong, c_longlong, c_longlong, c_longlong, _P, c_longlong, c_longlong, c_longlong, _P, _P, c_float,
-                                      _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),
-    "ogb_gdn_gate_norm": (c_int, [_P, _P, c_longlong, _P, c_float, _P, c_int, c_int, c_int, _P]),
-    "ogb_gated_delta": (c_int, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),
+                                      c_float, _P, c_longlong, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_gdn_gate_norm": (c_int, [_P, _P, c_longlong, _P, c_float, _P, c_longlong, c_int, c_int, c_int, c_int, _P]),
+    "ogb_gated_delta": (c_int, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_mamba2_scan_fused": (c_int, [_P, c_longlong, _P, c_longlong, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_mamba_gate_norm": (c_int, [_P, _P, c_longlong, _P, c_float, _P, c_int, c_int, _P]),
     "ogb_mamba2_scan": (c_int, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),

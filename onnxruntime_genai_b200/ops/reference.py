@@ -54,6 +54,16 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, norm_eps=0.0):
     return y if out_fp32 else y.to(x.dtype)
 
 
+def _act(g, act):
+    if act == "silu":
+        return torch.nn.functional.silu(g)
+    if act == "relu":
+        return torch.relu(g)
+    if act == "relu2":
+        return torch.relu(g) ** 2
+    return torch.nn.functional.gelu(g, approximate="none" if act == "gelu_erf" else "tanh")
+
+
 def gate_up_act(x, w, bias=None, act="silu", interleaved=False, norm_eps=0.0):
     """w is the stacked [gate; up] weight of shape [2I, K] (or 64-row interleaved blocks)."""
     if norm_eps > 0:
@@ -65,15 +75,13 @@ def gate_up_act(x, w, bias=None, act="silu", interleaved=False, norm_eps=0.0):
     if interleaved:
         y = y.view(-1, inter // 64, 2, 64).transpose(1, 2).reshape(-1, 2 * inter)
     g, u = y[..., :inter], y[..., inter:]
-    a = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
-    return (a * u).to(x.dtype)
+    return (_act(g, act) * u).to(x.dtype)
 
 
 def act_mul(x, act="silu"):
     inter = x.shape[-1] // 2
     g, u = x[..., :inter].float(), x[..., inter:].float()
-    a = torch.nn.functional.silu(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
-    return (a * u).to(x.dtype)
+    return (_act(g, act) * u).to(x.dtype)
 
 
 def activation(x, act="gelu"):
@@ -374,3 +382,45 @@ def mamba2_scan(x, dt, neg_a, Bm, Cm, Dv, state, slots, cu_seqlens, past_lens):
         state[slot] = S.to(state.dtype)
     return out.to(x.dtype)
 
+
+
+def head_project(x, w, heads, a_cols):
+    """out[:, h * N + n] = sum_k x[:, h * a_cols + k] * w[h * N + n, k]."""
+    N, K = w.shape[0] // heads, w.shape[1]
+    return torch.cat([x[:, h * a_cols:h * a_cols + K].float() @ w[h * N:(h + 1) * N].float().t() for h in range(heads)], 1).to(x.dtype)
+
+
+def latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache):
+    T, H, d, r, R = proj.shape[0], shape.H, shape.dim, shape.rot, shape.R
+    q, down = proj[:, :H * (d + r)].view(T, H, d + r), proj[:, H * (d + r):H * (d + r) + R + r]
+    c = down[:, :R].float()
+    c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * norm_w.float()
+    kr, qr = down[:, None, R:].float(), q[:, :, d:].float()
+    if cos is not None and shape.rot_dims:
+        pos = positions.long().clamp(0, cos.shape[0] - 1)
+        kr, qr = (_rotate(t, cos[pos], sin[pos], shape.rot_dims, False) for t in (kr, qr))
+    q[:, :, d:] = qr.to(proj.dtype)
+    ok = slots >= 0
+    cache[slots[ok].long(), :R + r] = torch.cat([c, kr[:, 0]], 1)[ok].to(cache.dtype)
+    return proj
+
+
+def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0):
+    T, H, d, r, R = qlat.shape[0], shape.H, shape.dim, shape.rot, shape.R
+    out = torch.zeros_like(qlat)
+    q = torch.cat([qlat.view(T, H, R).float(), proj[:, :H * (d + r)].view(T, H, d + r)[:, :, d:].float()], -1)
+    cu = cu_seqlens.tolist()
+    for b in range(past_lens.shape[0]):
+        t0, t1, past = cu[b], cu[b + 1], int(past_lens[b])
+        if t0 == t1:
+            continue
+        pos = torch.arange(past + t1 - t0, device=qlat.device)
+        rows = cache[block_table[b, pos // block_size].long() * block_size + pos % block_size, :R + r].float()
+        s = torch.einsum("qhd,kd->hqk", q[t0:t1], rows) * scale
+        qpos = past + torch.arange(t1 - t0, device=qlat.device)
+        vis = pos[None] <= qpos[:, None]
+        if window and window > 0:
+            vis = vis & (pos[None] > qpos[:, None] - window)
+        p = torch.softmax(s.masked_fill(~vis[None], float("-inf")), -1)
+        out[t0:t1] = torch.einsum("hqk,kd->qhd", p, rows[:, :R]).reshape(t1 - t0, H * R).to(out.dtype)
+    return out

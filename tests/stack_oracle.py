@@ -1,0 +1,147 @@
+"""A slow, plain restatement of declared-stack decoders (gated-delta and latent-attention mixers in parallel blocks), one function
+per mechanism, token by token where the mechanism is a recurrence.  It shares no code with the package: the tests compare the
+runtime against it.  Weights come as a dictionary of tensors under the checkpoint's names; all math runs in `dtype` (float64 by
+default).  A whole sequence is evaluated at once, from its first token: there is no cache here."""
+import math
+
+import torch
+
+
+# ------------------------------------------------------------------------------------------------ mechanisms
+def layer_norm(x, w, b, eps):
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w + b
+
+
+def rms_norm(x, w, eps):
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+
+
+def causal_conv_silu(x, taps):
+    """x [T, C], taps [C, K]: the newest position meets the last column."""
+    T, K = x.shape[0], taps.shape[1]
+    y = torch.zeros_like(x)
+    for t in range(T):
+        for k in range(K):
+            if t - k >= 0:
+                y[t] = y[t] + taps[:, K - 1 - k] * x[t - k]
+    return y * torch.sigmoid(y)
+
+
+def unit_vectors(x):
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def delta_recurrence(q, k, v, g, beta):
+    """q, k [T, Hk, dk] (prepared), v [T, H, dv], decay g and strength beta [T, H] -> [T, H, dv]."""
+    T, H, dv = v.shape
+    rep = H // q.shape[1]
+    S = torch.zeros(H, q.shape[2], dv, dtype=v.dtype)
+    out = torch.zeros_like(v)
+    for t in range(T):
+        for h in range(H):
+            kk, qq = k[t, h // rep], q[t, h // rep]
+            S[h] = S[h] * g[t, h]
+            u = beta[t, h] * (v[t, h] - kk @ S[h])
+            S[h] = S[h] + torch.outer(kk, u)
+            out[t, h] = qq @ S[h]
+    return out
+
+
+def delta_mixer(x, w, p, m, eps):
+    """x [T, width]; w: weights, p: prefix of the layer's mixer tensors, m: the mixer's sizes."""
+    T, H, Hk, dk, dv = x.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = causal_conv_silu(x @ w[p + "q"].T, w[p + "q.conv"]).view(T, Hk, dk)
+    k = causal_conv_silu(x @ w[p + "k"].T, w[p + "k.conv"]).view(T, Hk, dk)
+    v = causal_conv_silu(x @ w[p + "v"].T, w[p + "v.conv"]).view(T, H, dv)
+    q, k = unit_vectors(q) * dk ** -0.5, unit_vectors(k)
+    beta = torch.sigmoid(x @ w[p + "b"].T)
+    step = torch.log1p(torch.exp(-(x @ w[p + "a"].T + w[p + "dt_bias"]).abs())) + (x @ w[p + "a"].T + w[p + "dt_bias"]).clamp(min=0)
+    g = torch.exp(-torch.exp(w[p + "A_log"]) * step)
+    o = delta_recurrence(q, k, v, g, beta)
+    z = (x @ w[p + "g"].T).view(T, H, dv)
+    o = rms_norm(o, w[p + "norm"], eps) * (z * torch.sigmoid(z))
+    return o.reshape(T, H * dv) @ w[p + "o"].T
+
+
+def rotary_frequencies(rot):
+    """(frequency of every pair, factor on cos and sin)."""
+    d, base = rot["dims"], rot["base"]
+    f = [base ** (-2.0 * i / d) for i in range(d // 2)]
+    s = rot.get("scaling")
+    if not s:
+        return f, 1.0
+
+    def turns(t):
+        return d * math.log(s["original"] / (2 * math.pi * t)) / (2 * math.log(base))
+    lo, hi = max(math.floor(turns(s["fast"])), 0), min(math.ceil(turns(s["slow"])), d - 1)
+    out = []
+    for i, fi in enumerate(f):
+        r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(fi / s["factor"] * r + fi * (1 - r))
+    return out, 0.1 * math.log(s["factor"]) + 1.0
+
+
+def rotate(x, rot):
+    """x [T, heads, >= dims]: pairs (i, i + dims / 2) of the first dims entries turn with the position."""
+    if not rot:
+        return x
+    f, amp = rotary_frequencies(rot)
+    half = rot["dims"] // 2
+    y = x.clone()
+    for t in range(x.shape[0]):
+        for i in range(half):
+            c, s = math.cos(t * f[i]) * amp, math.sin(t * f[i]) * amp
+            u, v = x[t, :, i], x[t, :, i + half]
+            y[t, :, i], y[t, :, i + half] = u * c - v * s, v * c + u * s
+    return y
+
+
+def visible(T, mask):
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None]
+    ok = j <= i
+    if mask:
+        ok = ok & (i - j < mask["size"])
+    return ok
+
+
+def latent_mixer(x, w, p, m, eps):
+    T, H, d, r, dv, R = x.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    q = (x @ w[p + "q"].T).view(T, H, d + r)
+    down = x @ w[p + "dkv"].T
+    c = rms_norm(down[:, :R], w[p + "dkv.norm"], eps)
+    kr = rotate(down[:, R:].view(T, 1, r), m.get("rot"))[:, 0]
+    qr = rotate(q[:, :, d:], m.get("rot"))
+    kn = (c @ w[p + "uk"].T).view(T, H, d)
+    v = (c @ w[p + "uv"].T).view(T, H, dv)
+    ok = visible(T, m.get("mask"))
+    out = torch.zeros(T, H, dv, dtype=x.dtype)
+    for h in range(H):
+        s = (q[:, h, :d] @ kn[:, h].T + qr[:, h] @ kr.T) * m["scale"]
+        out[:, h] = torch.softmax(s.masked_fill(~ok, -math.inf), -1) @ v[:, h]
+    return out.reshape(T, H * dv) @ w[p + "o"].T
+
+
+def feed_forward(x, w, p):
+    return (torch.relu(x @ w[p + "gate"].T) * (x @ w[p + "up"].T)) @ w[p + "down"].T
+
+
+# ------------------------------------------------------------------------------------------------ the stack
+MIXERS = {"delta": delta_mixer, "latent_attention": latent_mixer}
+
+
+def stack_forward(cfg, weights, tokens, dtype=torch.float64):
+    """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
+    w = {k: v.to(dtype) for k, v in weights.items()}
+    eps = cfg["norm"]["eps"]
+    x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+    streams = []
+    for i, e in enumerate(cfg["layers"]):
+        p = f"l{e.get('weights_of', i) if e.get('weights_of') is not None else i}."
+        h = layer_norm(x, w[p + "norm1"], w[p + "norm1.b"], eps)
+        y = MIXERS[e["type"]](h, w, p + "mix.", e["mixer"], eps)
+        if e.get("mlp"):
+            y = y + feed_forward(h, w, p + "mlp.")
+        x = x + y
+        streams.append(x)
+    return layer_norm(x, w["final.norm"], w["final.norm.b"], eps) @ w["head"].T, torch.stack(streams)
