@@ -4,7 +4,9 @@
 
 cases: gemm_qkv gemm_o gemm_gate_up gemm_down gemm_lm_head gemm_prefill gemm_qkv_fused gemm_gate_up_fused w4_qkv w4_down attention_decode
        attention_prefill norm rope sample argmax all; moe_fp4_gate_up moe_fp4_down moe_fp4b_gate_up moe_fp4b_down moe_bf16_gate_up moe_bf16_down
-       (gpt-oss-20b experts, packed MXFP4 in the fp16 form, in the bf16 form (fp4b) or bf16 weights; not part of `all`)
+       gated_delta gated_delta_prefill mamba2_scan; latent_decode latent_absorb latent_value latent_prep latent_prefill latent_expand norm_stream
+       gemm_join (Luzatar layers at Llama-sized widths: 16 heads of 128 + 64 / 128 over a latent of 512; not part of `all`)
+       (moe_*: gpt-oss-20b experts, packed MXFP4 in the fp16 form, in the bf16 form (fp4b) or bf16 weights; not part of `all`)
 
 Each case runs the kernel at the Llama-3.1-8B (or, for w4_*, Phi-3-mini) shapes with `--layers` distinct
 weight sets rotated between launches (so weights come from HBM, not L2), captures `--iters` launches
@@ -107,7 +109,7 @@ def build_case(name, T, L, tp=1):
         kc, vc = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D)
         return (lambda i: ops.qkv_rope_append(x, ws[i % L], None, pos, slots, cos, sin, kc, vc, HQ, HKV, D, D, norm_eps=1e-5)), \
             N * H * 2 + T * (H + N) * 2, 2.0 * T * N * H
-    if name.startswith("gemm_") or name.startswith("w4_"):
+    if name != "gemm_join" and name.startswith(("gemm_", "w4_")):
         shapes = {"gemm_qkv": ((HQ + 2 * HKV) * D, H), "gemm_o": (H, HQ * D), "gemm_gate_up": (2 * I // tp, H), "gemm_down": (H, I // tp),
                   "gemm_lm_head": (V // tp, H), "gemm_prefill": (2 * I // tp, H), "w4_qkv": (9216 // tp, 3072), "w4_down": (3072, 8192 // tp)}
         N, K = shapes[name]
@@ -195,6 +197,68 @@ def build_case(name, T, L, tp=1):
         return (lambda i: ops.paged_attention(qkv, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ, HKV, D, 1 / math.sqrt(D),
                                               max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)),
                                               splits=ATTN_SPLITS, order=order)), nbytes, flops
+    if name.startswith("latent_"):
+        Hl, d, r, dv, R, bs = 16, 128, 64, 128, 512, 16
+        sh = ops.latent_shape(Hl, d, r, dv, R, r)
+        N, Lk = Hl * (d + r) + R + r, min(L, 8)
+        prefill = name in ("latent_prefill", "latent_expand")
+        if name == "latent_absorb":
+            x, ws = _bf(T, N, std=1.0), [_bf(Hl * R, d) for _ in range(L)]
+            return (lambda i: ops.head_project(x, ws[i % L], Hl, d + r)), Hl * R * d * 2 + T * Hl * (d + R) * 2, 2.0 * T * Hl * d * R
+        if name == "latent_value":
+            x, ws = _bf(T, Hl * R, std=1.0), [_bf(Hl * dv, R) for _ in range(L)]
+            return (lambda i: ops.head_project(x, ws[i % L], Hl, R)), Hl * R * dv * 2 + T * Hl * (dv + R) * 2, 2.0 * T * Hl * dv * R
+        rng = np.random.RandomState(2)
+        lens = [(0, 1024)] * (T // 1024) if prefill else [(int(p) + 64, 1) for p in rng.randint(128, 2049, size=T)]
+        if prefill and T <= 4096:
+            lens = [(0, T)]
+        nb = [(p + n + bs - 1) // bs for p, n in lens]
+        table = torch.zeros(len(lens), max(nb), dtype=torch.int32)
+        for b, k in enumerate(nb):
+            table[b, :k] = torch.arange(sum(nb[:b]), sum(nb[:b]) + k, dtype=torch.int32)
+        table = table.cuda()
+        caches = [_bf(sum(nb) * bs, R + r, std=1.0) for _ in range(Lk)]
+        Tq = sum(n for _, n in lens)
+        proj = _bf(Tq, N, std=1.0)
+        cu = torch.tensor(np.concatenate([[0], np.cumsum([n for _, n in lens])]), dtype=torch.int32).cuda()
+        pl = torch.tensor([p for p, _ in lens], dtype=torch.int32).cuda()
+        scale = 1 / math.sqrt(d + r)
+        if name == "latent_prep":
+            pos, slots = pl.clone(), (table[:, 0] * bs).contiguous()
+            cos, sin, w = torch.randn(4096, r // 2, device="cuda"), torch.randn(4096, r // 2, device="cuda"), torch.ones(R, device="cuda")
+            return (lambda i: ops.latent_prep(proj, sh, w, 1e-6, pos, cos, sin, slots, caches[i % Lk])), T * (Hl * r * 4 + (R + r) * 4), 0.0
+        if prefill:
+            w = _bf(Hl * (d + dv), R)
+            plan = ops.LatentPlan(lens, 0, "cuda")
+            if name == "latent_expand":
+                return (lambda i: ops.latent_expand(sh, w, caches[i % Lk], plan, table, bs)), plan.rows * ((R + r) * 6 + Hl * (d + dv) * 2), \
+                    2.0 * plan.rows * R * Hl * (d + dv)
+            lat, kv = ops.latent_expand(sh, w, caches[0], plan, table, bs)
+            out = torch.empty(Tq, Hl * dv, dtype=torch.bfloat16, device="cuda")
+            return (lambda i: ops.latent_attend_expanded(proj, sh, lat, kv, plan, cu, pl, scale, 0, out)), \
+                plan.rows * Hl * (d + dv) * 2 + Tq * Hl * (d + r + dv) * 2, sum(2.0 * Hl * (d + r + dv) * n * (n + 1) / 2 for _, n in lens)
+        qlat = _bf(Tq, Hl * R, std=0.3)
+        kv_tokens = sum(p + n for p, n in lens)
+        return (lambda i: ops.latent_attention(qlat, proj, sh, caches[i % Lk], cu, pl, table, bs, scale, 0, 1, max(p + n for p, n in lens),
+                                               splits=ATTN_SPLITS[0] if isinstance(ATTN_SPLITS, tuple) else ATTN_SPLITS)), \
+            kv_tokens * (R + r) * 2 + Tq * Hl * (2 * R + r) * 2, 2.0 * kv_tokens * Hl * (2 * R + r)
+    if name == "norm_stream":
+        xs, w, b = [torch.randn(T, H, device="cuda") for _ in range(8)], torch.randn(H, device="cuda"), torch.randn(H, device="cuda")
+        return (lambda i: ops.norm_stream(xs[i % 8], w, 1e-5, b, True)), T * H * 6, 0.0
+    if name == "gemm_join":
+        K = 2048 + I
+        x, ws, h = _bf(T, K, std=1.0), [_bf(H, K) for _ in range(L)], torch.zeros(T, H, device="cuda")
+        return (lambda i: ops.linear(x, ws[i % L], residual=h, out=h, out_fp32=True)), H * K * 2 + T * K * 2 + T * H * 8, 2.0 * T * H * K
+    if name == "gated_delta_prefill":
+        # prompts of 1024 tokens (one prompt below 4096 tokens) through one gated-delta-net layer, Qwen3.5 shapes
+        Hk, Hv, dk, dv = 16, 32, 128, 128
+        B = T // 1024 if T > 4096 else 1
+        q, k, v = _bf(T, Hk, dk, std=0.1), _bf(T, Hk, dk, std=0.1), _bf(T, Hv, dv, std=1.0)
+        g, beta = -torch.rand(T, Hv, device="cuda") * 0.2, torch.rand(T, Hv, device="cuda")
+        pool = torch.zeros(B, Hv, dk, dv, device="cuda")
+        slots, past = torch.arange(B, dtype=torch.int32, device="cuda"), torch.zeros(B, dtype=torch.int32, device="cuda")
+        cu = torch.arange(0, T + 1, T // B, dtype=torch.int32, device="cuda")
+        return (lambda i: ops.gated_delta(q, k, v, g, beta, pool, slots, cu, past, max_q_len=T // B)), T * (2 * Hk * dk + 2 * Hv * dv) * 2, 6.0 * T * Hv * dk * dv
     if name == "norm":
         x, r, w = _bf(T, H, std=1.0), _bf(T, H, std=1.0), _bf(H, std=1.0)
         return (lambda i: ops.norm(x, w, 1e-5, r)), T * H * 2 * 4, 0.0
@@ -216,7 +280,7 @@ def build_case(name, T, L, tp=1):
         slots = torch.arange(T, dtype=torch.int32, device="cuda")
         cu = torch.arange(T + 1, dtype=torch.int32, device="cuda")
         past = torch.full((T,), 7, dtype=torch.int32, device="cuda")
-        return (lambda i: ops.gated_delta(q, k, v, g, beta, pools[i % len(pools)], slots, cu, past)), \
+        return (lambda i: ops.gated_delta(q, k, v, g, beta, pools[i % len(pools)], slots, cu, past, max_q_len=1)), \
             T * Hv * dk * dv * 4 * 2 + T * (2 * Hk * dk + 2 * Hv * dv) * 2, 6.0 * T * Hv * dk * dv
     if name == "mamba2_scan":
         # one decode step of a Mamba-2 layer for T requests (heads 128, head size 64, state size 128, one B / C group): every request's
@@ -280,7 +344,7 @@ def main():
     hbm, tflops, src = _peaks()
     out = {}
     for name in (ALL if a.case == "all" else [a.case]):
-        T = a.tokens if name != "gemm_prefill" and name != "attention_prefill" else max(a.tokens, 2048)
+        T = max(a.tokens, 2048) if name in ("gemm_prefill", "attention_prefill", "latent_prefill", "latent_expand", "gated_delta_prefill") else a.tokens
         fn, nbytes, flops = build_case(name, T, a.layers, a.tp)
         iters = a.iters if name not in ("gemm_lm_head", "sample", "argmax") else min(a.iters, 4)
         us = _time_eager(fn, iters) if a.eager else _time_graph(fn, iters)

@@ -604,7 +604,8 @@ class SequenceState:
             self._tbl = self.block_table.cpu().numpy().copy()
         self._tbl = self._tbl[np.asarray(src_rows, dtype=np.int64)].copy()
         if self.kv.state is not None:       # recurrent states follow their hypotheses
-            self.kv.state = self.kv.state[:, torch.as_tensor(src_rows, dtype=torch.long, device=self.kv.state.device)].contiguous()
+            # in place: captured decode steps hold the pool's address
+            self.kv.state.copy_(self.kv.state[:, torch.as_tensor(src_rows, dtype=torch.long, device=self.kv.state.device)])
         self.kv_len = [self.kv_len[s] for s in src_rows]
         self._recount()
         self._tbl_dirty = True

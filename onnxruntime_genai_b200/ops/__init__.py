@@ -929,21 +929,31 @@ class LatentPlan:
         self.g_base, self.g_first, self.g_len, self.g_req = (dev[2 * B + i * k:2 * B + (i + 1) * k] for i in range(4))
 
 
-def latent_attention_long(proj, shape, w_ukv, cache, plan: LatentPlan, cu_seqlens, past_lens, block_table, block_size, scale, window, out):
-    """The long requests of a step (plan): their visible latents are gathered, expanded to per-head keys and values by one product with
-    w_ukv [H * (dim + vdim), kv_rank], and attended on the tensor cores.  Writes the requests' rows of out [T, >= H * vdim]."""
-    L = _lib.lib()
+def latent_expand(shape, w_ukv, cache, plan: LatentPlan, block_table, block_size):
+    """The cached rows the plan's requests can see as a dense matrix [rows, kv_rank + rot], and their per-head keys and values by one
+    product with w_ukv [H * (dim + vdim), kv_rank]."""
     width = shape.R + shape.rot
-    lat = torch.empty(plan.rows, width, dtype=torch.bfloat16, device=proj.device)
-    _lib.check(L.ogb_latent_gather(_ptr(cache), cache.stride(0), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(plan.g_base),
-                                   _ptr(plan.g_first), _ptr(plan.g_len), _ptr(plan.g_req), plan.n_req, plan.rows, width, _ptr(lat), width, _stream()),
-               "latent_gather")
-    kv = linear(lat[:, :shape.R], w_ukv)
-    _lib.check(L.ogb_attention_tc_latent(_ptr(proj), proj.stride(0), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), shape.R, plan.rows,
-                                         _ptr(cu_seqlens), _ptr(past_lens), _ptr(plan.row_base), _ptr(plan.first_kv), _ptr(out), out.stride(0),
-                                         float(scale), int(window), past_lens.shape[0], plan.max_q_len, shape.H, shape.dim, shape.rot, shape.vdim,
-                                         workspace(proj.device).status, _stream()), "attention_tc_latent")
+    lat = torch.empty(plan.rows, width, dtype=torch.bfloat16, device=cache.device)
+    _lib.check(_lib.lib().ogb_latent_gather(_ptr(cache), cache.stride(0), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(plan.g_base),
+                                           _ptr(plan.g_first), _ptr(plan.g_len), _ptr(plan.g_req), plan.n_req, plan.rows, width, _ptr(lat), width,
+                                           _stream()), "latent_gather")
+    return lat, linear(lat[:, :shape.R], w_ukv)
+
+
+def latent_attend_expanded(proj, shape, lat, kv, plan: LatentPlan, cu_seqlens, past_lens, scale, window, out):
+    """Tensor-memory attention of the plan's requests on expanded keys and values; writes their rows of out [T, >= H * vdim]."""
+    _lib.check(_lib.lib().ogb_attention_tc_latent(_ptr(proj), proj.stride(0), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), shape.R, plan.rows,
+                                                 _ptr(cu_seqlens), _ptr(past_lens), _ptr(plan.row_base), _ptr(plan.first_kv), _ptr(out), out.stride(0),
+                                                 float(scale), int(window), past_lens.shape[0], plan.max_q_len, shape.H, shape.dim, shape.rot,
+                                                 shape.vdim, workspace(proj.device).status, _stream()), "attention_tc_latent")
     return out
+
+
+def latent_attention_long(proj, shape, w_ukv, cache, plan: LatentPlan, cu_seqlens, past_lens, block_table, block_size, scale, window, out):
+    """The long requests of a step (plan): their visible latents are gathered, expanded to keys and values, and attended on the tensor
+    cores.  Writes the requests' rows of out [T, >= H * vdim]."""
+    lat, kv = latent_expand(shape, w_ukv, cache, plan, block_table, block_size)
+    return latent_attend_expanded(proj, shape, lat, kv, plan, cu_seqlens, past_lens, scale, window, out)
 
 
 # ------------------------------------------------------------------------------------------ logits processing
