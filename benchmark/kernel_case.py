@@ -239,8 +239,9 @@ def build_case(name, T, L, tp=1):
                 plan.rows * Hl * (d + dv) * 2 + Tq * Hl * (d + r + dv) * 2, sum(2.0 * Hl * (d + r + dv) * n * (n + 1) / 2 for _, n in lens)
         qlat = _bf(Tq, Hl * R, std=0.3)
         kv_tokens = sum(p + n for p, n in lens)
+        order = torch.argsort(-pl.long(), stable=True).to(torch.int32) if ATTN_ORDER else None
         return (lambda i: ops.latent_attention(qlat, proj, sh, caches[i % Lk], cu, pl, table, bs, scale, 0, 1, max(p + n for p, n in lens),
-                                               splits=ATTN_SPLITS[0] if isinstance(ATTN_SPLITS, tuple) else ATTN_SPLITS)), \
+                                               splits=ATTN_SPLITS[0] if isinstance(ATTN_SPLITS, tuple) else ATTN_SPLITS, order=order)), \
             kv_tokens * (R + r) * 2 + Tq * Hl * (2 * R + r) * 2, 2.0 * kv_tokens * Hl * (2 * R + r)
     if name == "norm_stream":
         xs, w, b = [torch.randn(T, H, device="cuda") for _ in range(8)], torch.randn(H, device="cuda"), torch.randn(H, device="cuda")

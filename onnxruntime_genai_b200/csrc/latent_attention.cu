@@ -5,9 +5,10 @@
 // and its result before the value map is sum_j p_j c_j: every head of a token reads the same rows, once, for scores and values.
 // Kernels:
 //   latent_prep_kernel   RMS norm of the latent and rotation of the key part into the cache; rotation of the queries' rotary parts.
-//   latent_mma_kernel    decode steps and short portions: one CTA = (request, up to 64 (token, head) rows, key split); tiles of 64
+//   latent_mma_kernel    decode steps and short portions: one CTA = (request, up to 64 (token, head) rows, key split); tiles of 32
 //                        cache rows through cp.async double buffering serve as K (all columns) and as V (the first R columns) of
-//                        warp-level MMAs.  Like paged_attention_kernel (attention.cu) it is bound by the cache stream and its rows are
+//                        warp-level MMAs; two CTAs share an SM (up to 16 rows of 576 columns), so that one's copies and softmax run
+//                        under the other's MMAs.  Like paged_attention_kernel (attention.cu) it is bound by the cache stream and its rows are
 //                        few; long prompts take the tensor-memory kernel (attention_tc.cu) on expanded keys and values instead.
 //   latent_simt_kernel   the same op in plain fp32 arithmetic for fp32 models and for sizes the other kernels cannot address.
 //   latent_gather_kernel cached rows of some requests into a dense matrix (input of the key / value expansion of long prompts).
@@ -79,28 +80,36 @@ struct LatentParams {
   float* part_o; float* part_ml;
   float scale;
   int window, B, H, R, rot, kp, pitch, splits, total_rows, skip_q_len;
+  const int32_t* order;           // [B] requests in issue order (longest first), or null
 };
 
-constexpr int LAT_BN = 64, LAT_THREADS = 256, LAT_PP = LAT_BN + 8;   // keys per tile; pitch of a P row
+constexpr int LAT_BN = 32, LAT_THREADS = 256, LAT_PP = LAT_BN + 8, LAT_SP = LAT_BN + 4;   // keys per tile; pitches of P and score rows
 
 template <int MT>
-__host__ __device__ constexpr int lat_smem_bytes(int pitch) {
-  return MT * 16 * pitch * 2 + 2 * LAT_BN * pitch * 2 + MT * 16 * LAT_PP * 2 + 8 * MT * 16 * 4 + 64;
-}
+struct LatCfg {
+  static constexpr int BM = MT * 16;
+  static constexpr int KH = MT == 4 ? 1 : 2;           // the score sums are divided over KH warps by columns of the rows
+  static constexpr int TPR = LAT_THREADS / BM;         // threads of one row in the softmax
+  static constexpr int KPT = LAT_BN / TPR;             // keys of each of them
+  static constexpr int smem(int pitch) { return (BM + 2 * LAT_BN) * pitch * 2 + BM * LAT_PP * 2 + KH * BM * LAT_SP * 4 + BM * 8 + 64; }
+};
 
 template <int MT, int NTW>
-__global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p) {
-  constexpr int BM = MT * 16, KG = 8 / MT;             // rows; key groups (warps of one row block)
+__global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kernel(LatentParams p) {
+  using Cfg = LatCfg<MT>;
+  constexpr int BM = Cfg::BM, KH = Cfg::KH, TPR = Cfg::TPR, KPT = Cfg::KPT;
   extern __shared__ __align__(128) uint8_t smem[];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);
-  __nv_bfloat16* sK = sQ + BM * p.pitch;               // [2][64][pitch]
+  __nv_bfloat16* sK = sQ + BM * p.pitch;               // [2][LAT_BN][pitch]
   __nv_bfloat16* sP = sK + 2 * LAT_BN * p.pitch;       // [BM][LAT_PP]
-  float* wred = reinterpret_cast<float*>(sP + BM * LAT_PP);   // [KG][BM] row maxima / sums of the key groups
+  float* sS = reinterpret_cast<float*>(sP + BM * LAT_PP);     // [KH][BM][LAT_SP] partial scores
+  float* sA = sS + KH * BM * LAT_SP;                   // [BM] factor of the old output; at the end the row sums
+  float* sM = sA + BM;                                 // [BM] at the end the row maxima
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int mt = warp % MT, kg = warp / MT;
-  const int b = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+  const int bz = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+  const int b = p.order ? p.order[bz] : bz;
   const int H = p.H, tok0 = p.cu[b], q_len = p.cu[b + 1] - tok0, rows = q_len * H;
   const int row0 = blockIdx.x * BM;
   if (row0 >= rows || (p.skip_q_len > 0 && q_len >= p.skip_q_len)) return;
@@ -121,13 +130,16 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p)
   }
   const int n_tiles = (hi - lo + LAT_BN - 1) / LAT_BN;
   const int kc = (p.R + p.rot) / 8, rc = p.R / 8;      // 16-byte chunks of a cache row; of its latent
-  auto load = [&](int it) {                            // a warp copies 8 rows of the tile; rows past the range become zeros
-    const int j = lo + it * LAT_BN + warp * 8 + (lane & 7);
-    int slot = -1;
-    if (j < hi) slot = table[j / p.block_size] * p.block_size + j % p.block_size;
-    __nv_bfloat16* dst = sK + ((it & 1) * LAT_BN + warp * 8) * p.pitch;
+  // A warp copies 4 rows of a tile; their cache slots are looked up one tile ahead of the copy, so that the copy does not wait for the
+  // table.  Rows past the range become zeros.
+  auto lookup = [&](int it) {
+    const int j = lo + it * LAT_BN + warp * 4 + (lane & 3);
+    return j < hi ? table[j / p.block_size] * p.block_size + j % p.block_size : -1;
+  };
+  auto load = [&](int it, int slot) {
+    __nv_bfloat16* dst = sK + ((it & 1) * LAT_BN + warp * 4) * p.pitch;
 #pragma unroll
-    for (int r = 0; r < 8; ++r) {
+    for (int r = 0; r < 4; ++r) {
       const int sl = __shfl_sync(0xffffffffu, slot, r);
       const __nv_bfloat16* src = p.cache + (sl >= 0 ? size_t(sl) * p.ldcache : 0);
       for (int c = lane; c < kc; c += 32) cp_async16(dst + r * p.pitch + c * 8, src + c * 8, sl >= 0);
@@ -148,111 +160,132 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p)
     for (int r = tid; r < BM; r += LAT_THREADS) *reinterpret_cast<uint4*>(sQ + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
     for (int r = tid; r < 2 * LAT_BN; r += LAT_THREADS) *reinterpret_cast<uint4*>(sK + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
   }
-  if (n_tiles > 0) load(0);
+  int slot_next = -1;
+  if (n_tiles > 0) {
+    load(0, lookup(0));
+    slot_next = lookup(1);
+  }
   cp_async_commit();
 
-  const int r_lo = mt * 16 + g, r_hi = r_lo + 8;       // score rows of this thread
-  const bool v_lo = row0 + r_lo < rows, v_hi = row0 + r_hi < rows;
-  const int q_lo = past + (row0 + r_lo) / H, q_hi = past + (row0 + r_hi) / H;
+  // softmax: TPR neighbouring threads share row sr, KPT keys each
+  const int sr = tid / TPR, sk0 = (tid % TPR) * KPT;
+  const bool s_valid = row0 + sr < rows;
+  const int s_pos = past + (row0 + sr) / H;
   const float sc2 = p.scale * LAT_LOG2E;
-  const int ksteps = p.kp / 16, c0 = warp * NTW * 8;   // output columns [c0, c0 + 8 * NTW) of every row
+  float mx = -INFINITY, l = 0.f;                       // the row's running maximum; the sum over this thread's keys
+  // scores: warp -> 16 rows (mt), a group of keys (kg), a share of the columns (kh)
+  const int ksteps = p.kp / 16;
+  const int mt = warp % MT, kg = MT == 1 ? warp & 3 : (warp / MT) & 1, kh = KH == 1 ? 0 : warp >> 2;
+  const int kmid = KH == 1 ? ksteps : (ksteps / 2 + 1) & ~1;                   // an even number of steps in the first share
+  const int ks0 = kh ? kmid : 0, ks1 = kh ? ksteps : kmid;
+  const int c0 = warp * NTW * 8;                       // output columns [c0, c0 + 8 * NTW) of every row
   float o[MT][NTW][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int n = 0; n < NTW; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
-  float mx[MT][2], l_lo = 0.f, l_hi = 0.f;             // running maxima of rows (16 m + g, + 8); sums over this thread's own keys
-#pragma unroll
-  for (int m = 0; m < MT; ++m) mx[m][0] = mx[m][1] = -INFINITY;
 
   for (int it = 0; it < n_tiles; ++it) {
     cp_async_wait<0>();
     __syncthreads();                                   // tile it has landed; every warp is done with tile it - 1
-    if (it + 1 < n_tiles) load(it + 1);
+    if (it + 1 < n_tiles) {
+      load(it + 1, slot_next);
+      slot_next = lookup(it + 2);
+    }
     cp_async_commit();
     const __nv_bfloat16* tk = sK + (it & 1) * LAT_BN * p.pitch;
-    // ---- scores of 16 rows x 8 * MT keys
-    float s[MT][4];
-#pragma unroll
-    for (int n = 0; n < MT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
     const __nv_bfloat16* qa = sQ + (mt * 16 + (lane & 15)) * p.pitch + (lane >> 4) * 8;
+    float* ps = sS + (kh * BM + mt * 16 + g) * LAT_SP + t4 * 2;
     if constexpr (MT == 1) {
-      float s2[4] = {0.f, 0.f, 0.f, 0.f};
+      // 16 rows x 8 keys; four accumulators: the MMAs of one sum would wait for each other
+      float s[4][4] = {};
       const __nv_bfloat16* ka = tk + (kg * 8 + (lane & 7)) * p.pitch + (lane >> 3) * 8;
+      int ks = ks0;
 #pragma unroll 2
-      for (int ks = 0; ks < ksteps; ks += 2) {
+      for (; ks + 4 <= ks1; ks += 4) {
+        uint32_t q0[4], q1[4], q2[4], q3[4], k0[4], k1[4];
+        ldmatrix_x4(k0, ka + ks * 16);
+        ldmatrix_x4(k1, ka + ks * 16 + 32);
+        ldmatrix_x4(q0, qa + ks * 16);
+        ldmatrix_x4(q1, qa + ks * 16 + 16);
+        ldmatrix_x4(q2, qa + ks * 16 + 32);
+        ldmatrix_x4(q3, qa + ks * 16 + 48);
+        mma_bf16_16816(s[0], q0, k0[0], k0[1]);
+        mma_bf16_16816(s[1], q1, k0[2], k0[3]);
+        mma_bf16_16816(s[2], q2, k1[0], k1[1]);
+        mma_bf16_16816(s[3], q3, k1[2], k1[3]);
+      }
+      for (; ks < ks1; ks += 2) {                      // (a last odd step reads 16 bytes past the row: the next row or P, unused)
         uint32_t qf[4], kb[4];
         ldmatrix_x4(kb, ka + ks * 16);
         ldmatrix_x4(qf, qa + ks * 16);
         mma_bf16_16816(s[0], qf, kb[0], kb[1]);
-        if (ks + 1 < ksteps) {
+        if (ks + 1 < ks1) {
           ldmatrix_x4(qf, qa + ks * 16 + 16);
-          mma_bf16_16816(s2, qf, kb[2], kb[3]);
+          mma_bf16_16816(s[1], qf, kb[2], kb[3]);
         }
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[0][e] += s2[e];
+      for (int e = 0; e < 4; ++e) s[0][e] = (s[0][e] + s[1][e]) + (s[2][e] + s[3][e]);
+      *reinterpret_cast<float2*>(ps + kg * 8) = make_float2(s[0][0], s[0][1]);
+      *reinterpret_cast<float2*>(ps + 8 * LAT_SP + kg * 8) = make_float2(s[0][2], s[0][3]);
     } else {
-      const __nv_bfloat16* ka = tk + (kg * 8 * MT + (lane >> 4) * 8 + (lane & 7)) * p.pitch + ((lane >> 3) & 1) * 8;
+      // 16 rows x 16 keys
+      float s[2][2][4] = {};
+      const __nv_bfloat16* ka = tk + (kg * 16 + (lane >> 4) * 8 + (lane & 7)) * p.pitch + ((lane >> 3) & 1) * 8;
 #pragma unroll 2
-      for (int ks = 0; ks < ksteps; ++ks) {
-        uint32_t qf[4];
+      for (int ks = ks0; ks < ks1; ks += 2) {
+        uint32_t qf[4], kb[4], qf2[4], kb2[4];
+        const int k2 = min(ks + 1, ks1 - 1);
         ldmatrix_x4(qf, qa + ks * 16);
-#pragma unroll
-        for (int np = 0; np < MT / 2; ++np) {
-          uint32_t kb[4];
-          ldmatrix_x4(kb, ka + np * 16 * p.pitch + ks * 16);
-          mma_bf16_16816(s[np * 2], qf, kb[0], kb[1]);
-          mma_bf16_16816(s[np * 2 + 1], qf, kb[2], kb[3]);
+        ldmatrix_x4(kb, ka + ks * 16);
+        ldmatrix_x4(qf2, qa + k2 * 16);
+        ldmatrix_x4(kb2, ka + k2 * 16);
+        mma_bf16_16816(s[0][0], qf, kb[0], kb[1]);
+        mma_bf16_16816(s[0][1], qf, kb[2], kb[3]);
+        if (ks + 1 < ks1) {
+          mma_bf16_16816(s[1][0], qf2, kb2[0], kb2[1]);
+          mma_bf16_16816(s[1][1], qf2, kb2[2], kb2[3]);
         }
       }
-    }
-    const int jb = lo + it * LAT_BN + kg * 8 * MT + t4 * 2;
-    float mlo = -INFINITY, mhi = -INFINITY;
 #pragma unroll
-    for (int n = 0; n < MT; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int j = jb + n * 8 + (e & 1), qp = e >= 2 ? q_hi : q_lo;
-        const bool ok = (e >= 2 ? v_hi : v_lo) && j < hi && j <= qp && (p.window <= 0 || j > qp - p.window);
-        s[n][e] = ok ? s[n][e] * sc2 : -INFINITY;
-        if (e >= 2) mhi = fmaxf(mhi, s[n][e]); else mlo = fmaxf(mlo, s[n][e]);
+      for (int n = 0; n < 2; ++n) {
+        *reinterpret_cast<float2*>(ps + kg * 16 + n * 8) = make_float2(s[0][n][0] + s[1][n][0], s[0][n][1] + s[1][n][1]);
+        *reinterpret_cast<float2*>(ps + 8 * LAT_SP + kg * 16 + n * 8) = make_float2(s[0][n][2] + s[1][n][2], s[0][n][3] + s[1][n][3]);
       }
-    mlo = fmaxf(mlo, __shfl_xor_sync(0xffffffffu, mlo, 1)); mlo = fmaxf(mlo, __shfl_xor_sync(0xffffffffu, mlo, 2));
-    mhi = fmaxf(mhi, __shfl_xor_sync(0xffffffffu, mhi, 1)); mhi = fmaxf(mhi, __shfl_xor_sync(0xffffffffu, mhi, 2));
-    if (t4 == 0) { wred[kg * BM + r_lo] = mlo; wred[kg * BM + r_hi] = mhi; }
+    }
     __syncthreads();
-    // ---- new maxima of all rows (every warp holds output columns of all of them), P of the own rows
-    float al[MT][2];
+    // ---- softmax of the tile's scores
+    float x[KPT], tmax = -INFINITY;
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        float n = mx[m][e];
-#pragma unroll
-        for (int k = 0; k < KG; ++k) n = fmaxf(n, wred[k * BM + m * 16 + g + e * 8]);
-        al[m][e] = n == -INFINITY ? 1.f : exp2f(mx[m][e] - n);
-        mx[m][e] = n;
-      }
-    float a_lo = 0.f, a_hi = 0.f, n_lo = 0.f, n_hi = 0.f;
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-      if (m == mt) { a_lo = al[m][0]; a_hi = al[m][1]; n_lo = mx[m][0] == -INFINITY ? 0.f : mx[m][0]; n_hi = mx[m][1] == -INFINITY ? 0.f : mx[m][1]; }
-    l_lo *= a_lo; l_hi *= a_hi;
-#pragma unroll
-    for (int n = 0; n < MT; ++n) {
-      const float p0 = exp2f(s[n][0] - n_lo), p1 = exp2f(s[n][1] - n_lo), p2 = exp2f(s[n][2] - n_hi), p3 = exp2f(s[n][3] - n_hi);
-      l_lo += p0 + p1; l_hi += p2 + p3;
-      const int kcol = kg * 8 * MT + n * 8 + t4 * 2;
-      *reinterpret_cast<uint32_t*>(sP + r_lo * LAT_PP + kcol) = pack_bf16x2(p0, p1);
-      *reinterpret_cast<uint32_t*>(sP + r_hi * LAT_PP + kcol) = pack_bf16x2(p2, p3);
+    for (int e = 0; e < KPT; ++e) {
+      float v = sS[sr * LAT_SP + sk0 + e];
+      if constexpr (KH == 2) v += sS[(BM + sr) * LAT_SP + sk0 + e];
+      const int j = lo + it * LAT_BN + sk0 + e;
+      x[e] = s_valid && j < hi && j <= s_pos && (p.window <= 0 || j > s_pos - p.window) ? v * sc2 : -INFINITY;
+      tmax = fmaxf(tmax, x[e]);
     }
+#pragma unroll
+    for (int w = TPR / 2; w > 0; w >>= 1) tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, w));
+    const float mn = fmaxf(mx, tmax), ms = mn == -INFINITY ? 0.f : mn;
+    const float al = mn == -INFINITY ? 1.f : exp2f(mx - mn);
+    mx = mn;
+    l *= al;
+#pragma unroll
+    for (int e = 0; e < KPT; e += 2) {
+      const float p0 = exp2f(x[e] - ms), p1 = exp2f(x[e + 1] - ms);
+      l += p0 + p1;
+      *reinterpret_cast<uint32_t*>(sP + sr * LAT_PP + sk0 + e) = pack_bf16x2(p0, p1);
+    }
+    if (sk0 == 0) sA[sr] = al;
     __syncthreads();
     // ---- O = O * alpha + P C
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int m = 0; m < MT; ++m) {
+      const float al0 = sA[m * 16 + g], al1 = sA[m * 16 + g + 8];
 #pragma unroll
-      for (int n = 0; n < NTW; ++n) { o[m][n][0] *= al[m][0]; o[m][n][1] *= al[m][0]; o[m][n][2] *= al[m][1]; o[m][n][3] *= al[m][1]; }
+      for (int n = 0; n < NTW; ++n) { o[m][n][0] *= al0; o[m][n][1] *= al0; o[m][n][2] *= al1; o[m][n][3] *= al1; }
+    }
 #pragma unroll
     for (int kk = 0; kk < LAT_BN / 16; ++kk) {
       uint32_t pa[MT][4];
@@ -272,11 +305,10 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p)
     }
   }
   cp_async_wait<0>();
-  // row sums: the quad's threads, then the key groups
-  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
-  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+#pragma unroll
+  for (int w = TPR / 2; w > 0; w >>= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
   __syncthreads();
-  if (t4 == 0) { wred[kg * BM + r_lo] = l_lo; wred[kg * BM + r_hi] = l_hi; }
+  if (sk0 == 0) { sA[sr] = l; sM[sr] = mx; }
   __syncthreads();
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -284,9 +316,7 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p)
     for (int e = 0; e < 2; ++e) {
       const int r = m * 16 + g + e * 8;
       if (row0 + r >= rows) continue;
-      float l = 0.f;
-#pragma unroll
-      for (int k = 0; k < KG; ++k) l += wred[k * BM + r];
+      const float lr = sA[r];
       const size_t orow = size_t(tok0) * H + row0 + r;
       if (p.splits > 1) {
         float* po = p.part_o + (size_t(split) * p.total_rows + orow) * p.R;
@@ -295,10 +325,10 @@ __global__ void __launch_bounds__(LAT_THREADS) latent_mma_kernel(LatentParams p)
           if (c0 + n * 8 < p.R) *reinterpret_cast<float2*>(po + c0 + n * 8 + t4 * 2) = make_float2(o[m][n][e * 2], o[m][n][e * 2 + 1]);
         if (warp == 0 && t4 == 0) {
           float* pm = p.part_ml + (size_t(split) * p.total_rows + orow) * 2;
-          pm[0] = mx[m][e]; pm[1] = l;
+          pm[0] = sM[r]; pm[1] = lr;
         }
       } else {
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = lr > 0.f ? 1.f / lr : 0.f;
         __nv_bfloat16* po = p.out + orow * p.R;
 #pragma unroll
         for (int n = 0; n < NTW; ++n)
@@ -430,7 +460,7 @@ static int LaunchLatentMma(const LatentParams& p, int max_q_len, cudaStream_t s)
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, 227 * 1024, configured)) return -3;
   const dim3 grid((max_q_len * p.H + MT * 16 - 1) / (MT * 16), 1, p.B * p.splits);
-  if (!launch_pdl(kern, grid, dim3(LAT_THREADS), lat_smem_bytes<MT>(p.pitch), s, p)) return -4;
+  if (!launch_pdl(kern, grid, dim3(LAT_THREADS), LatCfg<MT>::smem(p.pitch), s, p)) return -4;
   if (p.splits > 1 && !launch_pdl(latent_combine_kernel, dim3(p.total_rows), dim3(128), 0, s, static_cast<const float*>(p.part_o),
                                   static_cast<const float*>(p.part_ml), p.out, p.total_rows, p.R, p.splits))
     return -4;
@@ -464,7 +494,7 @@ OGB_API int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const
 
 // 1 when the warp-MMA kernel can address these sizes (16-byte pieces everywhere, the tile fits in shared memory).
 OGB_API int ogb_latent_mma_supported(const OgbLatentShape* sh) {
-  return sh->R % 8 == 0 && sh->rot % 8 == 0 && sh->dim % 8 == 0 && sh->R >= 8 && sh->R <= 512 && lat_smem_bytes<1>(lat_pitch(sh)) <= 227 * 1024;
+  return sh->R % 8 == 0 && sh->rot % 8 == 0 && sh->dim % 8 == 0 && sh->R >= 8 && sh->R <= 512 && LatCfg<1>::smem(lat_pitch(sh)) <= 227 * 1024;
 }
 
 // Rows of (token, head) a CTA takes for requests of at most max_q_len tokens.
@@ -481,7 +511,7 @@ OGB_API long long ogb_latent_scratch_bytes(int total_rows, int R, int splits) {
 OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                                  const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
                                  void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
-                                 long long scratch_bytes, void* stream) {
+                                 long long scratch_bytes, const int32_t* order, void* stream) {
   if (B <= 0 || T <= 0 || max_q_len <= 0) return 0;
   if (!ogb_latent_mma_supported(sh)) return -5;
   if ((ldp % 8) || (ldcache % 8) || block_size <= 0) return -1;
@@ -498,11 +528,11 @@ OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, co
   p.part_ml = p.part_o ? p.part_o + size_t(splits) * rows * sh->R : nullptr;
   p.scale = scale; p.window = window; p.B = B; p.H = sh->H; p.R = sh->R; p.rot = sh->rot;
   p.kp = (sh->R + sh->rot + 15) / 16 * 16; p.pitch = lat_pitch(sh);
-  p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len;
+  p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len; p.order = order;
   auto s = static_cast<cudaStream_t>(stream);
   int bm = ogb_latent_rows_per_tile(sh->H, skip_q_len > 0 && skip_q_len - 1 < max_q_len ? skip_q_len - 1 : max_q_len);
-  if (bm == 64 && lat_smem_bytes<4>(p.pitch) > 227 * 1024) bm = 32;
-  if (bm == 32 && lat_smem_bytes<2>(p.pitch) > 227 * 1024) bm = 16;
+  if (bm == 64 && LatCfg<4>::smem(p.pitch) > 227 * 1024) bm = 32;
+  if (bm == 32 && LatCfg<2>::smem(p.pitch) > 227 * 1024) bm = 16;
   if (skip_q_len > 0 && max_q_len > skip_q_len - 1) max_q_len = skip_q_len - 1;
   if (max_q_len <= 0) return 0;
   if (bm == 16) return LaunchLatentMt<1>(p, max_q_len, s);

@@ -7,8 +7,8 @@
 //   gated_delta_kernel        decode-shaped steps.  One CTA = (request, value head, 32 columns of the head's state S [dk, dv]); a thread
 //                             keeps 16 to 64 rows of one column, the lanes of a warp are neighbouring columns (the state streams in
 //                             full lines), the row splits of a column meet in shared memory.
-//   gated_delta_chunk_kernel  prompts.  The lanes of a warp are 8 columns x 4 row splits, so that the two dot products of a token are
-//                             finished by two shuffles and the token loop has no barrier; the keys and queries of a chunk of tokens
+//   gated_delta_chunk_kernel  prompts.  The row splits of a column are lanes of one warp, so that the two dot products of a token are
+//                             finished by shuffles and the token loop has no barrier; the keys and queries of a chunk of tokens
 //                             are normalised into shared memory by all warps beforehand.
 // Per token, with k_t, q_t of the head:
 //     S[:, j] *= exp(g);   mem = sum_i S[i, j] k[i];   delta = (v[j] - mem) * beta;   S[i, j] += k[i] * delta;   o[j] = sum_i S[i, j] q[i]
@@ -65,7 +65,8 @@ __device__ __forceinline__ void gdn_gates(const GdnParams<T>& p, int t, int h, f
 
 constexpr int GDN_MAX_DK = 1024, GDN_MAX_SPLITS = 16;
 
-template <typename T, int NPT>
+// FULL: dk is a multiple of NPT, no row is past the size.
+template <typename T, int NPT, bool FULL>
 __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams<T> p) {
   // thread (j, sp): column j of the state, rows [sp * NPT, (sp + 1) * NPT); the two dot products of a token (with k, then with q)
   // are summed over the splits through shared memory
@@ -86,8 +87,8 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams<T> p) {
   const bool live = j < dv;
   const bool fresh = p.past_lens[b] == 0;
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh && n0 + i < dk) ? S[size_t(i) * dv + j] : 0.f;
-  for (int i = dk + threadIdx.x; i < splits * NPT; i += blockDim.x) { sk[i] = 0.f; sq[i] = 0.f; }
+  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh && (FULL || n0 + i < dk)) ? S[size_t(i) * dv + j] : 0.f;
+  if (!FULL) for (int i = dk + threadIdx.x; i < splits * NPT; i += blockDim.x) { sk[i] = 0.f; sq[i] = 0.f; }
   for (int t = t0; t < t1; ++t) {
     __syncthreads();
     float ssk = 0.f, ssq = 0.f;
@@ -141,110 +142,142 @@ __global__ void __launch_bounds__(512) gated_delta_kernel(GdnParams<T> p) {
   }
   if (live) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) if (n0 + i < dk) S[size_t(i) * dv + j] = col[i];
+    for (int i = 0; i < NPT; ++i) if (FULL || n0 + i < dk) S[size_t(i) * dv + j] = col[i];
   }
 }
 
-// NPT rows per thread, 4 * NPT >= dk.  Row of thread split sp, register i: (i / 4) * 16 + sp * 4 + i % 4, so that a thread's rows come
-// as groups of four and the four splits of a warp read neighbouring 16-byte words of a key.  CH tokens per chunk.
+// A thread owns two columns and NPT rows of each, 8 * NPT >= dk; the lanes of a warp are 4 column pairs x 8 row splits.  Row of split sp,
+// register i: (i / 4) * 32 + sp * 4 + i % 4, so that a thread's rows come as groups of four and the splits of a warp read one
+// 128-byte line of a key together.  CH tokens per chunk.
+// Both dot products of a token are taken on the state before its update, which needs the two vectors once and one round of
+// shuffles: with m = S^T k and r = S^T q (old state), delta = beta * (v - g m), S <- g S + k delta^T and S_new^T q = g r + (k . q) delta.
 template <typename T, int NPT, int CH>
 __global__ void __launch_bounds__(128) gated_delta_chunk_kernel(GdnParams<T> p) {
-  constexpr int DKP = NPT * 4;
+  constexpr int DKP = NPT * 8, G4 = NPT / 4;
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y;
   const int Hv = p.Hv, dv = p.dv, dk = p.dk;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sp = lane & 3;
-  const int jj = warp * 8 + (lane >> 2), j = blockIdx.z * 32 + jj;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sp = lane & 7;
+  const int jj = warp * 8 + (lane >> 3) * 2, j = blockIdx.z * 32 + jj;      // columns j, j + 1
   const int hk = h / (Hv / p.Hk);
   const int t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
   if (t0 >= t1) return;
   __shared__ __align__(16) float sk[CH][DKP];
   __shared__ __align__(16) float sq[CH][DKP];
-  __shared__ float sv[CH][32], sgate[2][CH];
-  const bool live = j < dv, fresh = p.past_lens[b] == 0;
+  __shared__ __align__(8) float sv[CH][32];
+  __shared__ float sdot[CH], sgate[2][CH];
+  const bool live0 = j < dv, live1 = j + 1 < dv, fresh = p.past_lens[b] == 0;
   float* S = p.state + size_t(p.slots[b]) * p.slot_stride + size_t(h) * dk * dv;
-  auto row_of = [&](int i) { return (i >> 2) * 16 + sp * 4 + (i & 3); };
-  float col[NPT];
+  auto row_of = [&](int i) { return (i >> 2) * 32 + sp * 4 + (i & 3); };
+  float c0[NPT], c1[NPT];
 #pragma unroll
-  for (int i = 0; i < NPT; ++i) col[i] = (live && !fresh && row_of(i) < dk) ? S[size_t(row_of(i)) * dv + j] : 0.f;
+  for (int i = 0; i < NPT; ++i) {
+    const bool ok = !fresh && row_of(i) < dk;
+    c0[i] = ok && live0 ? S[size_t(row_of(i)) * dv + j] : 0.f;
+    c1[i] = ok && live1 ? S[size_t(row_of(i)) * dv + j + 1] : 0.f;
+  }
 
   // a chunk's raw keys / queries / values on their way from global memory: held in registers while the previous chunk is computed
   constexpr int PER = DKP / 32, TW = CH / 4;               // elements per lane of a row, rows per warp
-  float rk[TW][PER], rq[TW][PER], rv[TW], ga, gb;
-  auto fetch = [&](int c0) {
+  const T zero = act_from<T>(0.f);
+  T rk[TW][PER], rq[TW][PER], rv[TW];
+  float ga, gb;
+  auto fetch = [&](int f0) {
 #pragma unroll
     for (int w = 0; w < TW; ++w) {
-      const int t = c0 + w * 4 + warp;
+      const int t = f0 + w * 4 + warp;
 #pragma unroll
       for (int e = 0; e < PER; ++e) {
         const int i = e * 32 + lane;
         const bool ok = t < t1 && i < dk;
-        rk[w][e] = ok ? act_f32(p.k[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]) : 0.f;
-        rq[w][e] = ok ? act_f32(p.q[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i]) : 0.f;
+        rk[w][e] = ok ? p.k[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i] : zero;
+        rq[w][e] = ok ? p.q[size_t(t) * p.tok_stride_qk + size_t(hk) * dk + i] : zero;
       }
       const int jc = blockIdx.z * 32 + lane;
-      rv[w] = (t < t1 && jc < dv) ? act_f32(p.v[size_t(t) * p.tok_stride_v + size_t(h) * dv + jc]) : 0.f;
+      rv[w] = (t < t1 && jc < dv) ? p.v[size_t(t) * p.tok_stride_v + size_t(h) * dv + jc] : zero;
     }
     ga = gb = 0.f;
-    if (threadIdx.x < CH && c0 + int(threadIdx.x) < t1) gdn_gates(p, c0 + threadIdx.x, h, ga, gb);
+    if (threadIdx.x < CH && f0 + int(threadIdx.x) < t1) gdn_gates(p, f0 + threadIdx.x, h, ga, gb);
   };
   fetch(t0);
-  for (int c0 = t0; c0 < t1; c0 += CH) {
+  for (int f0 = t0; f0 < t1; f0 += CH) {
     __syncthreads();                                       // the previous chunk is no longer read
 #pragma unroll
     for (int w = 0; w < TW; ++w) {
-      float ssk = 0.f, ssq = 0.f;
+      float ssk = 0.f, ssq = 0.f, skq = 0.f;
 #pragma unroll
-      for (int e = 0; e < PER; ++e) { ssk += rk[w][e] * rk[w][e]; ssq += rq[w][e] * rq[w][e]; }
+      for (int e = 0; e < PER; ++e) {
+        const float kk = act_f32(rk[w][e]), qq = act_f32(rq[w][e]);
+        ssk += kk * kk; ssq += qq * qq; skq += kk * qq;
+      }
       float nk = 1.f, nq = 1.f;
       if (p.l2norm) {
         nk = inv_length(warp_sum(ssk), p.l2_eps);
         nq = p.q_scale * inv_length(warp_sum(ssq), p.l2_eps);
       }
+      skq = warp_sum(skq) * nk * nq;
       const int tt = w * 4 + warp;
 #pragma unroll
-      for (int e = 0; e < PER; ++e) { sk[tt][e * 32 + lane] = rk[w][e] * nk; sq[tt][e * 32 + lane] = rq[w][e] * nq; }
-      sv[tt][lane] = rv[w];
+      for (int e = 0; e < PER; ++e) {
+        sk[tt][e * 32 + lane] = act_f32(rk[w][e]) * nk;
+        sq[tt][e * 32 + lane] = act_f32(rq[w][e]) * nq;
+      }
+      sv[tt][lane] = act_f32(rv[w]);
+      if (lane == 0) sdot[tt] = skq;
     }
     if (threadIdx.x < CH) { sgate[0][threadIdx.x] = ga; sgate[1][threadIdx.x] = gb; }
     __syncthreads();
-    if (c0 + CH < t1) fetch(c0 + CH);
-    const int n = min(CH, t1 - c0);
+    if (f0 + CH < t1) fetch(f0 + CH);
+    const int n = min(CH, t1 - f0);
     for (int tt = 0; tt < n; ++tt) {
-      const float decay = sgate[0][tt], bt = sgate[1][tt], vj = sv[tt][jj];
+      const float decay = sgate[0][tt], bt = sgate[1][tt], kq = sdot[tt];
+      const float2 vj = *reinterpret_cast<const float2*>(&sv[tt][jj]);
       const float4* k4 = reinterpret_cast<const float4*>(sk[tt]) + sp;
       const float4* q4 = reinterpret_cast<const float4*>(sq[tt]) + sp;
-      float m4[4] = {0.f, 0.f, 0.f, 0.f};
+      float4 kk[G4];
+      float m0a = 0.f, m0b = 0.f, m1a = 0.f, m1b = 0.f, r0a = 0.f, r0b = 0.f, r1a = 0.f, r1b = 0.f;
 #pragma unroll
-      for (int i = 0; i < NPT / 4; ++i) {
-        const float4 kk = k4[i * 4];
-        col[4 * i] *= decay; col[4 * i + 1] *= decay; col[4 * i + 2] *= decay; col[4 * i + 3] *= decay;
-        m4[0] = fmaf(col[4 * i], kk.x, m4[0]); m4[1] = fmaf(col[4 * i + 1], kk.y, m4[1]);
-        m4[2] = fmaf(col[4 * i + 2], kk.z, m4[2]); m4[3] = fmaf(col[4 * i + 3], kk.w, m4[3]);
+      for (int i = 0; i < G4; ++i) {
+        kk[i] = k4[i * 8];
+        const float4 qq = q4[i * 8];
+        m0a = fmaf(c0[4 * i], kk[i].x, m0a); m1a = fmaf(c1[4 * i], kk[i].x, m1a);
+        m0b = fmaf(c0[4 * i + 1], kk[i].y, m0b); m1b = fmaf(c1[4 * i + 1], kk[i].y, m1b);
+        m0a = fmaf(c0[4 * i + 2], kk[i].z, m0a); m1a = fmaf(c1[4 * i + 2], kk[i].z, m1a);
+        m0b = fmaf(c0[4 * i + 3], kk[i].w, m0b); m1b = fmaf(c1[4 * i + 3], kk[i].w, m1b);
+        r0a = fmaf(c0[4 * i], qq.x, r0a); r1a = fmaf(c1[4 * i], qq.x, r1a);
+        r0b = fmaf(c0[4 * i + 1], qq.y, r0b); r1b = fmaf(c1[4 * i + 1], qq.y, r1b);
+        r0a = fmaf(c0[4 * i + 2], qq.z, r0a); r1a = fmaf(c1[4 * i + 2], qq.z, r1a);
+        r0b = fmaf(c0[4 * i + 3], qq.w, r0b); r1b = fmaf(c1[4 * i + 3], qq.w, r1b);
       }
-      float mem = (m4[0] + m4[1]) + (m4[2] + m4[3]);
-      mem += __shfl_xor_sync(0xffffffffu, mem, 1);
-      mem += __shfl_xor_sync(0xffffffffu, mem, 2);
-      const float delta = (vj - mem) * bt;
-      float o4[4] = {0.f, 0.f, 0.f, 0.f};
+      float m0 = m0a + m0b, m1 = m1a + m1b, r0 = r0a + r0b, r1 = r1a + r1b;
 #pragma unroll
-      for (int i = 0; i < NPT / 4; ++i) {
-        const float4 kk = k4[i * 4], qq = q4[i * 4];
-        col[4 * i] = fmaf(kk.x, delta, col[4 * i]); col[4 * i + 1] = fmaf(kk.y, delta, col[4 * i + 1]);
-        col[4 * i + 2] = fmaf(kk.z, delta, col[4 * i + 2]); col[4 * i + 3] = fmaf(kk.w, delta, col[4 * i + 3]);
-        o4[0] = fmaf(col[4 * i], qq.x, o4[0]); o4[1] = fmaf(col[4 * i + 1], qq.y, o4[1]);
-        o4[2] = fmaf(col[4 * i + 2], qq.z, o4[2]); o4[3] = fmaf(col[4 * i + 3], qq.w, o4[3]);
+      for (int o = 1; o < 8; o <<= 1) {
+        m0 += __shfl_xor_sync(0xffffffffu, m0, o);
+        m1 += __shfl_xor_sync(0xffffffffu, m1, o);
+        r0 += __shfl_xor_sync(0xffffffffu, r0, o);
+        r1 += __shfl_xor_sync(0xffffffffu, r1, o);
       }
-      float o = (o4[0] + o4[1]) + (o4[2] + o4[3]);
-      o += __shfl_xor_sync(0xffffffffu, o, 1);
-      o += __shfl_xor_sync(0xffffffffu, o, 2);
-      if (live && sp == 0) p.out[(size_t(c0 + tt) * Hv + h) * dv + j] = act_from<T>(o);
+      const float d0 = (vj.x - decay * m0) * bt, d1 = (vj.y - decay * m1) * bt;
+#pragma unroll
+      for (int i = 0; i < G4; ++i) {
+        c0[4 * i] = fmaf(kk[i].x, d0, decay * c0[4 * i]); c1[4 * i] = fmaf(kk[i].x, d1, decay * c1[4 * i]);
+        c0[4 * i + 1] = fmaf(kk[i].y, d0, decay * c0[4 * i + 1]); c1[4 * i + 1] = fmaf(kk[i].y, d1, decay * c1[4 * i + 1]);
+        c0[4 * i + 2] = fmaf(kk[i].z, d0, decay * c0[4 * i + 2]); c1[4 * i + 2] = fmaf(kk[i].z, d1, decay * c1[4 * i + 2]);
+        c0[4 * i + 3] = fmaf(kk[i].w, d0, decay * c0[4 * i + 3]); c1[4 * i + 3] = fmaf(kk[i].w, d1, decay * c1[4 * i + 3]);
+      }
+      if (sp == 0) {
+        T* dst = p.out + (size_t(f0 + tt) * Hv + h) * dv + j;
+        if (live0) dst[0] = act_from<T>(fmaf(decay, r0, kq * d0));
+        if (live1) dst[1] = act_from<T>(fmaf(decay, r1, kq * d1));
+      }
     }
   }
-  if (live) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) if (row_of(i) < dk) S[size_t(row_of(i)) * dv + j] = col[i];
+  for (int i = 0; i < NPT; ++i) {
+    if (row_of(i) >= dk) continue;
+    if (live0) S[size_t(row_of(i)) * dv + j] = c0[i];
+    if (live1) S[size_t(row_of(i)) * dv + j + 1] = c1[i];
   }
 }
 
@@ -276,7 +309,9 @@ using namespace ogb;
 
 template <typename T, int NPT>
 static bool LaunchGdnDecode(const GdnParams<T>& p, int B, int splits, cudaStream_t s) {
-  return launch_pdl(gated_delta_kernel<T, NPT>, dim3(B, p.Hv, (p.dv + 31) / 32), dim3(32 * splits), 0, s, p);
+  const dim3 grid(B, p.Hv, (p.dv + 31) / 32), block(32 * splits);
+  return p.dk % NPT == 0 ? launch_pdl(gated_delta_kernel<T, NPT, true>, grid, block, 0, s, p)
+                         : launch_pdl(gated_delta_kernel<T, NPT, false>, grid, block, 0, s, p);
 }
 template <typename T, int NPT, int CH>
 static bool LaunchGdnChunk(const GdnParams<T>& p, int B, cudaStream_t s) {
@@ -293,10 +328,10 @@ static int LaunchGatedDelta(const GdnParams<T>& p, int B, int max_q_len, void* s
   auto s = static_cast<cudaStream_t>(stream);
   bool ok;
   if (max_q_len != 1 && dk <= 256) {
-    if (dk <= 32) ok = LaunchGdnChunk<T, 8, 32>(p, B, s);
-    else if (dk <= 64) ok = LaunchGdnChunk<T, 16, 32>(p, B, s);
-    else if (dk <= 128) ok = LaunchGdnChunk<T, 32, 32>(p, B, s);
-    else ok = LaunchGdnChunk<T, 64, 16>(p, B, s);
+    if (dk <= 32) ok = LaunchGdnChunk<T, 4, 32>(p, B, s);
+    else if (dk <= 64) ok = LaunchGdnChunk<T, 8, 32>(p, B, s);
+    else if (dk <= 128) ok = LaunchGdnChunk<T, 16, 32>(p, B, s);
+    else ok = LaunchGdnChunk<T, 32, 16>(p, B, s);
     return ok ? 0 : -4;
   }
   // measured at Qwen3.5 shapes: 32 rows per thread 51 us, 16 rows 63 us, 64 rows 54 us (64 requests)

@@ -448,7 +448,7 @@ class DecoderModel:
         if n_short > 0:
             qlat = ops.head_project(proj[:n_short], lw.lat_uk_t, sp.heads, sp.dim + sp.rot_dim)
             olat = ops.latent_attention(qlat, proj, shape, cache, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale, sp.window,
-                                        s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0)
+                                        s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0, order=s.attn_order)
             ops.head_project(olat, lw.lat_uv, sp.heads, sp.kv_rank, out=out[:n_short])
         if plan is not None and plan.rows > 0:
             ops.latent_attention_long(proj, shape, lw.lat_ukv, cache, plan, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale,

@@ -864,10 +864,10 @@ def choose_latent_splits(batch: int, row_tiles: int, max_kv_len: int, window: in
 
 
 def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0, max_q_len=1, max_kv_len=1,
-                     skip_q_len=0, splits=None):
+                     skip_q_len=0, splits=None, order=None):
     """Attention of every head over the shared latent rows: qlat [T, H * kv_rank] (queries with the key map folded in), the rotated
     query parts in proj.  window > 0: position p sees (p - window, p].  skip_q_len > 0: requests with at least that many tokens are
-    not computed (their rows are unspecified).  Returns [T, H * kv_rank]."""
+    not computed (their rows are unspecified).  order [B]: requests in the order in which their CTAs are issued.  Returns [T, H * kv_rank]."""
     _check_index("latent_attention", "block_table", block_table, cache.shape[0] // block_size, -1)
     if not qlat.is_cuda:
         return ref.latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window)
@@ -890,7 +890,7 @@ def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_tabl
     _lib.check(L.ogb_latent_attention(_ptr(qlat), _ptr(proj), proj.stride(0), _sh(shape), _ptr(cache), cache.stride(0), _ptr(cu_seqlens), _ptr(past_lens),
                                       _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale), int(window), B, T,
                                       int(max_q_len), int(skip_q_len), int(splits), _ptr(scratch), scratch.numel() if scratch is not None else 0,
-                                      _stream()), "latent_attention")
+                                      _ptr(order), _stream()), "latent_attention")
     if splits > 1:
         _lib.LAUNCH_COUNT += 1      # the combine kernel
     return out
