@@ -81,7 +81,7 @@ long long ogb_latent_scratch_bytes(int total_rows, int R, int splits);
 int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                          const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
                          void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
-                         long long scratch_bytes, const int32_t* order, void* stream);
+                         long long scratch_bytes, const int32_t* order, int* status, void* stream);
 int ogb_latent_attention_simt(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                               const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
                               void* out, float scale, int window, int B, int T, int skip_q_len, int fp32, void* stream);

@@ -6,7 +6,7 @@
 // Kernels:
 //   latent_prep_kernel   RMS norm of the latent and rotation of the key part into the cache; rotation of the queries' rotary parts.
 //   latent_mma_kernel    decode steps and short portions: one CTA = (request, up to 64 (token, head) rows, key split); tiles of 32
-//                        cache rows through cp.async double buffering serve as K (all columns) and as V (the first R columns) of
+//                        cache rows, one bulk copy per row into a double buffer, serve as K (all columns) and as V (the first R columns) of
 //                        warp-level MMAs; two CTAs share an SM (up to 16 rows of 576 columns), so that one's copies and softmax run
 //                        under the other's MMAs.  Like paged_attention_kernel (attention.cu) it is bound by the cache stream and its rows are
 //                        few; long prompts take the tensor-memory kernel (attention_tc.cu) on expanded keys and values instead.
@@ -70,28 +70,40 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ proj, 
 }
 
 // ------------------------------------------------------------------------------------ warp-MMA kernel
+// Contiguous copy global -> shared (16-byte aligned addresses, a multiple of 16 bytes), completion on an mbarrier.
+__device__ __forceinline__ void bulk_load(void* smem_dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(smem_u32(smem_dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+
 struct LatentParams {
   const __nv_bfloat16* qlat;      // [T, H, R]
   const __nv_bfloat16* proj;      // rotary query parts at row t, column h * (dim + rot) + dim
   int ldp, dim;
   const __nv_bfloat16* cache; int ldcache;
-  const int32_t *cu, *past, *table; int table_cols, block_size;
+  const int32_t *cu, *past, *table; int table_cols, block_size, block_shift;      // log2(block_size) or -1
   __nv_bfloat16* out;             // [T, H, R]
   float* part_o; float* part_ml;
   float scale;
   int window, B, H, R, rot, kp, pitch, splits, total_rows, skip_q_len;
   const int32_t* order;           // [B] requests in issue order (longest first), or null
+  int* status;                    // device status word (bounded waits)
 };
 
+constexpr int LAT_MAX_SPLITS = 32, LAT_MAX_SMEM = 226 * 1024;          // (some static shared memory beside the dynamic part)
 constexpr int LAT_BN = 32, LAT_THREADS = 256, LAT_PP = LAT_BN + 8, LAT_SP = LAT_BN + 4;   // keys per tile; pitches of P and score rows
 
 template <int MT>
 struct LatCfg {
   static constexpr int BM = MT * 16;
-  static constexpr int KH = MT == 4 ? 1 : 2;           // the score sums are divided over KH warps by columns of the rows
+  // The score sums are divided over KH warps by columns of the rows.  16 rows: every warp takes all keys and an eighth of the columns,
+  // its part of the queries stays in registers (the staged queries make room for the partial scores), a cache row is read once.
+  static constexpr int KH = MT == 4 ? 1 : (MT == 2 ? 2 : 8);
   static constexpr int TPR = LAT_THREADS / BM;         // threads of one row in the softmax
   static constexpr int KPT = LAT_BN / TPR;             // keys of each of them
-  static constexpr int smem(int pitch) { return (BM + 2 * LAT_BN) * pitch * 2 + BM * LAT_PP * 2 + KH * BM * LAT_SP * 4 + BM * 8 + 64; }
+  static constexpr int S_BYTES = KH * BM * LAT_SP * 4;
+  static constexpr int q_bytes(int pitch) { return MT == 1 && S_BYTES > BM * pitch * 2 ? S_BYTES : BM * pitch * 2; }
+  static constexpr int smem(int pitch) { return q_bytes(pitch) + 2 * LAT_BN * pitch * 2 + BM * LAT_PP * 2 + (MT == 1 ? 0 : S_BYTES) + BM * 8 + 64; }
 };
 
 template <int MT, int NTW>
@@ -100,11 +112,14 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
   constexpr int BM = Cfg::BM, KH = Cfg::KH, TPR = Cfg::TPR, KPT = Cfg::KPT;
   extern __shared__ __align__(128) uint8_t smem[];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);
-  __nv_bfloat16* sK = sQ + BM * p.pitch;               // [2][LAT_BN][pitch]
+  __nv_bfloat16* sK = sQ + Cfg::q_bytes(p.pitch) / 2;  // [2][LAT_BN][pitch]
   __nv_bfloat16* sP = sK + 2 * LAT_BN * p.pitch;       // [BM][LAT_PP]
-  float* sS = reinterpret_cast<float*>(sP + BM * LAT_PP);     // [KH][BM][LAT_SP] partial scores
-  float* sA = sS + KH * BM * LAT_SP;                   // [BM] factor of the old output; at the end the row sums
+  float* sS = MT == 1 ? reinterpret_cast<float*>(sQ) : reinterpret_cast<float*>(sP + BM * LAT_PP);     // [KH][BM][LAT_SP] partial scores
+  float* sA = MT == 1 ? reinterpret_cast<float*>(sP + BM * LAT_PP) : sS + KH * BM * LAT_SP;             // [BM] factor of the old output; at the end the row sums
   float* sM = sA + BM;                                 // [BM] at the end the row maxima
+  __shared__ uint64_t full[2];                         // a tile's rows (tile 0: and the queries) have landed
+  __shared__ int abort_flag;
+  volatile int* abort_p = &abort_flag;
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -129,43 +144,46 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
     return;
   }
   const int n_tiles = (hi - lo + LAT_BN - 1) / LAT_BN;
-  const int kc = (p.R + p.rot) / 8, rc = p.R / 8;      // 16-byte chunks of a cache row; of its latent
-  // A warp copies 4 rows of a tile; their cache slots are looked up one tile ahead of the copy, so that the copy does not wait for the
-  // table.  Rows past the range become zeros.
-  auto lookup = [&](int it) {
-    const int j = lo + it * LAT_BN + warp * 4 + (lane & 3);
-    return j < hi ? table[j / p.block_size] * p.block_size + j % p.block_size : -1;
-  };
-  auto load = [&](int it, int slot) {
-    __nv_bfloat16* dst = sK + ((it & 1) * LAT_BN + warp * 4) * p.pitch;
-#pragma unroll
-    for (int r = 0; r < 4; ++r) {
-      const int sl = __shfl_sync(0xffffffffu, slot, r);
-      const __nv_bfloat16* src = p.cache + (sl >= 0 ? size_t(sl) * p.ldcache : 0);
-      for (int c = lane; c < kc; c += 32) cp_async16(dst + r * p.pitch + c * 8, src + c * 8, sl >= 0);
-    }
-  };
-  // queries: latent part from qlat, rotary part from the projection
-  for (int idx = tid; idx < BM * kc; idx += LAT_THREADS) {
-    const int r = idx / kc, c = idx - r * kc, gr = row0 + r;
-    const bool ok = gr < rows;
-    const __nv_bfloat16* src = p.qlat;
-    if (ok) {
-      const size_t tr = size_t(tok0) * H + gr;
-      src = c < rc ? p.qlat + tr * p.R + c * 8 : p.proj + (tr / H) * p.ldp + size_t(gr % H) * (p.dim + p.rot) + p.dim + (c - rc) * 8;
-    }
-    cp_async16(sQ + r * p.pitch + c * 8, src, ok);
+  const int kc = (p.R + p.rot) / 8;                    // 16-byte chunks of a cache row
+  const uint32_t row_bytes = (p.R + p.rot) * 2;
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    abort_flag = 0;
+    mbar_fence_init();
   }
   if (kc * 8 < p.kp) {                                 // columns between the row's end and the next multiple of 16 are zeros
     for (int r = tid; r < BM; r += LAT_THREADS) *reinterpret_cast<uint4*>(sQ + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
     for (int r = tid; r < 2 * LAT_BN; r += LAT_THREADS) *reinterpret_cast<uint4*>(sK + r * p.pitch + kc * 8) = make_uint4(0, 0, 0, 0);
   }
-  int slot_next = -1;
-  if (n_tiles > 0) {
+  __syncthreads();
+  // Warp 0 copies a tile, one row per lane; the rows' blocks are looked up one tile ahead of the copy and not touched before it, so that
+  // it does not wait for the table.  Rows past the range repeat its last row (their weights are zero).
+  auto key_of = [&](int it) { return min(lo + it * LAT_BN + lane, hi - 1); };
+  auto lookup = [&](int it) {
+    const int j = key_of(it);
+    return table[p.block_shift >= 0 ? j >> p.block_shift : j / p.block_size];
+  };
+  auto load = [&](int it, int block) {
+    const int j = key_of(it);
+    const int slot = p.block_shift >= 0 ? (block << p.block_shift) + (j & (p.block_size - 1)) : block * p.block_size + j % p.block_size;
+    bulk_load(sK + ((it & 1) * LAT_BN + lane) * p.pitch, p.cache + size_t(slot) * p.ldcache, row_bytes, &full[it & 1]);
+  };
+  int block_next = 0;
+  if (warp == 0) {
+    if (lane == 0) mbar_expect_tx(&full[0], (BM + LAT_BN) * row_bytes);
+    __syncwarp();
+    // queries: latent part from qlat, rotary part from the projection; rows past the request's repeat its last one
+    for (int r = lane; r < BM; r += 32) {
+      const int gr = min(row0 + r, rows - 1);
+      const size_t tr = size_t(tok0) * H + gr;
+      bulk_load(sQ + r * p.pitch, p.qlat + tr * p.R, p.R * 2, &full[0]);
+      if (p.rot > 0)
+        bulk_load(sQ + r * p.pitch + p.R, p.proj + size_t(tok0 + gr / H) * p.ldp + size_t(gr % H) * (p.dim + p.rot) + p.dim, p.rot * 2, &full[0]);
+    }
     load(0, lookup(0));
-    slot_next = lookup(1);
+    block_next = lookup(1);
   }
-  cp_async_commit();
 
   // softmax: TPR neighbouring threads share row sr, KPT keys each
   const int sr = tid / TPR, sk0 = (tid % TPR) * KPT;
@@ -175,9 +193,10 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
   float mx = -INFINITY, l = 0.f;                       // the row's running maximum; the sum over this thread's keys
   // scores: warp -> 16 rows (mt), a group of keys (kg), a share of the columns (kh)
   const int ksteps = p.kp / 16;
-  const int mt = warp % MT, kg = MT == 1 ? warp & 3 : (warp / MT) & 1, kh = KH == 1 ? 0 : warp >> 2;
-  const int kmid = KH == 1 ? ksteps : (ksteps / 2 + 1) & ~1;                   // an even number of steps in the first share
-  const int ks0 = kh ? kmid : 0, ks1 = kh ? ksteps : kmid;
+  constexpr int KS = NTW == 8 ? 5 : (NTW == 4 ? 3 : 2);                        // column steps of a warp (16 rows), at most
+  const int mt = warp % MT, kg = (warp / MT) & 1, kh = KH == 8 ? warp : (KH == 2 ? warp >> 2 : 0);
+  const int ks0 = kh * ksteps / KH, ks1 = (kh + 1) * ksteps / KH;
+  uint32_t qreg[KS][4];
   const int c0 = warp * NTW * 8;                       // output columns [c0, c0 + 8 * NTW) of every row
   float o[MT][NTW][4];
 #pragma unroll
@@ -186,49 +205,54 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
     for (int n = 0; n < NTW; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
 
   for (int it = 0; it < n_tiles; ++it) {
-    cp_async_wait<0>();
-    __syncthreads();                                   // tile it has landed; every warp is done with tile it - 1
-    if (it + 1 < n_tiles) {
-      load(it + 1, slot_next);
-      slot_next = lookup(it + 2);
+    if (!mbar_wait_bounded(&full[it & 1], (it >> 1) & 1, abort_p)) {
+      *abort_p = 1;
+      if (p.status) atomicMax(p.status, int(OGB_ERR_WAIT_TMA));
     }
-    cp_async_commit();
+    __syncthreads();                                   // tile it has landed; every warp is done with tile it - 1
+    if (*abort_p) break;                               // (set before the barrier or not at all: all threads leave together)
+    if (warp == 0 && it + 1 < n_tiles) {
+      if (lane == 0) mbar_expect_tx(&full[(it + 1) & 1], LAT_BN * row_bytes);
+      __syncwarp();
+      load(it + 1, block_next);
+      block_next = lookup(it + 2);
+    }
     const __nv_bfloat16* tk = sK + (it & 1) * LAT_BN * p.pitch;
     const __nv_bfloat16* qa = sQ + (mt * 16 + (lane & 15)) * p.pitch + (lane >> 4) * 8;
     float* ps = sS + (kh * BM + mt * 16 + g) * LAT_SP + t4 * 2;
     if constexpr (MT == 1) {
-      // 16 rows x 8 keys; four accumulators: the MMAs of one sum would wait for each other
-      float s[4][4] = {};
-      const __nv_bfloat16* ka = tk + (kg * 8 + (lane & 7)) * p.pitch + (lane >> 3) * 8;
-      int ks = ks0;
-#pragma unroll 2
-      for (; ks + 4 <= ks1; ks += 4) {
-        uint32_t q0[4], q1[4], q2[4], q3[4], k0[4], k1[4];
-        ldmatrix_x4(k0, ka + ks * 16);
-        ldmatrix_x4(k1, ka + ks * 16 + 32);
-        ldmatrix_x4(q0, qa + ks * 16);
-        ldmatrix_x4(q1, qa + ks * 16 + 16);
-        ldmatrix_x4(q2, qa + ks * 16 + 32);
-        ldmatrix_x4(q3, qa + ks * 16 + 48);
-        mma_bf16_16816(s[0], q0, k0[0], k0[1]);
-        mma_bf16_16816(s[1], q1, k0[2], k0[3]);
-        mma_bf16_16816(s[2], q2, k1[0], k1[1]);
-        mma_bf16_16816(s[3], q3, k1[2], k1[3]);
+      // 16 rows x 32 keys over this warp's columns
+      if (it == 0) {
+#pragma unroll
+        for (int i = 0; i < KS; ++i) if (ks0 + i < ks1) ldmatrix_x4(qreg[i], qa + (ks0 + i) * 16);
+        __syncthreads();                               // the staged queries are no longer needed: the scores take their place
       }
-      for (; ks < ks1; ks += 2) {                      // (a last odd step reads 16 bytes past the row: the next row or P, unused)
-        uint32_t qf[4], kb[4];
-        ldmatrix_x4(kb, ka + ks * 16);
-        ldmatrix_x4(qf, qa + ks * 16);
-        mma_bf16_16816(s[0], qf, kb[0], kb[1]);
-        if (ks + 1 < ks1) {
-          ldmatrix_x4(qf, qa + ks * 16 + 16);
-          mma_bf16_16816(s[1], qf, kb[2], kb[3]);
+      float s[4][4] = {};
+      const __nv_bfloat16* ka = tk + ((lane >> 4) * 8 + (lane & 7)) * p.pitch + ((lane >> 3) & 1) * 8 + ks0 * 16;
+      // the next step's fragments are read ahead of this step's MMAs
+      uint32_t k0[2][4], k1[2][4];
+      if (ks0 < ks1) {
+        ldmatrix_x4(k0[0], ka);
+        ldmatrix_x4(k1[0], ka + 16 * p.pitch);
+      }
+#pragma unroll
+      for (int i = 0; i < KS; ++i) {
+        if (i + 1 < KS && ks0 + i + 1 < ks1) {
+          ldmatrix_x4(k0[(i + 1) & 1], ka + (i + 1) * 16);
+          ldmatrix_x4(k1[(i + 1) & 1], ka + 16 * p.pitch + (i + 1) * 16);
+        }
+        if (ks0 + i < ks1) {
+          mma_bf16_16816(s[0], qreg[i], k0[i & 1][0], k0[i & 1][1]);
+          mma_bf16_16816(s[1], qreg[i], k0[i & 1][2], k0[i & 1][3]);
+          mma_bf16_16816(s[2], qreg[i], k1[i & 1][0], k1[i & 1][1]);
+          mma_bf16_16816(s[3], qreg[i], k1[i & 1][2], k1[i & 1][3]);
         }
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[0][e] = (s[0][e] + s[1][e]) + (s[2][e] + s[3][e]);
-      *reinterpret_cast<float2*>(ps + kg * 8) = make_float2(s[0][0], s[0][1]);
-      *reinterpret_cast<float2*>(ps + 8 * LAT_SP + kg * 8) = make_float2(s[0][2], s[0][3]);
+      for (int n = 0; n < 4; ++n) {
+        *reinterpret_cast<float2*>(ps + n * 8) = make_float2(s[n][0], s[n][1]);
+        *reinterpret_cast<float2*>(ps + 8 * LAT_SP + n * 8) = make_float2(s[n][2], s[n][3]);
+      }
     } else {
       // 16 rows x 16 keys
       float s[2][2][4] = {};
@@ -260,7 +284,8 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
 #pragma unroll
     for (int e = 0; e < KPT; ++e) {
       float v = sS[sr * LAT_SP + sk0 + e];
-      if constexpr (KH == 2) v += sS[(BM + sr) * LAT_SP + sk0 + e];
+#pragma unroll
+      for (int k = 1; k < KH; ++k) v += sS[(k * BM + sr) * LAT_SP + sk0 + e];
       const int j = lo + it * LAT_BN + sk0 + e;
       x[e] = s_valid && j < hi && j <= s_pos && (p.window <= 0 || j > s_pos - p.window) ? v * sc2 : -INFINITY;
       tmax = fmaxf(tmax, x[e]);
@@ -283,6 +308,7 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const float al0 = sA[m * 16 + g], al1 = sA[m * 16 + g + 8];
+      if (!__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) continue;        // no maximum moved
 #pragma unroll
       for (int n = 0; n < NTW; ++n) { o[m][n][0] *= al0; o[m][n][1] *= al0; o[m][n][2] *= al1; o[m][n][3] *= al1; }
     }
@@ -291,20 +317,27 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
       uint32_t pa[MT][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m) ldmatrix_x4(pa[m], sP + (m * 16 + (lane & 15)) * LAT_PP + kk * 16 + (lane >> 4) * 8);
+      uint32_t vb[NTW / 2][4];                         // (all fragments first: an MMA would hold back the reads behind it)
+#pragma unroll
+      for (int np = 0; np < NTW / 2; ++np)
+        if (c0 + np * 16 < p.R) ldmatrix_x4_trans(vb[np], tk + (kk * 16 + (lane & 15)) * p.pitch + c0 + np * 16 + (lane >> 4) * 8);
 #pragma unroll
       for (int np = 0; np < NTW / 2; ++np) {
         if (c0 + np * 16 >= p.R) break;
-        uint32_t vb[4];
-        ldmatrix_x4_trans(vb, tk + (kk * 16 + (lane & 15)) * p.pitch + c0 + np * 16 + (lane >> 4) * 8);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          mma_bf16_16816(o[m][np * 2], pa[m], vb[0], vb[1]);
-          mma_bf16_16816(o[m][np * 2 + 1], pa[m], vb[2], vb[3]);
+          mma_bf16_16816(o[m][np * 2], pa[m], vb[np][0], vb[np][1]);
+          mma_bf16_16816(o[m][np * 2 + 1], pa[m], vb[np][2], vb[np][3]);
         }
       }
     }
   }
-  cp_async_wait<0>();
+  if (*abort_p) {                                      // a wait ran out: let copies in flight land before the shared memory goes away
+    int never = 0;
+    mbar_wait_bounded(&full[0], 0, &never, 20000000ull);
+    mbar_wait_bounded(&full[1], 0, &never, 20000000ull);
+    return;
+  }
 #pragma unroll
   for (int w = TPR / 2; w > 0; w >>= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
   __syncthreads();
@@ -340,27 +373,28 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
 // One CTA per (token, head) row: merges the split partials.
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                              __nv_bfloat16* __restrict__ out, int total_rows, int R, int splits) {
+  __shared__ float w[LAT_MAX_SPLITS];
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x;
-  float M = -INFINITY;
-  for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[(size_t(s) * total_rows + row) * 2]);
-  float L = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float* ml = part_ml + (size_t(s) * total_rows + row) * 2;
-    if (ml[0] != -INFINITY) L += exp2f(ml[0] - M) * ml[1];
+  const int row = blockIdx.x, lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {
+    float2 ml = make_float2(-INFINITY, 0.f);
+    if (lane < splits) ml = *reinterpret_cast<const float2*>(part_ml + (size_t(lane) * total_rows + row) * 2);
+    const float M = warp_max(ml.x);
+    const float e = ml.x == -INFINITY ? 0.f : exp2f(ml.x - M);
+    const float L = warp_sum(e * ml.y);
+    w[lane] = L > 0.f ? e / L : 0.f;
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  __syncthreads();
   for (int c = threadIdx.x * 4; c < R; c += 512) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
     for (int s = 0; s < splits; ++s) {
-      const float m = part_ml[(size_t(s) * total_rows + row) * 2];
-      if (m == -INFINITY) continue;
-      const float w = exp2f(m - M);
+      const float f = w[s];
       const float4 v = *reinterpret_cast<const float4*>(part_o + (size_t(s) * total_rows + row) * R + c);
-      a.x += w * v.x; a.y += w * v.y; a.z += w * v.z; a.w += w * v.w;
+      if (f != 0.f) { a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w; }      // (an empty split's values are not defined)
     }
-    *reinterpret_cast<uint2*>(out + size_t(row) * R + c) = make_uint2(pack_bf16x2(a.x * inv, a.y * inv), pack_bf16x2(a.z * inv, a.w * inv));
+    *reinterpret_cast<uint2*>(out + size_t(row) * R + c) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
   }
 }
 
@@ -458,7 +492,7 @@ template <int MT, int NTW>
 static int LaunchLatentMma(const LatentParams& p, int max_q_len, cudaStream_t s) {
   auto kern = latent_mma_kernel<MT, NTW>;
   static bool configured[OGB_MAX_DEVICES] = {};
-  if (!set_max_dyn_smem(kern, 227 * 1024, configured)) return -3;
+  if (!set_max_dyn_smem(kern, LAT_MAX_SMEM, configured)) return -3;
   const dim3 grid((max_q_len * p.H + MT * 16 - 1) / (MT * 16), 1, p.B * p.splits);
   if (!launch_pdl(kern, grid, dim3(LAT_THREADS), LatCfg<MT>::smem(p.pitch), s, p)) return -4;
   if (p.splits > 1 && !launch_pdl(latent_combine_kernel, dim3(p.total_rows), dim3(128), 0, s, static_cast<const float*>(p.part_o),
@@ -494,7 +528,7 @@ OGB_API int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const
 
 // 1 when the warp-MMA kernel can address these sizes (16-byte pieces everywhere, the tile fits in shared memory).
 OGB_API int ogb_latent_mma_supported(const OgbLatentShape* sh) {
-  return sh->R % 8 == 0 && sh->rot % 8 == 0 && sh->dim % 8 == 0 && sh->R >= 8 && sh->R <= 512 && LatCfg<1>::smem(lat_pitch(sh)) <= 227 * 1024;
+  return sh->R % 8 == 0 && sh->rot % 8 == 0 && sh->dim % 8 == 0 && sh->R >= 8 && sh->R <= 512 && sh->rot <= 128 && LatCfg<1>::smem(lat_pitch(sh)) <= LAT_MAX_SMEM;
 }
 
 // Rows of (token, head) a CTA takes for requests of at most max_q_len tokens.
@@ -511,28 +545,30 @@ OGB_API long long ogb_latent_scratch_bytes(int total_rows, int R, int splits) {
 OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                                  const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
                                  void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
-                                 long long scratch_bytes, const int32_t* order, void* stream) {
+                                 long long scratch_bytes, const int32_t* order, int* status, void* stream) {
   if (B <= 0 || T <= 0 || max_q_len <= 0) return 0;
   if (!ogb_latent_mma_supported(sh)) return -5;
   if ((ldp % 8) || (ldcache % 8) || block_size <= 0) return -1;
   if ((reinterpret_cast<uintptr_t>(qlat) | reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) return -1;
-  if (splits < 1) splits = 1;
+  splits = splits < 1 ? 1 : (splits > LAT_MAX_SPLITS ? LAT_MAX_SPLITS : splits);
   const int rows = T * sh->H;
   if (ogb_latent_scratch_bytes(rows, sh->R, splits) > scratch_bytes || (long long)B * splits > 65535) return -2;
   LatentParams p;
   p.qlat = static_cast<const __nv_bfloat16*>(qlat); p.proj = static_cast<const __nv_bfloat16*>(proj); p.ldp = ldp; p.dim = sh->dim;
   p.cache = static_cast<const __nv_bfloat16*>(cache); p.ldcache = ldcache;
   p.cu = cu_seqlens; p.past = past_lens; p.table = block_table; p.table_cols = table_cols; p.block_size = block_size;
+  p.block_shift = -1;
+  for (int k = 0; k < 16; ++k) if (block_size == 1 << k) p.block_shift = k;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = static_cast<float*>(scratch);
   p.part_ml = p.part_o ? p.part_o + size_t(splits) * rows * sh->R : nullptr;
   p.scale = scale; p.window = window; p.B = B; p.H = sh->H; p.R = sh->R; p.rot = sh->rot;
   p.kp = (sh->R + sh->rot + 15) / 16 * 16; p.pitch = lat_pitch(sh);
-  p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len; p.order = order;
+  p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len; p.order = order; p.status = status;
   auto s = static_cast<cudaStream_t>(stream);
   int bm = ogb_latent_rows_per_tile(sh->H, skip_q_len > 0 && skip_q_len - 1 < max_q_len ? skip_q_len - 1 : max_q_len);
-  if (bm == 64 && LatCfg<4>::smem(p.pitch) > 227 * 1024) bm = 32;
-  if (bm == 32 && LatCfg<2>::smem(p.pitch) > 227 * 1024) bm = 16;
+  if (bm == 64 && LatCfg<4>::smem(p.pitch) > LAT_MAX_SMEM) bm = 32;
+  if (bm == 32 && LatCfg<2>::smem(p.pitch) > LAT_MAX_SMEM) bm = 16;
   if (skip_q_len > 0 && max_q_len > skip_q_len - 1) max_q_len = skip_q_len - 1;
   if (max_q_len <= 0) return 0;
   if (bm == 16) return LaunchLatentMt<1>(p, max_q_len, s);

@@ -82,7 +82,7 @@ _SIGS = {
     "ogb_latent_rows_per_tile": (c_int, [c_int, c_int]),
     "ogb_latent_scratch_bytes": (c_longlong, [c_int, c_int, c_int]),
     "ogb_latent_attention": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
-                                     _P, c_longlong, _P, _P]),
+                                     _P, c_longlong, _P, _P, _P]),
     "ogb_latent_attention_simt": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_latent_gather": (c_int, [_P, c_int, _P, c_int, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P, c_int, _P]),
     "ogb_attention_tc_latent_supported": (c_int, [c_int, c_int, c_int]),
