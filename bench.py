@@ -397,6 +397,26 @@ def ours(args):
     return 0
 
 
+def design_arm(args):
+    """Throughput of a declared-stack design beside the closest other model at equal size (not the headline workload)."""
+    import torch
+    from benchmark import stack_bench
+    torch.cuda.set_device(0)
+
+    class Sampler:      # one nvidia-smi process per measured model
+        def start(self):
+            self.s = ClockSampler(0)
+            self.s.start()
+
+        def stop(self):
+            return self.s.stop()
+    res = stack_bench.run(Sampler(), args.steps, max(3, args.warmup), args.design_sizes.split(",") if args.design_sizes else None)
+    print(json.dumps({"metric": "prefill_and_decode_tokens_per_s", "design": args.design, "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup),
+                      "dtype": "bf16", "data": "synthetic (random token ids, random weights drawn on the device)",
+                      "config": {"l2": "weights and caches larger than L2, no flush"}, "sizes": res}))
+    return 0
+
+
 def st_bytes(engine):
     return engine.staging.h2d_bytes
 
@@ -420,7 +440,12 @@ def main():
     ap.add_argument("--precision", default="bf16", choices=["bf16", "int4"],
                     help="weights of the checkpoint: bf16 (headline) or 4-bit (int4 block-32 linears; gpt-oss experts as packed MXFP4, the form "
                          "the reference publishes its gpt-oss numbers for); activations and the KV cache stay bf16")
+    ap.add_argument("--design", default="", choices=["", "luzatar"],
+                    help="measure this declared-stack design beside the closest other model at equal size instead of the headline workload")
+    ap.add_argument("--design_sizes", default="", help="comma-separated sizes of --design (default: all)")
     args = ap.parse_args()
+    if args.design:
+        return design_arm(args)
     if args.impl == "reference":
         return reference_arm(args)
     return ours(args)

@@ -1,0 +1,133 @@
+"""Prefill and decode throughput of a declared stack (Luzatar) beside the closest other model of the framework at equal size: the
+gated-delta-net + full-attention hybrid (Qwen3.5 style) with the same width, feed-forward, layer count, delta layers and attention
+heads.  Random weights drawn on the device; CUDA events around whole decoder forwards (decode steps replay a CUDA graph); the weights
+and caches of a step are larger than L2.  Reached through `python bench.py --design luzatar`."""
+import json
+import os
+import shutil
+import tempfile
+
+import numpy as np
+import torch
+
+SIZES = {
+    # name: width, ff, layers (alternating delta / attention), attention heads, kv heads of the hybrid, delta key heads, delta value heads
+    "2k": dict(width=2048, ff=6144, layers=16, heads=16, kv=4, dk=8, dv=16, vocab=65536),
+    "4k": dict(width=4096, ff=12288, layers=8, heads=32, kv=8, dk=16, dv=32, vocab=65536),
+}
+PREFILL = [(1, 4096), (8, 1024)]
+DECODE = [(1, 2048), (16, 2048), (64, 2048), (256, 1024)]
+BLOCK = 16
+
+
+def luzatar_dir(z, path):
+    delta = dict(type="delta", mixer=dict(heads=z["dv"], kv_heads=z["dk"], dim=128, vdim=128, conv=4), mlp=dict(kind="dense", ff=z["ff"]))
+    lat = dict(type="latent_attention", mixer=dict(heads=z["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, mask=dict(size=8192),
+                                                   rot=dict(base=1e6, dims=64)), mlp=dict(kind="dense", ff=z["ff"]))
+    cfg = dict(architecture="Luzatar", layers=[delta, lat] * (z["layers"] // 2), norm=dict(eps=1e-6), vocab=z["vocab"], width=z["width"])
+    os.makedirs(os.path.join(path, "src"), exist_ok=True)
+    with open(os.path.join(path, "src", "config.json"), "w") as f:
+        json.dump(cfg, f)
+    from onnxruntime_genai_b200.models.builder import create_model
+    return create_model(os.path.join(path, "src"), os.path.join(path, "model"), "bf16", "cuda", {"synthetic_weights": 1, "context_length": 8192})
+
+
+def hybrid_dir(z, path):
+    from onnxruntime_genai_b200.models.arch import ArchConfig
+    from onnxruntime_genai_b200.models.builder import export_model
+    a = ArchConfig(model_type="qwen3_next", vocab_size=z["vocab"], hidden_size=z["width"], num_layers=z["layers"], num_heads=z["heads"],
+                   num_kv_heads=z["kv"], head_dim=128, intermediate_size=z["ff"], context_length=8192, bos_token_id=0, eos_token_id=1, pad_token_id=0,
+                   layer_types=["linear_attention", "full_attention"] * (z["layers"] // 2), linear_num_key_heads=z["dk"], linear_num_value_heads=z["dv"],
+                   linear_key_head_dim=128, linear_value_head_dim=128, linear_conv_kernel_dim=4)
+    return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
+
+
+def _step(model, lens):
+    """(StepInputs, cache) of a step with the given (past, new) lengths over fresh zero caches."""
+    from onnxruntime_genai_b200.models.decoder import PagedKVCache, StepInputs
+    dec = model.decoder
+    nb = [(p + n + BLOCK - 1) // BLOCK for p, n in lens]
+    kv = PagedKVCache(dec.arch, sum(nb), BLOCK, "cuda", dec.dtype, kv_heads=dec.kv_heads_local, conv_channels=dec.conv_channels_local)
+    kv.ensure_state_slots(len(lens))
+    for pool in (kv.full, kv.conv, kv.latent, kv.state):
+        if pool is not None and pool.numel():
+            pool.normal_(0, 0.1)
+    table = np.zeros((len(lens), max(nb)), dtype=np.int32)
+    at, pos, slots = 0, [], []
+    for b, (p, n) in enumerate(lens):
+        table[b, :nb[b]] = np.arange(at, at + nb[b])
+        q = np.arange(p, p + n)
+        pos.append(q)
+        slots.append(at * BLOCK + q)
+        at += nb[b]
+    t = lambda x: torch.from_numpy(np.asarray(x, dtype=np.int32)).cuda()
+    cu = np.cumsum([0] + [n for _, n in lens])
+    ids = np.random.RandomState(1).randint(0, dec.arch.vocab_size, int(cu[-1]))
+    s = StepInputs(input_ids=t(ids), positions=t(np.concatenate(pos)), slot_mapping=t(np.concatenate(slots)), cu_seqlens=t(cu),
+                   past_lens=t([p for p, _ in lens]), block_table=t(table), logits_rows=t(cu[1:] - 1), max_q_len=max(n for _, n in lens),
+                   max_kv_len=max(p + n for p, n in lens), min_q_len=min(n for _, n in lens), host_lens=list(lens),
+                   state_slots=t(np.arange(len(lens))))
+    return s, kv
+
+
+def _time(fn, iters, warmup=3):
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(iters):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / iters
+
+
+def measure(model, steps, warmup):
+    from onnxruntime_genai_b200 import ops
+    from onnxruntime_genai_b200.ops import _lib
+    out = {}
+    with torch.no_grad():
+        for n, length in PREFILL:
+            s, kv = _step(model, [(0, length)] * n)
+            ms = _time(lambda: model.decoder.forward(s, kv), max(3, steps // 10), warmup)
+            out[f"prefill {n}x{length}"] = {"ms": round(ms, 3), "tokens_per_s": round(n * length / ms * 1e3)}
+            del s, kv
+        for n, past in DECODE:
+            s, kv = _step(model, [(past, 1)] * n)
+            model.decoder.forward(s, kv)
+            torch.cuda.synchronize()
+            before = _lib.LAUNCH_COUNT
+            g = torch.cuda.CUDAGraph()
+            with ops.graph_capture(g):
+                model.decoder.forward(s, kv)
+            launches = _lib.LAUNCH_COUNT - before
+            ms = _time(g.replay, steps, warmup)
+            out[f"decode {n} at {past}"] = {"ms": round(ms, 4), "tokens_per_s": round(n / ms * 1e3), "launches": launches}
+            del g, s, kv
+    ops.check_kernel_status()
+    torch.cuda.empty_cache()
+    return out
+
+
+def run(sampler, steps=50, warmup=3, sizes=None):
+    import onnxruntime_genai_b200 as og
+    result = {}
+    for name in sizes or SIZES:
+        z = SIZES[name]
+        result[name] = {"shape": z}
+        for label, make in (("luzatar", luzatar_dir), ("hybrid", hybrid_dir)):
+            d = tempfile.mkdtemp(prefix="ogb_stack_")
+            try:
+                model = og.Model(make(z, d))
+                sampler.start()
+                result[name][label] = measure(model, steps, warmup)
+                result[name][label]["clocks"] = sampler.stop()
+                result[name][label]["weight_gb"] = round(model.decoder.weight_bytes() / 1e9, 2)
+                del model
+            finally:
+                shutil.rmtree(d, ignore_errors=True)
+            torch.cuda.empty_cache()
+        pairs = [k for k in result[name]["luzatar"] if isinstance(result[name]["luzatar"][k], dict) and "ms" in result[name]["luzatar"][k]]
+        result[name]["time ratio luzatar / hybrid"] = {k: round(result[name]["luzatar"][k]["ms"] / result[name]["hybrid"][k]["ms"], 3) for k in pairs}
+    return result
