@@ -865,7 +865,11 @@ OGB_API int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_col
   if ((a_cols % 8) || (lda % 8) || (ldw % 8)) return -1;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -1;
   static const int pdl_enabled = [] { const char* e = getenv("OGB_PDL"); return (e && e[0] == '0') ? 0 : 1; }();
-  const int bt = ogb_gemm_token_tile(M, 0);
+  // The problems are small (a head's weight is a few tiles and a short K): the token tile shrinks until the launch covers the SMs, which
+  // divides the epilogues, the longest part of such a CTA.
+  int bt = min(128, ogb_gemm_token_tile(M, 0));         // (two CTAs per SM)
+  const long long wide = (long long)((N + GEMM_BLOCK_N - 1) / GEMM_BLOCK_N) * batch;
+  while (bt > 16 && wide * ((M + bt - 1) / bt) < ogb_sm_count_current()) bt /= 2;
   CUtensorMap tw, ta;
   if (!MakeMap(&tw, W, batch * N, K, ldw, GEMM_BLOCK_N)) return -2;
   if (!MakeMap(&ta, A, M, a_width, lda, bt)) return -2;
