@@ -49,7 +49,7 @@ MIXED = stack([delta(), latent(scale=0.5), latent(heads=5, window=7, scaled=Fals
 ODD = stack([latent(heads=1, dim=9, rot_dim=6, vdim=5, kv_rank=11, window=3, ff=13, scale=0.8), delta(heads=3, kv_heads=3, dim=7, vdim=5, conv=1, ff=0),
              delta(heads=1, kv_heads=1, dim=3, vdim=7, conv=6, ff=21)], vocab=37, width=45, eps=2e-2)
 # sizes that take the tensor-core and warp-MMA kernels of both attention forms, every kernel instantiation class of the recurrence
-WIDE = stack([latent(heads=4, dim=64, rot_dim=16, vdim=64, kv_rank=96, window=50, ff=128, scale=0.25), delta(heads=4, kv_heads=2, dim=64, vdim=48, ff=192),
+WIDE = stack([latent(heads=4, dim=56, rot_dim=24, vdim=64, kv_rank=88, window=50, ff=128, scale=0.25), delta(heads=4, kv_heads=2, dim=64, vdim=48, ff=192),
               latent(heads=9, dim=104, rot_dim=32, vdim=80, kv_rank=200, window=130, ff=64, scale=0.2, original=64),
               latent(heads=3, dim=136, rot_dim=64, vdim=128, kv_rank=384, window=33, ff=0, scale=0.2), delta(heads=2, kv_heads=1, dim=128, vdim=64, ff=64)],
              vocab=160, width=128)
@@ -287,7 +287,7 @@ def test_delta_recurrence_kernels(dt, Hk, Hv, dk, dv):
     assert (state[:, Hv * dk * dv:] == 99).all() and (state[1] == 99).all() and (state[2] == 99).all()
 
 
-SHAPES = [(3, 40, 8, 24, 48, 8), (1, 9, 6, 5, 11, 6), (6, 64, 16, 64, 128, 16), (17, 24, 32, 16, 256, 20), (4, 128, 64, 128, 512, 64), (40, 16, 8, 16, 40, 0)]
+SHAPES = [(3, 40, 8, 24, 48, 8), (1, 9, 6, 5, 11, 6), (5, 80, 24, 56, 112, 24), (17, 24, 32, 16, 256, 20), (4, 128, 64, 128, 512, 64), (40, 16, 8, 16, 40, 0)]
 
 
 def _latent_case(shape, lens, window, seed, dt, needles=()):
@@ -371,7 +371,7 @@ def test_latent_attention_over_pages(runtime, shape, window):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("shape", [(2, 64, 16, 64, 128, 16), (3, 40, 8, 24, 48, 8), (2, 128, 64, 128, 256, 64), (2, 72, 32, 104, 136, 32), (2, 192, 64, 128, 512, 64),
+@pytest.mark.parametrize("shape", [(2, 64, 24, 64, 144, 24), (3, 40, 8, 24, 48, 8), (2, 128, 64, 128, 256, 64), (2, 72, 32, 104, 136, 32), (2, 192, 64, 128, 512, 64),
                                    (2, 136, 8, 56, 64, 8)], ids=lambda s: "x".join(map(str, s)))
 @pytest.mark.parametrize("window", [0, 1, 33, 200])
 def test_latent_attention_of_long_prompts_on_expanded_keys(shape, window):
@@ -388,7 +388,7 @@ def test_window_edges_with_keys_that_stand_out(runtime, window, form):
     the same for the sequence's first tokens and at page borders."""
     if form == "long" and runtime != ("cuda", "bfloat16"):
         pytest.skip("the expanded form exists in bf16 on the GPU")
-    shape = (2, 64, 16, 64, 128, 16)
+    shape = (2, 56, 24, 64, 120, 24)
     for q in (window - 1, window, 64, 79, 80, 127):
         for dist in (0, 1, window - 1, window, window + 1):
             key = q - dist
