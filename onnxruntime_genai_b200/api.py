@@ -574,16 +574,10 @@ class SequenceState:
 
     def _flush_block_moves(self):
         if self._moves:
-            bs = self.block_size
             dev = self.kv.full.device
             src = torch.tensor([m[0] for m in self._moves], dtype=torch.int64, device=dev)
             dst = torch.tensor([m[1] for m in self._moves], dtype=torch.int64, device=dev)
-            ar = torch.arange(bs, device=dev)
-            s_idx, d_idx = (src[:, None] * bs + ar).reshape(-1), (dst[:, None] * bs + ar).reshape(-1)
-            self.kv.full[:, :, d_idx] = self.kv.full[:, :, s_idx]
-            for pool in (self.kv.conv, self.kv.latent):
-                if pool is not None:
-                    pool[:, d_idx] = pool[:, s_idx]
+            self.kv.copy_blocks(src, dst)
             self._moves = []
         if self._tbl_dirty:
             self.block_table.copy_(torch.from_numpy(self._tbl))

@@ -32,9 +32,9 @@ C_API_SO = os.path.join(C_API_DIR, "libogb200_genai.so")
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v"]
-# Sources compiled without --use_fast_math: recurrences, 32-bit models and the norms of an fp32 residual stream keep IEEE division,
+# Sources compiled without --use_fast_math: recurrences, routers, 32-bit models and the norms of an fp32 residual stream keep IEEE division,
 # square roots and denormals.
-PRECISE_SOURCES = {"gemm_simt.cu", "latent_attention.cu", "layer_ops.cu", "linear_attention.cu"}
+PRECISE_SOURCES = {"attention_simt.cu", "gemm_simt.cu", "latent_attention.cu", "layer_ops.cu", "linear_attention.cu", "moe.cu"}
 
 
 def _newer(sources, target) -> bool:

@@ -84,7 +84,8 @@ struct GemmParams {
   int ldc;
   int out_fp32;         // 0 bf16, 1 fp32, 2 fp16 output
   int act_pair;         // tiles hold 64 gate rows + 64 up rows, output has N/2 columns: 1 = silu(gate)*up,
-                        // 2 = clamped SwiGLU: g = min(gate, limit), u = clamp(up, +-limit), g*sigmoid(alpha*g)*(u+1)
+                        // 2 = clamped SwiGLU: g = min(gate, limit), u = clamp(up, +-limit), g*sigmoid(alpha*g)*(u+1),
+                        // 3 = max(gate, 0)*up, 4 = gelu_tanh(gate)*up
                         // 3 = max(gate, 0)*up
   float act_alpha, act_limit;
   const void* residual;
@@ -136,6 +137,8 @@ __device__ __forceinline__ uint32_t pack_f16x2(float a, float b) {
 }
 
 __device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+// 0.5 x (1 + tanh(y)) = x sigmoid(2 y), y = sqrt(2 / pi) (x + 0.044715 x^3)
+__device__ __forceinline__ float gelu_tanh(float x) { return x / (1.f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x))); }
 
 __device__ __forceinline__ uint32_t cluster_ctarank() { uint32_t r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }
 __device__ __forceinline__ void cluster_sync_all() {
@@ -433,6 +436,9 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, uint8_t* smem
         } else if (p.act_pair == 3) {
 #pragma unroll
           for (int j = 0; j < 8; ++j) v[j] = fmaxf(v[j], 0.f) * u[j];
+        } else if (p.act_pair == 4) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[j] = gelu_tanh(v[j]) * u[j];
         } else {
 #pragma unroll
           for (int j = 0; j < 8; ++j) {

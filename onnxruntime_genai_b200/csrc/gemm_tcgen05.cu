@@ -540,6 +540,9 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const
             } else if (p.act_pair == 3) {
 #pragma unroll
               for (int q = 0; q < 8; ++q) v[q] = fmaxf(v[q], 0.f) * u[q];
+            } else if (p.act_pair == 4) {
+#pragma unroll
+              for (int q = 0; q < 8; ++q) v[q] = gelu_tanh(v[q]) * u[q];
             } else {
 #pragma unroll
               for (int q = 0; q < 8; ++q) {
@@ -747,7 +750,7 @@ OGB_API long long ogb_comm_capacity(int device) {
 // interleaved in blocks of 64); bit 2: fused all-reduce over the registered symmetric buffers; bit 3: fused
 // reduce-scatter by token rows instead (rank r ends up with rows [r * ceil(M / world), ...) of the sum, written as
 // rows 0.. of C; residual, if given, is that slice too); bit 4: activations gathered from the ranks' pushes; bit 5: the residual
-// is fp32; bit 6: the paired activation is max(gate, 0) * up.
+// is fp32; bit 6: the paired activation is max(gate, 0) * up; bit 7: it is gelu_tanh(gate) * up.
 OGB_API int ogb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
                           const void* bias, const void* residual, int ldr, int flags, int splits, int device, int* status,
                           int sm_count, void* stream_) {
@@ -788,9 +791,9 @@ OGB_API int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, 
   GemmParams p = {};
   p.M = M; p.N = N; p.K = K;
   p.splits = splits; p.kb_per_split = kb_per; p.total_kb = total_kb;
-  p.C = C; p.ldc = ldc; p.out_fp32 = out_fp32; p.act_pair = act_pair ? ((flags >> 6) & 1 ? 3 : 1) : 0;
+  p.C = C; p.ldc = ldc; p.out_fp32 = out_fp32; p.act_pair = act_pair ? ((flags >> 6) & 1 ? 3 : ((flags >> 7) & 1 ? 4 : 1)) : 0;
   p.residual = residual; p.ldr = ldr; p.res_fp32 = (flags >> 5) & 1;
-  if ((p.res_fp32 || p.act_pair == 3) && fused_ar) return -1;      // the reductions carry bf16 rows
+  if ((p.res_fp32 || p.act_pair >= 3) && fused_ar) return -1;      // the reductions carry bf16 rows
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.status = status;
   p.pdl = pdl_enabled;

@@ -55,10 +55,27 @@ int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const
 int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K, int batch,
                   const float* residual, int ldr, int in_fp32, int out_fp32, void* stream);
 
+// Grouped expert product over token rows sorted by expert in plain arithmetic (tile list of ogb_moe_sort, tiles of at most 64 rows).
+int ogb_moe_gemm_simt(const void* A, int lda, const void* W, void* C, int ldc, int N, int K, const int32_t* tile_expert, const int32_t* tile_row0,
+                      const int32_t* tile_rows, const int32_t* num_tiles, int max_tiles, int token_tile, const int32_t* row_map, int fp32, void* stream);
+
 // ---- layer_ops.cu: fp32 residual stream
-int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, int T, int H, int vocab, float scale, void* stream);
+// (copy, may be null: the rows as bf16 beside the stream)
+int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, void* copy, int T, int H, int vocab, float scale, void* stream);
 int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const float* b, void* out, int out_fp32, int n_rows, int H, float eps,
                     int layernorm, void* stream);
+// Head norms, rotation and cache append of an attention layer: proj row t holds Hq query heads and Hkv key heads of key_row columns (the
+// first `dim` are the head, the rest zeros) and Hkv value heads of value_row columns.  Queries are replaced in place, keys and values go to
+// row slots[t] of the caches (slot < 0: nowhere).  Norm weights fp32 [dim] (null: no norm), cos / sin fp32 [max_pos, rot / 2] (rot 0: none).
+int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
+                 const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
+                 void* v_cache, int T, int fp32, void* stream);
+// h[t] += w * v / sqrt(mean(v^2) + eps), x[t] = h[t] as bf16 (x may be null).  v = y[t], or (inv_pos not null) the weighted sum of the
+// experts' rows sum_j topk_w[t, j] * y[inv_pos[t, j]], j < k.
+int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const float* w, float eps, void* x, const int32_t* inv_pos, const float* topk_w, int k,
+                   int T, int H, void* stream);
+// Expert activations on rows of alternating (gate, up) columns [n, 2 I]: kind 0 silu(g) * u, 1 clamped g * sigmoid(alpha g) * (u + 1).
+int ogb_expert_act(const void* gu, void* out, long long n, int I, int kind, float alpha, float limit, int fp32, void* stream);
 int ogb_act_mul_rows(const void* x, int ldx, void* out, int ldo, int T, int I, int act, int fp32, void* stream);
 int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const void* bias, void* cache, int ldcache, const int32_t* slots,
                          const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols,
@@ -70,6 +87,25 @@ int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldk
                             const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* row_base, const int32_t* first_kv, void* out,
                             int out_stride, float scale, int window, int B, int max_q_len, int H, int dim, int rot, int vdim, int* status,
                             void* stream);
+
+// ---- attention_mixed.cu, attention_tc_mixed.cu, attention_simt.cu: attention layers with sizes of their own.  Hq query heads over Hkv key /
+// value heads (q rows: Hq heads of dk columns first; caches [slots, Hkv, dk] and [slots, Hkv, dv]; out rows: Hq heads of dv columns).
+// window > 0: position p sees (p - window, p]; chunk > 0: the keys of p's own run of `chunk` positions; 0: every earlier key.
+// sinks (may be null) [Hq]: a logit in each head's denominator.  gate (may be null) [tokens, gate_stride], in the model's element type: a
+// head's output is multiplied by the sigmoid of its entry.
+typedef struct OgbAttnLayer { int Hq, Hkv, dk, dv, window, chunk, gate_stride; float scale; const float* sinks; const void* gate; } OgbAttnLayer;
+int ogb_attention_mixed_supported(int dk, int dv);
+int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
+                        const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
+                        int total_tokens, int max_q_len, int splits, int kv_chunk, void* scratch, long long scratch_bytes, const int32_t* order,
+                        int* status, void* stream, int skip_rows);
+int ogb_attention_tc_mixed_supported(int dk, int dv, int block_size, int cache_slots);
+int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
+                           const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
+                           int max_q_len, int min_rows, int cache_slots, int* status, void* stream);
+int ogb_attention_simt(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
+                       const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B, int T,
+                       int fp32, void* stream);
 
 // ---- latent_attention.cu: attention over a paged cache of latent rows [c (R) | rotated key (rot)]
 typedef struct OgbLatentShape { int H, dim, rot, vdim, R, rot_dims; } OgbLatentShape;

@@ -1,7 +1,8 @@
 // Per-token kernels of the models that keep their residual stream in fp32, for bf16 and fp32 activations and any width:
 //   embedding rows into the fp32 stream; RMS / layer norm of stream rows (optionally of selected rows only: the rows whose logits
-//   are wanted); the gated activation act(gate) * up between two strided matrices; the causal depthwise convolution over the paged
-//   window of earlier inputs.  Built without fast-math: the fp32 models are the exact form of the same code.
+//   are wanted); the norm of a sub-layer's output added to the stream (with the weighted sum of routed experts folded in); head norms,
+//   rotation and cache append of attention projections; the gated activation act(gate) * up between two strided matrices and the experts'
+//   form of it; the causal depthwise convolution over the paged window of earlier inputs.  Built without fast-math: the fp32 models are the exact form of the same code.
 #include "common.cuh"
 #include "kernels.h"
 
@@ -16,13 +17,17 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 
 // ------------------------------------------------------------------------------------ embedding into the fp32 stream
 template <typename T>
-__global__ void embedding_stream_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int H, int vocab,
-                                        float scale) {
+__global__ void embedding_stream_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
+                                        __nv_bfloat16* __restrict__ copy, int H, int vocab, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = min(max(ids[t], 0), vocab - 1);
-  for (int i = threadIdx.x; i < H; i += blockDim.x) out[size_t(t) * H + i] = to_f32(table[size_t(id) * H + i]) * scale;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = to_f32(table[size_t(id) * H + i]) * scale;
+    out[size_t(t) * H + i] = v;
+    if (copy) copy[size_t(t) * H + i] = f2bf(v);
+  }
 }
 
 // ------------------------------------------------------------------------------------ norm of the fp32 stream
@@ -90,6 +95,219 @@ __global__ void __launch_bounds__(256) norm_stream_kernel(const float* __restric
   }
 }
 
+// ------------------------------------------------------------------------------------ normed output of a sub-layer, added to the stream
+// One CTA per token.  The sub-layer's row v is y[t], or the weighted sum of the experts' rows that served the token (inv_pos: their rows in
+// y, topk_w: their weights, in the order of the choice).  h[t] += w * v / sqrt(mean(v^2) + eps); x[t]: the new row as bf16 (may be null).
+constexpr int ADN_VEC = 8, ADN_KEEP = 4;      // columns per piece, pieces a thread keeps in registers
+struct AddNormed {
+  float* h; const float* w; __nv_bfloat16* x;
+  const int32_t* inv_pos; const float* topk_w;
+  int k, ldy, H;
+  float eps;
+};
+
+template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 q = *reinterpret_cast<const uint4*>(p);
+  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y), c = unpack_bf16x2(q.z), d = unpack_bf16x2(q.w);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y; v[4] = c.x; v[5] = c.y; v[6] = d.x; v[7] = d.y;
+}
+
+template <typename T>
+__device__ __forceinline__ float add_normed_col(const AddNormed& p, const T* y, int t, int i) {
+  if (!p.inv_pos) return to_f32(y[size_t(t) * p.ldy + i]);
+  float v = 0.f;
+  for (int j = 0; j < p.k; ++j) {
+    const int r = p.inv_pos[size_t(t) * p.k + j];
+    if (r >= 0) v = fmaf(p.topk_w[size_t(t) * p.k + j], to_f32(y[size_t(r) * p.ldy + i]), v);
+  }
+  return v;
+}
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) add_normed_kernel(const T* __restrict__ y, AddNormed p) {
+  __shared__ float part[8];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  float sq = 0.f;
+  auto inv_rms = [&]() {
+    sq = warp_sum(sq);
+    if (lane == 0) part[warp] = sq;
+    __syncthreads();
+    float s = 0.f;
+    for (int i = 0; i < nw; ++i) s += part[i];
+    return 1.f / sqrtf(s / p.H + p.eps);
+  };
+  if constexpr (VEC) {
+    const int nv = p.H / ADN_VEC;
+    float v[ADN_KEEP][ADN_VEC];
+#pragma unroll
+    for (int c = 0; c < ADN_KEEP; ++c) {
+      const int i = c * blockDim.x + threadIdx.x;
+      if (i >= nv) break;
+      if (!p.inv_pos) {
+        load8(y + size_t(t) * p.ldy + i * ADN_VEC, v[c]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < ADN_VEC; ++e) v[c][e] = 0.f;
+        for (int j = 0; j < p.k; ++j) {
+          const int r = p.inv_pos[size_t(t) * p.k + j];
+          if (r < 0) continue;
+          const float wj = p.topk_w[size_t(t) * p.k + j];
+          float u[ADN_VEC];
+          load8(y + size_t(r) * p.ldy + i * ADN_VEC, u);
+#pragma unroll
+          for (int e = 0; e < ADN_VEC; ++e) v[c][e] = fmaf(wj, u[e], v[c][e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < ADN_VEC; ++e) sq = fmaf(v[c][e], v[c][e], sq);
+    }
+    const float inv = inv_rms();
+#pragma unroll
+    for (int c = 0; c < ADN_KEEP; ++c) {
+      const int i = c * blockDim.x + threadIdx.x;
+      if (i >= nv) break;
+      float hv[ADN_VEC], wv[ADN_VEC];
+      float* hp = p.h + size_t(t) * p.H + i * ADN_VEC;
+      load8<float>(hp, hv);
+      load8<float>(p.w + i * ADN_VEC, wv);
+#pragma unroll
+      for (int e = 0; e < ADN_VEC; ++e) hv[e] = fmaf(v[c][e] * inv, wv[e], hv[e]);
+      reinterpret_cast<float4*>(hp)[0] = make_float4(hv[0], hv[1], hv[2], hv[3]);
+      reinterpret_cast<float4*>(hp)[1] = make_float4(hv[4], hv[5], hv[6], hv[7]);
+      if (p.x)
+        *reinterpret_cast<uint4*>(p.x + size_t(t) * p.H + i * ADN_VEC) =
+            make_uint4(pack_bf16x2(hv[0], hv[1]), pack_bf16x2(hv[2], hv[3]), pack_bf16x2(hv[4], hv[5]), pack_bf16x2(hv[6], hv[7]));
+    }
+  } else {
+    for (int i = threadIdx.x; i < p.H; i += blockDim.x) {
+      const float v = add_normed_col(p, y, t, i);
+      sq = fmaf(v, v, sq);
+    }
+    const float inv = inv_rms();
+    for (int i = threadIdx.x; i < p.H; i += blockDim.x) {
+      const size_t at = size_t(t) * p.H + i;
+      const float n = fmaf(add_normed_col(p, y, t, i) * inv, p.w[i], p.h[at]);
+      p.h[at] = n;
+      if (p.x) p.x[at] = f2bf(n);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------ head norms, rotation, cache append
+// One warp per (token, head).  Query heads are replaced in place; key heads go to the token's cache row; value heads are copied there.
+// A lane handles pairs of columns (i, i + rot / 2) of the rotated part and single columns of the rest, V at a time.
+struct QkvPrep {
+  int ldp, Hq, Hkv, dim, key_row, value_row, rot, max_pos, T;
+  const float *q_norm, *k_norm, *cos, *sin;
+  const int32_t *positions, *slots;
+  float eps;
+};
+
+template <typename T, int V> __device__ __forceinline__ void ld_cols(const T* p, float (&f)[V]) {
+  if constexpr (V == 1) f[0] = to_f32(p[0]);
+  else if constexpr (sizeof(T) == 4) { const float2 a = *reinterpret_cast<const float2*>(p); f[0] = a.x; f[1] = a.y; }
+  else { const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p)); f[0] = a.x; f[1] = a.y; }
+}
+template <typename T, int V> __device__ __forceinline__ void st_cols(T* p, const float (&f)[V]) {
+  if constexpr (V == 1) p[0] = from_f32<T>(f[0]);
+  else if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+  else *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(f[0], f[1]);
+}
+
+// V = 2: two neighbouring columns at a time (dim and rot / 2 even, rows on even addresses), 1: any size.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) qkv_prep_kernel(T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int per = p.Hq + 2 * p.Hkv;
+  const long item = long(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (item >= long(p.T) * per) return;
+  const int t = int(item / per), head = int(item % per), lane = threadIdx.x & 31;
+  T* row = proj + size_t(t) * p.ldp;
+  const int slot = p.slots[t];
+  if (head >= p.Hq + p.Hkv) {
+    const int g = head - p.Hq - p.Hkv;
+    if (slot < 0) return;
+    const T* src = row + size_t(p.Hq + p.Hkv) * p.key_row + size_t(g) * p.value_row;
+    T* dst = v_cache + (size_t(slot) * p.Hkv + g) * p.value_row;
+    for (int i = lane * V; i < p.value_row; i += 32 * V) {
+      float f[V];
+      ld_cols<T, V>(src + i, f);
+      st_cols<T, V>(dst + i, f);
+    }
+    return;
+  }
+  const bool is_q = head < p.Hq;
+  if (!is_q && slot < 0) return;
+  T* src = row + size_t(head) * p.key_row;
+  T* dst = is_q ? src : k_cache + (size_t(slot) * p.Hkv + (head - p.Hq)) * p.key_row;
+  const float* w = is_q ? p.q_norm : p.k_norm;
+  float inv = 1.f;
+  if (w) {
+    float sq = 0.f;
+    for (int i = lane * V; i < p.dim; i += 32 * V) {
+      float f[V];
+      ld_cols<T, V>(src + i, f);
+#pragma unroll
+      for (int e = 0; e < V; ++e) sq = fmaf(f[e], f[e], sq);
+    }
+    inv = 1.f / sqrtf(warp_sum(sq) / p.dim + p.eps);
+  }
+  const int half = p.rot >> 1;
+  const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
+  auto normed = [&](int i, float (&f)[V]) {
+    ld_cols<T, V>(src + i, f);
+    if (w) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = f[e] * inv * w[i + e];
+    }
+  };
+  for (int i = lane * V; i < half; i += 32 * V) {
+    float a[V], b[V], u[V], v[V];
+    normed(i, a);
+    normed(i + half, b);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float c = p.cos[size_t(pos) * half + i + e], s = p.sin[size_t(pos) * half + i + e];
+      u[e] = a[e] * c - b[e] * s;
+      v[e] = b[e] * c + a[e] * s;
+    }
+    st_cols<T, V>(dst + i, u);
+    st_cols<T, V>(dst + i + half, v);
+  }
+  for (int i = p.rot + lane * V; i < p.dim; i += 32 * V) {
+    float f[V];
+    normed(i, f);
+    st_cols<T, V>(dst + i, f);
+  }
+  for (int i = p.dim + lane; i < p.key_row; i += 32) dst[i] = from_f32<T>(0.f);
+}
+
+// ------------------------------------------------------------------------------------ experts' activations
+// Rows of alternating (gate, up) columns.  kind 0: silu(g) * u; 1: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + 1).
+template <typename T>
+__global__ void expert_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long n, int kind, float alpha, float limit) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long i = long(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += long(gridDim.x) * blockDim.x) {
+    float g = to_f32(gu[2 * i]), u = to_f32(gu[2 * i + 1]), r;
+    if (kind == 0) {
+      r = g / (1.f + expf(-g)) * u;
+    } else {
+      if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
+      r = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    }
+    out[i] = from_f32<T>(r);
+  }
+}
+
 // ------------------------------------------------------------------------------------ act(gate) * up
 // x row t: gate in columns [0, I), up in [I, 2I); out row t has I columns.  act: 0 SiLU, 1 GELU(tanh), 2 ReLU, 3 GELU(erf), 4 ReLU^2.
 template <typename T>
@@ -146,13 +364,15 @@ __global__ void causal_conv_rows_kernel(const T* __restrict__ x, int ldx, const 
 
 using namespace ogb;
 
-OGB_API int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, int T, int H, int vocab, float scale, void* stream) {
+OGB_API int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, void* copy, int T, int H, int vocab, float scale,
+                                 void* stream) {
   if (T <= 0) return 0;
   auto s = static_cast<cudaStream_t>(stream);
   const dim3 block(H >= 256 ? 256 : 64);
-  const bool ok = table_fp32 ? launch_pdl(embedding_stream_kernel<float>, dim3(T), block, 0, s, ids, static_cast<const float*>(table), out, H, vocab, scale)
+  const bool ok = table_fp32 ? launch_pdl(embedding_stream_kernel<float>, dim3(T), block, 0, s, ids, static_cast<const float*>(table), out,
+                                          static_cast<__nv_bfloat16*>(copy), H, vocab, scale)
                              : launch_pdl(embedding_stream_kernel<__nv_bfloat16>, dim3(T), block, 0, s, ids, static_cast<const __nv_bfloat16*>(table), out,
-                                          H, vocab, scale);
+                                          static_cast<__nv_bfloat16*>(copy), H, vocab, scale);
   return ok ? 0 : -4;
 }
 
@@ -192,5 +412,58 @@ OGB_API int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const vo
   const bool ok = fp32 ? launch_pdl(causal_conv_rows_kernel<float>, dim3(T), block, 0, s, OGB_CONV_ARGS(float))
                        : launch_pdl(causal_conv_rows_kernel<__nv_bfloat16>, dim3(T), block, 0, s, OGB_CONV_ARGS(__nv_bfloat16));
 #undef OGB_CONV_ARGS
+  return ok ? 0 : -4;
+}
+
+OGB_API int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const float* w, float eps, void* x, const int32_t* inv_pos, const float* topk_w,
+                           int k, int T, int H, void* stream) {
+  if (T <= 0 || H <= 0) return 0;
+  auto s = static_cast<cudaStream_t>(stream);
+  const AddNormed p{h, w, static_cast<__nv_bfloat16*>(x), inv_pos, topk_w, k, ldy, H, eps};
+  const bool vec = H % ADN_VEC == 0 && ldy % ADN_VEC == 0 && H <= 256 * ADN_VEC * ADN_KEEP &&
+                   ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
+  // pieces of a row over the threads: every thread has one where the row has no more than 256
+  const int pieces = vec ? (H / ADN_VEC + 31) / 32 * 32 : (H + 31) / 32 * 32;
+  const dim3 block(pieces < 256 ? pieces : 256);
+  bool ok;
+  if (y_fp32) {
+    const float* yf = static_cast<const float*>(y);
+    ok = vec ? launch_pdl(add_normed_kernel<float, true>, dim3(T), block, 0, s, yf, p) : launch_pdl(add_normed_kernel<float, false>, dim3(T), block, 0, s, yf, p);
+  } else {
+    const __nv_bfloat16* yh = static_cast<const __nv_bfloat16*>(y);
+    ok = vec ? launch_pdl(add_normed_kernel<__nv_bfloat16, true>, dim3(T), block, 0, s, yh, p)
+             : launch_pdl(add_normed_kernel<__nv_bfloat16, false>, dim3(T), block, 0, s, yh, p);
+  }
+  return ok ? 0 : -4;
+}
+
+OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
+                         const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
+                         void* v_cache, int T, int fp32, void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || dim <= 0 || dim > key_row || rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (!cos || !sin || max_pos <= 0))) return -1;
+  const QkvPrep p{ldp, Hq, Hkv, dim, key_row, value_row, rot, max_pos > 0 ? max_pos : 1, T, q_norm, k_norm, cos, sin, positions, slots, eps};
+  const long items = long(T) * (Hq + 2 * Hkv);
+  const dim3 grid(unsigned((items + 7) / 8));
+  auto s = static_cast<cudaStream_t>(stream);
+  const int elem = fp32 ? 4 : 2;
+  const bool two = dim % 2 == 0 && (rot / 2) % 2 == 0 && ldp % 2 == 0 && key_row % 2 == 0 && value_row % 2 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & (2 * elem - 1)) == 0;
+#define OGB_PREP(TY, V) launch_pdl(qkv_prep_kernel<TY, V>, grid, dim3(256), 0, s, static_cast<TY*>(proj), static_cast<TY*>(k_cache), static_cast<TY*>(v_cache), p)
+  const bool ok = fp32 ? (two ? OGB_PREP(float, 2) : OGB_PREP(float, 1)) : (two ? OGB_PREP(__nv_bfloat16, 2) : OGB_PREP(__nv_bfloat16, 1));
+#undef OGB_PREP
+  return ok ? 0 : -4;
+}
+
+OGB_API int ogb_expert_act(const void* gu, void* out, long long n, int I, int kind, float alpha, float limit, int fp32, void* stream) {
+  const long total = long(n) * I;
+  if (total <= 0) return 0;
+  auto s = static_cast<cudaStream_t>(stream);
+  const long nb = (total + 255) / 256;
+  const dim3 grid(unsigned(nb < 148 * 16 ? nb : 148 * 16));
+  const bool ok = fp32 ? launch_pdl(expert_act_kernel<float>, grid, dim3(256), 0, s, static_cast<const float*>(gu), static_cast<float*>(out), total, kind,
+                                    alpha, limit)
+                       : launch_pdl(expert_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, static_cast<const __nv_bfloat16*>(gu),
+                                    static_cast<__nv_bfloat16*>(out), total, kind, alpha, limit);
   return ok ? 0 : -4;
 }

@@ -29,7 +29,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T,
   if (mode != 0) {
     for (int e = lane; e < E; e += 32) all_max = fmaxf(all_max, row[e]);
     all_max = warp_max(all_max);
-    for (int e = lane; e < E; e += 32) all_sum += __expf(row[e] - all_max);
+    for (int e = lane; e < E; e += 32) all_sum += expf(row[e] - all_max);
     all_sum = warp_sum(all_sum);
   }
   float my_val = 0.f;   // lane j keeps the j-th selected logit
@@ -55,10 +55,10 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T,
   }
   float w;
   if (mode == 0) {
-    const float ex = lane < k ? __expf(my_val - first) : 0.f;
+    const float ex = lane < k ? expf(my_val - first) : 0.f;
     w = ex / warp_sum(ex);
   } else {
-    const float pr = lane < k ? __expf(my_val - all_max) / all_sum : 0.f;
+    const float pr = lane < k ? expf(my_val - all_max) / all_sum : 0.f;
     w = mode == 2 ? pr / warp_sum(pr) : pr;
   }
   if (lane < k) {

@@ -17,7 +17,7 @@ LLM_TYPES = [
     "chatglm", "decoder", "ernie4_5", "gemma", "gemma2", "gemma3_text", "gptoss", "gpt_oss", "granite", "hunyuan", "hunyuandensev1", "hunyuan_v1_dense",
     "internlm2", "llama", "mistral", "nemotron", "olmo", "olmo2", "exaone4", "phi", "phi3", "phimoe", "qwen2", "qwen3",
     "smollm3", "lfm2", "gpt2", "helium", "mixtral", "qwen2_moe", "qwen3_moe", "granitemoe", "olmoe", "qwen2_vl", "qwen2_5_vl", "qwen3_vl",
-    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar",      # hybrids of gated-delta-net (linear attention) and full-attention layers
+    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar", "zevopel",      # hybrids of gated-delta-net (linear attention) and full-attention layers
 ]
 
 
@@ -30,7 +30,8 @@ ALM_TYPES = ["whisper"]
 @dataclass
 class RotarySpec:
     """Rotary positions of one layer: the first `dims` entries of a vector turn in pairs (i, i + dims / 2) with the frequencies
-    base^(-2 i / dims); scaling: None or the YaRN parameters {factor, original, fast, slow}."""
+    base^(-2 i / dims); scaling: None, the YaRN parameters {factor, original, fast, slow}, or {factor, original, low, high}: slowed down
+    by wavelength (Llama 3.1, see `wavelength_frequencies`)."""
     dims: int
     base: float
     scaling: Optional[Dict[str, float]] = None
@@ -40,8 +41,26 @@ class RotarySpec:
 
 
 @dataclass
+class MoeSpec:
+    """Routed experts of a layer: `top` of `experts` feed-forwards run per token.  act: "silu" silu(gate) * up, or "clamped"
+    g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).  weights: softmax over the "selected" router
+    logits, over "all" of them, or over all and "renormed" over the selected; "sparse_mixer": PhiMoE's margin rule."""
+    experts: int
+    top: int
+    act: str = "silu"
+    alpha: float = 1.702
+    limit: float = 0.0
+    weights: str = "all"
+    jitter_eps: float = 0.01
+
+
+@dataclass
 class LayerSpec:
     """One layer of a stack whose configuration lists its layers one by one (every layer has sizes of its own).  kind:
+      "attention"         `heads` query heads over `kv_heads` key / value heads, queries and keys of `dim`, values of `vdim` dimensions;
+                          chunk > 0: position p sees the keys of its own run of `chunk` positions (counted from position 0), 0: every
+                          earlier one; qk_norm: RMS norm of every query and key head before the rotation; sinks: a learned logit per head
+                          in the softmax's denominator; head_gate: a head's output times sigmoid of a projection of the mixer's input;
       "linear_attention"  gated delta rule: `kv_heads` query / key heads of `dim`, `heads` value heads of `vdim`, convolution of `conv` taps;
       "latent_attention"  `heads` heads of `dim` unrotated + `rot_dim` rotated query / key dimensions and `vdim` value dimensions over a
                           latent of `kv_rank` values per token; window 0: every earlier token is visible."""
@@ -55,8 +74,13 @@ class LayerSpec:
     rot_dim: int = 0
     scale: float = 1.0
     window: int = 0
+    chunk: int = 0
+    qk_norm: bool = False
+    sinks: bool = False
+    head_gate: bool = False
     rotary: Optional[RotarySpec] = None
-    ff: int = 0                       # width of the gated feed-forward (0: the layer has none)
+    ff: int = 0                       # width of the gated feed-forward, of one expert where there are experts (0: the layer has none)
+    moe: Optional[MoeSpec] = None
     weights_of: Optional[int] = None  # layer whose weights this one uses (cache and state are its own)
 
     @property
@@ -71,6 +95,15 @@ class LayerSpec:
     def latent_row(self) -> int:
         """Values a token keeps in the latent cache (rounded up to whole 16-byte pieces of 16-bit values)."""
         return (self.kv_rank + self.rot_dim + 7) // 8 * 8 if self.kind == "latent_attention" else 0
+
+    @property
+    def key_row(self) -> int:
+        """Columns of one key (and query) head of an attention layer: whole 16-byte pieces of 16-bit values, zeros past `dim`."""
+        return (self.dim + 7) // 8 * 8 if self.kind == "attention" else 0
+
+    @property
+    def value_row(self) -> int:
+        return (self.vdim + 7) // 8 * 8 if self.kind == "attention" else 0
 
 
 @dataclass
@@ -128,8 +161,11 @@ class ArchConfig:
     mamba_n_groups: int = 1
     mamba_conv_kernel: int = 4
     # Declared stacks: one entry per layer (see LayerSpec); layer_types then mirrors the entries' kinds.  Such stacks keep an fp32
-    # residual stream and join both sub-layers of a block in one output projection (parallel_block).
+    # residual stream.  Their blocks join both sub-layers in one output projection (parallel_block), or run them one after the other on
+    # the stream itself with a norm on each output (pre_norm False, post_sublayer_norms), scaled per element (layer_scale) and by
+    # residual_multiplier.
     layer_specs: Optional[List[LayerSpec]] = None
+    layer_scale: bool = False
     delta_l2_eps: float = 0.0        # gated delta rule: > 0 makes unit vectors x / sqrt(sum(x^2) + eps) instead of x / max(|x|, 1e-6)
     # Multimodal RoPE (Qwen2-VL): rotary pairs per position component (temporal, height, width); None: ordinary RoPE
     mrope_section: Optional[List[int]] = None
@@ -230,6 +266,20 @@ class ArchConfig:
     def mamba_conv_dim(self) -> int:
         return self.mamba_intermediate + 2 * self.mamba_n_groups * self.mamba_state_size
 
+    @property
+    def moe_spec(self) -> Optional[MoeSpec]:
+        """The experts of a model whose layers all have the same ones."""
+        if self.num_experts <= 0:
+            return None
+        std = self.moe_style == "standard"
+        weights = "sparse_mixer" if self.moe_sparse_mixer else ("all" if std and not self.moe_norm_topk else "selected")
+        return MoeSpec(self.num_experts, self.experts_per_token, "silu" if std else "clamped", self.moe_swiglu_alpha, self.moe_swiglu_limit, weights,
+                       self.moe_jitter_eps)
+
+    def is_spec_attention(self, layer: int) -> bool:
+        """Attention layers of declared stacks: keys and values have sizes of their own in every layer."""
+        return self.layer_specs is not None and self.layer_specs[layer].kind == "attention"
+
     def is_latent_layer(self, layer: int) -> bool:
         return self.layer_types is not None and self.layer_types[layer] == "latent_attention"
 
@@ -303,56 +353,86 @@ class ArchConfig:
 # "width"): what a design fixes for all its models.
 STACK_DESIGNS: Dict[str, Dict[str, Any]] = {
     # parallel blocks under one layer norm (weight and bias); gated delta rule and latent attention; ReLU-gated feed-forward
-    "Luzatar": dict(model_type="luzatar", layernorm=True, parallel_block=True, activation="relu", delta_l2_eps=1e-6),
+    "Luzatar": dict(arch=dict(model_type="luzatar", layernorm=True, parallel_block=True, activation="relu", delta_l2_eps=1e-6),
+                    mixers={"delta": "linear_attention", "latent_attention": "latent_attention"}, feed_forwards=("dense",)),
+    # sub-layers on the stream itself, RMS norms (stored around zero), layer scales and a residual multiplier on their outputs; chunked
+    # attention with normed queries and keys, sinks and a gate per head; GELU-gated feed-forward or clamped experts weighted by their
+    # probabilities among all experts
+    "Zevopel": dict(arch=dict(model_type="zevopel", pre_norm=False, post_sublayer_norms=True, norm_offset=1.0, layer_scale=True, activation="gelu_tanh"),
+                    mixers={"attention": "attention"}, feed_forwards=("dense", "moe"), attention=dict(qk_norm=True, sinks=True, head_gate=True),
+                    moe=dict(act="clamped", alpha=1.702, weights="all")),
 }
-_STACK_MIXERS = {"delta": "linear_attention", "latent_attention": "latent_attention"}
 
 
 def is_stack_config(cfg: Dict[str, Any]) -> bool:
     return isinstance(cfg, dict) and cfg.get("architecture") in STACK_DESIGNS and isinstance(cfg.get("layers"), list)
 
 
-def _stack_layer(i: int, e: Dict[str, Any]) -> LayerSpec:
-    kind = _STACK_MIXERS.get(e.get("type"))
+def _rotary_spec(i: int, rot: Optional[Dict[str, Any]], width: int) -> Optional[RotarySpec]:
+    if not rot or not int(rot["dims"]):
+        return None
+    sc = rot.get("scaling")
+    spec = RotarySpec(int(rot["dims"]), float(rot["base"]), {k: float(v) for k, v in sc.items()} if sc else None)
+    if spec.dims > width or spec.dims % 2:
+        raise ValueError(f"layer {i}: {spec.dims} rotary dimensions do not fit the {width} rotated ones")
+    return spec
+
+
+def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec:
+    kind = design["mixers"].get(e.get("type"))
     if kind is None:
         raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
     m, mlp = e["mixer"], e.get("mlp")
-    if mlp and mlp.get("kind", "dense") != "dense":
-        raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
-    sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), ff=int(mlp["ff"]) if mlp else 0,
+    ff_kind = mlp.get("kind", "dense") if mlp else None
+    if mlp and ff_kind not in design["feed_forwards"]:
+        raise ValueError(f"layer {i}: unknown feed-forward kind {ff_kind!r}")
+    sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                    weights_of=None if e.get("weights_of") is None else int(e["weights_of"]))
-    if kind == "linear_attention":
-        sp.kv_heads, sp.conv = int(m["kv_heads"]), int(m["conv"])
+    if ff_kind == "dense":
+        sp.ff = int(mlp["ff"])
+    elif ff_kind == "moe":
+        sp.ff = int(mlp["expert"]["ff"])
+        sp.moe = MoeSpec(int(mlp["router"]["experts"]), int(mlp["router"]["top"]), limit=float(mlp["expert"].get("limit") or 0.0), **design["moe"])
+        if not 0 < sp.moe.top <= sp.moe.experts:
+            raise ValueError(f"layer {i}: {sp.moe.top} of {sp.moe.experts} experts cannot be chosen")
+    if kind in ("linear_attention", "attention"):
+        sp.kv_heads = int(m["kv_heads"])
         if sp.heads % sp.kv_heads:
             raise ValueError(f"layer {i}: {sp.heads} heads do not divide over {sp.kv_heads} key heads")
+    mask = int((m.get("mask") or {}).get("size") or 0)
+    if kind == "linear_attention":
+        sp.conv = int(m["conv"])
+    elif kind == "attention":
+        sp.scale, sp.chunk = float(m["scale"]), mask
+        sp.rotary = _rotary_spec(i, m.get("rot"), sp.dim)
+        for k, v in design["attention"].items():
+            setattr(sp, k, v)
     else:
-        sp.kv_rank, sp.rot_dim, sp.scale = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"])
-        sp.window = int((m.get("mask") or {}).get("size") or 0)
-        if m.get("rot"):
-            sc = m["rot"].get("scaling")
-            sp.rotary = RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"]), {k: float(v) for k, v in sc.items()} if sc else None)
-            if sp.rotary.dims > sp.rot_dim or sp.rotary.dims % 2:
-                raise ValueError(f"layer {i}: {sp.rotary.dims} rotary dimensions do not fit the rotated part of {sp.rot_dim}")
+        sp.kv_rank, sp.rot_dim, sp.scale, sp.window = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"]), mask
+        sp.rotary = _rotary_spec(i, m.get("rot"), sp.rot_dim)
     return sp
 
 
 def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
     """config.json of a declared stack -> ArchConfig."""
-    specs = [_stack_layer(i, e) for i, e in enumerate(cfg["layers"])]
+    design = STACK_DESIGNS[cfg["architecture"]]
+    specs = [_stack_layer(i, e, design) for i, e in enumerate(cfg["layers"])]
     for i, sp in enumerate(specs):
         if sp.weights_of is not None and not (0 <= sp.weights_of < len(specs) and specs[sp.weights_of].weights_of is None and
                                               specs[sp.weights_of].kind == sp.kind and sp.weights_of != i):
             raise ValueError(f"layer {i}: weights_of {sp.weights_of} does not name a layer of its kind with weights of its own")
-    lat = [sp for sp in specs if sp.kind == "latent_attention"]
+    att = [sp for sp in specs if sp.kind != "linear_attention"]
     # longest sequence the rotary scaling was made for, and at least 32768 positions (recurrent and windowed layers have no limit)
-    span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in lat if sp.rotary and sp.rotary.scaling]
+    span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in att if sp.rotary and sp.rotary.scaling]
     eos = cfg.get("eos_token_id")
     return ArchConfig(vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=max(sp.heads for sp in specs),
-                      num_kv_heads=1, head_dim=max((sp.kv_rank + sp.rot_dim for sp in lat), default=specs[0].dim),
+                      num_kv_heads=max((sp.kv_heads for sp in specs if sp.kind == "attention"), default=1),
+                      head_dim=max((sp.kv_rank + sp.rot_dim or sp.dim for sp in att), default=specs[0].dim),
                       intermediate_size=max(sp.ff for sp in specs), context_length=int(cfg.get("context_length") or max([32768] + span)),
-                      norm_eps=float(cfg["norm"]["eps"]), layer_specs=specs, layer_types=[sp.kind for sp in specs], no_rope=not lat,
+                      norm_eps=float(cfg["norm"]["eps"]), layer_specs=specs, layer_types=[sp.kind for sp in specs], no_rope=not att,
+                      embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)), residual_multiplier=float(cfg.get("residual_mult", 1.0)),
                       bos_token_id=int(cfg.get("bos_token_id", 0)), eos_token_id=-1 if eos is None else eos, pad_token_id=int(cfg.get("pad_token_id", 0)),
-                      **STACK_DESIGNS[cfg["architecture"]])
+                      **design["arch"])
 
 
 def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
@@ -365,20 +445,36 @@ def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
         if sp.weights_of is not None:
             continue
         p, m = f"l{i}.", f"l{i}.mix."
-        out[p + "norm1"] = (W,)
-        if arch.layernorm:
-            out[p + "norm1.b"] = (W,)
+        # one norm for both sub-layers of a parallel block, else one for each
+        for n in range(1, 2 if arch.parallel_block or not sp.ff else 3):
+            out[f"{p}norm{n}"] = (W,)
+            if arch.layernorm:
+                out[f"{p}norm{n}.b"] = (W,)
+            if arch.layer_scale:
+                out[f"{p}ls{n}"] = (W,)
         if sp.kind == "linear_attention":
             kd, vd = sp.kv_heads * sp.dim, sp.heads * sp.vdim
             for n, c in (("q", kd), ("k", kd), ("v", vd)):
                 out[m + n], out[m + n + ".conv"] = (c, W), (c, sp.conv)
             out.update({m + "b": (sp.heads, W), m + "a": (sp.heads, W), m + "A_log": (sp.heads,), m + "dt_bias": (sp.heads,), m + "norm": (sp.vdim,),
                         m + "g": (vd, W), m + "o": (W, vd)})
+        elif sp.kind == "attention":
+            out.update({m + "q": (sp.heads * sp.dim, W), m + "k": (sp.kv_heads * sp.dim, W), m + "v": (sp.kv_heads * sp.vdim, W),
+                        m + "o": (W, sp.heads * sp.vdim)})
+            if sp.qk_norm:
+                out.update({m + "q.norm": (sp.dim,), m + "k.norm": (sp.dim,)})
+            if sp.sinks:
+                out[m + "sink"] = (sp.heads,)
+            if sp.head_gate:
+                out[m + "g"] = (sp.heads, W)
         else:
             out.update({m + "q": (sp.heads * (sp.dim + sp.rot_dim), W), m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
                         m + "uk": (sp.heads * sp.dim, sp.kv_rank), m + "uv": (sp.heads * sp.vdim, sp.kv_rank), m + "o": (W, sp.heads * sp.vdim)})
         if sp.ff:
-            out.update({p + "mlp.gate": (sp.ff, W), p + "mlp.up": (sp.ff, W), p + "mlp.down": (W, sp.ff)})
+            if sp.moe is not None:
+                out[p + "mlp.router"] = (sp.moe.experts, W)
+            for e in [""] if sp.moe is None else [f"e{k}." for k in range(sp.moe.experts)]:
+                out.update({f"{p}mlp.{e}gate": (sp.ff, W), f"{p}mlp.{e}up": (sp.ff, W), f"{p}mlp.{e}down": (W, sp.ff)})
     return out
 
 
@@ -654,11 +750,24 @@ def yarn_frequencies(inv_freq, rot: int, base: float, factor: float, original: f
     return inv_freq / factor * ramp + inv_freq * (1.0 - ramp)
 
 
+def wavelength_frequencies(inv_freq, factor: float, original: float, low: float, high: float):
+    """Llama 3.1: a pair whose wavelength is below original / high keeps its frequency, one above original / low is slowed down by
+    `factor`, between the two the frequency is blended linearly in original / wavelength."""
+    wavelen = 2 * math.pi / inv_freq
+    smooth = (original / wavelen - low) / (high - low) if high != low else np.ones_like(inv_freq)
+    scaled = np.where(wavelen > original / low, inv_freq / factor, inv_freq)
+    mid = (wavelen <= original / low) & (wavelen >= original / high)
+    return np.where(mid, (1 - smooth) * inv_freq / factor + smooth * inv_freq, scaled)
+
+
 def rotary_tables(spec: RotarySpec, n: int):
     """cos / sin [n, dims / 2] fp32 of a layer's rotary positions (angles in float64; YaRN multiplies both by 0.1 ln(factor) + 1)."""
     inv_freq = spec.base ** (-np.arange(0, spec.dims, 2, dtype=np.float64) / spec.dims)
     amp = 1.0
-    if spec.scaling:
+    if spec.scaling and "low" in spec.scaling:
+        sc = spec.scaling
+        inv_freq = wavelength_frequencies(inv_freq, sc["factor"], sc["original"], sc["low"], sc["high"])
+    elif spec.scaling:
         sc = spec.scaling
         inv_freq = yarn_frequencies(inv_freq, spec.dims, spec.base, sc["factor"], sc["original"], sc["fast"], sc["slow"], spec.dims - 1)
         amp = 0.1 * math.log(sc["factor"]) + 1.0
@@ -685,12 +794,7 @@ def rope_caches(arch: ArchConfig, max_positions: Optional[int] = None, local: bo
     elif kind == "llama3":
         factor = float(sc["factor"])
         low, high = float(sc.get("low_freq_factor", 1.0)), float(sc.get("high_freq_factor", 4.0))
-        old = float(sc.get("original_max_position_embeddings", 8192))
-        wavelen = 2 * math.pi / inv_freq
-        smooth = (old / wavelen - low) / (high - low)
-        scaled = np.where(wavelen > old / low, inv_freq / factor, inv_freq)
-        mid = (wavelen <= old / low) & (wavelen >= old / high)
-        inv_freq = np.where(mid, (1 - smooth) * inv_freq / factor + smooth * inv_freq, scaled)
+        inv_freq = wavelength_frequencies(inv_freq, factor, float(sc.get("original_max_position_embeddings", 8192)), low, high)
     elif kind == "yarn":
         factor = float(sc["factor"])
         old = float(sc.get("original_max_position_embeddings", arch.context_length / factor))

@@ -21,7 +21,7 @@ import torch
 
 from .. import ops
 from ..native_loader import native
-from .arch import ArchConfig
+from .arch import ArchConfig, MoeSpec
 
 
 @dataclass
@@ -80,7 +80,17 @@ class PagedKVCache:
                        if self.latent_index else None)
         if self.latent is not None and kv_bits != 16:
             raise RuntimeError("KV cache quantization is not available for latent-attention layers")
-        conv = [c or i in self.latent_index for i, c in enumerate(conv)]        # layers without key / value rows
+        # Attention layers of declared stacks: keys and values of each layer in pools as wide as its own heads, in the same paged slots.
+        self.spec_kv = {}
+        for i in range(arch.num_layers):
+            if arch.is_spec_attention(i):
+                if kv_bits != 16:
+                    raise RuntimeError("KV cache quantization is not available for declared stacks")
+                sp = arch.layer_specs[i]
+                self.spec_kv[i] = tuple(torch.zeros(num_blocks * block_size, sp.kv_heads, n, dtype=dtype, device=device)
+                                        for n in (sp.key_row, sp.value_row))
+        # layers without rows in the pools below
+        conv = [c or i in self.latent_index or i in self.spec_kv for i, c in enumerate(conv)]
         self.windowed = [num_window_blocks > 0 and arch.layer_window(i) > 0 and not conv[i] for i in range(arch.num_layers)]
         n_full = sum(1 for w, c in zip(self.windowed, conv) if not w and not c)
         n_win = sum(1 for w in self.windowed if w)
@@ -111,7 +121,22 @@ class PagedKVCache:
             else:
                 self._index.append((False, fi)); fi += 1
 
+    def copy_blocks(self, src, dst) -> None:
+        """Contents of the blocks src[i] (int64 ids) into the blocks dst[i], in every pool that is addressed by block."""
+        ar = torch.arange(self.block_size, device=src.device)
+        s_idx, d_idx = (src[:, None] * self.block_size + ar).reshape(-1), (dst[:, None] * self.block_size + ar).reshape(-1)
+        if self.full.numel():
+            self.full[:, :, d_idx] = self.full[:, :, s_idx]
+        for pool in (self.conv, self.latent):
+            if pool is not None:
+                pool[:, d_idx] = pool[:, s_idx]
+        for pools in self.spec_kv.values():
+            for pool in pools:
+                pool[d_idx] = pool[s_idx]
+
     def layer(self, i: int):
+        if i in self.spec_kv:
+            return (*self.spec_kv[i], False)
         win, j = self._index[i]
         pool = self.win if win else self.full
         return pool[j, 0], pool[j, 1], win
@@ -149,7 +174,9 @@ class PagedKVCache:
         es = torch.empty((), dtype=dtype).element_size()
         kv_row = arch.head_dim + 16 if kv_bits == 8 else arch.head_dim * es
         n_lat = sum(1 for i in range(arch.num_layers) if arch.is_latent_layer(i))
-        return ((arch.num_layers - n_conv - n_lat) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row) * es) * block_size
+        own = [sp for i, sp in enumerate(arch.layer_specs or []) if arch.is_spec_attention(i)]
+        own_row = sum(sp.kv_heads * (sp.key_row + sp.value_row) for sp in own)
+        return ((arch.num_layers - n_conv - n_lat - len(own)) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row + own_row) * es) * block_size
 
 
 class CrossKVCache:
@@ -250,6 +277,7 @@ class LayerWeights:
     exp_down_b: Optional[torch.Tensor] = None
     exp_lo: int = 0          # experts [exp_lo, exp_hi) live on this rank (expert parallelism)
     exp_hi: int = 0
+    moe: Optional[MoeSpec] = None  # experts of this layer where layers differ (None: the model's, arch.moe_spec)
     exp_blocked: bool = False  # gate/up rows in blocks of 64 gate + 64 up (grouped-GEMM layout) instead of even/odd
     lora: Dict[str, dict] = field(default_factory=dict)
     fold_ln1: Optional[torch.Tensor] = None    # norm weights that were multiplied into qkv_w / gate_up_w (see DecoderModel.fold_norms)
@@ -360,21 +388,27 @@ class DecoderModel:
             return ops.linear(x, w, bias, all_reduce=True)   # GEMM + all-reduce in one kernel over NVLink
         return self.tp.reduce(self._linear(x, w, bias, lora=lora))
 
-    def _attention(self, s: StepInputs, qkv, kc, vc, table, block_size: int, lw: LayerWeights):
+    def _attention(self, s: StepInputs, qkv, kc, vc, table, block_size: int, lw: LayerWeights, sp=None, gate=None, out=None):
         """Paged attention of one layer.  A mixed step (single-token requests first, then prompt chunks) runs as two launches:
         the single-token requests on the decode tiles (16 rows, the four warps share every K/V tile), the chunks on the
-        64-row tiles - in one launch every single-token request would occupy a 64-row tile that one warp walks alone."""
+        64-row tiles - in one launch every single-token request would occupy a 64-row tile that one warp walks alone.
+        sp: the layer's own sizes and mask (declared stacks); gate [T, heads]: logits of a gate on each head's output."""
         a = self.arch
-        args = (block_size, self.heads_local, self.kv_heads_local, a.head_dim, a.scale, lw.window, lw.sinks, a.softcap)
+        if sp is None:
+            args, kw, cols = (block_size, self.heads_local, self.kv_heads_local, a.head_dim, a.scale, lw.window, lw.sinks, a.softcap), {}, a.head_dim
+        else:
+            args, cols = (block_size, sp.heads, sp.kv_heads, sp.key_row, sp.scale, 0, lw.sinks, 0.0), sp.value_row
+            kw = dict(vdim=sp.value_row, chunk=sp.chunk, gate=gate)
         nd, B = s.num_decode, s.past_lens.shape[0]
         if not (qkv.is_cuda and 0 < nd < B and s.max_q_len > 1):
             return ops.paged_attention(qkv, kc, vc, s.cu_seqlens, s.past_lens, table, *args, max_q_len=s.max_q_len,
-                                       max_kv_len=s.max_kv_len, order=s.attn_order, min_q_len=s.min_q_len or None)
-        out = torch.empty(qkv.shape[0], self.heads_local * a.head_dim, dtype=qkv.dtype, device=qkv.device)
+                                       max_kv_len=s.max_kv_len, order=s.attn_order, min_q_len=s.min_q_len or None, out=out, **kw)
+        if out is None:
+            out = torch.empty(qkv.shape[0], args[1] * cols, dtype=qkv.dtype, device=qkv.device)
         ops.paged_attention(qkv, kc, vc, s.cu_seqlens[:nd + 1], s.past_lens[:nd], table[:nd], *args, max_q_len=1,
-                            max_kv_len=s.max_kv_len, out=out, total_tokens=nd)
+                            max_kv_len=s.max_kv_len, out=out, total_tokens=nd, **kw)
         ops.paged_attention(qkv, kc, vc, s.cu_seqlens[nd:], s.past_lens[nd:], table[nd:], *args, max_q_len=s.max_q_len,
-                            max_kv_len=s.max_kv_len, out=out)
+                            max_kv_len=s.max_kv_len, out=out, **kw)
         return out
 
     @staticmethod
@@ -455,14 +489,39 @@ class DecoderModel:
                                       sp.window, out)
         return out
 
+    def _spec_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """An attention layer of a declared stack: one projection [queries | keys | values | gate logits], norms, rotation and cache append
+        in one pass, attention over the paged cache whose epilogue gates the heads; writes them to `out` [T, heads * value_row]."""
+        sp = self.arch.layer_specs[li]
+        kc, vc, _ = kv.layer(li)
+        proj = self._wide_linear(x, lw.qkv_w)
+        ops.qkv_prep(proj, sp.heads, sp.kv_heads, sp.dim, sp.key_row, sp.value_row, lw.q_norm_w, lw.k_norm_w, self.arch.norm_eps, s.positions,
+                     lw.rope_cos, lw.rope_sin, s.slot_mapping, kc, vc)
+        g0 = (sp.heads + sp.kv_heads) * sp.key_row + sp.kv_heads * sp.value_row
+        return self._attention(s, proj, kc, vc, s.block_table, kv.block_size, lw, sp, proj[:, g0:g0 + sp.heads] if sp.head_gate else None, out)
+
+    def _stack_mixer(self, lw: LayerWeights, sp):
+        return {"linear_attention": self._linear_attention, "latent_attention": self._latent_attention, "attention": self._spec_attention}[sp.kind]
+
     def _forward_stream(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
-        """Parallel blocks on an fp32 residual stream (declared stacks): per layer one norm, the mixer and the gated feed-forward side by
-        side into the column ranges of one matrix, and one output projection of both whose epilogue adds to the stream in fp32."""
+        """Declared stacks: an fp32 residual stream between the embedding and the final norm (of the rows whose logits are wanted)."""
         a = self.arch
         if self.tp.size > 1:
             raise RuntimeError("declared stacks run on one GPU")
         if s.lora_ids is not None or self.active_adapter is not None:
             raise RuntimeError("LoRA adapters are not available for declared stacks")
+        if a.parallel_block:
+            h = self._parallel_blocks(s, kv)
+        else:
+            h = self._output_normed_blocks(s, kv)
+        x = ops.norm_stream(h, self.final_norm_w, a.norm_eps, self.final_norm_b, a.layernorm, self.dtype, rows=s.logits_rows)
+        self.last_hidden = x
+        return ops.linear(x, self.lm_head_w, out_fp32=True)
+
+    def _parallel_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
+        """Parallel blocks: per layer one norm, the mixer and the gated feed-forward side by side into the column ranges of one matrix,
+        and one output projection of both whose epilogue adds to the stream in fp32."""
+        a = self.arch
         h = s.inputs_embeds.float().clone() if s.inputs_embeds is not None else ops.embedding_stream(s.input_ids, self.embed, a.embed_scale)
         T = h.shape[0]
         for li, lw in enumerate(self.layers):
@@ -470,15 +529,36 @@ class DecoderModel:
             K = lw.join_w.shape[1]
             used = (lw.mlp_col == lw.mix_cols or lw.gate_up_w is None) and K == lw.mix_cols + (a.layer_specs[li].ff)
             y = (torch.empty if used else torch.zeros)(T, K, dtype=self.dtype, device=h.device)      # padding columns meet zero weights: finite
-            mixer = self._linear_attention if lw.lin_in_w is not None else self._latent_attention
-            mixer(s, kv, li, lw, x, out=y[:, :lw.mix_cols])
+            self._stack_mixer(lw, a.layer_specs[li])(s, kv, li, lw, x, out=y[:, :lw.mix_cols])
             if lw.gate_up_w is not None:
                 ops.gate_up_act(x, lw.gate_up_w, None, a.activation, out=y[:, lw.mlp_col:lw.mlp_col + a.layer_specs[li].ff],
                                 interleaved=lw.gate_up_interleaved)
             h = ops.linear(y, lw.join_w, residual=h, out=h, out_fp32=True)
-        x = ops.norm_stream(h, self.final_norm_w, a.norm_eps, self.final_norm_b, a.layernorm, self.dtype, rows=s.logits_rows)
-        self.last_hidden = x
-        return ops.linear(x, self.lm_head_w, out_fp32=True)
+        return h
+
+    def _output_normed_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
+        """Blocks whose sub-layers read the stream itself (x, its copy in the compute type): each sub-layer's result is normed, scaled
+        (norm weight, layer scale and residual multiplier are one vector) and added to the stream by one kernel, which also writes the
+        next sub-layer's x and folds the weighted sum of a mixture-of-experts layer."""
+        a = self.arch
+        if s.inputs_embeds is not None:
+            h = s.inputs_embeds.float().clone()
+            x = h.to(self.dtype)
+        else:
+            h, x = ops.embedding_stream(s.input_ids, self.embed, a.embed_scale, self.dtype)
+        for li, lw in enumerate(self.layers):
+            sp = a.layer_specs[li]
+            heads = torch.empty(h.shape[0], lw.mix_cols, dtype=self.dtype, device=h.device)
+            self._stack_mixer(lw, sp)(s, kv, li, lw, x, out=heads)
+            x = ops.add_normed(h, ops.linear(heads, lw.o_w), lw.post_attn_norm_w, a.norm_eps, self.dtype)
+            if sp.ff:
+                if sp.moe is not None:
+                    from .moe import moe_forward
+                    y = moe_forward(self, lw, x, defer=True)
+                else:
+                    y = ops.linear(ops.gate_up_act(x, lw.gate_up_w, None, a.activation, interleaved=lw.gate_up_interleaved), lw.down_w)
+                x = ops.add_normed(h, y, lw.post_ffn_norm_w, a.norm_eps, self.dtype)
+        return h
 
     def _mamba(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor) -> torch.Tensor:
         """A Mamba-2 layer (GraniteMoeHybrid).  Like the gated-delta-net layers, the causal convolution reads the projected

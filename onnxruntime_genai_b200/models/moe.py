@@ -1,6 +1,7 @@
 """Mixture-of-experts MLP: router -> top-k -> routing weights -> per-expert gated MLP -> weighted sum.
 Two styles: gpt-oss (biases, softmax over the selected logits, clamped SwiGLU(alpha, limit)) and standard (Mixtral, Qwen-MoE,
-PhiMoE, GraniteMoE: no biases, silu(gate) * up, softmax over all experts with or without renormalisation).
+PhiMoE, GraniteMoE: no biases, silu(gate) * up, softmax over all experts with or without renormalisation).  Declared stacks describe
+the experts of each layer by themselves (`LayerWeights.moe`, an arch.MoeSpec), with any mix of these rules.
 
 Semantics follow the MoE / QMoE contrib op the reference's builder emits
 (src/python/py/models/builders/base.py:4176-4408, builders/gptoss.py:653-847): `k` experts per token,
@@ -24,6 +25,7 @@ import os
 import torch
 
 from .. import ops
+from .arch import MoeSpec
 
 
 # OGB_MOE_ROW_MAP=0: the token rows of packed experts are gathered into a copy instead of being read through the row map
@@ -38,15 +40,23 @@ def swiglu_interleaved(gu: torch.Tensor, alpha: float, limit: float) -> torch.Te
     return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(gu.dtype)
 
 
+def spec_of(model, lw) -> MoeSpec:
+    """The routing rule and the activation of a layer: its own, or the model's."""
+    return lw.moe if lw.moe is not None else model.arch.moe_spec
+
+
+_TOPK_MODES = {"selected": 0, "all": 1, "renormed": 2}      # softmax over the selected logits / over all / over all, then over the selected
+
+
 def route(model, lw, x):
     """Routing weights and expert ids [T, k].  Softmax over the selected logits equals softmax over all experts renormalised
     over the selected; the standard style without renormalisation keeps the probabilities of the full softmax."""
-    a = model.arch
+    sp = spec_of(model, lw)
     logits = ops.linear(x, lw.router_w, lw.router_b).float()
-    if a.moe_sparse_mixer:
-        return sparse_mixer(logits, a.moe_jitter_eps)
-    top_v, top_i = torch.topk(logits, a.experts_per_token, dim=-1)
-    if a.moe_style == "standard" and not a.moe_norm_topk:
+    if sp.weights == "sparse_mixer":
+        return sparse_mixer(logits, sp.jitter_eps)
+    top_v, top_i = torch.topk(logits, sp.top, dim=-1)
+    if sp.weights == "all":
         return torch.softmax(logits, dim=-1).gather(-1, top_i), top_i
     return torch.softmax(top_v, dim=-1), top_i
 
@@ -85,27 +95,27 @@ def _unblock(t: torch.Tensor) -> torch.Tensor:
 
 def expert_mlp(model, lw, e: int, xs: torch.Tensor) -> torch.Tensor:
     """One expert (index into this rank's slice) over its rows: the unfused path (CPU, odd shapes)."""
-    a = model.arch
+    sp = spec_of(model, lw)
     packed = isinstance(lw.exp_gate_up_w, ops.Fp4Experts)   # MXFP4 experts: expand this one expert
     w = lw.exp_gate_up_w.dequantize(e).to(xs) if packed else lw.exp_gate_up_w[e]
     b = lw.exp_gate_up_b[e] if lw.exp_gate_up_b is not None else None
     if lw.exp_blocked:
         w, b = _unblock(w).contiguous(), _unblock(b).contiguous() if b is not None else None
     gu = ops.linear(xs, w, b)
-    act = silu_mul_interleaved(gu) if a.moe_style == "standard" else swiglu_interleaved(gu, a.moe_swiglu_alpha, a.moe_swiglu_limit)
+    act = silu_mul_interleaved(gu) if sp.act == "silu" else swiglu_interleaved(gu, sp.alpha, sp.limit)
     wd = lw.exp_down_w.dequantize(e).to(xs) if packed else lw.exp_down_w[e]
     return ops.linear(act.contiguous(), wd, lw.exp_down_b[e] if lw.exp_down_b is not None else None)
 
 
 def _forward_loop(model, lw, x):
-    a = model.arch
-    lo, hi = lw.exp_lo, lw.exp_hi or a.num_experts
+    sp = spec_of(model, lw)
+    lo, hi = lw.exp_lo, lw.exp_hi or sp.experts
     weights, experts = route(model, lw, x)
     out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
     flat_e = experts.reshape(-1)
     order = torch.argsort(flat_e, stable=True)
-    counts = torch.bincount(flat_e, minlength=a.num_experts).tolist()
-    tok = order // a.experts_per_token
+    counts = torch.bincount(flat_e, minlength=sp.experts).tolist()
+    tok = order // sp.top
     w_sorted = weights.reshape(-1)[order]
     start = 0
     for e, n in enumerate(counts):
@@ -117,46 +127,60 @@ def _forward_loop(model, lw, x):
     return out.to(x.dtype)
 
 
-def _forward_device(model, lw, x, defer=False):
-    a = model.arch
-    lo, hi = lw.exp_lo, lw.exp_hi or a.num_experts
-    standard = a.moe_style == "standard"
-    mode = 1 if standard and not a.moe_norm_topk else 0
+def _plan(model, lw, x, sp, token_tile=0):
+    """Routing of the tokens, on the device."""
+    lo, hi = lw.exp_lo, lw.exp_hi or sp.experts
     logits = ops.linear(x, lw.router_w, lw.router_b, out_fp32=True)
-    if a.moe_sparse_mixer:
-        tw, ti = sparse_mixer(logits, a.moe_jitter_eps)
-        plan = ops.moe_route(logits, 2, 0, (lo, hi), topk=(ti.to(torch.int32).contiguous(), tw.contiguous()))
-    else:
-        plan = ops.moe_route(logits, a.experts_per_token, mode, (lo, hi))
+    if sp.weights == "sparse_mixer":
+        tw, ti = sparse_mixer(logits, sp.jitter_eps)
+        return ops.moe_route(logits, 2, 0, (lo, hi), token_tile, topk=(ti.to(torch.int32).contiguous(), tw.contiguous()))
+    return ops.moe_route(logits, sp.top, _TOPK_MODES[sp.weights], (lo, hi), token_tile)
+
+
+def _forward_device(model, lw, x, defer=False):
+    sp = spec_of(model, lw)
+    plan = _plan(model, lw, x, sp)
     half = isinstance(lw.exp_gate_up_w, ops.Fp4Experts) and lw.exp_gate_up_w.half and lw.exp_down_w.half
     if half:
         # packed MXFP4 experts in their fp16 form: fp16 rows in, fp16 between the two grouped GEMMs, bf16 out; the streaming
         # kernel of decode-sized steps reads the token rows through the plan's row map instead of a gathered copy
         mapped = _ROW_MAP and ops.moe_fp4_reads_rows(lw.exp_gate_up_w, plan) and x.dtype == torch.bfloat16 and x.stride(0) % 8 == 0
         xs = x if mapped else ops.gather_rows(x, plan.sorted_token, f16=True)
-        h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=a.moe_swiglu_alpha, limit=a.moe_swiglu_limit,
+        h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=sp.alpha, limit=sp.limit,
                          out_dtype=torch.float16, row_map=mapped)
         y = ops.moe_gemm(h, lw.exp_down_w, plan, lw.exp_down_b)
         return ops.PendingCombine(y, plan) if defer else ops.moe_combine(y, plan)
     xs = ops.gather_rows(x, plan.sorted_token)
-    if standard:
+    if sp.act == "silu":
         h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, None, act_kind=1)
     else:
-        h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=a.moe_swiglu_alpha, limit=a.moe_swiglu_limit)
+        h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=sp.alpha, limit=sp.limit)
     y = ops.moe_gemm(h, lw.exp_down_w, plan, lw.exp_down_b)
     return ops.PendingCombine(y, plan) if defer else ops.moe_combine(y, plan)
+
+
+def _forward_simt(model, lw, x):
+    """32-bit models and sizes the tensor-core kernels cannot address: the same steps in plain arithmetic, experts' rows read through the
+    routing plan.  The result is pending: the caller's norm folds the weighted sum."""
+    sp = spec_of(model, lw)
+    plan = _plan(model, lw, x, sp, token_tile=64)
+    gu = ops.moe_gemm_simt(x, lw.exp_gate_up_w, plan, mapped=True)
+    h = ops.expert_act(gu, sp.act, sp.alpha, sp.limit)
+    return ops.PendingCombine(ops.moe_gemm_simt(h, lw.exp_down_w, plan), plan)
 
 
 def moe_forward(model, lw, x: torch.Tensor, defer: bool = False):
     """defer: the caller folds the combine step into the residual add + norm that follows (`ops.norm_moe_combine`); the
     result is then an `ops.PendingCombine` when the layer ran on the device path of a single rank."""
-    a = model.arch
-    fast = x.is_cuda and lw.exp_blocked and a.hidden_size % 8 == 0 and a.num_experts <= 1024 and a.experts_per_token <= 32
+    a, sp = model.arch, spec_of(model, lw)
+    fast = x.is_cuda and lw.exp_blocked and a.hidden_size % 8 == 0 and sp.experts <= 1024 and sp.top <= 32
     if model.tp.size > 1 and getattr(model.tp, "ep_mode", "replicated") == "all_to_all":
         # token-sharded expert parallelism: dispatch / combine all-to-all, the output is complete on every rank
         from ..parallel.ep import moe_all_to_all
         return moe_all_to_all(model, lw, x)
     if fast:
         return _forward_device(model, lw, x, defer and model.tp.size == 1) if model.tp.size == 1 else model.tp.reduce(_forward_device(model, lw, x))
+    if x.is_cuda and lw.moe is not None and defer and model.tp.size == 1:
+        return _forward_simt(model, lw, x)
     out = _forward_loop(model, lw, x)
     return model.tp.reduce(out) if model.tp.size > 1 else out

@@ -53,14 +53,15 @@ def _file_tensors(path: str) -> Callable[[str], torch.Tensor]:
     return get
 
 
-def _synthetic_tensors(path: str, shapes: Dict[str, tuple], device) -> Callable[[str], torch.Tensor]:
+def _synthetic_tensors(path: str, shapes: Dict[str, tuple], device, norm_offset: float = 0.0) -> Callable[[str], torch.Tensor]:
     from .builder import random_tensor
     with open(path) as f:
         meta = json.load(f)
 
     def get(name):
         t = random_tensor(name, shapes[name], int(meta.get("seed", 0)), float(meta.get("std", 0.02)), device=device)
-        return t + 1.0 if name.endswith("norm") or name.endswith("norm1") else t
+        around_one = name.endswith((".norm", "norm1", "norm2")) and (norm_offset == 0 or ".mix." in name) or name.endswith(("ls1", "ls2"))
+        return t + 1.0 if around_one else t
     return get
 
 
@@ -74,13 +75,15 @@ def load_stack_decoder(model_dir: str, filename: str, context_length: int, devic
     arch.context_length = context_length
     path = os.path.join(model_dir, filename)
     shapes = stack_weight_shapes(arch)
-    get = _synthetic_tensors(path, shapes, device) if filename.endswith(".synthetic.json") else _file_tensors(path)
+    get = _synthetic_tensors(path, shapes, device, arch.norm_offset) if filename.endswith(".synthetic.json") else _file_tensors(path)
     return build_stack_decoder(arch, get, device, dtype)
 
 
 def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], device, dtype) -> DecoderModel:
     """DecoderModel from a tensor source: input projections stacked per layer, the key map transposed per head, the output projections
-    of both sub-layers joined side by side, small vectors and recurrence constants in fp32."""
+    of both sub-layers of a parallel block joined side by side, the factors on a sub-layer's normed output multiplied into one vector,
+    experts stacked, heads and feed-forwards filled up with zeros where a kernel wants whole tiles, small vectors and recurrence constants
+    in fp32."""
     shapes = stack_weight_shapes(arch)
     model = DecoderModel(arch, device, dtype)
     cuda = torch.device(device).type == "cuda"
@@ -107,17 +110,70 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         return tables[spec.key()]
 
     up8 = lambda n: (n + 7) // 8 * 8      # columns of the joined input start on 16-byte boundaries
+    tiled = cuda and dtype == torch.bfloat16
+
+    def head_rows(name, heads, size, row):
+        """[heads * size, K] -> [heads * row, K]: every head filled up with zero rows."""
+        w = raw(name).to(dtype)
+        return w if size == row else torch.nn.functional.pad(w.view(heads, size, -1), (0, 0, 0, row - size)).reshape(heads * row, -1)
+
+    def attention_weights(lw, sp, m):
+        lw.qkv_w = torch.cat([head_rows(m + "q", sp.heads, sp.dim, sp.key_row), head_rows(m + "k", sp.kv_heads, sp.dim, sp.key_row),
+                              head_rows(m + "v", sp.kv_heads, sp.vdim, sp.value_row)] + ([raw(m + "g").to(dtype)] if sp.head_gate else []), 0).contiguous()
+        if sp.qk_norm:
+            lw.q_norm_w, lw.k_norm_w = vec(m + "q.norm"), vec(m + "k.norm")
+        if sp.sinks:
+            lw.sinks = vec(m + "sink")
+        lw.rope_cos, lw.rope_sin = rotary(sp.rotary)
+
+    def output_map(name, sp):
+        """The mixer's output map over its heads as they leave the mixer."""
+        w = raw(name).to(dtype)
+        if sp.kind != "attention" or sp.vdim == sp.value_row:
+            return w.contiguous()
+        return torch.nn.functional.pad(w.view(-1, sp.heads, sp.vdim), (0, sp.value_row - sp.vdim)).reshape(w.shape[0], -1).contiguous()
+
+    def output_factor(p, n):
+        """What multiplies a sub-layer's normalised output: norm weight, layer scale and residual multiplier."""
+        w = (vec(f"{p}norm{n}") + arch.norm_offset) * arch.residual_multiplier
+        return w * vec(f"{p}ls{n}") if arch.layer_scale else w
+
+    def feed_forward(lw, sp, p):
+        from ..ops import interleave_gate_up
+        lw.gate_up_w, lw.down_w = mat(p + "gate", p + "up"), mat(p + "down")
+        if tiled:      # whole blocks of 64 features (zero gates and zero ups give zero)
+            fill = (-sp.ff) % 64
+            w = torch.nn.functional.pad(lw.gate_up_w.view(2, sp.ff, -1), (0, 0, 0, fill)).reshape(2 * (sp.ff + fill), -1)
+            lw.gate_up_w, lw.gate_up_interleaved = interleave_gate_up(w), True
+            lw.down_w = torch.nn.functional.pad(lw.down_w, (0, fill)).contiguous()
+
+    def expert_weights(lw, sp, p):
+        from ..ops import interleave_experts_gate_up
+        E, W = sp.moe.experts, arch.hidden_size
+        lw.moe, lw.router_w, lw.exp_hi = sp.moe, mat(p + "router"), E
+        lw.exp_blocked = tiled and W % 8 == 0
+        F = (sp.ff + 63) // 64 * 64 if lw.exp_blocked else sp.ff      # (an expert's zero gates give zero, whatever its ups are)
+        gate_up = torch.zeros(E, 2, F, W, dtype=dtype, device=device)
+        lw.exp_down_w = torch.zeros(E, W, F, dtype=dtype, device=device)
+        for e in range(E):
+            gate_up[e, 0, :sp.ff], gate_up[e, 1, :sp.ff] = raw(f"{p}e{e}.gate").to(dtype), raw(f"{p}e{e}.up").to(dtype)
+            lw.exp_down_w[e, :, :sp.ff] = raw(f"{p}e{e}.down").to(dtype)
+        if lw.exp_blocked:
+            lw.exp_gate_up_w = interleave_experts_gate_up(gate_up.view(E, 2 * F, W), fused_interleaved=False)
+        else:
+            lw.exp_gate_up_w = gate_up.transpose(1, 2).reshape(E, 2 * F, W).contiguous()
 
     def layer(i) -> LayerWeights:
         sp, p, m = arch.layer_specs[i], f"l{i}.", f"l{i}.mix."
-        lw = LayerWeights(ln1_w=vec(p + "norm1"), qkv_w=None, o_w=None, ln2_w=None, ln1_b=vec(p + "norm1.b") if arch.layernorm else None)
-        lw.mix_cols = sp.heads * sp.vdim
-        lw.mlp_col = up8(lw.mix_cols)
+        lw = LayerWeights(ln1_w=None, qkv_w=None, o_w=None, ln2_w=None)
+        lw.mix_cols = sp.heads * (sp.value_row or sp.vdim)
         if sp.kind == "linear_attention":
             lw.lin_in_w = mat(m + "q", m + "k", m + "v", m + "g", m + "b", m + "a")
             lw.lin_conv_w = mat(m + "q.conv", m + "k.conv", m + "v.conv")
             lw.lin_neg_exp_a = -torch.exp(vec(m + "A_log"))
             lw.lin_dt_bias, lw.lin_norm_w = vec(m + "dt_bias"), vec(m + "norm")
+        elif sp.kind == "attention":
+            attention_weights(lw, sp, m)
         else:
             lw.lat_in_w = mat(m + "q", m + "dkv")
             lw.lat_norm_w = vec(m + "dkv.norm")
@@ -125,18 +181,26 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
             lw.lat_ukv = mat(m + "uk", m + "uv")
             lw.lat_uv = lw.lat_ukv[sp.heads * sp.dim:]
             lw.rope_cos, lw.rope_sin = rotary(sp.rotary)
+        if not arch.parallel_block:
+            lw.o_w, lw.post_attn_norm_w = output_map(m + "o", sp), output_factor(p, 1)
+            if sp.ff:
+                (feed_forward if sp.moe is None else expert_weights)(lw, sp, p + "mlp.")
+                lw.post_ffn_norm_w = output_factor(p, 2)
+            return lw
+        lw.ln1_w, lw.ln1_b = vec(p + "norm1"), vec(p + "norm1.b") if arch.layernorm else None
+        lw.mlp_col = up8(lw.mix_cols)
         lw.join_w = torch.zeros(arch.hidden_size, lw.mlp_col + up8(sp.ff), dtype=dtype, device=device)
-        lw.join_w[:, :lw.mix_cols] = raw(m + "o").to(dtype)
+        lw.join_w[:, :lw.mix_cols] = output_map(m + "o", sp)
         if sp.ff:
             lw.join_w[:, lw.mlp_col:lw.mlp_col + sp.ff] = raw(p + "mlp.down").to(dtype)
             lw.gate_up_w = mat(p + "mlp.gate", p + "mlp.up")
-            if cuda and dtype == torch.bfloat16 and sp.ff % 64 == 0:
+            if tiled and sp.ff % 64 == 0:
                 from ..ops import interleave_gate_up
                 lw.gate_up_w, lw.gate_up_interleaved = interleave_gate_up(lw.gate_up_w), True
         return lw
 
     model.embed, model.lm_head_w = mat("embed"), mat("head")
-    model.final_norm_w = vec("final.norm")
+    model.final_norm_w = vec("final.norm") + arch.norm_offset
     model.final_norm_b = vec("final.norm.b") if arch.layernorm else None
     own = {i: layer(i) for i, sp in enumerate(arch.layer_specs) if sp.weights_of is None}
     model.layers = [own[i if sp.weights_of is None else sp.weights_of] for i, sp in enumerate(arch.layer_specs)]

@@ -129,17 +129,40 @@ def embedding(ids: torch.Tensor, table, scale: float = 1.0) -> torch.Tensor:
     return out
 
 
-def embedding_stream(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
-    """Embedding rows as the start of an fp32 residual stream (bf16 or fp32 table, any width)."""
+def embedding_stream(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, dtype=None):
+    """Embedding rows as the start of an fp32 residual stream (bf16 or fp32 table, any width).  With `dtype`: (stream, the rows in that
+    type), the stream itself where it is fp32."""
     _check_index("embedding_stream", "ids", ids, table.shape[0])
     if not table.is_cuda:
-        return ref.embedding(ids, table).float() * scale
+        h = ref.embedding(ids, table).float() * scale
+        return h if dtype is None else (h, h if dtype == torch.float32 else h.to(dtype))
     assert ids.dtype == torch.int32 and table.is_contiguous() and table.dtype in (torch.bfloat16, torch.float32)
     T, H = ids.numel(), table.shape[1]
     out = torch.empty(T, H, dtype=torch.float32, device=table.device)
-    _lib.check(_lib.lib().ogb_embedding_stream(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), T, H, table.shape[0], float(scale),
-                                              _stream()), "embedding_stream")
-    return out
+    copy = torch.empty(T, H, dtype=torch.bfloat16, device=table.device) if dtype == torch.bfloat16 else None
+    _lib.check(_lib.lib().ogb_embedding_stream(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), _ptr(copy), T, H, table.shape[0],
+                                              float(scale), _stream()), "embedding_stream")
+    return out if dtype is None else (out, out if copy is None else copy)
+
+
+def add_normed(h, y, weight, eps, dtype=torch.bfloat16):
+    """h += weight * v / rms(v) in place: the normed output of a sub-layer joins the fp32 residual stream h [T, H].  v = y [T, H], or the
+    weighted sum of a mixture-of-experts layer whose combine step is pending.  weight fp32 [H].  Returns the new stream in `dtype` (the
+    stream itself where that is fp32)."""
+    if not h.is_cuda:
+        ref.add_normed(h, y, weight, eps)
+        return h if dtype == torch.float32 else h.to(dtype)
+    plan = None
+    if isinstance(y, PendingCombine):
+        y, plan = y.y, y.plan
+    T, H = h.shape
+    assert h.dtype == torch.float32 and h.is_contiguous() and weight.dtype == torch.float32 and y.stride(1) == 1 and y.shape[1] == H
+    assert y.dtype in (torch.bfloat16, torch.float32) and (plan is None or plan.T == T)
+    x = torch.empty(T, H, dtype=torch.bfloat16, device=h.device) if dtype == torch.bfloat16 else None
+    _lib.check(_lib.lib().ogb_add_normed(_ptr(h), _ptr(y), y.stride(0), int(y.dtype == torch.float32), _ptr(weight), float(eps), _ptr(x),
+                                        _ptr(plan.inv_pos) if plan else None, _ptr(plan.topk_w) if plan else None, plan.k if plan else 0, T, H, _stream()),
+               "add_normed")
+    return h if x is None else x
 
 
 def norm_stream(x, weight, eps, bias=None, layernorm=False, dtype=torch.bfloat16, rows=None):
@@ -199,7 +222,7 @@ def norm_moe_combine(pending: PendingCombine, weight, eps, residual, bias=None, 
 
 
 # ------------------------------------------------------------------------------------------ GEMM
-GEMM_FP32_OUT, GEMM_ACT_PAIR, GEMM_ALLREDUCE, GEMM_REDUCE_SCATTER, GEMM_GATHERED_A, GEMM_FP32_RESIDUAL, GEMM_PAIR_RELU = 1, 2, 4, 8, 16, 32, 64
+GEMM_FP32_OUT, GEMM_ACT_PAIR, GEMM_ALLREDUCE, GEMM_REDUCE_SCATTER, GEMM_GATHERED_A, GEMM_FP32_RESIDUAL, GEMM_PAIR_RELU, GEMM_PAIR_GELU = 1, 2, 4, 8, 16, 32, 64, 128
 
 
 FUSED_MAX_TOKENS = 128     # the decode-step fusions (folded norm, rotary + cache append) run in the decode-sized GEMM kernel
@@ -378,6 +401,9 @@ def interleave_gate_up(w: torch.Tensor, block: int = 64) -> torch.Tensor:
     return torch.cat([g, u], dim=1).reshape(w.shape).contiguous()
 
 
+_PAIR_FLAGS = {"silu": 0, "relu": GEMM_PAIR_RELU, "gelu_tanh": GEMM_PAIR_GELU, "gelu": GEMM_PAIR_GELU}      # activations the GEMM's epilogue pairs
+
+
 def gate_up_act(x, w, bias=None, act="silu", out=None, splits=0, interleaved=False, norm_eps=0.0):
     """act(x @ Wg.T) * (x @ Wu.T).  w is [2I, K]: stacked [Wg; Wu], or (interleaved=True) blocks of 64 gate
     rows + 64 up rows as produced by interleave_gate_up (the layout the fused kernel needs).  norm_eps: as in `linear`."""
@@ -406,14 +432,14 @@ def gate_up_act(x, w, bias=None, act="silu", out=None, splits=0, interleaved=Fal
         y = ref.gate_up_act(x, w, bias, act, interleaved)
         return y if out is None else out.copy_(y)
     inter = w.shape[0] // 2
-    if act not in ("silu", "relu") or not interleaved or inter % 64 or x.dtype != torch.bfloat16 or not _tma_ok(x, w):
+    if act not in _PAIR_FLAGS or not interleaved or inter % 64 or x.dtype != torch.bfloat16 or not _tma_ok(x, w):
         y = linear(x, w, bias)
         if interleaved:
             y = y.view(-1, inter // 64, 2, 64).transpose(1, 2).reshape(-1, 2 * inter)
         return act_mul(y.contiguous(), act, out)
     if out is None:
         out = torch.empty(x.shape[0], inter, dtype=torch.bfloat16, device=x.device)
-    return _gemm(x, w, out, bias, None, GEMM_ACT_PAIR | (GEMM_PAIR_RELU if act == "relu" else 0), splits, fused)
+    return _gemm(x, w, out, bias, None, GEMM_ACT_PAIR | _PAIR_FLAGS[act], splits, fused)
 
 
 def act_mul(x, act="silu", out=None):
@@ -698,6 +724,29 @@ def moe_gemm(xs: torch.Tensor, w: torch.Tensor, plan: MoePlan, bias=None, act_ki
     return out
 
 
+def moe_gemm_simt(xs: torch.Tensor, w: torch.Tensor, plan: MoePlan, mapped: bool = False) -> torch.Tensor:
+    """Grouped expert product in plain arithmetic (fp32, or bf16 sizes TMA cannot address): w [E, N, K]; xs holds the rows sorted by expert,
+    or (mapped) the token rows, read through the plan.  Returns [T * k, N] in xs's type."""
+    E, N, K = w.shape
+    assert xs.is_cuda and xs.dtype == w.dtype and xs.stride(1) == 1 and w.is_contiguous() and xs.dtype in (torch.float32, torch.bfloat16)
+    assert plan.bt <= 64 and xs.shape[1] == K
+    out = torch.empty(plan.T * plan.k, N, dtype=xs.dtype, device=xs.device)
+    _lib.check(_lib.lib().ogb_moe_gemm_simt(_ptr(xs), xs.stride(0), _ptr(w), _ptr(out), N, N, K, _ptr(plan.tile_expert), _ptr(plan.tile_row0),
+                                           _ptr(plan.tile_rows), _ptr(plan.num_tiles), plan.max_tiles, plan.bt, _ptr(plan.sorted_token) if mapped else None,
+                                           int(xs.dtype == torch.float32), _stream()), "moe_gemm_simt")
+    return out
+
+
+def expert_act(gu: torch.Tensor, kind: str, alpha: float = 1.702, limit: float = 0.0) -> torch.Tensor:
+    """Activation of expert rows whose columns alternate (gate, up): [n, 2 I] -> [n, I]."""
+    assert gu.is_cuda and gu.is_contiguous()
+    n, inter = gu.shape[0], gu.shape[1] // 2
+    out = torch.empty(n, inter, dtype=gu.dtype, device=gu.device)
+    _lib.check(_lib.lib().ogb_expert_act(_ptr(gu), _ptr(out), n, inter, {"silu": 0, "clamped": 1}[kind], float(alpha), float(limit),
+                                        int(gu.dtype == torch.float32), _stream()), "expert_act")
+    return out
+
+
 def moe_combine(y: torch.Tensor, plan: MoePlan, residual=None) -> torch.Tensor:
     """out[t] = (residual[t]) + sum_j w[t, j] * y[row(t, j)]; rows of experts that are not local are skipped."""
     out = torch.empty(plan.T, y.shape[1], dtype=torch.bfloat16, device=y.device)
@@ -735,6 +784,25 @@ def rope_kv_append(qkv, positions, slots, cos_cache, sin_cache, k_cache, v_cache
     return qkv
 
 
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache):
+    """Between the projection [Hq queries | Hkv keys | Hkv values | ...] of an attention layer and its attention: RMS norm of every query and
+    key head over its `dim` columns (weights fp32 [dim] or None), rotation of the first 2 * cos.shape[1] of them (cos / sin fp32 [positions,
+    rot / 2], or None), queries in place, keys and values to row slots[t] of the caches [slots, Hkv, key_row] and [slots, Hkv, value_row]
+    (slot < 0: to no row).  Any sizes, bf16 or fp32."""
+    _check_index("qkv_prep", "slots", slots[:proj.shape[0]], k_cache.shape[0], -1)
+    if cos is not None:
+        _check_index("qkv_prep", "positions", positions[:proj.shape[0]], cos.shape[0])
+    if not proj.is_cuda:
+        return ref.qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache)
+    assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == proj.dtype
+    assert proj.dtype in (torch.bfloat16, torch.float32) and all(w is None or w.dtype == torch.float32 for w in (q_norm_w, k_norm_w, cos, sin))
+    _lib.check(_lib.lib().ogb_qkv_prep(_ptr(proj), proj.stride(0), Hq, Hkv, dim, key_row, value_row, _ptr(q_norm_w), _ptr(k_norm_w), float(eps),
+                                      _ptr(positions), _ptr(cos), _ptr(sin), 2 * cos.shape[1] if cos is not None else 0,
+                                      cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(k_cache), _ptr(v_cache), proj.shape[0],
+                                      int(proj.dtype == torch.float32), _stream()), "qkv_prep")
+    return proj
+
+
 # ------------------------------------------------------------------------------------------ attention
 def choose_kv_splits(batch: int, Hkv: int, max_q_len: int, max_kv_len: int, sm_count: int = 148, group: int = 1, ordered: bool = False):
     """(splits, kv_chunk) of a paged-attention launch.  A launch whose (request, kv head) grid already fills the GPU
@@ -769,15 +837,22 @@ _TC_ATTENTION = os.environ.get("OGB_ATTN_TC", "1") != "0"
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale, window=0,
                     sinks=None, softcap=0.0, max_q_len=None, max_kv_len=None, splits=None, out=None, total_tokens=None, order=None,
-                    min_q_len=None):
+                    min_q_len=None, vdim=None, chunk=0, gate=None):
     """q: [T, stride] with the Hq*D query columns first.  Returns [T, Hq*D].  total_tokens: the requests of this call only cover
     the first `total_tokens` rows of q (sizes the split-KV scratch).  min_q_len: shortest request of the call when the caller
-    knows it (a call whose every request is long runs on the tensor-core prefill kernel alone)."""
+    knows it (a call whose every request is long runs on the tensor-core prefill kernel alone).  vdim (layers with sizes of their own): width
+    of a value head; chunk > 0: position p sees the keys from p // chunk * chunk on; gate [T, Hq]: each head's output is multiplied by its
+    sigmoid."""
     _check_index("paged_attention", "block_table", block_table, k_cache.shape[0] // block_size, -1)
     _check_index("paged_attention", "cu_seqlens", cu_seqlens[:past_lens.shape[0] + 1], q.shape[0] + 1)
     if not q.is_cuda:
-        return ref.paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                                   window, sinks, softcap)
+        o = ref.paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
+                                window, sinks, softcap, vdim, chunk, gate)
+        return o if out is None else out.copy_(o)
+    if vdim is not None or chunk > 0 or gate is not None:
+        assert softcap == 0.0
+        return _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, vdim or D, scale, window, chunk,
+                                      sinks, gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len)
     T = q.shape[0] if total_tokens is None else total_tokens
     B = past_lens.shape[0]
     if out is None:
@@ -825,6 +900,51 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
     _lib.check(rc, "paged_attention")
     if splits > 1:
         _lib.LAUNCH_COUNT += 1  # the combine kernel
+    return out
+
+
+def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, dk, dv, scale, window, chunk, sinks, gate,
+                           max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len):
+    """paged_attention of layers with sizes of their own: the tensor-memory kernel for requests with at least TC_ATTENTION_MIN_ROWS query
+    rows, the warp-MMA kernel for the others, plain arithmetic for fp32 and for sizes neither can address."""
+    import ctypes
+    T = q.shape[0] if total_tokens is None else total_tokens
+    B = past_lens.shape[0]
+    if out is None:
+        out = torch.empty(q.shape[0], Hq * dv, dtype=q.dtype, device=q.device)
+    max_q_len = max_q_len or T
+    L, G, ws = _lib.lib(), Hq // Hkv, workspace(q.device)
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and out.stride(1) == 1 and block_table.stride(1) == 1
+    assert sinks is None or sinks.dtype == torch.float32
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
+    layer = _lib.AttnLayer(Hq=Hq, Hkv=Hkv, dk=dk, dv=dv, window=int(window), chunk=int(chunk), gate_stride=gate.stride(0) if gate is not None else 0,
+                           scale=float(scale), sinks=_ptr(sinks), gate=_ptr(gate))
+    inputs = (ctypes.byref(layer), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(cu_seqlens), _ptr(past_lens), _ptr(block_table),
+              block_table.stride(0), int(block_size), _ptr(out), out.stride(0), B)
+    if (q.dtype == torch.float32 or not L.ogb_attention_mixed_supported(dk, dv) or q.stride(0) % 8 or out.stride(0) % 2 or q.data_ptr() % 16 or
+            out.data_ptr() % 4):
+        # (the grid covers the rows of the whole matrix: rows of requests outside this call are skipped)
+        _lib.check(L.ogb_attention_simt(*inputs, q.shape[0], int(q.dtype == torch.float32), _stream()), "attention_simt")
+        return out
+    slots = int(k_cache.shape[0])
+    long_rows = TC_ATTENTION_MIN_ROWS
+    use_tc = (_TC_ATTENTION and max_q_len * G >= long_rows and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and
+              bool(L.ogb_attention_tc_mixed_supported(dk, dv, int(block_size), slots)))
+    if not (use_tc and min_q_len is not None and min_q_len * G >= long_rows):
+        # (first: with splits the combine pass leaves unspecified values in the rows of the long requests)
+        if splits is None:
+            span = max_kv_len or 1024
+            if chunk > 0:
+                span = min(span, chunk + 63)
+            splits = choose_kv_splits(B, Hkv, max_q_len, span, group=G, ordered=order is not None)
+        sp, ch = splits if isinstance(splits, tuple) else (splits, 0)
+        scratch = ws.attn_scratch(L.ogb_attention_scratch_bytes(T, Hq, dv, sp)) if sp > 1 else None
+        _lib.check(L.ogb_attention_mixed(*inputs, T, int(max_q_len), int(sp), int(ch), _ptr(scratch), scratch.numel() if scratch is not None else 0,
+                                         _ptr(order), ws.status, _stream(), long_rows if use_tc else 0), "attention_mixed")
+        if sp > 1:
+            _lib.LAUNCH_COUNT += 1      # the combine kernel
+    if use_tc:
+        _lib.check(L.ogb_attention_tc_mixed(*inputs, int(max_q_len), long_rows, slots, ws.status, _stream()), "attention_tc_mixed")
     return out
 
 

@@ -29,7 +29,13 @@ class LatentShape(ctypes.Structure):
     _fields_ = [(n, c_int) for n in ("H", "dim", "rot", "vdim", "R", "rot_dims")]
 
 
+class AttnLayer(ctypes.Structure):
+    """OgbAttnLayer of csrc/kernels.h: an attention layer with sizes and a mask of its own."""
+    _fields_ = [(n, c_int) for n in ("Hq", "Hkv", "dk", "dv", "window", "chunk", "gate_stride")] + [("scale", c_float), ("sinks", _P), ("gate", _P)]
+
+
 _LS = ctypes.POINTER(LatentShape)
+_AL = ctypes.POINTER(AttnLayer)
 
 _SIGS = {
     "ogb_runtime_init": (c_int, [c_int]),
@@ -74,7 +80,17 @@ _SIGS = {
     "ogb_causal_conv_rows": (c_int, [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P]),
     "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_int, _P]),
-    "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, c_int, c_int, c_int, c_float, _P]),
+    "ogb_moe_gemm_simt": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P]),
+    "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_float, _P]),
+    "ogb_add_normed": (c_int, [_P, _P, c_int, c_int, _P, c_float, _P, _P, _P, c_int, c_int, c_int, _P]),
+    "ogb_qkv_prep": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, _P]),
+    "ogb_expert_act": (c_int, [_P, _P, c_longlong, c_int, c_int, c_float, c_float, c_int, _P]),
+    "ogb_attention_mixed_supported": (c_int, [c_int, c_int]),
+    "ogb_attention_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P,
+                                    _P, c_int]),
+    "ogb_attention_tc_mixed_supported": (c_int, [c_int, c_int, c_int, c_int]),
+    "ogb_attention_tc_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, _P]),
+    "ogb_attention_simt": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P]),
     "ogb_norm_stream": (c_int, [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P]),
     "ogb_act_mul_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_latent_prep": (c_int, [_P, c_int, _LS, _P, c_float, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P]),

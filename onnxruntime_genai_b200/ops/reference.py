@@ -200,15 +200,16 @@ def kv8_load(cache, Hkv, D):
 
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                    window=0, sinks=None, softcap=0.0):
-    """q: [T, >=Hq*D] (only the first Hq*D columns are read).  Returns [T, Hq*D]."""
-    T = q.shape[0]
-    out = torch.zeros(T, Hq * D, dtype=q.dtype, device=q.device)
+                    window=0, sinks=None, softcap=0.0, vdim=None, chunk=0, gate=None):
+    """q: [T, >=Hq*D] (only the first Hq*D columns are read).  vdim: width of a value head (None: D).  chunk > 0: position p sees the keys
+    from p // chunk * chunk on.  gate [T, Hq]: each head's output is multiplied by its sigmoid.  Returns [T, Hq*vdim]."""
+    T, DV = q.shape[0], vdim or D
+    out = torch.zeros(T, Hq * DV, dtype=q.dtype, device=q.device)
     if k_cache.dtype == torch.int8:
         kc, vc = kv8_load(k_cache, Hkv, D), kv8_load(v_cache, Hkv, D)
     else:
         kc = k_cache.view(-1, Hkv, D)
-        vc = v_cache.view(-1, Hkv, D)
+        vc = v_cache.view(-1, Hkv, DV)
     G = Hq // Hkv
     B = past_lens.shape[0]
     cu = cu_seqlens.tolist()
@@ -234,6 +235,8 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
         mask = (pos[None, :] <= qpos[:, None]) | full
         if window and window > 0:
             mask = mask & (pos[None, :] > qpos[:, None] - window)
+        if chunk > 0:
+            mask = mask & (pos[None, :] >= (qpos // chunk * chunk)[:, None])
         s = s.masked_fill(~mask[None], float("-inf"))
         if sinks is not None:
             sk = sinks.float().view(Hq, 1, 1).expand(Hq, n, 1)
@@ -241,7 +244,9 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
         else:
             p = torch.softmax(s, dim=-1)
         o = torch.einsum("hqk,khd->qhd", p, v)
-        out[t0:t1] = o.reshape(n, Hq * D).to(q.dtype)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t0:t1].float())[:, :, None]
+        out[t0:t1] = o.reshape(n, Hq * DV).to(q.dtype)
     return out
 
 
@@ -388,6 +393,31 @@ def head_project(x, w, heads, a_cols):
     """out[:, h * N + n] = sum_k x[:, h * a_cols + k] * w[h * N + n, k]."""
     N, K = w.shape[0] // heads, w.shape[1]
     return torch.cat([x[:, h * a_cols:h * a_cols + K].float() @ w[h * N:(h + 1) * N].float().t() for h in range(heads)], 1).to(x.dtype)
+
+
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache):
+    T, nq, nk = proj.shape[0], Hq * key_row, Hkv * key_row
+    q, k, v = proj[:, :nq].view(T, Hq, key_row), proj[:, nq:nq + nk].view(T, Hkv, key_row), proj[:, nq + nk:nq + nk + Hkv * value_row]
+    pos = positions.long().clamp(0, cos.shape[0] - 1) if cos is not None else None
+
+    def prepared(x, w):
+        x = x.float()
+        y = x.clone()
+        if w is not None:
+            y[..., :dim] = x[..., :dim] * torch.rsqrt(x[..., :dim].pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        return _rotate(y, cos[pos], sin[pos], 2 * cos.shape[1], False) if cos is not None else y
+    q.copy_(prepared(q, q_norm_w).to(proj.dtype))
+    ok = slots >= 0
+    at = slots[ok].long()
+    k_cache[at] = prepared(k, k_norm_w)[ok].to(k_cache.dtype)
+    v_cache[at] = v.view(T, Hkv, value_row)[ok].to(v_cache.dtype)
+    return proj
+
+
+def add_normed(h, y, weight, eps):
+    """h + weight * y / rms(y), in place."""
+    y = y.float()
+    return h.add_(y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight)
 
 
 def latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache):

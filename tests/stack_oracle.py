@@ -1,5 +1,6 @@
-"""A slow, plain restatement of declared-stack decoders (gated-delta and latent-attention mixers in parallel blocks), one function
-per mechanism, token by token where the mechanism is a recurrence.  It shares no code with the package: the tests compare the
+"""A slow, plain restatement of declared-stack decoders (gated-delta and latent-attention mixers in parallel blocks; chunked attention
+with sinks and routed experts in blocks whose norms follow the sub-layers), one function per mechanism, token by token where the
+mechanism is a recurrence.  It shares no code with the package: the tests compare the
 runtime against it.  Weights come as a dictionary of tensors under the checkpoint's names; all math runs in `dtype` (float64 by
 default).  A whole sequence is evaluated at once, from its first token: there is no cache here."""
 import math
@@ -64,6 +65,18 @@ def delta_mixer(x, w, p, m, eps):
     return o.reshape(T, H * dv) @ w[p + "o"].T
 
 
+def wavelength_scaled(f, s):
+    """Frequency f slowed down by s["factor"] where its wavelength is long against the original context, kept where it is short, blended
+    between."""
+    wave = 2 * math.pi / f
+    if wave < s["original"] / s["high"]:
+        return f
+    if wave > s["original"] / s["low"]:
+        return f / s["factor"]
+    keep = (s["original"] / wave - s["low"]) / (s["high"] - s["low"])
+    return keep * f + (1 - keep) * f / s["factor"]
+
+
 def rotary_frequencies(rot):
     """(frequency of every pair, factor on cos and sin)."""
     d, base = rot["dims"], rot["base"]
@@ -71,6 +84,8 @@ def rotary_frequencies(rot):
     s = rot.get("scaling")
     if not s:
         return f, 1.0
+    if "low" in s:
+        return [wavelength_scaled(fi, s) for fi in f], 1.0
 
     def turns(t):
         return d * math.log(s["original"] / (2 * math.pi * t)) / (2 * math.log(base))
@@ -122,26 +137,100 @@ def latent_mixer(x, w, p, m, eps):
     return out.reshape(T, H * dv) @ w[p + "o"].T
 
 
+def same_chunk(T, size):
+    """ok[i, j]: j is not after i and in the same run of `size` positions (runs are counted from position 0)."""
+    ok = torch.zeros(T, T, dtype=torch.bool)
+    for i in range(T):
+        ok[i, i // size * size:i + 1] = True
+    return ok
+
+
+def sink_attention(q, k, v, ok, scale, sink):
+    """q [T, H, d], k [T, G, d], v [T, G, dv]; sink [H]: a logit in the denominator that has no key and no value."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        g = h // (H // G)
+        s = (q[:, h] @ k[:, g].T * scale).masked_fill(~ok, -math.inf)
+        top = torch.maximum(s.max(-1).values, sink[h])[:, None]
+        e = torch.exp(s - top)
+        out[:, h] = (e @ v[:, g]) / (e.sum(-1, keepdim=True) + torch.exp(sink[h] - top))
+    return out
+
+
+def attention_mixer(x, w, p, m, eps):
+    T, H, G, d, dv = x.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = rms_norm((x @ w[p + "q"].T).view(T, H, d), w[p + "q.norm"], eps)
+    k = rms_norm((x @ w[p + "k"].T).view(T, G, d), w[p + "k.norm"], eps)
+    v = (x @ w[p + "v"].T).view(T, G, dv)
+    q, k = rotate(q, m.get("rot")), rotate(k, m.get("rot"))
+    o = sink_attention(q, k, v, same_chunk(T, m["mask"]["size"]), m["scale"], w[p + "sink"])
+    o = o * torch.sigmoid(x @ w[p + "g"].T)[:, :, None]
+    return o.reshape(T, H * dv) @ w[p + "o"].T
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def gelu_feed_forward(x, w, p, m=None):
+    return (gelu_tanh(x @ w[p + "gate"].T) * (x @ w[p + "up"].T)) @ w[p + "down"].T
+
+
+def clamped_expert(x, w, p, limit):
+    g, u = (x @ w[p + "gate"].T).clamp(max=limit), (x @ w[p + "up"].T).clamp(-limit, limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1)) @ w[p + "down"].T
+
+
+def routed_experts(x, w, p, m):
+    """Each token: the `top` experts of largest probability, weighted by their probabilities among all experts."""
+    s = torch.softmax(x @ w[p + "router"].T, -1)
+    out = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        for e in torch.argsort(s[t], descending=True)[:m["router"]["top"]].tolist():
+            out[t] = out[t] + s[t, e] * clamped_expert(x[t:t + 1], w, f"{p}e{e}.", m["expert"]["limit"])[0]
+    return out
+
+
 def feed_forward(x, w, p):
     return (torch.relu(x @ w[p + "gate"].T) * (x @ w[p + "up"].T)) @ w[p + "down"].T
 
 
 # ------------------------------------------------------------------------------------------------ the stack
-MIXERS = {"delta": delta_mixer, "latent_attention": latent_mixer}
+MIXERS = {"delta": delta_mixer, "latent_attention": latent_mixer, "attention": attention_mixer}
+FEED_FORWARDS = {"dense": gelu_feed_forward, "moe": routed_experts}
+
+
+def parallel_block(x, w, p, e, eps, cfg):
+    h = layer_norm(x, w[p + "norm1"], w[p + "norm1.b"], eps)
+    y = MIXERS[e["type"]](h, w, p + "mix.", e["mixer"], eps)
+    if e.get("mlp"):
+        y = y + feed_forward(h, w, p + "mlp.")
+    return x + y
+
+
+def output_normed_block(x, w, p, e, eps, cfg):
+    """The sub-layers read the stream itself; their results are normed, scaled per element and by the model's multiplier, and added."""
+    m = cfg["residual_mult"]
+    x = x + m * w[p + "ls1"] * rms_norm(MIXERS[e["type"]](x, w, p + "mix.", e["mixer"], eps), 1 + w[p + "norm1"], eps)
+    if e.get("mlp"):
+        x = x + m * w[p + "ls2"] * rms_norm(FEED_FORWARDS[e["mlp"]["kind"]](x, w, p + "mlp.", e["mlp"]), 1 + w[p + "norm2"], eps)
+    return x
 
 
 def stack_forward(cfg, weights, tokens, dtype=torch.float64):
     """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
     w = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
-    x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+    x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
+    block = {"Luzatar": parallel_block, "Zevopel": output_normed_block}[cfg["architecture"]]
     streams = []
     for i, e in enumerate(cfg["layers"]):
         p = f"l{e.get('weights_of', i) if e.get('weights_of') is not None else i}."
-        h = layer_norm(x, w[p + "norm1"], w[p + "norm1.b"], eps)
-        y = MIXERS[e["type"]](h, w, p + "mix.", e["mixer"], eps)
-        if e.get("mlp"):
-            y = y + feed_forward(h, w, p + "mlp.")
-        x = x + y
+        x = block(x, w, p, e, eps, cfg)
         streams.append(x)
-    return layer_norm(x, w["final.norm"], w["final.norm.b"], eps) @ w["head"].T, torch.stack(streams)
+    if cfg["architecture"] == "Luzatar":
+        x = layer_norm(x, w["final.norm"], w["final.norm.b"], eps)
+    else:
+        x = rms_norm(x, 1 + w["final.norm"], eps)
+    return x @ w["head"].T, torch.stack(streams)
