@@ -1,0 +1,121 @@
+"""What the tests of the declared stacks share: the runtimes they run on, models and engines over small random checkpoints, feeding a
+sequence in portions, paged inputs for single ops, and the comparison with the plain restatement (stack_oracle.py)."""
+import json
+
+import numpy as np
+import pytest
+import torch
+
+import onnxruntime_genai_b200 as og
+from stack_models import weights, write
+from stack_oracle import stack_forward
+
+RUNTIMES = [pytest.param(("cpu", "float32"), id="cpu"), pytest.param(("cuda", "float32"), id="cuda_fp32", marks=pytest.mark.gpu),
+            pytest.param(("cuda", "bfloat16"), id="cuda_bf16", marks=pytest.mark.gpu)]
+BLOCK = 16
+
+
+@pytest.fixture(autouse=True, scope="module")
+def one_thread():
+    """The matrices here are tiny: more threads than one only wait for each other.  (A test file takes this fixture by importing it.)"""
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
+
+def tol_of(runtime):
+    return 4e-2 if runtime[1] == "bfloat16" else 2e-4
+
+
+def dtype_of(runtime):
+    return torch.bfloat16 if runtime[1] == "bfloat16" else torch.float32
+
+
+def close(got, want, tol):
+    """Root mean square error of every row against the rows' own spread."""
+    got, want = got.double().cpu(), want.double().cpu()
+    assert got.shape == want.shape
+    err = (got - want).pow(2).mean(-1).sqrt() / want.std()
+    assert torch.isfinite(err).all() and float(err.max()) < tol, f"row {int(err.argmax())}: {float(err.max()):.3g} (limit {tol})"
+
+
+_CACHE = {}
+
+
+def open_model(tmp_path_factory, name, runtime, cfg, w=None):
+    """(model, configuration, weights) of a random checkpoint, opened once per runtime."""
+    key = (name, runtime)
+    if key not in _CACHE:
+        # (16-bit rounding must not decide which experts run: their routers get clear cases)
+        w = w or weights(cfg, seed=sum(map(ord, name)), clear_routes=runtime[1] == "bfloat16")
+        d = write(cfg, w, tmp_path_factory.mktemp(name))
+        c = og.Config(d, provider="cpu" if runtime[0] == "cpu" else "cuda")
+        if runtime[0] == "cuda":
+            c.set_provider_option("cuda", "compute_dtype", runtime[1])
+        _CACHE[key] = (og.Model(c), cfg, w)
+    return _CACHE[key]
+
+
+def open_engine(model, blocks=64, batch=4, tokens=512):
+    model.config.overlay(json.dumps({"engine": {"dynamic_batching": {"block_size": BLOCK, "num_blocks": blocks, "max_batch_size": batch,
+                                                                     "max_scheduled_tokens": tokens}}}))
+    return og.Engine(model)
+
+
+def random_tokens(cfg, n, seed=0):
+    return np.random.RandomState(seed).randint(0, cfg["vocab"], n)
+
+
+def feed(engine, model, toks, cuts):
+    """Logits of every token of one sequence fed in portions of the given sizes (the last size repeats)."""
+    r, at, out, i = og.Request(og.GeneratorParams(model)), 0, [], 0
+    while at < len(toks):
+        n = min(cuts[min(i, len(cuts) - 1)], len(toks) - at)
+        out.append(engine.run_given([(r, toks[at:at + n], list(range(n)))])[0])
+        at, i = at + n, i + 1
+    engine.remove_request(r)
+    return torch.cat(out).float().cpu()
+
+
+def paged(lens, blocks, seed=0):
+    """Block tables with shuffled blocks for requests of the given (past, new) lengths; slots and positions of the new tokens."""
+    order = np.random.RandomState(seed).permutation(blocks)
+    cols = max((p + n + BLOCK - 1) // BLOCK for p, n in lens)
+    table, at = np.full((len(lens), cols), -1, dtype=np.int32), 0
+    pos, slots = [], []
+    for b, (p, n) in enumerate(lens):
+        k = (p + n + BLOCK - 1) // BLOCK
+        table[b, :k] = order[at:at + k]
+        at += k
+        pos += list(range(p, p + n))
+    cu = np.cumsum([0] + [n for _, n in lens])
+    for b, (p, n) in enumerate(lens):
+        slots += [int(table[b, q // BLOCK]) * BLOCK + q % BLOCK for q in range(p, p + n)]
+    t = lambda x: torch.tensor(np.asarray(x), dtype=torch.int32)
+    return dict(table=t(table), pos=t(pos), slots=t(slots), cu=t(cu), past=t([p for p, _ in lens]))
+
+
+def rows_of(pg, b, n):
+    q = np.arange(n)
+    return torch.tensor(pg["table"][b].numpy()[q // BLOCK] * BLOCK + q % BLOCK).long()
+
+
+def greedy_ok(cfg, w, prompt, generated, tol):
+    """Every generated token is the oracle's argmax, or within rounding of it."""
+    lg = stack_forward(cfg, w, np.concatenate([prompt, generated]))[0]
+    for i, t in enumerate(generated):
+        row = lg[len(prompt) - 1 + i]
+        assert float(row.max() - row[int(t)]) <= tol * float(lg.std()), f"token {i}"
+
+
+def beam_search(cfg, w, prompt, n, beams):
+    """Plain beam search over the restatement: the best hypothesis of n tokens."""
+    hyps = [(0.0, list(map(int, prompt)))]
+    while len(hyps[0][1]) < n:
+        cand = []
+        for score, s in hyps:
+            row = torch.log_softmax(stack_forward(cfg, w, s)[0][-1], -1)
+            cand += [(score + float(v), s + [int(t)]) for v, t in zip(*torch.topk(row, beams))]
+        hyps = sorted(cand, key=lambda c: -c[0])[:beams]
+    return np.asarray(hyps[0][1])

@@ -103,12 +103,11 @@ def rotate(x, rot):
         return x
     f, amp = rotary_frequencies(rot)
     half = rot["dims"] // 2
-    y = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(half):
-            c, s = math.cos(t * f[i]) * amp, math.sin(t * f[i]) * amp
-            u, v = x[t, :, i], x[t, :, i + half]
-            y[t, :, i], y[t, :, i + half] = u * c - v * s, v * c + u * s
+    y, pos = x.clone(), torch.arange(x.shape[0], dtype=torch.float64)[:, None]
+    for i in range(half):
+        c, s = (torch.cos(pos * f[i]) * amp).to(x.dtype), (torch.sin(pos * f[i]) * amp).to(x.dtype)
+        u, v = x[:, :, i], x[:, :, i + half]
+        y[:, :, i], y[:, :, i + half] = u * c - v * s, v * c + u * s
     return y
 
 

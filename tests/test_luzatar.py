@@ -13,33 +13,13 @@ import onnxruntime_genai_b200 as og
 from onnxruntime_genai_b200 import ops
 from onnxruntime_genai_b200.models import arch as A
 from onnxruntime_genai_b200.models.decoder import PagedKVCache
+from stack_harness import BLOCK, RUNTIMES, beam_search, close, dtype_of, feed, greedy_ok, one_thread, open_engine, open_model, paged, random_tokens, rows_of, tol_of  # noqa: F401
 from stack_models import delta, latent, stack, weights, write
 from stack_oracle import causal_conv_silu, delta_recurrence, layer_norm, rms_norm, rotary_frequencies, rotate, stack_forward, unit_vectors, visible
-
-RUNTIMES = [pytest.param(("cpu", "float32"), id="cpu"), pytest.param(("cuda", "float32"), id="cuda_fp32", marks=pytest.mark.gpu),
-            pytest.param(("cuda", "bfloat16"), id="cuda_bf16", marks=pytest.mark.gpu)]
-BLOCK = 16
-
 
 @pytest.fixture(params=RUNTIMES)
 def runtime(request):
     return request.param
-
-
-def _tol(runtime):
-    return 4e-2 if runtime[1] == "bfloat16" else 2e-4
-
-
-def _dtype(runtime):
-    return torch.bfloat16 if runtime[1] == "bfloat16" else torch.float32
-
-
-def _close(got, want, tol):
-    """Root mean square error of every row against the rows' own spread."""
-    got, want = got.double().cpu(), want.double().cpu()
-    assert got.shape == want.shape
-    err = (got - want).pow(2).mean(-1).sqrt() / want.std()
-    assert torch.isfinite(err).all() and float(err.max()) < tol, f"row {int(err.argmax())}: {float(err.max()):.3g} (limit {tol})"
 
 
 # ------------------------------------------------------------------------------------------------ models and engines
@@ -54,43 +34,6 @@ WIDE = stack([latent(heads=4, dim=56, rot_dim=24, vdim=64, kv_rank=88, window=50
               latent(heads=3, dim=136, rot_dim=64, vdim=128, kv_rank=384, window=33, ff=0, scale=0.2), delta(heads=2, kv_heads=1, dim=128, vdim=64, ff=64)],
              vocab=160, width=128)
 STACKS = {"mixed": MIXED, "odd": ODD, "wide": WIDE}
-_CACHE = {}
-
-
-def _model(tmp_path_factory, name, runtime, cfg=None, w=None):
-    key = (name, runtime)
-    if key not in _CACHE:
-        cfg = cfg or STACKS[name]
-        w = w or weights(cfg, seed=sum(map(ord, name)))
-        d = write(cfg, w, tmp_path_factory.mktemp(name))
-        c = og.Config(d, provider="cpu" if runtime[0] == "cpu" else "cuda")
-        if runtime[0] == "cuda":
-            c.set_provider_option("cuda", "compute_dtype", runtime[1])
-        _CACHE[key] = (og.Model(c), cfg, w)
-    return _CACHE[key]
-
-
-def _engine(model, blocks=64, batch=4, tokens=512):
-    model.config.overlay(json.dumps({"engine": {"dynamic_batching": {"block_size": BLOCK, "num_blocks": blocks, "max_batch_size": batch,
-                                                                     "max_scheduled_tokens": tokens}}}))
-    return og.Engine(model)
-
-
-def _tokens(cfg, n, seed=0):
-    return np.random.RandomState(seed).randint(0, cfg["vocab"], n)
-
-
-def _feed(engine, model, toks, cuts):
-    """Logits of every token of one sequence fed in portions of the given sizes (the last size repeats)."""
-    r, at, out, i = og.Request(og.GeneratorParams(model)), 0, [], 0
-    while at < len(toks):
-        n = min(cuts[min(i, len(cuts) - 1)], len(toks) - at)
-        out.append(engine.run_given([(r, toks[at:at + n], list(range(n)))])[0])
-        at, i = at + n, i + 1
-    engine.remove_request(r)
-    return torch.cat(out).float().cpu()
-
-
 # ------------------------------------------------------------------------------------------------ configuration
 def test_config_is_read_into_layer_specs():
     a = A.from_stack_config(MIXED)
@@ -128,8 +71,8 @@ def test_builder_exports_a_model_directory(tmp_path):
     main(["-m", d, "-o", str(tmp_path / "out"), "-p", "bf16", "-e", "cpu", "--extra_options", "max_batch_size=3"])
     m = og.Model(str(tmp_path / "out"))
     assert m.type == "luzatar" and m.device_type == "cpu" and m.config.engine["dynamic_batching"]["max_batch_size"] == 3
-    toks = _tokens(ODD, 9)
-    _close(_feed(_engine(m), m, toks, [9]), stack_forward(ODD, weights(ODD, 3), toks)[0], 2e-4)
+    toks = random_tokens(ODD, 9)
+    close(feed(open_engine(m), m, toks, [9]), stack_forward(ODD, weights(ODD, 3), toks)[0], 2e-4)
     main(["-m", d, "-o", str(tmp_path / "syn"), "-p", "fp32", "-e", "cpu", "--extra_options", "synthetic_weights=1", "seed=5"])
     og.Model(str(tmp_path / "syn"))
 
@@ -150,12 +93,12 @@ def test_rotary_tables(rot):
 def test_stream_norm_and_embedding(runtime, H):
     g = torch.Generator().manual_seed(H)
     x, w, b = torch.randn(7, H, generator=g) * 3 + 2, torch.randn(H, generator=g), torch.randn(H, generator=g)
-    dev, dt = runtime[0], _dtype(runtime)
+    dev, dt = runtime[0], dtype_of(runtime)
     rows = torch.tensor([6, 0, 3], dtype=torch.int32)
     want = layer_norm(x.double(), w.double(), b.double(), 0.5)
-    _close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, b.to(dev), True, dt), want, _tol(runtime) / 4)
-    _close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, b.to(dev), True, dt, rows.to(dev)), want[rows.long()], _tol(runtime) / 4)
-    _close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, None, False, dt), rms_norm(x.double(), w.double(), 0.5), _tol(runtime) / 4)
+    close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, b.to(dev), True, dt), want, tol_of(runtime) / 4)
+    close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, b.to(dev), True, dt, rows.to(dev)), want[rows.long()], tol_of(runtime) / 4)
+    close(ops.norm_stream(x.to(dev), w.to(dev), 0.5, None, False, dt), rms_norm(x.double(), w.double(), 0.5), tol_of(runtime) / 4)
     table = torch.randn(11, H, generator=g).to(dt)
     ids = torch.tensor([3, 10, 0, 3], dtype=torch.int32)
     got = ops.embedding_stream(ids.to(dev), table.to(dev))
@@ -165,20 +108,20 @@ def test_stream_norm_and_embedding(runtime, H):
 @pytest.mark.parametrize("T,inter,width", [(3, 64, 40), (5, 128, 128), (70, 21, 45), (300, 192, 128)])
 def test_relu_gated_feed_forward_into_a_column_range(runtime, T, inter, width):
     g = torch.Generator().manual_seed(T)
-    dt, dev = _dtype(runtime), runtime[0]
+    dt, dev = dtype_of(runtime), runtime[0]
     x, w = torch.randn(T, width, generator=g).to(dt), (torch.randn(2 * inter, width, generator=g) / width ** 0.5).to(dt)
     il = runtime == ("cuda", "bfloat16") and inter % 64 == 0
     wide = torch.full((T, inter + 24), 7.0, dtype=dt, device=dev)
     ops.gate_up_act(x.to(dev), (ops.interleave_gate_up(w) if il else w).to(dev), None, "relu", out=wide[:, 8:8 + inter], interleaved=il)
     want = torch.relu(x.double() @ w[:inter].double().T) * (x.double() @ w[inter:].double().T)
-    _close(wide[:, 8:8 + inter], want, _tol(runtime))
+    close(wide[:, 8:8 + inter], want, tol_of(runtime))
     assert (wide[:, :8] == 7).all() and (wide[:, 8 + inter:] == 7).all()
 
 
 @pytest.mark.parametrize("T,K,N", [(1, 40, 72), (6, 45, 37), (64, 256, 512), (500, 128, 200)])
 def test_projection_adds_to_the_fp32_stream(runtime, T, K, N):
     g = torch.Generator().manual_seed(K)
-    dt, dev = _dtype(runtime), runtime[0]
+    dt, dev = dtype_of(runtime), runtime[0]
     x, w, h = torch.randn(T, K, generator=g).to(dt), torch.randn(N, K, generator=g).to(dt), torch.randn(T, N, generator=g) * 1000
     s = h.to(dev).clone()
     out = ops.linear(x.to(dev), w.to(dev), residual=s, out=s, out_fp32=True)
@@ -191,42 +134,19 @@ def test_projection_adds_to_the_fp32_stream(runtime, T, K, N):
 @pytest.mark.parametrize("T", [1, 20, 130])
 def test_per_head_projection(runtime, heads, a_cols, K, N, T):
     g = torch.Generator().manual_seed(N)
-    dt, dev = _dtype(runtime), runtime[0]
+    dt, dev = dtype_of(runtime), runtime[0]
     x, w = torch.randn(T, heads * a_cols + 8, generator=g).to(dt), torch.randn(heads * N, K, generator=g).to(dt)
     want = torch.cat([x[:, h * a_cols:h * a_cols + K].double() @ w[h * N:(h + 1) * N].double().T for h in range(heads)], 1)
-    _close(ops.head_project(x.to(dev), w.to(dev), heads, a_cols), want, _tol(runtime) / 4)
+    close(ops.head_project(x.to(dev), w.to(dev), heads, a_cols), want, tol_of(runtime) / 4)
     wide = torch.zeros(T, heads * N + 16, dtype=dt, device=dev)
     ops.head_project(x.to(dev), w.to(dev), heads, a_cols, out=wide[:, 8:8 + heads * N])
-    _close(wide[:, 8:8 + heads * N], want, _tol(runtime) / 4)
-
-
-def _paged(lens, blocks, seed=0):
-    """Block tables with shuffled blocks for requests of the given (past, new) lengths; slots and positions of the new tokens."""
-    order = np.random.RandomState(seed).permutation(blocks)
-    cols = max((p + n + BLOCK - 1) // BLOCK for p, n in lens)
-    table, at = np.full((len(lens), cols), -1, dtype=np.int32), 0
-    pos, slots = [], []
-    for b, (p, n) in enumerate(lens):
-        k = (p + n + BLOCK - 1) // BLOCK
-        table[b, :k] = order[at:at + k]
-        at += k
-        pos += list(range(p, p + n))
-    cu = np.cumsum([0] + [n for _, n in lens])
-    for b, (p, n) in enumerate(lens):
-        slots += [int(table[b, q // BLOCK]) * BLOCK + q % BLOCK for q in range(p, p + n)]
-    t = lambda x: torch.tensor(np.asarray(x), dtype=torch.int32)
-    return dict(table=t(table), pos=t(pos), slots=t(slots), cu=t(cu), past=t([p for p, _ in lens]))
-
-
-def _rows_of(pg, b, n):
-    q = np.arange(n)
-    return torch.tensor(pg["table"][b].numpy()[q // BLOCK] * BLOCK + q % BLOCK).long()
+    close(wide[:, 8:8 + heads * N], want, tol_of(runtime) / 4)
 
 
 @pytest.mark.parametrize("C,L", [(24, 4), (13, 3), (40, 1), (80, 6)])
 def test_convolution_continues_over_portions_and_pages(runtime, C, L):
     g = torch.Generator().manual_seed(C)
-    dt, dev = _dtype(runtime), runtime[0]
+    dt, dev = dtype_of(runtime), runtime[0]
     seqs = [torch.randn(n, C, generator=g).to(dt) for n in (37, 5, 18)]
     taps = torch.randn(C, L, generator=g).to(dt)
     cache = torch.zeros(12 * BLOCK, C + 3, dtype=dt, device=dev)[:, :C] if C % 8 else torch.zeros(12 * BLOCK, C + 8, dtype=dt, device=dev)[:, :C]
@@ -234,8 +154,8 @@ def test_convolution_continues_over_portions_and_pages(runtime, C, L):
     got, done = [[] for _ in seqs], [0, 0, 0]
     for cut in ((15, 1, 16), (2, 1, 2), (20, 3, 0)):
         lens = [(d, n) for d, n in zip(done, cut)]
-        pg = _paged([(d, len(s) - d) for d, s in zip(done, seqs)], 12)       # the same tables in every portion (total length fixed)
-        full = _paged([(0, len(s)) for s in seqs], 12)
+        pg = paged([(d, len(s) - d) for d, s in zip(done, seqs)], 12)       # the same tables in every portion (total length fixed)
+        full = paged([(0, len(s)) for s in seqs], 12)
         idx = [i for b, (d, n) in enumerate(lens) for i in range(int(full["cu"][b]) + d, int(full["cu"][b]) + d + n)]
         x = torch.cat([s[d:d + n] for s, (d, n) in zip(seqs, lens)])
         cu = torch.tensor(np.cumsum([0] + list(cut)), dtype=torch.int32)
@@ -246,7 +166,7 @@ def test_convolution_continues_over_portions_and_pages(runtime, C, L):
             done[b] += n
         del pg
     for s, y in zip(seqs, got):
-        _close(torch.cat(y), causal_conv_silu(s.double(), taps.double()), _tol(runtime))
+        close(torch.cat(y), causal_conv_silu(s.double(), taps.double()), tol_of(runtime))
 
 
 @pytest.mark.gpu
@@ -283,7 +203,7 @@ def test_delta_recurrence_kernels(dt, Hk, Hv, dk, dv):
                 done[b] += n
         for (c, p), y in zip(seqs, got):
             y = torch.cat(y)
-            _close(y, oracle(c[:len(y)], p[:len(y)]), 4e-2 if dt == torch.bfloat16 else 2e-4)
+            close(y, oracle(c[:len(y)], p[:len(y)]), 4e-2 if dt == torch.bfloat16 else 2e-4)
     assert (state[:, Hv * dk * dv:] == 99).all() and (state[1] == 99).all() and (state[2] == 99).all()
 
 
@@ -325,9 +245,9 @@ def _latent_case(shape, lens, window, seed, dt, needles=()):
 
 def _run_latent(case, shape, lens, window, runtime, splits=None, long_tokens=None):
     H, d, r, dv, R, rd = shape
-    dev, dt = runtime[0], _dtype(runtime)
+    dev, dt = runtime[0], dtype_of(runtime)
     sh = ops.latent_shape(H, d, r, dv, R, rd)
-    pg = _paged(lens, sum((p + n + BLOCK - 1) // BLOCK for p, n in lens) + 2, seed=5)
+    pg = paged(lens, sum((p + n + BLOCK - 1) // BLOCK for p, n in lens) + 2, seed=5)
     ld = (R + r + 7) // 8 * 8 + 8
     cache = torch.full(((int(pg["table"].max()) + 3) * BLOCK, ld), 3.0, dtype=dt, device=dev)
     cos = sin = None
@@ -338,7 +258,7 @@ def _run_latent(case, shape, lens, window, runtime, splits=None, long_tokens=Non
     for b, (p, n) in enumerate(lens):            # what earlier steps left in the cache
         if p:
             ops.latent_prep(wide(case["seqs"][b][:p].clone()), sh, case["nw"].to(dev), 1e-5, torch.arange(p, dtype=torch.int32, device=dev), cos, sin,
-                            _rows_of(pg, b, p).to(torch.int32).to(dev), cache)
+                            rows_of(pg, b, p).to(torch.int32).to(dev), cache)
     proj = wide(torch.cat([s[p:] for s, (p, _) in zip(case["seqs"], lens)]).clone())
     t = {k: v.to(dev) for k, v in pg.items()}
     ops.latent_prep(proj, sh, case["nw"].to(dev), 1e-5, t["pos"], cos, sin, t["slots"], cache)
@@ -365,9 +285,9 @@ def _run_latent(case, shape, lens, window, runtime, splits=None, long_tokens=Non
 @pytest.mark.parametrize("window", [0, 1, 23])
 def test_latent_attention_over_pages(runtime, shape, window):
     for lens in ([(0, 1), (70, 1), (15, 1), (16, 1), (200, 1)], [(0, 5), (31, 2), (40, 33), (17, 1)]):
-        case = _latent_case(shape, lens, window, 3, _dtype(runtime))
+        case = _latent_case(shape, lens, window, 3, dtype_of(runtime))
         for splits in (None, 1, 3):
-            _close(_run_latent(case, shape, lens, window, runtime, splits), case["want"], _tol(runtime))
+            close(_run_latent(case, shape, lens, window, runtime, splits), case["want"], tol_of(runtime))
 
 
 @pytest.mark.gpu
@@ -378,7 +298,7 @@ def test_latent_attention_of_long_prompts_on_expanded_keys(shape, window):
     rt = ("cuda", "bfloat16")
     for lens in ([(0, 300)], [(5, 1), (131, 140), (0, 3), (400, 129), (17, 64)]):
         case = _latent_case(shape, lens, window, 4, torch.bfloat16)
-        _close(_run_latent(case, shape, lens, window, rt, long_tokens=16), case["want"], _tol(rt))
+        close(_run_latent(case, shape, lens, window, rt, long_tokens=16), case["want"], tol_of(rt))
 
 
 @pytest.mark.parametrize("window", [17, 32, 50])
@@ -396,37 +316,37 @@ def test_window_edges_with_keys_that_stand_out(runtime, window, form):
                 continue
             n = {"decode": 1, "portion": 7, "long": min(q + 1, 70)}[form]
             lens = [(max(0, q + 1 - n), min(n, q + 1)), (3, 2)]
-            case = _latent_case(shape, lens, window, 11 + q + dist, _dtype(runtime), needles=[(0, key, q)])
+            case = _latent_case(shape, lens, window, 11 + q + dist, dtype_of(runtime), needles=[(0, key, q)])
             got = _run_latent(case, shape, lens, window, runtime, long_tokens=16 if form == "long" else None)
-            _close(got, case["want"], _tol(runtime))
+            close(got, case["want"], tol_of(runtime))
 
 
 # ------------------------------------------------------------------------------------------------ whole models
 @pytest.mark.parametrize("name", list(STACKS))
 def test_logits_of_a_whole_prompt(tmp_path_factory, runtime, name):
-    m, cfg, w = _model(tmp_path_factory, name, runtime)
+    m, cfg, w = open_model(tmp_path_factory, name, runtime, STACKS[name])
     for n in (1, 2, 47, 150):
-        toks = _tokens(cfg, n, n)
-        _close(_feed(_engine(m), m, toks, [n]), stack_forward(cfg, w, toks)[0], _tol(runtime))
+        toks = random_tokens(cfg, n, n)
+        close(feed(open_engine(m), m, toks, [n]), stack_forward(cfg, w, toks)[0], tol_of(runtime))
 
 
 @pytest.mark.parametrize("name", list(STACKS))
 @pytest.mark.parametrize("cuts", [[1], [2], [3, 2, 2, 17, 1, 1, 40], [100, 1], [64, 63, 2, 1], [15, 1, 1, 1, 16, 33]], ids=str)
 def test_portions_and_single_tokens(tmp_path_factory, runtime, name, cuts):
     """The same logits whatever the cut: token by token, pairs, ends and starts of pages and windows, long portions then decoding."""
-    m, cfg, w = _model(tmp_path_factory, name, runtime)
-    toks = _tokens(cfg, 130, 7)
-    _close(_feed(_engine(m), m, toks, cuts), stack_forward(cfg, w, toks)[0], _tol(runtime))
+    m, cfg, w = open_model(tmp_path_factory, name, runtime, STACKS[name])
+    toks = random_tokens(cfg, 130, 7)
+    close(feed(open_engine(m), m, toks, cuts), stack_forward(cfg, w, toks)[0], tol_of(runtime))
 
 
 @pytest.mark.parametrize("name", list(STACKS))
 def test_mixed_batches_reuse_pages_and_slots(tmp_path_factory, runtime, name):
     """More requests than fit at once come and go through a pool that is just large enough, portions beside single tokens, requests left
     out of some steps; every request gets the logits it gets alone."""
-    m, cfg, w = _model(tmp_path_factory, name, runtime)
-    eng = _engine(m, blocks=26, batch=4, tokens=300)
+    m, cfg, w = open_model(tmp_path_factory, name, runtime, STACKS[name])
+    eng = open_engine(m, blocks=26, batch=4, tokens=300)
     rng = np.random.RandomState(5)
-    waiting = [(i, _tokens(cfg, n, 20 + i)) for i, n in enumerate((90, 33, 120, 5, 64, 1, 77, 100, 16, 50))]
+    waiting = [(i, random_tokens(cfg, n, 20 + i)) for i, n in enumerate((90, 33, 120, 5, 64, 1, 77, 100, 16, 50))]
     live, got, seen = [], {i: [] for i, _ in waiting}, dict(waiting)
     used_blocks = set()
     while waiting or live:
@@ -454,51 +374,43 @@ def test_mixed_batches_reuse_pages_and_slots(tmp_path_factory, runtime, name):
     for i, parts in got.items():
         want = stack_forward(cfg, w, seen[i])[0]
         for at, n, lg in parts:
-            _close(lg, want[at:at + n] if i % 2 else want[at + n - 1:at + n], 1.5 * _tol(runtime))
+            close(lg, want[at:at + n] if i % 2 else want[at + n - 1:at + n], 1.5 * tol_of(runtime))
 
 
 def test_a_request_does_not_see_the_batch_around_it(tmp_path_factory, runtime):
-    m, cfg, _ = _model(tmp_path_factory, "wide", runtime)
-    a, b, c = (_tokens(cfg, n, s) for n, s in ((90, 1), (75, 2), (3, 3)))
-    alone = _feed(_engine(m), m, a, [80, 1])
-    eng = _engine(m)
+    m, cfg, _ = open_model(tmp_path_factory, "wide", runtime, STACKS["wide"])
+    a, b, c = (random_tokens(cfg, n, s) for n, s in ((90, 1), (75, 2), (3, 3)))
+    alone = feed(open_engine(m), m, a, [80, 1])
+    eng = open_engine(m)
     ra, rb, rc = (og.Request(og.GeneratorParams(m)) for _ in range(3))
     rows = [eng.run_given([(rb, b[:70], []), (ra, a[:80], list(range(80))), (rc, c, [0])])[1]]
     for j in range(10):
         rows.append(eng.run_given([(ra, a[80 + j:81 + j], [0])] + ([(rb, b[70 + j:71 + j], [0])] if j < 5 else []))[0])
-    _close(torch.cat(rows), alone.double(), _tol(runtime) / 4)
+    close(torch.cat(rows), alone.double(), tol_of(runtime) / 4)
 
 
 def test_long_decoding(tmp_path_factory, runtime):
     """Hundreds of single-token steps: windows slide over decoded tokens, states are carried on, pages fill up."""
-    m, cfg, w = _model(tmp_path_factory, "mixed", runtime)
-    toks = _tokens(cfg, 260, 9)
-    _close(_feed(_engine(m), m, toks, [20, 1]), stack_forward(cfg, w, toks)[0], _tol(runtime))
+    m, cfg, w = open_model(tmp_path_factory, "mixed", runtime, STACKS["mixed"])
+    toks = random_tokens(cfg, 260, 9)
+    close(feed(open_engine(m), m, toks, [20, 1]), stack_forward(cfg, w, toks)[0], tol_of(runtime))
 
 
 def test_run_given_rejects_what_does_not_fit(tmp_path_factory):
-    m, cfg, _ = _model(tmp_path_factory, "odd", ("cpu", "float32"))
-    eng = _engine(m, blocks=4, batch=2, tokens=64)
+    m, cfg, _ = open_model(tmp_path_factory, "odd", ("cpu", "float32"), STACKS["odd"])
+    eng = open_engine(m, blocks=4, batch=2, tokens=64)
     r = og.Request(og.GeneratorParams(m))
     with pytest.raises(RuntimeError):
-        eng.run_given([(r, _tokens(cfg, 3), [3])])
+        eng.run_given([(r, random_tokens(cfg, 3), [3])])
     with pytest.raises(RuntimeError):
-        eng.run_given([(og.Request(og.GeneratorParams(m)), _tokens(cfg, 65), [])])
+        eng.run_given([(og.Request(og.GeneratorParams(m)), random_tokens(cfg, 65), [])])
 
 
 # ------------------------------------------------------------------------------------------------ generation
-def _greedy_ok(cfg, w, prompt, generated, tol):
-    """Every generated token is the oracle's argmax, or within rounding of it."""
-    lg = stack_forward(cfg, w, np.concatenate([prompt, generated]))[0]
-    for i, t in enumerate(generated):
-        row = lg[len(prompt) - 1 + i]
-        assert float(row.max() - row[int(t)]) <= tol * float(lg.std()), f"token {i}"
-
-
 def test_greedy_generation_through_generator_and_engine(tmp_path_factory, runtime):
-    m, cfg, w = _model(tmp_path_factory, "wide", runtime)
+    m, cfg, w = open_model(tmp_path_factory, "wide", runtime, STACKS["wide"])
     tol = 0.2 if runtime[1] == "bfloat16" else 1e-3
-    prompts = [_tokens(cfg, n, 40 + n) for n in (70, 5, 33, 1, 18)]
+    prompts = [random_tokens(cfg, n, 40 + n) for n in (70, 5, 33, 1, 18)]
     p = og.GeneratorParams(m)
     p.set_search_options(max_length=100, do_sample=False)
     gen = og.Generator(m, p)
@@ -507,9 +419,9 @@ def test_greedy_generation_through_generator_and_engine(tmp_path_factory, runtim
         gen.generate_next_token()
     solo = np.asarray(gen.get_sequence(0))[70:]
     assert len(solo) == 30
-    _greedy_ok(cfg, w, prompts[0], solo, tol)
+    greedy_ok(cfg, w, prompts[0], solo, tol)
     # the scheduler: more requests than the batch holds, prompts cut by a small token budget, blocks that run short
-    eng = _engine(m, blocks=30, batch=3, tokens=40)
+    eng = open_engine(m, blocks=30, batch=3, tokens=40)
     reqs = []
     for t in prompts:
         gp = og.GeneratorParams(m)
@@ -529,13 +441,13 @@ def test_greedy_generation_through_generator_and_engine(tmp_path_factory, runtim
             eng.remove_request(r)
     for r, t in zip(reqs, prompts):
         assert len(r.kept) == len(t) + 25
-        _greedy_ok(cfg, w, t, r.kept[len(t):], tol)
+        greedy_ok(cfg, w, t, r.kept[len(t):], tol)
 
 
 def test_batched_generator_rewind_and_beams(tmp_path_factory, runtime):
-    m, cfg, w = _model(tmp_path_factory, "mixed", runtime)
+    m, cfg, w = open_model(tmp_path_factory, "mixed", runtime, STACKS["mixed"])
     tol = 0.2 if runtime[1] == "bfloat16" else 1e-3
-    prompt = np.stack([_tokens(cfg, 12, 3), _tokens(cfg, 12, 4)]).astype(np.int32)
+    prompt = np.stack([random_tokens(cfg, 12, 3), random_tokens(cfg, 12, 4)]).astype(np.int32)
     p = og.GeneratorParams(m)
     p.set_search_options(max_length=30, batch_size=2, do_sample=False)
     gen = og.Generator(m, p)
@@ -543,7 +455,7 @@ def test_batched_generator_rewind_and_beams(tmp_path_factory, runtime):
     while not gen.is_done():
         gen.generate_next_token()
     for r in range(2):
-        _greedy_ok(cfg, w, prompt[r], np.asarray(gen.get_sequence(r))[12:], tol)
+        greedy_ok(cfg, w, prompt[r], np.asarray(gen.get_sequence(r))[12:], tol)
     p = og.GeneratorParams(m)
     p.set_search_options(max_length=40, do_sample=False)
     gen = og.Generator(m, p)
@@ -554,7 +466,7 @@ def test_batched_generator_rewind_and_beams(tmp_path_factory, runtime):
     gen.rewind_to(15)
     for _ in range(7):
         gen.generate_next_token()
-    _greedy_ok(cfg, w, prompt[0], np.asarray(gen.get_sequence(0))[12:], tol)
+    greedy_ok(cfg, w, prompt[0], np.asarray(gen.get_sequence(0))[12:], tol)
     assert (np.asarray(gen.get_sequence(0))[:15] == first[:15]).all()
     p = og.GeneratorParams(m)
     p.set_search_options(max_length=24, num_beams=3, do_sample=False)
@@ -566,19 +478,8 @@ def test_batched_generator_rewind_and_beams(tmp_path_factory, runtime):
     lp = lambda s: float(sum(torch.log_softmax(stack_forward(cfg, w, s)[0], -1)[i, int(s[i + 1])] for i in range(11, len(s) - 1)))
     # beams follow their own states and pages: a plain beam search over the restatement finds a hypothesis of the same score (16-bit
     # rounding may pick another one where candidates are close)
-    best = lp(_beam_search(cfg, w, prompt[0], 24, 3))
+    best = lp(beam_search(cfg, w, prompt[0], 24, 3))
     assert abs(lp(seq) - best) < (4.0 if runtime[1] == "bfloat16" else 2e-2)
-
-
-def _beam_search(cfg, w, prompt, n, beams):
-    hyps = [(0.0, list(map(int, prompt)))]
-    while len(hyps[0][1]) < n:
-        cand = []
-        for score, s in hyps:
-            row = torch.log_softmax(stack_forward(cfg, w, s)[0][-1], -1)
-            cand += [(score + float(v), s + [int(t)]) for v, t in zip(*torch.topk(row, beams))]
-        hyps = sorted(cand, key=lambda c: -c[0])[:beams]
-    return np.asarray(hyps[0][1])
 
 
 # ------------------------------------------------------------------------------------------------ cache sizes, trace replay
@@ -597,8 +498,8 @@ def test_trace_replay_writes_the_wanted_rows(tmp_path):
     cfg, w = ODD, weights(ODD, 8)
     c = og.Config(write(cfg, w, tmp_path / "m"), provider="cpu")
     m = og.Model(c)
-    eng = _engine(m, blocks=8, batch=4, tokens=128)
-    a, b = _tokens(cfg, 30, 1).tolist(), _tokens(cfg, 12, 2).tolist()
+    eng = open_engine(m, blocks=8, batch=4, tokens=128)
+    a, b = random_tokens(cfg, 30, 1).tolist(), random_tokens(cfg, 12, 2).tolist()
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": a[:20], "want": [0, 19]}], "end": []},
              {"step": 1, "entries": [{"id": "y", "tokens": b[:11], "want": []}, {"id": "x", "tokens": a[20:21], "want": []}], "end": []},
              {"step": 2, "entries": [{"id": "x", "tokens": a[21:], "want": [8]}, {"id": "y", "tokens": b[11:], "want": [0]}], "end": ["x", "y"]}]
@@ -606,5 +507,5 @@ def test_trace_replay_writes_the_wanted_rows(tmp_path):
     trace_replay.replay(m, eng, [json.dumps(s) + "\n" for s in steps], str(tmp_path), said.append)
     assert said == ["done 0", "done 1", "done 2"] and not (tmp_path / "1.f32").exists() and eng.core.free_blocks == 8
     wa, wb = stack_forward(cfg, w, a)[0], stack_forward(cfg, w, b)[0]
-    _close(torch.from_numpy(np.fromfile(tmp_path / "0.f32", dtype="<f4")).view(2, -1), wa[[0, 19]], 2e-4)
-    _close(torch.from_numpy(np.fromfile(tmp_path / "2.f32", dtype="<f4")).view(2, -1), torch.stack([wa[29], wb[11]]), 2e-4)
+    close(torch.from_numpy(np.fromfile(tmp_path / "0.f32", dtype="<f4")).view(2, -1), wa[[0, 19]], 2e-4)
+    close(torch.from_numpy(np.fromfile(tmp_path / "2.f32", dtype="<f4")).view(2, -1), torch.stack([wa[29], wb[11]]), 2e-4)
