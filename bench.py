@@ -410,7 +410,7 @@ def design_arm(args):
 
         def stop(self):
             return self.s.stop()
-    res = stack_bench.run(Sampler(), args.steps, max(3, args.warmup), args.design_sizes.split(",") if args.design_sizes else None)
+    res = stack_bench.run(Sampler(), args.steps, max(3, args.warmup), args.design_sizes.split(",") if args.design_sizes else None, args.design)
     print(json.dumps({"metric": "prefill_and_decode_tokens_per_s", "design": args.design, "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup),
                       "dtype": "bf16", "data": "synthetic (random token ids, random weights drawn on the device)",
                       "config": {"l2": "weights and caches larger than L2, no flush"}, "sizes": res}))
@@ -440,7 +440,7 @@ def main():
     ap.add_argument("--precision", default="bf16", choices=["bf16", "int4"],
                     help="weights of the checkpoint: bf16 (headline) or 4-bit (int4 block-32 linears; gpt-oss experts as packed MXFP4, the form "
                          "the reference publishes its gpt-oss numbers for); activations and the KV cache stay bf16")
-    ap.add_argument("--design", default="", choices=["", "luzatar"],
+    ap.add_argument("--design", default="", choices=["", "luzatar", "zevopel"],
                     help="measure this declared-stack design beside the closest other model at equal size instead of the headline workload")
     ap.add_argument("--design_sizes", default="", help="comma-separated sizes of --design (default: all)")
     args = ap.parse_args()

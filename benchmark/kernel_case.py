@@ -5,6 +5,8 @@
 cases: gemm_qkv gemm_o gemm_gate_up gemm_down gemm_lm_head gemm_prefill gemm_qkv_fused gemm_gate_up_fused w4_qkv w4_down attention_decode
        attention_prefill norm rope sample argmax all; moe_fp4_gate_up moe_fp4_down moe_fp4b_gate_up moe_fp4b_down moe_bf16_gate_up moe_bf16_down
        gated_delta gated_delta_prefill mamba2_scan; latent_decode latent_absorb latent_value latent_prep latent_prefill latent_expand norm_stream
+       chunk_decode chunk_prefill chunk_decode_192 chunk_prefill_192 qkv_prep add_normed add_normed_experts gemm_gate_up_gelu expert_route (Zevopel
+       layers: attention with sinks and head gates, keys of 128 or 192 and values of 128 columns; norms of sub-layer outputs; not part of `all`)
        gemm_join (Luzatar layers at Llama-sized widths: 16 heads of 128 + 64 / 128 over a latent of 512; not part of `all`)
        (moe_*: gpt-oss-20b experts, packed MXFP4 in the fp16 form, in the bf16 form (fp4b) or bf16 weights; not part of `all`)
 
@@ -109,7 +111,7 @@ def build_case(name, T, L, tp=1):
         kc, vc = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D)
         return (lambda i: ops.qkv_rope_append(x, ws[i % L], None, pos, slots, cos, sin, kc, vc, HQ, HKV, D, D, norm_eps=1e-5)), \
             N * H * 2 + T * (H + N) * 2, 2.0 * T * N * H
-    if name != "gemm_join" and name.startswith(("gemm_", "w4_")):
+    if name not in ("gemm_join", "gemm_gate_up_gelu") and name.startswith(("gemm_", "w4_")):
         shapes = {"gemm_qkv": ((HQ + 2 * HKV) * D, H), "gemm_o": (H, HQ * D), "gemm_gate_up": (2 * I // tp, H), "gemm_down": (H, I // tp),
                   "gemm_lm_head": (V // tp, H), "gemm_prefill": (2 * I // tp, H), "w4_qkv": (9216 // tp, 3072), "w4_down": (3072, 8192 // tp)}
         N, K = shapes[name]
@@ -160,10 +162,11 @@ def build_case(name, T, L, tp=1):
         if gate_up:
             return (lambda i: ops.moe_gemm(xs, ws[i % L], plan, bias, act_kind=2, alpha=1.702, limit=7.0)), wbytes + T * k * (K + N // 2) * 2, 2.0 * T * k * N * K
         return (lambda i: ops.moe_gemm(xs, ws[i % L], plan, bias)), wbytes + T * k * (K + N) * 2, 2.0 * T * k * N * K
-    if name in ("attention_decode", "attention_prefill"):
+    if name in ("attention_decode", "attention_prefill") or name.startswith("chunk_"):
         bs = 16
         rng = np.random.RandomState(2)
-        decode = name == "attention_decode"
+        decode = "decode" in name
+        chunked, dk = name.startswith("chunk_"), 192 if name.endswith("192") else D
         B = T if decode else max(1, T // 1024)
         q_lens = [1] * B if decode else [T // B] * B
         past = (rng.randint(128, 2049, size=B) + 64).tolist() if decode else [0] * B
@@ -179,6 +182,8 @@ def build_case(name, T, L, tp=1):
         else:
             kc = [_bf(nblk * bs, HKV, D, std=1.0) for _ in range(Lk)]
             vc = [_bf(nblk * bs, HKV, D, std=1.0) for _ in range(Lk)]
+        if chunked:
+            kc = [_bf(nblk * bs, HKV, dk, std=1.0) for _ in range(Lk)]
         table = torch.zeros(B, cols, dtype=torch.int32)
         used = 0
         for b in range(B):
@@ -194,6 +199,13 @@ def build_case(name, T, L, tp=1):
         nbytes = kv_tokens * HKV * ((D + 16) if KV_BITS == 8 else D * 2) * 2 + Tq * HQ * D * 2 * 2
         flops = sum(4.0 * HQ * D * (q * p + q * (q + 1) / 2) for p, q in zip(past, q_lens))
         order = torch.argsort(-pl.long(), stable=True).to(torch.int32) if ATTN_ORDER else None   # longest request first
+        if chunked:
+            proj, sinks = _bf(Tq, HQ * dk + HQ, std=1.0), torch.randn(HQ, device="cuda")
+            nbytes = kv_tokens * HKV * (dk + D) * 2 + Tq * HQ * (dk + D) * 2
+            return (lambda i: ops.paged_attention(proj, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ, HKV, dk, 1 / math.sqrt(dk), sinks=sinks,
+                                                  max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)), splits=ATTN_SPLITS,
+                                                  order=order, min_q_len=min(q_lens), vdim=D, chunk=8192, gate=proj[:, HQ * dk:])), nbytes, \
+                flops * (dk + D) / (2 * D)
         return (lambda i: ops.paged_attention(qkv, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ, HKV, D, 1 / math.sqrt(D),
                                               max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)),
                                               splits=ATTN_SPLITS, order=order)), nbytes, flops
@@ -246,6 +258,26 @@ def build_case(name, T, L, tp=1):
     if name == "norm_stream":
         xs, w, b = [torch.randn(T, H, device="cuda") for _ in range(8)], torch.randn(H, device="cuda"), torch.randn(H, device="cuda")
         return (lambda i: ops.norm_stream(xs[i % 8], w, 1e-5, b, True)), T * H * 6, 0.0
+    if name == "gemm_gate_up_gelu":
+        x, ws = _bf(T, H, std=1.0), [ops.interleave_gate_up(_bf(2 * I, H)) for _ in range(L)]
+        return (lambda i: ops.gate_up_act(x, ws[i % L], act="gelu_tanh", interleaved=True)), 2 * I * H * 2 + T * (H + I) * 2, 4.0 * T * I * H
+    if name == "qkv_prep":
+        projs = [_bf(T, (HQ + 2 * HKV) * D + HQ, std=1.0) for _ in range(4)]
+        pos, slots = torch.arange(T, dtype=torch.int32, device="cuda") % 4096, torch.arange(T, dtype=torch.int32, device="cuda")
+        cos, sin, w = torch.randn(4096, D // 2, device="cuda"), torch.randn(4096, D // 2, device="cuda"), torch.ones(D, device="cuda")
+        kc, vc = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D)
+        return (lambda i: ops.qkv_prep(projs[i % 4], HQ, HKV, D, D, D, w, w, 1e-6, pos, cos, sin, slots, kc, vc)), T * (HQ + 2 * HKV) * D * 2 * 2, 0.0
+    if name in ("add_normed", "add_normed_experts"):
+        hs, w = [torch.randn(T, H, device="cuda") for _ in range(4)], torch.randn(H, device="cuda")
+        if name == "add_normed":
+            y, rows = _bf(T, H, std=1.0), T
+        else:
+            plan = ops.moe_route(torch.randn(T, 32, device="cuda"), 4, 1)
+            y, rows = ops.PendingCombine(_bf(T * 4, H, std=1.0), plan), 4 * T
+        return (lambda i: ops.add_normed(hs[i % 4], y, w, 1e-6)), rows * H * 2 + T * H * 10, 0.0
+    if name == "expert_route":
+        logits = torch.randn(T, 32, device="cuda")
+        return (lambda i: ops.moe_route(logits, 4, 1)), T * 32 * 4 + T * 4 * 16, 0.0
     if name == "gemm_join":
         K = 2048 + I
         x, ws, h = _bf(T, K, std=1.0), [_bf(H, K) for _ in range(L)], torch.zeros(T, H, device="cuda")
@@ -345,7 +377,8 @@ def main():
     hbm, tflops, src = _peaks()
     out = {}
     for name in (ALL if a.case == "all" else [a.case]):
-        T = max(a.tokens, 2048) if name in ("gemm_prefill", "attention_prefill", "latent_prefill", "latent_expand", "gated_delta_prefill") else a.tokens
+        T = max(a.tokens, 2048) if name in ("gemm_prefill", "attention_prefill", "latent_prefill", "latent_expand", "gated_delta_prefill",
+                                         "chunk_prefill", "chunk_prefill_192") else a.tokens
         fn, nbytes, flops = build_case(name, T, a.layers, a.tp)
         iters = a.iters if name not in ("gemm_lm_head", "sample", "argmax") else min(a.iters, 4)
         us = _time_eager(fn, iters) if a.eager else _time_graph(fn, iters)

@@ -1,7 +1,9 @@
-"""Prefill and decode throughput of a declared stack (Luzatar) beside the closest other model of the framework at equal size: the
-gated-delta-net + full-attention hybrid (Qwen3.5 style) with the same width, feed-forward, layer count, delta layers and attention
-heads.  Random weights drawn on the device; CUDA events around whole decoder forwards (decode steps replay a CUDA graph); the weights
-and caches of a step are larger than L2.  Reached through `python bench.py --design luzatar`."""
+"""Prefill and decode throughput of a declared stack beside the closest other model of the framework at equal size.  Luzatar: the
+gated-delta-net + full-attention hybrid (Qwen3.5 style) with the same width, feed-forward, layer count, delta layers and attention heads.
+Zevopel: Qwen3-style dense layers (normed query and key heads), and gpt-oss-style layers with bf16 experts (sinks, clamped experts), each
+with the same width, heads and feed-forwards; the chunks are as long as the context, so both attend to the same keys.  Random weights drawn
+on the device; CUDA events around whole decoder forwards (decode steps replay a CUDA graph); the weights and caches of a step are larger
+than L2.  Reached through `python bench.py --design luzatar | zevopel`."""
 import json
 import os
 import shutil
@@ -14,6 +16,12 @@ SIZES = {
     # name: width, ff, layers (alternating delta / attention), attention heads, kv heads of the hybrid, delta key heads, delta value heads
     "2k": dict(width=2048, ff=6144, layers=16, heads=16, kv=4, dk=8, dv=16, vocab=65536),
     "4k": dict(width=4096, ff=12288, layers=8, heads=32, kv=8, dk=16, dv=32, vocab=65536),
+}
+ZEVOPEL_SIZES = {
+    # name: width, feed-forward (of one expert where there are experts), layers, heads, kv heads, head size
+    "2k dense": dict(width=2048, ff=6144, layers=16, heads=16, kv=4, dim=128, vocab=65536),
+    "4k dense": dict(width=4096, ff=12288, layers=8, heads=32, kv=8, dim=128, vocab=65536),
+    "2.9k experts": dict(width=2880, ff=2880, layers=8, heads=64, kv=8, dim=64, vocab=65536, experts=32, top=4),
 }
 PREFILL = [(1, 4096), (8, 1024)]
 DECODE = [(1, 2048), (16, 2048), (64, 2048), (256, 1024)]
@@ -42,6 +50,36 @@ def hybrid_dir(z, path):
     return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
 
 
+def zevopel_dir(z, path):
+    mlp = dict(kind="dense", ff=z["ff"])
+    if z.get("experts"):
+        mlp = dict(kind="moe", expert=dict(ff=z["ff"], limit=7.0), router=dict(experts=z["experts"], top=z["top"]))
+    layer = dict(type="attention", mlp=mlp, mixer=dict(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5,
+                                                       mask=dict(size=8192), rot=dict(base=5e5, dims=z["dim"])))
+    cfg = dict(architecture="Zevopel", layers=[layer] * z["layers"], norm=dict(eps=1e-6), vocab=z["vocab"], width=z["width"], residual_mult=0.3,
+               embedding=dict(scale=1.0))
+    os.makedirs(os.path.join(path, "src"), exist_ok=True)
+    with open(os.path.join(path, "src", "config.json"), "w") as f:
+        json.dump(cfg, f)
+    from onnxruntime_genai_b200.models.builder import create_model
+    return create_model(os.path.join(path, "src"), os.path.join(path, "model"), "bf16", "cuda", {"synthetic_weights": 1, "context_length": 8192})
+
+
+def closest_to_zevopel_dir(z, path):
+    from onnxruntime_genai_b200.models.arch import ArchConfig
+    from onnxruntime_genai_b200.models.builder import export_model
+    a = ArchConfig(model_type="qwen3", vocab_size=z["vocab"], hidden_size=z["width"], num_layers=z["layers"], num_heads=z["heads"], num_kv_heads=z["kv"],
+                   head_dim=z["dim"], intermediate_size=z["ff"], context_length=8192, qk_norm=True, rope_theta=5e5, bos_token_id=0, eos_token_id=1,
+                   pad_token_id=0)
+    if z.get("experts"):
+        a.model_type, a.qk_norm, a.attn_bias, a.o_bias, a.mlp_bias, a.attn_sinks = "gptoss", False, True, True, True, True
+        a.num_experts, a.experts_per_token = z["experts"], z["top"]
+    return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
+
+
+DESIGNS = {"luzatar": (SIZES, luzatar_dir, "hybrid", hybrid_dir), "zevopel": (ZEVOPEL_SIZES, zevopel_dir, "closest", closest_to_zevopel_dir)}
+
+
 def _step(model, lens):
     """(StepInputs, cache) of a step with the given (past, new) lengths over fresh zero caches."""
     from onnxruntime_genai_b200.models.decoder import PagedKVCache, StepInputs
@@ -49,7 +87,7 @@ def _step(model, lens):
     nb = [(p + n + BLOCK - 1) // BLOCK for p, n in lens]
     kv = PagedKVCache(dec.arch, sum(nb), BLOCK, "cuda", dec.dtype, kv_heads=dec.kv_heads_local, conv_channels=dec.conv_channels_local)
     kv.ensure_state_slots(len(lens))
-    for pool in (kv.full, kv.conv, kv.latent, kv.state):
+    for pool in (kv.full, kv.conv, kv.latent, kv.state, *(p for pools in kv.spec_kv.values() for p in pools)):
         if pool is not None and pool.numel():
             pool.normal_(0, 0.1)
     table = np.zeros((len(lens), max(nb)), dtype=np.int32)
@@ -110,13 +148,14 @@ def measure(model, steps, warmup):
     return out
 
 
-def run(sampler, steps=50, warmup=3, sizes=None):
+def run(sampler, steps=50, warmup=3, sizes=None, design="luzatar"):
     import onnxruntime_genai_b200 as og
+    table, make_design, other, make_other = DESIGNS[design]
     result = {}
-    for name in sizes or SIZES:
-        z = SIZES[name]
+    for name in sizes or table:
+        z = table[name]
         result[name] = {"shape": z}
-        for label, make in (("luzatar", luzatar_dir), ("hybrid", hybrid_dir)):
+        for label, make in ((design, make_design), (other, make_other)):
             d = tempfile.mkdtemp(prefix="ogb_stack_")
             try:
                 model = og.Model(make(z, d))
@@ -128,6 +167,7 @@ def run(sampler, steps=50, warmup=3, sizes=None):
             finally:
                 shutil.rmtree(d, ignore_errors=True)
             torch.cuda.empty_cache()
-        pairs = [k for k in result[name]["luzatar"] if isinstance(result[name]["luzatar"][k], dict) and "ms" in result[name]["luzatar"][k]]
-        result[name]["time ratio luzatar / hybrid"] = {k: round(result[name]["luzatar"][k]["ms"] / result[name]["hybrid"][k]["ms"], 3) for k in pairs}
+        mine, theirs = result[name][design], result[name][other]
+        pairs = [k for k in mine if isinstance(mine[k], dict) and "ms" in mine[k]]
+        result[name][f"time ratio {design} / {other}"] = {k: round(mine[k]["ms"] / theirs[k]["ms"], 3) for k in pairs}
     return result

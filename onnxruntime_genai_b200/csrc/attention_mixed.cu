@@ -1,6 +1,6 @@
 // Attention over a paged cache for layers whose heads have sizes of their own (declared stacks): queries and keys of dk columns, values of
 // dv columns, an optional gate per head, keys limited to a window or to the query's own run of positions.  Decode rows and short portions:
-// the warp-MMA kernel of attention_paged.cuh with rows filled up with zeros to 64, 128 or 256 columns (heads that are 64, 96 or 128 wide
+// the warp-MMA kernel of attention_paged.cuh with rows filled up with zeros to 64, 128, 192 (keys) or 256 columns (heads that are 64, 96 or 128 wide
 // throughout take its exact forms).  Long portions are served by attention_tc_mixed.cu, fp32 models and other sizes by attention_simt.cu.
 #include "attention_paged.cuh"
 
@@ -56,5 +56,6 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
   if (a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
   if (a->dk <= 64) return LaunchMixedKeys<64>(p, max_q_len, stream);
   if (a->dk <= 128) return LaunchMixedKeys<128>(p, max_q_len, stream);
+  if (a->dk <= 192) return LaunchMixedKeys<192>(p, max_q_len, stream);
   return LaunchMixedKeys<256>(p, max_q_len, stream);
 }

@@ -33,8 +33,8 @@ namespace ogb {
 constexpr int ATT_BM = 64;   // query rows per CTA (4 warps x 16)
 constexpr int ATT_BN = 64;   // keys per tile
 constexpr int ATT_THREADS = 128;
-// K/V tiles in flight per CTA (two where three of the widest rows do not fit in shared memory)
-template <int DK, int DV> constexpr int att_stages() { return DK + DV > 384 ? 2 : 3; }
+// K/V tiles in flight per CTA: three, or two where three would keep a second CTA (or, for the widest rows, the first) off the SM
+template <int DK, int DV> constexpr int att_stages() { return DK + DV > 256 ? 2 : 3; }
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct AttnParams {
