@@ -101,6 +101,12 @@ def rows_of(pg, b, n):
     return torch.tensor(pg["table"][b].numpy()[q // BLOCK] * BLOCK + q % BLOCK).long()
 
 
+def wide_rows(x, dev):
+    """x [T, n] on the device with rows of whole 16-byte pieces (the form in which projections reach the attention kernels)."""
+    out = torch.zeros(x.shape[0], (x.shape[1] + 7) // 8 * 8, dtype=x.dtype, device=dev)[:, :x.shape[1]]
+    return out.copy_(x)
+
+
 def greedy_ok(cfg, w, prompt, generated, tol):
     """Every generated token is the oracle's argmax, or within rounding of it."""
     lg = stack_forward(cfg, w, np.concatenate([prompt, generated]))[0]

@@ -14,7 +14,7 @@ from onnxruntime_genai_b200 import ops
 from onnxruntime_genai_b200.models import arch as A
 from onnxruntime_genai_b200.models import moe
 from onnxruntime_genai_b200.models.decoder import LayerWeights, PagedKVCache
-from stack_harness import BLOCK, RUNTIMES, beam_search, close, dtype_of, feed, greedy_ok, one_thread, open_engine, open_model, paged, random_tokens, rows_of, tol_of  # noqa: F401
+from stack_harness import BLOCK, RUNTIMES, beam_search, close, dtype_of, feed, greedy_ok, one_thread, open_engine, open_model, paged, random_tokens, rows_of, tol_of, wide_rows  # noqa: F401
 from stack_models import chunked, output_normed_stack, weights, write
 from stack_oracle import (clamped_expert, gelu_feed_forward, rms_norm, rotary_frequencies, rotate, routed_experts, same_chunk, sink_attention, stack_forward,
                           wavelength_scaled)
@@ -31,8 +31,8 @@ MIXED = output_normed_stack([chunked(), chunked(heads=6, kv_heads=3, dim=16, vdi
                              chunked(heads=8, kv_heads=1, dim=8, vdim=8, dims=8, chunk=1, ff=64, experts=4, top=1, limit=1.5),
                              chunked(heads=2, kv_heads=2, dim=32, vdim=8, chunk=64, dims=32, ff=72, experts=3, top=3, limit=0.4)])
 # sizes no vector path can take: odd widths and head sizes, an odd number of rotated pairs, factors that are 1
-ODD = output_normed_stack([chunked(heads=3, kv_heads=3, dim=9, vdim=5, dims=6, chunk=11, ff=13, scale=0.9),
-                           chunked(heads=3, kv_heads=1, dim=7, vdim=3, dims=2, chunk=5, ff=7, experts=5, top=2, scale=1.0)],
+ODD = output_normed_stack([chunked(heads=3, kv_heads=3, dim=9, vdim=5, dims=6, chunk=11, ff=13, scale=0.4),
+                           chunked(heads=3, kv_heads=1, dim=7, vdim=3, dims=2, chunk=5, ff=7, experts=5, top=2, scale=0.4)],
                           vocab=37, width=45, eps=2e-2, residual_mult=1.0, embed_scale=1.0)
 # every class of the tensor-core and warp-MMA attention kernels, experts on the grouped GEMMs, heads too wide for either
 WIDE = output_normed_stack([chunked(heads=4, kv_heads=2, dim=128, vdim=64, chunk=64, dims=64, scale=0.15, ff=128),
@@ -171,7 +171,7 @@ def test_head_norms_rotation_and_append(runtime, shape):
     rot = dict(dims=rd, base=300.0, scaling=dict(factor=4.0, original=100, low=1.0, high=4.0)) if rd else None
     fill = lambda x, c: torch.nn.functional.pad(x, (0, c - x.shape[-1])).reshape(T, -1)
     proj = torch.cat([fill(q, kr), fill(k, kr), fill(v, vr), torch.randn(T, 3, generator=g).to(dt)], 1)
-    wide = torch.zeros(T, (proj.shape[1] + 7) // 8 * 8, dtype=dt)[:, :proj.shape[1]].copy_(proj).to(dev)
+    wide = wide_rows(proj, dev)
     kc, vc = torch.full((20 * BLOCK, G, kr), 7.0, dtype=dt, device=dev), torch.full((20 * BLOCK, G, vr), 7.0, dtype=dt, device=dev)
     cos = sin = None
     if rd:
@@ -235,7 +235,7 @@ def _run_attention(case, shape, lens, chunk, runtime, splits=None, order=None):
         kc[rows_of(pg, b, p + n).to(dev)], vc[rows_of(pg, b, p + n).to(dev)] = case["k"][b].to(dev), case["v"][b].to(dev)
     new = lambda x: torch.cat([t[p:] for t, (p, _) in zip(x, lens)])
     proj = torch.cat([new(case["q"]).reshape(-1, H * d), new(case["gate"])], 1)
-    wide = torch.zeros(proj.shape[0], (proj.shape[1] + 7) // 8 * 8, dtype=dt)[:, :proj.shape[1]].copy_(proj).to(dev)
+    wide = wide_rows(proj, dev)
     t = {n: x.to(dev) for n, x in pg.items()}
     out = torch.full((proj.shape[0], H * dv), 5.0, dtype=dt, device=dev)
     ops.paged_attention(wide, kc, vc, t["cu"], t["past"], t["table"], BLOCK, H, G, d, case["scale"], 0, case["sink"].to(dev), 0.0,
