@@ -405,10 +405,12 @@ class DecoderModel:
                                        max_kv_len=s.max_kv_len, order=s.attn_order, min_q_len=s.min_q_len or None, out=out, **kw)
         if out is None:
             out = torch.empty(qkv.shape[0], args[1] * cols, dtype=qkv.dtype, device=qkv.device)
-        ops.paged_attention(qkv, kc, vc, s.cu_seqlens[:nd + 1], s.past_lens[:nd], table[:nd], *args, max_q_len=1,
-                            max_kv_len=s.max_kv_len, out=out, total_tokens=nd, **kw)
+        # The chunks first: where their keys are split, the merge pass runs over all rows of the matrix and leaves unspecified values in
+        # the rows of the single-token requests, which the second launch then writes.
         ops.paged_attention(qkv, kc, vc, s.cu_seqlens[nd:], s.past_lens[nd:], table[nd:], *args, max_q_len=s.max_q_len,
                             max_kv_len=s.max_kv_len, out=out, **kw)
+        ops.paged_attention(qkv, kc, vc, s.cu_seqlens[:nd + 1], s.past_lens[:nd], table[:nd], *args, max_q_len=1,
+                            max_kv_len=s.max_kv_len, out=out, total_tokens=nd, **kw)
         return out
 
     @staticmethod

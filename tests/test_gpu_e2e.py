@@ -142,6 +142,27 @@ def test_engine_isolated_equals_batched_on_gpu(dirs):
     assert engine.core.free_blocks == engine.options.num_blocks
 
 
+def test_short_portions_beside_single_tokens_of_long_requests(dirs):
+    """A step with single tokens and two-token portions over long caches: both attention launches split their keys, and neither may touch
+    the other's rows."""
+    model = og.Model(dirs[0])
+    rng = np.random.RandomState(3)
+    seqs = [rng.randint(3, 1000, n) for n in (330, 212, 301)]
+    want = []
+    for t in seqs:
+        eng = og.Engine(model)
+        r = og.Request(og.GeneratorParams(model))
+        want.append(eng.run_given([(r, t, list(range(len(t) - 3, len(t))))])[0].float())
+    eng = og.Engine(model)
+    reqs = [og.Request(og.GeneratorParams(model)) for _ in seqs]
+    eng.run_given([(r, t[:-3], []) for r, t in zip(reqs, seqs)])
+    first = eng.run_given([(r, t[-3:-3 + n], list(range(n))) for r, t, n in zip(reqs, seqs, (1, 2, 1))])
+    rest = eng.run_given([(r, t[-3 + n:], list(range(3 - n))) for r, t, n in zip(reqs, seqs, (1, 2, 1))])
+    for w, a, b in zip(want, first, rest):
+        got = torch.cat([a.float(), b.float()])
+        assert float((got - w).abs().max()) < 0.05 * float(w.std())
+
+
 def test_smoke_entry():
     import __graft_entry__ as g
     g.smoke()

@@ -400,6 +400,25 @@ def test_a_request_does_not_see_the_batch_around_it(tmp_path_factory, runtime):
     close(torch.cat(rows), alone.double(), tol_of(runtime) / 4)
 
 
+def test_short_portions_beside_single_tokens_of_long_requests(tmp_path_factory, runtime):
+    """Keys of both are split between CTAs (few heads, long runs): neither launch may touch the rows of the other."""
+    cfg = output_normed_stack([chunked(heads=2, kv_heads=2, dim=64, vdim=128, chunk=400, dims=32, scale=0.2, ff=64),
+                               chunked(heads=2, kv_heads=1, dim=64, vdim=64, chunk=1000, dims=64, scale=0.2, ff=64)], width=64)
+    m, cfg, w = open_model(tmp_path_factory, "zev_split", runtime, cfg)
+    seqs = [random_tokens(cfg, n, 60 + n) for n in (330, 212, 301)]
+    eng = open_engine(m, tokens=1024)
+    reqs = [og.Request(og.GeneratorParams(m)) for _ in seqs]
+    eng.run_given([(r, t[:-10], []) for r, t in zip(reqs, seqs)])
+    got, at = [[], [], []], [len(t) - 10 for t in seqs]
+    for cut in ((1, 2, 1), (2, 1, 3), (1, 1, 2), (3, 3, 1), (1, 2, 2)):
+        out = eng.run_given([(r, t[a:a + n], list(range(n))) for r, t, a, n in zip(reqs, seqs, at, cut)])
+        for i, (o, n) in enumerate(zip(out, cut)):
+            got[i].append(o.float().cpu())
+            at[i] += n
+    for t, g, a in zip(seqs, got, at):
+        close(torch.cat(g), stack_forward(cfg, w, t)[0][len(t) - 10:a], tol_of(runtime))
+
+
 def test_long_decoding(tmp_path_factory, runtime):
     """Hundreds of single-token steps: runs end and begin among decoded tokens, pages fill up."""
     m, cfg, w = open_model(tmp_path_factory, "zev_mixed", runtime, MIXED)
