@@ -35,8 +35,8 @@ ODD = output_normed_stack([chunked(heads=3, kv_heads=3, dim=9, vdim=5, dims=6, c
                            chunked(heads=3, kv_heads=1, dim=7, vdim=3, dims=2, chunk=5, ff=7, experts=5, top=2, scale=0.4)],
                           vocab=37, width=45, eps=2e-2, residual_mult=1.0, embed_scale=1.0)
 # every class of the tensor-core and warp-MMA attention kernels, experts on the grouped GEMMs, heads too wide for either
-WIDE = output_normed_stack([chunked(heads=4, kv_heads=2, dim=128, vdim=64, chunk=64, dims=64, scale=0.15, ff=128),
-                            chunked(heads=8, kv_heads=1, dim=64, vdim=128, chunk=100, dims=64, scale=0.2, ff=96, experts=16, top=4),
+WIDE = output_normed_stack([chunked(heads=4, kv_heads=2, dim=128, vdim=56, chunk=48, dims=96, scale=0.15, ff=128),
+                            chunked(heads=8, kv_heads=1, dim=64, vdim=128, chunk=100, dims=64, scale=0.2, ff=104, experts=12, top=4),
                             chunked(heads=2, kv_heads=2, dim=192, vdim=128, chunk=50, dims=128, scale=0.1, ff=0),
                             chunked(heads=3, kv_heads=1, dim=256, vdim=256, chunk=300, dims=32, scale=0.1, ff=70),
                             chunked(heads=4, kv_heads=4, dim=128, vdim=128, chunk=130, dims=128, scale=0.15, ff=200, experts=6, top=2),
@@ -154,7 +154,7 @@ def test_gelu_gated_feed_forward(runtime, T, inter, width):
     close(got, gelu_feed_forward(x.double(), {k: v.double() for k, v in w.items()}, ""), tol_of(runtime))
 
 
-PREPS = [(4, 2, 24, 16, 16), (3, 3, 9, 5, 6), (6, 1, 128, 64, 64), (5, 5, 40, 40, 0), (2, 1, 264, 24, 264), (16, 4, 64, 128, 32), (8, 8, 8, 8, 2)]
+PREPS = [(4, 2, 24, 16, 16), (3, 3, 9, 5, 6), (5, 1, 128, 72, 80), (5, 5, 40, 40, 0), (2, 1, 264, 24, 264), (16, 4, 64, 128, 32), (8, 8, 8, 8, 2)]
 
 
 @pytest.mark.parametrize("shape", PREPS, ids=lambda s: "x".join(map(str, s)))
@@ -200,7 +200,7 @@ def test_head_norms_rotation_and_append(runtime, shape):
     assert (kc.cpu()[rest] == 7).all() and (vc.cpu()[rest] == 7).all() and torch.equal(got[:, -3:], proj[:, -3:])
 
 
-SHAPES = [(4, 2, 24, 16), (3, 3, 16, 8), (6, 3, 128, 64), (8, 1, 64, 128), (2, 2, 128, 128), (4, 2, 96, 96), (3, 1, 192, 128), (2, 1, 256, 256), (2, 2, 72, 200),
+SHAPES = [(4, 2, 24, 16), (3, 3, 16, 8), (6, 2, 128, 72), (8, 1, 64, 128), (2, 2, 128, 128), (4, 2, 96, 96), (3, 1, 192, 128), (2, 1, 256, 256), (2, 2, 72, 200),
           (2, 1, 264, 24), (20, 1, 40, 40)]
 
 
@@ -290,7 +290,7 @@ def test_a_sink_takes_its_share(runtime):
         assert (float(got.abs().max()) < 1e-6) == (s > 0)
 
 
-EXPERTS = [(8, 3, 40, 72), (5, 2, 7, 45), (16, 4, 96, 128), (3, 3, 64, 64), (4, 1, 130, 40), (64, 6, 32, 128)]
+EXPERTS = [(8, 3, 40, 72), (5, 2, 7, 45), (12, 4, 104, 128), (3, 3, 64, 64), (4, 1, 130, 40), (64, 6, 32, 128)]
 
 
 @pytest.mark.parametrize("E,top,ff,W", EXPERTS)
