@@ -38,7 +38,9 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
   if (reinterpret_cast<uintptr_t>(out) & 3) return -1;
   if (splits < 1) splits = 1;
   if (kv_chunk < 0 || (kv_chunk % ATT_BN) || (long long)B * splits > 65535) return -1;
-  if (splits > 1 && ogb_attention_scratch_bytes(total_tokens, a->Hq, a->dv, splits) > scratch_bytes) return -2;
+  if ((splits > 1 || a->raw) && (long long)splits * total_tokens * a->Hq * (a->dv + 2) * 4 > scratch_bytes) return -2;
+  const int maps = a->maps > 1 ? a->maps : 1;
+  if (a->dk % (8 * maps) || (a->raw && (a->sinks || !scratch))) return -1;
   AttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
   p.k_cache = static_cast<const __nv_bfloat16*>(k_cache); p.v_cache = static_cast<const __nv_bfloat16*>(v_cache);
@@ -47,11 +49,12 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
   p.total_rows = total_tokens * a->Hq;
   p.part_o = static_cast<float*>(scratch);
   p.part_ml = p.part_o ? p.part_o + size_t(splits) * p.total_rows * a->dv : nullptr;
-  p.sinks = a->sinks; p.scale = a->scale; p.softcap = 0.f; p.window = a->window; p.local = a->chunk;
+  p.sinks = a->sinks; p.scale = a->scale; p.softcap = a->softcap; p.window = a->window; p.local = a->chunk;
   p.B = B; p.Hq = a->Hq; p.Hkv = a->Hkv; p.splits = splits; p.chunk = splits > 1 ? kv_chunk : 0;
   p.status = status; p.order = order; p.skip_rows = skip_rows;
   p.dk = a->dk; p.dv = a->dv;
-  p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.gate_stride = a->gate_stride;
+  p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.gate_stride = a->gate_stride; p.gate_wide = a->gate && a->gate_wide;
+  p.maps = maps; p.raw = a->raw;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
   if (a->dk <= 64) return LaunchMixedKeys<64>(p, max_q_len, stream);

@@ -65,10 +65,21 @@ struct AttnParams {
   int local;
   // gate (may be null) [tokens, Hq]: every head's output is multiplied by the sigmoid of its entry.
   const __nv_bfloat16* gate; int gate_stride;
+  int gate_wide;     // gate [tokens, Hq * dv]: one entry per output column instead of one per head
+  // maps > 1: query vector h (dk / maps columns wide) belongs to map h % maps of its key head, whose row holds the maps' keys side by side: the
+  // query is staged at its map's columns among zeros, so keys and values are read once for all maps.
+  int maps;
+  int raw;           // partial results are written even without splits, and not merged here
 };
 
+__device__ __forceinline__ float attn_sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
 __device__ __forceinline__ float attn_gate(const __nv_bfloat16* gate, int stride, int tok, int hq) {
-  return gate ? 1.f / (1.f + __expf(-bf2f(gate[size_t(tok) * stride + hq]))) : 1.f;
+  return gate ? attn_sigmoid(bf2f(gate[size_t(tok) * stride + hq])) : 1.f;
+}
+// gate entries of two neighbouring output columns
+__device__ __forceinline__ float2 attn_gate2(const __nv_bfloat16* g) {
+  const float2 v = make_float2(bf2f(g[0]), bf2f(g[1]));
+  return make_float2(attn_sigmoid(v.x), attn_sigmoid(v.y));
 }
 
 template <int SROW>
@@ -131,8 +142,11 @@ paged_attention_kernel(AttnParams p) {
   const int last_tq = min(q_len - 1, (row0 + BM - 1) / G);
   int kv_hi = full ? past : past + last_tq + 1;
   int kv_lo = 0;
-  if (p.window > 0) kv_lo = max(0, past + row0 / G - p.window + 1);
   int split_base = 0;                // first key the splits divide
+  if (p.window > 0) {
+    kv_lo = max(0, past + row0 / G - p.window + 1);
+    split_base = kv_lo / ATT_BN * ATT_BN;
+  }
   if (p.local > 0) {
     kv_lo = (past + row0 / G) / p.local * p.local;
     split_base = kv_lo / ATT_BN * ATT_BN;
@@ -148,7 +162,8 @@ paged_attention_kernel(AttnParams p) {
   const int tile_begin = kv_lo / ATT_BN;
   const int tile_end = kv_hi > kv_lo ? (kv_hi + ATT_BN - 1) / ATT_BN : tile_begin;
   const int n_tiles = tile_end - tile_begin;
-  if (p.splits > 1 && n_tiles == 0) {
+  const bool partial = p.splits > 1 || p.raw;
+  if (partial && n_tiles == 0) {
     // Nothing in this split's range: mark its partials empty for the combine and leave before any copy is issued.
     for (int r = tid; r < BM; r += ATT_THREADS) {
       const int gr = row0 + r;
@@ -260,9 +275,15 @@ paged_attention_kernel(AttnParams p) {
   for (int c = tid; c < BM * CHUNKS; c += ATT_THREADS) {
     const int r = c / CHUNKS, ch = c % CHUNKS;
     const int gr = row0 + r;
-    const bool ok = gr < rows && ch * 8 < dk;
+    bool ok = gr < rows && ch * 8 < dk;
     const __nv_bfloat16* src = p.q;
-    if (ok) src = p.q + size_t(tok0 + gr / G) * p.q_stride + size_t(kvh * G + gr % G) * dk + ch * 8;
+    if (p.maps > 1) {
+      const int hq = kvh * G + gr % G, dm = dk / p.maps, c0 = (hq % p.maps) * dm;
+      ok = ok && ch * 8 >= c0 && ch * 8 < c0 + dm;
+      if (ok) src = p.q + size_t(tok0 + gr / G) * p.q_stride + size_t(hq) * dm + ch * 8 - c0;
+    } else if (ok) {
+      src = p.q + size_t(tok0 + gr / G) * p.q_stride + size_t(kvh * G + gr % G) * dk + ch * 8;
+    }
     cp_async16(sQ + swz<SROW>(r, ch), src, ok);
   }
   if (KV8) {
@@ -358,7 +379,7 @@ paged_attention_kernel(AttnParams p) {
           bool ok = (hi ? valid_hi : valid_lo) && j >= kv_lo && j < kv_hi && (full || j <= qpos);
           ok = ok && j >= (hi ? first_hi : first_lo);
           float x = s[nt][e];
-          if (p.softcap > 0.f) x = p.softcap * tanhf(x * p.scale / p.softcap) * LOG2E;
+          if (p.softcap > 0.f) x = p.softcap * tanh_capped(x * p.scale / p.softcap) * LOG2E;
           else x *= sc2;
           x = ok ? x : -INFINITY;
           s[nt][e] = x;
@@ -449,7 +470,7 @@ paged_attention_kernel(AttnParams p) {
       acc[d] = a;
     }
     const int tq = gr / G, hq = kvh * G + gr % G;
-    if (p.splits > 1) {
+    if (partial) {
       const size_t grow = size_t(tok0 + tq) * p.Hq + hq;
       float* po = p.part_o + (size_t(split) * p.total_rows + grow) * dv + seg * SEG;
 #pragma unroll
@@ -466,10 +487,15 @@ paged_attention_kernel(AttnParams p) {
         scale_o = exp2f(M - mm);
         L = L * scale_o + exp2f(sk - mm);
       }
-      const float inv = (L > 0.f ? scale_o / L : 0.f) * attn_gate(p.gate, p.gate_stride, tok0 + tq, hq);
+      const float inv = (L > 0.f ? scale_o / L : 0.f) * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * dv + seg * SEG;
+      const __nv_bfloat16* pg = p.gate + (p.gate_wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * dv + seg * SEG : 0);
 #pragma unroll
-      for (int d = 0; d < SEG; d += 2) if (FIT || seg * SEG + d < dv) *reinterpret_cast<uint32_t*>(po + d) = pack_bf16x2(acc[d] * inv, acc[d + 1] * inv);
+      for (int d = 0; d < SEG; d += 2)
+        if (FIT || seg * SEG + d < dv) {
+          const float2 g = p.gate_wide ? attn_gate2(pg + d) : make_float2(1.f, 1.f);
+          *reinterpret_cast<uint32_t*>(po + d) = pack_bf16x2(acc[d] * inv * g.x, acc[d + 1] * inv * g.y);
+        }
     }
     return;
   }
@@ -481,7 +507,7 @@ paged_attention_kernel(AttnParams p) {
     if (gr >= rows) continue;
     const int tq = gr / G, hq = kvh * G + gr % G;
     float m = half ? m_hi : m_lo, l = half ? l_hi : l_lo;
-    if (p.splits > 1) {
+    if (partial) {
       const size_t grow = size_t(tok0 + tq) * p.Hq + hq;
       float* po = p.part_o + (size_t(split) * p.total_rows + grow) * dv;
 #pragma unroll
@@ -499,11 +525,15 @@ paged_attention_kernel(AttnParams p) {
         scale_o = exp2f(m - mm);
         l = l * scale_o + exp2f(sk - mm);
       }
-      const float inv = (l > 0.f ? scale_o / l : 0.f) * attn_gate(p.gate, p.gate_stride, tok0 + tq, hq);
+      const float inv = (l > 0.f ? scale_o / l : 0.f) * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * dv;
+      const __nv_bfloat16* pg = p.gate + (p.gate_wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * dv : 0);
 #pragma unroll
       for (int i = 0; i < DTILES; ++i)
-        if (FIT || i * 8 < dv) *reinterpret_cast<uint32_t*>(po + i * 8 + t4 * 2) = pack_bf16x2(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
+        if (FIT || i * 8 < dv) {
+          const float2 g = p.gate_wide ? attn_gate2(pg + i * 8 + t4 * 2) : make_float2(1.f, 1.f);
+          *reinterpret_cast<uint32_t*>(po + i * 8 + t4 * 2) = pack_bf16x2(o[i][half * 2] * inv * g.x, o[i][half * 2 + 1] * inv * g.y);
+        }
     }
   }
 }
@@ -512,7 +542,7 @@ paged_attention_kernel(AttnParams p) {
 template <int DV, bool FIT>
 __global__ void attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out, int out_stride,
-                                         int total_rows, int Hq, int splits, int dv, const __nv_bfloat16* __restrict__ gate, int gate_stride) {
+                                         int total_rows, int Hq, int splits, int dv, const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_wide) {
   const int D = FIT ? DV : dv;
   pdl_launch_dependents();
   pdl_wait();
@@ -540,12 +570,13 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o, const
       if (d < D) acc[i] += w * po[d];
     }
   }
-  const float inv = (L > 0.f ? 1.f / L : 0.f) * attn_gate(gate, gate_stride, tok, hq);
+  const float inv = (L > 0.f ? 1.f / L : 0.f) * (gate_wide ? 1.f : attn_gate(gate, gate_stride, tok, hq));
   __nv_bfloat16* o = out + size_t(tok) * out_stride + size_t(hq) * D;
+  const __nv_bfloat16* pg = gate + (gate_wide ? size_t(tok) * gate_stride + size_t(hq) * D : 0);
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) o[d] = f2bf(acc[i] * inv);
+    if (d < D) o[d] = f2bf(acc[i] * inv * (gate_wide ? attn_sigmoid(bf2f(pg[d])) : 1.f));
   }
 }
 
@@ -566,10 +597,10 @@ static int LaunchAttentionMode(const AttnParams& p, int max_q_len, cudaStream_t 
   dim3 grid(q_tiles, p.Hkv, p.B * p.splits);
   launch_pdl(kern, grid, dim3(ATT_THREADS), SMEM, stream, p);
   if (cudaGetLastError() != cudaSuccess) return -4;
-  if (p.splits > 1) {
+  if (p.splits > 1 && !p.raw) {
     const int warps = 4;
     launch_pdl(attention_combine_kernel<DV, FIT>, dim3((p.total_rows + warps - 1) / warps), dim3(warps * 32), 0, stream,
-               static_cast<const float*>(p.part_o), static_cast<const float*>(p.part_ml), p.sinks, p.out, p.out_stride, p.total_rows, p.Hq, p.splits, p.dv, p.gate, p.gate_stride);
+               static_cast<const float*>(p.part_o), static_cast<const float*>(p.part_ml), p.sinks, p.out, p.out_stride, p.total_rows, p.Hq, p.splits, p.dv, p.gate, p.gate_stride, p.gate_wide);
     if (cudaGetLastError() != cudaSuccess) return -4;
   }
   return 0;

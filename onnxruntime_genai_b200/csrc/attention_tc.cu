@@ -59,20 +59,22 @@ OGB_API int ogb_attention_tc_latent_supported(int dim, int rot, int vdim) {
 // Long prompts of a latent-attention layer.  q: row t holds H heads of (dim | rot) rotated queries; kv [rows, >= H * (dim + vdim)]: the
 // expanded keys (head-major columns) then values; kr [rows, >= kr_col + rot]: the shared rotated key part from column kr_col on.
 // row_base / first_kv [B]: dense row of each request's first expanded position (a multiple of 16) and that position; row_base < 0
-// leaves the request out.  Output row t: H heads of vdim columns.
+// leaves the request out.  Output row t: H heads of vdim columns, times the sigmoid of gate [T, H * vdim] (may be null).  sinks (may be null) [H].
 OGB_API int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldkv, const void* kr, int ldkr, int kr_col, int rows,
                                     const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* row_base, const int32_t* first_kv, void* out,
-                                    int out_stride, float scale, int window, int B, int max_q_len, int H, int dim, int rot, int vdim, int* status,
-                                    void* stream_) {
+                                    int out_stride, float scale, int window, const float* sinks, const void* gate, int gate_stride, int B, int max_q_len,
+                                    int H, int dim, int rot, int vdim, int* status, void* stream_) {
   if (B <= 0 || max_q_len <= 0 || rows <= 0) return 0;
   if (!ogb_attention_tc_latent_supported(dim, rot, vdim)) return -5;
   if ((q_stride % 8) || (out_stride % 8) || (ldkv % 8) || (ldkr % 8) || (kr_col % 8)) return -1;
+  if (gate && ((gate_stride % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -1;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kr) | reinterpret_cast<uintptr_t>(out)) & 15) return -1;
   TcAttnParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
   p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.block_size = 16;
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;
   p.scale = scale; p.window = window; p.B = B; p.Hq = H; p.Hkv = H; p.min_rows = 1; p.status = status;
+  p.sinks = sinks; p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_stride = gate_stride; p.gate_wide = gate != nullptr;
   p.lat.row_base = row_base; p.lat.first_kv = first_kv; p.lat.dim = dim; p.lat.rot = rot; p.lat.vdim = vdim; p.lat.kr_col = kr_col;
   CUtensorMap mk, mv, mr;
   const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(kv);

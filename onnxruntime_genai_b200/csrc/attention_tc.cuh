@@ -74,7 +74,17 @@ struct TcAttnParams {
   int dk, dv;        // columns of a key (query) head and of a value head (MIX)
   int local;         // > 0: a query sees the keys of its own run of `local` positions only (runs are counted from position 0)
   const __nv_bfloat16* gate; int gate_stride;      // (may be null) [tokens, Hq]: a head's output is multiplied by the sigmoid of its entry
+  int gate_wide;     // gate [tokens, Hq * dv]: one entry per output column
+  // maps > 1 (MIX): Hkv counts the key vectors of all maps; key vector v meets the query vectors h of its group with h % maps == v % maps and
+  // the value head v / maps.
+  int maps;
+  // part_o (may be null; MIX): instead of `out`, sums [total_rows, dv], and (maximum, sum of weights) in part_ml [splits, total_rows, 2], whose
+  // entries of the other splits are marked empty.
+  float *part_o, *part_ml;
+  int splits, total_rows;
 };
+// entry of a query row in a grid of key vectors
+__device__ __forceinline__ int tca_query(int kvh, int i, int G, int maps) { return maps > 1 ? ((kvh / maps) * G + i) * maps + kvh % maps : kvh * G + i; }
 
 template <int DK, int DV, int BN>
 struct TcaCfg {
@@ -159,7 +169,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   // CTAs are dispatched in block-index order: the last row tiles of a causal prompt see the most keys, so they go first and
   // the tail of the grid is made of short CTAs
   const int row0 = int(gridDim.x - 1 - blockIdx.x) * TCA_BM;
-  if (rows < p.min_rows || row0 >= rows) return;      // before anything is allocated
+  if (rows * (MIX ? p.maps : 1) < p.min_rows || row0 >= rows) return;      // before anything is allocated
   if (LAT && p.lat.row_base[b] < 0) return;
   const int past = p.past_lens[b];
   const bool full = p.window < 0;
@@ -242,7 +252,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
               for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh * p.dk + h * 64, slot0);
             } else {
 #pragma unroll
-              for (int h = 0; h < Cfg::V_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh * p.dv + h * 64, slot0);
+              for (int h = 0; h < Cfg::V_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh / p.maps * p.dv + h * 64, slot0);
             }
           } else {
 #pragma unroll
@@ -320,7 +330,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     const int gr = row0 + r;
     const bool valid = gr < rows;
     const int tq = valid ? gr / G : q_len - 1;
-    const int hq = kvh * G + (valid ? gr % G : 0);
+    const int hq = MIX ? tca_query(kvh, valid ? gr % G : 0, G, p.maps) : kvh * G + (valid ? gr % G : 0);
     const int qpos = past + tq;
     const int first_local = p.local > 0 ? qpos / p.local * p.local : 0;
     // The two warps of a lane quarter meet on a named barrier.  It has no time limit, so no softmax warp ever leaves the tile loop
@@ -367,8 +377,17 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     // soft-cap / mask 16 scores of tile `it` in place and return their maximum (raw units: times kmul gives the exponent)
     auto prep16 = [&](int it, float (&x)[HC], int c, bool interior) -> float {
       if (capped) {
+        // (most scores lie where the polynomial holds: one vote spares the others the exponential and the division)
+        float far = 0.f;
 #pragma unroll
-        for (int e = 0; e < 16; ++e) x[c * 16 + e] = capl * tanhf(x[c * 16 + e] * inv_cap);
+        for (int e = 0; e < 16; ++e) { x[c * 16 + e] *= inv_cap; far = fmaxf(far, fabsf(x[c * 16 + e])); }
+        if (__any_sync(0xffffffffu, far > SOFT_CAP_NEAR)) {
+#pragma unroll
+          for (int e = 0; e < 16; ++e) x[c * 16 + e] = capl * tanh_capped(x[c * 16 + e]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 16; ++e) x[c * 16 + e] = capl * tanh_near(x[c * 16 + e]);
+        }
       }
       if (!interior) {
         const int jb = (tile_begin + it) * BN + half * HC + c * 16;
@@ -472,9 +491,18 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
         l = l * scale_o + exp2f(sk - mm);
       }
       float inv = l > 0.f ? scale_o / l : 0.f;
-      if (p.gate) inv /= 1.f + __expf(-bf2f(p.gate[size_t(tok0 + tq) * p.gate_stride + hq]));
+      const bool wide = p.gate_wide;
+      if (p.gate && !wide) inv /= 1.f + __expf(-bf2f(p.gate[size_t(tok0 + tq) * p.gate_stride + hq]));
       const int v_cols = LAT ? p.lat.vdim : (MIX ? p.dv : DV);
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * v_cols + half * OC;
+      const __nv_bfloat16* pg = p.gate + (wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * v_cols + half * OC : 0);
+      const bool raw = MIX && p.part_o;
+      const size_t part_row = size_t(tok0 + tq) * p.Hq + hq;
+      if (raw && valid && half == 0) {
+        p.part_ml[part_row * 2] = m_ref;
+        p.part_ml[part_row * 2 + 1] = l;
+        for (int s = 1; s < p.splits; ++s) p.part_ml[(size_t(s) * p.total_rows + part_row) * 2] = -INFINITY;
+      }
 #pragma unroll
       for (int c = 0; c < OC / 16; ++c) {
         uint32_t v[16];
@@ -485,7 +513,28 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
 #pragma unroll
           for (int e = 0; e < 16; ++e) v[e] = 0u;
         }
-        if (valid) {
+        if (wide) {
+          // (column ranges of a row start on 16-byte boundaries)
+#pragma unroll
+          for (int h8 = 0; h8 < 16; h8 += 8)
+            if (valid && half * OC + c * 16 + h8 < v_cols) {
+              const uint4 q = *reinterpret_cast<const uint4*>(pg + c * 16 + h8);
+              const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 g = unpack_bf16x2(qw[e]);
+                v[h8 + 2 * e] = __float_as_uint(__uint_as_float(v[h8 + 2 * e]) / (1.f + __expf(-g.x)));
+                v[h8 + 2 * e + 1] = __float_as_uint(__uint_as_float(v[h8 + 2 * e + 1]) / (1.f + __expf(-g.y)));
+              }
+            }
+        }
+        if (raw) {
+          float* pr = p.part_o + part_row * p.dv + half * OC + c * 16;
+#pragma unroll
+          for (int e = 0; e < 16; e += 4)
+            if (valid && half * OC + c * 16 + e < v_cols)
+              *reinterpret_cast<float4*>(pr + e) = make_float4(__uint_as_float(v[e]), __uint_as_float(v[e + 1]), __uint_as_float(v[e + 2]), __uint_as_float(v[e + 3]));
+        } else if (valid) {
           uint4 lo, hi;
           lo.x = pack_bf16x2(__uint_as_float(v[0]) * inv, __uint_as_float(v[1]) * inv);
           lo.y = pack_bf16x2(__uint_as_float(v[2]) * inv, __uint_as_float(v[3]) * inv);
@@ -510,7 +559,7 @@ template <int DK, int DV, int BN, bool MIX = false>
 static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
   using Cfg = TcaCfg<DK, DV, BN>;
   auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX>;
-  const int kw = p.Hkv * (MIX ? p.dk : DK), vw = p.Hkv * (MIX ? p.dv : DV);      // row widths of the caches
+  const int kw = p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
   CUtensorMap mk, mv;

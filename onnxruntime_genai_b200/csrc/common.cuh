@@ -36,6 +36,24 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t u) {
   return __bfloat1622float2(v);
 }
 
+// tanh for soft-capped scores.  |y| <= SOFT_CAP_NEAR: an odd polynomial, least squares over Chebyshev nodes in y^2 (absolute error below
+// 1e-7); beyond: 1 - 2 / (1 + e^(2 |y|)), where the difference no longer cancels.
+constexpr float SOFT_CAP_NEAR = 0.75f;
+constexpr float TANH_C1 = -0.3333296775817871f, TANH_C2 = 0.13325515389442444f, TANH_C3 = -0.053349819034338f, TANH_C4 = 0.01959378644824028f,
+                TANH_C5 = -0.004723952151834965f;
+__device__ __forceinline__ float tanh_near(float y) {
+  const float t = y * y;
+  float r = fmaf(t, TANH_C5, TANH_C4);
+  r = fmaf(t, r, TANH_C3);
+  r = fmaf(t, r, TANH_C2);
+  r = fmaf(t, r, TANH_C1);
+  return y * fmaf(t, r, 1.f);
+}
+__device__ __forceinline__ float tanh_capped(float y) {
+  const float a = fabsf(y);
+  return a <= SOFT_CAP_NEAR ? tanh_near(y) : copysignf(1.f - __fdividef(2.f, 1.f + exp2f(fminf(a, 40.f) * 2.885390081777927f)), y);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

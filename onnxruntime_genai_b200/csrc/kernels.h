@@ -53,7 +53,7 @@ int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const
 
 // ---- gemm_simt.cu: fp32 products and bf16 products TMA cannot address
 int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K, int batch,
-                  const float* residual, int ldr, int in_fp32, int out_fp32, void* stream);
+                  const float* residual, int ldr, const void* bias, int in_fp32, int out_fp32, void* stream);
 
 // Grouped expert product over token rows sorted by expert in plain arithmetic (tile list of ogb_moe_sort, tiles of at most 64 rows).
 int ogb_moe_gemm_simt(const void* A, int lda, const void* W, void* C, int ldc, int N, int K, const int32_t* tile_expert, const int32_t* tile_row0,
@@ -67,13 +67,38 @@ int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const f
 // Head norms, rotation and cache append of an attention layer: proj row t holds Hq query heads and Hkv key heads of key_row columns (the
 // first `dim` are the head, the rest zeros) and Hkv value heads of value_row columns.  Queries are replaced in place, keys and values go to
 // row slots[t] of the caches (slot < 0: nowhere).  Norm weights fp32 [dim] (null: no norm), cos / sin fp32 [max_pos, rot / 2] (rot 0: none).
-int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
+int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
                  const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
                  void* v_cache, int T, int fp32, void* stream);
 // h[t] += w * v / sqrt(mean(v^2) + eps), x[t] = h[t] as bf16 (x may be null).  v = y[t], or (inv_pos not null) the weighted sum of the
 // experts' rows sum_j topk_w[t, j] * y[inv_pos[t, j]], j < k.
 int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const float* w, float eps, void* x, const int32_t* inv_pos, const float* topk_w, int k,
                    int T, int H, void* stream);
+// Sum into the fp32 stream and tanh norm of the result: n = h_in[r] + v + y2[r] + first[r] + step, h_out[r] = n (h_out may be null, or h_in),
+// x[i] = tanh(alpha * n) * w + b, r = rows ? rows[i] : i.  v = y[r] (y may be null), or the weighted sum of experts' rows as above; y, y2 and x
+// in the compute type; first (fp32 rows) and step (one fp32 row) may be null.
+typedef struct OgbTanhNorm {
+  const float* h_in; float* h_out;
+  const void* y; const void* y2;
+  const int32_t* inv_pos; const float* topk_w;
+  const float* first; const float* step;
+  const float* w; const float* b;
+  void* x; const int32_t* rows;
+  int ldy, ldy2, k, n_rows, H, fp32;
+  float alpha;
+} OgbTanhNorm;
+int ogb_add_tanh_norm(const OgbTanhNorm* p, void* stream);
+// Token embedding plus a row hashed from (previous token, token): out[t] = table[id] * scale + bigram[(prev * mul_prev + id * mul_cur) mod buckets],
+// row `buckets` for a sequence's first token.  The previous token of a step's first token comes from the paged pool `tokens` [slots]; every
+// token of the step is stored there.
+typedef struct OgbBigram {
+  const int32_t *ids, *slots, *cu_seqlens, *past_lens, *block_table;
+  int32_t* tokens;
+  int table_cols, block_size, B, T, H, vocab, buckets, fp32;
+  long long mul_prev, mul_cur;
+  float scale;
+} OgbBigram;
+int ogb_embedding_bigram(const OgbBigram* p, const void* table, const void* bigram, float* out, void* stream);
 // Expert activations on rows of alternating (gate, up) columns [n, 2 I]: kind 0 silu(g) * u, 1 clamped g * sigmoid(alpha g) * (u + 1).
 int ogb_expert_act(const void* gu, void* out, long long n, int I, int kind, float alpha, float limit, int fp32, void* stream);
 int ogb_act_mul_rows(const void* x, int ldx, void* out, int ldo, int T, int I, int act, int fp32, void* stream);
@@ -85,15 +110,31 @@ int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const void* bias
 int ogb_attention_tc_latent_supported(int dim, int rot, int vdim);
 int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldkv, const void* kr, int ldkr, int kr_col, int rows,
                             const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* row_base, const int32_t* first_kv, void* out,
-                            int out_stride, float scale, int window, int B, int max_q_len, int H, int dim, int rot, int vdim, int* status,
-                            void* stream);
+                            int out_stride, float scale, int window, const float* sinks, const void* gate, int gate_stride, int B, int max_q_len,
+                            int H, int dim, int rot, int vdim, int* status, void* stream);
 
 // ---- attention_mixed.cu, attention_tc_mixed.cu, attention_simt.cu: attention layers with sizes of their own.  Hq query heads over Hkv key /
 // value heads (q rows: Hq heads of dk columns first; caches [slots, Hkv, dk] and [slots, Hkv, dv]; out rows: Hq heads of dv columns).
 // window > 0: position p sees (p - window, p]; chunk > 0: the keys of p's own run of `chunk` positions; 0: every earlier key.
 // sinks (may be null) [Hq]: a logit in each head's denominator.  gate (may be null) [tokens, gate_stride], in the model's element type: a
-// head's output is multiplied by the sigmoid of its entry.
-typedef struct OgbAttnLayer { int Hq, Hkv, dk, dv, window, chunk, gate_stride; float scale; const float* sinks; const void* gate; } OgbAttnLayer;
+// head's output is multiplied by the sigmoid of its entry (gate_wide: a row holds Hq * dv entries, one for every output column).
+// softcap > 0: a scaled score s becomes softcap * tanh(s / softcap).  maps > 1: query vector h belongs to map h % maps, is dk / maps columns
+// wide and meets only that map's columns of its key head (Hq counts query vectors, a key head holds the vectors of all maps side by side).
+// raw: instead of `out`, fp32 partial results go to scratch: [splits, tokens * Hq, dv] sums and, behind them, [splits, tokens * Hq, 2] (maximum
+// in log2 units, sum of the weights); ogb_attention_diff_merge reads them.
+typedef struct OgbAttnLayer {
+  int Hq, Hkv, dk, dv, window, chunk, gate_stride;
+  float scale;
+  const float* sinks;
+  const void* gate;
+  int gate_wide, maps, raw;
+  float softcap;
+} OgbAttnLayer;
+// Differential attention on raw partial results of H heads with two maps each (query vectors 2 h and 2 h + 1): with a1 and a2 the maps'
+// results, o = a1 - lambda * a2, out = o / sqrt(mean(o^2) + eps) * post over the head's first vdim columns (columns vdim .. dv - 1 are zeros),
+// times the sigmoid of gate [T, H * dv] (may be null).
+int ogb_attention_diff_merge(const float* part, int splits, int T, int part_tokens, int H, int dv, int vdim, float lambda, float post, float eps,
+                             const void* gate, int gate_stride, void* out, int out_stride, int fp32, void* stream);
 int ogb_attention_mixed_supported(int dk, int dv);
 int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
                         const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
@@ -102,25 +143,31 @@ int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stride, cons
 int ogb_attention_tc_mixed_supported(int dk, int dv, int block_size, int cache_slots);
 int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
                            const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
-                           int max_q_len, int min_rows, int cache_slots, int* status, void* stream);
+                           int max_q_len, int min_rows, int cache_slots, int splits, int total_tokens, void* scratch, long long scratch_bytes,
+                           int* status, void* stream);
 int ogb_attention_simt(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
                        const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B, int T,
-                       int fp32, void* stream);
+                       void* scratch, long long scratch_bytes, int fp32, void* stream);
 
 // ---- latent_attention.cu: attention over a paged cache of latent rows [c (R) | rotated key (rot)]
 typedef struct OgbLatentShape { int H, dim, rot, vdim, R, rot_dims; } OgbLatentShape;
-int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const float* norm_w, float eps, const int32_t* positions, const float* cos,
-                    const float* sin, int max_pos, const int32_t* slots, void* cache, int ldcache, int T, int fp32, void* stream);
+// q (may be null) [T, H * (dim | rot)]: the rotary parts are rotated in place; down (may be null) [T, R | rot]: normed and rotated into the cache;
+// cq (may be null) [T, q_rank]: RMS-normed in place with weight cq_w.
+int ogb_latent_prep(void* q, int ldq, const void* down, int ldd, void* cq, int ldcq, int q_rank, const float* cq_w, const OgbLatentShape* sh,
+                    const float* norm_w, float eps, const int32_t* positions, const float* cos, const float* sin, int max_pos, const int32_t* slots,
+                    void* cache, int ldcache, int T, int fp32, void* stream);
+// out[t, i] *= sigmoid(gate[t, i]), i < n
+int ogb_gate_rows(void* out, int ldo, const void* gate, int ldg, int T, int n, int fp32, void* stream);
 int ogb_latent_mma_supported(const OgbLatentShape* sh);
 int ogb_latent_rows_per_tile(int H, int max_q_len);
 long long ogb_latent_scratch_bytes(int total_rows, int R, int splits);
 int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                          const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
-                         void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
-                         long long scratch_bytes, const int32_t* order, int* status, void* stream);
+                         void* out, float scale, int window, const float* sinks, int B, int T, int max_q_len, int skip_q_len, int splits,
+                         void* scratch, long long scratch_bytes, const int32_t* order, int* status, void* stream);
 int ogb_latent_attention_simt(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                               const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
-                              void* out, float scale, int window, int B, int T, int skip_q_len, int fp32, void* stream);
+                              void* out, float scale, int window, const float* sinks, int B, int T, int skip_q_len, int fp32, void* stream);
 int ogb_latent_gather(const void* cache, int ldcache, const int32_t* block_table, int table_cols, int block_size, const int32_t* row_base,
                       const int32_t* first_kv, const int32_t* kv_len, const int32_t* req, int n_req, int rows, int width, void* out, int ldo,
                       void* stream);
@@ -137,7 +184,8 @@ int ogb_collective(int mode, const void* in, void* out, const void* residual, lo
                    void* stream);
 
 // ---- moe.cu
-int ogb_moe_topk(const float* logits, int ld, int T, int E, int k, int mode, int32_t* topk_idx, float* topk_w, void* stream);
+// shared: row t gets one more entry, expert E with weight 1 (rows of k + 1).
+int ogb_moe_topk(const float* logits, int ld, int T, int E, int k, int mode, int shared, int32_t* topk_idx, float* topk_w, void* stream);
 int ogb_moe_max_tiles(int n, int experts, int bt);
 int ogb_moe_fp4_reads_row_map(int token_tile, int K, int half);
 int ogb_moe_sort(const int32_t* topk_idx, int T, int k, int E, int e_lo, int e_hi, int bt, int32_t* expert_offsets,

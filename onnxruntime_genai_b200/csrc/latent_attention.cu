@@ -12,7 +12,8 @@
 //                        few; long prompts take the tensor-memory kernel (attention_tc.cu) on expanded keys and values instead.
 //   latent_simt_kernel   the same op in plain fp32 arithmetic for fp32 models and for sizes the other kernels cannot address.
 //   latent_gather_kernel cached rows of some requests into a dense matrix (input of the key / value expansion of long prompts).
-// A query at position p sees keys (p - window, p] (window > 0) or [0, p].  Built without fast-math.
+//   gate_rows_kernel     an output gate: rows times the sigmoid of other rows, in place.
+// A query at position p sees keys (p - window, p] (window > 0) or [0, p]; a head may have a sink, a logit in its denominator.  Built without fast-math.
 #include <cstdlib>
 #include "common.cuh"
 #include "kernels.h"
@@ -29,26 +30,36 @@ template <> __device__ __forceinline__ float lat_from<float>(float v) { return v
 template <> __device__ __forceinline__ __nv_bfloat16 lat_from<__nv_bfloat16>(float v) { return f2bf(v); }
 
 // ------------------------------------------------------------------------------------ norm + rotation + append
-// proj row t: [H heads of (dim | rot)] queries, R latent values, rot shared key values.  One CTA per token.
+// Row t of q (null: not here): H heads of (dim | rot); of down (null: not here): R latent values, rot shared key values; of cq (null: none):
+// the queries' own latent.  q and cq may be column ranges of down's matrix that do not overlap it.  One CTA per token.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ proj, int ldp, OgbLatentShape sh, const float* __restrict__ norm_w, float eps,
+__global__ void __launch_bounds__(128) latent_prep_kernel(T* q_, int ldq, const T* down_, int ldd, T* cq_, int ldcq, int q_rank,
+                                                          const float* __restrict__ cq_w, OgbLatentShape sh, const float* __restrict__ norm_w, float eps,
                                                           const int32_t* __restrict__ positions, const float* __restrict__ cosc,
                                                           const float* __restrict__ sinc, int max_pos, const int32_t* __restrict__ slots,
                                                           T* __restrict__ cache, int ldcache) {
-  __shared__ float part[4];
+  __shared__ float part[8];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  T* row = proj + size_t(t) * ldp;
-  const T* down = row + sh.H * (sh.dim + sh.rot);
-  const int pos = min(max(positions[t], 0), max_pos - 1), slot = slots[t];
+  const T* down = down_ ? down_ + size_t(t) * ldd : nullptr;
+  T* cq = cq_ ? cq_ + size_t(t) * ldcq : nullptr;
+  const int pos = min(max(positions[t], 0), max_pos - 1), slot = down ? slots[t] : -1;
   const int half = sh.rot_dims / 2;
   const float *cs = cosc + size_t(pos) * half, *sn = sinc + size_t(pos) * half;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < sh.R; i += 128) { const float v = lat_f32(down[i]); ss += v * v; }
+  float ss = 0.f, sq = 0.f;
+  if (down)
+    for (int i = threadIdx.x; i < sh.R; i += 128) { const float v = lat_f32(down[i]); ss += v * v; }
+  if (cq)
+    for (int i = threadIdx.x; i < q_rank; i += 128) { const float v = lat_f32(cq[i]); sq += v * v; }
   ss = warp_sum(ss);
-  if (lane == 0) part[warp] = ss;
+  sq = warp_sum(sq);
+  if (lane == 0) { part[warp] = ss; part[4 + warp] = sq; }
   __syncthreads();
+  if (cq) {
+    const float inv = 1.f / sqrtf((part[4] + part[5] + part[6] + part[7]) / q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += 128) cq[i] = lat_from<T>(lat_f32(cq[i]) * inv * cq_w[i]);
+  }
   if (slot >= 0) {
     const float inv = 1.f / sqrtf((part[0] + part[1] + part[2] + part[3]) / sh.R + eps);
     T* dst = cache + size_t(slot) * ldcache;
@@ -60,9 +71,10 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ proj, 
       dst[sh.R + i] = lat_from<T>(v);
     }
   }
+  if (!q_) return;
   for (int idx = threadIdx.x; idx < sh.H * half; idx += 128) {
     const int h = idx / half, i = idx - h * half;
-    T* q = row + h * (sh.dim + sh.rot) + sh.dim;
+    T* q = q_ + size_t(t) * ldq + h * (sh.dim + sh.rot) + sh.dim;
     const float u = lat_f32(q[i]), v = lat_f32(q[i + half]);
     q[i] = lat_from<T>(u * cs[i] - v * sn[i]);
     q[i + half] = lat_from<T>(v * cs[i] + u * sn[i]);
@@ -84,6 +96,7 @@ struct LatentParams {
   const int32_t *cu, *past, *table; int table_cols, block_size, block_shift;      // log2(block_size) or -1
   __nv_bfloat16* out;             // [T, H, R]
   float* part_o; float* part_ml;
+  const float* sinks;             // [H] a logit in each head's denominator, or null
   float scale;
   int window, B, H, R, rot, kp, pitch, splits, total_rows, skip_q_len;
   const int32_t* order;           // [B] requests in issue order (longest first), or null
@@ -361,7 +374,11 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
           pm[0] = sM[r]; pm[1] = lr;
         }
       } else {
-        const float inv = lr > 0.f ? 1.f / lr : 0.f;
+        float inv = lr > 0.f ? 1.f / lr : 0.f;
+        if (p.sinks) {
+          const float sk = p.sinks[(row0 + r) % H] * LAT_LOG2E, top = fmaxf(sM[r], sk), old = exp2f(sM[r] - top);
+          inv = old / (lr * old + exp2f(sk - top));
+        }
         __nv_bfloat16* po = p.out + orow * p.R;
 #pragma unroll
         for (int n = 0; n < NTW; ++n)
@@ -372,7 +389,8 @@ __global__ void __launch_bounds__(LAT_THREADS, MT == 4 ? 1 : 2) latent_mma_kerne
 
 // One CTA per (token, head) row: merges the split partials.
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                             __nv_bfloat16* __restrict__ out, int total_rows, int R, int splits) {
+                                                             __nv_bfloat16* __restrict__ out, int total_rows, int R, int splits,
+                                                             const float* __restrict__ sinks, int H) {
   __shared__ float w[LAT_MAX_SPLITS];
   pdl_launch_dependents();
   pdl_wait();
@@ -380,9 +398,10 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   if (threadIdx.x < 32) {
     float2 ml = make_float2(-INFINITY, 0.f);
     if (lane < splits) ml = *reinterpret_cast<const float2*>(part_ml + (size_t(lane) * total_rows + row) * 2);
-    const float M = warp_max(ml.x);
+    const float sk = sinks ? sinks[row % H] * LAT_LOG2E : -INFINITY;
+    const float M = fmaxf(warp_max(ml.x), sk);
     const float e = ml.x == -INFINITY ? 0.f : exp2f(ml.x - M);
-    const float L = warp_sum(e * ml.y);
+    const float L = warp_sum(e * ml.y) + (sinks ? exp2f(sk - M) : 0.f);
     w[lane] = L > 0.f ? e / L : 0.f;
   }
   __syncthreads();
@@ -404,7 +423,8 @@ template <typename T>
 __global__ void __launch_bounds__(128) latent_simt_kernel(const T* __restrict__ qlat, const T* __restrict__ proj, int ldp, OgbLatentShape sh,
                                                           const T* __restrict__ cache, int ldcache, const int32_t* __restrict__ cu,
                                                           const int32_t* __restrict__ past_lens, const int32_t* __restrict__ tables, int table_cols,
-                                                          int block_size, T* __restrict__ out, float scale, int window, int B, int skip_q_len) {
+                                                          int block_size, T* __restrict__ out, float scale, int window, const float* __restrict__ sinks, int B,
+                                                          int skip_q_len) {
   extern __shared__ float sq[];                        // [R + rot] query, then 32 scores
   float* ssc = sq + sh.R + sh.rot;
   pdl_launch_dependents();
@@ -425,7 +445,8 @@ __global__ void __launch_bounds__(128) latent_simt_kernel(const T* __restrict__ 
   float acc[LAT_SIMT_COLS];
 #pragma unroll
   for (int c = 0; c < LAT_SIMT_COLS; ++c) acc[c] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  // the sink takes part in the maximum and the sum from the start
+  float m = sinks ? sinks[h] : -INFINITY, l = sinks ? 1.f : 0.f;
   auto row_of = [&](int j) { return cache + (size_t(table[j / block_size]) * block_size + j % block_size) * ldcache; };
   for (int j0 = lo; j0 <= pos; j0 += 32) {
     __syncthreads();
@@ -466,6 +487,18 @@ __global__ void __launch_bounds__(128) latent_simt_kernel(const T* __restrict__ 
   }
 }
 
+// ------------------------------------------------------------------------------------ gate
+template <typename T>
+__global__ void gate_rows_kernel(T* __restrict__ out, int ldo, const T* __restrict__ gate, int ldg, int T_, int n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long all = long(T_) * n;
+  for (long i = long(blockIdx.x) * blockDim.x + threadIdx.x; i < all; i += long(gridDim.x) * blockDim.x) {
+    const long t = i / n, c = i % n;
+    out[t * ldo + c] = lat_from<T>(lat_f32(out[t * ldo + c]) / (1.f + expf(-lat_f32(gate[t * ldg + c]))));
+  }
+}
+
 // ------------------------------------------------------------------------------------ gather
 // Dense row i holds cached position first_kv[k] + i - row_base[k] of request req[k], k the last with row_base[k] <= i; rows past
 // kv_len[k] are zeros (a request's rows are padded to a multiple of 16).
@@ -496,7 +529,7 @@ static int LaunchLatentMma(const LatentParams& p, int max_q_len, cudaStream_t s)
   const dim3 grid((max_q_len * p.H + MT * 16 - 1) / (MT * 16), 1, p.B * p.splits);
   if (!launch_pdl(kern, grid, dim3(LAT_THREADS), LatCfg<MT>::smem(p.pitch), s, p)) return -4;
   if (p.splits > 1 && !launch_pdl(latent_combine_kernel, dim3(p.total_rows), dim3(128), 0, s, static_cast<const float*>(p.part_o),
-                                  static_cast<const float*>(p.part_ml), p.out, p.total_rows, p.R, p.splits))
+                                  static_cast<const float*>(p.part_ml), p.out, p.total_rows, p.R, p.splits, p.sinks, p.H))
     return -4;
   return 0;
 }
@@ -513,17 +546,29 @@ static int lat_pitch(const OgbLatentShape* sh) { return (sh->R + sh->rot + 15) /
 
 using namespace ogb;
 
-OGB_API int ogb_latent_prep(void* proj, int ldp, const OgbLatentShape* sh, const float* norm_w, float eps, const int32_t* positions, const float* cos,
-                            const float* sin, int max_pos, const int32_t* slots, void* cache, int ldcache, int T, int fp32, void* stream) {
+OGB_API int ogb_latent_prep(void* q, int ldq, const void* down, int ldd, void* cq, int ldcq, int q_rank, const float* cq_w, const OgbLatentShape* sh,
+                            const float* norm_w, float eps, const int32_t* positions, const float* cos, const float* sin, int max_pos,
+                            const int32_t* slots, void* cache, int ldcache, int T, int fp32, void* stream) {
   if (T <= 0) return 0;
   if (sh->rot_dims < 0 || sh->rot_dims > sh->rot || (sh->rot_dims & 1) || (sh->rot_dims > 0 && (!cos || !sin || max_pos <= 0))) return -1;
-  if (sh->R + sh->rot > ldcache) return -1;
+  if ((down && sh->R + sh->rot > ldcache) || (cq && (q_rank <= 0 || !cq_w))) return -1;
   auto s = static_cast<cudaStream_t>(stream);
+#define OGB_LAT_PREP(TY) launch_pdl(latent_prep_kernel<TY>, dim3(T), dim3(128), 0, s, static_cast<TY*>(q), ldq, static_cast<const TY*>(down), ldd, \
+                                    static_cast<TY*>(cq), ldcq, q_rank, cq_w, *sh, norm_w, eps, positions, cos, sin, max_pos, slots, \
+                                    static_cast<TY*>(cache), ldcache)
+  const bool ok = fp32 ? OGB_LAT_PREP(float) : OGB_LAT_PREP(__nv_bfloat16);
+#undef OGB_LAT_PREP
+  return ok ? 0 : -4;
+}
+
+OGB_API int ogb_gate_rows(void* out, int ldo, const void* gate, int ldg, int T, int n, int fp32, void* stream) {
+  if (T <= 0 || n <= 0) return 0;
+  auto s = static_cast<cudaStream_t>(stream);
+  const long nb = (long(T) * n + 255) / 256;
+  const dim3 grid(unsigned(nb < 148 * 16 ? nb : 148 * 16));
   using Hf = __nv_bfloat16;
-  return (fp32 ? launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), 0, s, static_cast<float*>(proj), ldp, *sh, norm_w, eps, positions, cos, sin,
-                            max_pos, slots, static_cast<float*>(cache), ldcache)
-               : launch_pdl(latent_prep_kernel<Hf>, dim3(T), dim3(128), 0, s, static_cast<Hf*>(proj), ldp, *sh, norm_w, eps, positions, cos, sin, max_pos,
-                            slots, static_cast<Hf*>(cache), ldcache)) ? 0 : -4;
+  return (fp32 ? launch_pdl(gate_rows_kernel<float>, grid, dim3(256), 0, s, static_cast<float*>(out), ldo, static_cast<const float*>(gate), ldg, T, n)
+               : launch_pdl(gate_rows_kernel<Hf>, grid, dim3(256), 0, s, static_cast<Hf*>(out), ldo, static_cast<const Hf*>(gate), ldg, T, n)) ? 0 : -4;
 }
 
 // 1 when the warp-MMA kernel can address these sizes (16-byte pieces everywhere, the tile fits in shared memory).
@@ -544,8 +589,8 @@ OGB_API long long ogb_latent_scratch_bytes(int total_rows, int R, int splits) {
 // bf16.  skip_q_len > 0: requests with at least that many tokens are left to another kernel (their rows of `out` are unspecified).
 OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                                  const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
-                                 void* out, float scale, int window, int B, int T, int max_q_len, int skip_q_len, int splits, void* scratch,
-                                 long long scratch_bytes, const int32_t* order, int* status, void* stream) {
+                                 void* out, float scale, int window, const float* sinks, int B, int T, int max_q_len, int skip_q_len, int splits,
+                                 void* scratch, long long scratch_bytes, const int32_t* order, int* status, void* stream) {
   if (B <= 0 || T <= 0 || max_q_len <= 0) return 0;
   if (!ogb_latent_mma_supported(sh)) return -5;
   if ((ldp % 8) || (ldcache % 8) || block_size <= 0) return -1;
@@ -562,7 +607,7 @@ OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, co
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = static_cast<float*>(scratch);
   p.part_ml = p.part_o ? p.part_o + size_t(splits) * rows * sh->R : nullptr;
-  p.scale = scale; p.window = window; p.B = B; p.H = sh->H; p.R = sh->R; p.rot = sh->rot;
+  p.sinks = sinks; p.scale = scale; p.window = window; p.B = B; p.H = sh->H; p.R = sh->R; p.rot = sh->rot;
   p.kp = (sh->R + sh->rot + 15) / 16 * 16; p.pitch = lat_pitch(sh);
   p.splits = splits; p.total_rows = rows; p.skip_q_len = skip_q_len; p.order = order; p.status = status;
   auto s = static_cast<cudaStream_t>(stream);
@@ -578,7 +623,7 @@ OGB_API int ogb_latent_attention(const void* qlat, const void* proj, int ldp, co
 
 OGB_API int ogb_latent_attention_simt(const void* qlat, const void* proj, int ldp, const OgbLatentShape* sh, const void* cache, int ldcache,
                                       const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size,
-                                      void* out, float scale, int window, int B, int T, int skip_q_len, int fp32, void* stream) {
+                                      void* out, float scale, int window, const float* sinks, int B, int T, int skip_q_len, int fp32, void* stream) {
   if (B <= 0 || T <= 0) return 0;
   if (sh->R > 128 * LAT_SIMT_COLS || sh->H > 65535 || block_size <= 0) return -5;
   const int smem = (sh->R + sh->rot + 32) * 4;
@@ -587,10 +632,10 @@ OGB_API int ogb_latent_attention_simt(const void* qlat, const void* proj, int ld
   using Hf = __nv_bfloat16;
   return (fp32 ? launch_pdl(latent_simt_kernel<float>, dim3(T, sh->H), dim3(128), smem, s, static_cast<const float*>(qlat), static_cast<const float*>(proj),
                             ldp, *sh, static_cast<const float*>(cache), ldcache, cu_seqlens, past_lens, block_table, table_cols, block_size,
-                            static_cast<float*>(out), scale, window, B, skip_q_len)
+                            static_cast<float*>(out), scale, window, sinks, B, skip_q_len)
                : launch_pdl(latent_simt_kernel<Hf>, dim3(T, sh->H), dim3(128), smem, s, static_cast<const Hf*>(qlat), static_cast<const Hf*>(proj), ldp, *sh,
                             static_cast<const Hf*>(cache), ldcache, cu_seqlens, past_lens, block_table, table_cols, block_size, static_cast<Hf*>(out), scale,
-                            window, B, skip_q_len)) ? 0 : -4;
+                            window, sinks, B, skip_q_len)) ? 0 : -4;
 }
 
 // width, ldcache, ldo in bf16 elements, multiples of 8

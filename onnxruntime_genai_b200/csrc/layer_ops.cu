@@ -1,5 +1,6 @@
 // Per-token kernels of the models that keep their residual stream in fp32, for bf16 and fp32 activations and any width:
-//   embedding rows into the fp32 stream; RMS / layer norm of stream rows (optionally of selected rows only: the rows whose logits
+//   embedding rows into the fp32 stream, alone or with a row hashed from the previous token and this one; sums into the stream with a tanh norm
+//   of the result; RMS / layer norm of stream rows (optionally of selected rows only: the rows whose logits
 //   are wanted); the norm of a sub-layer's output added to the stream (with the weighted sum of routed experts folded in); head norms,
 //   rotation and cache append of attention projections; the gated activation act(gate) * up between two strided matrices and the experts'
 //   form of it; the causal depthwise convolution over the paged window of earlier inputs.  Built without fast-math: the fp32 models are the exact form of the same code.
@@ -28,6 +29,37 @@ __global__ void embedding_stream_kernel(const int32_t* __restrict__ ids, const T
     out[size_t(t) * H + i] = v;
     if (copy) copy[size_t(t) * H + i] = f2bf(v);
   }
+}
+
+// ------------------------------------------------------------------------------------ embedding with hashed pairs
+// One CTA per token (see OgbBigram).
+template <typename T>
+__global__ void embedding_bigram_kernel(OgbBigram p, const T* __restrict__ table, const T* __restrict__ bigram, float* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  int lo = 0, hi = p.B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (p.cu_seqlens[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  const int t0 = p.cu_seqlens[lo], before = p.past_lens[lo] + t - t0, id = p.ids[t];
+  long long row = p.buckets;
+  if (before > 0) {
+    int prev = 0;
+    if (t > t0) {
+      prev = p.ids[t - 1];
+    } else {
+      const int q = before - 1, block = p.block_table[size_t(lo) * p.table_cols + q / p.block_size];
+      if (block >= 0) prev = p.tokens[size_t(block) * p.block_size + q % p.block_size];
+    }
+    row = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
+    if (row < 0) row += p.buckets;
+  }
+  if (threadIdx.x == 0 && p.slots[t] >= 0) p.tokens[p.slots[t]] = id;
+  const T* a = table + size_t(min(max(id, 0), p.vocab - 1)) * p.H;
+  const T* b = bigram + size_t(row) * p.H;
+  for (int i = threadIdx.x; i < p.H; i += blockDim.x) out[size_t(t) * p.H + i] = fmaf(to_f32(a[i]), p.scale, to_f32(b[i]));
 }
 
 // ------------------------------------------------------------------------------------ norm of the fp32 stream
@@ -200,11 +232,67 @@ __global__ void __launch_bounds__(256) add_normed_kernel(const T* __restrict__ y
   }
 }
 
+// ------------------------------------------------------------------------------------ sums into the stream, tanh norm of the result
+// (See OgbTanhNorm.)  Every column is on its own: blockIdx.y walks pieces of a row, VEC columns per thread.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) add_tanh_norm_kernel(OgbTanhNorm p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = p.rows ? p.rows[blockIdx.x] : blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+  if (i >= p.H) return;
+  auto load = [&](const auto* src, float (&v)[VEC]) {
+    if constexpr (VEC == 8) load8(src, v); else v[0] = to_f32(*src);
+  };
+  const size_t at = size_t(t) * p.H + i;
+  float n[VEC], u[VEC];
+  load(p.h_in + at, n);
+  auto add = [&](float w) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) n[e] = fmaf(w, u[e], n[e]);
+  };
+  const T* y = static_cast<const T*>(p.y);
+  if (p.inv_pos) {
+    for (int j = 0; j < p.k; ++j) {
+      const int r = p.inv_pos[size_t(t) * p.k + j];
+      if (r < 0) continue;
+      load(y + size_t(r) * p.ldy + i, u);
+      add(p.topk_w[size_t(t) * p.k + j]);
+    }
+  } else if (y) {
+    load(y + size_t(t) * p.ldy + i, u);
+    add(1.f);
+  }
+  if (p.y2) { load(static_cast<const T*>(p.y2) + size_t(t) * p.ldy2 + i, u); add(1.f); }
+  if (p.first) { load(p.first + at, u); add(1.f); }
+  if (p.step) { load(p.step + i, u); add(1.f); }
+  float w[VEC], b[VEC];
+  load(p.w + i, w);
+  load(p.b + i, b);
+  if constexpr (VEC == 8) {
+    if (p.h_out) {
+      reinterpret_cast<float4*>(p.h_out + at)[0] = make_float4(n[0], n[1], n[2], n[3]);
+      reinterpret_cast<float4*>(p.h_out + at)[1] = make_float4(n[4], n[5], n[6], n[7]);
+    }
+  } else {
+    if (p.h_out) p.h_out[at] = n[0];
+  }
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) n[e] = fmaf(tanhf(p.alpha * n[e]), w[e], b[e]);
+  T* dst = static_cast<T*>(p.x) + size_t(blockIdx.x) * p.H + i;
+  if constexpr (VEC == 1) dst[0] = from_f32<T>(n[0]);
+  else if constexpr (sizeof(T) == 4) {
+    reinterpret_cast<float4*>(dst)[0] = make_float4(n[0], n[1], n[2], n[3]);
+    reinterpret_cast<float4*>(dst)[1] = make_float4(n[4], n[5], n[6], n[7]);
+  } else {
+    *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(n[0], n[1]), pack_bf16x2(n[2], n[3]), pack_bf16x2(n[4], n[5]), pack_bf16x2(n[6], n[7]));
+  }
+}
+
 // ------------------------------------------------------------------------------------ head norms, rotation, cache append
 // One warp per (token, head).  Query heads are replaced in place; key heads go to the token's cache row; value heads are copied there.
 // A lane handles pairs of columns (i, i + rot / 2) of the rotated part and single columns of the rest, V at a time.
 struct QkvPrep {
-  int ldp, Hq, Hkv, dim, key_row, value_row, rot, max_pos, T;
+  int ldp, Hq, Hkv, Hv, dim, key_row, value_row, rot, max_pos, T;
   const float *q_norm, *k_norm, *cos, *sin;
   const int32_t *positions, *slots;
   float eps;
@@ -226,7 +314,7 @@ template <typename T, int V>
 __global__ void __launch_bounds__(256) qkv_prep_kernel(T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int per = p.Hq + 2 * p.Hkv;
+  const int per = p.Hq + p.Hkv + p.Hv;
   const long item = long(blockIdx.x) * 8 + (threadIdx.x >> 5);
   if (item >= long(p.T) * per) return;
   const int t = int(item / per), head = int(item % per), lane = threadIdx.x & 31;
@@ -236,7 +324,7 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(T* __restrict__ proj, T* 
     const int g = head - p.Hq - p.Hkv;
     if (slot < 0) return;
     const T* src = row + size_t(p.Hq + p.Hkv) * p.key_row + size_t(g) * p.value_row;
-    T* dst = v_cache + (size_t(slot) * p.Hkv + g) * p.value_row;
+    T* dst = v_cache + (size_t(slot) * p.Hv + g) * p.value_row;
     for (int i = lane * V; i < p.value_row; i += 32 * V) {
       float f[V];
       ld_cols<T, V>(src + i, f);
@@ -376,6 +464,34 @@ OGB_API int ogb_embedding_stream(const int32_t* ids, const void* table, int tabl
   return ok ? 0 : -4;
 }
 
+OGB_API int ogb_embedding_bigram(const OgbBigram* p, const void* table, const void* bigram, float* out, void* stream) {
+  if (p->T <= 0) return 0;
+  if (p->B <= 0 || p->H <= 0 || p->vocab <= 0 || p->buckets <= 0 || p->block_size <= 0) return -1;
+  auto s = static_cast<cudaStream_t>(stream);
+  const dim3 block(p->H >= 256 ? 256 : 64);
+  const bool ok = p->fp32 ? launch_pdl(embedding_bigram_kernel<float>, dim3(p->T), block, 0, s, *p, static_cast<const float*>(table),
+                                       static_cast<const float*>(bigram), out)
+                          : launch_pdl(embedding_bigram_kernel<__nv_bfloat16>, dim3(p->T), block, 0, s, *p, static_cast<const __nv_bfloat16*>(table),
+                                       static_cast<const __nv_bfloat16*>(bigram), out);
+  return ok ? 0 : -4;
+}
+
+OGB_API int ogb_add_tanh_norm(const OgbTanhNorm* p, void* stream) {
+  if (p->n_rows <= 0 || p->H <= 0) return 0;
+  if (!p->h_in || !p->w || !p->b || !p->x || (p->inv_pos && (!p->y || !p->topk_w))) return -1;
+  auto s = static_cast<cudaStream_t>(stream);
+  auto addr = [](const void* a) { return reinterpret_cast<uintptr_t>(a); };
+  const bool vec = p->H % 8 == 0 && (!p->y || p->ldy % 8 == 0) && (!p->y2 || p->ldy2 % 8 == 0) &&
+                   ((addr(p->h_in) | addr(p->h_out) | addr(p->y) | addr(p->y2) | addr(p->first) | addr(p->step) | addr(p->w) | addr(p->b) | addr(p->x)) & 15) == 0;
+  const int pieces = vec ? p->H / 8 : p->H;
+  const dim3 block(pieces < 128 ? (pieces + 31) / 32 * 32 : 128), grid(p->n_rows, (pieces + block.x - 1) / block.x);
+  if (grid.y > 65535) return -1;
+  const bool ok = p->fp32 ? (vec ? launch_pdl(add_tanh_norm_kernel<float, 8>, grid, block, 0, s, *p) : launch_pdl(add_tanh_norm_kernel<float, 1>, grid, block, 0, s, *p))
+                          : (vec ? launch_pdl(add_tanh_norm_kernel<__nv_bfloat16, 8>, grid, block, 0, s, *p)
+                                 : launch_pdl(add_tanh_norm_kernel<__nv_bfloat16, 1>, grid, block, 0, s, *p));
+  return ok ? 0 : -4;
+}
+
 // rows (may be null): out row i is the norm of x row rows[i].  w, b fp32 [H] (b may be null).
 OGB_API int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const float* b, void* out, int out_fp32, int n_rows, int H, float eps,
                             int layernorm, void* stream) {
@@ -437,13 +553,13 @@ OGB_API int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const f
   return ok ? 0 : -4;
 }
 
-OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
+OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
                          const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
                          void* v_cache, int T, int fp32, void* stream) {
   if (T <= 0) return 0;
-  if (Hq <= 0 || Hkv <= 0 || dim <= 0 || dim > key_row || rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (!cos || !sin || max_pos <= 0))) return -1;
-  const QkvPrep p{ldp, Hq, Hkv, dim, key_row, value_row, rot, max_pos > 0 ? max_pos : 1, T, q_norm, k_norm, cos, sin, positions, slots, eps};
-  const long items = long(T) * (Hq + 2 * Hkv);
+  if (Hq <= 0 || Hkv <= 0 || Hv <= 0 || dim <= 0 || dim > key_row || rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (!cos || !sin || max_pos <= 0))) return -1;
+  const QkvPrep p{ldp, Hq, Hkv, Hv, dim, key_row, value_row, rot, max_pos > 0 ? max_pos : 1, T, q_norm, k_norm, cos, sin, positions, slots, eps};
+  const long items = long(T) * (Hq + Hkv + Hv);
   const dim3 grid(unsigned((items + 7) / 8));
   auto s = static_cast<cudaStream_t>(stream);
   const int elem = fp32 ? 4 : 2;

@@ -18,8 +18,9 @@
 namespace ogb {
 
 // One warp per token.  mode 0: softmax over the k selected logits; mode 1: softmax over all experts, the
-// selected probabilities unchanged; mode 2: softmax over all experts, renormalised over the selected.
-__global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, int mode, int* __restrict__ topk_idx,
+// selected probabilities unchanged; mode 2: softmax over all experts, renormalised over the selected.  shared: every token also gets expert E
+// with weight 1 (rows of k + 1 entries).
+__global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, int mode, int shared, int* __restrict__ topk_idx,
                                 float* __restrict__ topk_w) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= T) return;
@@ -61,9 +62,10 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T,
     const float pr = lane < k ? expf(my_val - all_max) / all_sum : 0.f;
     w = mode == 2 ? pr / warp_sum(pr) : pr;
   }
-  if (lane < k) {
-    topk_idx[size_t(warp) * k + lane] = my_idx;
-    topk_w[size_t(warp) * k + lane] = w;
+  const int per = k + shared;
+  if (lane < per) {
+    topk_idx[size_t(warp) * per + lane] = lane < k ? my_idx : E;
+    topk_w[size_t(warp) * per + lane] = lane < k ? w : 1.f;
   }
 }
 
@@ -152,12 +154,13 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, int ldy,
 
 using namespace ogb;
 
-OGB_API int ogb_moe_topk(const float* logits, int ld, int T, int E, int k, int mode, int32_t* topk_idx, float* topk_w, void* stream) {
+OGB_API int ogb_moe_topk(const float* logits, int ld, int T, int E, int k, int mode, int shared, int32_t* topk_idx, float* topk_w, void* stream) {
   if (T <= 0) return 0;
-  if (E <= 0 || E > 1024 || k <= 0 || k > 32 || k > E || mode < 0 || mode > 2) return -1;
+  shared = shared ? 1 : 0;
+  if (E <= 0 || E > 1024 || k <= 0 || k + shared > 32 || k > E || mode < 0 || mode > 2) return -1;
   const int threads = 128, warps_per_block = threads / 32;
   moe_topk_kernel<<<(T + warps_per_block - 1) / warps_per_block, threads, 0, static_cast<cudaStream_t>(stream)>>>(
-      logits, ld, T, E, k, mode, topk_idx, topk_w);
+      logits, ld, T, E, k, mode, shared, topk_idx, topk_w);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -8,7 +8,7 @@ is a set of flag values, not a class.
 from __future__ import annotations
 
 import math
-from dataclasses import asdict, dataclass, field
+from dataclasses import asdict, dataclass, field, replace
 from typing import Any, Dict, List, Optional
 
 import numpy as np
@@ -17,7 +17,7 @@ LLM_TYPES = [
     "chatglm", "decoder", "ernie4_5", "gemma", "gemma2", "gemma3_text", "gptoss", "gpt_oss", "granite", "hunyuan", "hunyuandensev1", "hunyuan_v1_dense",
     "internlm2", "llama", "mistral", "nemotron", "olmo", "olmo2", "exaone4", "phi", "phi3", "phimoe", "qwen2", "qwen3",
     "smollm3", "lfm2", "gpt2", "helium", "mixtral", "qwen2_moe", "qwen3_moe", "granitemoe", "olmoe", "qwen2_vl", "qwen2_5_vl", "qwen3_vl",
-    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar", "zevopel",      # hybrids of gated-delta-net (linear attention) and full-attention layers
+    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar", "zevopel", "sugelix",      # hybrids of gated-delta-net (linear attention) and full-attention layers
 ]
 
 
@@ -29,12 +29,13 @@ ALM_TYPES = ["whisper"]
 
 @dataclass
 class RotarySpec:
-    """Rotary positions of one layer: the first `dims` entries of a vector turn in pairs (i, i + dims / 2) with the frequencies
-    base^(-2 i / dims); scaling: None, the YaRN parameters {factor, original, fast, slow}, or {factor, original, low, high}: slowed down
-    by wavelength (Llama 3.1, see `wavelength_frequencies`)."""
+    """Rotary positions of one layer: the first `dims` entries of a vector turn in pairs (i, i + dims / 2) (neighbours: in pairs
+    (2 i, 2 i + 1)) with the frequencies base^(-2 i / dims); scaling: None, {factor}: every frequency divided by it, the YaRN parameters
+    {factor, original, fast, slow}, or {factor, original, low, high}: slowed down by wavelength (Llama 3.1, see `wavelength_frequencies`)."""
     dims: int
     base: float
     scaling: Optional[Dict[str, float]] = None
+    neighbours: bool = False
 
     def key(self):
         return (self.dims, self.base, tuple(sorted((self.scaling or {}).items())))
@@ -44,7 +45,8 @@ class RotarySpec:
 class MoeSpec:
     """Routed experts of a layer: `top` of `experts` feed-forwards run per token.  act: "silu" silu(gate) * up, or "clamped"
     g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).  weights: softmax over the "selected" router
-    logits, over "all" of them, or over all and "renormed" over the selected; "sparse_mixer": PhiMoE's margin rule."""
+    logits, over "all" of them, or over all and "renormed" over the selected; "sparse_mixer": PhiMoE's margin rule.  shared_ff > 0: one more
+    expert of that width (with its own limit) runs for every token and is added with weight 1."""
     experts: int
     top: int
     act: str = "silu"
@@ -52,6 +54,8 @@ class MoeSpec:
     limit: float = 0.0
     weights: str = "all"
     jitter_eps: float = 0.01
+    shared_ff: int = 0
+    shared_limit: float = 0.0
 
 
 @dataclass
@@ -61,9 +65,16 @@ class LayerSpec:
                           chunk > 0: position p sees the keys of its own run of `chunk` positions (counted from position 0), 0: every
                           earlier one; qk_norm: RMS norm of every query and key head before the rotation; sinks: a learned logit per head
                           in the softmax's denominator; head_gate: a head's output times sigmoid of a projection of the mixer's input;
+                          window > 0: position p sees the keys in (p - window, p]; softcap > 0: a score s becomes
+                          softcap * tanh(s / softcap); qkv_bias: biases on the three projections; maps = 2 (differential attention):
+                          queries and keys hold two vectors of `dim` per head, each pair attends over the same values, and a head's result
+                          is the RMS-normed difference a1 - lambda * a2 times (1 - diff), lambda learned around `diff`;
       "linear_attention"  gated delta rule: `kv_heads` query / key heads of `dim`, `heads` value heads of `vdim`, convolution of `conv` taps;
       "latent_attention"  `heads` heads of `dim` unrotated + `rot_dim` rotated query / key dimensions and `vdim` value dimensions over a
-                          latent of `kv_rank` values per token; window 0: every earlier token is visible."""
+                          latent of `kv_rank` values per token; window 0: every earlier token is visible; q_rank > 0: the queries come
+                          out of an RMS-normed latent of their own; sinks as above.
+    out_gate (the attending kinds): the concatenated heads are multiplied element by element with the sigmoid of a projection of the mixer's
+    input.  A layer that runs several times is several entries: `weights_of` names the first run, every run has a cache of its own."""
     kind: str
     heads: int
     dim: int
@@ -78,10 +89,18 @@ class LayerSpec:
     qk_norm: bool = False
     sinks: bool = False
     head_gate: bool = False
+    out_gate: bool = False
+    qkv_bias: bool = False
+    softcap: float = 0.0
+    maps: int = 1
+    diff: float = 0.0
+    q_rank: int = 0
     rotary: Optional[RotarySpec] = None
     ff: int = 0                       # width of the gated feed-forward, of one expert where there are experts (0: the layer has none)
     moe: Optional[MoeSpec] = None
     weights_of: Optional[int] = None  # layer whose weights this one uses (cache and state are its own)
+    source: Optional[int] = None      # the layer's number in the checkpoint where that is not its place in the run
+    opens_pass: Optional[int] = None  # the layer is the first of this pass through a group of layers that runs several times
 
     @property
     def conv_channels(self) -> int:
@@ -98,7 +117,12 @@ class LayerSpec:
 
     @property
     def key_row(self) -> int:
-        """Columns of one key (and query) head of an attention layer: whole 16-byte pieces of 16-bit values, zeros past `dim`."""
+        """Columns of one key head of an attention layer: per map whole 16-byte pieces of 16-bit values, zeros past `dim`."""
+        return self.maps * self.map_row
+
+    @property
+    def map_row(self) -> int:
+        """Columns of one query vector of an attention layer (a head has `maps` of them)."""
         return (self.dim + 7) // 8 * 8 if self.kind == "attention" else 0
 
     @property
@@ -166,6 +190,10 @@ class ArchConfig:
     # residual_multiplier.
     layer_specs: Optional[List[LayerSpec]] = None
     layer_scale: bool = False
+    tanh_norm: bool = False          # norms are tanh(alpha * x) * w + b (Dynamic Tanh: no statistics), alpha a learned scalar per norm
+    bigram: Optional[Dict[str, int]] = None   # {buckets, mul_prev, mul_cur}: rows hashed from (previous token, token) join the embedding
+    passes: int = 0                  # > 0: a group of layers runs that many times (entries of layer_specs with `opens_pass`); before each pass
+                                     # a learned vector joins the stream, before each but the first also the embedding output
     delta_l2_eps: float = 0.0        # gated delta rule: > 0 makes unit vectors x / sqrt(sum(x^2) + eps) instead of x / max(|x|, 1e-6)
     # Multimodal RoPE (Qwen2-VL): rotary pairs per position component (temporal, height, width); None: ordinary RoPE
     mrope_section: Optional[List[int]] = None
@@ -354,13 +382,21 @@ class ArchConfig:
 STACK_DESIGNS: Dict[str, Dict[str, Any]] = {
     # parallel blocks under one layer norm (weight and bias); gated delta rule and latent attention; ReLU-gated feed-forward
     "Luzatar": dict(arch=dict(model_type="luzatar", layernorm=True, parallel_block=True, activation="relu", delta_l2_eps=1e-6),
-                    mixers={"delta": "linear_attention", "latent_attention": "latent_attention"}, feed_forwards=("dense",)),
+                    mixers={"delta": dict(kind="linear_attention"), "latent_attention": dict(kind="latent_attention")}, feed_forwards=("dense",)),
     # sub-layers on the stream itself, RMS norms (stored around zero), layer scales and a residual multiplier on their outputs; chunked
     # attention with normed queries and keys, sinks and a gate per head; GELU-gated feed-forward or clamped experts weighted by their
     # probabilities among all experts
     "Zevopel": dict(arch=dict(model_type="zevopel", pre_norm=False, post_sublayer_norms=True, norm_offset=1.0, layer_scale=True, activation="gelu_tanh"),
-                    mixers={"attention": "attention"}, feed_forwards=("dense", "moe"), attention=dict(qk_norm=True, sinks=True, head_gate=True),
+                    mixers={"attention": dict(kind="attention", mask="chunk", qk_norm=True, sinks=True, head_gate=True)}, feed_forwards=("dense", "moe"),
                     moe=dict(act="clamped", alpha=1.702, weights="all")),
+    # pre-norm blocks under tanh norms, a hashed bigram embedding, a group of layers that runs several times; soft-capped attention (pairs of
+    # neighbours rotate), differential attention over a window, latent attention with compressed queries and sinks, all with gated outputs;
+    # clamped experts weighted among the selected, with a shared one
+    "Sugelix": dict(arch=dict(model_type="sugelix", tanh_norm=True),
+                    mixers={"attention": dict(kind="attention", qkv_bias=True, out_gate=True, neighbours=True),
+                            "attention_2": dict(kind="attention", qkv_bias=True, out_gate=True, maps=2),
+                            "latent_attention": dict(kind="latent_attention", sinks=True, out_gate=True)},
+                    feed_forwards=("moe",), moe=dict(act="clamped", alpha=1.702, weights="selected")),
 }
 
 
@@ -368,26 +404,27 @@ def is_stack_config(cfg: Dict[str, Any]) -> bool:
     return isinstance(cfg, dict) and cfg.get("architecture") in STACK_DESIGNS and isinstance(cfg.get("layers"), list)
 
 
-def _rotary_spec(i: int, rot: Optional[Dict[str, Any]], width: int) -> Optional[RotarySpec]:
+def _rotary_spec(i: int, rot: Optional[Dict[str, Any]], width: int, neighbours: bool = False) -> Optional[RotarySpec]:
     if not rot or not int(rot["dims"]):
         return None
     sc = rot.get("scaling")
-    spec = RotarySpec(int(rot["dims"]), float(rot["base"]), {k: float(v) for k, v in sc.items()} if sc else None)
+    spec = RotarySpec(int(rot["dims"]), float(rot["base"]), {k: float(v) for k, v in sc.items()} if sc else None, neighbours)
     if spec.dims > width or spec.dims % 2:
         raise ValueError(f"layer {i}: {spec.dims} rotary dimensions do not fit the {width} rotated ones")
     return spec
 
 
 def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec:
-    kind = design["mixers"].get(e.get("type"))
-    if kind is None:
+    if e.get("type") not in design["mixers"]:
         raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
+    fixed = dict(design["mixers"][e["type"]])          # what the design fixes about this mixer
+    kind, mask_kind, neighbours = fixed.pop("kind"), fixed.pop("mask", "window"), fixed.pop("neighbours", False)
     m, mlp = e["mixer"], e.get("mlp")
     ff_kind = mlp.get("kind", "dense") if mlp else None
     if mlp and ff_kind not in design["feed_forwards"]:
         raise ValueError(f"layer {i}: unknown feed-forward kind {ff_kind!r}")
     sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                   weights_of=None if e.get("weights_of") is None else int(e["weights_of"]))
+                   weights_of=None if e.get("weights_of") is None else int(e["weights_of"]), **fixed)
     if ff_kind == "dense":
         sp.ff = int(mlp["ff"])
     elif ff_kind == "moe":
@@ -395,6 +432,8 @@ def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec
         sp.moe = MoeSpec(int(mlp["router"]["experts"]), int(mlp["router"]["top"]), limit=float(mlp["expert"].get("limit") or 0.0), **design["moe"])
         if not 0 < sp.moe.top <= sp.moe.experts:
             raise ValueError(f"layer {i}: {sp.moe.top} of {sp.moe.experts} experts cannot be chosen")
+        if mlp.get("shared"):
+            sp.moe.shared_ff, sp.moe.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"].get("limit") or 0.0)
     if kind in ("linear_attention", "attention"):
         sp.kv_heads = int(m["kv_heads"])
         if sp.heads % sp.kv_heads:
@@ -403,14 +442,30 @@ def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec
     if kind == "linear_attention":
         sp.conv = int(m["conv"])
     elif kind == "attention":
-        sp.scale, sp.chunk = float(m["scale"]), mask
-        sp.rotary = _rotary_spec(i, m.get("rot"), sp.dim)
-        for k, v in design["attention"].items():
-            setattr(sp, k, v)
+        sp.scale, sp.softcap, sp.diff = float(m["scale"]), float(m.get("softcap") or 0.0), float(m.get("diff") or 0.0)
+        setattr(sp, mask_kind, mask)
+        sp.rotary = _rotary_spec(i, m.get("rot"), sp.dim, neighbours)
     else:
         sp.kv_rank, sp.rot_dim, sp.scale, sp.window = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"]), mask
-        sp.rotary = _rotary_spec(i, m.get("rot"), sp.rot_dim)
+        sp.q_rank = int(m.get("q_rank") or 0)
+        sp.rotary = _rotary_spec(i, m.get("rot"), sp.rot_dim, neighbours)
     return sp
+
+
+def _run_order(specs: List[LayerSpec], loop: Optional[Dict[str, Any]]) -> List[LayerSpec]:
+    """The layers in the order in which they run: layers start .. stop - 1 `times` times in a row, the runs after the first with the
+    weights of the first."""
+    if not loop:
+        return specs
+    a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not (0 <= a < b <= len(specs) and times >= 1):
+        raise ValueError(f"layers {a} .. {b} of {len(specs)} cannot run {times} times")
+    if any(sp.weights_of is not None for sp in specs):
+        raise ValueError("layers that use another layer's weights cannot stand beside a group that runs several times")
+    out = [replace(sp, source=i) for i, sp in enumerate(specs[:a])]
+    for t in range(times):
+        out += [replace(sp, source=a + i, weights_of=a + i if t else None, opens_pass=t if i == 0 else None) for i, sp in enumerate(specs[a:b])]
+    return out + [replace(sp, source=b + i) for i, sp in enumerate(specs[b:])]
 
 
 def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
@@ -421,16 +476,21 @@ def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
         if sp.weights_of is not None and not (0 <= sp.weights_of < len(specs) and specs[sp.weights_of].weights_of is None and
                                               specs[sp.weights_of].kind == sp.kind and sp.weights_of != i):
             raise ValueError(f"layer {i}: weights_of {sp.weights_of} does not name a layer of its kind with weights of its own")
+    loop = cfg.get("loop")
+    specs = _run_order(specs, loop)
+    emb = cfg.get("embedding") or {}
     att = [sp for sp in specs if sp.kind != "linear_attention"]
     # longest sequence the rotary scaling was made for, and at least 32768 positions (recurrent and windowed layers have no limit)
-    span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in att if sp.rotary and sp.rotary.scaling]
+    span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in att
+            if sp.rotary and sp.rotary.scaling and "original" in sp.rotary.scaling]
     eos = cfg.get("eos_token_id")
     return ArchConfig(vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]), num_layers=len(specs), num_heads=max(sp.heads for sp in specs),
                       num_kv_heads=max((sp.kv_heads for sp in specs if sp.kind == "attention"), default=1),
                       head_dim=max((sp.kv_rank + sp.rot_dim or sp.dim for sp in att), default=specs[0].dim),
                       intermediate_size=max(sp.ff for sp in specs), context_length=int(cfg.get("context_length") or max([32768] + span)),
                       norm_eps=float(cfg["norm"]["eps"]), layer_specs=specs, layer_types=[sp.kind for sp in specs], no_rope=not att,
-                      embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)), residual_multiplier=float(cfg.get("residual_mult", 1.0)),
+                      embed_scale=float(emb.get("scale", 1.0)), passes=int(loop["times"]) if loop else 0,
+                      bigram={k: int(emb["bigram"][k]) for k in ("buckets", "mul_prev", "mul_cur")} if emb.get("bigram") else None, residual_multiplier=float(cfg.get("residual_mult", 1.0)),
                       bos_token_id=int(cfg.get("bos_token_id", 0)), eos_token_id=-1 if eos is None else eos, pad_token_id=int(cfg.get("pad_token_id", 0)),
                       **design["arch"])
 
@@ -439,17 +499,26 @@ def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
     """Names and shapes of a declared stack's checkpoint tensors."""
     W = arch.hidden_size
     out: Dict[str, tuple] = {"embed": (arch.vocab_size, W), "final.norm": (W,), "head": (arch.vocab_size, W)}
-    if arch.layernorm:
+    if arch.layernorm or arch.tanh_norm:
         out["final.norm.b"] = (W,)
+    if arch.tanh_norm:
+        out["final.norm.alpha"] = ()
+    if arch.bigram:
+        out["bigram"] = (arch.bigram["buckets"] + 1, W)
+    if arch.passes:
+        out["loop.step"] = (arch.passes, W)
     for i, sp in enumerate(arch.layer_specs):
         if sp.weights_of is not None:
             continue
-        p, m = f"l{i}.", f"l{i}.mix."
+        p = f"l{i if sp.source is None else sp.source}."
+        m = p + "mix."
         # one norm for both sub-layers of a parallel block, else one for each
         for n in range(1, 2 if arch.parallel_block or not sp.ff else 3):
             out[f"{p}norm{n}"] = (W,)
-            if arch.layernorm:
+            if arch.layernorm or arch.tanh_norm:
                 out[f"{p}norm{n}.b"] = (W,)
+            if arch.tanh_norm:
+                out[f"{p}norm{n}.alpha"] = ()
             if arch.layer_scale:
                 out[f"{p}ls{n}"] = (W,)
         if sp.kind == "linear_attention":
@@ -459,8 +528,14 @@ def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
             out.update({m + "b": (sp.heads, W), m + "a": (sp.heads, W), m + "A_log": (sp.heads,), m + "dt_bias": (sp.heads,), m + "norm": (sp.vdim,),
                         m + "g": (vd, W), m + "o": (W, vd)})
         elif sp.kind == "attention":
-            out.update({m + "q": (sp.heads * sp.dim, W), m + "k": (sp.kv_heads * sp.dim, W), m + "v": (sp.kv_heads * sp.vdim, W),
-                        m + "o": (W, sp.heads * sp.vdim)})
+            sizes = dict(q=sp.heads * sp.maps * sp.dim, k=sp.kv_heads * sp.maps * sp.dim, v=sp.kv_heads * sp.vdim)
+            for n, c in sizes.items():
+                out[m + n] = (c, W)
+                if sp.qkv_bias:
+                    out[f"{m}{n}.b"] = (c,)
+            out[m + "o"] = (W, sp.heads * sp.vdim)
+            if sp.maps == 2:
+                out.update({m + n: (sp.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
             if sp.qk_norm:
                 out.update({m + "q.norm": (sp.dim,), m + "k.norm": (sp.dim,)})
             if sp.sinks:
@@ -468,11 +543,23 @@ def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
             if sp.head_gate:
                 out[m + "g"] = (sp.heads, W)
         else:
-            out.update({m + "q": (sp.heads * (sp.dim + sp.rot_dim), W), m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
+            rows = sp.heads * (sp.dim + sp.rot_dim)
+            if sp.q_rank:
+                out.update({m + "dq": (sp.q_rank, W), m + "dq.norm": (sp.q_rank,), m + "uq": (rows, sp.q_rank)})
+            else:
+                out[m + "q"] = (rows, W)
+            out.update({m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
                         m + "uk": (sp.heads * sp.dim, sp.kv_rank), m + "uv": (sp.heads * sp.vdim, sp.kv_rank), m + "o": (W, sp.heads * sp.vdim)})
+            if sp.sinks:
+                out[m + "sink"] = (sp.heads,)
+        if sp.out_gate:
+            out[m + "g"] = (sp.heads * sp.vdim, W)
         if sp.ff:
             if sp.moe is not None:
                 out[p + "mlp.router"] = (sp.moe.experts, W)
+                if sp.moe.shared_ff:
+                    f = sp.moe.shared_ff
+                    out.update({p + "mlp.shared.gate": (f, W), p + "mlp.shared.up": (f, W), p + "mlp.shared.down": (W, f)})
             for e in [""] if sp.moe is None else [f"e{k}." for k in range(sp.moe.experts)]:
                 out.update({f"{p}mlp.{e}gate": (sp.ff, W), f"{p}mlp.{e}up": (sp.ff, W), f"{p}mlp.{e}down": (W, sp.ff)})
     return out
@@ -767,6 +854,8 @@ def rotary_tables(spec: RotarySpec, n: int):
     if spec.scaling and "low" in spec.scaling:
         sc = spec.scaling
         inv_freq = wavelength_frequencies(inv_freq, sc["factor"], sc["original"], sc["low"], sc["high"])
+    elif spec.scaling and "original" not in spec.scaling:
+        inv_freq = inv_freq / spec.scaling["factor"]
     elif spec.scaling:
         sc = spec.scaling
         inv_freq = yarn_frequencies(inv_freq, spec.dims, spec.base, sc["factor"], sc["original"], sc["fast"], sc["slow"], spec.dims - 1)

@@ -89,6 +89,8 @@ class PagedKVCache:
                 sp = arch.layer_specs[i]
                 self.spec_kv[i] = tuple(torch.zeros(num_blocks * block_size, sp.kv_heads, n, dtype=dtype, device=device)
                                         for n in (sp.key_row, sp.value_row))
+        # Models whose embedding also reads the token before: the ids of the cached positions, in the same paged slots.
+        self.tokens = torch.zeros(num_blocks * block_size, dtype=torch.int32, device=device) if arch.bigram else None
         # layers without rows in the pools below
         conv = [c or i in self.latent_index or i in self.spec_kv for i, c in enumerate(conv)]
         self.windowed = [num_window_blocks > 0 and arch.layer_window(i) > 0 and not conv[i] for i in range(arch.num_layers)]
@@ -133,6 +135,8 @@ class PagedKVCache:
         for pools in self.spec_kv.values():
             for pool in pools:
                 pool[d_idx] = pool[s_idx]
+        if self.tokens is not None:
+            self.tokens[d_idx] = self.tokens[s_idx]
 
     def layer(self, i: int):
         if i in self.spec_kv:
@@ -176,7 +180,8 @@ class PagedKVCache:
         n_lat = sum(1 for i in range(arch.num_layers) if arch.is_latent_layer(i))
         own = [sp for i, sp in enumerate(arch.layer_specs or []) if arch.is_spec_attention(i)]
         own_row = sum(sp.kv_heads * (sp.key_row + sp.value_row) for sp in own)
-        return ((arch.num_layers - n_conv - n_lat - len(own)) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row + own_row) * es) * block_size
+        ids = 4 if arch.bigram else 0
+        return ((arch.num_layers - n_conv - n_lat - len(own)) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row + own_row) * es + ids) * block_size
 
 
 class CrossKVCache:
@@ -252,6 +257,16 @@ class LayerWeights:
     lat_uk_t: Optional[torch.Tensor] = None    # per head the transposed key map [heads * kv_rank, dim]: folds keys into the query
     lat_uv: Optional[torch.Tensor] = None      # value map [heads * vdim, kv_rank]
     lat_ukv: Optional[torch.Tensor] = None     # [key map; value map]: expands cached latents for long prompts
+    lat_down_col: int = 0                      # column of the latent in that projection
+    lat_gate_col: int = 0                      # column of the output gate's logits (of an attention layer: in its projection; 0: no gate)
+    lat_q_norm_w: Optional[torch.Tensor] = None  # queries with a latent of their own: RMS weight (fp32) and map to the heads (lat_in_w starts with the down map)
+    lat_uq_w: Optional[torch.Tensor] = None
+    diff_lambda: float = 0.0                   # differential attention: factor of the second map
+    norm1: Optional[ops.TanhNorm] = None       # tanh norms of the two sub-layers
+    norm2: Optional[ops.TanhNorm] = None
+    shared_gate_up_w: Optional[torch.Tensor] = None  # a shared expert beside the routed ones: rows alternate (gate, up)
+    shared_down_w: Optional[torch.Tensor] = None
+    exp_shared: bool = False                   # the shared expert is the last of the stacked experts
     rope_cos: Optional[torch.Tensor] = None    # rotary tables of this layer
     rope_sin: Optional[torch.Tensor] = None
     join_w: Optional[torch.Tensor] = None      # parallel blocks on an fp32 stream: [mixer output map | down] over [mixer output (padded) | feed-forward]
@@ -296,6 +311,9 @@ class DecoderModel:
         self.embed: Optional[torch.Tensor] = None
         self.final_norm_w: Optional[torch.Tensor] = None
         self.final_norm_b: Optional[torch.Tensor] = None
+        self.final_norm: Optional[ops.TanhNorm] = None
+        self.bigram: Optional[torch.Tensor] = None       # rows of the hashed (previous token, token) pairs
+        self.loop_step: Optional[torch.Tensor] = None    # [passes, width] fp32
         self.lm_head_w: Optional[torch.Tensor] = None
         self.lm_head_b: Optional[torch.Tensor] = None
         self.cos: Optional[torch.Tensor] = None
@@ -397,14 +415,15 @@ class DecoderModel:
         if sp is None:
             args, kw, cols = (block_size, self.heads_local, self.kv_heads_local, a.head_dim, a.scale, lw.window, lw.sinks, a.softcap), {}, a.head_dim
         else:
-            args, cols = (block_size, sp.heads, sp.kv_heads, sp.key_row, sp.scale, 0, lw.sinks, 0.0), sp.value_row
-            kw = dict(vdim=sp.value_row, chunk=sp.chunk, gate=gate)
+            args, cols = (block_size, sp.heads * sp.maps, sp.kv_heads, sp.key_row, sp.scale, sp.window, lw.sinks, sp.softcap), sp.value_row
+            kw = dict(vdim=sp.value_row, chunk=sp.chunk, gate=gate, maps=sp.maps,
+                      diff=(lw.diff_lambda, 1.0 - sp.diff, a.norm_eps, sp.vdim) if sp.maps == 2 else None)
         nd, B = s.num_decode, s.past_lens.shape[0]
         if not (qkv.is_cuda and 0 < nd < B and s.max_q_len > 1):
             return ops.paged_attention(qkv, kc, vc, s.cu_seqlens, s.past_lens, table, *args, max_q_len=s.max_q_len,
                                        max_kv_len=s.max_kv_len, order=s.attn_order, min_q_len=s.min_q_len or None, out=out, **kw)
         if out is None:
-            out = torch.empty(qkv.shape[0], args[1] * cols, dtype=qkv.dtype, device=qkv.device)
+            out = torch.empty(qkv.shape[0], args[1] // kw.get("maps", 1) * cols, dtype=qkv.dtype, device=qkv.device)
         # The chunks first: where their keys are split, the merge pass runs over all rows of the matrix and leaves unspecified values in
         # the rows of the single-token requests, which the second launch then writes.
         ops.paged_attention(qkv, kc, vc, s.cu_seqlens[nd:], s.past_lens[nd:], table[nd:], *args, max_q_len=s.max_q_len,
@@ -414,13 +433,13 @@ class DecoderModel:
         return out
 
     @staticmethod
-    def _wide_linear(x, w):
-        """x @ w.T with rows of whole 16-byte pieces, so that column ranges of the result can be read in vectors."""
+    def _wide_linear(x, w, b=None):
+        """x @ w.T (+ b) with rows of whole 16-byte pieces, so that column ranges of the result can be read in vectors."""
         N = w.shape[0]
         if not x.is_cuda:
-            return ops.linear(x, w)
+            return ops.linear(x, w, b)
         out = torch.empty(x.shape[0], (N + 7) // 8 * 8, dtype=x.dtype, device=x.device)[:, :N]
-        return ops.linear(x, w, out=out)
+        return ops.linear(x, w, b, out=out)
 
     def _linear_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out=None) -> torch.Tensor:
         """A gated-delta-net layer (reference graph: builders/qwen.py:1776-1867).  The causal convolution reads the projected
@@ -462,15 +481,27 @@ class DecoderModel:
     def _latent_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         """A latent-attention layer: writes the value heads of every token to `out` [T, heads * vdim] (a column range).  Decode steps and
         short portions attend over the cached latents with the key map folded into the queries; requests that feed many tokens expand
-        the latents they can see to keys and values and run on the tensor-memory kernel."""
+        the latents they can see to keys and values and run on the tensor-memory kernel.  Queries with a latent of their own are projected
+        from it once it is normed; an output gate multiplies the value heads."""
         sp = self.arch.layer_specs[li]
         T = x.shape[0]
         shape = ops.latent_shape(sp.heads, sp.dim, sp.rot_dim, sp.vdim, sp.kv_rank, sp.rotary.dims if sp.rotary else 0)
         cache = kv.latent_layer(li)
         proj = self._wide_linear(x, lw.lat_in_w)
-        ops.latent_prep(proj, shape, lw.lat_norm_w, self.arch.norm_eps, s.positions, lw.rope_cos, lw.rope_sin, s.slot_mapping, cache)
+        eps, width = self.arch.norm_eps, sp.kv_rank + sp.rot_dim
+        own = dict(down=proj[:, lw.lat_down_col:lw.lat_down_col + width], norm_w=lw.lat_norm_w, slots=s.slot_mapping, cache=cache)
+        if lw.lat_uq_w is None:
+            q = proj[:, :sp.heads * (sp.dim + sp.rot_dim)]
+            ops.latent_prep_parts(shape, eps, s.positions, lw.rope_cos, lw.rope_sin, q=q, **own)
+        else:
+            cq = proj[:, :sp.q_rank]
+            ops.latent_prep_parts(shape, eps, s.positions, lw.rope_cos, lw.rope_sin, cq=cq, cq_w=lw.lat_q_norm_w, **own)
+            q = self._wide_linear(cq, lw.lat_uq_w)
+            if sp.rotary:
+                ops.latent_prep_parts(shape, eps, s.positions, lw.rope_cos, lw.rope_sin, q=q)
+        gate = proj[:, lw.lat_gate_col:lw.lat_gate_col + sp.heads * sp.vdim] if sp.out_gate else None
         plan = None
-        if s.host_lens is not None and s.max_q_len >= ops.LATENT_LONG_TOKENS and ops.latent_long_supported(shape, proj, cache, kv.block_size):
+        if s.host_lens is not None and s.max_q_len >= ops.LATENT_LONG_TOKENS and ops.latent_long_supported(shape, q, cache, kv.block_size):
             if s.latent_plans is None:
                 s.latent_plans = {}
             plan = s.latent_plans.get(sp.window)
@@ -482,25 +513,30 @@ class DecoderModel:
             ends = np.cumsum([n for _, n in s.host_lens])
             n_short = max([int(e) for e, (_, n) in zip(ends, s.host_lens) if n < ops.LATENT_LONG_TOKENS], default=0)
         if n_short > 0:
-            qlat = ops.head_project(proj[:n_short], lw.lat_uk_t, sp.heads, sp.dim + sp.rot_dim)
-            olat = ops.latent_attention(qlat, proj, shape, cache, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale, sp.window,
-                                        s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0, order=s.attn_order)
+            qlat = ops.head_project(q[:n_short], lw.lat_uk_t, sp.heads, sp.dim + sp.rot_dim)
+            olat = ops.latent_attention(qlat, q, shape, cache, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale, sp.window,
+                                        s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0, order=s.attn_order,
+                                        sinks=lw.sinks)
             ops.head_project(olat, lw.lat_uv, sp.heads, sp.kv_rank, out=out[:n_short])
+            if gate is not None:
+                ops.gate_rows(out[:n_short], gate[:n_short])
         if plan is not None and plan.rows > 0:
-            ops.latent_attention_long(proj, shape, lw.lat_ukv, cache, plan, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale,
-                                      sp.window, out)
+            ops.latent_attention_long(q, shape, lw.lat_ukv, cache, plan, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale,
+                                      sp.window, out, lw.sinks, gate)
         return out
 
     def _spec_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         """An attention layer of a declared stack: one projection [queries | keys | values | gate logits], norms, rotation and cache append
-        in one pass, attention over the paged cache whose epilogue gates the heads; writes them to `out` [T, heads * value_row]."""
+        in one pass, attention over the paged cache whose epilogue gates the heads (or their columns); writes them to `out`
+        [T, heads * value_row]."""
         sp = self.arch.layer_specs[li]
         kc, vc, _ = kv.layer(li)
-        proj = self._wide_linear(x, lw.qkv_w)
-        ops.qkv_prep(proj, sp.heads, sp.kv_heads, sp.dim, sp.key_row, sp.value_row, lw.q_norm_w, lw.k_norm_w, self.arch.norm_eps, s.positions,
-                     lw.rope_cos, lw.rope_sin, s.slot_mapping, kc, vc)
+        proj = self._wide_linear(x, lw.qkv_w, lw.qkv_b)
+        ops.qkv_prep(proj, sp.heads * sp.maps, sp.kv_heads * sp.maps, sp.dim, sp.map_row, sp.value_row, lw.q_norm_w, lw.k_norm_w, self.arch.norm_eps,
+                     s.positions, lw.rope_cos, lw.rope_sin, s.slot_mapping, kc, vc, Hv=sp.kv_heads)
         g0 = (sp.heads + sp.kv_heads) * sp.key_row + sp.kv_heads * sp.value_row
-        return self._attention(s, proj, kc, vc, s.block_table, kv.block_size, lw, sp, proj[:, g0:g0 + sp.heads] if sp.head_gate else None, out)
+        cols = sp.heads * sp.value_row if sp.out_gate else (sp.heads if sp.head_gate else 0)
+        return self._attention(s, proj, kc, vc, s.block_table, kv.block_size, lw, sp, proj[:, g0:g0 + cols] if cols else None, out)
 
     def _stack_mixer(self, lw: LayerWeights, sp):
         return {"linear_attention": self._linear_attention, "latent_attention": self._latent_attention, "attention": self._spec_attention}[sp.kind]
@@ -512,6 +548,9 @@ class DecoderModel:
             raise RuntimeError("declared stacks run on one GPU")
         if s.lora_ids is not None or self.active_adapter is not None:
             raise RuntimeError("LoRA adapters are not available for declared stacks")
+        if a.tanh_norm:
+            self.last_hidden = x = self._tanh_normed_blocks(s, kv)
+            return ops.linear(x, self.lm_head_w, out_fp32=True)
         if a.parallel_block:
             h = self._parallel_blocks(s, kv)
         else:
@@ -561,6 +600,34 @@ class DecoderModel:
                     y = ops.linear(ops.gate_up_act(x, lw.gate_up_w, None, a.activation, interleaved=lw.gate_up_interleaved), lw.down_w)
                 x = ops.add_normed(h, y, lw.post_ffn_norm_w, a.norm_eps, self.dtype)
         return h
+
+    def _tanh_normed_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
+        """Pre-norm blocks under tanh norms, to the final norm of the rows whose logits are wanted.  The mixer's output map adds to the stream
+        in its epilogue; one kernel per norm adds what is still missing from the stream (experts' rows, and where a pass through the looped
+        layers begins its learned vector and the embedding output) and writes the norm of the sum."""
+        a = self.arch
+        if s.inputs_embeds is not None:
+            raise RuntimeError("this model's embedding reads token ids (pairs of neighbours): inputs_embeds cannot replace them")
+        if a.bigram:
+            first = ops.embedding_bigram(s.input_ids, self.embed, a.embed_scale, self.bigram, a.bigram, kv.tokens, s.slot_mapping, s.positions,
+                                         s.cu_seqlens, s.past_lens, s.block_table, kv.block_size)
+        else:
+            first = ops.embedding_stream(s.input_ids, self.embed, a.embed_scale)
+        stream = torch.empty_like(first) if a.passes > 1 else first      # (the embedding output itself is needed again before later passes)
+        h, y = first, None
+        for li, lw in enumerate(self.layers):
+            sp = a.layer_specs[li]
+            opens = sp.opens_pass
+            x = ops.add_tanh_norm(h, y, lw.norm1, self.dtype, first if opens else None, None if opens is None else self.loop_step[opens], out=stream)
+            h = stream
+            heads = torch.empty(h.shape[0], lw.mix_cols, dtype=self.dtype, device=h.device)
+            self._stack_mixer(lw, sp)(s, kv, li, lw, x, out=heads)
+            ops.linear(heads, lw.o_w, residual=h, out=h, out_fp32=True)
+            y = None
+            if sp.ff:
+                from .moe import moe_forward
+                y = moe_forward(self, lw, ops.add_tanh_norm(h, None, lw.norm2, self.dtype), defer=True)
+        return ops.add_tanh_norm(h, y, self.final_norm, self.dtype, rows=s.logits_rows)
 
     def _mamba(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor) -> torch.Tensor:
         """A Mamba-2 layer (GraniteMoeHybrid).  Like the gated-delta-net layers, the causal convolution reads the projected

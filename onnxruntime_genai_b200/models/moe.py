@@ -1,7 +1,9 @@
 """Mixture-of-experts MLP: router -> top-k -> routing weights -> per-expert gated MLP -> weighted sum.
 Two styles: gpt-oss (biases, softmax over the selected logits, clamped SwiGLU(alpha, limit)) and standard (Mixtral, Qwen-MoE,
 PhiMoE, GraniteMoE: no biases, silu(gate) * up, softmax over all experts with or without renormalisation).  Declared stacks describe
-the experts of each layer by themselves (`LayerWeights.moe`, an arch.MoeSpec), with any mix of these rules.
+the experts of each layer by themselves (`LayerWeights.moe`, an arch.MoeSpec), with any mix of these rules, and may have a shared expert:
+of the same width and limit it is one more expert of the grouped products that every token is routed to with weight 1, else it runs
+beside them and the add + norm that follows folds it.
 
 Semantics follow the MoE / QMoE contrib op the reference's builder emits
 (src/python/py/models/builders/base.py:4176-4408, builders/gptoss.py:653-847): `k` experts per token,
@@ -107,6 +109,13 @@ def expert_mlp(model, lw, e: int, xs: torch.Tensor) -> torch.Tensor:
     return ops.linear(act.contiguous(), wd, lw.exp_down_b[e] if lw.exp_down_b is not None else None)
 
 
+def shared_expert(lw, x: torch.Tensor, sp: MoeSpec) -> torch.Tensor:
+    """The expert every token takes, where it stands beside the routed ones (sizes or limits of its own)."""
+    gu = ops.linear(x, lw.shared_gate_up_w)
+    h = ops.expert_act(gu, "clamped", sp.alpha, sp.shared_limit) if x.is_cuda else swiglu_interleaved(gu, sp.alpha, sp.shared_limit)
+    return ops.linear(h, lw.shared_down_w)
+
+
 def _forward_loop(model, lw, x):
     sp = spec_of(model, lw)
     lo, hi = lw.exp_lo, lw.exp_hi or sp.experts
@@ -124,6 +133,10 @@ def _forward_loop(model, lw, x):
             y = expert_mlp(model, lw, e - lo, x[idx].contiguous()).float()
             out.index_add_(0, idx, y * w_sorted[start:start + n, None])
         start += n
+    if lw.exp_shared:
+        out += expert_mlp(model, lw, sp.experts, x).float()
+    elif lw.shared_gate_up_w is not None:
+        out += shared_expert(lw, x, sp).float()
     return out.to(x.dtype)
 
 
@@ -131,6 +144,8 @@ def _plan(model, lw, x, sp, token_tile=0):
     """Routing of the tokens, on the device."""
     lo, hi = lw.exp_lo, lw.exp_hi or sp.experts
     logits = ops.linear(x, lw.router_w, lw.router_b, out_fp32=True)
+    if lw.exp_shared:
+        return ops.moe_route(logits, sp.top, _TOPK_MODES[sp.weights], None, token_tile, shared=True)
     if sp.weights == "sparse_mixer":
         tw, ti = sparse_mixer(logits, sp.jitter_eps)
         return ops.moe_route(logits, 2, 0, (lo, hi), token_tile, topk=(ti.to(torch.int32).contiguous(), tw.contiguous()))
@@ -140,6 +155,9 @@ def _plan(model, lw, x, sp, token_tile=0):
 def _forward_device(model, lw, x, defer=False):
     sp = spec_of(model, lw)
     plan = _plan(model, lw, x, sp)
+    beside = shared_expert(lw, x, sp) if lw.shared_gate_up_w is not None else None
+    if beside is not None and not defer:
+        raise RuntimeError("a shared expert beside the routed ones needs the add + norm that folds it")
     half = isinstance(lw.exp_gate_up_w, ops.Fp4Experts) and lw.exp_gate_up_w.half and lw.exp_down_w.half
     if half:
         # packed MXFP4 experts in their fp16 form: fp16 rows in, fp16 between the two grouped GEMMs, bf16 out; the streaming
@@ -156,7 +174,7 @@ def _forward_device(model, lw, x, defer=False):
     else:
         h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=sp.alpha, limit=sp.limit)
     y = ops.moe_gemm(h, lw.exp_down_w, plan, lw.exp_down_b)
-    return ops.PendingCombine(y, plan) if defer else ops.moe_combine(y, plan)
+    return ops.PendingCombine(y, plan, beside) if defer else ops.moe_combine(y, plan)
 
 
 def _forward_simt(model, lw, x):
@@ -166,14 +184,14 @@ def _forward_simt(model, lw, x):
     plan = _plan(model, lw, x, sp, token_tile=64)
     gu = ops.moe_gemm_simt(x, lw.exp_gate_up_w, plan, mapped=True)
     h = ops.expert_act(gu, sp.act, sp.alpha, sp.limit)
-    return ops.PendingCombine(ops.moe_gemm_simt(h, lw.exp_down_w, plan), plan)
+    return ops.PendingCombine(ops.moe_gemm_simt(h, lw.exp_down_w, plan), plan, shared_expert(lw, x, sp) if lw.shared_gate_up_w is not None else None)
 
 
 def moe_forward(model, lw, x: torch.Tensor, defer: bool = False):
     """defer: the caller folds the combine step into the residual add + norm that follows (`ops.norm_moe_combine`); the
     result is then an `ops.PendingCombine` when the layer ran on the device path of a single rank."""
     a, sp = model.arch, spec_of(model, lw)
-    fast = x.is_cuda and lw.exp_blocked and a.hidden_size % 8 == 0 and sp.experts <= 1024 and sp.top <= 32
+    fast = x.is_cuda and lw.exp_blocked and a.hidden_size % 8 == 0 and sp.experts + lw.exp_shared <= 1024 and sp.top + lw.exp_shared <= 32
     if model.tp.size > 1 and getattr(model.tp, "ep_mode", "replicated") == "all_to_all":
         # token-sharded expert parallelism: dispatch / combine all-to-all, the output is complete on every rank
         from ..parallel.ep import moe_all_to_all

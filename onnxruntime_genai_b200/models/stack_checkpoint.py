@@ -60,6 +60,8 @@ def _synthetic_tensors(path: str, shapes: Dict[str, tuple], device, norm_offset:
 
     def get(name):
         t = random_tensor(name, shapes[name], int(meta.get("seed", 0)), float(meta.get("std", 0.02)), device=device)
+        if name.endswith("alpha"):
+            return torch.full_like(t, 0.5)
         around_one = name.endswith((".norm", "norm1", "norm2")) and (norm_offset == 0 or ".mix." in name) or name.endswith(("ls1", "ls2"))
         return t + 1.0 if around_one else t
     return get
@@ -112,16 +114,41 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
     up8 = lambda n: (n + 7) // 8 * 8      # columns of the joined input start on 16-byte boundaries
     tiled = cuda and dtype == torch.bfloat16
 
-    def head_rows(name, heads, size, row):
-        """[heads * size, K] -> [heads * row, K]: every head filled up with zero rows."""
-        w = raw(name).to(dtype)
-        return w if size == row else torch.nn.functional.pad(w.view(heads, size, -1), (0, 0, 0, row - size)).reshape(heads * row, -1)
+    def padded(w, heads, size, row):
+        """[heads * size, ...] -> [heads * row, ...]: every head filled up with zero rows."""
+        if size == row:
+            return w
+        v = w.reshape(heads, size, -1)
+        return torch.nn.functional.pad(v, (0, 0, 0, row - size)).reshape(heads * row, *w.shape[1:])
 
     def attention_weights(lw, sp, m):
-        lw.qkv_w = torch.cat([head_rows(m + "q", sp.heads, sp.dim, sp.key_row), head_rows(m + "k", sp.kv_heads, sp.dim, sp.key_row),
-                              head_rows(m + "v", sp.kv_heads, sp.vdim, sp.value_row)] + ([raw(m + "g").to(dtype)] if sp.head_gate else []), 0).contiguous()
+        # neighbours that rotate as pairs are brought to the places of the two halves: the same permutation of queries and keys
+        def halves(t):
+            n = sp.rotary.dims if sp.rotary and sp.rotary.neighbours else 0
+            if not n:
+                return t
+            t = t.view(-1, sp.dim, *t.shape[1:])
+            return torch.cat([t[:, 0:n:2], t[:, 1:n:2], t[:, n:]], 1).flatten(0, 1)
+
+        def rows(name, heads, size, row, place=lambda t: t):
+            return padded(place(raw(name).to(dtype)), heads, size, row)
+        sizes = [("q", sp.heads * sp.maps, sp.dim, sp.map_row, halves), ("k", sp.kv_heads * sp.maps, sp.dim, sp.map_row, halves),
+                 ("v", sp.kv_heads, sp.vdim, sp.value_row, lambda t: t)]
+        parts = [rows(m + n, *z) for n, *z in sizes]
+        gates = []
+        if sp.head_gate:
+            gates = [raw(m + "g").to(dtype)]
+        elif sp.out_gate:
+            gates = [rows(m + "g", sp.heads, sp.vdim, sp.value_row)]
+        lw.qkv_w = torch.cat(parts + gates, 0).contiguous()
+        if sp.qkv_bias:
+            b = torch.cat([rows(f"{m}{n}.b", *z) for n, *z in sizes])
+            lw.qkv_b = torch.nn.functional.pad(b, (0, lw.qkv_w.shape[0] - b.numel())).contiguous()
         if sp.qk_norm:
-            lw.q_norm_w, lw.k_norm_w = vec(m + "q.norm"), vec(m + "k.norm")
+            lw.q_norm_w, lw.k_norm_w = halves(vec(m + "q.norm")).contiguous(), halves(vec(m + "k.norm")).contiguous()
+        if sp.maps == 2:
+            lam = [torch.exp((vec(f"{m}lq{i}") * vec(f"{m}lk{i}")).sum()) for i in (1, 2)]
+            lw.diff_lambda = float(lam[0] - lam[1]) + sp.diff
         if sp.sinks:
             lw.sinks = vec(m + "sink")
         lw.rope_cos, lw.rope_sin = rotary(sp.rotary)
@@ -153,18 +180,54 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         lw.moe, lw.router_w, lw.exp_hi = sp.moe, mat(p + "router"), E
         lw.exp_blocked = tiled and W % 8 == 0
         F = (sp.ff + 63) // 64 * 64 if lw.exp_blocked else sp.ff      # (an expert's zero gates give zero, whatever its ups are)
+        names = [f"{p}e{e}." for e in range(E)]
+        # a shared expert of the same width and limit is one more expert that every token takes
+        ff2 = sp.moe.shared_ff
+        lw.exp_shared = ff2 == sp.ff and sp.moe.shared_limit == sp.moe.limit and E < 1024 and sp.moe.top < 32
+        if lw.exp_shared:
+            names.append(p + "shared.")
+        elif ff2:
+            gate, up = raw(p + "shared.gate").to(dtype), raw(p + "shared.up").to(dtype)
+            fill = (-ff2) % 8                                          # rows of whole 16-byte pieces
+            lw.shared_gate_up_w = torch.nn.functional.pad(torch.stack([gate, up], 1), (0, 0, 0, 0, 0, fill)).reshape(2 * (ff2 + fill), W).contiguous()
+            lw.shared_down_w = torch.nn.functional.pad(raw(p + "shared.down").to(dtype), (0, fill)).contiguous()
+        E = len(names)
         gate_up = torch.zeros(E, 2, F, W, dtype=dtype, device=device)
         lw.exp_down_w = torch.zeros(E, W, F, dtype=dtype, device=device)
-        for e in range(E):
-            gate_up[e, 0, :sp.ff], gate_up[e, 1, :sp.ff] = raw(f"{p}e{e}.gate").to(dtype), raw(f"{p}e{e}.up").to(dtype)
-            lw.exp_down_w[e, :, :sp.ff] = raw(f"{p}e{e}.down").to(dtype)
+        for e, n in enumerate(names):
+            gate_up[e, 0, :sp.ff], gate_up[e, 1, :sp.ff] = raw(n + "gate").to(dtype), raw(n + "up").to(dtype)
+            lw.exp_down_w[e, :, :sp.ff] = raw(n + "down").to(dtype)
         if lw.exp_blocked:
             lw.exp_gate_up_w = interleave_experts_gate_up(gate_up.view(E, 2 * F, W), fused_interleaved=False)
         else:
             lw.exp_gate_up_w = gate_up.transpose(1, 2).reshape(E, 2 * F, W).contiguous()
 
+    def tanh_norm(name):
+        from ..ops import TanhNorm
+        return TanhNorm(vec(name), vec(name + ".b"), float(raw(name + ".alpha")))
+
+    def latent_input(lw, sp, m):
+        """Input projection of a latent-attention layer: [queries or their latent | latent and shared rotary key | gate logits], the parts
+        starting on 16-byte boundaries where there are more than the first two."""
+        parts = [raw(m + ("dq" if sp.q_rank else "q")).to(dtype), raw(m + "dkv").to(dtype)] + ([raw(m + "g").to(dtype)] if sp.out_gate else [])
+        starts, at, rows = [], 0, []
+        for t in parts:
+            if sp.q_rank or sp.out_gate:
+                rows.append(t.new_zeros(up8(at) - at, t.shape[1]))
+                at = up8(at)
+            starts.append(at)
+            rows.append(t)
+            at += t.shape[0]
+        lw.lat_in_w, lw.lat_down_col = torch.cat(rows, 0).contiguous(), starts[1]
+        if sp.out_gate:
+            lw.lat_gate_col = starts[2]
+        if sp.q_rank:
+            lw.lat_q_norm_w, lw.lat_uq_w = vec(m + "dq.norm"), mat(m + "uq")
+
     def layer(i) -> LayerWeights:
-        sp, p, m = arch.layer_specs[i], f"l{i}.", f"l{i}.mix."
+        sp = arch.layer_specs[i]
+        p = f"l{i if sp.source is None else sp.source}."
+        m = p + "mix."
         lw = LayerWeights(ln1_w=None, qkv_w=None, o_w=None, ln2_w=None)
         lw.mix_cols = sp.heads * (sp.value_row or sp.vdim)
         if sp.kind == "linear_attention":
@@ -175,12 +238,20 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         elif sp.kind == "attention":
             attention_weights(lw, sp, m)
         else:
-            lw.lat_in_w = mat(m + "q", m + "dkv")
+            latent_input(lw, sp, m)
+            if sp.sinks:
+                lw.sinks = vec(m + "sink")
             lw.lat_norm_w = vec(m + "dkv.norm")
             lw.lat_uk_t = mat(m + "uk").view(sp.heads, sp.dim, sp.kv_rank).transpose(1, 2).reshape(sp.heads * sp.kv_rank, sp.dim).contiguous()
             lw.lat_ukv = mat(m + "uk", m + "uv")
             lw.lat_uv = lw.lat_ukv[sp.heads * sp.dim:]
             lw.rope_cos, lw.rope_sin = rotary(sp.rotary)
+        if arch.tanh_norm:
+            lw.o_w, lw.norm1 = output_map(m + "o", sp), tanh_norm(p + "norm1")
+            if sp.ff:
+                expert_weights(lw, sp, p + "mlp.")
+                lw.norm2 = tanh_norm(p + "norm2")
+            return lw
         if not arch.parallel_block:
             lw.o_w, lw.post_attn_norm_w = output_map(m + "o", sp), output_factor(p, 1)
             if sp.ff:
@@ -200,8 +271,15 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         return lw
 
     model.embed, model.lm_head_w = mat("embed"), mat("head")
-    model.final_norm_w = vec("final.norm") + arch.norm_offset
-    model.final_norm_b = vec("final.norm.b") if arch.layernorm else None
+    if arch.tanh_norm:
+        model.final_norm = tanh_norm("final.norm")
+    else:
+        model.final_norm_w = vec("final.norm") + arch.norm_offset
+        model.final_norm_b = vec("final.norm.b") if arch.layernorm else None
+    if arch.bigram:
+        model.bigram = mat("bigram")
+    if arch.passes:
+        model.loop_step = vec("loop.step")
     own = {i: layer(i) for i, sp in enumerate(arch.layer_specs) if sp.weights_of is None}
     model.layers = [own[i if sp.weights_of is None else sp.weights_of] for i, sp in enumerate(arch.layer_specs)]
     return model

@@ -154,6 +154,7 @@ def add_normed(h, y, weight, eps, dtype=torch.bfloat16):
         return h if dtype == torch.float32 else h.to(dtype)
     plan = None
     if isinstance(y, PendingCombine):
+        assert y.shared is None
         y, plan = y.y, y.plan
     T, H = h.shape
     assert h.dtype == torch.float32 and h.is_contiguous() and weight.dtype == torch.float32 and y.stride(1) == 1 and y.shape[1] == H
@@ -163,6 +164,57 @@ def add_normed(h, y, weight, eps, dtype=torch.bfloat16):
                                         _ptr(plan.inv_pos) if plan else None, _ptr(plan.topk_w) if plan else None, plan.k if plan else 0, T, H, _stream()),
                "add_normed")
     return h if x is None else x
+
+
+def embedding_bigram(ids, table, scale, bigram, spec, tokens, slots, positions, cu_seqlens, past_lens, block_table, block_size: int):
+    """Start of an fp32 residual stream: table[id] * scale + bigram[(previous * mul_prev + id * mul_cur) mod buckets] (row `buckets` for the first
+    token of a sequence), spec = {buckets, mul_prev, mul_cur}.  The token before a request's first one of the step is read from the paged pool
+    `tokens` [slots] int32, to which this step's tokens are written (slot < 0: not)."""
+    _check_index("embedding_bigram", "slots", slots[:ids.numel()], tokens.shape[0], -1)
+    if not table.is_cuda:
+        return ref.embedding_bigram(ids, table, scale, bigram, spec, tokens, slots, positions, cu_seqlens, past_lens, block_table, block_size)
+    import ctypes
+    assert ids.dtype == torch.int32 and tokens.dtype == torch.int32 and table.is_contiguous() and bigram.is_contiguous() and bigram.dtype == table.dtype
+    assert bigram.shape == (spec["buckets"] + 1, table.shape[1]) and block_table.stride(1) == 1 and table.dtype in (torch.bfloat16, torch.float32)
+    T, H = ids.numel(), table.shape[1]
+    out = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    p = _lib.Bigram(ids=_ptr(ids), slots=_ptr(slots), cu_seqlens=_ptr(cu_seqlens), past_lens=_ptr(past_lens), block_table=_ptr(block_table),
+                    tokens=_ptr(tokens), table_cols=block_table.stride(0), block_size=int(block_size), B=past_lens.shape[0], T=T, H=H, vocab=table.shape[0],
+                    fp32=int(table.dtype == torch.float32), scale=float(scale), **spec)
+    _lib.check(_lib.lib().ogb_embedding_bigram(ctypes.byref(p), _ptr(table), _ptr(bigram), _ptr(out), _stream()), "embedding_bigram")
+    return out
+
+
+class TanhNorm:
+    """A norm without statistics: tanh(alpha * x) * weight + bias (weight and bias fp32)."""
+    __slots__ = ("weight", "bias", "alpha")
+
+    def __init__(self, weight, bias, alpha: float):
+        self.weight, self.bias, self.alpha = weight, bias, float(alpha)
+
+
+def add_tanh_norm(h, y, norm: TanhNorm, dtype=torch.bfloat16, first=None, step=None, rows=None, out=None):
+    """n = h + y (+ first) (+ step), tanh norm of n in `dtype`; n is written to `out` (h itself: in place; None: nowhere).  h [T, H] the fp32 residual
+    stream; y: the sub-layer's rows [T, H], a mixture-of-experts output whose combine step is pending, or None; first fp32 [T, H], step fp32 [H].
+    rows (int32): only these rows are summed and normed (out must be None)."""
+    if not h.is_cuda:
+        return ref.add_tanh_norm(h, y, norm, dtype, first, step, rows, out)
+    import ctypes
+    plan = y2 = None
+    if isinstance(y, PendingCombine):
+        y, plan, y2 = y.y, y.plan, y.shared
+    T, H = h.shape
+    n = T if rows is None else rows.numel()
+    assert h.dtype == torch.float32 and h.is_contiguous() and (out is None or (rows is None and out.is_contiguous() and out.dtype == torch.float32))
+    assert all(t is None or (t.dtype == dtype and t.stride(1) == 1 and t.shape[1] == H) for t in (y, y2)) and norm.weight.dtype == torch.float32
+    assert all(t is None or (t.dtype == torch.float32 and t.is_contiguous()) for t in (first, step)) and (plan is None or plan.T == T)
+    x = torch.empty(n, H, dtype=dtype, device=h.device)
+    p = _lib.TanhNorm(h_in=_ptr(h), h_out=_ptr(out), y=_ptr(y), y2=_ptr(y2), inv_pos=_ptr(plan.inv_pos) if plan else None,
+                      topk_w=_ptr(plan.topk_w) if plan else None, first=_ptr(first), step=_ptr(step), w=_ptr(norm.weight), b=_ptr(norm.bias), x=_ptr(x),
+                      rows=_ptr(rows), ldy=y.stride(0) if y is not None else 0, ldy2=y2.stride(0) if y2 is not None else 0, k=plan.k if plan else 0,
+                      n_rows=n, H=H, fp32=int(dtype == torch.float32), alpha=norm.alpha)
+    _lib.check(_lib.lib().ogb_add_tanh_norm(ctypes.byref(p), _stream()), "add_tanh_norm")
+    return x
 
 
 def norm_stream(x, weight, eps, bias=None, layernorm=False, dtype=torch.bfloat16, rows=None):
@@ -202,17 +254,18 @@ def norm(x, weight, eps, residual=None, bias=None, layernorm=False, out=None) ->
 
 class PendingCombine:
     """The output of a mixture-of-experts layer before its combine step: the experts' rows `y` and the routing plan.
-    `norm_moe_combine` folds the weighted sum into the residual add + norm that consumes it."""
-    __slots__ = ("y", "plan")
+    `norm_moe_combine` folds the weighted sum into the residual add + norm that consumes it.  shared: rows [T, H] of an expert that runs for
+    every token outside the routing plan (added with weight 1)."""
+    __slots__ = ("y", "plan", "shared")
 
-    def __init__(self, y, plan):
-        self.y, self.plan = y, plan
+    def __init__(self, y, plan, shared=None):
+        self.y, self.plan, self.shared = y, plan, shared
 
 
 def norm_moe_combine(pending: PendingCombine, weight, eps, residual, bias=None, layernorm=False):
     """norm(moe_combine(pending.y, pending.plan), weight, eps, residual, ...) in one launch; same results bit for bit."""
     y, plan = pending.y, pending.plan
-    assert y.is_cuda and y.dtype == torch.bfloat16 and y.stride(-1) == 1 and residual is not None
+    assert pending.shared is None and y.is_cuda and y.dtype == torch.bfloat16 and y.stride(-1) == 1 and residual is not None
     H = y.shape[1]
     out = torch.empty(plan.T, H, dtype=torch.bfloat16, device=y.device)
     _lib.check(_lib.lib().ogb_norm_moe_combine(_ptr(y), y.stride(0), _ptr(plan.inv_pos), _ptr(plan.topk_w), plan.k, _ptr(residual),
@@ -276,12 +329,13 @@ def _tma_ok(x, w) -> bool:
     return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0
 
 
-def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None):
+def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None, bias=None):
     """The fp32 / unaligned form of a product (csrc/gemm_simt.cu)."""
+    assert bias is None or bias.dtype == x.dtype
     assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and out.dtype in (torch.float32, torch.bfloat16)
     _lib.check(_lib.lib().ogb_gemm_simt(_ptr(x), x.stride(0), int(a_cols), _ptr(w), w.stride(0), _ptr(out), out.stride(0), int(c_cols), x.shape[0],
                                        w.shape[0] // batch, K or x.shape[1], int(batch), _ptr(residual), residual.stride(0) if residual is not None else 0,
-                                       int(x.dtype == torch.float32), int(out.dtype == torch.float32), _stream()), "gemm_simt")
+                                       _ptr(bias), int(x.dtype == torch.float32), int(out.dtype == torch.float32), _stream()), "gemm_simt")
     return out
 
 
@@ -323,13 +377,13 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, out=None, splits=0, a
         y = ref.linear(x, w, bias, residual, out_fp32, norm_eps)
         return y if out is None else out.copy_(y)
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.stride(-1) == 1
-    if x.dtype == torch.float32 or (bias is None and norm_eps == 0 and not all_reduce and reduce_scatter is None and not _tma_ok(x, w) and
+    if x.dtype == torch.float32 or (norm_eps == 0 and not all_reduce and reduce_scatter is None and not _tma_ok(x, w) and
                                     (residual is None or residual.dtype == torch.float32)):
         # 32-bit models, and bf16 shapes TMA cannot address
-        assert bias is None and norm_eps == 0 and not all_reduce and reduce_scatter is None
+        assert norm_eps == 0 and not all_reduce and reduce_scatter is None
         if out is None:
             out = torch.empty(x.shape[0], w.shape[0], dtype=torch.float32 if out_fp32 else x.dtype, device=x.device)
-        return _gemm_simt(x, w, out, residual)
+        return _gemm_simt(x, w, out, residual, bias=bias)
     assert x.dtype == torch.bfloat16
     fused = None
     if norm_eps > 0:
@@ -648,16 +702,19 @@ class MoePlan:
                  "tile_row0", "tile_rows", "num_tiles")
 
 
-def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=None, token_tile: int = 0, topk=None) -> MoePlan:
+def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=None, token_tile: int = 0, topk=None, shared: bool = False) -> MoePlan:
     """router_logits [T, E] fp32 -> MoePlan (top-k, routing weights, rows grouped by expert, GEMM tile list).
     mode 0: softmax over the selected logits; 1: softmax over all experts; 2: the latter renormalised.
     expert_range (lo, hi): only these experts are local (expert parallelism).  topk = (idx int32 [T, k], weights fp32 [T, k]):
-    a selection made elsewhere (PhiMoE's sparse mixer); only the grouping by expert is computed."""
+    a selection made elsewhere (PhiMoE's sparse mixer); only the grouping by expert is computed.  shared: every token is also served by
+    expert E, with weight 1 (the plan then has E + 1 experts and k + 1 of them per token)."""
     assert router_logits.is_cuda and router_logits.dtype == torch.float32 and router_logits.stride(-1) == 1
-    T, E = router_logits.shape
+    T, routed = router_logits.shape
+    top, k, E = k, k + int(shared), routed + int(shared)
     L = _lib.lib()
     dev = router_logits.device
     lo, hi = expert_range if expert_range is not None else (0, E)
+    assert not shared or (topk is None and (lo, hi) == (0, E))
     pl = MoePlan()
     n = T * k
     bt = token_tile or L.ogb_gemm_token_tile(max(1, min(T, -(-2 * n // max(1, hi - lo)))), 0)
@@ -677,7 +734,7 @@ def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=N
     pl.tile_expert, pl.tile_row0, pl.tile_rows = tiles[:pl.max_tiles], tiles[pl.max_tiles:2 * pl.max_tiles], tiles[2 * pl.max_tiles:3 * pl.max_tiles]
     pl.num_tiles = tiles[3 * pl.max_tiles:]
     if topk is None:
-        _lib.check(L.ogb_moe_topk(_ptr(router_logits), router_logits.stride(0), T, E, k, mode, _ptr(pl.topk_idx), _ptr(pl.topk_w), _stream()),
+        _lib.check(L.ogb_moe_topk(_ptr(router_logits), router_logits.stride(0), T, routed, top, mode, int(shared), _ptr(pl.topk_idx), _ptr(pl.topk_w), _stream()),
                    "moe_topk")
     _lib.check(L.ogb_moe_sort(_ptr(pl.topk_idx), T, k, E, lo, hi, bt, _ptr(pl.expert_offsets), _ptr(pl.sorted_token), _ptr(pl.inv_pos),
                               _ptr(pl.tile_expert), _ptr(pl.tile_row0), _ptr(pl.tile_rows), _ptr(pl.num_tiles), pl.max_tiles, _stream()),
@@ -784,19 +841,20 @@ def rope_kv_append(qkv, positions, slots, cos_cache, sin_cache, k_cache, v_cache
     return qkv
 
 
-def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache):
-    """Between the projection [Hq queries | Hkv keys | Hkv values | ...] of an attention layer and its attention: RMS norm of every query and
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv=None):
+    """Between the projection [Hq queries | Hkv keys | Hv (None: Hkv) values | ...] of an attention layer and its attention: RMS norm of every query and
     key head over its `dim` columns (weights fp32 [dim] or None), rotation of the first 2 * cos.shape[1] of them (cos / sin fp32 [positions,
-    rot / 2], or None), queries in place, keys and values to row slots[t] of the caches [slots, Hkv, key_row] and [slots, Hkv, value_row]
+    rot / 2], or None), queries in place, keys and values to row slots[t] of the caches [slots, Hkv, key_row] and [slots, Hv, value_row]
     (slot < 0: to no row).  Any sizes, bf16 or fp32."""
+    Hv = Hv or Hkv
     _check_index("qkv_prep", "slots", slots[:proj.shape[0]], k_cache.shape[0], -1)
     if cos is not None:
         _check_index("qkv_prep", "positions", positions[:proj.shape[0]], cos.shape[0])
     if not proj.is_cuda:
-        return ref.qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache)
+        return ref.qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv)
     assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == proj.dtype
     assert proj.dtype in (torch.bfloat16, torch.float32) and all(w is None or w.dtype == torch.float32 for w in (q_norm_w, k_norm_w, cos, sin))
-    _lib.check(_lib.lib().ogb_qkv_prep(_ptr(proj), proj.stride(0), Hq, Hkv, dim, key_row, value_row, _ptr(q_norm_w), _ptr(k_norm_w), float(eps),
+    _lib.check(_lib.lib().ogb_qkv_prep(_ptr(proj), proj.stride(0), Hq, Hkv, Hv, dim, key_row, value_row, _ptr(q_norm_w), _ptr(k_norm_w), float(eps),
                                       _ptr(positions), _ptr(cos), _ptr(sin), 2 * cos.shape[1] if cos is not None else 0,
                                       cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(k_cache), _ptr(v_cache), proj.shape[0],
                                       int(proj.dtype == torch.float32), _stream()), "qkv_prep")
@@ -837,22 +895,23 @@ _TC_ATTENTION = os.environ.get("OGB_ATTN_TC", "1") != "0"
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale, window=0,
                     sinks=None, softcap=0.0, max_q_len=None, max_kv_len=None, splits=None, out=None, total_tokens=None, order=None,
-                    min_q_len=None, vdim=None, chunk=0, gate=None):
+                    min_q_len=None, vdim=None, chunk=0, gate=None, maps=1, diff=None):
     """q: [T, stride] with the Hq*D query columns first.  Returns [T, Hq*D].  total_tokens: the requests of this call only cover
     the first `total_tokens` rows of q (sizes the split-KV scratch).  min_q_len: shortest request of the call when the caller
     knows it (a call whose every request is long runs on the tensor-core prefill kernel alone).  vdim (layers with sizes of their own): width
     of a value head; chunk > 0: position p sees the keys from p // chunk * chunk on; gate [T, Hq]: each head's output is multiplied by its
-    sigmoid."""
+    sigmoid, or [T, heads * vdim]: each output column.  maps = 2, diff = (lambda, post, eps, columns): differential attention - q holds Hq vectors of
+    D / 2 columns, 2 h and 2 h + 1 for head h, a key head both maps' keys; returns the Hq / 2 heads (see csrc/kernels.h, ogb_attention_diff_merge),
+    RMS-normed over the first `columns` of each."""
     _check_index("paged_attention", "block_table", block_table, k_cache.shape[0] // block_size, -1)
     _check_index("paged_attention", "cu_seqlens", cu_seqlens[:past_lens.shape[0] + 1], q.shape[0] + 1)
     if not q.is_cuda:
         o = ref.paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                                window, sinks, softcap, vdim, chunk, gate)
+                                window, sinks, softcap, vdim, chunk, gate, maps, diff)
         return o if out is None else out.copy_(o)
-    if vdim is not None or chunk > 0 or gate is not None:
-        assert softcap == 0.0
+    if vdim is not None or chunk > 0 or gate is not None or maps > 1:
         return _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, vdim or D, scale, window, chunk,
-                                      sinks, gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len)
+                                      sinks, softcap, gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps, diff)
     T = q.shape[0] if total_tokens is None else total_tokens
     B = past_lens.shape[0]
     if out is None:
@@ -903,49 +962,73 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
     return out
 
 
-def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, dk, dv, scale, window, chunk, sinks, gate,
-                           max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len):
+def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, dk, dv, scale, window, chunk, sinks, softcap,
+                           gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps=1, diff=None):
     """paged_attention of layers with sizes of their own: the tensor-memory kernel for requests with at least TC_ATTENTION_MIN_ROWS query
     rows, the warp-MMA kernel for the others, plain arithmetic for fp32 and for sizes neither can address."""
     import ctypes
     T = q.shape[0] if total_tokens is None else total_tokens
     B = past_lens.shape[0]
+    assert (maps == 1) == (diff is None) and maps <= 2 and (diff is None or sinks is None)
     if out is None:
-        out = torch.empty(q.shape[0], Hq * dv, dtype=q.dtype, device=q.device)
+        out = torch.empty(q.shape[0], Hq // maps * dv, dtype=q.dtype, device=q.device)
     max_q_len = max_q_len or T
     L, G, ws = _lib.lib(), Hq // Hkv, workspace(q.device)
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and out.stride(1) == 1 and block_table.stride(1) == 1
     assert sinks is None or sinks.dtype == torch.float32
-    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[1] in (Hq, Hq // maps * dv))
+    wide = gate is not None and gate.shape[1] == Hq // maps * dv and (dv > 1 or maps > 1)
+    in_kernel = gate if diff is None else None             # (a differential layer's gate belongs to the merge of its maps)
     layer = _lib.AttnLayer(Hq=Hq, Hkv=Hkv, dk=dk, dv=dv, window=int(window), chunk=int(chunk), gate_stride=gate.stride(0) if gate is not None else 0,
-                           scale=float(scale), sinks=_ptr(sinks), gate=_ptr(gate))
+                           scale=float(scale), sinks=_ptr(sinks), gate=_ptr(in_kernel), gate_wide=int(wide), maps=maps, raw=int(diff is not None),
+                           softcap=float(softcap or 0.0))
+
+    def merge(part, sp, part_tokens):
+        """Differential layers: the two maps' partial results of the call's tokens become the heads."""
+        lam, post, eps, cols = diff
+        _lib.check(L.ogb_attention_diff_merge(_ptr(part), int(sp), min(T, out.shape[0]), int(part_tokens), Hq // 2, dv, int(cols), float(lam), float(post),
+                                              float(eps), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0),
+                                              int(out.dtype == torch.float32), _stream()), "attention_diff_merge")
+        return out
+
+    def part_bytes(tokens, sp):
+        return int(sp) * tokens * Hq * (dv + 2) * 4
     inputs = (ctypes.byref(layer), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(cu_seqlens), _ptr(past_lens), _ptr(block_table),
               block_table.stride(0), int(block_size), _ptr(out), out.stride(0), B)
     if (q.dtype == torch.float32 or not L.ogb_attention_mixed_supported(dk, dv) or q.stride(0) % 8 or out.stride(0) % 2 or q.data_ptr() % 16 or
             out.data_ptr() % 4):
         # (the grid covers the rows of the whole matrix: rows of requests outside this call are skipped)
-        _lib.check(L.ogb_attention_simt(*inputs, q.shape[0], int(q.dtype == torch.float32), _stream()), "attention_simt")
-        return out
+        n = q.shape[0]
+        scratch = ws.attn_scratch(part_bytes(n, 1)) if diff is not None else None
+        _lib.check(L.ogb_attention_simt(*inputs, n, _ptr(scratch), scratch.numel() if scratch is not None else 0, int(q.dtype == torch.float32), _stream()),
+                   "attention_simt")
+        return out if diff is None else merge(scratch, 1, n)
     slots = int(k_cache.shape[0])
     long_rows = TC_ATTENTION_MIN_ROWS
     use_tc = (_TC_ATTENTION and max_q_len * G >= long_rows and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and
-              bool(L.ogb_attention_tc_mixed_supported(dk, dv, int(block_size), slots)))
-    if not (use_tc and min_q_len is not None and min_q_len * G >= long_rows):
+              bool(L.ogb_attention_tc_mixed_supported(dk // maps, dv, int(block_size), slots)) and
+              (not wide or diff is not None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)))
+    sp, ch, scratch = 1, 0, None
+    all_long = use_tc and min_q_len is not None and min_q_len * G >= long_rows
+    if not all_long:
         # (first: with splits the combine pass leaves unspecified values in the rows of the long requests)
         if splits is None:
             span = max_kv_len or 1024
-            if chunk > 0:
-                span = min(span, chunk + 63)
+            if chunk > 0 or window > 0:
+                span = min(span, (chunk or window) + 63)
             splits = choose_kv_splits(B, Hkv, max_q_len, span, group=G, ordered=order is not None)
         sp, ch = splits if isinstance(splits, tuple) else (splits, 0)
-        scratch = ws.attn_scratch(L.ogb_attention_scratch_bytes(T, Hq, dv, sp)) if sp > 1 else None
+    if sp > 1 or diff is not None:
+        scratch = ws.attn_scratch(part_bytes(T, sp))
+    if not all_long:
         _lib.check(L.ogb_attention_mixed(*inputs, T, int(max_q_len), int(sp), int(ch), _ptr(scratch), scratch.numel() if scratch is not None else 0,
                                          _ptr(order), ws.status, _stream(), long_rows if use_tc else 0), "attention_mixed")
-        if sp > 1:
+        if sp > 1 and diff is None:
             _lib.LAUNCH_COUNT += 1      # the combine kernel
     if use_tc:
-        _lib.check(L.ogb_attention_tc_mixed(*inputs, int(max_q_len), long_rows, slots, ws.status, _stream()), "attention_tc_mixed")
-    return out
+        _lib.check(L.ogb_attention_tc_mixed(*inputs, int(max_q_len), long_rows, slots, int(sp), T, _ptr(scratch),
+                                            scratch.numel() if scratch is not None else 0, ws.status, _stream()), "attention_tc_mixed")
+    return out if diff is None else merge(scratch, sp, T)
 
 
 # ------------------------------------------------------------------------------------------ latent attention
@@ -962,19 +1045,41 @@ def _sh(shape):
 
 
 def latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache):
-    """In place: rotates the rotary part of every query head of proj ([H heads of (dim | rot)] then [latent | shared rotary key]), and
+    """`latent_prep_parts` of one projection [H heads of (dim | rot) | latent | shared rotary key].  In place: rotates the rotary part of every query head of proj ([H heads of (dim | rot)] then [latent | shared rotary key]), and
     writes the RMS-normalised latent and the rotated key of each token to its row of `cache` [slots, >= kv_rank + rot] (slot < 0: to no
     row).  cos / sin [positions, rot_dims / 2] fp32, or None for a layer that does not rotate."""
     _check_index("latent_prep", "slots", slots[:proj.shape[0]], cache.shape[0], -1)
     if cos is not None:
         _check_index("latent_prep", "positions", positions[:proj.shape[0]], cos.shape[0])
-    if not proj.is_cuda:
-        return ref.latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache)
-    assert proj.stride(1) == 1 and cache.stride(1) == 1 and cache.dtype == proj.dtype and norm_w.dtype == torch.float32
-    _lib.check(_lib.lib().ogb_latent_prep(_ptr(proj), proj.stride(0), _sh(shape), _ptr(norm_w), float(eps), _ptr(positions), _ptr(cos), _ptr(sin),
-                                         cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(cache), cache.stride(0), proj.shape[0],
-                                         int(proj.dtype == torch.float32), _stream()), "latent_prep")
+    n = shape.H * (shape.dim + shape.rot)
+    latent_prep_parts(shape, eps, positions, cos, sin, q=proj[:, :n], down=proj[:, n:], norm_w=norm_w, slots=slots, cache=cache)
     return proj
+
+
+def latent_prep_parts(shape, eps, positions, cos, sin, q=None, down=None, norm_w=None, slots=None, cache=None, cq=None, cq_w=None):
+    """The steps around a latent-attention layer's projections, each where its matrix is given: q [T, H * (dim | rot)]: the rotary parts are rotated in
+    place; down [T, latent | shared rotary key]: normed (weight norm_w) and rotated into `cache`; cq [T, q_rank]: RMS norm with weight cq_w in
+    place (the queries' own latent)."""
+    some = next(t for t in (q, down, cq) if t is not None)
+    if not some.is_cuda:
+        return ref.latent_prep_parts(shape, eps, positions, cos, sin, q, down, norm_w, slots, cache, cq, cq_w)
+    assert all(t is None or (t.stride(1) == 1 and t.dtype == some.dtype) for t in (q, down, cq, cache))
+    assert all(t is None or t.dtype == torch.float32 for t in (norm_w, cq_w)) and (down is None or (cache is not None and slots is not None))
+    ld = lambda t: t.stride(0) if t is not None else 0
+    _lib.check(_lib.lib().ogb_latent_prep(_ptr(q), ld(q), _ptr(down), ld(down), _ptr(cq), ld(cq), cq.shape[1] if cq is not None else 0, _ptr(cq_w),
+                                         _sh(shape), _ptr(norm_w), float(eps), _ptr(positions), _ptr(cos), _ptr(sin),
+                                         cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(cache), ld(cache), some.shape[0],
+                                         int(some.dtype == torch.float32), _stream()), "latent_prep")
+
+
+def gate_rows(x, gate):
+    """x *= sigmoid(gate) in place; both [T, n] (column ranges of wider matrices)."""
+    if not x.is_cuda:
+        return x.copy_((x.float() * torch.sigmoid(gate.float())).to(x.dtype))
+    assert x.stride(1) == 1 and gate.stride(1) == 1 and gate.shape == x.shape and gate.dtype == x.dtype
+    _lib.check(_lib.lib().ogb_gate_rows(_ptr(x), x.stride(0), _ptr(gate), gate.stride(0), x.shape[0], x.shape[1], int(x.dtype == torch.float32), _stream()),
+               "gate_rows")
+    return x
 
 
 def choose_latent_splits(batch: int, row_tiles: int, tile_rows: int, max_kv_len: int, window: int, sm_count: int = 148) -> int:
@@ -987,13 +1092,14 @@ def choose_latent_splits(batch: int, row_tiles: int, tile_rows: int, max_kv_len:
 
 
 def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0, max_q_len=1, max_kv_len=1,
-                     skip_q_len=0, splits=None, order=None):
+                     skip_q_len=0, splits=None, order=None, sinks=None):
     """Attention of every head over the shared latent rows: qlat [T, H * kv_rank] (queries with the key map folded in), the rotated
     query parts in proj.  window > 0: position p sees (p - window, p].  skip_q_len > 0: requests with at least that many tokens are
-    not computed (their rows are unspecified).  order [B]: requests in the order in which their CTAs are issued.  Returns [T, H * kv_rank]."""
+    not computed (their rows are unspecified).  order [B]: requests in the order in which their CTAs are issued.  sinks [H] fp32: a logit in each
+    head's denominator.  Returns [T, H * kv_rank]."""
     _check_index("latent_attention", "block_table", block_table, cache.shape[0] // block_size, -1)
     if not qlat.is_cuda:
-        return ref.latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window)
+        return ref.latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window, sinks)
     T, B, H, R = qlat.shape[0], past_lens.shape[0], shape.H, shape.R
     out = torch.empty_like(qlat)
     L = _lib.lib()
@@ -1002,7 +1108,7 @@ def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_tabl
             (qlat.data_ptr() | proj.data_ptr() | cache.data_ptr()) % 16):
         _lib.check(L.ogb_latent_attention_simt(_ptr(qlat), _ptr(proj), proj.stride(0), _sh(shape), _ptr(cache), cache.stride(0), _ptr(cu_seqlens),
                                                _ptr(past_lens), _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale),
-                                               int(window), B, T, int(skip_q_len), int(f32), _stream()), "latent_attention_simt")
+                                               int(window), _ptr(sinks), B, T, int(skip_q_len), int(f32), _stream()), "latent_attention_simt")
         return out
     q_len = min(max_q_len, skip_q_len - 1) if skip_q_len > 0 else max_q_len
     if splits is None:
@@ -1011,7 +1117,7 @@ def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_tabl
     need = L.ogb_latent_scratch_bytes(T * H, R, splits)
     scratch = workspace(qlat.device).attn_scratch(need) if splits > 1 else None
     _lib.check(L.ogb_latent_attention(_ptr(qlat), _ptr(proj), proj.stride(0), _sh(shape), _ptr(cache), cache.stride(0), _ptr(cu_seqlens), _ptr(past_lens),
-                                      _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale), int(window), B, T,
+                                      _ptr(block_table), block_table.stride(0), int(block_size), _ptr(out), float(scale), int(window), _ptr(sinks), B, T,
                                       int(max_q_len), int(skip_q_len), int(splits), _ptr(scratch), scratch.numel() if scratch is not None else 0,
                                       _ptr(order), workspace(qlat.device).status, _stream()), "latent_attention")
     if splits > 1:
@@ -1063,20 +1169,23 @@ def latent_expand(shape, w_ukv, cache, plan: LatentPlan, block_table, block_size
     return lat, linear(lat[:, :shape.R], w_ukv)
 
 
-def latent_attend_expanded(proj, shape, lat, kv, plan: LatentPlan, cu_seqlens, past_lens, scale, window, out):
-    """Tensor-memory attention of the plan's requests on expanded keys and values; writes their rows of out [T, >= H * vdim]."""
+def latent_attend_expanded(proj, shape, lat, kv, plan: LatentPlan, cu_seqlens, past_lens, scale, window, out, sinks=None, gate=None):
+    """Tensor-memory attention of the plan's requests on expanded keys and values; writes their rows of out [T, >= H * vdim], times the sigmoid
+    of gate [T, H * vdim] where one is given (rows of whole 16-byte pieces)."""
     _lib.check(_lib.lib().ogb_attention_tc_latent(_ptr(proj), proj.stride(0), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), shape.R, plan.rows,
                                                  _ptr(cu_seqlens), _ptr(past_lens), _ptr(plan.row_base), _ptr(plan.first_kv), _ptr(out), out.stride(0),
-                                                 float(scale), int(window), past_lens.shape[0], plan.max_q_len, shape.H, shape.dim, shape.rot,
+                                                 float(scale), int(window), _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                                 past_lens.shape[0], plan.max_q_len, shape.H, shape.dim, shape.rot,
                                                  shape.vdim, workspace(proj.device).status, _stream()), "attention_tc_latent")
     return out
 
 
-def latent_attention_long(proj, shape, w_ukv, cache, plan: LatentPlan, cu_seqlens, past_lens, block_table, block_size, scale, window, out):
+def latent_attention_long(proj, shape, w_ukv, cache, plan: LatentPlan, cu_seqlens, past_lens, block_table, block_size, scale, window, out, sinks=None,
+                          gate=None):
     """The long requests of a step (plan): their visible latents are gathered, expanded to keys and values, and attended on the tensor
     cores.  Writes the requests' rows of out [T, >= H * vdim]."""
     lat, kv = latent_expand(shape, w_ukv, cache, plan, block_table, block_size)
-    return latent_attend_expanded(proj, shape, lat, kv, plan, cu_seqlens, past_lens, scale, window, out)
+    return latent_attend_expanded(proj, shape, lat, kv, plan, cu_seqlens, past_lens, scale, window, out, sinks, gate)
 
 
 # ------------------------------------------------------------------------------------------ logits processing

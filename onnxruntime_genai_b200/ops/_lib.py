@@ -31,7 +31,21 @@ class LatentShape(ctypes.Structure):
 
 class AttnLayer(ctypes.Structure):
     """OgbAttnLayer of csrc/kernels.h: an attention layer with sizes and a mask of its own."""
-    _fields_ = [(n, c_int) for n in ("Hq", "Hkv", "dk", "dv", "window", "chunk", "gate_stride")] + [("scale", c_float), ("sinks", _P), ("gate", _P)]
+    _fields_ = ([(n, c_int) for n in ("Hq", "Hkv", "dk", "dv", "window", "chunk", "gate_stride")] + [("scale", c_float), ("sinks", _P), ("gate", _P)] +
+                [(n, c_int) for n in ("gate_wide", "maps", "raw")] + [("softcap", c_float)])
+
+
+class TanhNorm(ctypes.Structure):
+    """OgbTanhNorm of csrc/kernels.h: a sum into the residual stream and the tanh norm of the result."""
+    _fields_ = ([(n, _P) for n in ("h_in", "h_out", "y", "y2", "inv_pos", "topk_w", "first", "step", "w", "b", "x", "rows")] +
+                [(n, c_int) for n in ("ldy", "ldy2", "k", "n_rows", "H", "fp32")] + [("alpha", c_float)])
+
+
+class Bigram(ctypes.Structure):
+    """OgbBigram of csrc/kernels.h: token embedding with rows hashed from (previous token, token)."""
+    _fields_ = ([(n, _P) for n in ("ids", "slots", "cu_seqlens", "past_lens", "block_table", "tokens")] +
+                [(n, c_int) for n in ("table_cols", "block_size", "B", "T", "H", "vocab", "buckets", "fp32")] +
+                [("mul_prev", c_longlong), ("mul_cur", c_longlong), ("scale", c_float)])
 
 
 _LS = ctypes.POINTER(LatentShape)
@@ -62,7 +76,7 @@ _SIGS = {
                                  _P, c_int, c_int, c_int, _P, _P, _P]),
     "ogb_moe_fp4_reads_row_map": (c_int, [c_int, c_int, c_int]),
     "ogb_collective": (c_int, [c_int, _P, _P, _P, c_longlong, c_int, _P, c_int, _P]),
-    "ogb_moe_topk": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P]),
+    "ogb_moe_topk": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P]),
     "ogb_moe_max_tiles": (c_int, [c_int, c_int, c_int]),
     "ogb_moe_sort": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P]),
     "ogb_moe_combine": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_int, _P, c_int, _P, c_int, _P]),
@@ -79,30 +93,35 @@ _SIGS = {
     "ogb_causal_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_causal_conv_rows": (c_int, [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P]),
-    "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_int, _P]),
+    "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, _P]),
     "ogb_moe_gemm_simt": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P]),
     "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_float, _P]),
     "ogb_add_normed": (c_int, [_P, _P, c_int, c_int, _P, c_float, _P, _P, _P, c_int, c_int, c_int, _P]),
-    "ogb_qkv_prep": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, _P]),
+    "ogb_qkv_prep": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, _P]),
     "ogb_expert_act": (c_int, [_P, _P, c_longlong, c_int, c_int, c_float, c_float, c_int, _P]),
     "ogb_attention_mixed_supported": (c_int, [c_int, c_int]),
     "ogb_attention_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P,
                                     _P, c_int]),
     "ogb_attention_tc_mixed_supported": (c_int, [c_int, c_int, c_int, c_int]),
-    "ogb_attention_tc_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, _P]),
-    "ogb_attention_simt": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P]),
+    "ogb_attention_tc_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P,
+                                       c_longlong, _P, _P]),
+    "ogb_attention_simt": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, _P, c_longlong, c_int, _P]),
+    "ogb_attention_diff_merge": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, _P, c_int, _P, c_int, c_int, _P]),
+    "ogb_add_tanh_norm": (c_int, [ctypes.POINTER(TanhNorm), _P]),
+    "ogb_embedding_bigram": (c_int, [ctypes.POINTER(Bigram), _P, _P, _P, _P]),
     "ogb_norm_stream": (c_int, [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P]),
     "ogb_act_mul_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),
-    "ogb_latent_prep": (c_int, [_P, c_int, _LS, _P, c_float, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P]),
+    "ogb_latent_prep": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, _P, _LS, _P, c_float, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P]),
+    "ogb_gate_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, _P]),
     "ogb_latent_mma_supported": (c_int, [_LS]),
     "ogb_latent_rows_per_tile": (c_int, [c_int, c_int]),
     "ogb_latent_scratch_bytes": (c_longlong, [c_int, c_int, c_int]),
-    "ogb_latent_attention": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, c_int,
+    "ogb_latent_attention": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, _P, c_int, c_int, c_int, c_int, c_int,
                                      _P, c_longlong, _P, _P, _P]),
-    "ogb_latent_attention_simt": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P]),
+    "ogb_latent_attention_simt": (c_int, [_P, _P, c_int, _LS, _P, c_int, _P, _P, _P, c_int, c_int, _P, c_float, c_int, _P, c_int, c_int, c_int, c_int, _P]),
     "ogb_latent_gather": (c_int, [_P, c_int, _P, c_int, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P, c_int, _P]),
     "ogb_attention_tc_latent_supported": (c_int, [c_int, c_int, c_int]),
-    "ogb_attention_tc_latent": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_float, c_int, c_int, c_int, c_int,
+    "ogb_attention_tc_latent": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_float, c_int, _P, _P, c_int, c_int, c_int, c_int,
                                         c_int, c_int, c_int, _P, _P]),
     "ogb_short_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, _P]),
     "ogb_decode_advance": (c_int, [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),

@@ -19,6 +19,35 @@ def embedding(ids, table, scale=1.0):
     return out
 
 
+def embedding_bigram(ids, table, scale, bigram, spec, tokens, slots, positions, cu_seqlens, past_lens, block_table, block_size):
+    cu, ids_ = cu_seqlens.tolist(), ids.tolist()
+    rows = []
+    for b in range(past_lens.shape[0]):
+        for t in range(cu[b], cu[b + 1]):
+            at = int(past_lens[b]) + t - cu[b]
+            if at == 0:
+                rows.append(spec["buckets"])
+                continue
+            q = at - 1
+            prev = ids_[t - 1] if t > cu[b] else int(tokens[int(block_table[b, q // block_size]) * block_size + q % block_size])
+            rows.append((prev * spec["mul_prev"] + ids_[t] * spec["mul_cur"]) % spec["buckets"])
+    ok = slots >= 0
+    tokens[slots[ok].long()] = ids[ok]
+    return table[ids.long()].float() * scale + bigram[torch.tensor(rows, dtype=torch.long)].float()
+
+
+def add_tanh_norm(h, y, norm, dtype, first=None, step=None, rows=None, out=None):
+    n = h
+    for t in (y, first, step):
+        if t is not None:
+            n = n + t.float()
+    if out is not None:
+        out.copy_(n)
+    if rows is not None:
+        n = n[rows.long()]
+    return (torch.tanh(norm.alpha * n) * norm.weight + norm.bias).to(dtype)
+
+
 def norm(x, weight, eps, residual=None, bias=None, layernorm=False):
     h = x.float()
     new_res = None
@@ -200,10 +229,20 @@ def kv8_load(cache, Hkv, D):
 
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                    window=0, sinks=None, softcap=0.0, vdim=None, chunk=0, gate=None):
+                    window=0, sinks=None, softcap=0.0, vdim=None, chunk=0, gate=None, maps=1, diff=None):
     """q: [T, >=Hq*D] (only the first Hq*D columns are read).  vdim: width of a value head (None: D).  chunk > 0: position p sees the keys
-    from p // chunk * chunk on.  gate [T, Hq]: each head's output is multiplied by its sigmoid.  Returns [T, Hq*vdim]."""
+    from p // chunk * chunk on.  gate [T, Hq]: each head's output is multiplied by its sigmoid ([T, Hq*vdim]: each column).  Returns [T, Hq*vdim].
+    maps = 2: differential attention (see ops.paged_attention), returns [T, Hq/2*vdim]."""
     T, DV = q.shape[0], vdim or D
+    if maps == 2:
+        lam, post, eps, cols = diff
+        slots, d, H = v_cache.shape[0], D // 2, Hq // 2
+        qq, kk = q[:, :Hq * d].float().view(T, H, 2, d), k_cache.view(slots, Hkv, 2, d)
+        a = [paged_attention(qq[:, :, m].reshape(T, H * d), kk[:, :, m].contiguous(), v_cache, cu_seqlens, past_lens, block_table, block_size, H, Hkv, d,
+                             scale, window, None, softcap, DV, chunk) for m in (0, 1)]
+        o = (a[0] - lam * a[1]).view(T, H, DV)
+        o = o * torch.rsqrt(o[:, :, :cols].pow(2).mean(-1, keepdim=True) + eps) * post
+        return (o.reshape(T, -1) * (1.0 if gate is None else torch.sigmoid(gate.float()))).to(q.dtype)
     out = torch.zeros(T, Hq * DV, dtype=q.dtype, device=q.device)
     if k_cache.dtype == torch.int8:
         kc, vc = kv8_load(k_cache, Hkv, D), kv8_load(v_cache, Hkv, D)
@@ -245,7 +284,8 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
             p = torch.softmax(s, dim=-1)
         o = torch.einsum("hqk,khd->qhd", p, v)
         if gate is not None:
-            o = o * torch.sigmoid(gate[t0:t1].float())[:, :, None]
+            g = torch.sigmoid(gate[t0:t1].float())
+            o = o * (g[:, :, None] if gate.shape[1] == Hq else g.view(n, Hq, DV))
         out[t0:t1] = o.reshape(n, Hq * DV).to(q.dtype)
     return out
 
@@ -395,9 +435,9 @@ def head_project(x, w, heads, a_cols):
     return torch.cat([x[:, h * a_cols:h * a_cols + K].float() @ w[h * N:(h + 1) * N].float().t() for h in range(heads)], 1).to(x.dtype)
 
 
-def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache):
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv):
     T, nq, nk = proj.shape[0], Hq * key_row, Hkv * key_row
-    q, k, v = proj[:, :nq].view(T, Hq, key_row), proj[:, nq:nq + nk].view(T, Hkv, key_row), proj[:, nq + nk:nq + nk + Hkv * value_row]
+    q, k, v = proj[:, :nq].view(T, Hq, key_row), proj[:, nq:nq + nk].view(T, Hkv, key_row), proj[:, nq + nk:nq + nk + Hv * value_row]
     pos = positions.long().clamp(0, cos.shape[0] - 1) if cos is not None else None
 
     def prepared(x, w):
@@ -409,8 +449,8 @@ def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, po
     q.copy_(prepared(q, q_norm_w).to(proj.dtype))
     ok = slots >= 0
     at = slots[ok].long()
-    k_cache[at] = prepared(k, k_norm_w)[ok].to(k_cache.dtype)
-    v_cache[at] = v.view(T, Hkv, value_row)[ok].to(v_cache.dtype)
+    k_cache.view(-1, Hkv, key_row)[at] = prepared(k, k_norm_w)[ok].to(k_cache.dtype)
+    v_cache.view(-1, Hv, value_row)[at] = v.view(T, Hv, value_row)[ok].to(v_cache.dtype)
     return proj
 
 
@@ -420,22 +460,27 @@ def add_normed(h, y, weight, eps):
     return h.add_(y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight)
 
 
-def latent_prep(proj, shape, norm_w, eps, positions, cos, sin, slots, cache):
-    T, H, d, r, R = proj.shape[0], shape.H, shape.dim, shape.rot, shape.R
-    q, down = proj[:, :H * (d + r)].view(T, H, d + r), proj[:, H * (d + r):H * (d + r) + R + r]
-    c = down[:, :R].float()
-    c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * norm_w.float()
-    kr, qr = down[:, None, R:].float(), q[:, :, d:].float()
-    if cos is not None and shape.rot_dims:
+def latent_prep_parts(shape, eps, positions, cos, sin, q, down, norm_w, slots, cache, cq, cq_w):
+    H, d, r, R = shape.H, shape.dim, shape.rot, shape.R
+    unit = lambda x, w: x.float() * torch.rsqrt(x.float().pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+    def turned(x):
+        if cos is None or not shape.rot_dims:
+            return x.float()
         pos = positions.long().clamp(0, cos.shape[0] - 1)
-        kr, qr = (_rotate(t, cos[pos], sin[pos], shape.rot_dims, False) for t in (kr, qr))
-    q[:, :, d:] = qr.to(proj.dtype)
-    ok = slots >= 0
-    cache[slots[ok].long(), :R + r] = torch.cat([c, kr[:, 0]], 1)[ok].to(cache.dtype)
-    return proj
+        return _rotate(x.float(), cos[pos], sin[pos], shape.rot_dims, False)
+    if q is not None:
+        for h in range(H):
+            part = q[:, h * (d + r) + d:(h + 1) * (d + r)]
+            part.copy_(turned(part[:, None])[:, 0].to(q.dtype))
+    if cq is not None:
+        cq.copy_(unit(cq, cq_w).to(cq.dtype))
+    if down is not None:
+        ok = slots >= 0
+        cache[slots[ok].long(), :R + r] = torch.cat([unit(down[:, :R], norm_w), turned(down[:, None, R:R + r])[:, 0]], 1)[ok].to(cache.dtype)
 
 
-def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0):
+def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_table, block_size, scale, window=0, sinks=None):
     T, H, d, r, R = qlat.shape[0], shape.H, shape.dim, shape.rot, shape.R
     out = torch.zeros_like(qlat)
     q = torch.cat([qlat.view(T, H, R).float(), proj[:, :H * (d + r)].view(T, H, d + r)[:, :, d:].float()], -1)
@@ -451,6 +496,9 @@ def latent_attention(qlat, proj, shape, cache, cu_seqlens, past_lens, block_tabl
         vis = pos[None] <= qpos[:, None]
         if window and window > 0:
             vis = vis & (pos[None] > qpos[:, None] - window)
-        p = torch.softmax(s.masked_fill(~vis[None], float("-inf")), -1)
+        s = s.masked_fill(~vis[None], float("-inf"))
+        if sinks is not None:
+            s = torch.cat([s, sinks.float().view(H, 1, 1).expand(H, t1 - t0, 1)], -1)
+        p = torch.softmax(s, -1)[..., :len(pos)]
         out[t0:t1] = torch.einsum("hqk,kd->qhd", p, rows[:, :R]).reshape(t1 - t0, H * R).to(out.dtype)
     return out

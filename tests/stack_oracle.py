@@ -1,6 +1,6 @@
 """A slow, plain restatement of declared-stack decoders (gated-delta and latent-attention mixers in parallel blocks; chunked attention
-with sinks and routed experts in blocks whose norms follow the sub-layers), one function per mechanism, token by token where the
-mechanism is a recurrence.  It shares no code with the package: the tests compare the
+with sinks and routed experts in blocks whose norms follow the sub-layers; soft-capped, differential and query-compressed latent attention with
+output gates in pre-norm blocks that run several times), one function per mechanism, token by token where the mechanism is a recurrence.  It shares no code with the package: the tests compare the
 runtime against it.  Weights come as a dictionary of tensors under the checkpoint's names; all math runs in `dtype` (float64 by
 default).  A whole sequence is evaluated at once, from its first token: there is no cache here."""
 import math
@@ -86,6 +86,8 @@ def rotary_frequencies(rot):
         return f, 1.0
     if "low" in s:
         return [wavelength_scaled(fi, s) for fi in f], 1.0
+    if "original" not in s:
+        return [fi / s["factor"] for fi in f], 1.0
 
     def turns(t):
         return d * math.log(s["original"] / (2 * math.pi * t)) / (2 * math.log(base))
@@ -108,6 +110,20 @@ def rotate(x, rot):
         c, s = (torch.cos(pos * f[i]) * amp).to(x.dtype), (torch.sin(pos * f[i]) * amp).to(x.dtype)
         u, v = x[:, :, i], x[:, :, i + half]
         y[:, :, i], y[:, :, i + half] = u * c - v * s, v * c + u * s
+    return y
+
+
+def rotate_neighbours(x, rot):
+    """x [T, heads, >= dims]: pairs (2 i, 2 i + 1) of the first dims entries turn with the position."""
+    if not rot:
+        return x
+    f, amp = rotary_frequencies(rot)
+    y = x.clone()
+    for t in range(x.shape[0]):
+        for i, fi in enumerate(f):
+            c, s = math.cos(t * fi) * amp, math.sin(t * fi) * amp
+            u, v = x[t, :, 2 * i], x[t, :, 2 * i + 1]
+            y[t, :, 2 * i], y[t, :, 2 * i + 1] = u * c - v * s, v * c + u * s
     return y
 
 
@@ -195,6 +211,86 @@ def feed_forward(x, w, p):
     return (torch.relu(x @ w[p + "gate"].T) * (x @ w[p + "up"].T)) @ w[p + "down"].T
 
 
+def bounded_norm(x, w, p):
+    """Norm without statistics: a scaled hyperbolic tangent of every entry, weight and bias."""
+    return torch.tanh(w[p + ".alpha"] * x) * w[p] + w[p + ".b"]
+
+
+def bigram_rows(tokens, buckets, mul_prev, mul_cur):
+    """Row of every token in a table over hashed pairs (previous token, token); a first token has the row behind the buckets."""
+    return [buckets if t == 0 else (int(tokens[t - 1]) * mul_prev + int(tokens[t]) * mul_cur) % buckets for t in range(len(tokens))]
+
+
+def capped(s, cap):
+    return cap * torch.tanh(s / cap) if cap else s
+
+
+def softmax_attention(q, k, v, ok, scale, cap=0.0):
+    """q [T, H, d], k [T, G, d], v [T, G, dv] -> [T, H, dv]."""
+    rep = q.shape[1] // k.shape[1]
+    out = torch.zeros(q.shape[0], q.shape[1], v.shape[2], dtype=q.dtype)
+    for h in range(q.shape[1]):
+        s = capped(q[:, h] @ k[:, h // rep].T * scale, cap)
+        out[:, h] = torch.softmax(s.masked_fill(~ok, -math.inf), -1) @ v[:, h // rep]
+    return out
+
+
+def gated_output(o, x, w, p):
+    """Concatenated heads, element by element times the sigmoid of a projection of the mixer's input; output map."""
+    return (o.reshape(o.shape[0], -1) * torch.sigmoid(x @ w[p + "g"].T)) @ w[p + "o"].T
+
+
+def capped_mixer(x, w, p, m, eps):
+    T, H, G, d, dv = x.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k, v = ((x @ w[p + n].T + w[p + n + ".b"]).view(T, h, c) for n, h, c in (("q", H, d), ("k", G, d), ("v", G, dv)))
+    q, k = rotate_neighbours(q, m.get("rot")), rotate_neighbours(k, m.get("rot"))
+    return gated_output(softmax_attention(q, k, v, visible(T, m.get("mask")), m["scale"], m.get("softcap")), x, w, p)
+
+
+def difference_factor(w, p, diff):
+    return torch.exp((w[p + "lq1"] * w[p + "lk1"]).sum()) - torch.exp((w[p + "lq2"] * w[p + "lk2"]).sum()) + diff
+
+
+def difference_of_maps(a1, a2, factor, diff, eps):
+    """a1, a2 [T, H, dv]: what two attention maps make of the same values."""
+    o = a1 - factor * a2
+    return o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * (1 - diff)
+
+
+def differential_mixer(x, w, p, m, eps):
+    T, H, G, d, dv = x.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = (x @ w[p + "q"].T + w[p + "q.b"]).view(T, H, 2, d)
+    k = (x @ w[p + "k"].T + w[p + "k.b"]).view(T, G, 2, d)
+    v = (x @ w[p + "v"].T + w[p + "v.b"]).view(T, G, dv)
+    ok = visible(T, m.get("mask"))
+    a = [softmax_attention(rotate(q[:, :, i], m.get("rot")), rotate(k[:, :, i], m.get("rot")), v, ok, m["scale"]) for i in (0, 1)]
+    return gated_output(difference_of_maps(*a, difference_factor(w, p, m["diff"]), m["diff"], eps), x, w, p)
+
+
+def compressed_latent_mixer(x, w, p, m, eps):
+    """Latent attention whose queries come out of a normed latent of their own, with sinks and an output gate."""
+    T, H, d, r, dv, R = x.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    q = (rms_norm(x @ w[p + "dq"].T, w[p + "dq.norm"], eps) @ w[p + "uq"].T).view(T, H, d + r)
+    down = x @ w[p + "dkv"].T
+    c = rms_norm(down[:, :R], w[p + "dkv.norm"], eps)
+    kr = rotate(down[:, R:].view(T, 1, r), m.get("rot"))
+    q = torch.cat([q[:, :, :d], rotate(q[:, :, d:], m.get("rot"))], -1)
+    k = torch.cat([(c @ w[p + "uk"].T).view(T, H, d), kr.expand(T, H, r)], -1)
+    o = sink_attention(q, k, (c @ w[p + "uv"].T).view(T, H, dv), visible(T, m.get("mask")), m["scale"], w[p + "sink"])
+    return gated_output(o, x, w, p)
+
+
+def selected_experts(x, w, p, m):
+    """Each token: the `top` experts of largest router logit, weighted by a softmax over these logits; a shared expert for every token."""
+    z = x @ w[p + "router"].T
+    out = clamped_expert(x, w, p + "shared.", m["shared"]["limit"]) if m.get("shared") else torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        chosen = torch.argsort(z[t], descending=True)[:m["router"]["top"]]
+        for e, share in zip(chosen.tolist(), torch.softmax(z[t, chosen], -1)):
+            out[t] = out[t] + share * clamped_expert(x[t:t + 1], w, f"{p}e{e}.", m["expert"]["limit"])[0]
+    return out
+
+
 # ------------------------------------------------------------------------------------------------ the stack
 MIXERS = {"delta": delta_mixer, "latent_attention": latent_mixer, "attention": attention_mixer}
 FEED_FORWARDS = {"dense": gelu_feed_forward, "moe": routed_experts}
@@ -217,8 +313,45 @@ def output_normed_block(x, w, p, e, eps, cfg):
     return x
 
 
+GATED_MIXERS = {"attention": capped_mixer, "attention_2": differential_mixer, "latent_attention": compressed_latent_mixer}
+
+
+def bounded_norm_block(x, w, p, e, eps):
+    x = x + GATED_MIXERS[e["type"]](bounded_norm(x, w, p + "norm1"), w, p + "mix.", e["mixer"], eps)
+    if e.get("mlp"):
+        x = x + selected_experts(bounded_norm(x, w, p + "norm2"), w, p + "mlp.", e["mlp"])
+    return x
+
+
+def passes(cfg):
+    """(layer, pass that starts with it or None) in the order in which the layers run."""
+    n, loop = len(cfg["layers"]), cfg.get("loop")
+    if not loop:
+        return [(i, None) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    return [(i, None) for i in range(a)] + [(i, t if i == a else None) for t in range(loop["times"]) for i in range(a, b)] + [(i, None) for i in range(b, n)]
+
+
+def looped_forward(cfg, weights, tokens, dtype=torch.float64):
+    """stack_forward of stacks with a hashed-pair embedding, bounded norms and layers that run several times."""
+    w = {k: v.to(dtype) for k, v in weights.items()}
+    emb = cfg["embedding"]
+    x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * emb["scale"]
+    if emb.get("bigram"):
+        x = x + w["bigram"][bigram_rows(tokens, **emb["bigram"])]
+    first, streams = x, []
+    for i, t in passes(cfg):
+        if t is not None:
+            x = x + (first if t > 0 else 0) + w["loop.step"][t]
+        x = bounded_norm_block(x, w, f"l{i}.", cfg["layers"][i], cfg["norm"]["eps"])
+        streams.append(x)
+    return bounded_norm(x, w, "final.norm") @ w["head"].T, torch.stack(streams)
+
+
 def stack_forward(cfg, weights, tokens, dtype=torch.float64):
     """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
+    if cfg["architecture"] == "Sugelix":
+        return looped_forward(cfg, weights, tokens, dtype)
     w = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * cfg.get("embedding", {}).get("scale", 1.0)
