@@ -1,9 +1,11 @@
 """Prefill and decode throughput of a declared stack beside the closest other model of the framework at equal size.  Luzatar: the
 gated-delta-net + full-attention hybrid (Qwen3.5 style) with the same width, feed-forward, layer count, delta layers and attention heads.
 Zevopel: Qwen3-style dense layers (normed query and key heads), and gpt-oss-style layers with bf16 experts (sinks, clamped experts), each
-with the same width, heads and feed-forwards; the chunks are as long as the context, so both attend to the same keys.  Random weights drawn
+with the same width, heads and feed-forwards; the chunks are as long as the context, so both attend to the same keys.  Sugelix: gpt-oss-style
+layers again, as many as the design runs, with the same width, head count, key and value sizes and as many experts per token (one of the
+design's is the shared one); soft-capped scores on both sides where the design's layers have them.  Random weights drawn
 on the device; CUDA events around whole decoder forwards (decode steps replay a CUDA graph); the weights and caches of a step are larger
-than L2.  Reached through `python bench.py --design luzatar | zevopel`."""
+than L2.  Reached through `python bench.py --design luzatar | zevopel | sugelix`."""
 import json
 import os
 import shutil
@@ -22,6 +24,14 @@ ZEVOPEL_SIZES = {
     "2k dense": dict(width=2048, ff=6144, layers=16, heads=16, kv=4, dim=128, vocab=65536),
     "4k dense": dict(width=4096, ff=12288, layers=8, heads=32, kv=8, dim=128, vocab=65536),
     "2.9k experts": dict(width=2880, ff=2880, layers=8, heads=64, kv=8, dim=64, vocab=65536, experts=32, top=4),
+}
+SUGELIX_SIZES = {
+    # name: the layers' mixers ("a" soft-capped, "d" differential, "l" latent), how often the stack runs, width, one expert's feed-forward, heads,
+    # kv heads, head size (of both maps together where there are two), experts (one more is shared), experts per token with the shared one
+    "2.9k capped": dict(mixers="aaaaaaaa", times=1, width=2880, ff=2880, heads=32, kv=8, dim=128, vocab=65536, experts=32, top=4, softcap=50.0),
+    "2.9k differential": dict(mixers="dddddddd", times=1, width=2880, ff=2880, heads=32, kv=8, dim=128, vocab=65536, experts=32, top=4),
+    "2.9k latent": dict(mixers="llllllll", times=1, width=2880, ff=2880, heads=32, kv=8, dim=128, vocab=65536, experts=32, top=4),
+    "2k mixed, twice": dict(mixers="adal", times=2, width=2048, ff=1024, heads=16, kv=4, dim=128, vocab=65536, experts=64, top=6, softcap=50.0),
 }
 PREFILL = [(1, 4096), (8, 1024)]
 DECODE = [(1, 2048), (16, 2048), (64, 2048), (256, 1024)]
@@ -77,7 +87,38 @@ def closest_to_zevopel_dir(z, path):
     return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
 
 
-DESIGNS = {"luzatar": (SIZES, luzatar_dir, "hybrid", hybrid_dir), "zevopel": (ZEVOPEL_SIZES, zevopel_dir, "closest", closest_to_zevopel_dir)}
+def sugelix_dir(z, path):
+    d, mlp = z["dim"], dict(kind="moe", expert=dict(ff=z["ff"], limit=7.0), shared=dict(ff=z["ff"], limit=7.0), router=dict(experts=z["experts"], top=z["top"] - 1))
+    kinds = {"a": ("attention", dict(heads=z["heads"], kv_heads=z["kv"], dim=d, vdim=d, scale=d ** -0.5, softcap=z.get("softcap"), rot=dict(base=5e5, dims=d))),
+             "d": ("attention_2", dict(heads=z["heads"], kv_heads=z["kv"], dim=d // 2, vdim=d, scale=(d // 2) ** -0.5, diff=0.5, mask=dict(size=8192),
+                                       rot=dict(base=5e5, dims=d // 2, scaling=dict(factor=8.0)))),
+             "l": ("latent_attention", dict(heads=z["heads"], dim=d, rot_dim=64, vdim=d, kv_rank=512, q_rank=1024, scale=(d + 64) ** -0.5, mask=dict(size=8192),
+                                            rot=dict(base=5e5, dims=64)))}
+    cfg = dict(architecture="Sugelix", layers=[dict(type=kinds[m][0], mixer=kinds[m][1], mlp=mlp) for m in z["mixers"]], norm=dict(eps=1e-6), vocab=z["vocab"],
+               width=z["width"], embedding=dict(scale=z["width"] ** 0.5, bigram=dict(buckets=50021, mul_prev=31, mul_cur=17)))
+    if z["times"] > 1:
+        cfg["loop"] = dict(start=0, stop=len(z["mixers"]), times=z["times"])
+    os.makedirs(os.path.join(path, "src"), exist_ok=True)
+    with open(os.path.join(path, "src", "config.json"), "w") as f:
+        json.dump(cfg, f)
+    from onnxruntime_genai_b200.models.builder import create_model
+    return create_model(os.path.join(path, "src"), os.path.join(path, "model"), "bf16", "cuda", {"synthetic_weights": 1, "context_length": 8192})
+
+
+def closest_to_sugelix_dir(z, path):
+    from onnxruntime_genai_b200.models.arch import ArchConfig
+    from onnxruntime_genai_b200.models.builder import export_model
+    a = ArchConfig(model_type="gptoss", vocab_size=z["vocab"], hidden_size=z["width"], num_layers=len(z["mixers"]) * z["times"], num_heads=z["heads"],
+                   num_kv_heads=z["kv"], head_dim=z["dim"], intermediate_size=z["ff"], context_length=8192, rope_theta=5e5, attn_bias=True, o_bias=True,
+                   mlp_bias=True, num_experts=z["experts"] + 1, experts_per_token=z["top"], bos_token_id=0, eos_token_id=1, pad_token_id=0)
+    if z.get("softcap"):
+        a.softcap = z["softcap"]
+    else:
+        a.attn_sinks = True
+    return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
+
+
+DESIGNS = {"sugelix": (SUGELIX_SIZES, sugelix_dir, "closest", closest_to_sugelix_dir), "luzatar": (SIZES, luzatar_dir, "hybrid", hybrid_dir), "zevopel": (ZEVOPEL_SIZES, zevopel_dir, "closest", closest_to_zevopel_dir)}
 
 
 def _step(model, lens):

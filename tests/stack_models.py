@@ -41,6 +41,37 @@ def output_normed_stack(layers, vocab=90, width=72, eps=3e-5, residual_mult=0.6,
                 embedding=dict(scale=embed_scale))
 
 
+def experts(ff=40, n=6, top=2, limit=0.8, shared_ff=None, shared_limit=None):
+    """Routed experts; shared_ff: width of a shared expert (None: as wide as the others, 0: none)."""
+    mlp = dict(kind="moe", expert=dict(ff=ff, limit=limit), router=dict(experts=n, top=top))
+    if shared_ff != 0:
+        mlp["shared"] = dict(ff=shared_ff or ff, limit=shared_limit or limit)
+    return mlp
+
+
+def capped(heads=4, kv_heads=2, dim=24, vdim=16, scale=0.3, softcap=6.0, dims=16, base=3000.0, mlp=experts()):
+    return dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, softcap=softcap, rot=dict(base=base, dims=dims)),
+                mlp=mlp)
+
+
+def differential(heads=4, kv_heads=2, dim=16, vdim=24, window=20, scale=0.35, diff=0.4, dims=12, base=900.0, factor=3.0, mlp=experts()):
+    return dict(type="attention_2", mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, diff=diff, mask=dict(size=window),
+                                               rot=dict(base=base, dims=dims, scaling=dict(factor=factor))), mlp=mlp)
+
+
+def compressed_latent(heads=3, dim=40, rot_dim=8, vdim=24, kv_rank=48, q_rank=56, window=25, scale=0.17, base=5000.0, mlp=experts()):
+    return dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, q_rank=q_rank, scale=scale,
+                                                    mask=dict(size=window) if window else None, rot=dict(base=base, dims=rot_dim)), mlp=mlp)
+
+
+def looped_stack(layers, vocab=90, width=72, eps=3e-5, embed_scale=1.7, buckets=53, mul_prev=31, mul_cur=7, loop=(0, None, 2)):
+    cfg = dict(architecture="Sugelix", layers=copy.deepcopy(layers), norm=dict(eps=eps), vocab=vocab, width=width,
+               embedding=dict(scale=embed_scale, bigram=dict(buckets=buckets, mul_prev=mul_prev, mul_cur=mul_cur)))
+    if loop:
+        cfg["loop"] = dict(start=loop[0], stop=len(layers) if loop[1] is None else loop[1], times=loop[2])
+    return cfg
+
+
 def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
     """Random weights of useful magnitude (projections near unit gain, decays between slow and fast).  clear_routes: a router reads one
     column of the stream per expert, these columns hold well separated values in every embedding row, and no sub-layer writes them."""
@@ -49,9 +80,15 @@ def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
     out = {}
     for name, shape in stack_weight_shapes(from_stack_config(cfg)).items():
         x = torch.randn(shape, generator=g)
-        if cfg["architecture"] == "Zevopel" and (name == "final.norm" or name.endswith(("norm1", "norm2"))):
+        if name.endswith("alpha"):
+            x = 0.35 + 0.1 * torch.rand((), generator=g)
+        elif name == "bigram" or name == "loop.step":
+            x = 0.7 * x
+        elif name.endswith(("lq1", "lk1", "lq2", "lk2")):
+            x = x / shape[0] ** 0.5                       # a factor well away from its starting value
+        elif cfg["architecture"] == "Zevopel" and (name == "final.norm" or name.endswith(("norm1", "norm2"))):
             x = 0.2 * x                                   # stored around zero
-        elif name.endswith(("norm", "norm1", "ls1", "ls2")):
+        elif name.endswith(("norm", "norm1", "norm2", "ls1", "ls2")):
             x = 1.0 + 0.2 * x
         elif name.endswith("router"):
             x = 2.0 * x / shape[1] ** 0.5
@@ -69,7 +106,24 @@ def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
             x = gain * x / shape[1] ** 0.5
         out[name] = x.to(dtype)
     most = max([e["mlp"]["router"]["experts"] for e in cfg["layers"] if (e.get("mlp") or {}).get("kind") == "moe"], default=0)
-    if clear_routes and most:
+    if clear_routes and most and cfg["architecture"] == "Sugelix":
+        assert most < cfg["width"]
+        turns = (cfg.get("loop") or dict(times=1))["times"]
+        for v in range(cfg["vocab"]):
+            out["embed"][v, :most] = ((torch.randperm(most, generator=g).float() / most * 3 - 1.5) / turns / cfg["embedding"]["scale"]).to(dtype)
+        out["bigram"][:, :most] = 0
+        if "loop.step" in out:
+            out["loop.step"][:, :most] = 0
+        for name, x in out.items():
+            if name.endswith(("mix.o", ".down")):
+                x[:most] = 0
+            elif name.endswith("norm2"):
+                x[:most] = 1
+            elif name.endswith("norm2.b"):
+                x[:most] = 0
+            elif name.endswith("router"):
+                x.zero_()[:, :most].fill_diagonal_(3.0)
+    elif clear_routes and most:
         assert most < cfg["width"]
         for v in range(cfg["vocab"]):
             out["embed"][v, :most] = (torch.randperm(most, generator=g).float() / most * 3 - 1.5).to(dtype)

@@ -118,12 +118,11 @@ def rotate_neighbours(x, rot):
     if not rot:
         return x
     f, amp = rotary_frequencies(rot)
-    y = x.clone()
-    for t in range(x.shape[0]):
-        for i, fi in enumerate(f):
-            c, s = math.cos(t * fi) * amp, math.sin(t * fi) * amp
-            u, v = x[t, :, 2 * i], x[t, :, 2 * i + 1]
-            y[t, :, 2 * i], y[t, :, 2 * i + 1] = u * c - v * s, v * c + u * s
+    y, pos = x.clone(), torch.arange(x.shape[0], dtype=torch.float64)[:, None]
+    for i, fi in enumerate(f):
+        c, s = (torch.cos(pos * fi) * amp).to(x.dtype), (torch.sin(pos * fi) * amp).to(x.dtype)
+        u, v = x[:, :, 2 * i], x[:, :, 2 * i + 1]
+        y[:, :, 2 * i], y[:, :, 2 * i + 1] = u * c - v * s, v * c + u * s
     return y
 
 

@@ -14,7 +14,8 @@ from onnxruntime_genai_b200 import ops
 from onnxruntime_genai_b200.models import arch as A
 from onnxruntime_genai_b200.models import moe
 from onnxruntime_genai_b200.models.decoder import LayerWeights, PagedKVCache
-from stack_harness import BLOCK, RUNTIMES, beam_search, close, dtype_of, feed, greedy_ok, one_thread, open_engine, open_model, paged, random_tokens, rows_of, tol_of, wide_rows  # noqa: F401
+from stack_harness import (BLOCK, RUNTIMES, close, dtype_of, feed, greedy_generation, mixed_batches, one_thread, open_engine, open_model, paged,  # noqa: F401
+                           random_tokens, rewind_and_beams, rows_of, tol_of, wide_rows)
 from stack_models import chunked, output_normed_stack, weights, write
 from stack_oracle import (clamped_expert, gelu_feed_forward, rms_norm, rotary_frequencies, rotate, routed_experts, same_chunk, sink_attention, stack_forward,
                           wavelength_scaled)
@@ -354,38 +355,7 @@ def test_portions_and_single_tokens(tmp_path_factory, runtime, name, cuts):
 
 @pytest.mark.parametrize("name", list(STACKS))
 def test_mixed_batches_reuse_pages(tmp_path_factory, runtime, name):
-    """More requests than fit at once come and go through a pool that is just large enough, portions beside single tokens, requests left
-    out of some steps; every request gets the logits it gets alone."""
-    m, cfg, w = open_model(tmp_path_factory, name, runtime, STACKS[name])
-    eng = open_engine(m, blocks=26, batch=4, tokens=300)
-    rng = np.random.RandomState(5)
-    waiting = [(i, random_tokens(cfg, n, 20 + i)) for i, n in enumerate((90, 33, 120, 5, 64, 1, 77, 100, 16, 50))]
-    live, got, seen, used = [], {i: [] for i, _ in waiting}, dict(waiting), []
-    while waiting or live:
-        while waiting and len(live) < 4 and sum((len(t) + BLOCK - 1) // BLOCK for _, t, _, _ in live) + (len(waiting[0][1]) + BLOCK - 1) // BLOCK <= 26:
-            i, t = waiting.pop(0)
-            live.append([i, t, 0, og.Request(og.GeneratorParams(m))])
-        step = []
-        for e in live:
-            if len(live) > 1 and rng.rand() < 0.25:
-                continue                                    # left out of this step
-            step.append((e, min(int(rng.choice([1, 1, 2, 3, 17, 40, 70])), len(e[1]) - e[2])))
-        if not step:
-            continue
-        out = eng.run_given([(e[3], e[1][e[2]:e[2] + n], list(range(n)) if e[0] % 2 else [n - 1]) for e, n in step])
-        eng.core.check_invariants()
-        for (e, n), lg in zip(step, out):
-            got[e[0]].append((e[2], n, lg.float().cpu()))
-            e[2] += n
-        for e in [e for e in live if e[2] == len(e[1])]:
-            used += e[3]._native.blocks()
-            eng.remove_request(e[3])
-            live.remove(e)
-    assert eng.core.free_blocks == 26 and len(used) > len(set(used))      # blocks were used again
-    for i, parts in got.items():
-        want = stack_forward(cfg, w, seen[i])[0]
-        for at, n, lg in parts:
-            close(lg, want[at:at + n] if i % 2 else want[at + n - 1:at + n], 1.5 * tol_of(runtime))
+    mixed_batches(*open_model(tmp_path_factory, name, runtime, STACKS[name]), runtime)
 
 
 def test_a_request_does_not_see_the_batch_around_it(tmp_path_factory, runtime):
@@ -437,75 +407,11 @@ def test_positions_count_from_the_first_token_of_the_sequence(tmp_path_factory, 
 
 # ------------------------------------------------------------------------------------------------ generation
 def test_greedy_generation_through_generator_and_engine(tmp_path_factory, runtime):
-    m, cfg, w = open_model(tmp_path_factory, "zev_wide", runtime, WIDE)
-    tol = 0.2 if runtime[1] == "bfloat16" else 1e-3
-    prompts = [random_tokens(cfg, n, 40 + n) for n in (70, 5, 33, 1, 18)]
-    p = og.GeneratorParams(m)
-    p.set_search_options(max_length=100, do_sample=False)
-    gen = og.Generator(m, p)
-    gen.append_tokens(prompts[0].astype(np.int32).reshape(1, -1))
-    while not gen.is_done():
-        gen.generate_next_token()
-    solo = np.asarray(gen.get_sequence(0))[70:]
-    assert len(solo) == 30
-    greedy_ok(cfg, w, prompts[0], solo, tol)
-    # the scheduler: more requests than the batch holds, prompts cut by a small token budget, blocks that run short
-    eng = open_engine(m, blocks=30, batch=3, tokens=40)
-    reqs = []
-    for t in prompts:
-        gp = og.GeneratorParams(m)
-        gp.set_search_options(max_length=len(t) + 25, do_sample=False)
-        r = og.Request(gp)
-        r.add_tokens(t.astype(np.int32))
-        eng.add_request(r)
-        reqs.append(r)
-    while eng.has_pending_requests():
-        r = eng.step()
-        if r is None:
-            continue
-        while r.has_unseen_tokens():
-            r.get_unseen_token()
-        if r.is_turn_complete():
-            r.kept = r.tokens()
-            eng.remove_request(r)
-    for r, t in zip(reqs, prompts):
-        assert len(r.kept) == len(t) + 25
-        greedy_ok(cfg, w, t, r.kept[len(t):], tol)
+    greedy_generation(*open_model(tmp_path_factory, "zev_wide", runtime, WIDE), runtime)
 
 
 def test_batched_generator_rewind_and_beams(tmp_path_factory, runtime):
-    m, cfg, w = open_model(tmp_path_factory, "zev_mixed", runtime, MIXED)
-    tol = 0.2 if runtime[1] == "bfloat16" else 1e-3
-    prompt = np.stack([random_tokens(cfg, 12, 3), random_tokens(cfg, 12, 4)]).astype(np.int32)
-    p = og.GeneratorParams(m)
-    p.set_search_options(max_length=30, batch_size=2, do_sample=False)
-    gen = og.Generator(m, p)
-    gen.append_tokens(prompt)
-    while not gen.is_done():
-        gen.generate_next_token()
-    for r in range(2):
-        greedy_ok(cfg, w, prompt[r], np.asarray(gen.get_sequence(r))[12:], tol)
-    p = og.GeneratorParams(m)
-    p.set_search_options(max_length=40, do_sample=False)
-    gen = og.Generator(m, p)
-    gen.append_tokens(prompt[:1])
-    for _ in range(10):
-        gen.generate_next_token()
-    gen.rewind_to(15)
-    for _ in range(7):
-        gen.generate_next_token()
-    greedy_ok(cfg, w, prompt[0], np.asarray(gen.get_sequence(0))[12:], tol)
-    p = og.GeneratorParams(m)
-    p.set_search_options(max_length=24, num_beams=3, do_sample=False)
-    gen = og.Generator(m, p)
-    gen.append_tokens(prompt[:1])
-    while not gen.is_done():
-        gen.generate_next_token()
-    seq = np.asarray(gen.get_sequence(0))
-    lp = lambda s: float(sum(torch.log_softmax(stack_forward(cfg, w, s)[0], -1)[i, int(s[i + 1])] for i in range(11, len(s) - 1)))
-    # beams follow their own pages: a plain beam search over the restatement finds a hypothesis of the same score (16-bit rounding may pick
-    # another one where candidates are close)
-    assert abs(lp(seq) - lp(beam_search(cfg, w, prompt[0], 24, 3))) < (4.0 if runtime[1] == "bfloat16" else 2e-2)
+    rewind_and_beams(*open_model(tmp_path_factory, "zev_mixed", runtime, MIXED), runtime)
 
 
 def test_sampled_generation_is_reproducible(tmp_path_factory, runtime):
