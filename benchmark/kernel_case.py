@@ -7,6 +7,9 @@ cases: gemm_qkv gemm_o gemm_gate_up gemm_down gemm_lm_head gemm_prefill gemm_qkv
        gated_delta gated_delta_prefill mamba2_scan; latent_decode latent_absorb latent_value latent_prep latent_prefill latent_expand norm_stream
        chunk_decode chunk_prefill chunk_decode_192 chunk_prefill_192 qkv_prep add_normed add_normed_experts gemm_gate_up_gelu expert_route (Zevopel
        layers: attention with sinks and head gates, keys of 128 or 192 and values of 128 columns; norms of sub-layer outputs; not part of `all`)
+       capped_decode capped_prefill softcap_decode softcap_prefill diff_decode diff_prefill qkv_prep_plain tanh_norm tanh_norm_experts
+       embed_pairs embed latent_value_gated shared_route (Sugelix layers: soft-capped attention with a gate per column beside the older models' soft
+       cap, differential attention with two maps of 64 over values of 128 columns, sums into the stream with their tanh norm; not part of `all`)
        gemm_join (Luzatar layers at Llama-sized widths: 16 heads of 128 + 64 / 128 over a latent of 512; not part of `all`)
        (moe_*: gpt-oss-20b experts, packed MXFP4 in the fp16 form, in the bf16 form (fp4b) or bf16 weights; not part of `all`)
 
@@ -96,6 +99,15 @@ def build_case(name, T, L, tp=1):
     """Returns (fn(i), algorithmic_bytes, flops).  tp > 1: the per-rank shapes of tensor parallelism; the row-parallel
     projections then run the fused all-reduce against a world of one (protocol cost without a peer)."""
     HQ, HKV = globals()["HQ"] // tp, max(1, globals()["HKV"] // tp)
+    if name in ("embed", "embed_pairs"):
+        table, ids = _bf(65536, H), torch.randint(0, 65536, (T,), device="cuda", dtype=torch.int32)
+        if name == "embed":
+            return (lambda i: ops.embedding(ids, table)), T * H * 4, 0.0
+        spec = dict(buckets=50021, mul_prev=31, mul_cur=17)
+        pairs, tokens = _bf(50022, H), torch.zeros(T + 16, dtype=torch.int32, device="cuda")
+        ar = torch.arange(T + 1, dtype=torch.int32, device="cuda")
+        past, tab = torch.full((T,), 7, dtype=torch.int32, device="cuda"), ar[:T, None].contiguous()
+        return (lambda i: ops.embedding_bigram(ids, table, 2.0, pairs, spec, tokens, ar[:T], past, ar, past, tab, 16)), T * H * 8, 0.0
     if name in ("gemm_qkv_fused", "gemm_gate_up_fused"):
         # the decode-step fusions: RMS norm folded into the projection (+ rotary embedding and KV-cache append for QKV)
         x = _bf(T, H, std=1.0)
@@ -162,7 +174,7 @@ def build_case(name, T, L, tp=1):
         if gate_up:
             return (lambda i: ops.moe_gemm(xs, ws[i % L], plan, bias, act_kind=2, alpha=1.702, limit=7.0)), wbytes + T * k * (K + N // 2) * 2, 2.0 * T * k * N * K
         return (lambda i: ops.moe_gemm(xs, ws[i % L], plan, bias)), wbytes + T * k * (K + N) * 2, 2.0 * T * k * N * K
-    if name in ("attention_decode", "attention_prefill") or name.startswith("chunk_"):
+    if name in ("attention_decode", "attention_prefill") or name.startswith(("chunk_", "capped_", "softcap_", "diff_")):
         bs = 16
         rng = np.random.RandomState(2)
         decode = "decode" in name
@@ -206,8 +218,17 @@ def build_case(name, T, L, tp=1):
                                                   max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)), splits=ATTN_SPLITS,
                                                   order=order, min_q_len=min(q_lens), vdim=D, chunk=8192, gate=proj[:, HQ * dk:])), nbytes, \
                 flops * (dk + D) / (2 * D)
+        if name.startswith(("capped_", "diff_")):
+            maps = 2 if name.startswith("diff_") else 1      # (a key head holds both maps' 64 columns)
+            proj = _bf(Tq, 2 * HQ * D, std=1.0)
+            diff = (0.6, 0.5, 1e-6, D) if maps == 2 else None
+            return (lambda i: ops.paged_attention(proj, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ * maps, HKV, D, 1 / math.sqrt(D // maps),
+                                                  softcap=0.0 if maps == 2 else 50.0, max_q_len=max(q_lens),
+                                                  max_kv_len=max(p + q for p, q in zip(past, q_lens)), splits=ATTN_SPLITS, order=order,
+                                                  min_q_len=min(q_lens), vdim=D, gate=proj[:, HQ * D:], maps=maps, diff=diff)), \
+                nbytes + Tq * HQ * D * 2, flops * (1.5 if maps == 2 else 1.0)
         return (lambda i: ops.paged_attention(qkv, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ, HKV, D, 1 / math.sqrt(D),
-                                              max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)),
+                                              softcap=50.0 if name.startswith("softcap") else 0.0, max_q_len=max(q_lens), max_kv_len=max(p + q for p, q in zip(past, q_lens)),
                                               splits=ATTN_SPLITS, order=order)), nbytes, flops
     if name.startswith("latent_"):
         Hl, d, r, dv, R, bs = 16, 128, 64, 128, 512, 16
@@ -217,9 +238,10 @@ def build_case(name, T, L, tp=1):
         if name == "latent_absorb":
             x, ws = _bf(T, N, std=1.0), [_bf(Hl * R, d) for _ in range(L)]
             return (lambda i: ops.head_project(x, ws[i % L], Hl, d + r)), Hl * R * d * 2 + T * Hl * (d + R) * 2, 2.0 * T * Hl * d * R
-        if name == "latent_value":
+        if name in ("latent_value", "latent_value_gated"):
             x, ws = _bf(T, Hl * R, std=1.0), [_bf(Hl * dv, R) for _ in range(L)]
-            return (lambda i: ops.head_project(x, ws[i % L], Hl, R)), Hl * R * dv * 2 + T * Hl * (dv + R) * 2, 2.0 * T * Hl * dv * R
+            gate = _bf(T, Hl * dv, std=1.0) if name.endswith("gated") else None
+            return (lambda i: ops.head_project(x, ws[i % L], Hl, R, gate=gate)), Hl * R * dv * 2 + T * Hl * (dv + R) * 2, 2.0 * T * Hl * dv * R
         rng = np.random.RandomState(2)
         lens = [(0, 1024)] * (T // 1024) if prefill else [(int(p) + 64, 1) for p in rng.randint(128, 2049, size=T)]
         if prefill and T <= 4096:
@@ -261,12 +283,12 @@ def build_case(name, T, L, tp=1):
     if name == "gemm_gate_up_gelu":
         x, ws = _bf(T, H, std=1.0), [ops.interleave_gate_up(_bf(2 * I, H)) for _ in range(L)]
         return (lambda i: ops.gate_up_act(x, ws[i % L], act="gelu_tanh", interleaved=True)), 2 * I * H * 2 + T * (H + I) * 2, 4.0 * T * I * H
-    if name == "qkv_prep":
+    if name in ("qkv_prep", "qkv_prep_plain"):
         projs = [_bf(T, (HQ + 2 * HKV) * D + HQ, std=1.0) for _ in range(4)]
         pos, slots = torch.arange(T, dtype=torch.int32, device="cuda") % 4096, torch.arange(T, dtype=torch.int32, device="cuda")
         cos, sin, w = torch.randn(4096, D // 2, device="cuda"), torch.randn(4096, D // 2, device="cuda"), torch.ones(D, device="cuda")
         kc, vc = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D)
-        return (lambda i: ops.qkv_prep(projs[i % 4], HQ, HKV, D, D, D, w, w, 1e-6, pos, cos, sin, slots, kc, vc)), T * (HQ + 2 * HKV) * D * 2 * 2, 0.0
+        return (lambda i: ops.qkv_prep(projs[i % 4], HQ, HKV, D, D, D, *((w, w) if name == "qkv_prep" else (None, None)), 1e-6, pos, cos, sin, slots, kc, vc)), T * (HQ + 2 * HKV) * D * 2 * 2, 0.0
     if name in ("add_normed", "add_normed_experts"):
         hs, w = [torch.randn(T, H, device="cuda") for _ in range(4)], torch.randn(H, device="cuda")
         if name == "add_normed":
@@ -275,6 +297,17 @@ def build_case(name, T, L, tp=1):
             plan = ops.moe_route(torch.randn(T, 32, device="cuda"), 4, 1)
             y, rows = ops.PendingCombine(_bf(T * 4, H, std=1.0), plan), 4 * T
         return (lambda i: ops.add_normed(hs[i % 4], y, w, 1e-6)), rows * H * 2 + T * H * 10, 0.0
+    if name in ("tanh_norm", "tanh_norm_experts"):
+        hs, norm = [torch.randn(T, H, device="cuda") for _ in range(4)], ops.TanhNorm(torch.randn(H, device="cuda"), torch.randn(H, device="cuda"), 0.5)
+        if name == "tanh_norm":
+            y, rows = _bf(T, H, std=1.0), T
+        else:
+            plan = ops.moe_route(torch.randn(T, 32, device="cuda"), 3, 0, shared=True)
+            y, rows = ops.PendingCombine(_bf(T * 4, H, std=1.0), plan), 4 * T
+        return (lambda i: ops.add_tanh_norm(hs[i % 4], y, norm, out=hs[i % 4])), rows * H * 2 + T * H * 10, 0.0
+    if name == "shared_route":
+        logits = torch.randn(T, 32, device="cuda")
+        return (lambda i: ops.moe_route(logits, 3, 0, shared=True)), T * 32 * 4 + T * 4 * 16, 0.0
     if name == "expert_route":
         logits = torch.randn(T, 32, device="cuda")
         return (lambda i: ops.moe_route(logits, 4, 1)), T * 32 * 4 + T * 4 * 16, 0.0
@@ -378,7 +411,7 @@ def main():
     out = {}
     for name in (ALL if a.case == "all" else [a.case]):
         T = max(a.tokens, 2048) if name in ("gemm_prefill", "attention_prefill", "latent_prefill", "latent_expand", "gated_delta_prefill",
-                                         "chunk_prefill", "chunk_prefill_192") else a.tokens
+                                         "chunk_prefill", "chunk_prefill_192", "capped_prefill", "softcap_prefill", "diff_prefill") else a.tokens
         fn, nbytes, flops = build_case(name, T, a.layers, a.tp)
         iters = a.iters if name not in ("gemm_lm_head", "sample", "argmax") else min(a.iters, 4)
         us = _time_eager(fn, iters) if a.eager else _time_graph(fn, iters)

@@ -104,69 +104,169 @@ __global__ void __launch_bounds__(ASM_THREADS) attention_simt_kernel(OgbAttnLaye
   }
 }
 
-// Differential attention on partial results: one warp per (token, head).  KEEP > 0: a lane keeps its columns (dv <= 32 * KEEP) in registers.
-template <typename T, int KEEP>
-__global__ void __launch_bounds__(128) attention_diff_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits,
-                                                                   int rows_all, int T_, int H, int dv, int vdim, float lambda, float post, float eps,
-                                                                   const T* __restrict__ gate, int gate_stride, T* __restrict__ out, int out_stride) {
+// ------------------------------------------------------------------------------------ differential merge
+template <typename T> __device__ __forceinline__ void load4(const T* p, float (&v)[4]);
+template <> __device__ __forceinline__ void load4<float>(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+template <> __device__ __forceinline__ void load4<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
+struct DiffMerge {
+  const float *part_o, *part_ml;
+  int splits, rows_all, T, H, dv, vdim;
+  float lambda, post, eps;
+  int gate_stride, out_stride;
+};
+
+// Both maps' (maximum, sum) of a head in split s.
+__device__ __forceinline__ float4 diff_stats(const DiffMerge& p, size_t row, int s) {
+  const float2* ml = reinterpret_cast<const float2*>(p.part_ml) + size_t(s) * p.rows_all + row;
+  const float2 a = ml[0], b = ml[1];
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// The weights of up to 32 splits (from s0 on) of the two rows of a head in the difference a1 - lambda * a2, one split per lane.
+__device__ __forceinline__ float2 diff_weights(const DiffMerge& p, size_t row, int s0, const float (&top)[2], const float (&inv)[2], int lane) {
+  float2 w = make_float2(0.f, 0.f);
+  if (s0 + lane < p.splits) {
+    const float4 ml = diff_stats(p, row, s0 + lane);
+    if (ml.x != -INFINITY) w.x = exp2f(ml.x - top[0]) * inv[0];
+    if (ml.z != -INFINITY) w.y = -exp2f(ml.z - top[1]) * inv[1];
+  }
+  return w;
+}
+
+// KEEP > 0: dv <= 128 * KEEP, a lane owns columns 4 lane .. 4 lane + 3 of every 128 (dv a multiple of 4); 0: any dv, recomputed where it is
+// needed twice.  WARPS: warps of a head, the splits are divided over them (1: four heads per CTA).
+template <typename T, int KEEP, int WARPS>
+__global__ void __launch_bounds__(128) attention_diff_merge_kernel(DiffMerge p, const T* __restrict__ gate, T* __restrict__ out) {
+  __shared__ float part[WARPS > 1 ? WARPS : 1][KEEP > 0 ? KEEP * 128 : 1];
   pdl_launch_dependents();
   pdl_wait();
-  const long item = long(blockIdx.x) * 4 + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (item >= long(T_) * H) return;
-  const int t = int(item / H), h = int(item % H);
-  const size_t row = size_t(t) * 2 * H + 2 * h;
-  float top[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
-  for (int s = 0; s < splits; ++s)
-#pragma unroll
-    for (int m = 0; m < 2; ++m) top[m] = fmaxf(top[m], part_ml[(size_t(s) * rows_all + row + m) * 2]);
-  for (int s = 0; s < splits; ++s)
-#pragma unroll
-    for (int m = 0; m < 2; ++m) {
-      const float* ml = part_ml + (size_t(s) * rows_all + row + m) * 2;
-      if (ml[0] != -INFINITY) sum[m] += exp2f(ml[0] - top[m]) * ml[1];
-    }
-  const float inv1 = sum[0] > 0.f ? 1.f / sum[0] : 0.f, inv2 = sum[1] > 0.f ? lambda / sum[1] : 0.f;
-  auto column = [&](int d) {
-    float a = 0.f, b = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const size_t r = size_t(s) * rows_all + row;
-      const float m1 = part_ml[r * 2], m2 = part_ml[r * 2 + 2];
-      if (m1 != -INFINITY) a += exp2f(m1 - top[0]) * part_o[r * dv + d];
-      if (m2 != -INFINITY) b += exp2f(m2 - top[1]) * part_o[(r + 1) * dv + d];
-    }
-    return a * inv1 - b * inv2;
-  };
-  float keep[KEEP > 0 ? KEEP : 1], sq = 0.f;
-  if constexpr (KEEP > 0) {
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-      const int d = lane + 32 * i;
-      keep[i] = d < vdim ? column(d) : 0.f;
-      sq = fmaf(keep[i], keep[i], sq);
-    }
-  } else {
-    for (int d = lane; d < vdim; d += 32) { const float v = column(d); sq = fmaf(v, v, sq); }
+  const int lane = threadIdx.x & 31, warp = WARPS > 1 ? threadIdx.x >> 5 : 0;
+  const long item = WARPS > 1 ? long(blockIdx.x) : long(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= long(p.T) * p.H) return;
+  const int t = int(item / p.H), h = int(item % p.H);
+  const size_t row = size_t(t) * 2 * p.H + 2 * h;
+  float top[2] = {-INFINITY, -INFINITY}, inv[2] = {0.f, 0.f};
+  for (int s = lane; s < p.splits; s += 32) {
+    const float4 ml = diff_stats(p, row, s);
+    top[0] = fmaxf(top[0], ml.x);
+    top[1] = fmaxf(top[1], ml.z);
   }
-  const float f = post / sqrtf(warp_sum(sq) / vdim + eps);
-  T* dst = out + size_t(t) * out_stride + size_t(h) * dv;
-  const T* pg = gate ? gate + size_t(t) * gate_stride + size_t(h) * dv : nullptr;
-  auto store = [&](int d, float v) { dst[d] = of_f32<T>(pg ? v * f / (1.f + expf(-as_f32(pg[d]))) : v * f); };
+  top[0] = warp_max(top[0]);
+  top[1] = warp_max(top[1]);
+  for (int s = lane; s < p.splits; s += 32) {
+    const float4 ml = diff_stats(p, row, s);
+    if (ml.x != -INFINITY) inv[0] += exp2f(ml.x - top[0]) * ml.y;
+    if (ml.z != -INFINITY) inv[1] += exp2f(ml.z - top[1]) * ml.w;
+  }
+  inv[0] = warp_sum(inv[0]);
+  inv[1] = warp_sum(inv[1]);
+  inv[0] = inv[0] > 0.f ? 1.f / inv[0] : 0.f;
+  inv[1] = inv[1] > 0.f ? p.lambda / inv[1] : 0.f;
+  T* dst = out + size_t(t) * p.out_stride + size_t(h) * p.dv;
+  const T* pg = gate ? gate + size_t(t) * p.gate_stride + size_t(h) * p.dv : nullptr;
   if constexpr (KEEP > 0) {
+    float o[KEEP][4] = {};
+    for (int s0 = 0; s0 < p.splits; s0 += 32) {
+      const float2 w = diff_weights(p, row, s0, top, inv, lane);
+      const int n = min(32, p.splits - s0);
+#pragma unroll 4
+      for (int s = warp; s < n; s += WARPS) {
+        const float w1 = __shfl_sync(0xffffffffu, w.x, s), w2 = __shfl_sync(0xffffffffu, w.y, s);
+        const float* r = p.part_o + (size_t(s0 + s) * p.rows_all + row) * p.dv;
 #pragma unroll
-    for (int i = 0; i < KEEP; ++i) if (lane + 32 * i < dv) store(lane + 32 * i, keep[i]);
+        for (int k = 0; k < KEEP; ++k) {
+          const int d = k * 128 + lane * 4;
+          if (d >= p.dv) continue;
+          float a[4], b[4];
+          load4(r + d, a);
+          load4(r + p.dv + d, b);
+          // (an empty split's values are not defined)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            if (w1 != 0.f) o[k][e] = fmaf(w1, a[e], o[k][e]);
+            if (w2 != 0.f) o[k][e] = fmaf(w2, b[e], o[k][e]);
+          }
+        }
+      }
+    }
+    if constexpr (WARPS > 1) {
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) store4(&part[warp][k * 128 + lane * 4], o[k]);
+      __syncthreads();
+      if (warp != 0) return;
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k)
+        for (int q = 1; q < WARPS; ++q) {
+          float a[4];
+          load4(&part[q][k * 128 + lane * 4], a);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) o[k][e] += a[e];
+        }
+    }
+    float sq = 0.f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (k * 128 + lane * 4 + e >= p.vdim) o[k][e] = 0.f;
+        sq = fmaf(o[k][e], o[k][e], sq);
+      }
+    const float f = p.post / sqrtf(warp_sum(sq) / p.vdim + p.eps);
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int d = k * 128 + lane * 4;
+      if (d >= p.dv) continue;
+      float g[4];
+      if (pg) load4(pg + d, g);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[k][e] = pg ? o[k][e] * f / (1.f + expf(-g[e])) : o[k][e] * f;
+      store4(dst + d, o[k]);
+    }
   } else {
-    for (int d = lane; d < dv; d += 32) store(d, d < vdim ? column(d) : 0.f);
+    auto column = [&](int d) {
+      float v = 0.f;
+      for (int s = 0; s < p.splits; ++s) {
+        const size_t r = size_t(s) * p.rows_all + row;
+        const float m1 = p.part_ml[r * 2], m2 = p.part_ml[r * 2 + 2];
+        if (m1 != -INFINITY) v += exp2f(m1 - top[0]) * inv[0] * p.part_o[r * p.dv + d];
+        if (m2 != -INFINITY) v -= exp2f(m2 - top[1]) * inv[1] * p.part_o[(r + 1) * p.dv + d];
+      }
+      return v;
+    };
+    float sq = 0.f;
+    for (int d = lane; d < p.vdim; d += 32) { const float v = column(d); sq = fmaf(v, v, sq); }
+    const float f = p.post / sqrtf(warp_sum(sq) / p.vdim + p.eps);
+    for (int d = lane; d < p.dv; d += 32) {
+      const float v = d < p.vdim ? column(d) * f : 0.f;
+      dst[d] = of_f32<T>(pg ? v / (1.f + expf(-as_f32(pg[d]))) : v);
+    }
   }
 }
 
 template <typename T>
-static int LaunchDiffMerge(const float* po, const float* ml, int splits, int rows_all, int T_, int H, int dv, int vdim, float lambda, float post, float eps,
-                           const void* gate, int gate_stride, void* out, int out_stride, cudaStream_t s) {
-  const dim3 grid(unsigned((long(T_) * H + 3) / 4));
-#define OGB_DIFF(K) launch_pdl(attention_diff_merge_kernel<T, K>, grid, dim3(128), 0, s, po, ml, splits, rows_all, T_, H, dv, vdim, lambda, post, eps, \
-                               static_cast<const T*>(gate), gate_stride, static_cast<T*>(out), out_stride)
-  const bool ok = dv <= 128 ? OGB_DIFF(4) : (dv <= 256 ? OGB_DIFF(8) : OGB_DIFF(0));
+static int LaunchDiffMerge(const DiffMerge& p, const void* gate, void* out, cudaStream_t s) {
+  const long items = long(p.T) * p.H;
+  const bool vec = p.dv % 4 == 0 && p.dv <= 256 && p.gate_stride % 4 == 0 && p.out_stride % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & (4 * sizeof(T) - 1)) == 0;
+  const bool spread = p.splits > 4 && items < (1l << 30);      // several warps per head
+  const dim3 grid(unsigned(spread && vec ? items : (items + 3) / 4));
+#define OGB_DIFF(K, W) launch_pdl(attention_diff_merge_kernel<T, K, W>, grid, dim3(128), 0, s, p, static_cast<const T*>(gate), static_cast<T*>(out))
+  bool ok;
+  if (!vec) ok = OGB_DIFF(0, 1);
+  else if (p.dv <= 128) ok = spread ? OGB_DIFF(1, 4) : OGB_DIFF(1, 1);
+  else ok = spread ? OGB_DIFF(2, 4) : OGB_DIFF(2, 1);
 #undef OGB_DIFF
   return ok ? 0 : -4;
 }
@@ -211,8 +311,7 @@ OGB_API int ogb_attention_diff_merge(const float* part, int splits, int T, int p
   if (T <= 0 || H <= 0) return 0;
   if (!part || splits < 1 || T > part_tokens || vdim <= 0 || vdim > dv) return -1;
   const int rows = part_tokens * 2 * H;
-  const float* ml = part + size_t(splits) * rows * dv;
+  const DiffMerge p{part, part + size_t(splits) * rows * dv, splits, rows, T, H, dv, vdim, lambda, post, eps, gate ? gate_stride : 0, out_stride};
   cudaStream_t s = static_cast<cudaStream_t>(stream_);
-  return fp32 ? LaunchDiffMerge<float>(part, ml, splits, rows, T, H, dv, vdim, lambda, post, eps, gate, gate_stride, out, out_stride, s)
-              : LaunchDiffMerge<__nv_bfloat16>(part, ml, splits, rows, T, H, dv, vdim, lambda, post, eps, gate, gate_stride, out, out_stride, s);
+  return fp32 ? LaunchDiffMerge<float>(p, gate, out, s) : LaunchDiffMerge<__nv_bfloat16>(p, gate, out, s);
 }

@@ -473,6 +473,16 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       tc_fence_before();
       mbar_arrive(&p_full[it % Cfg::S_BUFS]);
     }
+    // the gate's columns of this row are fetched while the last P V runs (ranges start on 16-byte boundaries)
+    const bool wide = p.gate_wide;
+    const int v_cols = LAT ? p.lat.vdim : (MIX ? p.dv : DV);
+    uint4 gq[OC / 8];
+#pragma unroll
+    for (int c = 0; c < OC / 8; ++c) {
+      gq[c] = make_uint4(0u, 0u, 0u, 0u);
+      if (wide && valid && half * OC + c * 8 < v_cols)
+        gq[c] = *reinterpret_cast<const uint4*>(p.gate + size_t(tok0 + tq) * p.gate_stride + size_t(hq) * v_cols + half * OC + c * 8);
+    }
     ok = ok && !*abort_p;
     if (ok && n_tiles > 0 && !mbar_wait_bounded(&o_done[(n_tiles - 1) % Cfg::S_BUFS], ((n_tiles - 1) / Cfg::S_BUFS) & 1, abort_p)) { fail(OGB_ERR_WAIT_MMA); ok = false; }
     tc_fence_after();
@@ -491,11 +501,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
         l = l * scale_o + exp2f(sk - mm);
       }
       float inv = l > 0.f ? scale_o / l : 0.f;
-      const bool wide = p.gate_wide;
       if (p.gate && !wide) inv /= 1.f + __expf(-bf2f(p.gate[size_t(tok0 + tq) * p.gate_stride + hq]));
-      const int v_cols = LAT ? p.lat.vdim : (MIX ? p.dv : DV);
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * v_cols + half * OC;
-      const __nv_bfloat16* pg = p.gate + (wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * v_cols + half * OC : 0);
       const bool raw = MIX && p.part_o;
       const size_t part_row = size_t(tok0 + tq) * p.Hq + hq;
       if (raw && valid && half == 0) {
@@ -514,19 +521,18 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           for (int e = 0; e < 16; ++e) v[e] = 0u;
         }
         if (wide) {
-          // (column ranges of a row start on 16-byte boundaries)
 #pragma unroll
-          for (int h8 = 0; h8 < 16; h8 += 8)
-            if (valid && half * OC + c * 16 + h8 < v_cols) {
-              const uint4 q = *reinterpret_cast<const uint4*>(pg + c * 16 + h8);
-              const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
+          for (int h8 = 0; h8 < 2; ++h8) {
+            const uint4 q = gq[c * 2 + h8];
+            const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                const float2 g = unpack_bf16x2(qw[e]);
-                v[h8 + 2 * e] = __float_as_uint(__uint_as_float(v[h8 + 2 * e]) / (1.f + __expf(-g.x)));
-                v[h8 + 2 * e + 1] = __float_as_uint(__uint_as_float(v[h8 + 2 * e + 1]) / (1.f + __expf(-g.y)));
-              }
+            for (int e = 0; e < 4; ++e) {
+              const float2 g = unpack_bf16x2(qw[e]);
+              const int i = h8 * 8 + 2 * e;
+              v[i] = __float_as_uint(__fdividef(__uint_as_float(v[i]), 1.f + __expf(-g.x)));
+              v[i + 1] = __float_as_uint(__fdividef(__uint_as_float(v[i + 1]), 1.f + __expf(-g.y)));
             }
+          }
         }
         if (raw) {
           float* pr = p.part_o + part_row * p.dv + half * OC + c * 16;

@@ -62,7 +62,8 @@ struct GroupParams {
 // A batch of products that share A's rows (per-head projections): problem z multiplies the K columns of A that start at
 // z * a_cols with weight rows [z * N, (z + 1) * N) and writes C + z * c_cols.  K columns past a problem's own may hold other
 // problems' values: the weight map ends at K, so they meet zeros.  m_tiles > 0 switches it on (blockIdx.y = z * m_tiles + tile).
-struct BatchParams { int m_tiles, a_cols, c_cols; };
+// gate (may be null) [M, ...]: problem z's output column n is multiplied by the sigmoid of gate[m, z * c_cols + n].
+struct BatchParams { int m_tiles, a_cols, c_cols; const __nv_bfloat16* gate; int ldg; };
 
 // Rotary embedding + KV-cache append fused into the epilogue of a QKV projection (positions == nullptr: off).  Output
 // columns are [Hq query heads | Hkv key heads | Hkv value heads] of D each; the rotation pairs element i with i + rot / 2
@@ -306,6 +307,23 @@ static __device__ __noinline__ void epi_store8(const StoreArgs a, int m, int col
   }
 }
 
+// v *= sigmoid of the gate's columns of token row m (see BatchParams)
+static __device__ __noinline__ void epi_gate8(const __nv_bfloat16* g, int cols, float (&v)[8]) {
+  if (cols >= 8 && (reinterpret_cast<uintptr_t>(g) & 15) == 0) {
+    const uint4 q = *reinterpret_cast<const uint4*>(g);
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 x = unpack_bf16x2(w[j]);
+      v[2 * j] /= 1.f + __expf(-x.x);
+      v[2 * j + 1] /= 1.f + __expf(-x.y);
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) if (j < cols) v[j] /= 1.f + __expf(-bf2f(g[j]));
+  }
+}
+
 // Epilogue shared by the linear-layer kernels.  Called by all threads of the CTA once the MMA issuer has committed the last
 // k-block to `accum_bar`; `smem` is the (idle) pipeline memory, reused for the fp32 tile.
 // COMM: 0 = results stay on this GPU; 1 = tensor-parallel reduction with flagged lines over peer memory; 2 = through the
@@ -483,6 +501,7 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, uint8_t* smem
         }
       }
       if (COMM == 0) {
+        if (p.bat.gate) epi_gate8(p.bat.gate + size_t(m) * p.bat.ldg + size_t(blockIdx.y / p.bat.m_tiles) * p.bat.c_cols + col, n_out - col, v);
         epi_store8(sa, m, col, make_float4(v[0], v[1], v[2], v[3]), make_float4(v[4], v[5], v[6], v[7]));
       } else if (COMM == 2) {
         // this rank's partial stays in its own plane; the switch adds the planes when a rank reads through the multicast mapping

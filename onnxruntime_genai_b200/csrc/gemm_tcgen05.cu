@@ -860,9 +860,9 @@ OGB_API int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, 
 }
 
 // A batch of `batch` products over the same M rows of A (per-head projections): C[:, z * c_cols + n] = sum_k A[:, z * a_cols + k] *
-// W[z * N + n, k], k < K.  A [M, a_width] bf16 (a_cols a multiple of 8, every column finite), W [batch * N, K] bf16, C bf16.
+// W[z * N + n, k], k < K, times the sigmoid of gate[:, z * c_cols + n] (gate may be null).  A [M, a_width] bf16 (a_cols a multiple of 8, every column finite), W [batch * N, K] bf16, C bf16.
 OGB_API int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M,
-                                  int N, int K, int batch, int* status, void* stream_) {
+                                  int N, int K, int batch, const void* gate, int ldg, int* status, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   if ((a_cols % 8) || (lda % 8) || (ldw % 8)) return -1;
@@ -884,6 +884,7 @@ OGB_API int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_col
   p.status = status;
   p.pdl = pdl_enabled;
   p.bat.m_tiles = (M + bt - 1) / bt; p.bat.a_cols = a_cols; p.bat.c_cols = c_cols;
+  p.bat.gate = static_cast<const __nv_bfloat16*>(gate); p.bat.ldg = ldg;
   if ((long long)p.bat.m_tiles * batch > 65535) return -1;
   dim3 grid((N + GEMM_BLOCK_N - 1) / GEMM_BLOCK_N, p.bat.m_tiles * batch, 1);
   switch (bt) {

@@ -49,7 +49,7 @@ int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, void* C,
 
 // Per-head products over the same rows of A: C[:, z * c_cols + n] = sum_k A[:, z * a_cols + k] * W[z * N + n, k]
 int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N,
-                          int K, int batch, int* status, void* stream);
+                          int K, int batch, const void* gate, int ldg, int* status, void* stream);
 
 // ---- gemm_simt.cu: fp32 products and bf16 products TMA cannot address
 int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K, int batch,
@@ -89,10 +89,10 @@ typedef struct OgbTanhNorm {
 } OgbTanhNorm;
 int ogb_add_tanh_norm(const OgbTanhNorm* p, void* stream);
 // Token embedding plus a row hashed from (previous token, token): out[t] = table[id] * scale + bigram[(prev * mul_prev + id * mul_cur) mod buckets],
-// row `buckets` for a sequence's first token.  The previous token of a step's first token comes from the paged pool `tokens` [slots]; every
+// row `buckets` for a sequence's first token (position 0).  The previous token of a step's first token comes from the paged pool `tokens` [slots]; every
 // token of the step is stored there.
 typedef struct OgbBigram {
-  const int32_t *ids, *slots, *cu_seqlens, *past_lens, *block_table;
+  const int32_t *ids, *slots, *positions, *cu_seqlens, *block_table;
   int32_t* tokens;
   int table_cols, block_size, B, T, H, vocab, buckets, fp32;
   long long mul_prev, mul_cur;

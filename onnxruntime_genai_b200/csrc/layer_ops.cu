@@ -16,6 +16,17 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return f2bf(v); }
 
+template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 q = *reinterpret_cast<const uint4*>(p);
+  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y), c = unpack_bf16x2(q.z), d = unpack_bf16x2(q.w);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y; v[4] = c.x; v[5] = c.y; v[6] = d.x; v[7] = d.y;
+}
+
 // ------------------------------------------------------------------------------------ embedding into the fp32 stream
 template <typename T>
 __global__ void embedding_stream_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
@@ -32,34 +43,50 @@ __global__ void embedding_stream_kernel(const int32_t* __restrict__ ids, const T
 }
 
 // ------------------------------------------------------------------------------------ embedding with hashed pairs
-// One CTA per token (see OgbBigram).
-template <typename T>
-__global__ void embedding_bigram_kernel(OgbBigram p, const T* __restrict__ table, const T* __restrict__ bigram, float* __restrict__ out) {
+// One CTA per token (see OgbBigram).  The request of a token is found by all threads at once: a decode step is a chain of dependent loads.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) embedding_bigram_kernel(OgbBigram p, const T* __restrict__ table, const T* __restrict__ bigram,
+                                                               float* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
-  int lo = 0, hi = p.B - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (p.cu_seqlens[mid] <= t) lo = mid; else hi = mid - 1;
+  const int id = p.ids[t], before = p.positions[t], slot = p.slots[t];
+  const int prev_id = t > 0 ? p.ids[t - 1] : 0;
+  int n = 0;                                           // requests that start at or before the token
+  for (int i0 = 0; i0 < p.B; i0 += blockDim.x) {
+    const int i = i0 + threadIdx.x;
+    const int c = __syncthreads_count(i < p.B && p.cu_seqlens[i] <= t);
+    n += c;
+    if (c < int(blockDim.x)) break;
   }
-  const int t0 = p.cu_seqlens[lo], before = p.past_lens[lo] + t - t0, id = p.ids[t];
+  const int r = n - 1;
   long long row = p.buckets;
   if (before > 0) {
-    int prev = 0;
-    if (t > t0) {
-      prev = p.ids[t - 1];
-    } else {
-      const int q = before - 1, block = p.block_table[size_t(lo) * p.table_cols + q / p.block_size];
-      if (block >= 0) prev = p.tokens[size_t(block) * p.block_size + q % p.block_size];
+    int prev = prev_id;
+    if (p.cu_seqlens[r] == t) {
+      const int q = before - 1, block = p.block_table[size_t(r) * p.table_cols + q / p.block_size];
+      prev = block >= 0 ? p.tokens[size_t(block) * p.block_size + q % p.block_size] : 0;
     }
     row = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
     if (row < 0) row += p.buckets;
   }
-  if (threadIdx.x == 0 && p.slots[t] >= 0) p.tokens[p.slots[t]] = id;
+  if (threadIdx.x == 0 && slot >= 0) p.tokens[slot] = id;
   const T* a = table + size_t(min(max(id, 0), p.vocab - 1)) * p.H;
   const T* b = bigram + size_t(row) * p.H;
-  for (int i = threadIdx.x; i < p.H; i += blockDim.x) out[size_t(t) * p.H + i] = fmaf(to_f32(a[i]), p.scale, to_f32(b[i]));
+  float* dst = out + size_t(t) * p.H;
+  for (int i = threadIdx.x * VEC; i < p.H; i += blockDim.x * VEC) {
+    if constexpr (VEC == 8) {
+      float x[8], y[8];
+      load8(a + i, x);
+      load8(b + i, y);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = fmaf(x[e], p.scale, y[e]);
+      reinterpret_cast<float4*>(dst + i)[0] = make_float4(x[0], x[1], x[2], x[3]);
+      reinterpret_cast<float4*>(dst + i)[1] = make_float4(x[4], x[5], x[6], x[7]);
+    } else {
+      dst[i] = fmaf(to_f32(a[i]), p.scale, to_f32(b[i]));
+    }
+  }
 }
 
 // ------------------------------------------------------------------------------------ norm of the fp32 stream
@@ -137,17 +164,6 @@ struct AddNormed {
   int k, ldy, H;
   float eps;
 };
-
-template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
-template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 q = *reinterpret_cast<const uint4*>(p);
-  const float2 a = unpack_bf16x2(q.x), b = unpack_bf16x2(q.y), c = unpack_bf16x2(q.z), d = unpack_bf16x2(q.w);
-  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y; v[4] = c.x; v[5] = c.y; v[6] = d.x; v[7] = d.y;
-}
 
 template <typename T>
 __device__ __forceinline__ float add_normed_col(const AddNormed& p, const T* y, int t, int i) {
@@ -378,6 +394,60 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(T* __restrict__ proj, T* 
   for (int i = p.dim + lane; i < p.key_row; i += 32) dst[i] = from_f32<T>(0.f);
 }
 
+// The same without norms, where every part is whole pieces of 8 columns (dim, rot / 2, value_row): one thread per piece, a rotated piece with its
+// partner half a rotation away.
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_prep_pieces_kernel(T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int half = p.rot >> 1, turn = half / 8, kp = p.key_row / 8 - turn, vp = p.value_row / 8;      // pieces of a query or key head, of a value head
+  const int t = blockIdx.x, n_qk = (p.Hq + p.Hkv) * kp, n = n_qk + p.Hv * vp;
+  T* row = proj + size_t(t) * p.ldp;
+  const int slot = p.slots[t];
+  const size_t at = size_t(min(max(p.positions[t], 0), p.max_pos - 1)) * half;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
+    float a[8], b[8];
+    auto st8 = [](T* dst, const float (&v)[8]) {
+      if constexpr (sizeof(T) == 4) {
+        reinterpret_cast<float4*>(dst)[0] = make_float4(v[0], v[1], v[2], v[3]);
+        reinterpret_cast<float4*>(dst)[1] = make_float4(v[4], v[5], v[6], v[7]);
+      } else {
+        *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+      }
+    };
+    if (i >= n_qk) {
+      if (slot < 0) continue;
+      const int j = (i - n_qk) * 8;
+      load8(row + size_t(p.Hq + p.Hkv) * p.key_row + j, a);
+      st8(v_cache + size_t(slot) * p.Hv * p.value_row + j, a);
+      continue;
+    }
+    const int head = i / kp, c = i - head * kp;
+    const bool is_q = head < p.Hq;
+    if (!is_q && slot < 0) continue;
+    T* src = row + size_t(head) * p.key_row;
+    T* dst = is_q ? src : k_cache + (size_t(slot) * p.Hkv + (head - p.Hq)) * p.key_row;
+    if (c < turn) {
+      float cs[8], sn[8], u[8], v[8];
+      load8(src + c * 8, a);
+      load8(src + half + c * 8, b);
+      load8(p.cos + at + c * 8, cs);
+      load8(p.sin + at + c * 8, sn);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        u[e] = a[e] * cs[e] - b[e] * sn[e];
+        v[e] = b[e] * cs[e] + a[e] * sn[e];
+      }
+      st8(dst + c * 8, u);
+      st8(dst + half + c * 8, v);
+    } else if (!is_q) {                                // (unrotated columns of a query stay where they are)
+      const int j = p.rot + (c - turn) * 8;
+      load8(src + j, a);
+      st8(dst + j, a);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------ experts' activations
 // Rows of alternating (gate, up) columns.  kind 0: silu(g) * u; 1: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + 1).
 template <typename T>
@@ -468,11 +538,12 @@ OGB_API int ogb_embedding_bigram(const OgbBigram* p, const void* table, const vo
   if (p->T <= 0) return 0;
   if (p->B <= 0 || p->H <= 0 || p->vocab <= 0 || p->buckets <= 0 || p->block_size <= 0) return -1;
   auto s = static_cast<cudaStream_t>(stream);
-  const dim3 block(p->H >= 256 ? 256 : 64);
-  const bool ok = p->fp32 ? launch_pdl(embedding_bigram_kernel<float>, dim3(p->T), block, 0, s, *p, static_cast<const float*>(table),
-                                       static_cast<const float*>(bigram), out)
-                          : launch_pdl(embedding_bigram_kernel<__nv_bfloat16>, dim3(p->T), block, 0, s, *p, static_cast<const __nv_bfloat16*>(table),
-                                       static_cast<const __nv_bfloat16*>(bigram), out);
+  const bool vec = p->H % 8 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(bigram) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int pieces = vec ? p->H / 8 : p->H;
+  const dim3 block(pieces >= 256 ? 256 : (pieces + 31) / 32 * 32);
+#define OGB_PAIRS(TY, V) launch_pdl(embedding_bigram_kernel<TY, V>, dim3(p->T), block, 0, s, *p, static_cast<const TY*>(table), static_cast<const TY*>(bigram), out)
+  const bool ok = p->fp32 ? (vec ? OGB_PAIRS(float, 8) : OGB_PAIRS(float, 1)) : (vec ? OGB_PAIRS(__nv_bfloat16, 8) : OGB_PAIRS(__nv_bfloat16, 1));
+#undef OGB_PAIRS
   return ok ? 0 : -4;
 }
 
@@ -563,6 +634,16 @@ OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, 
   const dim3 grid(unsigned((items + 7) / 8));
   auto s = static_cast<cudaStream_t>(stream);
   const int elem = fp32 ? 4 : 2;
+  if (!q_norm && !k_norm && dim == key_row && dim % 8 == 0 && rot % 16 == 0 && value_row % 8 == 0 && ldp % 8 == 0 &&
+      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(cos) |
+        reinterpret_cast<uintptr_t>(sin)) & 15) == 0) {
+    const int pieces = (Hq + Hkv) * (key_row / 8 - rot / 16) + Hv * (value_row / 8);
+    const dim3 g2(T, T >= 1024 ? 1 : (pieces + 255) / 256), block(pieces < 256 ? (pieces + 31) / 32 * 32 : 256);
+    const bool done = fp32 ? launch_pdl(qkv_prep_pieces_kernel<float>, g2, block, 0, s, static_cast<float*>(proj), static_cast<float*>(k_cache), static_cast<float*>(v_cache), p)
+                           : launch_pdl(qkv_prep_pieces_kernel<__nv_bfloat16>, g2, block, 0, s, static_cast<__nv_bfloat16*>(proj),
+                                        static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), p);
+    return done ? 0 : -4;
+  }
   const bool two = dim % 2 == 0 && (rot / 2) % 2 == 0 && ldp % 2 == 0 && key_row % 2 == 0 && value_row % 2 == 0 &&
                    ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & (2 * elem - 1)) == 0;
 #define OGB_PREP(TY, V) launch_pdl(qkv_prep_kernel<TY, V>, grid, dim3(256), 0, s, static_cast<TY*>(proj), static_cast<TY*>(k_cache), static_cast<TY*>(v_cache), p)

@@ -517,9 +517,7 @@ class DecoderModel:
             olat = ops.latent_attention(qlat, q, shape, cache, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale, sp.window,
                                         s.max_q_len, s.max_kv_len, skip_q_len=ops.LATENT_LONG_TOKENS if plan is not None else 0, order=s.attn_order,
                                         sinks=lw.sinks)
-            ops.head_project(olat, lw.lat_uv, sp.heads, sp.kv_rank, out=out[:n_short])
-            if gate is not None:
-                ops.gate_rows(out[:n_short], gate[:n_short])
+            ops.head_project(olat, lw.lat_uv, sp.heads, sp.kv_rank, out=out[:n_short], gate=None if gate is None else gate[:n_short])
         if plan is not None and plan.rows > 0:
             ops.latent_attention_long(q, shape, lw.lat_ukv, cache, plan, s.cu_seqlens, s.past_lens, s.block_table, kv.block_size, sp.scale,
                                       sp.window, out, lw.sinks, gate)
@@ -602,9 +600,9 @@ class DecoderModel:
         return h
 
     def _tanh_normed_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
-        """Pre-norm blocks under tanh norms, to the final norm of the rows whose logits are wanted.  The mixer's output map adds to the stream
-        in its epilogue; one kernel per norm adds what is still missing from the stream (experts' rows, and where a pass through the looped
-        layers begins its learned vector and the embedding output) and writes the norm of the sum."""
+        """Pre-norm blocks under tanh norms, to the final norm of the rows whose logits are wanted.  One kernel per sub-layer adds its result to the
+        fp32 stream (folding the weighted sum of experts' rows, and where a pass through the looped layers begins its learned vector and the
+        embedding output) and writes the next sub-layer's norm of the sum."""
         a = self.arch
         if s.inputs_embeds is not None:
             raise RuntimeError("this model's embedding reads token ids (pairs of neighbours): inputs_embeds cannot replace them")
@@ -622,11 +620,10 @@ class DecoderModel:
             h = stream
             heads = torch.empty(h.shape[0], lw.mix_cols, dtype=self.dtype, device=h.device)
             self._stack_mixer(lw, sp)(s, kv, li, lw, x, out=heads)
-            ops.linear(heads, lw.o_w, residual=h, out=h, out_fp32=True)
-            y = None
+            y = ops.linear(heads, lw.o_w)
             if sp.ff:
                 from .moe import moe_forward
-                y = moe_forward(self, lw, ops.add_tanh_norm(h, None, lw.norm2, self.dtype), defer=True)
+                y = moe_forward(self, lw, ops.add_tanh_norm(h, y, lw.norm2, self.dtype, out=h), defer=True)
         return ops.add_tanh_norm(h, y, self.final_norm, self.dtype, rows=s.logits_rows)
 
     def _mamba(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor) -> torch.Tensor:

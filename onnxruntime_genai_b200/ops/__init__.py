@@ -178,7 +178,7 @@ def embedding_bigram(ids, table, scale, bigram, spec, tokens, slots, positions, 
     assert bigram.shape == (spec["buckets"] + 1, table.shape[1]) and block_table.stride(1) == 1 and table.dtype in (torch.bfloat16, torch.float32)
     T, H = ids.numel(), table.shape[1]
     out = torch.empty(T, H, dtype=torch.float32, device=table.device)
-    p = _lib.Bigram(ids=_ptr(ids), slots=_ptr(slots), cu_seqlens=_ptr(cu_seqlens), past_lens=_ptr(past_lens), block_table=_ptr(block_table),
+    p = _lib.Bigram(ids=_ptr(ids), slots=_ptr(slots), positions=_ptr(positions), cu_seqlens=_ptr(cu_seqlens), block_table=_ptr(block_table),
                     tokens=_ptr(tokens), table_cols=block_table.stride(0), block_size=int(block_size), B=past_lens.shape[0], T=T, H=H, vocab=table.shape[0],
                     fp32=int(table.dtype == torch.float32), scale=float(scale), **spec)
     _lib.check(_lib.lib().ogb_embedding_bigram(ctypes.byref(p), _ptr(table), _ptr(bigram), _ptr(out), _stream()), "embedding_bigram")
@@ -339,20 +339,24 @@ def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None, bi
     return out
 
 
-def head_project(x, w, heads: int, a_cols: int, out=None):
+def head_project(x, w, heads: int, a_cols: int, out=None, gate=None):
     """Per-head products over the same token rows: out[:, h * N + n] = sum_k x[:, h * a_cols + k] * w[h * N + n, k] with
-    w [heads * N, K]; x may be wider than the heads need.  Returns [T, heads * N] (or writes `out`, which may be a column range)."""
+    w [heads * N, K]; x may be wider than the heads need; gate [T, heads * N]: the result is multiplied by its sigmoid.  Returns [T, heads * N] (or
+    writes `out`, which may be a column range)."""
     K, N = w.shape[1], w.shape[0] // heads
     if out is None:
         out = torch.empty(x.shape[0], heads * N, dtype=x.dtype, device=x.device)
     if not x.is_cuda:
         out.copy_(ref.head_project(x, w, heads, a_cols))
-        return out
+        return out if gate is None else gate_rows(out, gate)
     if x.dtype == torch.float32 or a_cols % 8 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8 or (x.data_ptr() | w.data_ptr()) % 16:
-        return _gemm_simt(x, w, out, batch=heads, a_cols=a_cols, c_cols=N, K=K)
+        _gemm_simt(x, w, out, batch=heads, a_cols=a_cols, c_cols=N, K=K)
+        return out if gate is None else gate_rows(out, gate)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1 and gate.shape == (x.shape[0], heads * N))
     _lib.check(_lib.lib().ogb_gemm_bf16_batched(_ptr(x), x.stride(0), x.shape[1], int(a_cols), _ptr(w), w.stride(0), _ptr(out), out.stride(0), N,
-                                               x.shape[0], N, K, heads, workspace(x.device).status, _stream()), "gemm_bf16_batched")
+                                               x.shape[0], N, K, heads, _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                               workspace(x.device).status, _stream()), "gemm_bf16_batched")
     return out
 
 

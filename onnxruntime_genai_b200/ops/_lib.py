@@ -43,7 +43,7 @@ class TanhNorm(ctypes.Structure):
 
 class Bigram(ctypes.Structure):
     """OgbBigram of csrc/kernels.h: token embedding with rows hashed from (previous token, token)."""
-    _fields_ = ([(n, _P) for n in ("ids", "slots", "cu_seqlens", "past_lens", "block_table", "tokens")] +
+    _fields_ = ([(n, _P) for n in ("ids", "slots", "positions", "cu_seqlens", "block_table", "tokens")] +
                 [(n, c_int) for n in ("table_cols", "block_size", "B", "T", "H", "vocab", "buckets", "fp32")] +
                 [("mul_prev", c_longlong), ("mul_cur", c_longlong), ("scale", c_float)])
 
@@ -92,7 +92,7 @@ _SIGS = {
     "ogb_act": (c_int, [_P, _P, c_longlong, c_int, _P]),
     "ogb_causal_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_causal_conv_rows": (c_int, [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
-    "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P]),
+    "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P]),
     "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, _P]),
     "ogb_moe_gemm_simt": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P]),
     "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_float, _P]),

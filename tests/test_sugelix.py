@@ -182,6 +182,59 @@ def test_sum_into_the_stream_and_its_tanh_norm(runtime, T, H):
     assert torch.allclose(ops.add_tanh_norm(tiny, None, zero, torch.float32).cpu(), torch.full((1, H), 2e-5), rtol=1e-5)
 
 
+@pytest.mark.parametrize("T,heads,K,N", [(1, 3, 48, 24), (5, 4, 128, 64), (70, 2, 512, 128), (200, 3, 13, 7), (33, 5, 24, 20)])
+def test_per_head_products_with_a_gate(runtime, T, heads, K, N):
+    g = torch.Generator().manual_seed(T)
+    dev, dt = runtime[0], dtype_of(runtime)
+    x, w, gate = torch.randn(T, heads * K, generator=g).to(dt), (torch.randn(heads * N, K, generator=g) / K ** 0.5).to(dt), (2 * torch.randn(T, heads * N, generator=g)).to(dt)
+    want = torch.cat([x[:, h * K:(h + 1) * K].double() @ w[h * N:(h + 1) * N].double().T for h in range(heads)], 1) * torch.sigmoid(gate.double())
+    out = torch.zeros(T, heads * N + 5, dtype=dt, device=dev)
+    ops.head_project(wide_rows(x, dev), w.to(dev), heads, K, out=out[:, 3:3 + heads * N], gate=wide_rows(gate, dev))
+    close(out[:, 3:3 + heads * N], want, 8e-3 if dt == torch.bfloat16 else 1e-5)
+    assert (out[:, :3] == 0).all() and (out[:, -2:] == 0).all()
+
+
+@pytest.mark.parametrize("shape", [(4, 2, 24, 16, 16), (3, 1, 9, 5, 6), (5, 1, 128, 72, 80), (8, 2, 64, 128, 64), (6, 3, 40, 40, 0), (4, 4, 32, 8, 32)],
+                         ids=lambda s: "x".join(map(str, s)))
+def test_rotation_and_append_without_norms(runtime, shape):
+    """Two key vectors per value head; a token whose slot is negative is not kept."""
+    H, G, d, dv, rd = shape
+    dev, dt = runtime[0], dtype_of(runtime)
+    g = torch.Generator().manual_seed(d)
+    kr, vr = (d + 7) // 8 * 8, (dv + 7) // 8 * 8
+    lens = [(0, 5), (30, 1), (15, 3), (200, 1)]
+    pg = paged(lens, 20)
+    T = sum(n for _, n in lens)
+    q, k, v = (torch.randn(T, n, c, generator=g).to(dt) for n, c in ((2 * H, d), (2 * G, d), (G, dv)))
+    fill = lambda x, c: torch.nn.functional.pad(x, (0, c - x.shape[-1])).reshape(T, -1)
+    proj = torch.cat([fill(q, kr), fill(k, kr), fill(v, vr), torch.randn(T, 3, generator=g).to(dt)], 1)
+    wide = wide_rows(proj, dev)
+    kc, vc = torch.full((20 * BLOCK, G, 2 * kr), 7.0, dtype=dt, device=dev), torch.full((20 * BLOCK, G, vr), 7.0, dtype=dt, device=dev)
+    rot = dict(dims=rd, base=300.0, scaling=dict(factor=3.0)) if rd else None
+    cos = sin = None
+    if rd:
+        cos, sin = (torch.from_numpy(t).to(dev) for t in A.rotary_tables(A.RotarySpec(rd, 300.0, rot["scaling"]), 256))
+    slots = pg["slots"].clone()
+    slots[-1] = -1
+    ops.qkv_prep(wide, 2 * H, 2 * G, d, kr, vr, None, None, 0.0, pg["pos"].to(dev), cos, sin, slots.to(dev), kc, vc, Hv=G)
+
+    def want(x):
+        out = torch.empty(x.shape, dtype=torch.float64)
+        for t, p in enumerate(pg["pos"].tolist()):         # rotate() counts positions from the first row
+            full = torch.zeros(p + 1, *x.shape[1:], dtype=torch.float64)
+            full[p] = x[t].double()
+            out[t] = rotate(full, rot)[p]
+        return out
+    got = wide.cpu()
+    close(got[:, :2 * H * kr].reshape(T * 2 * H, kr)[:, :d], want(q).reshape(-1, d), tol_of(runtime) / 4)
+    at = slots[slots >= 0].long()
+    close(kc.cpu()[at].view(-1, 2 * G, kr)[:, :, :d].reshape(-1, d), want(k)[slots >= 0].reshape(-1, d), tol_of(runtime) / 4)
+    assert torch.equal(vc.cpu()[at][:, :, :dv], v[slots >= 0]) and (kc.cpu()[at].view(-1, 2 * G, kr)[:, :, d:] == 0).all()
+    rest = torch.ones(20 * BLOCK, dtype=torch.bool)
+    rest[at] = False
+    assert (kc.cpu()[rest] == 7).all() and (vc.cpu()[rest] == 7).all() and torch.equal(got[:, -3:], proj[:, -3:])
+
+
 SHAPES = [(4, 2, 24, 16), (3, 3, 16, 8), (6, 2, 128, 72), (8, 1, 64, 128), (2, 2, 128, 128), (4, 2, 96, 96), (4, 4, 64, 64), (2, 1, 256, 256), (2, 1, 264, 24),
           (20, 1, 40, 40)]
 
