@@ -145,6 +145,49 @@ __device__ __forceinline__ float2 diff_weights(const DiffMerge& p, size_t row, i
   return w;
 }
 
+// One split (prompts): a1 / l1 - lambda * a2 / l2, everything loaded before anything is used.
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(128) attention_diff_single_kernel(DiffMerge p, const T* __restrict__ gate, T* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long item = long(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= long(p.T) * p.H) return;
+  const int t = int(item / p.H), h = int(item - long(t) * p.H);
+  const size_t row = size_t(t) * 2 * p.H + 2 * h;
+  const float* r = p.part_o + row * p.dv;
+  const T* pg = gate ? gate + size_t(t) * p.gate_stride + size_t(h) * p.dv : nullptr;
+  float a[KEEP][4], b[KEEP][4], g[KEEP][4];
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = k * 128 + lane * 4;
+    if (d >= p.dv) continue;
+    load4(r + d, a[k]);
+    load4(r + p.dv + d, b[k]);
+    if (pg) load4(pg + d, g[k]);
+  }
+  const float4 ml = diff_stats(p, row, 0);
+  const float f1 = ml.y > 0.f ? 1.f / ml.y : 0.f, f2 = ml.w > 0.f ? p.lambda / ml.w : 0.f;
+  float sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      a[k][e] = k * 128 + lane * 4 + e < p.vdim ? a[k][e] * f1 - b[k][e] * f2 : 0.f;
+      sq = fmaf(a[k][e], a[k][e], sq);
+    }
+  const float f = p.post / sqrtf(warp_sum(sq) / p.vdim + p.eps);
+  T* dst = out + size_t(t) * p.out_stride + size_t(h) * p.dv;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = k * 128 + lane * 4;
+    if (d >= p.dv) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) a[k][e] = pg ? a[k][e] * f / (1.f + expf(-g[k][e])) : a[k][e] * f;
+    store4(dst + d, a[k]);
+  }
+}
+
 // KEEP > 0: dv <= 128 * KEEP, a lane owns columns 4 lane .. 4 lane + 3 of every 128 (dv a multiple of 4); 0: any dv, recomputed where it is
 // needed twice.  WARPS: warps of a head, the splits are divided over them (1: four heads per CTA).
 template <typename T, int KEEP, int WARPS>
@@ -263,11 +306,14 @@ static int LaunchDiffMerge(const DiffMerge& p, const void* gate, void* out, cuda
   const bool spread = p.splits > 4 && items < (1l << 30);      // several warps per head
   const dim3 grid(unsigned(spread && vec ? items : (items + 3) / 4));
 #define OGB_DIFF(K, W) launch_pdl(attention_diff_merge_kernel<T, K, W>, grid, dim3(128), 0, s, p, static_cast<const T*>(gate), static_cast<T*>(out))
+#define OGB_DIFF1(K) launch_pdl(attention_diff_single_kernel<T, K>, grid, dim3(128), 0, s, p, static_cast<const T*>(gate), static_cast<T*>(out))
   bool ok;
   if (!vec) ok = OGB_DIFF(0, 1);
+  else if (p.splits == 1) ok = p.dv <= 128 ? OGB_DIFF1(1) : OGB_DIFF1(2);
   else if (p.dv <= 128) ok = spread ? OGB_DIFF(1, 4) : OGB_DIFF(1, 1);
   else ok = spread ? OGB_DIFF(2, 4) : OGB_DIFF(2, 1);
 #undef OGB_DIFF
+#undef OGB_DIFF1
   return ok ? 0 : -4;
 }
 
