@@ -140,8 +140,9 @@ __device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.p
 
 // DK: width of the staged query and key rows; DV: width of the value rows; LAT: the latent form, whose first NOPE of the DK columns
 // are the unrotated part; MIX: heads of p.dk and p.dv columns (multiples of 8).  The boxes of a head narrower than the staged rows reach
-// into the next head's columns, which meet zeros in Q (keys) or give output columns that are not stored (values).
-template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false>
+// into the next head's columns, which meet zeros in Q (keys) or give output columns that are not stored (values).  CAP: scores are soft-capped
+// (a kernel of its own: the loop body of the others has to stay within the instruction cache).
+template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false, bool CAP = false>
 __global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN>::CTAS_PER_SM)
 attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_r,
                     TcAttnParams p) {
@@ -354,9 +355,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       mbar_arrive(&q_full);
     }
     const uint32_t lane_base = tmem_base + (uint32_t(quarter * 32) << 16);
-    const bool capped = p.softcap > 0.f;
-    const float kmul = capped ? 1.f : p.scale * TCA_LOG2E;        // exponent = s * kmul - reference maximum
-    const float inv_cap = capped ? p.scale / p.softcap : 0.f, capl = p.softcap * TCA_LOG2E;
+    const float kmul = CAP ? 1.f : p.scale * TCA_LOG2E;        // exponent = s * kmul - reference maximum
+    const float inv_cap = CAP ? p.scale / p.softcap : 0.f, capl = p.softcap * TCA_LOG2E;
     // a tile every key of which every row of this lane quarter sees needs no masks
     const int wq_lo = past + min(q_len - 1, (row0 + quarter * 32) / G), wq_hi = past + min(q_len - 1, (row0 + quarter * 32 + 31) / G);
     const bool rows_full = row0 + quarter * 32 + 31 < rows;
@@ -376,7 +376,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     };
     // soft-cap / mask 16 scores of tile `it` in place and return their maximum (raw units: times kmul gives the exponent)
     auto prep16 = [&](int it, float (&x)[HC], int c, bool interior) -> float {
-      if (capped) {
+      if constexpr (CAP) {
         // (most scores lie where the polynomial holds: one vote spares the others the exponential and the division)
         float far = 0.f;
 #pragma unroll
@@ -561,10 +561,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   if (warp == TCA_K_WARP) tmem_dealloc(tmem_base, Cfg::TMEM_COLS);
 }
 
-template <int DK, int DV, int BN, bool MIX = false>
-static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
+template <int DK, int DV, int BN, bool MIX, bool CAP>
+static int LaunchTcForm(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
   using Cfg = TcaCfg<DK, DV, BN>;
-  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX>;
+  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP>;
   const int kw = p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
@@ -577,6 +577,12 @@ static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_ca
   dim3 grid((max_q_len * G + TCA_BM - 1) / TCA_BM, p.Hkv, p.B);
   launch_pdl(kern, grid, dim3(TCA_THREADS), Cfg::SMEM, stream, mk, mv, mv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <int DK, int DV, int BN, bool MIX = false>
+static int LaunchTc(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
+  return p.softcap > 0.f ? LaunchTcForm<DK, DV, BN, MIX, true>(p, k_cache, v_cache, max_q_len, cache_slots, stream)
+                         : LaunchTcForm<DK, DV, BN, MIX, false>(p, k_cache, v_cache, max_q_len, cache_slots, stream);
 }
 
 }  // namespace ogb

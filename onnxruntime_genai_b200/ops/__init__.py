@@ -1087,11 +1087,12 @@ def gate_rows(x, gate):
 
 
 def choose_latent_splits(batch: int, row_tiles: int, tile_rows: int, max_kv_len: int, window: int, sm_count: int = 148) -> int:
-    """Key splits of a latent-attention launch: about three CTAs per SM for 16-row tiles (two are resident at a time, the third evens out
-    requests of different lengths), half of that for taller tiles, each split at least two tiles of 32 keys.  Measured on B200 with
-    requests of 192..2112 keys: 64 requests 6 - 8 splits 36 us (4: 45), 256 requests 2 splits 96 us (1: 153, 3: 105), 8 requests 24."""
+    """Key splits of a latent-attention launch: 3.5 CTAs per SM for 16-row tiles (two are resident at a time, the others even out requests of
+    different lengths), 1.5 for taller tiles, each split at least two tiles of 32 keys.  Measured on B200 with requests of 192..2112 keys:
+    16 heads, 64 requests 6 - 8 splits 36 us (4: 45), 256 requests 2 splits 96 us (1: 153, 3: 105); 32 heads, 64 requests longest first 4 splits
+    55 us (3: 59, 6: 60), all of 2049 keys 95 us (3: 115, 6: 98)."""
     span = max_kv_len if window <= 0 else min(max_kv_len, window + 64)
-    want = (3 if tile_rows <= 16 else 1.5) * sm_count / max(1, batch * row_tiles)
+    want = (3.5 if tile_rows <= 16 else 1.5) * sm_count / max(1, batch * row_tiles)
     return max(1, min(int(round(want)), span // 64, 32))
 
 
