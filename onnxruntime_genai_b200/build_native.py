@@ -34,7 +34,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v"]
 # Sources compiled without --use_fast_math: recurrences, routers, 32-bit models and the norms of an fp32 residual stream keep IEEE division,
 # square roots and denormals.
-PRECISE_SOURCES = {"attention_simt.cu", "gemm_simt.cu", "latent_attention.cu", "layer_ops.cu", "linear_attention.cu", "moe.cu"}
+PRECISE_SOURCES = {"attention_simt.cu", "gemm_simt.cu", "latent_attention.cu", "layer_ops.cu", "linear_attention.cu", "moe.cu", "recurrent.cu"}
 
 
 def _newer(sources, target) -> bool:

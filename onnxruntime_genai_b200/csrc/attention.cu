@@ -47,6 +47,7 @@ static int PagedAttention(const void* q, int q_stride, const void* k_cache, cons
   if (kv_chunk < 0 || (kv_chunk % ATT_BN)) return -1;
   if (splits > 1 && ogb_attention_scratch_bytes(total_tokens, Hq, D, splits) > scratch_bytes) return -2;
   AttnParams p{};
+  p.out_scale = 1.f;
   p.chunk = splits > 1 ? kv_chunk : 0;
   p.status = status;
   p.order = order;

@@ -54,9 +54,10 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
   p.status = status; p.order = order; p.skip_rows = skip_rows;
   p.dk = a->dk; p.dv = a->dv;
   p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.gate_stride = a->gate_stride; p.gate_wide = a->gate && a->gate_wide;
-  p.maps = maps; p.raw = a->raw;
+  p.maps = maps; p.raw = a->raw; p.joint = a->joint; p.out_scale = a->out_scale;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
+  if (a->joint && maps > 1) return -1;
+  if (!a->joint && a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
   if (a->dk <= 64) return LaunchMixedKeys<64>(p, max_q_len, stream);
   if (a->dk <= 128) return LaunchMixedKeys<128>(p, max_q_len, stream);
   if (a->dk <= 192) return LaunchMixedKeys<192>(p, max_q_len, stream);

@@ -69,6 +69,9 @@ struct AttnParams {
   // maps > 1: query vector h (dk / maps columns wide) belongs to map h % maps of its key head, whose row holds the maps' keys side by side: the
   // query is staged at its map's columns among zeros, so keys and values are read once for all maps.
   int maps;
+  // joint: a cache row holds the keys of all key heads side by side as one key of dk columns, which every query head meets; values by key head
+  int joint;
+  float out_scale;   // multiplies the result (not of raw calls)
   int raw;           // partial results are written even without splits, and not merged here
 };
 
@@ -206,7 +209,7 @@ paged_attention_kernel(AttnParams p) {
         const int kl = item / CHUNKS, ch = item % CHUNKS;
         const int sl = __shfl_sync(0xffffffffu, slot, kl);
         const bool ok = sl >= 0 && ch * 8 < dk;
-        cp_async16(tk + koff(warp * 16 + kl, ch), p.k_cache + (ok ? (size_t(sl) * p.Hkv + kvh) * dk + ch * 8 : 0), ok);
+        cp_async16(tk + koff(warp * 16 + kl, ch), p.k_cache + (ok ? (p.joint ? size_t(sl) : size_t(sl) * p.Hkv + kvh) * dk + ch * 8 : 0), ok);
       }
 #pragma unroll
       for (int c = 0; c < CHUNKS_V / 2; ++c) {
@@ -487,7 +490,7 @@ paged_attention_kernel(AttnParams p) {
         scale_o = exp2f(M - mm);
         L = L * scale_o + exp2f(sk - mm);
       }
-      const float inv = (L > 0.f ? scale_o / L : 0.f) * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
+      const float inv = (L > 0.f ? scale_o / L : 0.f) * p.out_scale * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * dv + seg * SEG;
       const __nv_bfloat16* pg = p.gate + (p.gate_wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * dv + seg * SEG : 0);
 #pragma unroll
@@ -525,7 +528,7 @@ paged_attention_kernel(AttnParams p) {
         scale_o = exp2f(m - mm);
         l = l * scale_o + exp2f(sk - mm);
       }
-      const float inv = (l > 0.f ? scale_o / l : 0.f) * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
+      const float inv = (l > 0.f ? scale_o / l : 0.f) * p.out_scale * (p.gate_wide ? 1.f : attn_gate(p.gate, p.gate_stride, tok0 + tq, hq));
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * dv;
       const __nv_bfloat16* pg = p.gate + (p.gate_wide ? size_t(tok0 + tq) * p.gate_stride + size_t(hq) * dv : 0);
 #pragma unroll
@@ -542,7 +545,7 @@ paged_attention_kernel(AttnParams p) {
 template <int DV, bool FIT>
 __global__ void attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out, int out_stride,
-                                         int total_rows, int Hq, int splits, int dv, const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_wide) {
+                                         int total_rows, int Hq, int splits, int dv, const __nv_bfloat16* __restrict__ gate, int gate_stride, int gate_wide, float out_scale) {
   const int D = FIT ? DV : dv;
   pdl_launch_dependents();
   pdl_wait();
@@ -570,7 +573,7 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o, const
       if (d < D) acc[i] += w * po[d];
     }
   }
-  const float inv = (L > 0.f ? 1.f / L : 0.f) * (gate_wide ? 1.f : attn_gate(gate, gate_stride, tok, hq));
+  const float inv = (L > 0.f ? 1.f / L : 0.f) * out_scale * (gate_wide ? 1.f : attn_gate(gate, gate_stride, tok, hq));
   __nv_bfloat16* o = out + size_t(tok) * out_stride + size_t(hq) * D;
   const __nv_bfloat16* pg = gate + (gate_wide ? size_t(tok) * gate_stride + size_t(hq) * D : 0);
 #pragma unroll
@@ -600,7 +603,7 @@ static int LaunchAttentionMode(const AttnParams& p, int max_q_len, cudaStream_t 
   if (p.splits > 1 && !p.raw) {
     const int warps = 4;
     launch_pdl(attention_combine_kernel<DV, FIT>, dim3((p.total_rows + warps - 1) / warps), dim3(warps * 32), 0, stream,
-               static_cast<const float*>(p.part_o), static_cast<const float*>(p.part_ml), p.sinks, p.out, p.out_stride, p.total_rows, p.Hq, p.splits, p.dv, p.gate, p.gate_stride, p.gate_wide);
+               static_cast<const float*>(p.part_o), static_cast<const float*>(p.part_ml), p.sinks, p.out, p.out_stride, p.total_rows, p.Hq, p.splits, p.dv, p.gate, p.gate_stride, p.gate_wide, p.out_scale);
     if (cudaGetLastError() != cudaSuccess) return -4;
   }
   return 0;

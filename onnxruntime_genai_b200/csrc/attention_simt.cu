@@ -40,6 +40,7 @@ __global__ void __launch_bounds__(ASM_THREADS) attention_simt_kernel(OgbAttnLaye
   const int pos = past_lens[b] + t - cu[b], g = h / (a.Hq / a.Hkv);
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : (a.chunk > 0 ? pos / a.chunk * a.chunk : 0);
   const int32_t* table = tables + size_t(b) * table_cols;
+  const int kh = a.joint ? 1 : a.Hkv, kg = a.joint ? 0 : g;  // key heads of a cache row, the one this query meets
   const int dm = a.dk / a.maps, c0 = (h % a.maps) * dm;      // this query vector's columns of a key
   for (int i = threadIdx.x; i < dm; i += ASM_THREADS) sq[i] = as_f32(q[size_t(t) * q_stride + size_t(h) * dm + i]);
   float acc[COLS];
@@ -56,7 +57,7 @@ __global__ void __launch_bounds__(ASM_THREADS) attention_simt_kernel(OgbAttnLaye
     }
     __syncthreads();
     for (int k = warp; k < nk; k += ASM_THREADS / 32) {
-      const T* row = k_cache + (size_t(sslot[k]) * a.Hkv + g) * a.dk + c0;
+      const T* row = k_cache + (size_t(sslot[k]) * kh + kg) * a.dk + c0;
       float d = 0.f;
       for (int i = lane; i < dm; i += 32) d = fmaf(sq[i], as_f32(row[i]), d);
       d = warp_sum(d) * a.scale;
@@ -92,6 +93,7 @@ __global__ void __launch_bounds__(ASM_THREADS) attention_simt_kernel(OgbAttnLaye
     if (threadIdx.x == 0) { part_ml[row * 2] = 0.f; part_ml[row * 2 + 1] = 1.f; }
     return;
   }
+  inv *= a.out_scale;
   const T* gate = static_cast<const T*>(a.gate);
   if (gate && !a.gate_wide) inv *= 1.f / (1.f + expf(-as_f32(gate[size_t(t) * a.gate_stride + h])));
 #pragma unroll
@@ -341,7 +343,7 @@ OGB_API int ogb_attention_simt(const OgbAttnLayer* a, const void* q, int q_strid
   if (a->dv > 16 * ASM_THREADS || a->dk > 8192 || a->Hq > 65535) return -5;
   OgbAttnLayer l = *a;
   if (l.maps < 1) l.maps = 1;
-  if (l.Hkv <= 0 || l.Hq % l.Hkv || l.dk % l.maps || block_size <= 0 || (l.raw && l.sinks)) return -1;
+  if ((l.joint && l.maps > 1) || l.Hkv <= 0 || l.Hq % l.Hkv || l.dk % l.maps || block_size <= 0 || (l.raw && l.sinks)) return -1;
   if (l.raw && (long long)T * l.Hq * (l.dv + 2) * 4 > scratch_bytes) return -2;
   float* po = l.raw ? static_cast<float*>(scratch) : nullptr;
   float* ml = po ? po + size_t(T) * l.Hq * l.dv : nullptr;

@@ -41,6 +41,7 @@ OGB_API int ogb_attention_tc(const void* q, int q_stride, const void* k_cache, c
   if (Hkv <= 0 || Hq % Hkv || (q_stride % 8) || (out_stride % 8)) return -1;
   if (((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out)) & 15) != 0) return -1;
   TcAttnParams p{};
+  p.out_scale = 1.f;
   p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
   p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.block_table = block_table; p.table_cols = table_cols; p.block_size = block_size;
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;
@@ -70,6 +71,7 @@ OGB_API int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv,
   if (gate && ((gate_stride % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -1;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kr) | reinterpret_cast<uintptr_t>(out)) & 15) return -1;
   TcAttnParams p{};
+  p.out_scale = 1.f;
   p.q = static_cast<const __nv_bfloat16*>(q); p.q_stride = q_stride;
   p.cu_seqlens = cu_seqlens; p.past_lens = past_lens; p.block_size = 16;
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;

@@ -82,6 +82,8 @@ struct TcAttnParams {
   // entries of the other splits are marked empty.
   float *part_o, *part_ml;
   int splits, total_rows;
+  int joint;         // (MIX) one key of dk columns per cache row, which every query head meets; values by key head
+  float out_scale;   // multiplies the result
 };
 // entry of a query row in a grid of key vectors
 __device__ __forceinline__ int tca_query(int kvh, int i, int G, int maps) { return maps > 1 ? ((kvh / maps) * G + i) * maps + kvh % maps : kvh * G + i; }
@@ -250,7 +252,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           if constexpr (MIX) {
             if (is_k) {
 #pragma unroll
-              for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh * p.dk + h * 64, slot0);
+              for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], (p.joint ? 0 : kvh * p.dk) + h * 64, slot0);
             } else {
 #pragma unroll
               for (int h = 0; h < Cfg::V_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh / p.maps * p.dv + h * 64, slot0);
@@ -500,7 +502,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
         scale_o = m_ref == -INFINITY ? 0.f : exp2f(m_ref - mm);
         l = l * scale_o + exp2f(sk - mm);
       }
-      float inv = l > 0.f ? scale_o / l : 0.f;
+      float inv = l > 0.f ? scale_o / l * p.out_scale : 0.f;
       if (p.gate && !wide) inv /= 1.f + __expf(-bf2f(p.gate[size_t(tok0 + tq) * p.gate_stride + hq]));
       __nv_bfloat16* po = p.out + size_t(tok0 + tq) * p.out_stride + size_t(hq) * v_cols + half * OC;
       const bool raw = MIX && p.part_o;
@@ -565,7 +567,7 @@ template <int DK, int DV, int BN, bool MIX, bool CAP>
 static int LaunchTcForm(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
   using Cfg = TcaCfg<DK, DV, BN>;
   auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP>;
-  const int kw = p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
+  const int kw = MIX && p.joint ? p.dk : p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
   CUtensorMap mk, mv;

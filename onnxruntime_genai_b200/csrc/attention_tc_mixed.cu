@@ -47,6 +47,8 @@ OGB_API int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_s
   p.out = static_cast<__nv_bfloat16*>(out); p.out_stride = out_stride;
   p.sinks = a->sinks; p.scale = a->scale; p.softcap = a->softcap; p.window = a->window; p.local = a->chunk;
   p.B = B; p.Hq = a->Hq; p.Hkv = a->Hkv * maps; p.min_rows = min_rows; p.status = status;
+  p.joint = a->joint; p.out_scale = a->out_scale;
+  if (a->joint && maps > 1) return -1;
   p.dk = a->dk / maps; p.dv = a->dv; p.maps = maps;
   p.gate_wide = a->gate && a->gate_wide;
   if (a->raw) {
@@ -56,7 +58,7 @@ OGB_API int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_s
   }
   p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.gate_stride = a->gate_stride;
   cudaStream_t s = static_cast<cudaStream_t>(stream_);
-  if (maps == 1 && !a->raw && a->dk == a->dv && (a->dk == 64 || a->dk == 128)) return LaunchTcUniform(p, a->dk, k_cache, v_cache, max_q_len, cache_slots, s);
+  if (maps == 1 && !a->raw && !a->joint && a->dk == a->dv && (a->dk == 64 || a->dk == 128)) return LaunchTcUniform(p, a->dk, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 64) return LaunchTcMixedKeys<64>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 128) return LaunchTcMixedKeys<128>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 192) return LaunchTcMixedKeys<192>(p, k_cache, v_cache, max_q_len, cache_slots, s);

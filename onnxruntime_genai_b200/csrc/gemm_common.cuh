@@ -87,7 +87,7 @@ struct GemmParams {
   int act_pair;         // tiles hold 64 gate rows + 64 up rows, output has N/2 columns: 1 = silu(gate)*up,
                         // 2 = clamped SwiGLU: g = min(gate, limit), u = clamp(up, +-limit), g*sigmoid(alpha*g)*(u+1),
                         // 3 = max(gate, 0)*up, 4 = gelu_tanh(gate)*up
-                        // 3 = max(gate, 0)*up
+  int act_one;          // > 0: 1 + activation of every output column (see act_one)
   float act_alpha, act_limit;
   const void* residual;
   int ldr;
@@ -140,6 +140,20 @@ __device__ __forceinline__ uint32_t pack_f16x2(float a, float b) {
 __device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
 // 0.5 x (1 + tanh(y)) = x sigmoid(2 y), y = sqrt(2 / pi) (x + 0.044715 x^3)
 __device__ __forceinline__ float gelu_tanh(float x) { return x / (1.f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x))); }
+
+// kind - 1: 0 SiLU, 1 GELU(tanh), 2 ReLU, 3 GELU(erf), 4 ReLU^2
+__device__ __forceinline__ float act_one(int kind, float x) {
+  if (kind == 1) return x / (1.f + expf(-x));
+  if (kind == 2) return x / (1.f + expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+  if (kind == 4) return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
+  x = fmaxf(x, 0.f);
+  return kind == 5 ? x * x : x;
+}
+// (out of line: fetched cold by the epilogues)
+static __device__ __noinline__ void epi_act8(int kind, float (&v)[8]) {
+#pragma unroll
+  for (int j = 0; j < 8; ++j) v[j] = act_one(kind, v[j]);
+}
 
 __device__ __forceinline__ uint32_t cluster_ctarank() { uint32_t r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }
 __device__ __forceinline__ void cluster_sync_all() {
@@ -471,6 +485,7 @@ __device__ __forceinline__ void gemm_epilogue(const GemmParams& p, uint8_t* smem
         const int pos_raw = roped ? p.rope.positions[m] : 0;
         const int slot = roped ? p.rope.slots[m] : -1;
         reduce8(mc, oc * 8, rs, v);
+        if (p.act_one) epi_act8(p.act_one, v);
         if (roped) {
           // Fused rotary embedding + KV-cache append of a QKV projection (heads never straddle a tile: 128 % D == 0).
           // Query heads go to C rotated; key heads go rotated, value heads as they are, to this token's cache slot.

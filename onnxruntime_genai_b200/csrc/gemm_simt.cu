@@ -4,6 +4,7 @@
 // and the grouped form over token rows sorted by expert (tile list of moe.cu): C[r, n] = sum_k A[map(r), k] * W[expert(r) * N + n, k].
 // One CTA = a 64 x 64 output tile, 16 columns of K at a time through shared memory, 4 x 4 outputs per thread.
 #include "common.cuh"
+#include "gemm_common.cuh"
 #include "kernels.h"
 
 namespace ogb {
@@ -12,6 +13,7 @@ struct SimtGemmParams {
   const void* A; const void* W; void* C; const float* residual; const void* bias;
   int lda, a_cols, ldw, ldc, c_cols, ldr;
   int M, N, K;
+  int act;      // 0 none, else 1 + activation (see act_one)
   // grouped form: per token tile (blockIdx.y) its expert, first row and rows; row_map (may be null): row of A for every sorted row
   const int32_t *tile_expert, *tile_row0, *tile_rows, *num_tiles, *row_map;
 };
@@ -65,6 +67,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(SimtGemmParams p) {
       if (n >= p.N) continue;
       float v = acc[i][j];
       if (p.bias) v += ld_f32(static_cast<const T*>(p.bias) + n);
+      if (p.act) v = act_one(p.act, v);
       if (p.residual) v += p.residual[size_t(m) * p.ldr + n];
       TO* dst = static_cast<TO*>(p.C) + size_t(m) * p.ldc + size_t(z) * p.c_cols + n;
       if constexpr (sizeof(TO) == 4) *dst = v; else *dst = f2bf(v);
@@ -77,13 +80,13 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(SimtGemmParams p) {
 using namespace ogb;
 
 // in_fp32 / out_fp32: element types of A and W / of C (else bf16).  residual (fp32, may be C itself) and bias [N] (in A's type)
-// only with batch == 1.
+// only with batch == 1.  act: 0, or 1 + the activation of the result (numbers as in ogb_gemm_bf16), before the residual.
 OGB_API int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K,
-                          int batch, const float* residual, int ldr, const void* bias, int in_fp32, int out_fp32, void* stream_) {
+                          int batch, const float* residual, int ldr, const void* bias, int act, int in_fp32, int out_fp32, void* stream_) {
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   if ((residual || bias) && batch != 1) return -1;
   if (M > 64 * 65535 || batch > 65535) return -1;
-  SimtGemmParams p{A, W, C, residual, bias, lda, a_cols, ldw, ldc, c_cols, ldr, M, N, K, nullptr, nullptr, nullptr, nullptr, nullptr};
+  SimtGemmParams p{A, W, C, residual, bias, lda, a_cols, ldw, ldc, c_cols, ldr, M, N, K, act, nullptr, nullptr, nullptr, nullptr, nullptr};
   const dim3 grid((N + 63) / 64, (M + 63) / 64, batch);
   auto s = static_cast<cudaStream_t>(stream_);
   bool ok;
@@ -101,7 +104,7 @@ OGB_API int ogb_moe_gemm_simt(const void* A, int lda, const void* W, void* C, in
                               void* stream_) {
   if (N <= 0 || K <= 0 || max_tiles <= 0) return 0;
   if (token_tile > 64 || max_tiles > 65535 || !tile_expert || !tile_row0 || !tile_rows || !num_tiles) return -1;
-  SimtGemmParams p{A, W, C, nullptr, nullptr, lda, 0, K, ldc, 0, 0, 0, N, K, tile_expert, tile_row0, tile_rows, num_tiles, row_map};
+  SimtGemmParams p{A, W, C, nullptr, nullptr, lda, 0, K, ldc, 0, 0, 0, N, K, 0, tile_expert, tile_row0, tile_rows, num_tiles, row_map};
   const dim3 grid((N + 63) / 64, max_tiles, 1);
   auto s = static_cast<cudaStream_t>(stream_);
   const bool ok = fp32 ? launch_pdl(gemm_simt_kernel<float, float>, grid, dim3(256), 0, s, p)

@@ -552,6 +552,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const
               }
             }
           }
+          if (p.act_one) epi_act8(p.act_one, v);
           const int col = col0 + oc * 8;
           if (col >= n_out) continue;
           if (p.residual && p.res_fp32) {
@@ -750,7 +751,8 @@ OGB_API long long ogb_comm_capacity(int device) {
 // interleaved in blocks of 64); bit 2: fused all-reduce over the registered symmetric buffers; bit 3: fused
 // reduce-scatter by token rows instead (rank r ends up with rows [r * ceil(M / world), ...) of the sum, written as
 // rows 0.. of C; residual, if given, is that slice too); bit 4: activations gathered from the ranks' pushes; bit 5: the residual
-// is fp32; bit 6: the paired activation is max(gate, 0) * up; bit 7: it is gelu_tanh(gate) * up.
+// is fp32; bit 6: the paired activation is max(gate, 0) * up; bit 7: it is gelu_tanh(gate) * up; bits 8 .. 10: 1 + the
+// activation of every output column (see act_one), before the residual.
 OGB_API int ogb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
                           const void* bias, const void* residual, int ldr, int flags, int splits, int device, int* status,
                           int sm_count, void* stream_) {
@@ -793,7 +795,9 @@ OGB_API int ogb_gemm_bf16_fused(const void* A, int lda, const void* W, int ldw, 
   p.splits = splits; p.kb_per_split = kb_per; p.total_kb = total_kb;
   p.C = C; p.ldc = ldc; p.out_fp32 = out_fp32; p.act_pair = act_pair ? ((flags >> 6) & 1 ? 3 : ((flags >> 7) & 1 ? 4 : 1)) : 0;
   p.residual = residual; p.ldr = ldr; p.res_fp32 = (flags >> 5) & 1;
-  if ((p.res_fp32 || p.act_pair >= 3) && fused_ar) return -1;      // the reductions carry bf16 rows
+  p.act_one = (flags >> 8) & 7;
+  if ((p.res_fp32 || p.act_pair >= 3 || p.act_one) && fused_ar) return -1;      // the reductions carry bf16 rows (of sums that are not complete)
+  if (p.act_one > 5 || (p.act_one && act_pair)) return -1;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.status = status;
   p.pdl = pdl_enabled;
@@ -901,7 +905,8 @@ OGB_API int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_col
 // [experts * N, K], the device-built tile list (ogb_moe_sort) gives for every token tile its expert, first
 // row and row count.  C[row, :] = A[row, :] * W[expert(row)]^T (+ bias[expert]) (+ paired activation).
 // `token_tile` must be the tile size the list was built for; `max_tiles` bounds the list length (the grid).
-// flags bit 1: paired activation; act_kind selects it (1 = silu(gate)*up, 2 = clamped SwiGLU(alpha, limit)).
+// flags bit 1: paired activation; act_kind selects it (1 = silu(gate)*up, 2 = clamped SwiGLU(alpha, limit)).  Without it: act_kind > 0 is 1 + the
+// activation of every output column (see act_one).
 OGB_API int ogb_moe_gemm(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int rows_total, int N, int K, int experts,
                          const void* bias, int flags, int act_kind, float act_alpha, float act_limit, const int* tile_expert,
                          const int* tile_row0, const int* tile_rows, const int* num_tiles, int max_tiles, int token_tile,
@@ -923,6 +928,8 @@ OGB_API int ogb_moe_gemm(const void* A, int lda, const void* W, int ldw, void* C
   p.total_kb = (K + GEMM_BLOCK_K - 1) / GEMM_BLOCK_K;
   p.splits = 1; p.kb_per_split = p.total_kb;
   p.C = C; p.ldc = ldc; p.out_fp32 = flags & 1; p.act_pair = act_pair ? act_kind : 0;
+  p.act_one = act_pair ? 0 : act_kind;
+  if (act_kind < 0 || p.act_one > 5) return -1;
   p.act_alpha = act_alpha; p.act_limit = act_limit;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.status = status;

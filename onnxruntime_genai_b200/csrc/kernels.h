@@ -28,7 +28,7 @@ int ogb_comm_set_options(int use_nvls, long long two_shot_bytes, int p2p_two_hop
 long long ogb_comm_capacity(int device);
 // flags: bit 0 fp32 output, bit 1 paired silu(gate)*up epilogue, bit 2 fused tensor-parallel all-reduce,
 // bit 3 fused reduce-scatter by token rows (sequence-parallel form), bit 5 the residual is fp32, bit 6 the paired activation is
-// max(gate, 0) * up
+// max(gate, 0) * up, bits 8 .. 10: 1 + the activation of every output column (0: none; 0 SiLU, 1 GELU(tanh), 2 ReLU, 3 GELU(erf), 4 ReLU^2)
 int ogb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, const void* bias,
                   const void* residual, int ldr, int flags, int splits, int device, int* status, int sm_count, void* stream);
 
@@ -53,7 +53,7 @@ int ogb_gemm_bf16_batched(const void* A, int lda, int a_width, int a_cols, const
 
 // ---- gemm_simt.cu: fp32 products and bf16 products TMA cannot address
 int ogb_gemm_simt(const void* A, int lda, int a_cols, const void* W, int ldw, void* C, int ldc, int c_cols, int M, int N, int K, int batch,
-                  const float* residual, int ldr, const void* bias, int in_fp32, int out_fp32, void* stream);
+                  const float* residual, int ldr, const void* bias, int act, int in_fp32, int out_fp32, void* stream);
 
 // Grouped expert product over token rows sorted by expert in plain arithmetic (tile list of ogb_moe_sort, tiles of at most 64 rows).
 int ogb_moe_gemm_simt(const void* A, int lda, const void* W, void* C, int ldc, int N, int K, const int32_t* tile_expert, const int32_t* tile_row0,
@@ -62,14 +62,28 @@ int ogb_moe_gemm_simt(const void* A, int lda, const void* W, void* C, int ldc, i
 // ---- layer_ops.cu: fp32 residual stream
 // (copy, may be null: the rows as bf16 beside the stream)
 int ogb_embedding_stream(const int32_t* ids, const void* table, int table_fp32, float* out, void* copy, int T, int H, int vocab, float scale, void* stream);
-int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const float* b, void* out, int out_fp32, int n_rows, int H, float eps,
-                    int layernorm, void* stream);
+// Norm of rows of the fp32 stream x [.., H]: out[i] = norm(x[r]) * w + b, r = rows ? rows[i] : i; w2 (may be null): out2[i] = norm(x[r]) * w2.  RMS norm, or
+// layer norm.  y (may be null): y[r] (in the compute type, like out), or (inv_pos not null) the weighted sum of experts' rows sum_j topk_w[r, j] *
+// y[inv_pos[r, j]], j < k, is added to the row first, in place where rows is null.
+typedef struct OgbNormStream {
+  float* x;
+  const int32_t* rows;
+  const float *w, *b, *w2;
+  void *out, *out2;
+  const void* y;
+  const int32_t* inv_pos; const float* topk_w;
+  int ldy, k, n_rows, H, layernorm, fp32;
+  float eps;
+} OgbNormStream;
+int ogb_norm_stream(const OgbNormStream* p, void* stream);
 // Head norms, rotation and cache append of an attention layer: proj row t holds Hq query heads and Hkv key heads of key_row columns (the
 // first `dim` are the head, the rest zeros) and Hkv value heads of value_row columns.  Queries are replaced in place, keys and values go to
 // row slots[t] of the caches (slot < 0: nowhere).  Norm weights fp32 [dim] (null: no norm), cos / sin fp32 [max_pos, rot / 2] (rot 0: none).
+// talk (may be null) fp32 [Hq, Hq]: the queries are not replaced; mixed row t [Hq][Hkv][key_row] gets sum over the heads g of key head c's group
+// of talk[h, g] * q_g as part c of head h.
 int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
                  const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
-                 void* v_cache, int T, int fp32, void* stream);
+                 void* v_cache, int T, const float* talk, void* mixed, int fp32, void* stream);
 // h[t] += w * v / sqrt(mean(v^2) + eps), x[t] = h[t] as bf16 (x may be null).  v = y[t], or (inv_pos not null) the weighted sum of the
 // experts' rows sum_j topk_w[t, j] * y[inv_pos[t, j]], j < k.
 int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const float* w, float eps, void* x, const int32_t* inv_pos, const float* topk_w, int k,
@@ -99,12 +113,33 @@ typedef struct OgbBigram {
   float scale;
 } OgbBigram;
 int ogb_embedding_bigram(const OgbBigram* p, const void* table, const void* bigram, float* out, void* stream);
-// Expert activations on rows of alternating (gate, up) columns [n, 2 I]: kind 0 silu(g) * u, 1 clamped g * sigmoid(alpha g) * (u + 1).
+// Expert activations on rows of alternating (gate, up) columns [n, 2 I]: kind 0 silu(g) * u, 1 clamped g * sigmoid(alpha g) * (u + 1);
+// on rows [n, I]: kind 2 max(x, 0)^2.
 int ogb_expert_act(const void* gu, void* out, long long n, int I, int kind, float alpha, float limit, int fp32, void* stream);
 int ogb_act_mul_rows(const void* x, int ldx, void* out, int ldo, int T, int I, int act, int fp32, void* stream);
 int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const void* bias, void* cache, int ldcache, const int32_t* slots,
                          const int32_t* positions, const int32_t* cu_seqlens, const int32_t* past_lens, const int32_t* block_table, int table_cols,
                          int block_size, void* out, int T, int B, int C, int L, int silu, int fp32, void* stream);
+
+// ---- recurrent.cu: recurrent mixers over packed sequences (states fp32, at state + slot * slot_stride; a request without a past starts from zero)
+// Gated average per column: S <- (1 - sigmoid(z)) S + sigmoid(z) * c(x), c(x) = x + 1/2 for x >= 0, sigmoid(x) below; out = S * silu(g) * scale.
+// z, x, g: columns of rows of ld elements, W each.
+int ogb_min_gru(const void* z, const void* x, const void* g, int ld, float* state, long long slot_stride, const int32_t* slots, const int32_t* cu_seqlens,
+                const int32_t* past_lens, void* out, int ldo, int B, int W, float scale, int max_q_len, int fp32, void* stream);
+// Matrix memories of H heads with keys of d and values of dv columns.  q, k, v, g: columns of rows of ld elements ([H, d], [H, d], [H, dv], [H, dv]); gates:
+// fp32 rows of ldg, H logits of the input gates and H of the forget gates, to which gate_b [2 H] is added; out rows of ldo.  State of a slot: memories
+// [H, d, dv], normalisers [H, d], maxima [H].  max_q_len: the most tokens a request of the step feeds, T the step's tokens.
+typedef struct OgbMlstm {
+  const void *q, *k, *v, *g;
+  const float *gates, *gate_b, *norm_w;
+  void* out;
+  float* state;
+  const int32_t *slots, *cu_seqlens, *past_lens;
+  long long slot_stride;
+  int ld, ldg, ldo, B, H, d, dv, T, max_q_len, fp32;
+  float cap, eps;
+} OgbMlstm;
+int ogb_mlstm(const OgbMlstm* a, void* stream);
 
 // ---- attention_tc.cu, latent form (long prompts over expanded keys and values)
 int ogb_attention_tc_latent_supported(int dim, int rot, int vdim);
@@ -118,6 +153,8 @@ int ogb_attention_tc_latent(const void* q, int q_stride, const void* kv, int ldk
 // window > 0: position p sees (p - window, p]; chunk > 0: the keys of p's own run of `chunk` positions; 0: every earlier key.
 // sinks (may be null) [Hq]: a logit in each head's denominator.  gate (may be null) [tokens, gate_stride], in the model's element type: a
 // head's output is multiplied by the sigmoid of its entry (gate_wide: a row holds Hq * dv entries, one for every output column).
+// joint: dk counts the columns of all key heads of a position (caches [slots, dk] and [slots, Hkv, dv]); every query is that wide and meets all of
+// them.  The result is multiplied by out_scale (not in raw calls).
 // softcap > 0: a scaled score s becomes softcap * tanh(s / softcap).  maps > 1: query vector h belongs to map h % maps, is dk / maps columns
 // wide and meets only that map's columns of its key head (Hq counts query vectors, a key head holds the vectors of all maps side by side).
 // raw: instead of `out`, fp32 partial results go to scratch: [splits, tokens * Hq, dv] sums and, behind them, [splits, tokens * Hq, 2] (maximum
@@ -129,6 +166,8 @@ typedef struct OgbAttnLayer {
   const void* gate;
   int gate_wide, maps, raw;
   float softcap;
+  int joint;
+  float out_scale;
 } OgbAttnLayer;
 // Differential attention on raw partial results of H heads with two maps each (query vectors 2 h and 2 h + 1): with a1 and a2 the maps'
 // results, o = a1 - lambda * a2, out = o / sqrt(mean(o^2) + eps) * post over the head's first vdim columns (columns vdim .. dv - 1 are zeros),

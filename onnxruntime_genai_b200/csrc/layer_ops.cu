@@ -90,26 +90,73 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(OgbBigram p, cons
 }
 
 // ------------------------------------------------------------------------------------ norm of the fp32 stream
-// One CTA per output row; the row is kept in shared memory, the variance is taken from the deviations (a second pass over them).
+// (See OgbNormStream.)  One CTA per output row; the row is kept in shared memory, the variance is taken from the deviations (a second pass over
+// them).  ADD: rows in T are added to the stream's row first.
 template <typename T>
-__global__ void __launch_bounds__(256) norm_stream_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, const float* __restrict__ w,
-                                                          const float* __restrict__ b, T* __restrict__ out, int H, float eps, int layernorm) {
+__device__ __forceinline__ float4 added4(const OgbNormStream& p, int t, int i, float4 v) {
+  auto one = [&](const T* y, float w) {
+    float2 a, c;
+    if constexpr (sizeof(T) == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(y);
+      a = make_float2(q.x, q.y); c = make_float2(q.z, q.w);
+    } else {
+      const uint2 q = *reinterpret_cast<const uint2*>(y);
+      a = unpack_bf16x2(q.x); c = unpack_bf16x2(q.y);
+    }
+    v.x = fmaf(w, a.x, v.x); v.y = fmaf(w, a.y, v.y); v.z = fmaf(w, c.x, v.z); v.w = fmaf(w, c.y, v.w);
+  };
+  const T* y = static_cast<const T*>(p.y) + i;
+  if (!p.inv_pos) {
+    one(y + size_t(t) * p.ldy, 1.f);
+    return v;
+  }
+#pragma unroll 4
+  for (int j = 0; j < p.k; ++j) {
+    const int r = p.inv_pos[size_t(t) * p.k + j];
+    if (r >= 0) one(y + size_t(r) * p.ldy, p.topk_w[size_t(t) * p.k + j]);
+  }
+  return v;
+}
+
+template <typename T, bool ADD>
+__global__ void __launch_bounds__(256) norm_stream_kernel(OgbNormStream p) {
   extern __shared__ float row[];
   __shared__ float part[2][8];
   pdl_launch_dependents();
   pdl_wait();
-  const float* src = x + size_t(rows ? rows[blockIdx.x] : blockIdx.x) * H;
+  const int H = p.H, t0 = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+  float* src = p.x + size_t(t0) * H;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  const bool vec = (H & 3) == 0;
+  const bool vec = (H & 3) == 0 && (!ADD || (p.ldy & 3) == 0);
+  const float eps = p.eps;
+  const int layernorm = p.layernorm;
   float sum = 0.f;
   if (vec) {
     for (int i = threadIdx.x; i < H / 4; i += blockDim.x) {
-      const float4 v = reinterpret_cast<const float4*>(src)[i];
+      float4 v = reinterpret_cast<const float4*>(src)[i];
+      if constexpr (ADD) {
+        v = added4<T>(p, t0, i * 4, v);
+        if (!p.rows) reinterpret_cast<float4*>(src)[i] = v;
+      }
       reinterpret_cast<float4*>(row)[i] = v;
       sum += (v.x + v.y) + (v.z + v.w);
     }
   } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = src[i]; row[i] = v; sum += v; }
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      float v = src[i];
+      if constexpr (ADD) {
+        const T* y = static_cast<const T*>(p.y) + i;
+        if (!p.inv_pos) v += to_f32(y[size_t(t0) * p.ldy]);
+        else
+          for (int j = 0; j < p.k; ++j) {
+            const int r = p.inv_pos[size_t(t0) * p.k + j];
+            if (r >= 0) v = fmaf(p.topk_w[size_t(t0) * p.k + j], to_f32(y[size_t(r) * p.ldy]), v);
+          }
+        if (!p.rows) src[i] = v;
+      }
+      row[i] = v;
+      sum += v;
+    }
   }
   float mean = 0.f;
   if (layernorm) {
@@ -137,20 +184,33 @@ __global__ void __launch_bounds__(256) norm_stream_kernel(const float* __restric
   float t = 0.f;
   for (int i = 0; i < nw; ++i) t += part[1][i];
   const float inv = 1.f / sqrtf(t / H + eps);
-  T* dst = out + size_t(blockIdx.x) * H;
+  T* dst = static_cast<T*>(p.out) + size_t(blockIdx.x) * H;
+  T* dst2 = p.w2 ? static_cast<T*>(p.out2) + size_t(blockIdx.x) * H : nullptr;
   if (vec) {
+    auto put = [&](T* d, int i, float4 o) {
+      if constexpr (sizeof(T) == 4) reinterpret_cast<float4*>(d)[i] = o;
+      else reinterpret_cast<uint2*>(d)[i] = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+    };
     for (int i = threadIdx.x; i < H / 4; i += blockDim.x) {
-      const float4 v = reinterpret_cast<const float4*>(row)[i], g = reinterpret_cast<const float4*>(w)[i];
-      float4 o = make_float4((v.x - mean) * inv * g.x, (v.y - mean) * inv * g.y, (v.z - mean) * inv * g.z, (v.w - mean) * inv * g.w);
-      if (b) {
-        const float4 c = reinterpret_cast<const float4*>(b)[i];
+      const float4 v = reinterpret_cast<const float4*>(row)[i], g = reinterpret_cast<const float4*>(p.w)[i];
+      const float4 u = make_float4((v.x - mean) * inv, (v.y - mean) * inv, (v.z - mean) * inv, (v.w - mean) * inv);
+      float4 o = make_float4(u.x * g.x, u.y * g.y, u.z * g.z, u.w * g.w);
+      if (p.b) {
+        const float4 c = reinterpret_cast<const float4*>(p.b)[i];
         o.x += c.x; o.y += c.y; o.z += c.z; o.w += c.w;
       }
-      if constexpr (sizeof(T) == 4) reinterpret_cast<float4*>(dst)[i] = o;
-      else reinterpret_cast<uint2*>(dst)[i] = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+      put(dst, i, o);
+      if (dst2) {
+        const float4 e = reinterpret_cast<const float4*>(p.w2)[i];
+        put(dst2, i, make_float4(u.x * e.x, u.y * e.y, u.z * e.z, u.w * e.w));
+      }
     }
   } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = from_f32<T>((row[i] - mean) * inv * w[i] + (b ? b[i] : 0.f));
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float u = (row[i] - mean) * inv;
+      dst[i] = from_f32<T>(u * p.w[i] + (p.b ? p.b[i] : 0.f));
+      if (dst2) dst2[i] = from_f32<T>(u * p.w2[i]);
+    }
   }
 }
 
@@ -448,13 +508,81 @@ __global__ void __launch_bounds__(256) qkv_prep_pieces_kernel(T* __restrict__ pr
   }
 }
 
+// The same for heads whose scores are mixed: head h's scores are sum_g talk[h, g] * (scores of g), so with the queries of a key head's group G_c mixed
+// into one query part, m[h, c] = sum over g in G_c of talk[h, g] q_g, they are the product of [m[h, 0] | m[h, 1] | ...] with the keys of all key
+// heads side by side.  The parts are summed in fp32 from the normed and rotated queries and rounded once.  One CTA per token: its warps prepare heads
+// (queries into shared memory, keys and values to the cache), then every thread mixes columns; rows of `mixed` are [Hq][Hkv][key_row].
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_prep_mixed_kernel(const T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p,
+                                                             const float* __restrict__ talk, T* __restrict__ mixed) {
+  extern __shared__ float sm[];
+  float* st = sm;                            // [Hq][Hq]
+  float* sq = sm + (p.Hq * p.Hq + 1) / 2 * 2;      // [Hq][key_row]
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < p.Hq * p.Hq; i += blockDim.x) st[i] = talk[i];
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const T* row = proj + size_t(t) * p.ldp;
+  const int slot = p.slots[t], half = p.rot >> 1;
+  const size_t at = size_t(min(max(p.positions[t], 0), p.max_pos - 1)) * half;
+  for (int head = warp; head < p.Hq + p.Hkv; head += nw) {
+    const bool is_q = head < p.Hq;
+    const T* src = row + size_t(head) * p.key_row;
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    float inv = 1.f;
+    if (w) {
+      float sq2 = 0.f;
+      for (int i = lane; i < p.dim; i += 32) { const float f = to_f32(src[i]); sq2 = fmaf(f, f, sq2); }
+      inv = 1.f / sqrtf(warp_sum(sq2) / p.dim + p.eps);
+    }
+    auto normed = [&](int i) { const float f = to_f32(src[i]); return w ? f * inv * w[i] : f; };
+    T* dst = is_q || slot < 0 ? nullptr : k_cache + (size_t(slot) * p.Hkv + (head - p.Hq)) * p.key_row;
+    auto put = [&](int i, float f) {
+      if (is_q) sq[head * p.key_row + i] = f;
+      else if (dst) dst[i] = from_f32<T>(f);
+    };
+    for (int i = lane; i < half; i += 32) {
+      const float a = normed(i), b = normed(i + half), c = p.cos[at + i], s = p.sin[at + i];
+      put(i, a * c - b * s);
+      put(i + half, b * c + a * s);
+    }
+    for (int i = p.rot + lane; i < p.key_row; i += 32) put(i, i < p.dim ? normed(i) : 0.f);
+  }
+  if (slot >= 0) {
+    const T* src = row + size_t(p.Hq + p.Hkv) * p.key_row;
+    T* dst = v_cache + size_t(slot) * p.Hv * p.value_row;
+    for (int i = threadIdx.x; i < p.Hv * p.value_row; i += blockDim.x) dst[i] = src[i];
+  }
+  __syncthreads();
+  const int G = p.Hq / p.Hkv, cols = p.Hkv * p.key_row;
+  T* out = mixed + size_t(t) * p.Hq * cols;
+  for (int i = threadIdx.x * 2; i < p.Hq * cols; i += blockDim.x * 2) {      // (key_row is a multiple of 8)
+    const int h = i / cols, c = (i - h * cols) / p.key_row, d = i % p.key_row;
+    const float* q = sq + c * G * p.key_row + d;
+    const float* m = st + h * p.Hq + c * G;
+    float f[2] = {0.f, 0.f};
+    for (int g = 0; g < G; ++g) {
+      const float2 v = *reinterpret_cast<const float2*>(q + g * p.key_row);
+      f[0] = fmaf(m[g], v.x, f[0]);
+      f[1] = fmaf(m[g], v.y, f[1]);
+    }
+    st_cols<T, 2>(out + i, f);
+  }
+}
+
 // ------------------------------------------------------------------------------------ experts' activations
 // Rows of alternating (gate, up) columns.  kind 0: silu(g) * u; 1: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + 1).
+// Rows without gates: kind 2: max(x, 0)^2.
 template <typename T>
 __global__ void expert_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long n, int kind, float alpha, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   for (long i = long(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += long(gridDim.x) * blockDim.x) {
+    if (kind == 2) {
+      const float x = fmaxf(to_f32(gu[i]), 0.f);
+      out[i] = from_f32<T>(x * x);
+      continue;
+    }
     float g = to_f32(gu[2 * i]), u = to_f32(gu[2 * i + 1]), r;
     if (kind == 0) {
       r = g / (1.f + expf(-g)) * u;
@@ -563,16 +691,17 @@ OGB_API int ogb_add_tanh_norm(const OgbTanhNorm* p, void* stream) {
   return ok ? 0 : -4;
 }
 
-// rows (may be null): out row i is the norm of x row rows[i].  w, b fp32 [H] (b may be null).
-OGB_API int ogb_norm_stream(const float* x, const int32_t* rows, const float* w, const float* b, void* out, int out_fp32, int n_rows, int H, float eps,
-                            int layernorm, void* stream) {
-  if (n_rows <= 0) return 0;
-  if (H <= 0 || H > 48 * 1024 / 4 - 64) return -1;
+OGB_API int ogb_norm_stream(const OgbNormStream* p, void* stream) {
+  if (p->n_rows <= 0) return 0;
+  if (p->H <= 0 || p->H > 48 * 1024 / 4 - 64 || (p->inv_pos && (!p->y || !p->topk_w)) || (p->w2 && !p->out2)) return -1;
+  auto addr = [](const void* a) { return reinterpret_cast<uintptr_t>(a); };
+  if (p->H % 4 == 0 && ((addr(p->x) | addr(p->w) | addr(p->b) | addr(p->w2) | addr(p->out) | addr(p->out2) | addr(p->y)) & (p->fp32 ? 15 : 7))) return -1;
   auto s = static_cast<cudaStream_t>(stream);
-  const dim3 block(H >= 1024 ? 256 : 128);
-  const bool ok = out_fp32 ? launch_pdl(norm_stream_kernel<float>, dim3(n_rows), block, size_t(H) * 4, s, x, rows, w, b, static_cast<float*>(out), H, eps, layernorm)
-                           : launch_pdl(norm_stream_kernel<__nv_bfloat16>, dim3(n_rows), block, size_t(H) * 4, s, x, rows, w, b,
-                                        static_cast<__nv_bfloat16*>(out), H, eps, layernorm);
+  const dim3 block(p->H >= 1024 ? 256 : 128), grid(p->n_rows);
+  const size_t smem = size_t(p->H) * 4;
+  using H = __nv_bfloat16;
+  const bool ok = p->fp32 ? (p->y ? launch_pdl(norm_stream_kernel<float, true>, grid, block, smem, s, *p) : launch_pdl(norm_stream_kernel<float, false>, grid, block, smem, s, *p))
+                          : (p->y ? launch_pdl(norm_stream_kernel<H, true>, grid, block, smem, s, *p) : launch_pdl(norm_stream_kernel<H, false>, grid, block, smem, s, *p));
   return ok ? 0 : -4;
 }
 
@@ -626,7 +755,7 @@ OGB_API int ogb_add_normed(float* h, const void* y, int ldy, int y_fp32, const f
 
 OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, int key_row, int value_row, const float* q_norm, const float* k_norm, float eps,
                          const int32_t* positions, const float* cos, const float* sin, int rot, int max_pos, const int32_t* slots, void* k_cache,
-                         void* v_cache, int T, int fp32, void* stream) {
+                         void* v_cache, int T, const float* talk, void* mixed, int fp32, void* stream) {
   if (T <= 0) return 0;
   if (Hq <= 0 || Hkv <= 0 || Hv <= 0 || dim <= 0 || dim > key_row || rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (!cos || !sin || max_pos <= 0))) return -1;
   const QkvPrep p{ldp, Hq, Hkv, Hv, dim, key_row, value_row, rot, max_pos > 0 ? max_pos : 1, T, q_norm, k_norm, cos, sin, positions, slots, eps};
@@ -634,6 +763,21 @@ OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, 
   const dim3 grid(unsigned((items + 7) / 8));
   auto s = static_cast<cudaStream_t>(stream);
   const int elem = fp32 ? 4 : 2;
+  if (talk) {
+    const size_t smem = (size_t(Hq) * (Hq + key_row) + 1) * 4;
+    if (!mixed || Hq % Hkv || key_row % 8 || smem > 200 * 1024 || (reinterpret_cast<uintptr_t>(mixed) & 15)) return -1;
+    static bool done32[OGB_MAX_DEVICES] = {}, done16[OGB_MAX_DEVICES] = {};
+    const dim3 block(256);
+    if (fp32) {
+      if (!set_max_dyn_smem(qkv_prep_mixed_kernel<float>, 200 * 1024, done32)) return -3;
+      return launch_pdl(qkv_prep_mixed_kernel<float>, dim3(T), block, smem, s, static_cast<const float*>(proj), static_cast<float*>(k_cache), static_cast<float*>(v_cache),
+                        p, talk, static_cast<float*>(mixed)) ? 0 : -4;
+    }
+    using B = __nv_bfloat16;
+    if (!set_max_dyn_smem(qkv_prep_mixed_kernel<B>, 200 * 1024, done16)) return -3;
+    return launch_pdl(qkv_prep_mixed_kernel<B>, dim3(T), block, smem, s, static_cast<const B*>(proj), static_cast<B*>(k_cache), static_cast<B*>(v_cache), p, talk,
+                      static_cast<B*>(mixed)) ? 0 : -4;
+  }
   if (!q_norm && !k_norm && dim == key_row && dim % 8 == 0 && rot % 16 == 0 && value_row % 8 == 0 && ldp % 8 == 0 &&
       ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(cos) |
         reinterpret_cast<uintptr_t>(sin)) & 15) == 0) {

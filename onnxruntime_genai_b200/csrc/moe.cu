@@ -69,6 +69,75 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T,
   }
 }
 
+// One warp per token: experts chosen by sigmoid(logit) + correction among the `keep` of `groups` groups of neighbours whose two largest choice
+// scores have the largest sums; weights: the chosen sigmoids divided by their sum (+ 1e-20), times scale.  Choice scores sit in shared memory.
+__global__ void moe_topk_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, const float* __restrict__ correction, int groups,
+                                        int keep, float scale, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
+  extern __shared__ float choice_all[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= T) return;
+  float* c = choice_all + size_t(warp) * (E + groups);
+  float* gs = c + E;                       // the groups' sums
+  const float* row = logits + size_t(t) * ld;
+  for (int e = lane; e < E; e += 32) c[e] = 1.f / (1.f + expf(-row[e])) + correction[e];
+  __syncwarp();
+  auto best_of = [&](const float* v, int n, int& arg) {
+    float best = -INFINITY;
+    arg = 0x7fffffff;
+    for (int e = lane; e < n; e += 32) if (v[e] > best) { best = v[e]; arg = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, arg, o);
+      if (ov > best || (ov == best && oe < arg)) { best = ov; arg = oe; }
+    }
+  };
+  if (groups > 1) {
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = c[e];
+        if (v > a) { b = a; a = v; } else if (v > b) b = v;
+      }
+      gs[g] = per > 1 ? a + b : a;
+    }
+    __syncwarp();
+    // the kept groups are marked by +inf, the others' experts leave the choice
+    for (int j = 0; j < keep; ++j) {
+      float best = -INFINITY;
+      int arg = 0x7fffffff;
+      for (int g = lane; g < groups; g += 32) if (gs[g] != INFINITY && gs[g] > best) { best = gs[g]; arg = g; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (ov > best || (ov == best && oe < arg)) { best = ov; arg = oe; }
+      }
+      if (lane == 0 && arg < groups) gs[arg] = INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32) if (gs[e / per] != INFINITY) c[e] = -INFINITY;
+    __syncwarp();
+  }
+  float s = 0.f;
+  int mine = 0;
+  for (int j = 0; j < k; ++j) {
+    int e;
+    best_of(c, E, e);
+    e = e < E ? e : 0;
+    if (lane == j) { mine = e; s = 1.f / (1.f + expf(-row[e])); }
+    __syncwarp();
+    if (lane == 0) c[e] = -INFINITY;
+    __syncwarp();
+  }
+  const float sum = warp_sum(s) + 1e-20f;
+  if (lane < k) {
+    topk_idx[size_t(t) * k + lane] = mine;
+    topk_w[size_t(t) * k + lane] = s / sum * scale;
+  }
+}
+
 // Single CTA: counting sort of the n = T*k assignments by expert (local experts [e_lo, e_hi) only).
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* __restrict__ topk_idx, int n, int k, int E, int e_lo, int e_hi, int bt, int* __restrict__ expert_offsets,
@@ -161,6 +230,16 @@ OGB_API int ogb_moe_topk(const float* logits, int ld, int T, int E, int k, int m
   const int threads = 128, warps_per_block = threads / 32;
   moe_topk_kernel<<<(T + warps_per_block - 1) / warps_per_block, threads, 0, static_cast<cudaStream_t>(stream)>>>(
       logits, ld, T, E, k, mode, shared, topk_idx, topk_w);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+OGB_API int ogb_moe_topk_grouped(const float* logits, int ld, int T, int E, int k, const float* correction, int groups, int keep, float scale,
+                                 int32_t* topk_idx, float* topk_w, void* stream) {
+  if (T <= 0) return 0;
+  if (E <= 0 || E > 1024 || k <= 0 || k > 32 || k > E || groups < 1 || E % groups || keep < 1 || keep > groups || k > E / groups * keep || !correction) return -1;
+  const int warps = 4;
+  moe_topk_grouped_kernel<<<(T + warps - 1) / warps, warps * 32, size_t(warps) * (E + groups) * sizeof(float), static_cast<cudaStream_t>(stream)>>>(
+      logits, ld, T, E, k, correction, groups, keep, scale, topk_idx, topk_w);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

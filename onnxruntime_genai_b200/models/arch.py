@@ -17,7 +17,7 @@ LLM_TYPES = [
     "chatglm", "decoder", "ernie4_5", "gemma", "gemma2", "gemma3_text", "gptoss", "gpt_oss", "granite", "hunyuan", "hunyuandensev1", "hunyuan_v1_dense",
     "internlm2", "llama", "mistral", "nemotron", "olmo", "olmo2", "exaone4", "phi", "phi3", "phimoe", "qwen2", "qwen3",
     "smollm3", "lfm2", "gpt2", "helium", "mixtral", "qwen2_moe", "qwen3_moe", "granitemoe", "olmoe", "qwen2_vl", "qwen2_5_vl", "qwen3_vl",
-    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar", "zevopel", "sugelix",      # hybrids of gated-delta-net (linear attention) and full-attention layers
+    "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "granitemoehybrid", "granitemoeshared", "luzatar", "zevopel", "sugelix", "tevilix",      # hybrids of gated-delta-net (linear attention) and full-attention layers
 ]
 
 
@@ -43,10 +43,12 @@ class RotarySpec:
 
 @dataclass
 class MoeSpec:
-    """Routed experts of a layer: `top` of `experts` feed-forwards run per token.  act: "silu" silu(gate) * up, or "clamped"
-    g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).  weights: softmax over the "selected" router
-    logits, over "all" of them, or over all and "renormed" over the selected; "sparse_mixer": PhiMoE's margin rule.  shared_ff > 0: one more
-    expert of that width (with its own limit) runs for every token and is added with weight 1."""
+    """Routed experts of a layer: `top` of `experts` feed-forwards run per token.  act: "silu" silu(gate) * up, "clamped"
+    g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit), or (experts without a gate matrix) "relu2"
+    max(up, 0)^2.  weights: softmax over the "selected" router logits, over "all" of them, or over all and "renormed" over the selected;
+    "sparse_mixer": PhiMoE's margin rule; "sigmoid": the selected experts' sigmoid scores divided by their sum, times `scale`, where the choice
+    goes by the scores plus a learned correction and (groups > 1) only among the `keep` groups of neighbours whose two best experts have the
+    largest sums.  shared_ff > 0: one more expert of that width (with its own limit) runs for every token and is added with weight 1."""
     experts: int
     top: int
     act: str = "silu"
@@ -56,6 +58,13 @@ class MoeSpec:
     jitter_eps: float = 0.01
     shared_ff: int = 0
     shared_limit: float = 0.0
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+
+    @property
+    def gated(self) -> bool:
+        return self.act != "relu2"
 
 
 @dataclass
@@ -72,7 +81,12 @@ class LayerSpec:
       "linear_attention"  gated delta rule: `kv_heads` query / key heads of `dim`, `heads` value heads of `vdim`, convolution of `conv` taps;
       "latent_attention"  `heads` heads of `dim` unrotated + `rot_dim` rotated query / key dimensions and `vdim` value dimensions over a
                           latent of `kv_rank` values per token; window 0: every earlier token is visible; q_rank > 0: the queries come
-                          out of an RMS-normed latent of their own; sinks as above.
+                          out of an RMS-normed latent of their own; sinks as above;
+      "mlstm"             matrix memories (xLSTM): per head a state [dim, vdim] with exponential input and sigmoid forget gates, both soft-capped
+                          at gate_cap, a normaliser [dim] and a running maximum;
+      "min_gru"           a gated average per column (minGRU): vdim columns whose gates read only the current token.
+    talk ("attention"): a head's scores are a learned mix of all heads' scores.  beside: a second mixer on the same input; the results, each times
+    its mix_scale, are added.  prefix: what follows "mix." in the names of the mixer's tensors.
     out_gate (the attending kinds): the concatenated heads are multiplied element by element with the sigmoid of a projection of the mixer's
     input.  A layer that runs several times is several entries: `weights_of` names the first run, every run has a cache of its own."""
     kind: str
@@ -95,6 +109,12 @@ class LayerSpec:
     maps: int = 1
     diff: float = 0.0
     q_rank: int = 0
+    talk: bool = False
+    o_bias: bool = False
+    gate_cap: float = 0.0
+    beside: Optional["LayerSpec"] = None
+    mix_scale: float = 1.0
+    prefix: str = ""
     rotary: Optional[RotarySpec] = None
     ff: int = 0                       # width of the gated feed-forward, of one expert where there are experts (0: the layer has none)
     moe: Optional[MoeSpec] = None
@@ -107,8 +127,21 @@ class LayerSpec:
         return 2 * self.kv_heads * self.dim + self.heads * self.vdim if self.kind == "linear_attention" else 0
 
     @property
+    def own_state(self) -> int:
+        """Floats of the mixer's recurrent state."""
+        if self.kind == "mlstm":          # memories, normalisers, maxima
+            return self.heads * (self.dim * self.vdim + self.dim + 1)
+        return {"linear_attention": self.heads * self.dim * self.vdim, "min_gru": self.vdim}.get(self.kind, 0)
+
+    @property
+    def beside_state(self) -> int:
+        """Where the state of the mixer beside this one starts in a request's slot."""
+        return (self.own_state + 3) // 4 * 4
+
+    @property
     def state_elems(self) -> int:
-        return self.heads * self.dim * self.vdim if self.kind == "linear_attention" else 0
+        """Floats of a request's slot: the state of the mixer, then of the one beside it."""
+        return self.beside_state + self.beside.own_state if self.beside else self.own_state
 
     @property
     def latent_row(self) -> int:
@@ -190,6 +223,8 @@ class ArchConfig:
     # residual_multiplier.
     layer_specs: Optional[List[LayerSpec]] = None
     layer_scale: bool = False
+    sublayer_norms: bool = False     # parallel blocks: each sub-layer reads a norm of its own of the same stream
+    norm_bias: bool = True           # layer norms of declared stacks have a bias
     tanh_norm: bool = False          # norms are tanh(alpha * x) * w + b (Dynamic Tanh: no statistics), alpha a learned scalar per norm
     bigram: Optional[Dict[str, int]] = None   # {buckets, mul_prev, mul_cur}: rows hashed from (previous token, token) join the embedding
     passes: int = 0                  # > 0: a group of layers runs that many times (entries of layer_specs with `opens_pass`); before each pass
@@ -275,11 +310,15 @@ class ArchConfig:
         return self.layer_types is not None and self.layer_types[layer] == "mamba"
 
     def is_recurrent_layer(self, layer: int) -> bool:
+        if self.layer_specs is not None:
+            return self.layer_specs[layer].state_elems > 0
         return self.is_linear_layer(layer) or self.is_mamba_layer(layer)
 
     @property
     def has_linear_layers(self) -> bool:
-        """True for models with layers that carry a recurrent state per request (gated-delta-net or Mamba-2 layers)."""
+        """True for models with layers that carry a recurrent state per request (gated-delta-net, Mamba-2 and other recurrent layers)."""
+        if self.layer_specs is not None:
+            return any(sp.state_elems > 0 for sp in self.layer_specs)
         return self.layer_types is not None and ("linear_attention" in self.layer_types or "mamba" in self.layer_types)
 
     @property
@@ -397,6 +436,14 @@ STACK_DESIGNS: Dict[str, Dict[str, Any]] = {
                             "attention_2": dict(kind="attention", qkv_bias=True, out_gate=True, maps=2),
                             "latent_attention": dict(kind="latent_attention", sinks=True, out_gate=True)},
                     feed_forwards=("moe",), moe=dict(act="clamped", alpha=1.702, weights="selected")),
+    # parallel blocks with a layer norm (no bias) per sub-layer, a group of layers that runs several times; windowed attention with normed and
+    # mixed heads beside a gated average, matrix memories; plain GELU feed-forward or squared-ReLU experts chosen in groups by corrected scores
+    "Tevilix": dict(arch=dict(model_type="tevilix", layernorm=True, norm_bias=False, parallel_block=True, sublayer_norms=True, mlp_gated=False,
+                              activation="gelu_erf"),
+                    mixers={"parallel": dict(left=dict(kind="attention", qkv_bias=True, o_bias=True, qk_norm=True, talk=True, out_gate=True),
+                                             right=dict(kind="min_gru")),
+                            "mlstm": dict(kind="mlstm")},
+                    feed_forwards=("dense", "moe"), moe=dict(act="relu2", weights="sigmoid")),
 }
 
 
@@ -414,26 +461,13 @@ def _rotary_spec(i: int, rot: Optional[Dict[str, Any]], width: int, neighbours: 
     return spec
 
 
-def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec:
-    if e.get("type") not in design["mixers"]:
-        raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
-    fixed = dict(design["mixers"][e["type"]])          # what the design fixes about this mixer
+def _mixer_spec(i: int, m: Dict[str, Any], fixed: Dict[str, Any]) -> LayerSpec:
+    """One mixer of layer i: m, its sizes in config.json; fixed, what the design says about it."""
+    fixed = dict(fixed)
     kind, mask_kind, neighbours = fixed.pop("kind"), fixed.pop("mask", "window"), fixed.pop("neighbours", False)
-    m, mlp = e["mixer"], e.get("mlp")
-    ff_kind = mlp.get("kind", "dense") if mlp else None
-    if mlp and ff_kind not in design["feed_forwards"]:
-        raise ValueError(f"layer {i}: unknown feed-forward kind {ff_kind!r}")
-    sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                   weights_of=None if e.get("weights_of") is None else int(e["weights_of"]), **fixed)
-    if ff_kind == "dense":
-        sp.ff = int(mlp["ff"])
-    elif ff_kind == "moe":
-        sp.ff = int(mlp["expert"]["ff"])
-        sp.moe = MoeSpec(int(mlp["router"]["experts"]), int(mlp["router"]["top"]), limit=float(mlp["expert"].get("limit") or 0.0), **design["moe"])
-        if not 0 < sp.moe.top <= sp.moe.experts:
-            raise ValueError(f"layer {i}: {sp.moe.top} of {sp.moe.experts} experts cannot be chosen")
-        if mlp.get("shared"):
-            sp.moe.shared_ff, sp.moe.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"].get("limit") or 0.0)
+    if kind == "min_gru":
+        return LayerSpec(kind=kind, heads=1, dim=1, vdim=int(m["width"]), **fixed)
+    sp = LayerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), **fixed)
     if kind in ("linear_attention", "attention"):
         sp.kv_heads = int(m["kv_heads"])
         if sp.heads % sp.kv_heads:
@@ -441,6 +475,8 @@ def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec
     mask = int((m.get("mask") or {}).get("size") or 0)
     if kind == "linear_attention":
         sp.conv = int(m["conv"])
+    elif kind == "mlstm":
+        sp.gate_cap = float(m["gate_cap"])
     elif kind == "attention":
         sp.scale, sp.softcap, sp.diff = float(m["scale"]), float(m.get("softcap") or 0.0), float(m.get("diff") or 0.0)
         setattr(sp, mask_kind, mask)
@@ -449,6 +485,37 @@ def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec
         sp.kv_rank, sp.rot_dim, sp.scale, sp.window = int(m["kv_rank"]), int(m["rot_dim"]), float(m["scale"]), mask
         sp.q_rank = int(m.get("q_rank") or 0)
         sp.rotary = _rotary_spec(i, m.get("rot"), sp.rot_dim, neighbours)
+    return sp
+
+
+def _stack_layer(i: int, e: Dict[str, Any], design: Dict[str, Any]) -> LayerSpec:
+    if e.get("type") not in design["mixers"]:
+        raise ValueError(f"layer {i}: unknown mixer type {e.get('type')!r}")
+    fixed, m, mlp = design["mixers"][e["type"]], e["mixer"], e.get("mlp")
+    ff_kind = mlp.get("kind", "dense") if mlp else None
+    if mlp and ff_kind not in design["feed_forwards"]:
+        raise ValueError(f"layer {i}: unknown feed-forward kind {ff_kind!r}")
+    if "left" in fixed:               # two mixers side by side
+        sp, sp2 = (_mixer_spec(i, m[side], dict(fixed[side], prefix=side + ".")) for side in ("left", "right"))
+        sp.mix_scale, sp2.mix_scale = float(m["left_scale"]), float(m["right_scale"])
+        sp.beside = sp2
+    else:
+        sp = _mixer_spec(i, m, fixed)
+    sp.weights_of = None if e.get("weights_of") is None else int(e["weights_of"])
+    if ff_kind == "dense":
+        sp.ff = int(mlp["ff"])
+    elif ff_kind == "moe":
+        r = mlp["router"]
+        groups = r.get("groups") or {}
+        sp.ff = int(mlp["expert"]["ff"])
+        sp.moe = MoeSpec(int(r["experts"]), int(r["top"]), limit=float(mlp["expert"].get("limit") or 0.0), groups=int(groups.get("count") or 1),
+                         keep=int(groups.get("keep") or 1), scale=float(r.get("scale", 1.0)), **design["moe"])
+        if sp.moe.experts % sp.moe.groups or not 0 < sp.moe.keep <= sp.moe.groups:
+            raise ValueError(f"layer {i}: {sp.moe.keep} of {sp.moe.groups} groups of {sp.moe.experts} experts cannot be kept")
+        if not 0 < sp.moe.top <= sp.moe.experts // sp.moe.groups * sp.moe.keep:
+            raise ValueError(f"layer {i}: {sp.moe.top} of {sp.moe.experts} experts cannot be chosen")
+        if mlp.get("shared"):
+            sp.moe.shared_ff, sp.moe.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"].get("limit") or 0.0)
     return sp
 
 
@@ -479,7 +546,7 @@ def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
     loop = cfg.get("loop")
     specs = _run_order(specs, loop)
     emb = cfg.get("embedding") or {}
-    att = [sp for sp in specs if sp.kind != "linear_attention"]
+    att = [sp for sp in specs if sp.kind in ("attention", "latent_attention")]
     # longest sequence the rotary scaling was made for, and at least 32768 positions (recurrent and windowed layers have no limit)
     span = [int(sp.rotary.scaling["original"] * sp.rotary.scaling["factor"]) for sp in att
             if sp.rotary and sp.rotary.scaling and "original" in sp.rotary.scaling]
@@ -495,73 +562,98 @@ def from_stack_config(cfg: Dict[str, Any]) -> ArchConfig:
                       **design["arch"])
 
 
+def _mixer_weight_shapes(sp: LayerSpec, W: int, m: str) -> Dict[str, tuple]:
+    """Names (m: their prefix) and shapes of a mixer's tensors, W the model's width."""
+    out: Dict[str, tuple] = {}
+    if sp.kind == "linear_attention":
+        kd, vd = sp.kv_heads * sp.dim, sp.heads * sp.vdim
+        for n, c in (("q", kd), ("k", kd), ("v", vd)):
+            out[m + n], out[m + n + ".conv"] = (c, W), (c, sp.conv)
+        out.update({m + "b": (sp.heads, W), m + "a": (sp.heads, W), m + "A_log": (sp.heads,), m + "dt_bias": (sp.heads,), m + "norm": (sp.vdim,),
+                    m + "g": (vd, W), m + "o": (W, vd)})
+    elif sp.kind == "attention":
+        sizes = dict(q=sp.heads * sp.maps * sp.dim, k=sp.kv_heads * sp.maps * sp.dim, v=sp.kv_heads * sp.vdim)
+        for n, c in sizes.items():
+            out[m + n] = (c, W)
+            if sp.qkv_bias:
+                out[f"{m}{n}.b"] = (c,)
+        out[m + "o"] = (W, sp.heads * sp.vdim)
+        if sp.o_bias:
+            out[m + "o.b"] = (W,)
+        if sp.talk:
+            out[m + "talk"] = (sp.heads, sp.heads)
+        if sp.maps == 2:
+            out.update({m + n: (sp.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        if sp.qk_norm:
+            out.update({m + "q.norm": (sp.dim,), m + "k.norm": (sp.dim,)})
+        if sp.sinks:
+            out[m + "sink"] = (sp.heads,)
+        if sp.head_gate:
+            out[m + "g"] = (sp.heads, W)
+    elif sp.kind == "mlstm":
+        for n, c in (("q", sp.heads * sp.dim), ("k", sp.heads * sp.dim), ("v", sp.heads * sp.vdim), ("g", sp.heads * sp.vdim)):
+            out[m + n] = (c, W)
+        out.update({m + "i": (sp.heads, W), m + "i.b": (sp.heads,), m + "f": (sp.heads, W), m + "f.b": (sp.heads,), m + "norm": (sp.heads * sp.vdim,),
+                    m + "o": (W, sp.heads * sp.vdim)})
+    elif sp.kind == "min_gru":
+        out.update({m + "z": (sp.vdim, W), m + "z.b": (sp.vdim,), m + "x": (sp.vdim, W), m + "x.b": (sp.vdim,), m + "g": (sp.vdim, W), m + "o": (W, sp.vdim)})
+    else:
+        rows = sp.heads * (sp.dim + sp.rot_dim)
+        if sp.q_rank:
+            out.update({m + "dq": (sp.q_rank, W), m + "dq.norm": (sp.q_rank,), m + "uq": (rows, sp.q_rank)})
+        else:
+            out[m + "q"] = (rows, W)
+        out.update({m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
+                    m + "uk": (sp.heads * sp.dim, sp.kv_rank), m + "uv": (sp.heads * sp.vdim, sp.kv_rank), m + "o": (W, sp.heads * sp.vdim)})
+        if sp.sinks:
+            out[m + "sink"] = (sp.heads,)
+    if sp.out_gate:
+        out[m + "g"] = (sp.heads * sp.vdim, W)
+    return out
+
+
 def stack_weight_shapes(arch: ArchConfig) -> Dict[str, tuple]:
     """Names and shapes of a declared stack's checkpoint tensors."""
     W = arch.hidden_size
     out: Dict[str, tuple] = {"embed": (arch.vocab_size, W), "final.norm": (W,), "head": (arch.vocab_size, W)}
-    if arch.layernorm or arch.tanh_norm:
+    norm_bias = arch.layernorm and arch.norm_bias or arch.tanh_norm
+    if norm_bias:
         out["final.norm.b"] = (W,)
     if arch.tanh_norm:
         out["final.norm.alpha"] = ()
     if arch.bigram:
         out["bigram"] = (arch.bigram["buckets"] + 1, W)
-    if arch.passes:
+    if arch.passes and arch.tanh_norm:
         out["loop.step"] = (arch.passes, W)
     for i, sp in enumerate(arch.layer_specs):
         if sp.weights_of is not None:
             continue
         p = f"l{i if sp.source is None else sp.source}."
         m = p + "mix."
-        # one norm for both sub-layers of a parallel block, else one for each
-        for n in range(1, 2 if arch.parallel_block or not sp.ff else 3):
+        # one norm for both sub-layers of a parallel block (where they have none of their own), else one for each
+        for n in range(1, 2 if arch.parallel_block and not arch.sublayer_norms or not sp.ff else 3):
             out[f"{p}norm{n}"] = (W,)
-            if arch.layernorm or arch.tanh_norm:
+            if norm_bias:
                 out[f"{p}norm{n}.b"] = (W,)
             if arch.tanh_norm:
                 out[f"{p}norm{n}.alpha"] = ()
             if arch.layer_scale:
                 out[f"{p}ls{n}"] = (W,)
-        if sp.kind == "linear_attention":
-            kd, vd = sp.kv_heads * sp.dim, sp.heads * sp.vdim
-            for n, c in (("q", kd), ("k", kd), ("v", vd)):
-                out[m + n], out[m + n + ".conv"] = (c, W), (c, sp.conv)
-            out.update({m + "b": (sp.heads, W), m + "a": (sp.heads, W), m + "A_log": (sp.heads,), m + "dt_bias": (sp.heads,), m + "norm": (sp.vdim,),
-                        m + "g": (vd, W), m + "o": (W, vd)})
-        elif sp.kind == "attention":
-            sizes = dict(q=sp.heads * sp.maps * sp.dim, k=sp.kv_heads * sp.maps * sp.dim, v=sp.kv_heads * sp.vdim)
-            for n, c in sizes.items():
-                out[m + n] = (c, W)
-                if sp.qkv_bias:
-                    out[f"{m}{n}.b"] = (c,)
-            out[m + "o"] = (W, sp.heads * sp.vdim)
-            if sp.maps == 2:
-                out.update({m + n: (sp.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
-            if sp.qk_norm:
-                out.update({m + "q.norm": (sp.dim,), m + "k.norm": (sp.dim,)})
-            if sp.sinks:
-                out[m + "sink"] = (sp.heads,)
-            if sp.head_gate:
-                out[m + "g"] = (sp.heads, W)
-        else:
-            rows = sp.heads * (sp.dim + sp.rot_dim)
-            if sp.q_rank:
-                out.update({m + "dq": (sp.q_rank, W), m + "dq.norm": (sp.q_rank,), m + "uq": (rows, sp.q_rank)})
-            else:
-                out[m + "q"] = (rows, W)
-            out.update({m + "dkv": (sp.kv_rank + sp.rot_dim, W), m + "dkv.norm": (sp.kv_rank,),
-                        m + "uk": (sp.heads * sp.dim, sp.kv_rank), m + "uv": (sp.heads * sp.vdim, sp.kv_rank), m + "o": (W, sp.heads * sp.vdim)})
-            if sp.sinks:
-                out[m + "sink"] = (sp.heads,)
-        if sp.out_gate:
-            out[m + "g"] = (sp.heads * sp.vdim, W)
+        for mx in (sp, sp.beside):
+            if mx is not None:
+                out.update(_mixer_weight_shapes(mx, W, m + mx.prefix))
         if sp.ff:
             if sp.moe is not None:
                 out[p + "mlp.router"] = (sp.moe.experts, W)
+                if sp.moe.weights == "sigmoid":
+                    out[p + "mlp.correction"] = (sp.moe.experts,)
                 if sp.moe.shared_ff:
                     f = sp.moe.shared_ff
                     out.update({p + "mlp.shared.gate": (f, W), p + "mlp.shared.up": (f, W), p + "mlp.shared.down": (W, f)})
+            gated = arch.mlp_gated if sp.moe is None else sp.moe.gated
             for e in [""] if sp.moe is None else [f"e{k}." for k in range(sp.moe.experts)]:
-                out.update({f"{p}mlp.{e}gate": (sp.ff, W), f"{p}mlp.{e}up": (sp.ff, W), f"{p}mlp.{e}down": (W, sp.ff)})
+                out.update({f"{p}mlp.{e}{n}": (sp.ff, W) for n in (("gate", "up") if gated else ("up",))})
+                out[f"{p}mlp.{e}down"] = (W, sp.ff)
     return out
 
 

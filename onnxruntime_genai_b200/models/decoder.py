@@ -92,7 +92,7 @@ class PagedKVCache:
         # Models whose embedding also reads the token before: the ids of the cached positions, in the same paged slots.
         self.tokens = torch.zeros(num_blocks * block_size, dtype=torch.int32, device=device) if arch.bigram else None
         # layers without rows in the pools below
-        conv = [c or i in self.latent_index or i in self.spec_kv for i, c in enumerate(conv)]
+        conv = [c or arch.layer_specs is not None for c in conv]
         self.windowed = [num_window_blocks > 0 and arch.layer_window(i) > 0 and not conv[i] for i in range(arch.num_layers)]
         n_full = sum(1 for w, c in zip(self.windowed, conv) if not w and not c)
         n_win = sum(1 for w in self.windowed if w)
@@ -163,17 +163,22 @@ class PagedKVCache:
 
     def state_layer(self, i: int) -> torch.Tensor:
         """[slots, heads, ...] state of one layer; slots may be further apart than a state is long (stacks whose layers differ)."""
-        st = self.state[self.lin_index[i]]
         if self.arch.layer_specs is None:
-            return st
+            return self.state[self.lin_index[i]]
         sp = self.arch.layer_specs[i]
-        return st[:, :sp.state_elems].view(st.shape[0], sp.heads, sp.dim, sp.vdim)
+        return self.state_rows(i).view(-1, sp.heads, sp.dim, sp.vdim)
+
+    def state_rows(self, i: int, beside: bool = False) -> torch.Tensor:
+        """[slots, floats] state of the mixer of a declared layer, or of the mixer beside it."""
+        sp, st = self.arch.layer_specs[i], self.state[self.lin_index[i]]
+        return st[:, sp.beside_state:sp.state_elems] if beside else st[:, :sp.own_state]
 
     @staticmethod
     def bytes_per_block(arch: ArchConfig, block_size: int, dtype, kv_heads: Optional[int] = None, conv_channels: Optional[int] = None,
                         kv_bits: int = 16) -> int:
         hk = kv_heads if kv_heads is not None else arch.num_kv_heads
         n_conv = sum(1 for i in range(arch.num_layers) if arch.conv_state_channels(i) > 0)
+        n_plain = 0 if arch.layer_specs is not None else arch.num_layers - n_conv
         cc = arch.recurrent_conv_dim if arch.has_linear_layers else (conv_channels if conv_channels is not None else arch.hidden_size)
         es = torch.empty((), dtype=dtype).element_size()
         kv_row = arch.head_dim + 16 if kv_bits == 8 else arch.head_dim * es
@@ -181,7 +186,7 @@ class PagedKVCache:
         own = [sp for i, sp in enumerate(arch.layer_specs or []) if arch.is_spec_attention(i)]
         own_row = sum(sp.kv_heads * (sp.key_row + sp.value_row) for sp in own)
         ids = 4 if arch.bigram else 0
-        return ((arch.num_layers - n_conv - n_lat - len(own)) * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row + own_row) * es + ids) * block_size
+        return max(1, (n_plain * 2 * hk * kv_row + (n_conv * cc + n_lat * arch.latent_row + own_row) * es + ids) * block_size)
 
 
 class CrossKVCache:
@@ -228,6 +233,7 @@ class LayerWeights:
     q_norm_w: Optional[torch.Tensor] = None
     k_norm_w: Optional[torch.Tensor] = None
     sinks: Optional[torch.Tensor] = None
+    talk: Optional[torch.Tensor] = None          # [heads, heads] fp32: every head's scores are a mix of all heads'
     post_attn_norm_w: Optional[torch.Tensor] = None
     post_ffn_norm_w: Optional[torch.Tensor] = None
     gate_up_w: Optional[torch.Tensor] = None
@@ -269,9 +275,17 @@ class LayerWeights:
     exp_shared: bool = False                   # the shared expert is the last of the stacked experts
     rope_cos: Optional[torch.Tensor] = None    # rotary tables of this layer
     rope_sin: Optional[torch.Tensor] = None
+    mem_in_w: Optional[torch.Tensor] = None    # matrix memories: stacked [queries | keys | values | output gate] projection,
+    mem_gate_w: Optional[torch.Tensor] = None  # that of the input and forget gates [2 heads, width], their biases (fp32),
+    mem_gate_b: Optional[torch.Tensor] = None
+    mem_norm_w: Optional[torch.Tensor] = None  # and the weight of the heads' norm (fp32)
     join_w: Optional[torch.Tensor] = None      # parallel blocks on an fp32 stream: [mixer output map | down] over [mixer output (padded) | feed-forward]
-    mix_cols: int = 0                          # columns of the mixer output in the joined input, and where the feed-forward starts
+    join_b: Optional[torch.Tensor] = None
+    mix_cols: int = 0                          # columns of the mixer output in the joined input, where that of the mixer beside it and the
+    beside_col: int = 0                        # feed-forward start, and columns in use
     mlp_col: int = 0
+    join_cols: int = 0
+    beside_in: int = 0                         # first column of the mixer beside this one in their joint projection
     cross_ln_w: Optional[torch.Tensor] = None  # encoder-decoder cross-attention (whisper)
     cross_ln_b: Optional[torch.Tensor] = None
     cross_q_w: Optional[torch.Tensor] = None
@@ -416,7 +430,10 @@ class DecoderModel:
             args, kw, cols = (block_size, self.heads_local, self.kv_heads_local, a.head_dim, a.scale, lw.window, lw.sinks, a.softcap), {}, a.head_dim
         else:
             args, cols = (block_size, sp.heads * sp.maps, sp.kv_heads, sp.key_row, sp.scale, sp.window, lw.sinks, sp.softcap), sp.value_row
-            kw = dict(vdim=sp.value_row, chunk=sp.chunk, gate=gate, maps=sp.maps,
+            if sp.talk:
+                cols_k = sp.kv_heads * sp.key_row
+                args = args[:3] + (cols_k,) + args[4:]
+            kw = dict(vdim=sp.value_row, chunk=sp.chunk, gate=gate, maps=sp.maps, joint=sp.talk, out_scale=sp.mix_scale,
                       diff=(lw.diff_lambda, 1.0 - sp.diff, a.norm_eps, sp.vdim) if sp.maps == 2 else None)
         nd, B = s.num_decode, s.past_lens.shape[0]
         if not (qkv.is_cuda and 0 < nd < B and s.max_q_len > 1):
@@ -523,21 +540,47 @@ class DecoderModel:
                                       sp.window, out, lw.sinks, gate)
         return out
 
-    def _spec_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    def _spec_attention(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor,
+                        beside: Optional[torch.Tensor] = None) -> torch.Tensor:
         """An attention layer of a declared stack: one projection [queries | keys | values | gate logits], norms, rotation and cache append
         in one pass, attention over the paged cache whose epilogue gates the heads (or their columns); writes them to `out`
-        [T, heads * value_row]."""
+        [T, heads * value_row].  Heads whose scores are mixed: the mix is a mix of the queries, one part per key head, so that a query meets the
+        keys of all key heads as one vector.  A mixer beside the attention has its columns in the same projection and writes `beside`."""
         sp = self.arch.layer_specs[li]
         kc, vc, _ = kv.layer(li)
         proj = self._wide_linear(x, lw.qkv_w, lw.qkv_b)
+        q = proj if lw.talk is None else torch.empty(x.shape[0], sp.heads * sp.kv_heads * sp.key_row, dtype=x.dtype, device=x.device)
         ops.qkv_prep(proj, sp.heads * sp.maps, sp.kv_heads * sp.maps, sp.dim, sp.map_row, sp.value_row, lw.q_norm_w, lw.k_norm_w, self.arch.norm_eps,
-                     s.positions, lw.rope_cos, lw.rope_sin, s.slot_mapping, kc, vc, Hv=sp.kv_heads)
+                     s.positions, lw.rope_cos, lw.rope_sin, s.slot_mapping, kc, vc, Hv=sp.kv_heads, talk=lw.talk, mixed=q if lw.talk is not None else None)
+        if beside is not None:
+            self._min_gru(s, kv, li, sp.beside, proj[:, lw.beside_in:], beside)
         g0 = (sp.heads + sp.kv_heads) * sp.key_row + sp.kv_heads * sp.value_row
         cols = sp.heads * sp.value_row if sp.out_gate else (sp.heads if sp.head_gate else 0)
-        return self._attention(s, proj, kc, vc, s.block_table, kv.block_size, lw, sp, proj[:, g0:g0 + cols] if cols else None, out)
+        return self._attention(s, q, kc, vc, s.block_table, kv.block_size, lw, sp, proj[:, g0:g0 + cols] if cols else None, out)
+
+    def _need_slots(self, s: StepInputs) -> None:
+        if s.state_slots is None:
+            raise RuntimeError("this model has recurrent layers: the caller must provide StepInputs.state_slots")
+
+    def _min_gru(self, s: StepInputs, kv: PagedKVCache, li: int, sp, proj: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """Gated average beside another mixer: proj [T, (update gate | candidate | output gate) of up8(vdim) columns each]."""
+        self._need_slots(s)
+        W, row = sp.vdim, (sp.vdim + 7) // 8 * 8
+        return ops.min_gru(proj[:, :W], proj[:, row:row + W], proj[:, 2 * row:2 * row + W], kv.state_rows(li, beside=True), s.state_slots, s.cu_seqlens,
+                           s.past_lens, out, sp.mix_scale, s.max_q_len)
+
+    def _mlstm(self, s: StepInputs, kv: PagedKVCache, li: int, lw: LayerWeights, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """Matrix memories: writes the normed and gated heads to `out` [T, heads * vdim].  The gates' logits stay in fp32."""
+        self._need_slots(s)
+        sp = self.arch.layer_specs[li]
+        proj = self._wide_linear(x, lw.mem_in_w)
+        gates = ops.linear(x, lw.mem_gate_w, out_fp32=True)
+        return ops.mlstm(proj, gates, lw.mem_gate_b, sp.heads, sp.dim, sp.vdim, sp.gate_cap, lw.mem_norm_w, self.arch.norm_eps, kv.state_rows(li), s.state_slots,
+                         s.cu_seqlens, s.past_lens, out, s.max_q_len)
 
     def _stack_mixer(self, lw: LayerWeights, sp):
-        return {"linear_attention": self._linear_attention, "latent_attention": self._latent_attention, "attention": self._spec_attention}[sp.kind]
+        return {"linear_attention": self._linear_attention, "latent_attention": self._latent_attention, "attention": self._spec_attention,
+                "mlstm": self._mlstm}[sp.kind]
 
     def _forward_stream(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
         """Declared stacks: an fp32 residual stream between the embedding and the final norm (of the rows whose logits are wanted)."""
@@ -549,31 +592,41 @@ class DecoderModel:
         if a.tanh_norm:
             self.last_hidden = x = self._tanh_normed_blocks(s, kv)
             return ops.linear(x, self.lm_head_w, out_fp32=True)
+        pending = None
         if a.parallel_block:
-            h = self._parallel_blocks(s, kv)
+            h, pending = self._parallel_blocks(s, kv)
         else:
             h = self._output_normed_blocks(s, kv)
-        x = ops.norm_stream(h, self.final_norm_w, a.norm_eps, self.final_norm_b, a.layernorm, self.dtype, rows=s.logits_rows)
+        x = ops.norm_stream(h, self.final_norm_w, a.norm_eps, self.final_norm_b, a.layernorm, self.dtype, rows=s.logits_rows, add=pending)
         self.last_hidden = x
         return ops.linear(x, self.lm_head_w, out_fp32=True)
 
-    def _parallel_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
-        """Parallel blocks: per layer one norm, the mixer and the gated feed-forward side by side into the column ranges of one matrix,
-        and one output projection of both whose epilogue adds to the stream in fp32."""
+    def _parallel_blocks(self, s: StepInputs, kv: PagedKVCache):
+        """Parallel blocks: per layer one norm (or one per sub-layer, by one kernel), the mixer (or two) and the dense feed-forward side by side into
+        the column ranges of one matrix, and one output projection of all whose epilogue adds to the stream in fp32.  Routed experts read the
+        stream's norm too; the weighted sum of their rows joins the stream in the kernel of the next norm.  Returns the stream and what still
+        has to be added to it."""
+        from .moe import moe_forward
         a = self.arch
         h = s.inputs_embeds.float().clone() if s.inputs_embeds is not None else ops.embedding_stream(s.input_ids, self.embed, a.embed_scale)
-        T = h.shape[0]
+        T, pending = h.shape[0], None
         for li, lw in enumerate(self.layers):
-            x = ops.norm_stream(h, lw.ln1_w, a.norm_eps, lw.ln1_b, a.layernorm, self.dtype)
+            sp = a.layer_specs[li]
+            x = x2 = ops.norm_stream(h, lw.ln1_w, a.norm_eps, lw.ln1_b, a.layernorm, self.dtype, add=pending, weight2=lw.ln2_w)
+            if lw.ln2_w is not None:
+                x, x2 = x
             K = lw.join_w.shape[1]
-            used = (lw.mlp_col == lw.mix_cols or lw.gate_up_w is None) and K == lw.mix_cols + (a.layer_specs[li].ff)
-            y = (torch.empty if used else torch.zeros)(T, K, dtype=self.dtype, device=h.device)      # padding columns meet zero weights: finite
-            self._stack_mixer(lw, a.layer_specs[li])(s, kv, li, lw, x, out=y[:, :lw.mix_cols])
+            y = (torch.empty if lw.join_cols == K else torch.zeros)(T, K, dtype=self.dtype, device=h.device)      # padding columns meet zero weights: finite
+            beside = dict(beside=y[:, lw.beside_col:lw.beside_col + sp.beside.vdim]) if sp.beside else {}
+            self._stack_mixer(lw, sp)(s, kv, li, lw, x, out=y[:, :lw.mix_cols], **beside)
+            ff = y[:, lw.mlp_col:lw.mlp_col + sp.ff]
             if lw.gate_up_w is not None:
-                ops.gate_up_act(x, lw.gate_up_w, None, a.activation, out=y[:, lw.mlp_col:lw.mlp_col + a.layer_specs[li].ff],
-                                interleaved=lw.gate_up_interleaved)
-            h = ops.linear(y, lw.join_w, residual=h, out=h, out_fp32=True)
-        return h
+                ops.gate_up_act(x2, lw.gate_up_w, None, a.activation, out=ff, interleaved=lw.gate_up_interleaved)
+            elif lw.fc1_w is not None:
+                ops.linear_act(x2, lw.fc1_w, a.activation, out=ff)
+            pending = moe_forward(self, lw, x2, defer=True) if sp.moe is not None else None
+            h = ops.linear(y, lw.join_w, lw.join_b, residual=h, out=h, out_fp32=True)
+        return h, pending
 
     def _output_normed_blocks(self, s: StepInputs, kv: PagedKVCache) -> torch.Tensor:
         """Blocks whose sub-layers read the stream itself (x, its copy in the compute type): each sub-layer's result is normed, scaled

@@ -3,7 +3,7 @@ Two styles: gpt-oss (biases, softmax over the selected logits, clamped SwiGLU(al
 PhiMoE, GraniteMoE: no biases, silu(gate) * up, softmax over all experts with or without renormalisation).  Declared stacks describe
 the experts of each layer by themselves (`LayerWeights.moe`, an arch.MoeSpec), with any mix of these rules, and may have a shared expert:
 of the same width and limit it is one more expert of the grouped products that every token is routed to with weight 1, else it runs
-beside them and the add + norm that follows folds it.
+beside them and the add + norm that follows folds it.  Experts without a gate matrix keep their up matrix in `exp_gate_up_w`.
 
 Semantics follow the MoE / QMoE contrib op the reference's builder emits
 (src/python/py/models/builders/base.py:4176-4408, builders/gptoss.py:653-847): `k` experts per token,
@@ -54,6 +54,8 @@ def route(model, lw, x):
     """Routing weights and expert ids [T, k].  Softmax over the selected logits equals softmax over all experts renormalised
     over the selected; the standard style without renormalisation keeps the probabilities of the full softmax."""
     sp = spec_of(model, lw)
+    if sp.weights == "sigmoid":
+        return corrected_choice(ops.linear(x, lw.router_w, out_fp32=True), lw.router_b, sp)
     logits = ops.linear(x, lw.router_w, lw.router_b).float()
     if sp.weights == "sparse_mixer":
         return sparse_mixer(logits, sp.jitter_eps)
@@ -61,6 +63,20 @@ def route(model, lw, x):
     if sp.weights == "all":
         return torch.softmax(logits, dim=-1).gather(-1, top_i), top_i
     return torch.softmax(top_v, dim=-1), top_i
+
+
+def corrected_choice(logits: torch.Tensor, correction: torch.Tensor, sp: MoeSpec):
+    """Sigmoid scores; the choice goes by score + correction, among the `keep` groups of neighbours with the largest sums of two."""
+    s = torch.sigmoid(logits.float())
+    c = s + correction
+    if sp.groups > 1:
+        g = c.view(c.shape[0], sp.groups, -1)
+        best = g.topk(min(2, g.shape[-1]), dim=-1).values.sum(-1).topk(sp.keep, dim=-1).indices
+        open_ = torch.zeros(g.shape[:2], dtype=torch.bool, device=c.device).scatter_(1, best, True)
+        c = g.masked_fill(~open_[:, :, None], float("-inf")).reshape(c.shape)
+    ids = torch.topk(c, sp.top, dim=-1).indices
+    w = s.gather(-1, ids)
+    return w / (w.sum(-1, keepdim=True) + 1e-20) * sp.scale, ids
 
 
 def sparse_mixer(logits: torch.Tensor, eps: float):
@@ -101,6 +117,8 @@ def expert_mlp(model, lw, e: int, xs: torch.Tensor) -> torch.Tensor:
     packed = isinstance(lw.exp_gate_up_w, ops.Fp4Experts)   # MXFP4 experts: expand this one expert
     w = lw.exp_gate_up_w.dequantize(e).to(xs) if packed else lw.exp_gate_up_w[e]
     b = lw.exp_gate_up_b[e] if lw.exp_gate_up_b is not None else None
+    if not sp.gated:
+        return ops.linear(ops.linear_act(xs, w, sp.act), lw.exp_down_w[e])
     if lw.exp_blocked:
         w, b = _unblock(w).contiguous(), _unblock(b).contiguous() if b is not None else None
     gu = ops.linear(xs, w, b)
@@ -143,6 +161,9 @@ def _forward_loop(model, lw, x):
 def _plan(model, lw, x, sp, token_tile=0):
     """Routing of the tokens, on the device."""
     lo, hi = lw.exp_lo, lw.exp_hi or sp.experts
+    if sp.weights == "sigmoid":
+        return ops.moe_route(ops.linear(x, lw.router_w, out_fp32=True), sp.top, 3, (lo, hi), token_tile, correction=lw.router_b, groups=sp.groups, keep=sp.keep,
+                             scale=sp.scale)
     logits = ops.linear(x, lw.router_w, lw.router_b, out_fp32=True)
     if lw.exp_shared:
         return ops.moe_route(logits, sp.top, _TOPK_MODES[sp.weights], None, token_tile, shared=True)
@@ -169,7 +190,9 @@ def _forward_device(model, lw, x, defer=False):
         y = ops.moe_gemm(h, lw.exp_down_w, plan, lw.exp_down_b)
         return ops.PendingCombine(y, plan) if defer else ops.moe_combine(y, plan)
     xs = ops.gather_rows(x, plan.sorted_token)
-    if sp.act == "silu":
+    if not sp.gated:
+        h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, None, act_kind=ops.MOE_ACTS[sp.act], pair=False)
+    elif sp.act == "silu":
         h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, None, act_kind=1)
     else:
         h = ops.moe_gemm(xs, lw.exp_gate_up_w, plan, lw.exp_gate_up_b, act_kind=2, alpha=sp.alpha, limit=sp.limit)

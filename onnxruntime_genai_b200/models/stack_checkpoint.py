@@ -84,7 +84,7 @@ def load_stack_decoder(model_dir: str, filename: str, context_length: int, devic
 def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], device, dtype) -> DecoderModel:
     """DecoderModel from a tensor source: input projections stacked per layer, the key map transposed per head, the output projections
     of both sub-layers of a parallel block joined side by side, the factors on a sub-layer's normed output multiplied into one vector,
-    experts stacked, heads and feed-forwards filled up with zeros where a kernel wants whole tiles, small vectors and recurrence constants
+    experts stacked, two mixers' input projections joined where they stand side by side, heads and feed-forwards filled up with zeros where a kernel wants whole tiles, small vectors and recurrence constants
     in fp32."""
     shapes = stack_weight_shapes(arch)
     model = DecoderModel(arch, device, dtype)
@@ -151,7 +151,22 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
             lw.diff_lambda = float(lam[0] - lam[1]) + sp.diff
         if sp.sinks:
             lw.sinks = vec(m + "sink")
+        if sp.talk:
+            lw.talk = vec(m + "talk")
         lw.rope_cos, lw.rope_sin = rotary(sp.rotary)
+
+    def add_beside(lw, sp, m):
+        """The projections [update gate | candidate | output gate] of a gated average, each filled up to whole 16-byte pieces, behind the projection of
+        the mixer it stands beside."""
+        W = lw.qkv_w.shape[1]
+        fill = (0, (-sp.vdim) % 8)
+        parts = [torch.nn.functional.pad(raw(m + n).to(dtype), (0, 0) + fill) for n in ("z", "x", "g")]
+        bias = [torch.nn.functional.pad(raw(m + n).to(dtype), fill) for n in ("z.b", "x.b")]
+        lw.beside_in = up8(lw.qkv_w.shape[0])
+        gap = lw.beside_in - lw.qkv_w.shape[0]
+        first = lw.qkv_b if lw.qkv_b is not None else lw.qkv_w.new_zeros(lw.qkv_w.shape[0])
+        lw.qkv_w = torch.cat([lw.qkv_w, lw.qkv_w.new_zeros(gap, W)] + parts, 0).contiguous()
+        lw.qkv_b = torch.cat([first, first.new_zeros(gap)] + bias + [torch.zeros_like(bias[0])]).contiguous()
 
     def output_map(name, sp):
         """The mixer's output map over its heads as they leave the mixer."""
@@ -180,7 +195,16 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         lw.moe, lw.router_w, lw.exp_hi = sp.moe, mat(p + "router"), E
         lw.exp_blocked = tiled and W % 8 == 0
         F = (sp.ff + 63) // 64 * 64 if lw.exp_blocked else sp.ff      # (an expert's zero gates give zero, whatever its ups are)
+        if sp.moe.weights == "sigmoid":
+            lw.router_b = vec(p + "correction")
         names = [f"{p}e{e}." for e in range(E)]
+        if not sp.moe.gated:
+            F = up8(sp.ff) if lw.exp_blocked else sp.ff
+            lw.exp_gate_up_w = torch.zeros(E, F, W, dtype=dtype, device=device)
+            lw.exp_down_w = torch.zeros(E, W, F, dtype=dtype, device=device)
+            for e, n in enumerate(names):
+                lw.exp_gate_up_w[e, :sp.ff], lw.exp_down_w[e, :, :sp.ff] = raw(n + "up").to(dtype), raw(n + "down").to(dtype)
+            return
         # a shared expert of the same width and limit is one more expert that every token takes
         ff2 = sp.moe.shared_ff
         lw.exp_shared = ff2 == sp.ff and sp.moe.shared_limit == sp.moe.limit and E < 1024 and sp.moe.top < 32
@@ -236,7 +260,12 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
             lw.lin_neg_exp_a = -torch.exp(vec(m + "A_log"))
             lw.lin_dt_bias, lw.lin_norm_w = vec(m + "dt_bias"), vec(m + "norm")
         elif sp.kind == "attention":
-            attention_weights(lw, sp, m)
+            attention_weights(lw, sp, m + sp.prefix)
+            if sp.beside:
+                add_beside(lw, sp.beside, m + sp.beside.prefix)
+        elif sp.kind == "mlstm":
+            lw.mem_in_w, lw.mem_gate_w = mat(m + "q", m + "k", m + "v", m + "g"), mat(m + "i", m + "f")
+            lw.mem_gate_b, lw.mem_norm_w = torch.cat([vec(m + "i.b"), vec(m + "f.b")]), vec(m + "norm")
         else:
             latent_input(lw, sp, m)
             if sp.sinks:
@@ -258,11 +287,25 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
                 (feed_forward if sp.moe is None else expert_weights)(lw, sp, p + "mlp.")
                 lw.post_ffn_norm_w = output_factor(p, 2)
             return lw
-        lw.ln1_w, lw.ln1_b = vec(p + "norm1"), vec(p + "norm1.b") if arch.layernorm else None
-        lw.mlp_col = up8(lw.mix_cols)
-        lw.join_w = torch.zeros(arch.hidden_size, lw.mlp_col + up8(sp.ff), dtype=dtype, device=device)
-        lw.join_w[:, :lw.mix_cols] = output_map(m + "o", sp)
-        if sp.ff:
+        lw.ln1_w, lw.ln1_b = vec(p + "norm1"), vec(p + "norm1.b") if arch.layernorm and arch.norm_bias else None
+        if sp.ff and arch.sublayer_norms:
+            lw.ln2_w = vec(p + "norm2")
+        ff, side = sp.ff if sp.moe is None else 0, sp.beside.vdim if sp.beside else 0
+        lw.beside_col = up8(lw.mix_cols)
+        lw.mlp_col = lw.beside_col + up8(side)
+        lw.join_cols = lw.mix_cols + side + ff
+        lw.join_w = torch.zeros(arch.hidden_size, lw.mlp_col + up8(ff), dtype=dtype, device=device)
+        lw.join_w[:, :lw.mix_cols] = output_map(m + sp.prefix + "o", sp)
+        if side:
+            lw.join_w[:, lw.beside_col:lw.beside_col + side] = raw(m + sp.beside.prefix + "o").to(dtype)
+        if sp.o_bias:
+            lw.join_b = (vec(m + sp.prefix + "o.b") * sp.mix_scale).to(dtype)
+        if sp.moe is not None:
+            expert_weights(lw, sp, p + "mlp.")
+        elif sp.ff and not arch.mlp_gated:
+            lw.fc1_w = mat(p + "mlp.up")
+            lw.join_w[:, lw.mlp_col:lw.mlp_col + sp.ff] = raw(p + "mlp.down").to(dtype)
+        elif sp.ff:
             lw.join_w[:, lw.mlp_col:lw.mlp_col + sp.ff] = raw(p + "mlp.down").to(dtype)
             lw.gate_up_w = mat(p + "mlp.gate", p + "mlp.up")
             if tiled and sp.ff % 64 == 0:
@@ -275,10 +318,10 @@ def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], de
         model.final_norm = tanh_norm("final.norm")
     else:
         model.final_norm_w = vec("final.norm") + arch.norm_offset
-        model.final_norm_b = vec("final.norm.b") if arch.layernorm else None
+        model.final_norm_b = vec("final.norm.b") if arch.layernorm and arch.norm_bias else None
     if arch.bigram:
         model.bigram = mat("bigram")
-    if arch.passes:
+    if arch.passes and arch.tanh_norm:
         model.loop_step = vec("loop.step")
     own = {i: layer(i) for i, sp in enumerate(arch.layer_specs) if sp.weights_of is None}
     model.layers = [own[i if sp.weights_of is None else sp.weights_of] for i, sp in enumerate(arch.layer_specs)]

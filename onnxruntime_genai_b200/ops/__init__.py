@@ -217,20 +217,33 @@ def add_tanh_norm(h, y, norm: TanhNorm, dtype=torch.bfloat16, first=None, step=N
     return x
 
 
-def norm_stream(x, weight, eps, bias=None, layernorm=False, dtype=torch.bfloat16, rows=None):
+def norm_stream(x, weight, eps, bias=None, layernorm=False, dtype=torch.bfloat16, rows=None, add=None, weight2=None):
     """Norm of the rows of an fp32 residual stream [T, H] (of the rows listed in `rows`, int32, when given) as `dtype`; weight and bias
-    are fp32."""
+    are fp32.  add: rows [T, H] in `dtype`, or a mixture-of-experts output whose combine step is pending, that join the stream first (in place,
+    where all its rows are normed).  weight2: returns the pair (norm with weight and bias, norm with weight2)."""
     if rows is not None:
         _check_index("norm_stream", "rows", rows, x.shape[0])
     if not x.is_cuda:
+        if add is not None:
+            x = x.add_(add.float()) if rows is None else x + add.float()
         h = x if rows is None else x[rows.long()]
-        return ref.norm(h.float(), weight, eps, None, bias, layernorm)[0].to(dtype)
-    assert x.dtype == torch.float32 and x.is_contiguous() and weight.dtype == torch.float32 and (bias is None or bias.dtype == torch.float32)
+        one = lambda w, b: ref.norm(h.float(), w, eps, None, b, layernorm)[0].to(dtype)
+        return one(weight, bias) if weight2 is None else (one(weight, bias), one(weight2, None))
+    import ctypes
+    plan = None
+    if isinstance(add, PendingCombine):
+        assert add.shared is None
+        add, plan = add.y, add.plan
+    assert x.dtype == torch.float32 and x.is_contiguous() and all(t is None or t.dtype == torch.float32 for t in (weight, bias, weight2))
     n, H = (x.shape[0] if rows is None else rows.numel()), x.shape[1]
+    assert add is None or (add.dtype == dtype and add.stride(1) == 1 and add.shape[1] == H) and (plan is None or plan.T == x.shape[0])
     out = torch.empty(n, H, dtype=dtype, device=x.device)
-    _lib.check(_lib.lib().ogb_norm_stream(_ptr(x), _ptr(rows), _ptr(weight), _ptr(bias), _ptr(out), int(dtype == torch.float32), n, H, float(eps),
-                                         int(layernorm), _stream()), "norm_stream")
-    return out
+    out2 = torch.empty_like(out) if weight2 is not None else None
+    p = _lib.NormStream(x=_ptr(x), rows=_ptr(rows), w=_ptr(weight), b=_ptr(bias), w2=_ptr(weight2), out=_ptr(out), out2=_ptr(out2), y=_ptr(add),
+                        inv_pos=_ptr(plan.inv_pos) if plan else None, topk_w=_ptr(plan.topk_w) if plan else None, ldy=add.stride(0) if add is not None else 0,
+                        k=plan.k if plan else 0, n_rows=n, H=H, layernorm=int(layernorm), fp32=int(dtype == torch.float32), eps=float(eps))
+    _lib.check(_lib.lib().ogb_norm_stream(ctypes.byref(p), _stream()), "norm_stream")
+    return out if out2 is None else (out, out2)
 
 
 # ------------------------------------------------------------------------------------------ norm
@@ -329,13 +342,13 @@ def _tma_ok(x, w) -> bool:
     return x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and (x.data_ptr() | w.data_ptr()) % 16 == 0
 
 
-def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None, bias=None):
+def _gemm_simt(x, w, out, residual=None, batch=1, a_cols=0, c_cols=0, K=None, bias=None, act=0):
     """The fp32 / unaligned form of a product (csrc/gemm_simt.cu)."""
     assert bias is None or bias.dtype == x.dtype
     assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and out.dtype in (torch.float32, torch.bfloat16)
     _lib.check(_lib.lib().ogb_gemm_simt(_ptr(x), x.stride(0), int(a_cols), _ptr(w), w.stride(0), _ptr(out), out.stride(0), int(c_cols), x.shape[0],
                                        w.shape[0] // batch, K or x.shape[1], int(batch), _ptr(residual), residual.stride(0) if residual is not None else 0,
-                                       _ptr(bias), int(x.dtype == torch.float32), int(out.dtype == torch.float32), _stream()), "gemm_simt")
+                                       _ptr(bias), int(act), int(x.dtype == torch.float32), int(out.dtype == torch.float32), _stream()), "gemm_simt")
     return out
 
 
@@ -406,6 +419,19 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, out=None, splits=0, a
     if residual is not None and residual.dtype == torch.float32:
         flags |= GEMM_FP32_RESIDUAL       # an fp32 residual stream, updated in place by the epilogue when `out` is the residual itself
     return _gemm(x, w, out, bias, residual, flags, splits, fused)
+
+
+def linear_act(x, w, act, out=None):
+    """act(x @ w.T), the activation in the product's epilogue; `out` may be a column range of a wider matrix."""
+    if not x.is_cuda:
+        y = ref.linear_act(x, w, act)
+        return y if out is None else out.copy_(y)
+    if out is None:
+        out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
+    assert x.dtype == w.dtype == out.dtype and x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
+    if x.dtype == torch.float32 or not _tma_ok(x, w):
+        return _gemm_simt(x, w, out, act=1 + _ACT[act])
+    return _gemm(x, w, out, None, None, (1 + _ACT[act]) << 8, 0)
 
 
 def qkv_rope_append(x, w, bias, positions, slots, cos_cache, sin_cache, k_cache, v_cache, Hq, Hkv, D, rot, norm_eps=0.0):
@@ -706,9 +732,11 @@ class MoePlan:
                  "tile_row0", "tile_rows", "num_tiles")
 
 
-def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=None, token_tile: int = 0, topk=None, shared: bool = False) -> MoePlan:
+def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=None, token_tile: int = 0, topk=None, shared: bool = False, correction=None,
+              groups: int = 1, keep: int = 1, scale: float = 1.0) -> MoePlan:
     """router_logits [T, E] fp32 -> MoePlan (top-k, routing weights, rows grouped by expert, GEMM tile list).
-    mode 0: softmax over the selected logits; 1: softmax over all experts; 2: the latter renormalised.
+    mode 0: softmax over the selected logits; 1: softmax over all experts; 2: the latter renormalised; 3: the selected sigmoid scores divided by their
+    sum, times `scale`, the selection by score + correction (fp32 [E]) within the `keep` best of `groups` groups.
     expert_range (lo, hi): only these experts are local (expert parallelism).  topk = (idx int32 [T, k], weights fp32 [T, k]):
     a selection made elsewhere (PhiMoE's sparse mixer); only the grouping by expert is computed.  shared: every token is also served by
     expert E, with weight 1 (the plan then has E + 1 experts and k + 1 of them per token)."""
@@ -737,7 +765,11 @@ def moe_route(router_logits: torch.Tensor, k: int, mode: int = 0, expert_range=N
     tiles = torch.empty(3 * pl.max_tiles + 1, **i32)
     pl.tile_expert, pl.tile_row0, pl.tile_rows = tiles[:pl.max_tiles], tiles[pl.max_tiles:2 * pl.max_tiles], tiles[2 * pl.max_tiles:3 * pl.max_tiles]
     pl.num_tiles = tiles[3 * pl.max_tiles:]
-    if topk is None:
+    if mode == 3:
+        assert topk is None and not shared and correction.dtype == torch.float32 and correction.numel() == E
+        _lib.check(L.ogb_moe_topk_grouped(_ptr(router_logits), router_logits.stride(0), T, E, k, _ptr(correction), int(groups), int(keep), float(scale),
+                                          _ptr(pl.topk_idx), _ptr(pl.topk_w), _stream()), "moe_topk_grouped")
+    elif topk is None:
         _lib.check(L.ogb_moe_topk(_ptr(router_logits), router_logits.stride(0), T, routed, top, mode, int(shared), _ptr(pl.topk_idx), _ptr(pl.topk_w), _stream()),
                    "moe_topk")
     _lib.check(L.ogb_moe_sort(_ptr(pl.topk_idx), T, k, E, lo, hi, bt, _ptr(pl.expert_offsets), _ptr(pl.sorted_token), _ptr(pl.inv_pos),
@@ -751,11 +783,14 @@ def moe_fp4_reads_rows(w, plan: MoePlan) -> bool:
     return isinstance(w, Fp4Experts) and w.half and bool(_lib.lib().ogb_moe_fp4_reads_row_map(plan.bt, w.K, 1))
 
 
+MOE_ACTS = {"relu2": 1 + _ACT["relu2"]}      # activations of experts without a gate matrix (act_kind of moe_gemm with pair=False)
+
+
 def moe_gemm(xs: torch.Tensor, w: torch.Tensor, plan: MoePlan, bias=None, act_kind: int = 0, alpha: float = 1.0, limit: float = 0.0,
-             out_dtype=torch.bfloat16, row_map: bool = False):
+             out_dtype=torch.bfloat16, row_map: bool = False, pair: bool = True):
     """Grouped expert GEMM over rows sorted by expert.  xs [T*k, K] bf16; w [E, N, K] bf16; bias [E, N].
     act_kind 0: plain; 1: silu(gate)*up; 2: clamped SwiGLU(alpha, limit) — both need the 64-row gate/up blocks
-    of interleave_experts_gate_up and return N/2 columns."""
+    of interleave_experts_gate_up and return N/2 columns.  pair=False: act_kind is 0 or an entry of MOE_ACTS, for every column."""
     E, N, K = w.shape
     assert xs.is_cuda and xs.stride(-1) == 1
     ws = workspace(xs.device)
@@ -776,9 +811,10 @@ def moe_gemm(xs: torch.Tensor, w: torch.Tensor, plan: MoePlan, bias=None, act_ki
         _lib.check(rc, "moe_gemm_fp4")
         return out
     assert xs.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous()
-    out = torch.empty(xs.shape[0], N // 2 if act_kind else N, dtype=torch.bfloat16, device=xs.device)
+    pair = pair and act_kind != 0
+    out = torch.empty(xs.shape[0], N // 2 if pair else N, dtype=torch.bfloat16, device=xs.device)
     rc = _lib.lib().ogb_moe_gemm(_ptr(xs), xs.stride(0), _ptr(w), K, _ptr(out), out.stride(0), xs.shape[0], N, K, E, _ptr(bias),
-                                 GEMM_ACT_PAIR if act_kind else 0, int(act_kind), float(alpha), float(limit), _ptr(plan.tile_expert),
+                                 GEMM_ACT_PAIR if pair else 0, int(act_kind), float(alpha), float(limit), _ptr(plan.tile_expert),
                                  _ptr(plan.tile_row0), _ptr(plan.tile_rows), _ptr(plan.num_tiles), plan.max_tiles, plan.bt, ws.status,
                                  _stream())
     _lib.check(rc, "moe_gemm")
@@ -799,11 +835,11 @@ def moe_gemm_simt(xs: torch.Tensor, w: torch.Tensor, plan: MoePlan, mapped: bool
 
 
 def expert_act(gu: torch.Tensor, kind: str, alpha: float = 1.702, limit: float = 0.0) -> torch.Tensor:
-    """Activation of expert rows whose columns alternate (gate, up): [n, 2 I] -> [n, I]."""
+    """Activation of expert rows whose columns alternate (gate, up): [n, 2 I] -> [n, I]; of rows without gates ("relu2"): [n, I] -> [n, I]."""
     assert gu.is_cuda and gu.is_contiguous()
-    n, inter = gu.shape[0], gu.shape[1] // 2
+    n, inter = gu.shape[0], gu.shape[1] // (1 if kind == "relu2" else 2)
     out = torch.empty(n, inter, dtype=gu.dtype, device=gu.device)
-    _lib.check(_lib.lib().ogb_expert_act(_ptr(gu), _ptr(out), n, inter, {"silu": 0, "clamped": 1}[kind], float(alpha), float(limit),
+    _lib.check(_lib.lib().ogb_expert_act(_ptr(gu), _ptr(out), n, inter, {"silu": 0, "clamped": 1, "relu2": 2}[kind], float(alpha), float(limit),
                                         int(gu.dtype == torch.float32), _stream()), "expert_act")
     return out
 
@@ -845,22 +881,26 @@ def rope_kv_append(qkv, positions, slots, cos_cache, sin_cache, k_cache, v_cache
     return qkv
 
 
-def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv=None):
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv=None, talk=None,
+             mixed=None):
     """Between the projection [Hq queries | Hkv keys | Hv (None: Hkv) values | ...] of an attention layer and its attention: RMS norm of every query and
     key head over its `dim` columns (weights fp32 [dim] or None), rotation of the first 2 * cos.shape[1] of them (cos / sin fp32 [positions,
     rot / 2], or None), queries in place, keys and values to row slots[t] of the caches [slots, Hkv, key_row] and [slots, Hv, value_row]
-    (slot < 0: to no row).  Any sizes, bf16 or fp32."""
+    (slot < 0: to no row).  Any sizes, bf16 or fp32.  talk [Hq, Hq] fp32: the queries stay; row t of `mixed` [T, Hq * Hkv * key_row] gets, for head h and
+    key head c, the sum of talk[h, g] times query g over the heads g of c's group."""
     Hv = Hv or Hkv
     _check_index("qkv_prep", "slots", slots[:proj.shape[0]], k_cache.shape[0], -1)
     if cos is not None:
         _check_index("qkv_prep", "positions", positions[:proj.shape[0]], cos.shape[0])
     if not proj.is_cuda:
-        return ref.qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv)
+        return ref.qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv, talk, mixed)
+    assert talk is None or (talk.dtype == torch.float32 and talk.is_contiguous() and mixed.is_contiguous() and mixed.dtype == proj.dtype and
+                            mixed.shape == (proj.shape[0], Hq * Hkv * key_row))
     assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == proj.dtype
     assert proj.dtype in (torch.bfloat16, torch.float32) and all(w is None or w.dtype == torch.float32 for w in (q_norm_w, k_norm_w, cos, sin))
     _lib.check(_lib.lib().ogb_qkv_prep(_ptr(proj), proj.stride(0), Hq, Hkv, Hv, dim, key_row, value_row, _ptr(q_norm_w), _ptr(k_norm_w), float(eps),
                                       _ptr(positions), _ptr(cos), _ptr(sin), 2 * cos.shape[1] if cos is not None else 0,
-                                      cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(k_cache), _ptr(v_cache), proj.shape[0],
+                                      cos.shape[0] if cos is not None else 1, _ptr(slots), _ptr(k_cache), _ptr(v_cache), proj.shape[0], _ptr(talk), _ptr(mixed),
                                       int(proj.dtype == torch.float32), _stream()), "qkv_prep")
     return proj
 
@@ -899,23 +939,24 @@ _TC_ATTENTION = os.environ.get("OGB_ATTN_TC", "1") != "0"
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale, window=0,
                     sinks=None, softcap=0.0, max_q_len=None, max_kv_len=None, splits=None, out=None, total_tokens=None, order=None,
-                    min_q_len=None, vdim=None, chunk=0, gate=None, maps=1, diff=None):
+                    min_q_len=None, vdim=None, chunk=0, gate=None, maps=1, diff=None, joint=False, out_scale=1.0):
     """q: [T, stride] with the Hq*D query columns first.  Returns [T, Hq*D].  total_tokens: the requests of this call only cover
     the first `total_tokens` rows of q (sizes the split-KV scratch).  min_q_len: shortest request of the call when the caller
     knows it (a call whose every request is long runs on the tensor-core prefill kernel alone).  vdim (layers with sizes of their own): width
     of a value head; chunk > 0: position p sees the keys from p // chunk * chunk on; gate [T, Hq]: each head's output is multiplied by its
     sigmoid, or [T, heads * vdim]: each output column.  maps = 2, diff = (lambda, post, eps, columns): differential attention - q holds Hq vectors of
     D / 2 columns, 2 h and 2 h + 1 for head h, a key head both maps' keys; returns the Hq / 2 heads (see csrc/kernels.h, ogb_attention_diff_merge),
-    RMS-normed over the first `columns` of each."""
+    RMS-normed over the first `columns` of each.  joint: the key heads of a cache row are one key of D columns, which every query head (D wide) meets.
+    The result is multiplied by out_scale."""
     _check_index("paged_attention", "block_table", block_table, k_cache.shape[0] // block_size, -1)
     _check_index("paged_attention", "cu_seqlens", cu_seqlens[:past_lens.shape[0] + 1], q.shape[0] + 1)
     if not q.is_cuda:
         o = ref.paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                                window, sinks, softcap, vdim, chunk, gate, maps, diff)
+                                window, sinks, softcap, vdim, chunk, gate, maps, diff, joint, out_scale)
         return o if out is None else out.copy_(o)
-    if vdim is not None or chunk > 0 or gate is not None or maps > 1:
+    if vdim is not None or chunk > 0 or gate is not None or maps > 1 or joint or out_scale != 1.0:
         return _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, vdim or D, scale, window, chunk,
-                                      sinks, softcap, gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps, diff)
+                                      sinks, softcap, gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps, diff, joint, out_scale)
     T = q.shape[0] if total_tokens is None else total_tokens
     B = past_lens.shape[0]
     if out is None:
@@ -967,7 +1008,7 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
 
 
 def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, dk, dv, scale, window, chunk, sinks, softcap,
-                           gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps=1, diff=None):
+                           gate, max_q_len, max_kv_len, splits, out, total_tokens, order, min_q_len, maps=1, diff=None, joint=False, out_scale=1.0):
     """paged_attention of layers with sizes of their own: the tensor-memory kernel for requests with at least TC_ATTENTION_MIN_ROWS query
     rows, the warp-MMA kernel for the others, plain arithmetic for fp32 and for sizes neither can address."""
     import ctypes
@@ -985,7 +1026,7 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
     in_kernel = gate if diff is None else None             # (a differential layer's gate belongs to the merge of its maps)
     layer = _lib.AttnLayer(Hq=Hq, Hkv=Hkv, dk=dk, dv=dv, window=int(window), chunk=int(chunk), gate_stride=gate.stride(0) if gate is not None else 0,
                            scale=float(scale), sinks=_ptr(sinks), gate=_ptr(in_kernel), gate_wide=int(wide), maps=maps, raw=int(diff is not None),
-                           softcap=float(softcap or 0.0))
+                           softcap=float(softcap or 0.0), joint=int(joint), out_scale=float(out_scale))
 
     def merge(part, sp, part_tokens):
         """Differential layers: the two maps' partial results of the call's tokens become the heads."""
@@ -1033,6 +1074,40 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
         _lib.check(L.ogb_attention_tc_mixed(*inputs, int(max_q_len), long_rows, slots, int(sp), T, _ptr(scratch),
                                             scratch.numel() if scratch is not None else 0, ws.status, _stream()), "attention_tc_mixed")
     return out if diff is None else merge(scratch, sp, T)
+
+
+# ------------------------------------------------------------------------------------------ recurrent mixers of declared stacks
+def min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale=1.0, max_q_len=0):
+    """Gated average per column over packed sequences: S <- (1 - sigmoid(z)) S + sigmoid(z) * c(x) with c(x) = x + 1/2 for x >= 0 and sigmoid(x) below;
+    out = S * silu(g) * scale.  z, x, g [T, W]: columns of one matrix; state [slots, W] fp32 (rows may be further apart), updated in place; a request whose
+    past length is 0 starts from zero.  max_q_len: the most tokens a request feeds (0: unknown)."""
+    if not z.is_cuda:
+        return ref.min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale)
+    T, W = z.shape
+    assert z.dtype == x.dtype == g.dtype == out.dtype and z.stride() == x.stride() == g.stride() and z.stride(1) == out.stride(1) == 1
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and out.shape == (T, W)
+    _lib.check(_lib.lib().ogb_min_gru(_ptr(z), _ptr(x), _ptr(g), z.stride(0), _ptr(state), state.stride(0), _ptr(slots), _ptr(cu_seqlens), _ptr(past_lens),
+                                     _ptr(out), out.stride(0), past_lens.shape[0], W, float(scale), int(max_q_len or T), int(z.dtype == torch.float32),
+                                     _stream()), "min_gru")
+    return out
+
+
+def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out, max_q_len=0):
+    """Matrix memories over packed sequences (see csrc/recurrent.cu): proj [T, queries | keys | values | output gate], gates fp32 [T, input | forget logits],
+    their biases gate_b and the heads' norm weight fp32; state [slots, heads * (dim * vdim + dim + 1)] fp32, updated in place; out [T, heads * vdim]."""
+    if not proj.is_cuda:
+        return ref.mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out)
+    import ctypes
+    nk, nv, es = heads * dim, heads * vdim, proj.element_size()
+    assert proj.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype and gates.dtype == torch.float32 and gates.stride(1) == 1
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * (dim * vdim + dim + 1)
+    at = proj.data_ptr()
+    p = _lib.Mlstm(q=at, k=at + nk * es, v=at + 2 * nk * es, g=at + (2 * nk + nv) * es, gates=_ptr(gates), gate_b=_ptr(gate_b), norm_w=_ptr(norm_w),
+                   out=_ptr(out), state=_ptr(state), slots=_ptr(slots), cu_seqlens=_ptr(cu_seqlens), past_lens=_ptr(past_lens), slot_stride=state.stride(0),
+                   ld=proj.stride(0), ldg=gates.stride(0), ldo=out.stride(0), B=past_lens.shape[0], H=heads, d=dim, dv=vdim, T=proj.shape[0],
+                   max_q_len=int(max_q_len or proj.shape[0]), fp32=int(proj.dtype == torch.float32), cap=float(cap), eps=float(eps))
+    _lib.check(_lib.lib().ogb_mlstm(ctypes.byref(p), _stream()), "mlstm")
+    return out
 
 
 # ------------------------------------------------------------------------------------------ latent attention

@@ -32,7 +32,20 @@ class LatentShape(ctypes.Structure):
 class AttnLayer(ctypes.Structure):
     """OgbAttnLayer of csrc/kernels.h: an attention layer with sizes and a mask of its own."""
     _fields_ = ([(n, c_int) for n in ("Hq", "Hkv", "dk", "dv", "window", "chunk", "gate_stride")] + [("scale", c_float), ("sinks", _P), ("gate", _P)] +
-                [(n, c_int) for n in ("gate_wide", "maps", "raw")] + [("softcap", c_float)])
+                [(n, c_int) for n in ("gate_wide", "maps", "raw")] + [("softcap", c_float), ("joint", c_int), ("out_scale", c_float)])
+
+
+class NormStream(ctypes.Structure):
+    """OgbNormStream of csrc/kernels.h: norms of rows of the fp32 residual stream."""
+    _fields_ = ([(n, _P) for n in ("x", "rows", "w", "b", "w2", "out", "out2", "y", "inv_pos", "topk_w")] +
+                [(n, c_int) for n in ("ldy", "k", "n_rows", "H", "layernorm", "fp32")] + [("eps", c_float)])
+
+
+class Mlstm(ctypes.Structure):
+    """OgbMlstm of csrc/kernels.h: matrix memories."""
+    _fields_ = ([(n, _P) for n in ("q", "k", "v", "g", "gates", "gate_b", "norm_w", "out", "state", "slots", "cu_seqlens", "past_lens")] +
+                [("slot_stride", c_longlong)] + [(n, c_int) for n in ("ld", "ldg", "ldo", "B", "H", "d", "dv", "T", "max_q_len", "fp32")] +
+                [("cap", c_float), ("eps", c_float)])
 
 
 class TanhNorm(ctypes.Structure):
@@ -93,11 +106,11 @@ _SIGS = {
     "ogb_causal_conv": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_causal_conv_rows": (c_int, [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_gemm_bf16_batched": (c_int, [_P, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P]),
-    "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, _P]),
+    "ogb_gemm_simt": (c_int, [_P, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, _P]),
     "ogb_moe_gemm_simt": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P, _P, c_int, c_int, _P, c_int, _P]),
     "ogb_embedding_stream": (c_int, [_P, _P, c_int, _P, _P, c_int, c_int, c_int, c_float, _P]),
     "ogb_add_normed": (c_int, [_P, _P, c_int, c_int, _P, c_float, _P, _P, _P, c_int, c_int, c_int, _P]),
-    "ogb_qkv_prep": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, _P]),
+    "ogb_qkv_prep": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, _P, _P, c_int, _P]),
     "ogb_expert_act": (c_int, [_P, _P, c_longlong, c_int, c_int, c_float, c_float, c_int, _P]),
     "ogb_attention_mixed_supported": (c_int, [c_int, c_int]),
     "ogb_attention_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P,
@@ -109,7 +122,10 @@ _SIGS = {
     "ogb_attention_diff_merge": (c_int, [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, _P, c_int, _P, c_int, c_int, _P]),
     "ogb_add_tanh_norm": (c_int, [ctypes.POINTER(TanhNorm), _P]),
     "ogb_embedding_bigram": (c_int, [ctypes.POINTER(Bigram), _P, _P, _P, _P]),
-    "ogb_norm_stream": (c_int, [_P, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, _P]),
+    "ogb_norm_stream": (c_int, [ctypes.POINTER(NormStream), _P]),
+    "ogb_min_gru": (c_int, [_P, _P, _P, c_int, _P, c_longlong, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, c_int, _P]),
+    "ogb_mlstm": (c_int, [ctypes.POINTER(Mlstm), _P]),
+    "ogb_moe_topk_grouped": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_float, _P, _P, _P]),
     "ogb_act_mul_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),
     "ogb_latent_prep": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, _P, _LS, _P, c_float, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P]),
     "ogb_gate_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, _P]),

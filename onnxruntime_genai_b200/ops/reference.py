@@ -83,6 +83,10 @@ def linear(x, w, bias=None, residual=None, out_fp32=False, norm_eps=0.0):
     return y if out_fp32 else y.to(x.dtype)
 
 
+def linear_act(x, w, act):
+    return _act(x.float() @ w.float().t(), act).to(x.dtype)
+
+
 def _act(g, act):
     if act == "silu":
         return torch.nn.functional.silu(g)
@@ -229,10 +233,11 @@ def kv8_load(cache, Hkv, D):
 
 
 def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, block_size, Hq, Hkv, D, scale,
-                    window=0, sinks=None, softcap=0.0, vdim=None, chunk=0, gate=None, maps=1, diff=None):
+                    window=0, sinks=None, softcap=0.0, vdim=None, chunk=0, gate=None, maps=1, diff=None, joint=False, out_scale=1.0):
     """q: [T, >=Hq*D] (only the first Hq*D columns are read).  vdim: width of a value head (None: D).  chunk > 0: position p sees the keys
     from p // chunk * chunk on.  gate [T, Hq]: each head's output is multiplied by its sigmoid ([T, Hq*vdim]: each column).  Returns [T, Hq*vdim].
-    maps = 2: differential attention (see ops.paged_attention), returns [T, Hq/2*vdim]."""
+    maps = 2: differential attention (see ops.paged_attention), returns [T, Hq/2*vdim].  joint: the key heads of a position are one key of D columns
+    that every query head meets.  The result is multiplied by out_scale."""
     T, DV = q.shape[0], vdim or D
     if maps == 2:
         lam, post, eps, cols = diff
@@ -247,7 +252,7 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
     if k_cache.dtype == torch.int8:
         kc, vc = kv8_load(k_cache, Hkv, D), kv8_load(v_cache, Hkv, D)
     else:
-        kc = k_cache.view(-1, Hkv, D)
+        kc = k_cache.view(-1, 1, D).expand(-1, Hkv, D) if joint else k_cache.view(-1, Hkv, D)
         vc = v_cache.view(-1, Hkv, DV)
     G = Hq // Hkv
     B = past_lens.shape[0]
@@ -286,6 +291,7 @@ def paged_attention(q, k_cache, v_cache, cu_seqlens, past_lens, block_table, blo
         if gate is not None:
             g = torch.sigmoid(gate[t0:t1].float())
             o = o * (g[:, :, None] if gate.shape[1] == Hq else g.view(n, Hq, DV))
+        o = o * out_scale
         out[t0:t1] = o.reshape(n, Hq * DV).to(q.dtype)
     return out
 
@@ -435,7 +441,47 @@ def head_project(x, w, heads, a_cols):
     return torch.cat([x[:, h * a_cols:h * a_cols + K].float() @ w[h * N:(h + 1) * N].float().t() for h in range(heads)], 1).to(x.dtype)
 
 
-def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv):
+def min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale):
+    cu = cu_seqlens.tolist()
+    zf, xf, gf = torch.sigmoid(z.float()), x.float(), torch.nn.functional.silu(g.float()) * scale
+    c = torch.where(xf >= 0, xf + 0.5, torch.sigmoid(xf))
+    for r in range(past_lens.shape[0]):
+        S = torch.zeros_like(zf[0]) if int(past_lens[r]) == 0 else state[int(slots[r])].clone()
+        for t in range(cu[r], cu[r + 1]):
+            S = (1 - zf[t]) * S + zf[t] * c[t]
+            out[t] = (S * gf[t]).to(out.dtype)
+        if cu[r + 1] > cu[r]:
+            state[int(slots[r])] = S
+    return out
+
+
+def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out):
+    T, nk, nv = proj.shape[0], heads * dim, heads * vdim
+    q = proj[:, :nk].float().view(T, heads, dim) * dim ** -0.5
+    k, v, g = proj[:, nk:2 * nk].float().view(T, heads, dim), proj[:, 2 * nk:2 * nk + nv].float().view(T, heads, vdim), proj[:, 2 * nk + nv:2 * nk + 2 * nv].float()
+    lg = cap * torch.tanh((gates.float() + gate_b) / cap)
+    li, lf = lg[:, :heads], torch.nn.functional.logsigmoid(lg[:, heads:])
+    cu = cu_seqlens.tolist()
+    for r in range(past_lens.shape[0]):
+        if cu[r] == cu[r + 1]:
+            continue
+        st = state[int(slots[r])]
+        st = torch.zeros_like(st) if int(past_lens[r]) == 0 else st.clone()
+        S, n, m = st[:nk * vdim].view(heads, dim, vdim), st[nk * vdim:nk * vdim + nk].view(heads, dim), st[nk * vdim + nk:]
+        for t in range(cu[r], cu[r + 1]):
+            new = torch.maximum(lf[t] + m, li[t])
+            keep, add = torch.exp(lf[t] + m - new), torch.exp(li[t] - new)
+            S = keep[:, None, None] * S + (add[:, None] * k[t])[:, :, None] * v[t][:, None, :]
+            n = keep[:, None] * n + add[:, None] * k[t]
+            m = new
+            o = torch.einsum("hd,hdv->hv", q[t], S) / (torch.maximum((q[t] * n).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+            out[t] = (o.reshape(-1) * norm_w * torch.sigmoid(g[t])).to(out.dtype)
+        state[int(slots[r])] = torch.cat([S.reshape(-1), n.reshape(-1), m])
+    return out
+
+
+def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, positions, cos, sin, slots, k_cache, v_cache, Hv, talk=None, mixed=None):
     T, nq, nk = proj.shape[0], Hq * key_row, Hkv * key_row
     q, k, v = proj[:, :nq].view(T, Hq, key_row), proj[:, nq:nq + nk].view(T, Hkv, key_row), proj[:, nq + nk:nq + nk + Hv * value_row]
     pos = positions.long().clamp(0, cos.shape[0] - 1) if cos is not None else None
@@ -446,7 +492,12 @@ def qkv_prep(proj, Hq, Hkv, dim, key_row, value_row, q_norm_w, k_norm_w, eps, po
         if w is not None:
             y[..., :dim] = x[..., :dim] * torch.rsqrt(x[..., :dim].pow(2).mean(-1, keepdim=True) + eps) * w.float()
         return _rotate(y, cos[pos], sin[pos], 2 * cos.shape[1], False) if cos is not None else y
-    q.copy_(prepared(q, q_norm_w).to(proj.dtype))
+    turned = prepared(q, q_norm_w)
+    if talk is None:
+        q.copy_(turned.to(proj.dtype))
+    else:
+        parts = torch.einsum("hcg,tcgd->thcd", talk.view(Hq, Hkv, Hq // Hkv), turned.view(T, Hkv, Hq // Hkv, key_row))
+        mixed.copy_(parts.reshape(T, -1).to(mixed.dtype))
     ok = slots >= 0
     at = slots[ok].long()
     k_cache.view(-1, Hkv, key_row)[at] = prepared(k, k_norm_w)[ok].to(k_cache.dtype)

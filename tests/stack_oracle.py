@@ -1,6 +1,7 @@
 """A slow, plain restatement of declared-stack decoders (gated-delta and latent-attention mixers in parallel blocks; chunked attention
 with sinks and routed experts in blocks whose norms follow the sub-layers; soft-capped, differential and query-compressed latent attention with
-output gates in pre-norm blocks that run several times), one function per mechanism, token by token where the mechanism is a recurrence.  It shares no code with the package: the tests compare the
+output gates in pre-norm blocks that run several times; attention with mixed heads beside a gated recurrence, and matrix memories, in parallel blocks
+with a norm per sub-layer), one function per mechanism, token by token where the mechanism is a recurrence.  It shares no code with the package: the tests compare the
 runtime against it.  Weights come as a dictionary of tensors under the checkpoint's names; all math runs in `dtype` (float64 by
 default).  A whole sequence is evaluated at once, from its first token: there is no cache here."""
 import math
@@ -290,6 +291,102 @@ def selected_experts(x, w, p, m):
     return out
 
 
+def mixed_scores(q, k, mix, scale):
+    """Scores [H, T, T] of q [T, H, d] and k [T, G, d], head h a sum of all heads' scores weighted by mix[h]."""
+    H, rep = q.shape[1], q.shape[1] // k.shape[1]
+    own = torch.stack([q[:, h] @ k[:, h // rep].T * scale for h in range(H)])
+    return torch.stack([sum(mix[h, g] * own[g] for g in range(H)) for h in range(H)])
+
+
+def mixed_heads_attention(q, k, v, ok, scale, mix):
+    """q [T, H, d], k [T, G, d], v [T, G, dv], mix [H, H] -> [T, H, dv]."""
+    rep = q.shape[1] // k.shape[1]
+    s = mixed_scores(q, k, mix, scale)
+    return torch.stack([torch.softmax(s[h].masked_fill(~ok, -math.inf), -1) @ v[:, h // rep] for h in range(q.shape[1])], 1)
+
+
+def mixed_heads_mixer(x, w, p, m, eps):
+    T, H, G, d, dv = x.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q, k, v = ((x @ w[p + n].T + w[p + n + ".b"]).view(T, h, c) for n, h, c in (("q", H, d), ("k", G, d), ("v", G, dv)))
+    q, k = (rotate(rms_norm(t, w[p + n + ".norm"], eps), m.get("rot")) for t, n in ((q, "q"), (k, "k")))
+    o = mixed_heads_attention(q, k, v, visible(T, m.get("mask")), m["scale"], w[p + "talk"])
+    return gated_output(o, x, w, p) + w[p + "o.b"]
+
+
+def gated_average(z, u):
+    """S_t = (1 - z_t) S_(t-1) + z_t c(u_t) from S = 0, per column; c(u) = u + 1/2 above zero, sigmoid(u) below."""
+    S, out = torch.zeros_like(u[0]), torch.zeros_like(u)
+    for t in range(u.shape[0]):
+        c = torch.where(u[t] >= 0, u[t] + 0.5, torch.sigmoid(u[t]))
+        S = (1 - z[t]) * S + z[t] * c
+        out[t] = S
+    return out
+
+
+def gated_average_mixer(x, w, p, m, eps):
+    S = gated_average(torch.sigmoid(x @ w[p + "z"].T + w[p + "z.b"]), x @ w[p + "x"].T + w[p + "x.b"])
+    g = x @ w[p + "g"].T
+    return (S * g * torch.sigmoid(g)) @ w[p + "o"].T
+
+
+def side_by_side_mixer(x, w, p, m, eps):
+    return (m["left_scale"] * mixed_heads_mixer(x, w, p + "left.", m["left"], eps) + m["right_scale"] * gated_average_mixer(x, w, p + "right.", m["right"], eps))
+
+
+def matrix_memory(q, k, v, i, f):
+    """q, k [T, H, d], v [T, H, dv], log gates i (input) and f (forget) [T, H] -> [T, H, dv]; the stored sums are kept relative to exp(m)."""
+    T, H, dv = v.shape
+    out = torch.zeros_like(v)
+    for h in range(H):
+        S, n, m = torch.zeros(q.shape[2], dv, dtype=v.dtype), torch.zeros(q.shape[2], dtype=v.dtype), torch.zeros((), dtype=v.dtype)
+        for t in range(T):
+            new = torch.maximum(f[t, h] + m, i[t, h])
+            keep, add = torch.exp(f[t, h] + m - new), torch.exp(i[t, h] - new)
+            S, n, m = keep * S + add * torch.outer(k[t, h], v[t, h]), keep * n + add * k[t, h], new
+            out[t, h] = (q[t, h] @ S) / (torch.maximum((q[t, h] @ n).abs(), torch.exp(-m)) + 1e-6)
+    return out
+
+
+def matrix_memory_mixer(x, w, p, m, eps):
+    T, H, d, dv, cap = x.shape[0], m["heads"], m["dim"], m["vdim"], m["gate_cap"]
+    q, k, v = (x @ w[p + "q"].T).view(T, H, d) * d ** -0.5, (x @ w[p + "k"].T).view(T, H, d), (x @ w[p + "v"].T).view(T, H, dv)
+    i = capped(x @ w[p + "i"].T + w[p + "i.b"], cap)
+    f = -torch.log1p(torch.exp(-capped(x @ w[p + "f"].T + w[p + "f.b"], cap)))
+    o = rms_norm(matrix_memory(q, k, v, i, f), 1.0, eps).reshape(T, H * dv) * w[p + "norm"]
+    return gated_output(o, x, w, p)
+
+
+def erf_feed_forward(x, w, p, m=None):
+    y = x @ w[p + "up"].T
+    return (0.5 * y * (1 + torch.erf(y / math.sqrt(2)))) @ w[p + "down"].T
+
+
+def squared_relu_expert(x, w, p):
+    return torch.relu(x @ w[p + "up"].T) ** 2 @ w[p + "down"].T
+
+
+def grouped_choice(c, count, keep, top):
+    """Indices of the `top` largest of c [E] among the `keep` groups of neighbours whose two largest entries have the largest sums."""
+    group = c.view(count, -1)
+    best = torch.sort(group, -1, descending=True).values[:, :2].sum(-1)
+    open_ = torch.zeros(count, dtype=torch.bool)
+    open_[torch.argsort(best, descending=True)[:keep]] = True
+    return torch.argsort(group.masked_fill(~open_[:, None], -math.inf).reshape(-1), descending=True)[:top]
+
+
+def grouped_experts(x, w, p, m):
+    """Each token: experts chosen by sigmoid scores plus a correction, weighted by the scores' shares times the router's scale."""
+    r = m["router"]
+    s = torch.sigmoid(x @ w[p + "router"].T)
+    out = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        chosen = grouped_choice(s[t] + w[p + "correction"], r["groups"]["count"], r["groups"]["keep"], r["top"])
+        share = s[t, chosen] / (s[t, chosen].sum() + 1e-20) * r["scale"]
+        for e, a in zip(chosen.tolist(), share):
+            out[t] = out[t] + a * squared_relu_expert(x[t:t + 1], w, f"{p}e{e}.")[0]
+    return out
+
+
 # ------------------------------------------------------------------------------------------------ the stack
 MIXERS = {"delta": delta_mixer, "latent_attention": latent_mixer, "attention": attention_mixer}
 FEED_FORWARDS = {"dense": gelu_feed_forward, "moe": routed_experts}
@@ -347,8 +444,32 @@ def looped_forward(cfg, weights, tokens, dtype=torch.float64):
     return bounded_norm(x, w, "final.norm") @ w["head"].T, torch.stack(streams)
 
 
+TWO_NORM_MIXERS = {"parallel": side_by_side_mixer, "mlstm": matrix_memory_mixer}
+TWO_NORM_FEED_FORWARDS = {"dense": erf_feed_forward, "moe": grouped_experts}
+
+
+def two_norm_parallel_block(x, w, p, e, eps):
+    y = TWO_NORM_MIXERS[e["type"]](layer_norm(x, w[p + "norm1"], 0, eps), w, p + "mix.", e["mixer"], eps)
+    if e.get("mlp"):
+        y = y + TWO_NORM_FEED_FORWARDS[e["mlp"]["kind"]](layer_norm(x, w[p + "norm2"], 0, eps), w, p + "mlp.", e["mlp"])
+    return x + y
+
+
+def two_norm_forward(cfg, weights, tokens, dtype=torch.float64):
+    """stack_forward of parallel blocks with a norm per sub-layer."""
+    w, eps = {k: v.to(dtype) for k, v in weights.items()}, cfg["norm"]["eps"]
+    x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)] * cfg["embedding"]["scale"]
+    streams = []
+    for i, _ in passes(cfg):
+        x = two_norm_parallel_block(x, w, f"l{i}.", cfg["layers"][i], eps)
+        streams.append(x)
+    return layer_norm(x, w["final.norm"], 0, eps) @ w["head"].T, torch.stack(streams)
+
+
 def stack_forward(cfg, weights, tokens, dtype=torch.float64):
     """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
+    if cfg["architecture"] == "Tevilix":
+        return two_norm_forward(cfg, weights, tokens, dtype)
     if cfg["architecture"] == "Sugelix":
         return looped_forward(cfg, weights, tokens, dtype)
     w = {k: v.to(dtype) for k, v in weights.items()}
