@@ -128,7 +128,9 @@ int ogb_min_gru(const void* z, const void* x, const void* g, int ld, float* stat
                 const int32_t* past_lens, void* out, int ldo, int B, int W, float scale, int max_q_len, int fp32, void* stream);
 // Matrix memories of H heads with keys of d and values of dv columns.  q, k, v, g: columns of rows of ld elements ([H, d], [H, d], [H, dv], [H, dv]); gates:
 // fp32 rows of ldg, H logits of the input gates and H of the forget gates, to which gate_b [2 H] is added; out rows of ldo.  State of a slot: memories
-// [H, d, dv], normalisers [H, d], maxima [H].  max_q_len: the most tokens a request of the step feeds, T the step's tokens.
+// [H, d, dv], normalisers [H, d], maxima [H].  max_q_len: the most tokens a request of the step feeds, T the step's tokens.  long_tokens > 0 (bf16):
+// requests with at least that many tokens run in the chunk form, in ogb_mlstm_scratch_bytes of scratch (0: these sizes have none); all_long: no request of the
+// step has fewer.
 typedef struct OgbMlstm {
   const void *q, *k, *v, *g;
   const float *gates, *gate_b, *norm_w;
@@ -136,9 +138,12 @@ typedef struct OgbMlstm {
   float* state;
   const int32_t *slots, *cu_seqlens, *past_lens;
   long long slot_stride;
-  int ld, ldg, ldo, B, H, d, dv, T, max_q_len, fp32;
+  int ld, ldg, ldo, B, H, d, dv, T, max_q_len, fp32, long_tokens, all_long;
   float cap, eps;
+  void* scratch;
+  long long scratch_bytes;
 } OgbMlstm;
+long long ogb_mlstm_scratch_bytes(int T, int B, int H, int d, int dv);
 int ogb_mlstm(const OgbMlstm* a, void* stream);
 
 // ---- attention_tc.cu, latent form (long prompts over expanded keys and values)

@@ -12,6 +12,13 @@
 //   m' = max(f + m, i),  S <- exp(f + m - m') S + exp(i - m') k v^T,  n likewise with k alone,  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6),
 //   out = o / rms(o) * norm * sigmoid(g).
 //   mlstm_step_kernel     any step.  A cluster of CTAs shares the columns of a head; the state streams through registers once per token.
+//   chunk form (bf16)     requests with many tokens, 64 at a time.  With b_t the sum of the chunk's log forget gates up to t, c_t = i_t - b_t and
+//                         M_t = max(m before the chunk, c_s for s <= t), the running maximum is b_t + M_t and the chunk's outputs and its end state are
+//                         products:  num_t = e^(m - M_t) q_t S + sum_{s <= t} e^(c_s - M_t) (q_t . k_s) v_s,  S' = e^(m - M_L) S + sum_s e^(c_s - M_L) k_s v_s^T
+//                         (every exponent is at most 0).  Four kernels: the gates of all tokens (prefix sums and maxima); every chunk's own sum of
+//                         k v^T; the scan of these over a request's chunks, elementwise; every chunk's outputs.  Sums, decays and states are fp32; as operands of
+//                         the tensor cores, weighted keys, states and weighted scores are split into two bf16 numbers (16 bits of mantissa), queries,
+//                         keys and values are bf16 as the projection left them.
 #include "common.cuh"
 #include "kernels.h"
 
@@ -283,6 +290,428 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, i
   if (C > 1) { rec_cluster_arrive(); rec_cluster_wait(); }          // no CTA leaves while another may read its sums
 }
 
+// ------------------------------------------------------------------------------------ matrix memory, chunks of a prompt
+constexpr int MC_L = 64;               // tokens of a chunk
+
+struct MlstmChunk {
+  float *c, *M, *floor;                // [H, T] per token: c_t, M_t, e^-(running maximum)
+  float *m_in, *M_last;                // [chunks, H]: maximum before the chunk, M of its last token
+  float* sums;                         // [chunks, H, KS, NT, 32 lanes, 4]: first a chunk's own sums (fp32), then the state before it (bf16 pairs)
+  float* nsums;                        // [chunks, H, dp]: the same for the normalisers (fp32 throughout)
+  int T, KS, NT;                       // 16-row groups of the keys' columns, 8-column groups of the values' (both padded to whole 16s)
+  int min_tokens;                      // shorter requests are not served here
+};
+// chunk j of request b: ids are unique because a request starts at least as many ids after the one before it as that one has chunks
+__device__ __forceinline__ int mc_chunk(int t0, int b, int j) { return t0 / MC_L + b + j; }
+
+// One CTA per (head, request).  A warp takes chunks, a lane two of a chunk's tokens; then the maxima are chained over the chunks.
+__global__ void __launch_bounds__(256) mlstm_gates_kernel(MlstmParams p, MlstmChunk k) {
+  extern __shared__ float sm[];        // per chunk: sum of log forget gates, largest c, maximum before the chunk
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y, t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len < k.min_tokens || len <= 0) return;
+  const int n = (len + MC_L - 1) / MC_L, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float *sb = sm, *sc = sm + n, *si = sm + 2 * n;
+  const float bi = p.gate_b[h], bf = p.gate_b[p.H + h];
+  float *gc = k.c + size_t(h) * k.T + t0, *gM = k.M + size_t(h) * k.T + t0, *gf = k.floor + size_t(h) * k.T + t0;
+  for (int j = warp; j < n; j += 8) {
+    float i[2], f[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = j * MC_L + 2 * lane + e;
+      i[e] = -INFINITY;
+      f[e] = 0.f;
+      if (t < len) {
+        const float* gp = p.gates + size_t(t0 + t) * p.ldg;
+        i[e] = p.cap * tanhf((gp[h] + bi) / p.cap);
+        const float y = p.cap * tanhf((gp[p.H + h] + bf) / p.cap);
+        f[e] = -(y < -20.f ? -y : log1pf(expf(-y)));
+      }
+    }
+    float s = f[0] + f[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += v; }
+    const float b1 = s, b0 = s - f[1], c0 = i[0] - b0, c1 = i[1] - b1;
+    float x = fmaxf(c0, c1);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, x, o); if (lane >= o) x = fmaxf(x, v); }
+    float before = __shfl_up_sync(0xffffffffu, x, 1);
+    if (lane == 0) before = -INFINITY;
+    const int t = j * MC_L + 2 * lane;
+    if (t < len) { gc[t] = c0; gM[t] = fmaxf(before, c0); gf[t] = b0; }
+    if (t + 1 < len) { gc[t + 1] = c1; gM[t + 1] = x; gf[t + 1] = b1; }
+    if (lane == 31) { sb[j] = b1; sc[j] = x; }
+  }
+  __syncthreads();
+  float* gm = p.state + size_t(p.slots[b]) * p.slot_stride + size_t(p.H) * p.d * (p.dv + 1) + h;
+  if (threadIdx.x == 0) {
+    float m = p.past_lens[b] == 0 ? 0.f : *gm;
+    for (int j = 0; j < n; ++j) {
+      const float M = fmaxf(m, sc[j]);
+      const size_t at = size_t(mc_chunk(t0, b, j)) * p.H + h;
+      k.m_in[at] = m;
+      k.M_last[at] = M;
+      si[j] = m;
+      m = sb[j] + M;
+    }
+    *gm = m;
+  }
+  __syncthreads();
+  for (int t = threadIdx.x; t < len; t += blockDim.x) {
+    const float M = fmaxf(si[t / MC_L], gM[t]);
+    gM[t] = M;
+    gf[t] = expf(-(gf[t] + M));
+  }
+}
+
+__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+  hi = f2bf(v);
+  lo = f2bf(v - bf2f(hi));
+}
+__device__ __forceinline__ uint32_t pair_bits(__nv_bfloat16 a, __nv_bfloat16 b) {
+  return uint32_t(__bfloat16_as_ushort(a)) | uint32_t(__bfloat16_as_ushort(b)) << 16;
+}
+
+// A chunk's own sums, transposed: rows are value columns, so that a thread's results are the two halves of its B operand in the output kernel.
+// Grid (tiles of 64 key columns x 64 value columns, chunks of the longest request, requests x heads).
+constexpr int MC_PITCH = 64 + 8;
+__global__ void __launch_bounds__(128) mlstm_sums_kernel(MlstmParams p, MlstmChunk k) {
+  __shared__ __align__(16) __nv_bfloat16 sv[MC_L * MC_PITCH], shi[MC_L * MC_PITCH], slo[MC_L * MC_PITCH];
+  __shared__ float sw[MC_L];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.z % p.H, b = blockIdx.z / p.H, j = blockIdx.y, t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len < k.min_tokens || j * MC_L >= len) return;
+  const int v_tiles = (k.NT + 7) / 8, v0 = blockIdx.x % v_tiles * 64, d0 = blockIdx.x / v_tiles * 64;
+  const int n = min(MC_L, len - j * MC_L), first = t0 + j * MC_L, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int chunk = mc_chunk(t0, b, j);
+  const float M = k.M_last[size_t(chunk) * p.H + h];
+  if (tid < MC_L) sw[tid] = tid < n ? expf(k.c[size_t(h) * k.T + first + tid] - M) : 0.f;
+  __syncthreads();
+  for (int i = tid; i < MC_L * 8; i += 128) {
+    const int t = i / 8, c = i % 8 * 8;
+    const bool ok = t < n;
+    const size_t row = size_t(first + t) * p.ld;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u), kk = v, hi, lo;
+    if (ok && v0 + c < p.dv) v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.v) + row + size_t(h) * p.dv + v0 + c);
+    if (ok && d0 + c < p.d) kk = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.k) + row + size_t(h) * p.d + d0 + c);
+    const uint32_t* in = &kk.x;
+    uint32_t *ph = &hi.x, *pl = &lo.x;
+    const float w = sw[t];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = unpack_bf16x2(in[e]);
+      __nv_bfloat16 h0, l0, h1, l1;
+      split_bf16(f.x * w, h0, l0);
+      split_bf16(f.y * w, h1, l1);
+      ph[e] = pair_bits(h0, h1);
+      pl[e] = pair_bits(l0, l1);
+    }
+    *reinterpret_cast<uint4*>(sv + t * MC_PITCH + c) = v;
+    *reinterpret_cast<uint4*>(shi + t * MC_PITCH + c) = hi;
+    *reinterpret_cast<uint4*>(slo + t * MC_PITCH + c) = lo;
+  }
+  __syncthreads();
+  if (v0 == 0 && tid < 64 && d0 + tid < k.KS * 16) {
+    float s = 0.f;
+    for (int t = 0; t < MC_L; ++t) s += bf2f(shi[t * MC_PITCH + tid]) + bf2f(slo[t * MC_PITCH + tid]);
+    k.nsums[(size_t(chunk) * p.H + h) * k.KS * 16 + d0 + tid] = s;
+  }
+  if (v0 + warp * 16 >= k.NT * 8) return;
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
+#pragma unroll
+  for (int ks = 0; ks < MC_L / 16; ++ks) {
+    uint32_t a[4];
+    ldmatrix_x4_trans(a, sv + (ks * 16 + (lane & 7) + (lane >> 4) * 8) * MC_PITCH + warp * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+    for (int g = 0; g < 4; ++g) {
+      const int at = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * MC_PITCH + g * 16 + (lane >> 4) * 8;
+      uint32_t w[4];
+      ldmatrix_x4_trans(w, shi + at);
+      mma_bf16_16816(acc[2 * g], a, w[0], w[1]);
+      mma_bf16_16816(acc[2 * g + 1], a, w[2], w[3]);
+      ldmatrix_x4_trans(w, slo + at);
+      mma_bf16_16816(acc[2 * g], a, w[0], w[1]);
+      mma_bf16_16816(acc[2 * g + 1], a, w[2], w[3]);
+    }
+  }
+  float4* dst = reinterpret_cast<float4*>(k.sums) + (size_t(chunk) * p.H + h) * k.KS * k.NT * 32;
+  const int nt = (v0 + warp * 16) / 8;
+#pragma unroll
+  for (int g = 0; g < 4; ++g) {
+    const int ks = d0 / 16 + g;
+    if (ks >= k.KS) break;
+    dst[(size_t(ks) * k.NT + nt) * 32 + lane] = make_float4(acc[2 * g][0], acc[2 * g][1], acc[2 * g + 1][0], acc[2 * g + 1][1]);
+    dst[(size_t(ks) * k.NT + nt + 1) * 32 + lane] = make_float4(acc[2 * g][2], acc[2 * g][3], acc[2 * g + 1][2], acc[2 * g + 1][3]);
+  }
+}
+
+// The states before every chunk: S <- decay * S + sums, the four entries of a thread (rows 2 i, 2 i + 1, 2 i + 8, 2 i + 9 of a 16-row group, one column) kept
+// over the chunks.  The last column of CTAs takes the normalisers.  Grid (.., heads, requests).
+__global__ void __launch_bounds__(256) mlstm_scan_kernel(MlstmParams p, MlstmChunk k) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.y, b = blockIdx.z, t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len < k.min_tokens || len <= 0) return;
+  const int n = (len + MC_L - 1) / MC_L, chunk0 = mc_chunk(t0, b, 0);
+  const bool fresh = p.past_lens[b] == 0;
+  float* slot = p.state + size_t(p.slots[b]) * p.slot_stride;
+  const float *m_in = k.m_in + size_t(chunk0) * p.H + h, *M_last = k.M_last + size_t(chunk0) * p.H + h;
+  if (blockIdx.x == gridDim.x - 1) {
+    const int dp = k.KS * 16;
+    for (int i = threadIdx.x; i < dp; i += blockDim.x) {
+      float* g = slot + size_t(p.H) * p.d * p.dv + size_t(h) * p.d + i;
+      float S = fresh || i >= p.d ? 0.f : *g;
+      for (int j = 0; j < n; ++j) {
+        float* at = k.nsums + (size_t(chunk0 + j) * p.H + h) * dp + i;
+        const float u = *at;
+        *at = S;
+        S = fmaf(expf(m_in[size_t(j) * p.H] - M_last[size_t(j) * p.H]), S, u);
+      }
+      if (i < p.d) *g = S;
+    }
+    return;
+  }
+  const int f = blockIdx.x * blockDim.x + threadIdx.x;
+  if (f >= k.KS * k.NT * 32) return;
+  const int lane = f & 31, nt = (f >> 5) % k.NT, ks = (f >> 5) / k.NT;
+  const int v = nt * 8 + (lane >> 2), d = ks * 16 + (lane & 3) * 2;
+  float* g = slot + size_t(h) * p.d * p.dv + v;
+  float S[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const int r = d + (e >> 1) * 8 + (e & 1);
+    S[e] = fresh || r >= p.d || v >= p.dv ? 0.f : g[size_t(r) * p.dv];
+  }
+  const size_t stride = size_t(p.H) * k.KS * k.NT * 32;
+  float4* u = reinterpret_cast<float4*>(k.sums) + (size_t(chunk0) * p.H + h) * k.KS * k.NT * 32 + f;
+  constexpr int AHEAD = 8;
+  for (int j0 = 0; j0 < n; j0 += AHEAD) {
+    float4 x[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) if (j0 + i < n) x[i] = u[size_t(j0 + i) * stride];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      if (j0 + i >= n) break;
+      const float w = expf(m_in[size_t(j0 + i) * p.H] - M_last[size_t(j0 + i) * p.H]);
+      __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) split_bf16(S[e], hi[e], lo[e]);
+      reinterpret_cast<uint4*>(u)[size_t(j0 + i) * stride] =
+          make_uint4(pair_bits(hi[0], hi[1]), pair_bits(hi[2], hi[3]), pair_bits(lo[0], lo[1]), pair_bits(lo[2], lo[3]));
+      S[0] = fmaf(w, S[0], x[i].x); S[1] = fmaf(w, S[1], x[i].y); S[2] = fmaf(w, S[2], x[i].z); S[3] = fmaf(w, S[3], x[i].w);
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const int r = d + (e >> 1) * 8 + (e & 1);
+    if (r < p.d && v < p.dv) g[size_t(r) * p.dv] = S[e];
+  }
+}
+
+// Outputs of a chunk.  Warp (rg, cg): rows rg * 32 .. + 31; scores of 16 keys each, then NTW 8-column groups of the values.  Grid (chunks, heads, requests).
+template <int NTW>
+__global__ void __launch_bounds__(256, NTW <= 8 ? 2 : 1) mlstm_out_kernel(MlstmParams p, MlstmChunk k) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float sc[MC_L], sM[MC_L], sfl[MC_L], snq[MC_L], srow[4][MC_L];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int j = blockIdx.x, h = blockIdx.y, b = blockIdx.z, t0 = p.cu_seqlens[b], len = p.cu_seqlens[b + 1] - t0;
+  if (len < k.min_tokens || j * MC_L >= len) return;
+  const int dp = k.KS * 16, vp = k.NT * 8, qpitch = dp + 8, vpitch = vp + 8;
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* sk = sq + MC_L * qpitch;
+  __nv_bfloat16* sv = sk + MC_L * qpitch;
+  __nv_bfloat16* phi = sv + MC_L * vpitch;
+  __nv_bfloat16* plo = phi + MC_L * MC_PITCH;
+  const int n = min(MC_L, len - j * MC_L), first = t0 + j * MC_L, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+  const int rg = warp >> 2, cg = warp & 3, chunk = mc_chunk(t0, b, j);
+  const bool empty = j == 0 && p.past_lens[b] == 0;        // the state before the chunk is zero
+  for (int i = tid; i < MC_L * (dp / 8); i += 256) {
+    const int t = i / (dp / 8), c = i % (dp / 8) * 8;
+    const bool ok = t < n && c < p.d;
+    const size_t at = size_t(first + (ok ? t : 0)) * p.ld + size_t(h) * p.d + (ok ? c : 0);
+    cp_async16(sq + t * qpitch + c, static_cast<const __nv_bfloat16*>(p.q) + at, ok);
+    cp_async16(sk + t * qpitch + c, static_cast<const __nv_bfloat16*>(p.k) + at, ok);
+  }
+  cp_async_commit();
+  for (int i = tid; i < MC_L * (vp / 8); i += 256) {
+    const int t = i / (vp / 8), c = i % (vp / 8) * 8;
+    const bool ok = t < n && c < p.dv;
+    cp_async16(sv + t * vpitch + c, static_cast<const __nv_bfloat16*>(p.v) + size_t(first + (ok ? t : 0)) * p.ld + size_t(h) * p.dv + (ok ? c : 0), ok);
+  }
+  cp_async_commit();
+  const float m = k.m_in[size_t(chunk) * p.H + h];
+  if (tid < MC_L) {
+    const size_t at = size_t(h) * k.T + first + tid;
+    sc[tid] = tid < n ? k.c[at] : -INFINITY;
+    sM[tid] = tid < n ? k.M[at] : 0.f;
+    sfl[tid] = tid < n ? k.floor[at] : 1.f;
+  }
+  cp_async_wait<1>();
+  __syncthreads();
+  // ---- weighted scores
+  {
+    float acc[2][2][4] = {};
+    if (cg * 16 <= rg * 32 + 31) {
+      for (int ks = 0; ks < k.KS; ++ks) {
+        uint32_t kb[4];
+        ldmatrix_x4(kb, sk + (cg * 16 + (lane >> 4) * 8 + (lane & 7)) * qpitch + ks * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt) {
+          uint32_t a[4];
+          ldmatrix_x4(a, sq + (rg * 32 + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * qpitch + ks * 16 + (lane >> 4) * 8);
+          mma_bf16_16816(acc[mt][0], a, kb[0], kb[1]);
+          mma_bf16_16816(acc[mt][1], a, kb[2], kb[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = rg * 32 + mt * 16 + g + half * 8;
+        const float M = sM[t];
+        float sum = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const int s = cg * 16 + nt * 8 + t4 * 2;
+          __nv_bfloat16 hi[2], lo[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float w = s + e <= t ? acc[mt][nt][half * 2 + e] * p.q_scale * expf(sc[s + e] - M) : 0.f;
+            sum += w;
+            split_bf16(w, hi[e], lo[e]);
+          }
+          *reinterpret_cast<uint32_t*>(phi + t * MC_PITCH + s) = pair_bits(hi[0], hi[1]);
+          *reinterpret_cast<uint32_t*>(plo + t * MC_PITCH + s) = pair_bits(lo[0], lo[1]);
+        }
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+        if (t4 == 0) srow[cg][t] = sum;
+      }
+  }
+  // ---- q . n of the state before the chunk: four threads per row
+  {
+    const int t = tid >> 2;
+    float s = 0.f;
+    if (!empty) {
+      const float* nn = k.nsums + (size_t(chunk) * p.H + h) * dp;
+      for (int i = tid & 3; i < dp; i += 4) s = fmaf(bf2f(sq[t * qpitch + i]), nn[i], s);
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+    }
+    if ((tid & 3) == 0) snq[t] = s * p.q_scale * expf(m - sM[t]);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // ---- numerators
+  float o[2][NTW][4];
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) { o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f; }
+  const int nt0 = cg * NTW;
+  if (!empty) {
+    const uint4* S = reinterpret_cast<const uint4*>(k.sums) + (size_t(chunk) * p.H + h) * k.KS * k.NT * 32 + lane;
+    for (int ks = 0; ks < k.KS; ++ks) {
+      uint32_t a[2][4];
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt) ldmatrix_x4(a[mt], sq + (rg * 32 + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * qpitch + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int i = 0; i < NTW; ++i) {
+        if (nt0 + i >= k.NT) break;
+        const uint4 f = S[(size_t(ks) * k.NT + nt0 + i) * 32];
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt) {
+          mma_bf16_16816(o[mt][i], a[mt], f.x, f.y);
+          mma_bf16_16816(o[mt][i], a[mt], f.z, f.w);
+        }
+      }
+    }
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt) {
+      const float w0 = p.q_scale * expf(m - sM[rg * 32 + mt * 16 + g]), w1 = p.q_scale * expf(m - sM[rg * 32 + mt * 16 + g + 8]);
+#pragma unroll
+      for (int i = 0; i < NTW; ++i) { o[mt][i][0] *= w0; o[mt][i][1] *= w0; o[mt][i][2] *= w1; o[mt][i][3] *= w1; }
+    }
+  }
+#pragma unroll
+  for (int ks = 0; ks < MC_L / 16; ++ks) {
+    if (ks * 16 > rg * 32 + 31) break;
+    uint32_t a[2][4], c[2][4];
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt) {
+      const int at = (rg * 32 + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * MC_PITCH + ks * 16 + (lane >> 4) * 8;
+      ldmatrix_x4(a[mt], phi + at);
+      ldmatrix_x4(c[mt], plo + at);
+    }
+#pragma unroll
+    for (int i = 0; i < NTW; i += 2) {
+      if (nt0 + i >= k.NT) break;                          // (whole pairs of groups: NT is even)
+      uint32_t vb[4];
+      ldmatrix_x4_trans(vb, sv + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vpitch + (nt0 + i + (lane >> 4)) * 8);
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt) {
+        mma_bf16_16816(o[mt][i], a[mt], vb[0], vb[1]);
+        mma_bf16_16816(o[mt][i], c[mt], vb[0], vb[1]);
+        mma_bf16_16816(o[mt][i + 1], a[mt], vb[2], vb[3]);
+        mma_bf16_16816(o[mt][i + 1], c[mt], vb[2], vb[3]);
+      }
+    }
+  }
+  // ---- denominators, norm over the head, gate
+  float inv[2][2];
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = rg * 32 + mt * 16 + g + half * 8;
+      const float nq = snq[t] + ((srow[0][t] + srow[1][t]) + (srow[2][t] + srow[3][t]));
+      inv[mt][half] = 1.f / (fmaxf(fabsf(nq), sfl[t]) + 1e-6f);
+    }
+  __syncthreads();                                          // (the row sums have been read)
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NTW; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float x = o[mt][i][half * 2 + e] * inv[mt][half];
+          o[mt][i][half * 2 + e] = x;
+          ss = fmaf(x, x, ss);
+        }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (t4 == 0) srow[cg][rg * 32 + mt * 16 + g + half * 8] = ss;
+    }
+  __syncthreads();
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = rg * 32 + mt * 16 + g + half * 8;
+      if (t >= n) continue;
+      const float r = 1.f / sqrtf(((srow[0][t] + srow[1][t]) + (srow[2][t] + srow[3][t])) / p.dv + p.eps);
+      const __nv_bfloat16* gp = static_cast<const __nv_bfloat16*>(p.g) + size_t(first + t) * p.ld + size_t(h) * p.dv;
+      __nv_bfloat16* op = static_cast<__nv_bfloat16*>(p.out) + size_t(first + t) * p.ldo + size_t(h) * p.dv;
+#pragma unroll
+      for (int i = 0; i < NTW; ++i) {
+        const int c = (nt0 + i) * 8 + t4 * 2;
+        if (c >= p.dv) break;
+        const float2 w = *reinterpret_cast<const float2*>(p.norm_w + size_t(h) * p.dv + c), gg = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(gp + c));
+        *reinterpret_cast<uint32_t*>(op + c) =
+            pack_bf16x2(o[mt][i][half * 2] * r * w.x * rec_sigmoid(gg.x), o[mt][i][half * 2 + 1] * r * w.y * rec_sigmoid(gg.y));
+      }
+    }
+}
+
 }  // namespace ogb
 
 using namespace ogb;
@@ -322,6 +751,54 @@ static bool LaunchMlstmStep(const MlstmParams& p, int B, int cw, int C, cudaStre
   return cudaLaunchKernelEx(&cfg, mlstm_step_kernel<T, VEC>, p, cw) == cudaSuccess;
 }
 
+// Sizes of the chunk form's scratch, or false where its kernels cannot run.
+static bool MlstmChunkSizes(int T, int B, int H, int d, int dv, MlstmChunk* k, long long* floats) {
+  if (d % 8 || dv % 8 || d > 256 || dv > 512) return false;
+  k->T = T; k->KS = (d + 15) / 16; k->NT = (dv + 15) / 16 * 2;
+  const long long chunks = T / MC_L + B, per = (long long)H * k->KS * k->NT * 128;
+  *floats = 3LL * H * T + 2 * chunks * H + chunks * per + chunks * H * k->KS * 16 + 64;
+  return true;
+}
+
+OGB_API long long ogb_mlstm_scratch_bytes(int T, int B, int H, int d, int dv) {
+  MlstmChunk k;
+  long long n = 0;
+  return MlstmChunkSizes(T, B, H, d, dv, &k, &n) ? n * 4 : 0;
+}
+
+template <int NTW>
+static bool LaunchMlstmOut(const MlstmParams& p, const MlstmChunk& k, dim3 grid, cudaStream_t s) {
+  const int smem = (MC_L * (2 * (k.KS * 16 + 8) + k.NT * 8 + 8) + 2 * MC_L * MC_PITCH) * 2;
+  static bool done[OGB_MAX_DEVICES] = {};
+  return set_max_dyn_smem(mlstm_out_kernel<NTW>, 200 * 1024, done) && launch_pdl(mlstm_out_kernel<NTW>, grid, dim3(256), smem, s, p, k);
+}
+
+static int LaunchMlstmChunks(const MlstmParams& p, const OgbMlstm* a, cudaStream_t s) {
+  MlstmChunk k;
+  long long floats = 0;
+  if (!MlstmChunkSizes(a->T, a->B, a->H, a->d, a->dv, &k, &floats)) return -5;
+  if (floats * 4 > a->scratch_bytes) return -2;
+  auto addr = [](const void* x) { return reinterpret_cast<uintptr_t>(x); };
+  if (((addr(a->q) | addr(a->k) | addr(a->v) | addr(a->scratch)) & 15) || a->ld % 8 || a->ldo % 2 || ((addr(a->g) | addr(a->out)) & 3) || (addr(a->norm_w) & 7)) return -1;
+  k.min_tokens = a->long_tokens;
+  const long long chunks = a->T / MC_L + a->B, HT = (long long)a->H * a->T;
+  k.sums = static_cast<float*>(a->scratch);                 // (16-byte pieces: first)
+  k.nsums = k.sums + chunks * a->H * k.KS * k.NT * 128;
+  k.c = k.nsums + chunks * a->H * k.KS * 16;
+  k.M = k.c + HT; k.floor = k.M + HT;
+  k.m_in = k.floor + HT; k.M_last = k.m_in + chunks * a->H;
+  const int n = (a->max_q_len + MC_L - 1) / MC_L;
+  if (n > 65535 || (long long)a->B * a->H > 65535) return -1;
+  const size_t gsmem = size_t(3) * n * 4;
+  if (gsmem > 48 * 1024) return -5;
+  if (!launch_pdl(mlstm_gates_kernel, dim3(a->H, a->B), dim3(256), gsmem, s, p, k)) return -4;
+  if (!launch_pdl(mlstm_sums_kernel, dim3(((k.NT + 7) / 8) * ((k.KS + 3) / 4), n, a->B * a->H), dim3(128), 0, s, p, k)) return -4;
+  if (!launch_pdl(mlstm_scan_kernel, dim3((k.KS * k.NT * 32 + 255) / 256 + 1, a->H, a->B), dim3(256), 0, s, p, k)) return -4;
+  const dim3 grid(n, a->H, a->B);
+  const bool ok = k.NT <= 16 ? LaunchMlstmOut<4>(p, k, grid, s) : (k.NT <= 32 ? LaunchMlstmOut<8>(p, k, grid, s) : LaunchMlstmOut<16>(p, k, grid, s));
+  return ok ? 0 : -4;
+}
+
 OGB_API int ogb_mlstm(const OgbMlstm* a, void* stream) {
   if (a->B <= 0 || a->H <= 0) return 0;
   if (a->d <= 0 || a->d > ML_MAX_D || a->dv <= 0 || a->B > 65535 || a->H > 65535 || a->cap <= 0.f) return -5;
@@ -331,6 +808,12 @@ OGB_API int ogb_mlstm(const OgbMlstm* a, void* stream) {
   p.ld = a->ld; p.ldg = a->ldg; p.ldo = a->ldo; p.H = a->H; p.d = a->d; p.dv = a->dv; p.cap = a->cap; p.eps = a->eps;
   p.q_scale = 1.f / sqrtf(float(a->d));
   auto s = static_cast<cudaStream_t>(stream);
+  if (a->long_tokens > 0) {
+    if (a->fp32) return -5;
+    const int rc = LaunchMlstmChunks(p, a, s);
+    if (rc != 0 || a->all_long) return rc;
+    p.long_tokens = a->long_tokens;
+  }
   // states in whole 16-byte pieces (a slot's first float is on a 16-byte boundary, heads and rows are multiples of four)
   const bool vec = a->dv % 4 == 0 && a->slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 15) == 0;
   const int unit = vec ? 4 : 1;

@@ -576,7 +576,7 @@ class DecoderModel:
         proj = self._wide_linear(x, lw.mem_in_w)
         gates = ops.linear(x, lw.mem_gate_w, out_fp32=True)
         return ops.mlstm(proj, gates, lw.mem_gate_b, sp.heads, sp.dim, sp.vdim, sp.gate_cap, lw.mem_norm_w, self.arch.norm_eps, kv.state_rows(li), s.state_slots,
-                         s.cu_seqlens, s.past_lens, out, s.max_q_len)
+                         s.cu_seqlens, s.past_lens, out, s.max_q_len, s.min_q_len)
 
     def _stack_mixer(self, lw: LayerWeights, sp):
         return {"linear_attention": self._linear_attention, "latent_attention": self._latent_attention, "attention": self._spec_attention,

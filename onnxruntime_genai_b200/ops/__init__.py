@@ -1092,9 +1092,12 @@ def min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale=1.0, max_q_
     return out
 
 
-def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out, max_q_len=0):
+MLSTM_LONG_TOKENS = 24      # requests that feed at least this many tokens run in the chunk form of the matrix memories
+
+
+def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out, max_q_len=0, min_q_len=0):
     """Matrix memories over packed sequences (see csrc/recurrent.cu): proj [T, queries | keys | values | output gate], gates fp32 [T, input | forget logits],
-    their biases gate_b and the heads' norm weight fp32; state [slots, heads * (dim * vdim + dim + 1)] fp32, updated in place; out [T, heads * vdim]."""
+    their biases gate_b and the heads' norm weight fp32; state [slots, heads * (dim * vdim + dim + 1)] fp32, updated in place; out [T, heads * vdim].  max_q_len, min_q_len: most and fewest tokens a request feeds (0: unknown)."""
     if not proj.is_cuda:
         return ref.mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out)
     import ctypes
@@ -1106,6 +1109,13 @@ def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots,
                    out=_ptr(out), state=_ptr(state), slots=_ptr(slots), cu_seqlens=_ptr(cu_seqlens), past_lens=_ptr(past_lens), slot_stride=state.stride(0),
                    ld=proj.stride(0), ldg=gates.stride(0), ldo=out.stride(0), B=past_lens.shape[0], H=heads, d=dim, dv=vdim, T=proj.shape[0],
                    max_q_len=int(max_q_len or proj.shape[0]), fp32=int(proj.dtype == torch.float32), cap=float(cap), eps=float(eps))
+    scratch = None
+    if p.max_q_len >= MLSTM_LONG_TOKENS and not p.fp32 and p.ld % 8 == 0 and at % 16 == 0 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0:
+        need = _lib.lib().ogb_mlstm_scratch_bytes(p.T, p.B, heads, dim, vdim)
+        if need:
+            scratch = torch.empty(need, dtype=torch.uint8, device=proj.device)
+            p.scratch, p.scratch_bytes, p.long_tokens, p.all_long = _ptr(scratch), need, MLSTM_LONG_TOKENS, int(min_q_len >= MLSTM_LONG_TOKENS)
+            _lib.LAUNCH_COUNT += 3 + (1 - p.all_long)
     _lib.check(_lib.lib().ogb_mlstm(ctypes.byref(p), _stream()), "mlstm")
     return out
 

@@ -44,8 +44,8 @@ class NormStream(ctypes.Structure):
 class Mlstm(ctypes.Structure):
     """OgbMlstm of csrc/kernels.h: matrix memories."""
     _fields_ = ([(n, _P) for n in ("q", "k", "v", "g", "gates", "gate_b", "norm_w", "out", "state", "slots", "cu_seqlens", "past_lens")] +
-                [("slot_stride", c_longlong)] + [(n, c_int) for n in ("ld", "ldg", "ldo", "B", "H", "d", "dv", "T", "max_q_len", "fp32")] +
-                [("cap", c_float), ("eps", c_float)])
+                [("slot_stride", c_longlong)] + [(n, c_int) for n in ("ld", "ldg", "ldo", "B", "H", "d", "dv", "T", "max_q_len", "fp32", "long_tokens", "all_long")] +
+                [("cap", c_float), ("eps", c_float), ("scratch", _P), ("scratch_bytes", c_longlong)])
 
 
 class TanhNorm(ctypes.Structure):
@@ -124,6 +124,7 @@ _SIGS = {
     "ogb_embedding_bigram": (c_int, [ctypes.POINTER(Bigram), _P, _P, _P, _P]),
     "ogb_norm_stream": (c_int, [ctypes.POINTER(NormStream), _P]),
     "ogb_min_gru": (c_int, [_P, _P, _P, c_int, _P, c_longlong, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, c_int, _P]),
+    "ogb_mlstm_scratch_bytes": (c_longlong, [c_int, c_int, c_int, c_int, c_int]),
     "ogb_mlstm": (c_int, [ctypes.POINTER(Mlstm), _P]),
     "ogb_moe_topk_grouped": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_float, _P, _P, _P]),
     "ogb_act_mul_rows": (c_int, [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P]),

@@ -72,6 +72,33 @@ def looped_stack(layers, vocab=90, width=72, eps=3e-5, embed_scale=1.7, buckets=
     return cfg
 
 
+def grouped(ff=40, n=6, top=2, groups=2, keep=1, scale=1.5):
+    """Experts without gates, chosen among the best groups."""
+    return dict(kind="moe", expert=dict(ff=ff), router=dict(experts=n, top=top, groups=dict(count=groups, keep=keep), scale=scale))
+
+
+def plain(ff=80):
+    return dict(kind="dense", ff=ff)
+
+
+def side_by_side(heads=4, kv_heads=2, dim=24, vdim=16, window=20, scale=0.3, dims=16, base=3000.0, factor=5.0, width=40, scales=(0.7, 0.45), mlp=plain()):
+    """Attention with mixed heads beside a gated average of `width` columns."""
+    rot = dict(base=base, dims=dims, **(dict(scaling=dict(factor=factor)) if factor else {})) if dims else None
+    left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, mask=dict(size=window) if window else None, rot=rot)
+    return dict(type="parallel", mixer=dict(left=left, right=dict(width=width), left_scale=scales[0], right_scale=scales[1]), mlp=mlp)
+
+
+def memories(heads=3, dim=16, vdim=24, gate_cap=9.0, mlp=plain()):
+    return dict(type="mlstm", mixer=dict(heads=heads, dim=dim, vdim=vdim, gate_cap=gate_cap), mlp=mlp)
+
+
+def two_norm_stack(layers, vocab=90, width=72, eps=3e-5, embed_scale=1.7, loop=(0, None, 2)):
+    cfg = dict(architecture="Tevilix", layers=copy.deepcopy(layers), norm=dict(eps=eps), vocab=vocab, width=width, embedding=dict(scale=embed_scale))
+    if loop:
+        cfg["loop"] = dict(start=loop[0], stop=len(layers) if loop[1] is None else loop[1], times=loop[2])
+    return cfg
+
+
 def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
     """Random weights of useful magnitude (projections near unit gain, decays between slow and fast).  clear_routes: a router reads one
     column of the stream per expert, these columns hold well separated values in every embedding row, and no sub-layer writes them."""
@@ -94,6 +121,12 @@ def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
             x = 2.0 * x / shape[1] ** 0.5
         elif name.endswith("sink"):
             x = x + 0.5
+        elif name.endswith("talk"):
+            x = torch.eye(shape[0]) + 0.5 * x             # every head's scores show in the others'
+        elif name.endswith("correction"):
+            x = 0.4 * x
+        elif name.endswith(".f.b"):
+            x = 2.0 + 1.5 * x                             # memories of a few and of many tokens
         elif name.endswith(".b") and len(shape) == 1 or name.endswith("dt_bias"):
             x = 0.3 * x
         elif name.endswith("A_log"):
@@ -106,7 +139,21 @@ def weights(cfg, seed=0, dtype=torch.bfloat16, gain=1.0, clear_routes=False):
             x = gain * x / shape[1] ** 0.5
         out[name] = x.to(dtype)
     most = max([e["mlp"]["router"]["experts"] for e in cfg["layers"] if (e.get("mlp") or {}).get("kind") == "moe"], default=0)
-    if clear_routes and most and cfg["architecture"] == "Sugelix":
+    if clear_routes and most and cfg["architecture"] == "Tevilix":
+        assert most < cfg["width"]
+        for v in range(cfg["vocab"]):
+            out["embed"][v, :most] = (torch.randperm(most, generator=g).float() / most * 4 - 2).to(dtype)
+        for name, x in out.items():
+            if name.endswith((".o", ".o.b", ".down")):
+                x[:most] = 0
+            elif name.endswith("norm2"):
+                x[:most] = 1
+            elif name.endswith("router"):
+                x.zero_()[:, :most].fill_diagonal_(4.0)
+            elif name.endswith("correction"):             # groups far apart: their choice is constant
+                r = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]
+                x.copy_((3 * torch.randperm(r["groups"]["count"], generator=g)).repeat_interleave(r["experts"] // r["groups"]["count"]))
+    elif clear_routes and most and cfg["architecture"] == "Sugelix":
         assert most < cfg["width"]
         turns = (cfg.get("loop") or dict(times=1))["times"]
         for v in range(cfg["vocab"]):
