@@ -440,7 +440,7 @@ def main():
     ap.add_argument("--precision", default="bf16", choices=["bf16", "int4"],
                     help="weights of the checkpoint: bf16 (headline) or 4-bit (int4 block-32 linears; gpt-oss experts as packed MXFP4, the form "
                          "the reference publishes its gpt-oss numbers for); activations and the KV cache stay bf16")
-    ap.add_argument("--design", default="", choices=["", "luzatar", "zevopel", "sugelix"],
+    ap.add_argument("--design", default="", choices=["", "luzatar", "zevopel", "sugelix", "tevilix"],
                     help="measure this declared-stack design beside the closest other model at equal size instead of the headline workload")
     ap.add_argument("--design_sizes", default="", help="comma-separated sizes of --design (default: all)")
     args = ap.parse_args()

@@ -10,6 +10,8 @@ cases: gemm_qkv gemm_o gemm_gate_up gemm_down gemm_lm_head gemm_prefill gemm_qkv
        capped_decode capped_prefill softcap_decode softcap_prefill diff_decode diff_prefill qkv_prep_plain tanh_norm tanh_norm_experts
        embed_pairs embed latent_value_gated shared_route (Sugelix layers: soft-capped attention with a gate per column beside the older models' soft
        cap, differential attention with two maps of 64 over values of 128 columns, sums into the stream with their tanh norm; not part of `all`)
+       talk_decode talk_prefill qkv_prep_mixed min_gru min_gru_prefill mlstm mlstm_prefill two_norms two_norms_experts gemm_up_gelu_erf grouped_route
+       (Tevilix layers: mixed heads over 8, or 4 with --tp 2, key heads, gated averages of 4096 columns, 32 memories of 128 x 128; not part of `all`)
        gemm_join (Luzatar layers at Llama-sized widths: 16 heads of 128 + 64 / 128 over a latent of 512; not part of `all`)
        (moe_*: gpt-oss-20b experts, packed MXFP4 in the fp16 form, in the bf16 form (fp4b) or bf16 weights; not part of `all`)
 
@@ -123,7 +125,7 @@ def build_case(name, T, L, tp=1):
         kc, vc = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D)
         return (lambda i: ops.qkv_rope_append(x, ws[i % L], None, pos, slots, cos, sin, kc, vc, HQ, HKV, D, D, norm_eps=1e-5)), \
             N * H * 2 + T * (H + N) * 2, 2.0 * T * N * H
-    if name not in ("gemm_join", "gemm_gate_up_gelu") and name.startswith(("gemm_", "w4_")):
+    if name not in ("gemm_join", "gemm_gate_up_gelu", "gemm_up_gelu_erf") and name.startswith(("gemm_", "w4_")):
         shapes = {"gemm_qkv": ((HQ + 2 * HKV) * D, H), "gemm_o": (H, HQ * D), "gemm_gate_up": (2 * I // tp, H), "gemm_down": (H, I // tp),
                   "gemm_lm_head": (V // tp, H), "gemm_prefill": (2 * I // tp, H), "w4_qkv": (9216 // tp, 3072), "w4_down": (3072, 8192 // tp)}
         N, K = shapes[name]
@@ -277,6 +279,67 @@ def build_case(name, T, L, tp=1):
         return (lambda i: ops.latent_attention(qlat, proj, sh, caches[i % Lk], cu, pl, table, bs, scale, 0, 1, max(p + n for p, n in lens),
                                                splits=ATTN_SPLITS[0] if isinstance(ATTN_SPLITS, tuple) else ATTN_SPLITS, order=order)), \
             kv_tokens * (R + r) * 2 + Tq * Hl * (2 * R + r) * 2, 2.0 * kv_tokens * Hl * (2 * R + r)
+    if name in ("talk_decode", "talk_prefill"):
+        # a query meets the keys of all key heads; window 8192
+        bs, decode = 16, name == "talk_decode"
+        rng = np.random.RandomState(2)
+        B = T if decode else max(1, T // 1024 if T > 4096 else 1)
+        lens = [(int(p) + 64, 1) for p in rng.randint(128, 2049, size=B)] if decode else [(0, T // B)] * B
+        nb = [(p + n + bs - 1) // bs for p, n in lens]
+        table = torch.zeros(B, max(nb), dtype=torch.int32)
+        for b, k in enumerate(nb):
+            table[b, :k] = torch.arange(sum(nb[:b]), sum(nb[:b]) + k, dtype=torch.int32)
+        table, Lk = table.cuda(), min(L, 4)
+        kc, vc = ([_bf(sum(nb) * bs, HKV, D, std=1.0) for _ in range(Lk)] for _ in range(2))
+        Tq = sum(n for _, n in lens)
+        q, gate = _bf(Tq, HQ * HKV * D, std=0.3), _bf(Tq, HQ * D, std=1.0)
+        cu = torch.tensor(np.concatenate([[0], np.cumsum([n for _, n in lens])]), dtype=torch.int32).cuda()
+        pl = torch.tensor([p for p, _ in lens], dtype=torch.int32).cuda()
+        order = torch.argsort(-pl.long(), stable=True).to(torch.int32) if ATTN_ORDER else None
+        pairs = sum(n * p + n * (n + 1) / 2 for p, n in lens)
+        return (lambda i: ops.paged_attention(q, kc[i % Lk], vc[i % Lk], cu, pl, table, bs, HQ, HKV, HKV * D, 1 / math.sqrt(D), 8192, max_q_len=lens[0][1],
+                                              max_kv_len=max(p + n for p, n in lens), splits=ATTN_SPLITS, order=order, min_q_len=lens[0][1], vdim=D, gate=gate, joint=True)), \
+            sum(p + n for p, n in lens) * HKV * D * 4 + Tq * HQ * (HKV + 2) * D * 2, 2.0 * HQ * (HKV + 1) * D * pairs
+    if name == "qkv_prep_mixed":
+        projs = [_bf(T, (2 * HQ + 2 * HKV) * D, std=1.0) for _ in range(4)]
+        pos, slots = torch.arange(T, dtype=torch.int32, device="cuda") % 4096, torch.arange(T, dtype=torch.int32, device="cuda")
+        cos, sin, w, talk = torch.randn(4096, D // 2, device="cuda"), torch.randn(4096, D // 2, device="cuda"), torch.ones(D, device="cuda"), torch.randn(HQ, HQ, device="cuda")
+        kc, vc, out = _bf(T + 16, HKV, D), _bf(T + 16, HKV, D), torch.empty(T, HQ * HKV * D, dtype=torch.bfloat16, device="cuda")
+        return (lambda i: ops.qkv_prep(projs[i % 4], HQ, HKV, D, D, D, w, w, 1e-6, pos, cos, sin, slots, kc, vc, talk=talk, mixed=out)), \
+            T * (HQ + 4 * HKV + HQ * HKV) * D * 2, 0.0
+    if name in ("min_gru", "min_gru_prefill"):
+        B = T if name == "min_gru" else max(1, T // 1024 if T > 4096 else 1)
+        projs = [_bf(T, 3 * H, std=1.0) for _ in range(4)]
+        state, out = torch.zeros(B, H, device="cuda"), torch.empty(T, H, dtype=torch.bfloat16, device="cuda")
+        slots, past = torch.arange(B, dtype=torch.int32, device="cuda"), torch.full((B,), 7, dtype=torch.int32, device="cuda")
+        cu = torch.arange(0, T + 1, T // B, dtype=torch.int32, device="cuda")
+        return (lambda i: ops.min_gru(projs[i % 4][:, :H], projs[i % 4][:, H:2 * H], projs[i % 4][:, 2 * H:], state, slots, cu, past, out, 0.5, T // B)), \
+            T * H * 8 + B * H * 8, 0.0
+    if name in ("mlstm", "mlstm_prefill"):
+        Hm, d, dv = 32, 128, 128
+        B = T if name == "mlstm" else max(1, T // 1024 if T > 4096 else 1)
+        projs = [_bf(T, 2 * Hm * (d + dv), std=1.0) for _ in range(4)]
+        gates, gb, nw = torch.randn(T, 2 * Hm, device="cuda"), torch.ones(2 * Hm, device="cuda"), torch.ones(Hm * dv, device="cuda")
+        elems = Hm * (d * dv + d + 1)
+        pools = [torch.randn(B, elems, device="cuda") * 0.1 for _ in range(2 if B > 1 else 8)]
+        out = torch.empty(T, Hm * dv, dtype=torch.bfloat16, device="cuda")
+        slots, past = torch.arange(B, dtype=torch.int32, device="cuda"), torch.full((B,), 7, dtype=torch.int32, device="cuda")
+        cu = torch.arange(0, T + 1, T // B, dtype=torch.int32, device="cuda")
+        return (lambda i: ops.mlstm(projs[i % 4], gates, gb, Hm, d, dv, 15.0, nw, 1e-6, pools[i % len(pools)], slots, cu, past, out, T // B, T // B)), \
+            B * elems * 8 + T * Hm * (2 * d + 3 * dv) * 2, T * Hm * 4.0 * d * dv
+    if name in ("two_norms", "two_norms_experts"):
+        hs, w = [torch.randn(T, H, device="cuda") for _ in range(4)], torch.randn(H, device="cuda")
+        if name == "two_norms":
+            return (lambda i: ops.norm_stream(hs[i % 4], w, 1e-6, None, True, weight2=w)), T * H * 8, 0.0
+        plan = ops.moe_route(torch.randn(T, 32, device="cuda"), 4, 1)
+        y = ops.PendingCombine(_bf(T * 4, H, std=1.0), plan)
+        return (lambda i: ops.norm_stream(hs[i % 4], w, 1e-6, None, True, add=y, weight2=w)), T * H * 20, 0.0
+    if name == "gemm_up_gelu_erf":
+        x, ws = _bf(T, H, std=1.0), [_bf(I, H) for _ in range(L)]
+        return (lambda i: ops.linear_act(x, ws[i % L], "gelu_erf")), I * H * 2 + T * (H + I) * 2, 2.0 * T * I * H
+    if name == "grouped_route":
+        logits, corr = torch.randn(T, 64, device="cuda"), torch.randn(64, device="cuda")
+        return (lambda i: ops.moe_route(logits, 6, 3, correction=corr, groups=8, keep=4)), T * 64 * 4 + T * 6 * 16, 0.0
     if name == "norm_stream":
         xs, w, b = [torch.randn(T, H, device="cuda") for _ in range(8)], torch.randn(H, device="cuda"), torch.randn(H, device="cuda")
         return (lambda i: ops.norm_stream(xs[i % 8], w, 1e-5, b, True)), T * H * 6, 0.0
@@ -411,7 +474,7 @@ def main():
     out = {}
     for name in (ALL if a.case == "all" else [a.case]):
         T = max(a.tokens, 2048) if name in ("gemm_prefill", "attention_prefill", "latent_prefill", "latent_expand", "gated_delta_prefill",
-                                         "chunk_prefill", "chunk_prefill_192", "capped_prefill", "softcap_prefill", "diff_prefill") else a.tokens
+                                         "chunk_prefill", "chunk_prefill_192", "capped_prefill", "softcap_prefill", "diff_prefill", "talk_prefill", "mlstm_prefill", "min_gru_prefill") else a.tokens
         fn, nbytes, flops = build_case(name, T, a.layers, a.tp)
         iters = a.iters if name not in ("gemm_lm_head", "sample", "argmax") else min(a.iters, 4)
         us = _time_eager(fn, iters) if a.eager else _time_graph(fn, iters)

@@ -3,9 +3,11 @@ gated-delta-net + full-attention hybrid (Qwen3.5 style) with the same width, fee
 Zevopel: Qwen3-style dense layers (normed query and key heads), and gpt-oss-style layers with bf16 experts (sinks, clamped experts), each
 with the same width, heads and feed-forwards; the chunks are as long as the context, so both attend to the same keys.  Sugelix: gpt-oss-style
 layers again, as many as the design runs, with the same width, head count, key and value sizes and as many experts per token (one of the
-design's is the shared one); soft-capped scores on both sides where the design's layers have them.  Random weights drawn
+design's is the shared one); soft-capped scores on both sides where the design's layers have them.  Tevilix: the Qwen3.5-style hybrid again, its
+delta layers in the places of the matrix memories (as many states of the same size), its attention in those of the pairs of attention and gated
+average, with the same heads and the same feed-forward (dense, or as many experts of the same width); windows as long as the context.  Random weights drawn
 on the device; CUDA events around whole decoder forwards (decode steps replay a CUDA graph); the weights and caches of a step are larger
-than L2.  Reached through `python bench.py --design luzatar | zevopel | sugelix`."""
+than L2.  Reached through `python bench.py --design luzatar | zevopel | sugelix | tevilix`."""
 import json
 import os
 import shutil
@@ -33,6 +35,13 @@ SUGELIX_SIZES = {
     "2.9k latent": dict(mixers="llllllll", times=1, width=2880, ff=2880, heads=32, kv=8, dim=128, vocab=65536, experts=32, top=4),
     "2k mixed, twice": dict(mixers="adal", times=2, width=2048, ff=1024, heads=16, kv=4, dim=128, vocab=65536, experts=64, top=6, softcap=50.0),
 }
+TEVILIX_SIZES = {
+    # name: width, feed-forward (of one expert where there are experts), layers (alternating memories / attention beside a gated average), attention heads,
+    # kv heads, head size, columns of the gated average, heads of the memories (128 x 128 each; dk, dv: the hybrid's key and value heads)
+    "2k dense": dict(width=2048, ff=6144, layers=16, heads=16, kv=4, dim=128, gru=1024, dk=8, dv=16, vocab=65536),
+    "4k dense": dict(width=4096, ff=12288, layers=8, heads=32, kv=4, dim=128, gru=2048, dk=16, dv=32, vocab=65536),
+    "2k experts": dict(width=2048, ff=1024, layers=16, heads=16, kv=2, dim=128, gru=1024, dk=8, dv=16, vocab=65536, experts=64, top=6, groups=8, keep=4),
+}
 PREFILL = [(1, 4096), (8, 1024)]
 DECODE = [(1, 2048), (16, 2048), (64, 2048), (256, 1024)]
 BLOCK = 16
@@ -50,6 +59,22 @@ def luzatar_dir(z, path):
     return create_model(os.path.join(path, "src"), os.path.join(path, "model"), "bf16", "cuda", {"synthetic_weights": 1, "context_length": 8192})
 
 
+def tevilix_dir(z, path):
+    mlp = dict(kind="dense", ff=z["ff"])
+    if z.get("experts"):
+        mlp = dict(kind="moe", expert=dict(ff=z["ff"]), router=dict(experts=z["experts"], top=z["top"], groups=dict(count=z["groups"], keep=z["keep"]), scale=1.0))
+    d = z["dim"]
+    pair = dict(left=dict(heads=z["heads"], kv_heads=z["kv"], dim=d, vdim=d, scale=d ** -0.5, mask=dict(size=8192),
+                          rot=dict(base=5e5, dims=d, scaling=dict(factor=4.0))), right=dict(width=z["gru"]), left_scale=0.7, right_scale=0.5)
+    layers = [dict(type="mlstm", mixer=dict(heads=z["dv"], dim=128, vdim=128, gate_cap=15.0), mlp=mlp), dict(type="parallel", mixer=pair, mlp=mlp)] * (z["layers"] // 2)
+    cfg = dict(architecture="Tevilix", layers=layers, norm=dict(eps=1e-6), vocab=z["vocab"], width=z["width"], embedding=dict(scale=1.0))
+    os.makedirs(os.path.join(path, "src"), exist_ok=True)
+    with open(os.path.join(path, "src", "config.json"), "w") as f:
+        json.dump(cfg, f)
+    from onnxruntime_genai_b200.models.builder import create_model
+    return create_model(os.path.join(path, "src"), os.path.join(path, "model"), "bf16", "cuda", {"synthetic_weights": 1, "context_length": 8192})
+
+
 def hybrid_dir(z, path):
     from onnxruntime_genai_b200.models.arch import ArchConfig
     from onnxruntime_genai_b200.models.builder import export_model
@@ -57,6 +82,8 @@ def hybrid_dir(z, path):
                    num_kv_heads=z["kv"], head_dim=128, intermediate_size=z["ff"], context_length=8192, bos_token_id=0, eos_token_id=1, pad_token_id=0,
                    layer_types=["linear_attention", "full_attention"] * (z["layers"] // 2), linear_num_key_heads=z["dk"], linear_num_value_heads=z["dv"],
                    linear_key_head_dim=128, linear_value_head_dim=128, linear_conv_kernel_dim=4)
+    if z.get("experts"):
+        a.moe_style, a.num_experts, a.experts_per_token = "standard", z["experts"], z["top"]
     return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
 
 
@@ -118,7 +145,7 @@ def closest_to_sugelix_dir(z, path):
     return export_model(a, path, precision="bf16", execution_provider="cuda", paged=True, block_size=BLOCK, synthetic_weights=True)
 
 
-DESIGNS = {"sugelix": (SUGELIX_SIZES, sugelix_dir, "closest", closest_to_sugelix_dir), "luzatar": (SIZES, luzatar_dir, "hybrid", hybrid_dir), "zevopel": (ZEVOPEL_SIZES, zevopel_dir, "closest", closest_to_zevopel_dir)}
+DESIGNS = {"tevilix": (TEVILIX_SIZES, tevilix_dir, "hybrid", hybrid_dir), "sugelix": (SUGELIX_SIZES, sugelix_dir, "closest", closest_to_sugelix_dir), "luzatar": (SIZES, luzatar_dir, "hybrid", hybrid_dir), "zevopel": (ZEVOPEL_SIZES, zevopel_dir, "closest", closest_to_zevopel_dir)}
 
 
 def _step(model, lens):

@@ -32,7 +32,7 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
                                 int total_tokens, int max_q_len, int splits, int kv_chunk, void* scratch, long long scratch_bytes, const int32_t* order,
                                 int* status, void* stream_, int skip_rows) {
   if (B <= 0 || total_tokens <= 0 || max_q_len <= 0) return 0;
-  if (!ogb_attention_mixed_supported(a->dk, a->dv)) return -5;
+  if (a->joint || !ogb_attention_mixed_supported(a->dk, a->dv)) return -5;
   if (a->Hkv <= 0 || a->Hq % a->Hkv || (q_stride % 8) || (out_stride % 2) || block_size <= 0 || a->Hkv > 65535) return -1;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) return -1;
   if (reinterpret_cast<uintptr_t>(out) & 3) return -1;
@@ -54,10 +54,9 @@ OGB_API int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stri
   p.status = status; p.order = order; p.skip_rows = skip_rows;
   p.dk = a->dk; p.dv = a->dv;
   p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.gate_stride = a->gate_stride; p.gate_wide = a->gate && a->gate_wide;
-  p.maps = maps; p.raw = a->raw; p.joint = a->joint; p.out_scale = a->out_scale;
+  p.maps = maps; p.raw = a->raw; p.out_scale = a->out_scale;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
-  if (a->joint && maps > 1) return -1;
-  if (!a->joint && a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
+  if (a->dk == a->dv && (a->dk == 64 || a->dk == 96 || a->dk == 128)) return LaunchAttentionUniform(p, a->dk, max_q_len, stream);
   if (a->dk <= 64) return LaunchMixedKeys<64>(p, max_q_len, stream);
   if (a->dk <= 128) return LaunchMixedKeys<128>(p, max_q_len, stream);
   if (a->dk <= 192) return LaunchMixedKeys<192>(p, max_q_len, stream);

@@ -69,8 +69,6 @@ struct AttnParams {
   // maps > 1: query vector h (dk / maps columns wide) belongs to map h % maps of its key head, whose row holds the maps' keys side by side: the
   // query is staged at its map's columns among zeros, so keys and values are read once for all maps.
   int maps;
-  // joint: a cache row holds the keys of all key heads side by side as one key of dk columns, which every query head meets; values by key head
-  int joint;
   float out_scale;   // multiplies the result (not of raw calls)
   int raw;           // partial results are written even without splits, and not merged here
 };
@@ -209,7 +207,7 @@ paged_attention_kernel(AttnParams p) {
         const int kl = item / CHUNKS, ch = item % CHUNKS;
         const int sl = __shfl_sync(0xffffffffu, slot, kl);
         const bool ok = sl >= 0 && ch * 8 < dk;
-        cp_async16(tk + koff(warp * 16 + kl, ch), p.k_cache + (ok ? (p.joint ? size_t(sl) : size_t(sl) * p.Hkv + kvh) * dk + ch * 8 : 0), ok);
+        cp_async16(tk + koff(warp * 16 + kl, ch), p.k_cache + (ok ? (size_t(sl) * p.Hkv + kvh) * dk + ch * 8 : 0), ok);
       }
 #pragma unroll
       for (int c = 0; c < CHUNKS_V / 2; ++c) {

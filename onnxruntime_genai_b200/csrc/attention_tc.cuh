@@ -88,18 +88,21 @@ struct TcAttnParams {
 // entry of a query row in a grid of key vectors
 __device__ __forceinline__ int tca_query(int kvh, int i, int G, int maps) { return maps > 1 ? ((kvh / maps) * G + i) * maps + kvh % maps : kvh * G + i; }
 
-template <int DK, int DV, int BN>
+// KC: key columns of a ring slot (DK, or a part of it where whole tiles of wide keys would not fit twice beside the queries).
+template <int DK, int DV, int BN, int KC = DK>
 struct TcaCfg {
-  static constexpr int K_HALVES = DK / 64, V_HALVES = DV / 64;
+  static constexpr int K_PARTS = DK / KC, K_HALVES = KC / 64, V_HALVES = DV / 64;
+  static_assert(DK % KC == 0, "a key row is whole parts");
   static constexpr int Q_BYTES = TCA_BM * DK * 2;
-  static constexpr int K_TILE = BN * DK * 2, V_TILE = BN * DV * 2;
+  static constexpr int K_TILE = BN * KC * 2, V_TILE = BN * DV * 2;
   // K and V tiles have rings of their own: a K tile is free as soon as its Q K^T is done (one tile period earlier than the
   // V tile of the same keys), and the loads must run two to three tile periods ahead of their use to hide their latency.
   static constexpr int BUDGET = 227 * 1024 - 1024 - 1536 - Q_BYTES;      // 1 KiB of alignment slack, static shared memory
-  static constexpr int PAIRS = BUDGET / (K_TILE + V_TILE) >= 4 ? 4 : BUDGET / (K_TILE + V_TILE);
+  static constexpr int PAIRS = K_PARTS > 1 ? 2 : (BUDGET / (K_TILE + V_TILE) >= 4 ? 4 : BUDGET / (K_TILE + V_TILE));
   static constexpr int V_STAGES = PAIRS;
-  static constexpr int K_STAGES = PAIRS < 4 && BUDGET - PAIRS * (K_TILE + V_TILE) >= K_TILE ? PAIRS + 1 : PAIRS;
-  static_assert(PAIRS >= 2, "the rings need two stages each");
+  static constexpr int K_STAGES = K_PARTS > 1 ? (BUDGET - 2 * V_TILE) / K_TILE
+                                              : (PAIRS < 4 && BUDGET - PAIRS * (K_TILE + V_TILE) >= K_TILE ? PAIRS + 1 : PAIRS);
+  static_assert(PAIRS >= 2 && K_STAGES >= 2, "the rings need two stages each");
   static constexpr int SMEM = 1024 + Q_BYTES + K_STAGES * K_TILE + V_STAGES * V_TILE;
   static constexpr int S_BUFS = 3;
   static constexpr int S_COLS = BN, O_COL = S_BUFS * BN;
@@ -144,11 +147,12 @@ __device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.p
 // are the unrotated part; MIX: heads of p.dk and p.dv columns (multiples of 8).  The boxes of a head narrower than the staged rows reach
 // into the next head's columns, which meet zeros in Q (keys) or give output columns that are not stored (values).  CAP: scores are soft-capped
 // (a kernel of its own: the loop body of the others has to stay within the instruction cache).
-template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false, bool CAP = false>
-__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN>::CTAS_PER_SM)
+template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false, bool CAP = false, int KC = DK>
+__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN, KC>::CTAS_PER_SM)
 attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_r,
                     TcAttnParams p) {
-  using Cfg = TcaCfg<DK, DV, BN>;
+  using Cfg = TcaCfg<DK, DV, BN, KC>;
+  static_assert(KC == DK || (MIX && !LAT), "keys in parts: only layers with sizes of their own");
   constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ __align__(128) uint8_t smem_dyn[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~uintptr_t(1023));
@@ -225,9 +229,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     if (lane == 0) tma_prefetch_desc(tmap);
     const int last_group = max(0, (kv_hi - 1) / 16 * 16);
     int issued = 0;
-    for (int it = 0; it < n_tiles; ++it) {
-      const int st = it % NS;
-      if (it >= NS && !mbar_wait_bounded(&empty[st], ((it / NS) - 1) & 1, abort_p)) { if (lane == 0) fail(OGB_ERR_WAIT_TMA); break; }
+    const int parts = is_k ? Cfg::K_PARTS : 1;             // slots per tile
+    for (int n = 0; n < n_tiles * parts; ++n) {
+      const int st = n % NS, it = Cfg::K_PARTS > 1 ? n / parts : n, part = Cfg::K_PARTS > 1 ? n - it * parts : 0;
+      if (n >= NS && !mbar_wait_bounded(&empty[st], ((n / NS) - 1) & 1, abort_p)) { if (lane == 0) fail(OGB_ERR_WAIT_TMA); break; }
       if (lane == 0) mbar_expect_tx(&full[st], tile_bytes);
       __syncwarp();
       // Key groups past the end of the range re-read the last valid group (their scores are masked), so every stage
@@ -252,7 +257,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           if constexpr (MIX) {
             if (is_k) {
 #pragma unroll
-              for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], (p.joint ? 0 : kvh * p.dk) + h * 64, slot0);
+              for (int h = 0; h < Cfg::K_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], (p.joint ? 0 : kvh * p.dk) + part * KC + h * 64, slot0);
             } else {
 #pragma unroll
               for (int h = 0; h < Cfg::V_HALVES; ++h) tma_load_2d(dst + h * (BN * 128), tmap, &full[st], kvh / p.maps * p.dv + h * 64, slot0);
@@ -263,7 +268,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           }
         }
       }
-      issued = it + 1;
+      issued = n + 1;
     }
     if (*abort_p) {
       // copies in flight must land before the shared memory goes away
@@ -281,21 +286,24 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     bool ok = mbar_wait_bounded(&q_full, 0, abort_p);
     if (!ok && lane == 0) fail(OGB_ERR_WAIT_MMA);
     auto issue_qk = [&](int it) -> bool {
-      const int st = it % KS;
-      if (!mbar_wait_bounded(&k_full[st], (it / KS) & 1, abort_p)) return false;
-      tc_fence_after();
-      if (lane == 0) {
-        const uint32_t k_addr = k_ring + st * Cfg::K_TILE;
+#pragma unroll 1
+      for (int part = 0; part < Cfg::K_PARTS; ++part) {
+        const int n = it * Cfg::K_PARTS + part, st = n % KS;
+        if (!mbar_wait_bounded(&k_full[st], (n / KS) & 1, abort_p)) return false;
+        tc_fence_after();
+        if (lane == 0) {
+          const uint32_t k_addr = k_ring + st * Cfg::K_TILE, q_part = q_addr + part * (KC / 64) * (TCA_BM * 128);
 #pragma unroll
-        for (int ks = 0; ks < DK / 16; ++ks) {
-          const uint64_t da = umma_desc_sw128(q_addr + (ks >> 2) * (TCA_BM * 128) + (ks & 3) * 32);
-          const uint64_t db = umma_desc_sw128(k_addr + (ks >> 2) * (BN * 128) + (ks & 3) * 32);
-          umma_f16(tmem_base + (it % Cfg::S_BUFS) * Cfg::S_COLS, da, db, idesc_qk, ks > 0);
+          for (int ks = 0; ks < KC / 16; ++ks) {
+            const uint64_t da = umma_desc_sw128(q_part + (ks >> 2) * (TCA_BM * 128) + (ks & 3) * 32);
+            const uint64_t db = umma_desc_sw128(k_addr + (ks >> 2) * (BN * 128) + (ks & 3) * 32);
+            umma_f16(tmem_base + (it % Cfg::S_BUFS) * Cfg::S_COLS, da, db, idesc_qk, part > 0 || ks > 0);
+          }
+          if (part == Cfg::K_PARTS - 1) umma_commit(&s_full[it % Cfg::S_BUFS]);
+          umma_commit(&k_empty[st]);
         }
-        umma_commit(&s_full[it % Cfg::S_BUFS]);
-        umma_commit(&k_empty[st]);
+        __syncwarp();
       }
-      __syncwarp();
       return true;
     };
     // Q K^T runs three tiles ahead (three S buffers; P_j replaces S_j in place and the buffer is free again after P_j V_j,
@@ -563,10 +571,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   if (warp == TCA_K_WARP) tmem_dealloc(tmem_base, Cfg::TMEM_COLS);
 }
 
-template <int DK, int DV, int BN, bool MIX, bool CAP>
+template <int DK, int DV, int BN, bool MIX, bool CAP, int KC = DK>
 static int LaunchTcForm(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
-  using Cfg = TcaCfg<DK, DV, BN>;
-  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP>;
+  using Cfg = TcaCfg<DK, DV, BN, KC>;
+  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP, KC>;
   const int kw = MIX && p.joint ? p.dk : p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;

@@ -1,5 +1,6 @@
 // Prefill attention on the tensor cores (attention_tc.cuh) for layers whose heads have sizes of their own: queries and keys of dk columns
-// staged as 64, 128, 192 or 256, values of dv columns staged as 64, 128 or 256.
+// staged as 64, 128, 192 or 256, values of dv columns staged as 64, 128 or 256.  Joint layers (a query meets the keys of all key heads) also with keys of up to 512
+// columns, which arrive in parts of 128.
 #include "attention_tc.cuh"
 
 namespace ogb {
@@ -19,9 +20,25 @@ static int LaunchTcMixedKeys(const TcAttnParams& p, const void* k, const void* v
   return LaunchTcMixed<DK, 256>(p, k, v, max_q_len, cache_slots, s);
 }
 
+template <int DK, int DV>
+static int LaunchTcWide(const TcAttnParams& p, const void* k, const void* v, int max_q_len, int cache_slots, cudaStream_t s) {
+  return p.softcap > 0.f ? LaunchTcForm<DK, DV, 64, true, true, 128>(p, k, v, max_q_len, cache_slots, s)
+                         : LaunchTcForm<DK, DV, 64, true, false, 128>(p, k, v, max_q_len, cache_slots, s);
+}
+template <int DK>
+static int LaunchTcWideKeys(const TcAttnParams& p, const void* k, const void* v, int max_q_len, int cache_slots, cudaStream_t s) {
+  if (p.dv <= 64) return LaunchTcWide<DK, 64>(p, k, v, max_q_len, cache_slots, s);
+  if (p.dv <= 128) return LaunchTcWide<DK, 128>(p, k, v, max_q_len, cache_slots, s);
+  return LaunchTcWide<DK, 256>(p, k, v, max_q_len, cache_slots, s);
+}
+
 }  // namespace ogb
 
 using namespace ogb;
+
+OGB_API int ogb_attention_tc_joint_supported(int dk, int dv, int block_size, int cache_slots) {
+  return dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && dk <= 512 && dv <= 256 && block_size % 16 == 0 && cache_slots >= 16;
+}
 
 OGB_API int ogb_attention_tc_mixed_supported(int dk, int dv, int block_size, int cache_slots) {
   return dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && dv <= 256 && block_size % 16 == 0 && cache_slots >= 16;
@@ -33,7 +50,7 @@ OGB_API int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_s
                                    int max_q_len, int min_rows, int cache_slots, int splits, int total_tokens, void* scratch,
                                    long long scratch_bytes, int* status, void* stream_) {
   if (B <= 0 || max_q_len <= 0) return 0;
-  if (!ogb_attention_tc_mixed_supported(a->dk, a->dv, block_size, cache_slots)) return -5;
+  if (!(a->joint ? ogb_attention_tc_joint_supported(a->dk, a->dv, block_size, cache_slots) : ogb_attention_tc_mixed_supported(a->dk, a->dv, block_size, cache_slots))) return -5;
   const int maps = a->maps > 1 ? a->maps : 1;
   if (splits < 1) splits = 1;
   if (a->dk % (8 * maps) || a->Hkv * maps > 65535 || (a->Hq / a->Hkv) % maps || (a->raw && (a->sinks || !scratch))) return -1;
@@ -62,5 +79,7 @@ OGB_API int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_s
   if (p.dk <= 64) return LaunchTcMixedKeys<64>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 128) return LaunchTcMixedKeys<128>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 192) return LaunchTcMixedKeys<192>(p, k_cache, v_cache, max_q_len, cache_slots, s);
-  return LaunchTcMixedKeys<256>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  if (p.dk <= 256) return LaunchTcMixedKeys<256>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  if (p.dk <= 384) return LaunchTcWideKeys<384>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  return LaunchTcWideKeys<512>(p, k_cache, v_cache, max_q_len, cache_slots, s);
 }

@@ -149,10 +149,34 @@ __device__ __forceinline__ float act_one(int kind, float x) {
   x = fmaxf(x, 0.f);
   return kind == 5 ? x * x : x;
 }
-// (out of line: fetched cold by the epilogues)
-static __device__ __noinline__ void epi_act8(int kind, float (&v)[8]) {
+// The tensor-core kernels' form, for results that are rounded to 16 bits.  GELU(erf): erf by formula 7.1.26 of Abramowitz and Stegun, Handbook of
+// Mathematical Functions (absolute error below 1.5e-7): 1 - (a1 t + .. + a5 t^5) e^(-y^2), t = 1 / (1 + 0.3275911 y), y >= 0.
+__device__ __forceinline__ float gelu_erf_fast(float x) {
+  const float y = fabsf(x) * 0.7071067811865476f, t = __fdividef(1.f, fmaf(0.3275911f, y, 1.f));
+  float r = fmaf(t, 1.061405429f, -1.453152027f);
+  r = fmaf(t, r, 1.421413741f);
+  r = fmaf(t, r, -0.284496736f);
+  r = fmaf(t, r, 0.254829592f);
+  const float tail = 0.5f * t * r * __expf(-y * y);       // (1 - erf) / 2
+  return x * (x > 0.f ? 1.f - tail : tail);
+}
+__device__ __forceinline__ void epi_act8(int kind, float (&v)[8]) {
+  if (kind == 4) {
 #pragma unroll
-  for (int j = 0; j < 8; ++j) v[j] = act_one(kind, v[j]);
+    for (int j = 0; j < 8; ++j) v[j] = gelu_erf_fast(v[j]);
+  } else if (kind == 5) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { const float r = fmaxf(v[j], 0.f); v[j] = r * r; }
+  } else if (kind == 3) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = fmaxf(v[j], 0.f);
+  } else if (kind == 2) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = gelu_tanh(v[j]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = silu(v[j]);
+  }
 }
 
 __device__ __forceinline__ uint32_t cluster_ctarank() { uint32_t r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }

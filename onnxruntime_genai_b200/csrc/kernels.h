@@ -123,9 +123,11 @@ int ogb_causal_conv_rows(const void* x, int ldx, const void* w, const void* bias
 
 // ---- recurrent.cu: recurrent mixers over packed sequences (states fp32, at state + slot * slot_stride; a request without a past starts from zero)
 // Gated average per column: S <- (1 - sigmoid(z)) S + sigmoid(z) * c(x), c(x) = x + 1/2 for x >= 0, sigmoid(x) below; out = S * silu(g) * scale.
-// z, x, g: columns of rows of ld elements, W each.
+// z, x, g: columns of rows of ld elements, W each.  scratch (may be null) of ogb_min_gru_scratch_bytes: requests of many tokens, T in the step.
 int ogb_min_gru(const void* z, const void* x, const void* g, int ld, float* state, long long slot_stride, const int32_t* slots, const int32_t* cu_seqlens,
-                const int32_t* past_lens, void* out, int ldo, int B, int W, float scale, int max_q_len, int fp32, void* stream);
+                const int32_t* past_lens, void* out, int ldo, int T, int B, int W, float scale, int max_q_len, void* scratch, long long scratch_bytes, int fp32,
+                void* stream);
+long long ogb_min_gru_scratch_bytes(int T, int B, int W);
 // Matrix memories of H heads with keys of d and values of dv columns.  q, k, v, g: columns of rows of ld elements ([H, d], [H, d], [H, dv], [H, dv]); gates:
 // fp32 rows of ldg, H logits of the input gates and H of the forget gates, to which gate_b [2 H] is added; out rows of ldo.  State of a slot: memories
 // [H, d, dv], normalisers [H, d], maxima [H].  max_q_len: the most tokens a request of the step feeds, T the step's tokens.  long_tokens > 0 (bf16):
@@ -184,7 +186,15 @@ int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stride, cons
                         const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
                         int total_tokens, int max_q_len, int splits, int kv_chunk, void* scratch, long long scratch_bytes, const int32_t* order,
                         int* status, void* stream, int skip_rows);
+// attention_joint.cu: joint layers, decode steps and short portions
+int ogb_attention_joint_supported(int dk, int v_cols);
+int ogb_attention_joint_form(int Hq, int dk, int v_cols);
+int ogb_attention_joint(const OgbAttnLayer* l, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
+                        const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
+                        int total_tokens, int max_q_len, int splits, void* scratch, long long scratch_bytes, const int32_t* order, int* status,
+                        void* stream, int skip_rows);
 int ogb_attention_tc_mixed_supported(int dk, int dv, int block_size, int cache_slots);
+int ogb_attention_tc_joint_supported(int dk, int dv, int block_size, int cache_slots);
 int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
                            const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
                            int max_q_len, int min_rows, int cache_slots, int splits, int total_tokens, void* scratch, long long scratch_bytes,

@@ -570,6 +570,97 @@ __global__ void __launch_bounds__(256) qkv_prep_mixed_kernel(const T* __restrict
   }
 }
 
+// The same where every part is whole pieces of 8 columns (dim = key_row, rot / 2, value_row) and a head at most 32 pieces: LPH lanes per head (a power of two),
+// one piece each, norms and the partners of a rotation by shuffles; then a thread mixes a piece of a key head's queries into four heads at a time.
+template <typename T> __device__ __forceinline__ void store8(T* dst, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    reinterpret_cast<float4*>(dst)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(dst)[1] = make_float4(v[4], v[5], v[6], v[7]);
+  } else {
+    *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_prep_mixed_pieces_kernel(const T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p,
+                                                                    const float* __restrict__ talk, T* __restrict__ mixed, int LPH) {
+  extern __shared__ __align__(16) float sm[];
+  float* sq = sm;                            // [Hq][dim]
+  float* st = sm + p.Hq * p.dim;             // [Hq][Hq]
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < p.Hq * p.Hq; i += blockDim.x) st[i] = talk[i];
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, dim = p.dim, half = p.rot >> 1, turn = half / 8;
+  const T* row = proj + size_t(t) * p.ldp;
+  const int slot = p.slots[t], heads = p.Hq + p.Hkv;
+  const size_t at = size_t(min(max(p.positions[t], 0), p.max_pos - 1)) * half;
+  const int l = tid % LPH, per = blockDim.x / LPH;
+  for (int h0 = 0; h0 < heads; h0 += per) {
+    const int head = h0 + tid / LPH;
+    const bool is_q = head < p.Hq, live = head < heads && l * 8 < dim;
+    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (live) load8(row + size_t(head) * dim + l * 8, f);
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    if (p.q_norm || p.k_norm) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(f[e], f[e], ss);
+      for (int o = LPH >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (w && live) {
+        const float inv = 1.f / sqrtf(ss / dim + p.eps);
+        float g[8];
+        load8(w + l * 8, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = f[e] * inv * g[e];
+      }
+    }
+    if (turn > 0) {
+      // lanes [0, turn) hold the first halves, [turn, 2 turn) the second ones
+      const bool first = l < turn, turns = l < 2 * turn;
+      const int lane = tid & 31, from = turns ? (first ? lane + turn : lane - turn) : lane;
+      float cs[8], sn[8], o[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = __shfl_sync(0xffffffffu, f[e], from);
+      if (turns) {
+        load8(p.cos + at + (first ? l : l - turn) * 8, cs);
+        load8(p.sin + at + (first ? l : l - turn) * 8, sn);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = first ? f[e] * cs[e] - o[e] * sn[e] : f[e] * cs[e] + o[e] * sn[e];
+      }
+    }
+    if (live) {
+      if (is_q) store8(sq + head * dim + l * 8, f);
+      else if (slot >= 0) store8(k_cache + (size_t(slot) * p.Hkv + (head - p.Hq)) * dim + l * 8, f);
+    }
+  }
+  if (slot >= 0)
+    for (int i = tid; i < p.Hv * p.value_row / 8; i += blockDim.x) {
+      float f[8];
+      load8(row + size_t(heads) * dim + i * 8, f);
+      store8(v_cache + size_t(slot) * p.Hv * p.value_row + i * 8, f);
+    }
+  __syncthreads();
+  const int G = p.Hq / p.Hkv, dp = dim / 8, items = p.Hkv * dp;      // item: (key head, piece)
+  T* out = mixed + size_t(t) * p.Hq * p.Hkv * dim;
+  for (int i = tid; i < (p.Hq + 3) / 4 * items; i += blockDim.x) {
+    const int hb = i / items * 4, item = i % items, c = item / dp, d = (item - c * dp) * 8;
+    float acc[4][8] = {};
+    for (int g = 0; g < G; ++g) {
+      float q[8];
+      load8<float>(sq + (c * G + g) * dim + d, q);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float m = hb + j < p.Hq ? st[(hb + j) * p.Hq + c * G + g] : 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[j][e] = fmaf(m, q[e], acc[j][e]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (hb + j < p.Hq) store8(out + (size_t(hb + j) * p.Hkv + c) * dim + d, acc[j]);
+  }
+}
+
 // ------------------------------------------------------------------------------------ experts' activations
 // Rows of alternating (gate, up) columns.  kind 0: silu(g) * u; 1: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, +-limit) + 1).
 // Rows without gates: kind 2: max(x, 0)^2.
@@ -766,8 +857,23 @@ OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, 
   if (talk) {
     const size_t smem = (size_t(Hq) * (Hq + key_row) + 1) * 4;
     if (!mixed || Hq % Hkv || key_row % 8 || smem > 200 * 1024 || (reinterpret_cast<uintptr_t>(mixed) & 15)) return -1;
-    static bool done32[OGB_MAX_DEVICES] = {}, done16[OGB_MAX_DEVICES] = {};
     const dim3 block(256);
+    const bool pieces = dim == key_row && dim % 8 == 0 && dim <= 256 && rot % 16 == 0 && value_row % 8 == 0 && ldp % 8 == 0 &&
+                        ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
+                          reinterpret_cast<uintptr_t>(cos) | reinterpret_cast<uintptr_t>(sin) | reinterpret_cast<uintptr_t>(q_norm) |
+                          reinterpret_cast<uintptr_t>(k_norm)) & 15) == 0;
+    if (pieces) {
+      int lph = 1;
+      while (lph * 8 < dim) lph *= 2;
+      static bool p32[OGB_MAX_DEVICES] = {}, p16[OGB_MAX_DEVICES] = {};
+      using B = __nv_bfloat16;
+      if (fp32 ? !set_max_dyn_smem(qkv_prep_mixed_pieces_kernel<float>, 200 * 1024, p32) : !set_max_dyn_smem(qkv_prep_mixed_pieces_kernel<B>, 200 * 1024, p16)) return -3;
+      return (fp32 ? launch_pdl(qkv_prep_mixed_pieces_kernel<float>, dim3(T), block, smem, s, static_cast<const float*>(proj), static_cast<float*>(k_cache),
+                                static_cast<float*>(v_cache), p, talk, static_cast<float*>(mixed), lph)
+                   : launch_pdl(qkv_prep_mixed_pieces_kernel<B>, dim3(T), block, smem, s, static_cast<const B*>(proj), static_cast<B*>(k_cache),
+                                static_cast<B*>(v_cache), p, talk, static_cast<B*>(mixed), lph)) ? 0 : -4;
+    }
+    static bool done32[OGB_MAX_DEVICES] = {}, done16[OGB_MAX_DEVICES] = {};
     if (fp32) {
       if (!set_max_dyn_smem(qkv_prep_mixed_kernel<float>, 200 * 1024, done32)) return -3;
       return launch_pdl(qkv_prep_mixed_kernel<float>, dim3(T), block, smem, s, static_cast<const float*>(proj), static_cast<float*>(k_cache), static_cast<float*>(v_cache),

@@ -69,72 +69,98 @@ __global__ void moe_topk_kernel(const float* __restrict__ logits, int ld, int T,
   }
 }
 
+// A float as an unsigned number of the same order.
+__device__ __forceinline__ uint32_t order_bits(float v) {
+  const uint32_t u = __float_as_uint(v);
+  return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+// Entry with the largest key of the warp's lanes (each brings its best and where that is; 0: nothing), the smallest place among equal ones.
+__device__ __forceinline__ int warp_argmax(uint32_t key, int at) {
+  const uint32_t top = __reduce_max_sync(0xffffffffu, key);
+  return int(__reduce_min_sync(0xffffffffu, key == top ? uint32_t(at) : 0x7fffffffu));
+}
+
 // One warp per token: experts chosen by sigmoid(logit) + correction among the `keep` of `groups` groups of neighbours whose two largest choice
-// scores have the largest sums; weights: the chosen sigmoids divided by their sum (+ 1e-20), times scale.  Choice scores sit in shared memory.
-__global__ void moe_topk_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, const float* __restrict__ correction, int groups,
-                                        int keep, float scale, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
+// scores have the largest sums; weights: the chosen sigmoids divided by their sum (+ 1e-20), times scale.  A lane holds every 32nd expert, PER of them; the
+// scores also sit in shared memory for the groups' sums.
+template <int PER>
+__global__ void __launch_bounds__(128) moe_topk_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, const float* __restrict__ correction,
+                                                               int groups, int keep, float scale, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
   extern __shared__ float choice_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= T) return;
-  float* c = choice_all + size_t(warp) * (E + groups);
-  float* gs = c + E;                       // the groups' sums
+  float* c = choice_all + size_t(warp) * E;
   const float* row = logits + size_t(t) * ld;
-  for (int e = lane; e < E; e += 32) c[e] = 1.f / (1.f + expf(-row[e])) + correction[e];
-  __syncwarp();
-  auto best_of = [&](const float* v, int n, int& arg) {
-    float best = -INFINITY;
-    arg = 0x7fffffff;
-    for (int e = lane; e < n; e += 32) if (v[e] > best) { best = v[e]; arg = e; }
+  float s[PER];
+  uint32_t key[PER];                       // 0: not to be chosen
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, arg, o);
-      if (ov > best || (ov == best && oe < arg)) { best = ov; arg = oe; }
-    }
-  };
-  if (groups > 1) {
-    const int per = E / groups;
-    for (int g = lane; g < groups; g += 32) {
-      float a = -INFINITY, b = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) {
-        const float v = c[e];
-        if (v > a) { b = a; a = v; } else if (v > b) b = v;
-      }
-      gs[g] = per > 1 ? a + b : a;
-    }
-    __syncwarp();
-    // the kept groups are marked by +inf, the others' experts leave the choice
-    for (int j = 0; j < keep; ++j) {
-      float best = -INFINITY;
-      int arg = 0x7fffffff;
-      for (int g = lane; g < groups; g += 32) if (gs[g] != INFINITY && gs[g] > best) { best = gs[g]; arg = g; }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oe = __shfl_xor_sync(0xffffffffu, arg, o);
-        if (ov > best || (ov == best && oe < arg)) { best = ov; arg = oe; }
-      }
-      if (lane == 0 && arg < groups) gs[arg] = INFINITY;
-      __syncwarp();
-    }
-    for (int e = lane; e < E; e += 32) if (gs[e / per] != INFINITY) c[e] = -INFINITY;
-    __syncwarp();
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    s[i] = 0.f;
+    key[i] = 0;
+    if (e >= E) continue;
+    s[i] = 1.f / (1.f + expf(-row[e]));
+    const float v = s[i] + correction[e];
+    key[i] = order_bits(v);
+    if (groups > 1) c[e] = v;
   }
-  float s = 0.f;
+  if (groups > 1) {
+    __syncwarp();
+    const int per = E / groups;
+    // groups in rounds of 32, one per lane; a round's kept groups compete with those kept so far
+    uint32_t kept[32];                     // bit g % 32 of word g / 32
+    const int words = (groups + 31) / 32;
+#pragma unroll 1
+    for (int w = 0; w < words; ++w) {
+      const int g = w * 32 + lane;
+      uint32_t mine = 0;
+      if (g < groups) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int e = g * per; e < (g + 1) * per; ++e) {
+          const float v = c[e];
+          b = fmaxf(b, fminf(a, v));
+          a = fmaxf(a, v);
+        }
+        mine = order_bits(per > 1 ? a + b : a);
+      }
+      kept[w] = mine;
+    }
+    // `keep` times the best group that is left
+    uint32_t open_[32];
+    for (int w = 0; w < words; ++w) open_[w] = 0;
+    for (int j = 0; j < keep; ++j) {
+      uint32_t best = 0;
+      int at = 0x7fffffff;
+      for (int w = 0; w < words; ++w) if (kept[w] > best) { best = kept[w]; at = w * 32 + lane; }
+      const int g = warp_argmax(best, at);
+      if (g >= groups) break;
+      if ((g & 31) == lane) kept[g >> 5] = 0;
+      open_[g >> 5] |= 1u << (g & 31);
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int g = min(i * 32 + lane, E - 1) / per;
+      if (!(open_[g >> 5] >> (g & 31) & 1)) key[i] = 0;
+    }
+  }
+  float w = 0.f;
   int mine = 0;
   for (int j = 0; j < k; ++j) {
-    int e;
-    best_of(c, E, e);
-    e = e < E ? e : 0;
-    if (lane == j) { mine = e; s = 1.f / (1.f + expf(-row[e])); }
-    __syncwarp();
-    if (lane == 0) c[e] = -INFINITY;
-    __syncwarp();
+    uint32_t best = 0;
+    int at = 0x7fffffff;
+    float sv = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) if (key[i] > best) { best = key[i]; at = i * 32 + lane; sv = s[i]; }
+    const int e = min(warp_argmax(best, at), E - 1);       // (there are always enough experts to choose from)
+    sv = __shfl_sync(0xffffffffu, sv, e & 31);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) if (i * 32 + lane == e) key[i] = 0;
+    if (lane == j) { mine = e; w = sv; }
   }
-  const float sum = warp_sum(s) + 1e-20f;
+  const float sum = warp_sum(w) + 1e-20f;
   if (lane < k) {
     topk_idx[size_t(t) * k + lane] = mine;
-    topk_w[size_t(t) * k + lane] = s / sum * scale;
+    topk_w[size_t(t) * k + lane] = w / sum * scale;
   }
 }
 
@@ -238,8 +264,16 @@ OGB_API int ogb_moe_topk_grouped(const float* logits, int ld, int T, int E, int 
   if (T <= 0) return 0;
   if (E <= 0 || E > 1024 || k <= 0 || k > 32 || k > E || groups < 1 || E % groups || keep < 1 || keep > groups || k > E / groups * keep || !correction) return -1;
   const int warps = 4;
-  moe_topk_grouped_kernel<<<(T + warps - 1) / warps, warps * 32, size_t(warps) * (E + groups) * sizeof(float), static_cast<cudaStream_t>(stream)>>>(
-      logits, ld, T, E, k, correction, groups, keep, scale, topk_idx, topk_w);
+  const dim3 grid((T + warps - 1) / warps), block(warps * 32);
+  const size_t smem = groups > 1 ? size_t(warps) * E * sizeof(float) : 0;
+  auto st = static_cast<cudaStream_t>(stream);
+#define OGB_GROUPED(PER) moe_topk_grouped_kernel<PER><<<grid, block, smem, st>>>(logits, ld, T, E, k, correction, groups, keep, scale, topk_idx, topk_w)
+  if (E <= 32) OGB_GROUPED(1);
+  else if (E <= 64) OGB_GROUPED(2);
+  else if (E <= 128) OGB_GROUPED(4);
+  else if (E <= 256) OGB_GROUPED(8);
+  else OGB_GROUPED(32);
+#undef OGB_GROUPED
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -4,14 +4,14 @@
 //
 // Gated average, every column on its own:   z = sigmoid(z'),  c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0),  S <- (1 - z) S + z c,  out = S * silu(g) * scale.
 //   min_gru_step_kernel   decode-shaped steps: a thread walks the tokens of its columns.
-//   min_gru_scan_kernel   prompts: a CTA takes 16 columns and 512 tokens at a time, a thread 8 tokens of two columns.  S_t is an affine function of the
-//                         state before the thread's tokens, these functions are composed by a scan over the threads of a column, and the thread's
-//                         tokens are replayed from the state found.
+//   min_gru_chunk_kernel  prompts, in two passes over chunks of tokens: what a chunk does to a state is an affine function per column; the second pass
+//                         applies the functions of the chunks before its own to the first state and walks its tokens.
 //
 // Matrix memory, per head, with i and f the capped log gates and m the running maximum:
 //   m' = max(f + m, i),  S <- exp(f + m - m') S + exp(i - m') k v^T,  n likewise with k alone,  o = S^T q / (max(|n . q|, exp(-m')) + 1e-6),
 //   out = o / rms(o) * norm * sigmoid(g).
-//   mlstm_step_kernel     any step.  A cluster of CTAs shares the columns of a head; the state streams through registers once per token.
+//   mlstm_step_kernel     any step.  A CTA, or a cluster that shares the columns, has a head of a request; the state passes through registers, where it
+//                         stays over the tokens of a short portion.
 //   chunk form (bf16)     requests with many tokens, 64 at a time.  With b_t the sum of the chunk's log forget gates up to t, c_t = i_t - b_t and
 //                         M_t = max(m before the chunk, c_s for s <= t), the running maximum is b_t + M_t and the chunk's outputs and its end state are
 //                         products:  num_t = e^(m - M_t) q_t S + sum_{s <= t} e^(c_s - M_t) (q_t . k_s) v_s,  S' = e^(m - M_L) S + sum_s e^(c_s - M_L) k_s v_s^T
@@ -70,76 +70,59 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(MinGruParams p) {
   *st = S;
 }
 
-constexpr int MG_COLS = 16, MG_L = 8, MG_SEGS = 64, MG_THREADS = MG_SEGS * MG_COLS / 2;
+// Prompts, in chunks of MG_L tokens.  Pass 1: what a chunk does to a state, S -> A S + D, per column; the state before the request's first token is kept beside
+// (the last chunk of pass 2 overwrites it).  Pass 2: the state before the chunk from the chunks before it, then the chunk's tokens.  A thread has two
+// neighbouring columns.  Column count, strides and the columns' addresses are even.  Grid (.., chunks of the longest request, requests).
+constexpr int MG_L = 64, MG_AHEAD = 8, MG_THREADS = 128;
 
-// Column count, strides and the columns' addresses are even.
-template <typename T>
-__global__ void __launch_bounds__(MG_THREADS) min_gru_scan_kernel(MinGruParams p) {
-  __shared__ float sa[MG_COLS][MG_SEGS + 1], sb[MG_COLS][MG_SEGS + 1];
-  __shared__ float carry[MG_COLS];
+__device__ __forceinline__ size_t mg_chunk(int t0, int b, int j) { return size_t(t0 / MG_L + b + j); }      // (unique: see mc_chunk)
+
+template <typename T, bool OUT>
+__global__ void __launch_bounds__(MG_THREADS) min_gru_chunk_kernel(MinGruParams p, float4* __restrict__ maps, float2* __restrict__ first) {
   pdl_launch_dependents();
   pdl_wait();
-  const int b = blockIdx.y, t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
-  if (t0 >= t1) return;
-  const int tid = threadIdx.x, seg = tid / (MG_COLS / 2), cc = tid % (MG_COLS / 2) * 2, c = blockIdx.x * MG_COLS + cc;
-  const bool live = c < p.W;
-  float* st = p.state + size_t(p.slots[b]) * p.slot_stride;
+  const int b = blockIdx.z, j = blockIdx.y, t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
+  const int pair = blockIdx.x * MG_THREADS + threadIdx.x, c = 2 * pair, begin = t0 + j * MG_L, end = min(t1, begin + MG_L);
+  if (begin >= t1 || c >= p.W) return;
+  const int pairs = p.W / 2;
+  float* st = p.state + size_t(p.slots[b]) * p.slot_stride + c;
   const T *z = static_cast<const T*>(p.z) + c, *x = static_cast<const T*>(p.x) + c, *g = static_cast<const T*>(p.g) + c;
   T* out = static_cast<T*>(p.out) + c;
-  if (tid < MG_COLS) carry[tid] = p.past_lens[b] == 0 || blockIdx.x * MG_COLS + tid >= p.W ? 0.f : st[blockIdx.x * MG_COLS + tid];
-  for (int base = t0; base < t1; base += MG_SEGS * MG_L) {
-    // S after a token: a * S + d
-    float2 a[MG_L], d[MG_L], gate[MG_L];
-    const int ts = base + seg * MG_L;
-    float2 A = make_float2(1.f, 1.f), D = make_float2(0.f, 0.f);
-#pragma unroll
-    for (int i = 0; i < MG_L; ++i) {
-      const bool ok = live && ts + i < t1;
-      float2 zz = make_float2(0.f, 0.f), u = zz;
-      gate[i] = zz;
-      if (ok) {
-        zz = rec_ld2(z + size_t(ts + i) * p.ld);
-        u = rec_ld2(x + size_t(ts + i) * p.ld);
-        gate[i] = rec_ld2(g + size_t(ts + i) * p.ld);
-      }
-      const float s0 = ok ? rec_sigmoid(zz.x) : 0.f, s1 = ok ? rec_sigmoid(zz.y) : 0.f;
-      a[i] = make_float2(1.f - s0, 1.f - s1);
-      d[i] = make_float2(s0 * mg_candidate(u.x), s1 * mg_candidate(u.y));
-      D = make_float2(fmaf(a[i].x, D.x, d[i].x), fmaf(a[i].y, D.y, d[i].y));
-      A = make_float2(A.x * a[i].x, A.y * a[i].y);
+  float2 A = make_float2(1.f, 1.f), S = make_float2(0.f, 0.f);
+  if constexpr (OUT) {
+    S = first[size_t(b) * pairs + pair];
+    const float4* m = maps + mg_chunk(t0, b, 0) * pairs + pair;
+#pragma unroll 8
+    for (int i = 0; i < j; ++i) {
+      const float4 v = m[size_t(i) * pairs];
+      S = make_float2(fmaf(v.x, S.x, v.z), fmaf(v.y, S.y, v.w));
     }
-    sa[cc][seg] = A.x; sa[cc + 1][seg] = A.y;
-    sb[cc][seg] = D.x; sb[cc + 1][seg] = D.y;
-    __syncthreads();
-    // one warp per column: the state before every segment
-    {
-      const int w = tid >> 5, lane = tid & 31;
-      float a0 = sa[w][2 * lane], a1 = sa[w][2 * lane + 1], b0 = sb[w][2 * lane], b1 = sb[w][2 * lane + 1];
-      float pa = a0 * a1, pb = fmaf(a1, b0, b1);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float qa = __shfl_up_sync(0xffffffffu, pa, o), qb = __shfl_up_sync(0xffffffffu, pb, o);
-        if (lane >= o) { pb = fmaf(pa, qb, pb); pa *= qa; }
-      }
-      const float ea = __shfl_up_sync(0xffffffffu, pa, 1), eb = __shfl_up_sync(0xffffffffu, pb, 1), s0 = carry[w];
-      const float before = lane ? fmaf(ea, s0, eb) : s0;
-      sb[w][2 * lane] = before;
-      sb[w][2 * lane + 1] = fmaf(a0, before, b0);
-      const float end = __shfl_sync(0xffffffffu, fmaf(pa, s0, pb), 31);
-      __syncwarp();
-      if (lane == 0) carry[w] = end;
-    }
-    __syncthreads();
-    float2 S = make_float2(sb[cc][seg], sb[cc + 1][seg]);
-#pragma unroll
-    for (int i = 0; i < MG_L; ++i) {
-      S = make_float2(fmaf(a[i].x, S.x, d[i].x), fmaf(a[i].y, S.y, d[i].y));
-      if (live && ts + i < t1)
-        rec_st2(out + size_t(ts + i) * p.ldo, S.x * gate[i].x * rec_sigmoid(gate[i].x) * p.scale, S.y * gate[i].y * rec_sigmoid(gate[i].y) * p.scale);
-    }
-    __syncthreads();
+  } else if (j == 0) {
+    first[size_t(b) * pairs + pair] = p.past_lens[b] == 0 ? S : make_float2(st[0], st[1]);
   }
-  if (tid < MG_COLS && blockIdx.x * MG_COLS + tid < p.W) st[blockIdx.x * MG_COLS + tid] = carry[tid];
+  for (int t = begin; t < end; t += MG_AHEAD) {
+    float2 zz[MG_AHEAD], u[MG_AHEAD], gg[MG_AHEAD];
+#pragma unroll
+    for (int i = 0; i < MG_AHEAD; ++i) {
+      const int r = min(t + i, end - 1);
+      zz[i] = rec_ld2(z + size_t(r) * p.ld);
+      u[i] = rec_ld2(x + size_t(r) * p.ld);
+      if constexpr (OUT) gg[i] = rec_ld2(g + size_t(r) * p.ld);
+    }
+#pragma unroll
+    for (int i = 0; i < MG_AHEAD; ++i) {
+      if (t + i >= end) break;
+      const float s0 = rec_sigmoid(zz[i].x), s1 = rec_sigmoid(zz[i].y), a0 = 1.f - s0, a1 = 1.f - s1;
+      S = make_float2(fmaf(a0, S.x, s0 * mg_candidate(u[i].x)), fmaf(a1, S.y, s1 * mg_candidate(u[i].y)));
+      if constexpr (OUT) rec_st2(out + size_t(t + i) * p.ldo, S.x * gg[i].x * rec_sigmoid(gg[i].x) * p.scale, S.y * gg[i].y * rec_sigmoid(gg[i].y) * p.scale);
+      else A = make_float2(A.x * a0, A.y * a1);
+    }
+  }
+  if constexpr (OUT) {
+    if (end == t1) { st[0] = S.x; st[1] = S.y; }
+  } else {
+    maps[mg_chunk(t0, b, j) * pairs + pair] = make_float4(A.x, A.y, S.x, S.y);
+  }
 }
 
 // ------------------------------------------------------------------------------------ matrix memory
@@ -177,10 +160,9 @@ __device__ __forceinline__ float rec_ld_peer(const float* local, uint32_t rank) 
   return v;
 }
 
-// Grid (cluster, heads, requests).  The CTA owns columns [rank * cw, rank * cw + cw) of the head, cw = a multiple of VEC of at most 256; thread
-// (row group, column group of VEC).  Every token: the factors, n . q (by all CTAs alike), then the state's rows through registers.  The state of a step
-// of several tokens is read back by the thread that wrote it.
-template <typename T, int VEC>
+// Grid (cluster, heads, requests).  The CTA owns columns [rank * cw, rank * cw + cw) of the head (cw a multiple of VEC, at most 256), a thread VEC columns of every
+// groups-th row: NR rows in registers from the first token to the last, or (NR = 0) any number, read and written back at every token.
+template <typename T, int VEC, int NR>
 __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, int cw) {
   __shared__ float sk[ML_MAX_D], sq[ML_MAX_D], sn[ML_MAX_D];
   __shared__ float red[ML_THREADS * VEC];
@@ -194,20 +176,43 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, i
   if (t0 >= t1 || (p.long_tokens > 0 && t1 - t0 >= p.long_tokens)) return;      // (alike in all CTAs of a cluster)
   const bool fresh = p.past_lens[b] == 0;
   float* slot = p.state + size_t(p.slots[b]) * p.slot_stride;
-  float* S = slot + size_t(h) * d * dv;
-  float* gn = slot + size_t(p.H) * d * dv + size_t(h) * d;
-  float* gm = slot + size_t(p.H) * d * (dv + 1) + h;
   const int c0 = rank * cw, cols = min(cw, dv - c0);                // (may be <= 0)
   const int lanes = (cw + VEC - 1) / VEC;                           // column groups
   const int groups = ML_THREADS / lanes, cg = tid % lanes, rg = tid / lanes, col = cg * VEC;
   const bool mine = rg < groups && col < cols;
+  float* S = slot + size_t(h) * d * dv + c0 + col;
+  float* gn = slot + size_t(p.H) * d * dv + size_t(h) * d;
+  float* gm = slot + size_t(p.H) * d * (dv + 1) + h;
+  auto load = [&](int r, float (&s)[VEC]) {
+    if constexpr (VEC == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(S + size_t(r) * dv);
+      s[0] = f.x; s[1] = f.y; s[2] = f.z; s[3] = f.w;
+    } else {
+      s[0] = S[size_t(r) * dv];
+    }
+  };
+  auto store = [&](int r, const float (&s)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(S + size_t(r) * dv) = make_float4(s[0], s[1], s[2], s[3]);
+    else S[size_t(r) * dv] = s[0];
+  };
+  float st[NR > 0 ? NR : 1][VEC];
+  if constexpr (NR > 0) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[i][e] = 0.f;
+      if (mine && !fresh && rg + i * groups < d) load(rg + i * groups, st[i]);
+    }
+  }
   for (int i = tid; i < d; i += ML_THREADS) sn[i] = fresh ? 0.f : gn[i];
   float m = fresh ? 0.f : *gm;
-  if (C > 1) { __syncthreads(); rec_cluster_arrive(); rec_cluster_wait(); }      // n and m have been read by every CTA
   for (int t = t0; t < t1; ++t) {
     const T* qp = static_cast<const T*>(p.q) + size_t(t) * p.ld + size_t(h) * d;
     const T* kp = static_cast<const T*>(p.k) + size_t(t) * p.ld + size_t(h) * d;
     const float* gp = p.gates + size_t(t) * p.ldg;
+    float v[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = mine ? rec_f32(static_cast<const T*>(p.v)[size_t(t) * p.ld + size_t(h) * dv + c0 + col + e]) : 0.f;
     const MlstmGate gt = mlstm_gate(gp[h] + p.gate_b[h], gp[p.H + h] + p.gate_b[p.H + h], p.cap, m);
     m = gt.m;
     float nq = 0.f;
@@ -222,35 +227,30 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, i
     nq = 0.f;
 #pragma unroll
     for (int w = 0; w < ML_THREADS / 32; ++w) nq += part[w];
-    float o[VEC], v[VEC];
+    float o[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) o[e] = 0.f;
-    if (mine) {
-      const T* vp = static_cast<const T*>(p.v) + size_t(t) * p.ld + size_t(h) * dv + c0 + col;
+    auto step = [&](int r, float (&s)[VEC]) {
+      const float kk = sk[r], qq = sq[r];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[e] = rec_f32(vp[e]);
-      const bool zero = fresh && t == t0;
-#pragma unroll 4
-      for (int r = rg; r < d; r += groups) {
-        float* sp = S + size_t(r) * dv + c0 + col;
-        float s[VEC];
-        if (zero) {
+      for (int e = 0; e < VEC; ++e) {
+        s[e] = fmaf(gt.keep, s[e], kk * v[e]);
+        o[e] = fmaf(qq, s[e], o[e]);
+      }
+    };
+    if (mine) {
+      if constexpr (NR > 0) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) if (rg + i * groups < d) step(rg + i * groups, st[i]);
+      } else {
+        for (int r = rg; r < d; r += groups) {
+          float s[VEC];
 #pragma unroll
           for (int e = 0; e < VEC; ++e) s[e] = 0.f;
-        } else if constexpr (VEC == 4) {
-          const float4 f = *reinterpret_cast<const float4*>(sp);
-          s[0] = f.x; s[1] = f.y; s[2] = f.z; s[3] = f.w;
-        } else {
-          s[0] = *sp;
+          if (!(fresh && t == t0)) load(r, s);
+          step(r, s);
+          store(r, s);
         }
-        const float kk = sk[r], qq = sq[r];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-          s[e] = fmaf(gt.keep, s[e], kk * v[e]);
-          o[e] = fmaf(qq, s[e], o[e]);
-        }
-        if constexpr (VEC == 4) *reinterpret_cast<float4*>(sp) = make_float4(s[0], s[1], s[2], s[3]);
-        else *sp = s[0];
       }
     }
 #pragma unroll
@@ -259,6 +259,7 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, i
     // column sums over the row groups: thread tid takes column tid
     float val = 0.f;
     if (tid < cols) {
+#pragma unroll 8
       for (int r = 0; r < groups; ++r) val += red[r * lanes * VEC + tid];
       val /= fmaxf(fabsf(nq), gt.floor) + 1e-6f;
     }
@@ -281,8 +282,15 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_step_kernel(MlstmParams p, i
       const float gate = rec_sigmoid(rec_f32(static_cast<const T*>(p.g)[size_t(t) * p.ld + at]));
       static_cast<T*>(p.out)[size_t(t) * p.ldo + at] = rec_from<T>(val / sqrtf(ss / dv + p.eps) * p.norm_w[at] * gate);
     }
-    __syncthreads();
+    if (t + 1 < t1) __syncthreads();
   }
+  if constexpr (NR > 0) {
+    if (mine) {
+#pragma unroll
+      for (int i = 0; i < NR; ++i) if (rg + i * groups < d) store(rg + i * groups, st[i]);
+    }
+  }
+  // (every CTA of the cluster has read the normaliser and the maximum: all have met at a token)
   if (rank == 0) {
     for (int i = tid; i < d; i += ML_THREADS) gn[i] = sn[i];
     if (tid == 0) *gm = m;
@@ -716,10 +724,12 @@ __global__ void __launch_bounds__(256, NTW <= 8 ? 2 : 1) mlstm_out_kernel(MlstmP
 
 using namespace ogb;
 
+OGB_API long long ogb_min_gru_scratch_bytes(int T, int B, int W) { return ((long long)(T / MG_L + B) * 16 + (long long)B * 8) * ((W + 1) / 2); }
+
 // See kernels.h.
 OGB_API int ogb_min_gru(const void* z, const void* x, const void* g, int ld, float* state, long long slot_stride, const int32_t* slots,
-                        const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int ldo, int B, int W, float scale, int max_q_len, int fp32,
-                        void* stream) {
+                        const int32_t* cu_seqlens, const int32_t* past_lens, void* out, int ldo, int T, int B, int W, float scale, int max_q_len,
+                        void* scratch, long long scratch_bytes, int fp32, void* stream) {
   if (B <= 0 || W <= 0) return 0;
   if (B > 65535 || slot_stride < W) return -1;
   const MinGruParams p{z, x, g, out, state, slots, cu_seqlens, past_lens, slot_stride, ld, ldo, W, scale};
@@ -727,28 +737,41 @@ OGB_API int ogb_min_gru(const void* z, const void* x, const void* g, int ld, flo
   auto addr = [](const void* a) { return reinterpret_cast<uintptr_t>(a); };
   const bool even = W % 2 == 0 && ld % 2 == 0 && ldo % 2 == 0 && ((addr(z) | addr(x) | addr(g) | addr(out)) & (fp32 ? 7 : 3)) == 0;
   using H = __nv_bfloat16;
-  if (max_q_len <= 16 || !even) {
+  if (!scratch || !even) {
     const dim3 grid((W + 127) / 128, B), block(128);
     return (fp32 ? launch_pdl(min_gru_step_kernel<float>, grid, block, 0, s, p) : launch_pdl(min_gru_step_kernel<H>, grid, block, 0, s, p)) ? 0 : -4;
   }
-  const dim3 grid((W + MG_COLS - 1) / MG_COLS, B), block(MG_THREADS);
-  return (fp32 ? launch_pdl(min_gru_scan_kernel<float>, grid, block, 0, s, p) : launch_pdl(min_gru_scan_kernel<H>, grid, block, 0, s, p)) ? 0 : -4;
+  if (scratch_bytes < ogb_min_gru_scratch_bytes(T, B, W) || (addr(scratch) & 15)) return -2;
+  auto* maps = static_cast<float4*>(scratch);
+  auto* first = reinterpret_cast<float2*>(maps + size_t(T / MG_L + B) * (W / 2));
+  const dim3 grid((W / 2 + MG_THREADS - 1) / MG_THREADS, (max_q_len + MG_L - 1) / MG_L, B), block(MG_THREADS);
+  if (grid.y > 65535) return -1;
+  const bool ok = fp32 ? launch_pdl(min_gru_chunk_kernel<float, false>, grid, block, 0, s, p, maps, first) && launch_pdl(min_gru_chunk_kernel<float, true>, grid, block, 0, s, p, maps, first)
+                       : launch_pdl(min_gru_chunk_kernel<H, false>, grid, block, 0, s, p, maps, first) && launch_pdl(min_gru_chunk_kernel<H, true>, grid, block, 0, s, p, maps, first);
+  return ok ? 0 : -4;
 }
 
-template <typename T, int VEC>
-static bool LaunchMlstmStep(const MlstmParams& p, int B, int cw, int C, cudaStream_t s) {
+template <typename T, int VEC, int NR>
+static bool LaunchMlstmStepRows(const MlstmParams& p, int B, int cw, int C, cudaStream_t s) {
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(C, p.H, B);
   cfg.blockDim = dim3(ML_THREADS);
   cfg.stream = s;
   cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = C; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
-  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = C; attr[1].val.clusterDim.y = 1; attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr;
-  cfg.numAttrs = 2;
-  return cudaLaunchKernelEx(&cfg, mlstm_step_kernel<T, VEC>, p, cw) == cudaSuccess;
+  cfg.numAttrs = C > 1 ? 2 : 1;
+  return cudaLaunchKernelEx(&cfg, mlstm_step_kernel<T, VEC, NR>, p, cw) == cudaSuccess;
+}
+template <typename T, int VEC>
+static bool LaunchMlstmStep(const MlstmParams& p, int B, int cw, int C, int rows, cudaStream_t s) {
+  if (rows <= 4) return LaunchMlstmStepRows<T, VEC, 4>(p, B, cw, C, s);
+  if (rows <= 8) return LaunchMlstmStepRows<T, VEC, 8>(p, B, cw, C, s);
+  if (rows <= 16) return LaunchMlstmStepRows<T, VEC, 16>(p, B, cw, C, s);
+  return LaunchMlstmStepRows<T, VEC, 0>(p, B, cw, C, s);
 }
 
 // Sizes of the chunk form's scratch, or false where its kernels cannot run.
@@ -817,14 +840,15 @@ OGB_API int ogb_mlstm(const OgbMlstm* a, void* stream) {
   // states in whole 16-byte pieces (a slot's first float is on a 16-byte boundary, heads and rows are multiples of four)
   const bool vec = a->dv % 4 == 0 && a->slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a->state) & 15) == 0;
   const int unit = vec ? 4 : 1;
-  // columns of a CTA: 32 where that needs no more than a cluster of eight (so that few requests still use many SMs), at most 256
-  int cw = 32;
-  while ((a->dv + cw - 1) / cw > ML_MAX_CLUSTER) cw *= 2;
+  // CTAs that share a head: no more than it takes for two CTAs per SM, and for 16 rows of a thread to hold the state; no fewer than 32 columns each
+  int C = 1, cw = 0, rows = 0;
+  for (;; C *= 2) {
+    cw = ((a->dv + C - 1) / C + unit - 1) / unit * unit;
+    rows = cw <= 256 ? (a->d + ML_THREADS / ((cw + unit - 1) / unit) - 1) / (ML_THREADS / ((cw + unit - 1) / unit)) : 1 << 20;
+    if (C == ML_MAX_CLUSTER || (cw <= 256 && (cw < 64 || (rows <= 16 && (long long)a->B * a->H * C >= 296)))) break;
+  }
   if (cw > 256) return -5;
-  int C = (a->dv + cw - 1) / cw;
-  while (C & (C - 1)) ++C;              // (a CTA without columns only meets the others)
-  if (C == 1) cw = (a->dv + unit - 1) / unit * unit;
-  const bool ok = a->fp32 ? (vec ? LaunchMlstmStep<float, 4>(p, a->B, cw, C, s) : LaunchMlstmStep<float, 1>(p, a->B, cw, C, s))
-                          : (vec ? LaunchMlstmStep<__nv_bfloat16, 4>(p, a->B, cw, C, s) : LaunchMlstmStep<__nv_bfloat16, 1>(p, a->B, cw, C, s));
+  const bool ok = a->fp32 ? (vec ? LaunchMlstmStep<float, 4>(p, a->B, cw, C, rows, s) : LaunchMlstmStep<float, 1>(p, a->B, cw, C, rows, s))
+                          : (vec ? LaunchMlstmStep<__nv_bfloat16, 4>(p, a->B, cw, C, rows, s) : LaunchMlstmStep<__nv_bfloat16, 1>(p, a->B, cw, C, rows, s));
   return ok ? 0 : -4;
 }

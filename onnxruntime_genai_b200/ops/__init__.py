@@ -933,6 +933,15 @@ def choose_kv_splits(batch: int, Hkv: int, max_q_len: int, max_kv_len: int, sm_c
     return int(splits), int(chunk)
 
 
+def choose_joint_splits(batch: int, Hq: int, dk: int, v_cols: int, max_q_len: int, span: int, sm_count: int = 148) -> int:
+    """Key splits of a launch for heads whose scores are mixed (one CTA per token and 32 heads): about two waves of the CTAs that are resident at a time,
+    each split at least two tiles of keys."""
+    form = _lib.lib().ogb_attention_joint_form(int(Hq), int(dk), int(v_cols))
+    tile, resident = form // 4, form % 4
+    ctas = max(1, batch * max_q_len * ((Hq + 31) // 32))
+    return max(1, min(int(round(2.0 * resident * sm_count / ctas)), span // (2 * tile), 32))
+
+
 TC_ATTENTION_MIN_ROWS = 128      # query rows (tokens x heads of a GQA group) from which a request takes the tcgen05 prefill kernel
 _TC_ATTENTION = os.environ.get("OGB_ATTN_TC", "1") != "0"
 
@@ -1040,8 +1049,9 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
         return int(sp) * tokens * Hq * (dv + 2) * 4
     inputs = (ctypes.byref(layer), _ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(cu_seqlens), _ptr(past_lens), _ptr(block_table),
               block_table.stride(0), int(block_size), _ptr(out), out.stride(0), B)
-    if (q.dtype == torch.float32 or not L.ogb_attention_mixed_supported(dk, dv) or q.stride(0) % 8 or out.stride(0) % 2 or q.data_ptr() % 16 or
-            out.data_ptr() % 4):
+    served = L.ogb_attention_joint_supported(dk, Hkv * dv) if joint else L.ogb_attention_mixed_supported(dk, dv)
+    if (q.dtype == torch.float32 or not served or q.stride(0) % 8 or out.stride(0) % 2 or q.data_ptr() % 16 or out.data_ptr() % 4 or
+            (joint and (dv % 8 or chunk > 0 or (wide and (gate.stride(0) % 2 or gate.data_ptr() % 4))))):
         # (the grid covers the rows of the whole matrix: rows of requests outside this call are skipped)
         n = q.shape[0]
         scratch = ws.attn_scratch(part_bytes(n, 1)) if diff is not None else None
@@ -1051,7 +1061,8 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
     slots = int(k_cache.shape[0])
     long_rows = TC_ATTENTION_MIN_ROWS
     use_tc = (_TC_ATTENTION and max_q_len * G >= long_rows and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and
-              bool(L.ogb_attention_tc_mixed_supported(dk // maps, dv, int(block_size), slots)) and
+              bool(L.ogb_attention_tc_joint_supported(dk, dv, int(block_size), slots) if joint else
+                   L.ogb_attention_tc_mixed_supported(dk // maps, dv, int(block_size), slots)) and
               (not wide or diff is not None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)))
     sp, ch, scratch = 1, 0, None
     all_long = use_tc and min_q_len is not None and min_q_len * G >= long_rows
@@ -1061,11 +1072,19 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
             span = max_kv_len or 1024
             if chunk > 0 or window > 0:
                 span = min(span, (chunk or window) + 63)
-            splits = choose_kv_splits(B, Hkv, max_q_len, span, group=G, ordered=order is not None)
+            if joint:
+                splits = choose_joint_splits(B, Hq, dk, Hkv * dv, max_q_len, span, ws.sm_count)
+            else:
+                splits = choose_kv_splits(B, Hkv, max_q_len, span, group=G, ordered=order is not None)
         sp, ch = splits if isinstance(splits, tuple) else (splits, 0)
     if sp > 1 or diff is not None:
         scratch = ws.attn_scratch(part_bytes(T, sp))
-    if not all_long:
+    if not all_long and joint:
+        _lib.check(L.ogb_attention_joint(*inputs, T, int(max_q_len), int(sp), _ptr(scratch), scratch.numel() if scratch is not None else 0, _ptr(order),
+                                         ws.status, _stream(), long_rows if use_tc else 0), "attention_joint")
+        if sp > 1:
+            _lib.LAUNCH_COUNT += 1      # the combine kernel
+    elif not all_long:
         _lib.check(L.ogb_attention_mixed(*inputs, T, int(max_q_len), int(sp), int(ch), _ptr(scratch), scratch.numel() if scratch is not None else 0,
                                          _ptr(order), ws.status, _stream(), long_rows if use_tc else 0), "attention_mixed")
         if sp > 1 and diff is None:
@@ -1077,6 +1096,9 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
 
 
 # ------------------------------------------------------------------------------------------ recurrent mixers of declared stacks
+MIN_GRU_STEP_TOKENS = 16    # portions of at most this many tokens are walked token by token
+
+
 def min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale=1.0, max_q_len=0):
     """Gated average per column over packed sequences: S <- (1 - sigmoid(z)) S + sigmoid(z) * c(x) with c(x) = x + 1/2 for x >= 0 and sigmoid(x) below;
     out = S * silu(g) * scale.  z, x, g [T, W]: columns of one matrix; state [slots, W] fp32 (rows may be further apart), updated in place; a request whose
@@ -1086,9 +1108,14 @@ def min_gru(z, x, g, state, slots, cu_seqlens, past_lens, out, scale=1.0, max_q_
     T, W = z.shape
     assert z.dtype == x.dtype == g.dtype == out.dtype and z.stride() == x.stride() == g.stride() and z.stride(1) == out.stride(1) == 1
     assert state.dtype == torch.float32 and state.stride(1) == 1 and out.shape == (T, W)
+    max_q_len = int(max_q_len or T)
+    scratch = None
+    if max_q_len > MIN_GRU_STEP_TOKENS:
+        scratch = torch.empty(_lib.lib().ogb_min_gru_scratch_bytes(T, past_lens.shape[0], W), dtype=torch.uint8, device=z.device)
+        _lib.LAUNCH_COUNT += 1
     _lib.check(_lib.lib().ogb_min_gru(_ptr(z), _ptr(x), _ptr(g), z.stride(0), _ptr(state), state.stride(0), _ptr(slots), _ptr(cu_seqlens), _ptr(past_lens),
-                                     _ptr(out), out.stride(0), past_lens.shape[0], W, float(scale), int(max_q_len or T), int(z.dtype == torch.float32),
-                                     _stream()), "min_gru")
+                                     _ptr(out), out.stride(0), T, past_lens.shape[0], W, float(scale), max_q_len, _ptr(scratch),
+                                     scratch.numel() if scratch is not None else 0, int(z.dtype == torch.float32), _stream()), "min_gru")
     return out
 
 

@@ -115,6 +115,10 @@ _SIGS = {
     "ogb_attention_mixed_supported": (c_int, [c_int, c_int]),
     "ogb_attention_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P,
                                     _P, c_int]),
+    "ogb_attention_joint_supported": (c_int, [c_int, c_int]),
+    "ogb_attention_joint_form": (c_int, [c_int, c_int, c_int]),
+    "ogb_attention_joint": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P, _P, c_int]),
+    "ogb_attention_tc_joint_supported": (c_int, [c_int, c_int, c_int, c_int]),
     "ogb_attention_tc_mixed_supported": (c_int, [c_int, c_int, c_int, c_int]),
     "ogb_attention_tc_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P,
                                        c_longlong, _P, _P]),
@@ -123,7 +127,8 @@ _SIGS = {
     "ogb_add_tanh_norm": (c_int, [ctypes.POINTER(TanhNorm), _P]),
     "ogb_embedding_bigram": (c_int, [ctypes.POINTER(Bigram), _P, _P, _P, _P]),
     "ogb_norm_stream": (c_int, [ctypes.POINTER(NormStream), _P]),
-    "ogb_min_gru": (c_int, [_P, _P, _P, c_int, _P, c_longlong, _P, _P, _P, _P, c_int, c_int, c_int, c_float, c_int, c_int, _P]),
+    "ogb_min_gru": (c_int, [_P, _P, _P, c_int, _P, c_longlong, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_float, c_int, _P, c_longlong, c_int, _P]),
+    "ogb_min_gru_scratch_bytes": (c_longlong, [c_int, c_int, c_int]),
     "ogb_mlstm_scratch_bytes": (c_longlong, [c_int, c_int, c_int, c_int, c_int]),
     "ogb_mlstm": (c_int, [ctypes.POINTER(Mlstm), _P]),
     "ogb_moe_topk_grouped": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, c_int, c_float, _P, _P, _P]),
