@@ -188,7 +188,6 @@ int ogb_attention_mixed(const OgbAttnLayer* a, const void* q, int q_stride, cons
                         int* status, void* stream, int skip_rows);
 // attention_joint.cu: joint layers, decode steps and short portions
 int ogb_attention_joint_supported(int dk, int v_cols);
-int ogb_attention_joint_form(int Hq, int dk, int v_cols);
 int ogb_attention_joint(const OgbAttnLayer* l, const void* q, int q_stride, const void* k_cache, const void* v_cache, const int32_t* cu_seqlens,
                         const int32_t* past_lens, const int32_t* block_table, int table_cols, int block_size, void* out, int out_stride, int B,
                         int total_tokens, int max_q_len, int splits, void* scratch, long long scratch_bytes, const int32_t* order, int* status,

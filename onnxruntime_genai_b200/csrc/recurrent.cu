@@ -38,6 +38,11 @@ __device__ __forceinline__ void rec_st2(float* p, float a, float b) { *reinterpr
 __device__ __forceinline__ void rec_st2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b); }
 
 __device__ __forceinline__ float rec_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+// The same for models with 16-bit activations, with the hardware's exponential and reciprocal (relative error of a few 1e-7 where the argument is of the order of one).
+template <typename T> __device__ __forceinline__ float rec_gate(float x) {
+  if constexpr (sizeof(T) == 4) return rec_sigmoid(x);
+  else return __fdividef(1.f, 1.f + __expf(-fmaxf(x, -80.f)));
+}
 
 // ------------------------------------------------------------------------------------ gated average
 struct MinGruParams {
@@ -50,7 +55,7 @@ struct MinGruParams {
   float scale;
 };
 
-__device__ __forceinline__ float mg_candidate(float u) { return u >= 0.f ? u + 0.5f : rec_sigmoid(u); }
+template <typename T> __device__ __forceinline__ float mg_candidate(float u) { return u >= 0.f ? u + 0.5f : rec_gate<T>(u); }
 
 template <typename T>
 __global__ void __launch_bounds__(128) min_gru_step_kernel(MinGruParams p) {
@@ -63,9 +68,9 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(MinGruParams p) {
   const T *z = static_cast<const T*>(p.z) + c, *x = static_cast<const T*>(p.x) + c, *g = static_cast<const T*>(p.g) + c;
   float S = p.past_lens[b] == 0 ? 0.f : *st;
   for (int t = t0; t < t1; ++t) {
-    const float zz = rec_sigmoid(rec_f32(z[size_t(t) * p.ld])), gg = rec_f32(g[size_t(t) * p.ld]);
-    S = fmaf(zz, mg_candidate(rec_f32(x[size_t(t) * p.ld])), (1.f - zz) * S);
-    static_cast<T*>(p.out)[size_t(t) * p.ldo + c] = rec_from<T>(S * gg * rec_sigmoid(gg) * p.scale);
+    const float zz = rec_gate<T>(rec_f32(z[size_t(t) * p.ld])), gg = rec_f32(g[size_t(t) * p.ld]);
+    S = fmaf(zz, mg_candidate<T>(rec_f32(x[size_t(t) * p.ld])), (1.f - zz) * S);
+    static_cast<T*>(p.out)[size_t(t) * p.ldo + c] = rec_from<T>(S * gg * rec_gate<T>(gg) * p.scale);
   }
   *st = S;
 }
@@ -112,9 +117,9 @@ __global__ void __launch_bounds__(MG_THREADS) min_gru_chunk_kernel(MinGruParams 
 #pragma unroll
     for (int i = 0; i < MG_AHEAD; ++i) {
       if (t + i >= end) break;
-      const float s0 = rec_sigmoid(zz[i].x), s1 = rec_sigmoid(zz[i].y), a0 = 1.f - s0, a1 = 1.f - s1;
-      S = make_float2(fmaf(a0, S.x, s0 * mg_candidate(u[i].x)), fmaf(a1, S.y, s1 * mg_candidate(u[i].y)));
-      if constexpr (OUT) rec_st2(out + size_t(t + i) * p.ldo, S.x * gg[i].x * rec_sigmoid(gg[i].x) * p.scale, S.y * gg[i].y * rec_sigmoid(gg[i].y) * p.scale);
+      const float s0 = rec_gate<T>(zz[i].x), s1 = rec_gate<T>(zz[i].y), a0 = 1.f - s0, a1 = 1.f - s1;
+      S = make_float2(fmaf(a0, S.x, s0 * mg_candidate<T>(u[i].x)), fmaf(a1, S.y, s1 * mg_candidate<T>(u[i].y)));
+      if constexpr (OUT) rec_st2(out + size_t(t + i) * p.ldo, S.x * gg[i].x * rec_gate<T>(gg[i].x) * p.scale, S.y * gg[i].y * rec_gate<T>(gg[i].y) * p.scale);
       else A = make_float2(A.x * a0, A.y * a1);
     }
   }
@@ -313,7 +318,7 @@ struct MlstmChunk {
 __device__ __forceinline__ int mc_chunk(int t0, int b, int j) { return t0 / MC_L + b + j; }
 
 // One CTA per (head, request).  A warp takes chunks, a lane two of a chunk's tokens; then the maxima are chained over the chunks.
-__global__ void __launch_bounds__(256) mlstm_gates_kernel(MlstmParams p, MlstmChunk k) {
+__global__ void __launch_bounds__(1024) mlstm_gates_kernel(MlstmParams p, MlstmChunk k) {
   extern __shared__ float sm[];        // per chunk: sum of log forget gates, largest c, maximum before the chunk
   pdl_launch_dependents();
   pdl_wait();
@@ -323,7 +328,7 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(MlstmParams p, MlstmCh
   float *sb = sm, *sc = sm + n, *si = sm + 2 * n;
   const float bi = p.gate_b[h], bf = p.gate_b[p.H + h];
   float *gc = k.c + size_t(h) * k.T + t0, *gM = k.M + size_t(h) * k.T + t0, *gf = k.floor + size_t(h) * k.T + t0;
-  for (int j = warp; j < n; j += 8) {
+  for (int j = warp; j < n; j += blockDim.x >> 5) {
     float i[2], f[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
@@ -624,15 +629,29 @@ __global__ void __launch_bounds__(256, NTW <= 8 ? 2 : 1) mlstm_out_kernel(MlstmP
     for (int i = 0; i < NTW; ++i) { o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f; }
   const int nt0 = cg * NTW;
   if (!empty) {
+    // (the next step's fragments are on their way while this one's are multiplied; groups past the last read it again)
     const uint4* S = reinterpret_cast<const uint4*>(k.sums) + (size_t(chunk) * p.H + h) * k.KS * k.NT * 32 + lane;
+    constexpr int PF = NTW <= 8 ? NTW : 1;
+    uint4 next[PF];
+    auto fetch = [&](int ks, int i) { return S[(size_t(ks) * k.NT + min(nt0 + i, k.NT - 1)) * 32]; };
+    if constexpr (PF == NTW) {
+#pragma unroll
+      for (int i = 0; i < PF; ++i) next[i] = fetch(0, i);
+    }
     for (int ks = 0; ks < k.KS; ++ks) {
       uint32_t a[2][4];
+      uint4 now[PF];
+      if constexpr (PF == NTW) {
+        const int after = min(ks + 1, k.KS - 1);
+#pragma unroll
+        for (int i = 0; i < PF; ++i) { now[i] = next[i]; next[i] = fetch(after, i); }
+      }
 #pragma unroll
       for (int mt = 0; mt < 2; ++mt) ldmatrix_x4(a[mt], sq + (rg * 32 + mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * qpitch + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
       for (int i = 0; i < NTW; ++i) {
         if (nt0 + i >= k.NT) break;
-        const uint4 f = S[(size_t(ks) * k.NT + nt0 + i) * 32];
+        const uint4 f = PF == NTW ? now[i % PF] : fetch(ks, i);
 #pragma unroll
         for (int mt = 0; mt < 2; ++mt) {
           mma_bf16_16816(o[mt][i], a[mt], f.x, f.y);
@@ -814,7 +833,7 @@ static int LaunchMlstmChunks(const MlstmParams& p, const OgbMlstm* a, cudaStream
   if (n > 65535 || (long long)a->B * a->H > 65535) return -1;
   const size_t gsmem = size_t(3) * n * 4;
   if (gsmem > 48 * 1024) return -5;
-  if (!launch_pdl(mlstm_gates_kernel, dim3(a->H, a->B), dim3(256), gsmem, s, p, k)) return -4;
+  if (!launch_pdl(mlstm_gates_kernel, dim3(a->H, a->B), dim3(n >= 16 ? 1024 : (n >= 8 ? 512 : 256)), gsmem, s, p, k)) return -4;
   if (!launch_pdl(mlstm_sums_kernel, dim3(((k.NT + 7) / 8) * ((k.KS + 3) / 4), n, a->B * a->H), dim3(128), 0, s, p, k)) return -4;
   if (!launch_pdl(mlstm_scan_kernel, dim3((k.KS * k.NT * 32 + 255) / 256 + 1, a->H, a->B), dim3(256), 0, s, p, k)) return -4;
   const dim3 grid(n, a->H, a->B);

@@ -116,7 +116,6 @@ _SIGS = {
     "ogb_attention_mixed": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P,
                                     _P, c_int]),
     "ogb_attention_joint_supported": (c_int, [c_int, c_int]),
-    "ogb_attention_joint_form": (c_int, [c_int, c_int, c_int]),
     "ogb_attention_joint": (c_int, [_AL, _P, c_int, _P, _P, _P, _P, _P, c_int, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, c_longlong, _P, _P, _P, c_int]),
     "ogb_attention_tc_joint_supported": (c_int, [c_int, c_int, c_int, c_int]),
     "ogb_attention_tc_mixed_supported": (c_int, [c_int, c_int, c_int, c_int]),
