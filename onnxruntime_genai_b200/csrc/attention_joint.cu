@@ -23,9 +23,10 @@ struct JointParams {
 };
 
 // MT: 16-head tiles; KSW: 16-column steps of the keys per warp; NP: pairs of 8-column groups of the values per warp; BN: keys per tile; CTAS: per SM.
-template <int AJ_WARPS, int MT, int KSW, int NP, int BN, int CTAS>
+// ONE: the heads of a key head's group are all in one head tile (16 is a multiple of the group), so that a group of value columns needs one accumulator.
+template <int AJ_WARPS, int MT, int KSW, int NP, int BN, int CTAS, bool ONE>
 __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(JointParams jp) {
-  constexpr int AJ_THREADS = AJ_WARPS * 32, ROWS = 16 * MT, TPR = AJ_THREADS / ROWS, KPT = BN / TPR, SP = BN + 2, PP = BN + 8;
+  constexpr int AJ_THREADS = AJ_WARPS * 32, ROWS = 16 * MT, TPR = AJ_THREADS / ROWS, MO = ONE ? 1 : MT, KPT = BN / TPR, SP = BN + 2, PP = BN + 8;
   // elements between the rows of a tile: an odd number of 16-byte pieces, as wide as the form's widest rows (fixed, so that addresses are offsets)
   constexpr int KPITCH = AJ_WARPS * KSW * 16 + 8, VPITCH = AJ_WARPS * NP * 16 + 8;
   static_assert(KPT >= 1 && BN % TPR == 0, "a row's keys are divided over its threads");
@@ -133,13 +134,13 @@ __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(Jo
   const int sr = tid / TPR, sk0 = (tid % TPR) * KPT;      // softmax: row and first key of this thread
   const float sc2 = p.scale * LOG2E;
   float mx = -INFINITY, l = 0.f;
-  float o[NP][2][MT][4];
+  float o[NP][2][MO][4];
 #pragma unroll
   for (int i = 0; i < NP; ++i)
 #pragma unroll
     for (int e = 0; e < 2; ++e)
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) { o[i][e][mt][0] = o[i][e][mt][1] = o[i][e][mt][2] = o[i][e][mt][3] = 0.f; }
+      for (int mt = 0; mt < MO; ++mt) { o[i][e][mt][0] = o[i][e][mt][1] = o[i][e][mt][2] = o[i][e][mt][3] = 0.f; }
 
   bool ok = true;
   uint32_t phase = 0;
@@ -221,14 +222,20 @@ __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(Jo
     }
     __syncthreads();
     {
-      if (it > 0 && *moved == it)
+      if (it > 0 && *moved == it) {
+        float a[MT][2];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        const float a0 = sA[mt * 16 + g], a1 = sA[mt * 16 + g + 8];
+        for (int mt = 0; mt < MT; ++mt) { a[mt][0] = sA[mt * 16 + g]; a[mt][1] = sA[mt * 16 + g + 8]; }
 #pragma unroll
         for (int i = 0; i < NP; ++i)
 #pragma unroll
-          for (int e = 0; e < 2; ++e) { o[i][e][mt][0] *= a0; o[i][e][mt][1] *= a0; o[i][e][mt][2] *= a1; o[i][e][mt][3] *= a1; }
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int mo = 0; mo < MO; ++mo) {
+              const bool second = MT > 1 && (ONE ? hit >> ((i * 2 + e) * MT + 1) & 1 : mo > 0);
+              const float a0 = second ? a[MT - 1][0] : a[0][0], a1 = second ? a[MT - 1][1] : a[0][1];
+              o[i][e][mo][0] *= a0; o[i][e][mo][1] *= a0; o[i][e][mo][2] *= a1; o[i][e][mo][3] *= a1;
+            }
       }
 #pragma unroll
       for (int kk = 0; kk < BN / 16; ++kk) {
@@ -243,8 +250,8 @@ __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(Jo
           ldmatrix_x4_trans(vb, tv + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VPITCH + (pair * 2 + (lane >> 4)) * 8);
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
-            if (MT == 1 || (hit >> (i * 2 * MT + mt) & 1)) mma_bf16_16816(o[i][0][mt], pa[mt], vb[0], vb[1]);
-            if (MT == 1 || (hit >> ((i * 2 + 1) * MT + mt) & 1)) mma_bf16_16816(o[i][1][mt], pa[mt], vb[2], vb[3]);
+            if (MT == 1 || (hit >> (i * 2 * MT + mt) & 1)) mma_bf16_16816(o[i][0][mt % MO], pa[mt], vb[0], vb[1]);
+            if (MT == 1 || (hit >> ((i * 2 + 1) * MT + mt) & 1)) mma_bf16_16816(o[i][1][mt % MO], pa[mt], vb[2], vb[3]);
           }
         }
       }
@@ -290,7 +297,7 @@ __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(Jo
         for (int half = 0; half < 2; ++half) {
           const int r = mt * 16 + g + half * 8, h = h0 + r;
           if (h >= p.Hq || h / G != c) continue;
-          const float x = o[i][e][mt][half * 2], y = o[i][e][mt][half * 2 + 1];
+          const float x = o[i][e][mt % MO][half * 2], y = o[i][e][mt % MO][half * 2 + 1];
           if (partial) {
             *reinterpret_cast<float2*>(p.part_o + (size_t(split) * p.total_rows + size_t(tok) * p.Hq + h) * p.dv + col) = make_float2(x, y);
           } else {
@@ -302,7 +309,7 @@ __global__ void __launch_bounds__(AJ_WARPS * 32, CTAS) attention_joint_kernel(Jo
     }
 }
 
-template <int AJ_WARPS, int MT, int KSW, int NP, int BN, int CTAS>
+template <int AJ_WARPS, int MT, int KSW, int NP, int BN, int CTAS, bool ONE = false>
 static int LaunchJoint(const AttnParams& a, int max_q_len, cudaStream_t stream) {
   JointParams jp{};
   jp.a = a;
@@ -315,7 +322,7 @@ static int LaunchJoint(const AttnParams& a, int max_q_len, cudaStream_t stream) 
   jp.head_tiles = (a.Hq + rows - 1) / rows;
   const long long gx = (long long)max_q_len * jp.head_tiles;
   if (gx > 0x7fffffff) return -1;
-  auto kern = attention_joint_kernel<AJ_WARPS, MT, KSW, NP, BN, CTAS>;
+  auto kern = attention_joint_kernel<AJ_WARPS, MT, KSW, NP, BN, CTAS, ONE>;
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, 224 * 1024, configured)) return -3;
   if (!launch_pdl(kern, dim3(unsigned(gx), 1, a.B * a.splits), dim3(AJ_WARPS * 32), size_t(jp.stages) * stage + rest, stream, jp)) return -4;
@@ -368,6 +375,7 @@ OGB_API int ogb_attention_joint(const OgbAttnLayer* l, const void* q, int q_stri
   auto s = static_cast<cudaStream_t>(stream_);
   const int cols = max(p.dk, p.Hkv * p.dv);
   const bool one = p.Hq <= 16;
+  if (cols > 512 && !one && 16 % (p.Hq / p.Hkv) == 0) return LaunchJoint<16, 2, 4, 4, 16, 1, true>(p, max_q_len, s);
   if (cols > 512) return one ? LaunchJoint<8, 1, 8, 8, 16, 1>(p, max_q_len, s) : LaunchJoint<16, 2, 4, 4, 16, 1>(p, max_q_len, s);
   if (cols <= 256) return one ? LaunchJoint<4, 1, 4, 4, 32, 2>(p, max_q_len, s) : LaunchJoint<4, 2, 4, 4, 32, 2>(p, max_q_len, s);
   // few CTAs: taller tiles, one CTA per SM; else two, whose phases overlap (64 requests: 46.5 us against 50.1, 16 requests: 27.7 against 26.1)

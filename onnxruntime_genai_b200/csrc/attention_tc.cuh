@@ -88,12 +88,14 @@ struct TcAttnParams {
 // entry of a query row in a grid of key vectors
 __device__ __forceinline__ int tca_query(int kvh, int i, int G, int maps) { return maps > 1 ? ((kvh / maps) * G + i) * maps + kvh % maps : kvh * G + i; }
 
-// KC: key columns of a ring slot (DK, or a part of it where whole tiles of wide keys would not fit twice beside the queries).
-template <int DK, int DV, int BN, int KC = DK>
+// KC: key columns of a ring slot (DK, or a part of it where whole tiles of wide keys would not fit twice beside the queries).  QR: query rows of a tile, 128, or
+// 64 where 128 rows of queries would not leave room for the rings: the lower half of the accumulators then belongs to no row (as operand rows 64 .. 127
+// the MMA reads whatever follows 64 rows in shared memory; rows do not mix).
+template <int DK, int DV, int BN, int KC = DK, int QR = TCA_BM>
 struct TcaCfg {
   static constexpr int K_PARTS = DK / KC, K_HALVES = KC / 64, V_HALVES = DV / 64;
-  static_assert(DK % KC == 0, "a key row is whole parts");
-  static constexpr int Q_BYTES = TCA_BM * DK * 2;
+  static_assert(DK % KC == 0 && (QR == 64 || QR == TCA_BM), "a key row is whole parts");
+  static constexpr int Q_BYTES = QR * DK * 2, Q_HALF = QR * 128;      // 64 columns of the rows
   static constexpr int K_TILE = BN * KC * 2, V_TILE = BN * DV * 2;
   // K and V tiles have rings of their own: a K tile is free as soon as its Q K^T is done (one tile period earlier than the
   // V tile of the same keys), and the loads must run two to three tile periods ahead of their use to hide their latency.
@@ -147,16 +149,16 @@ __device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.p
 // are the unrotated part; MIX: heads of p.dk and p.dv columns (multiples of 8).  The boxes of a head narrower than the staged rows reach
 // into the next head's columns, which meet zeros in Q (keys) or give output columns that are not stored (values).  CAP: scores are soft-capped
 // (a kernel of its own: the loop body of the others has to stay within the instruction cache).
-template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false, bool CAP = false, int KC = DK>
-__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN, KC>::CTAS_PER_SM)
+template <int DK, int DV, int BN, bool LAT = false, int NOPE = DK, bool MIX = false, bool CAP = false, int KC = DK, int QR = TCA_BM>
+__global__ void __launch_bounds__(TCA_THREADS, TcaCfg<DK, DV, BN, KC, QR>::CTAS_PER_SM)
 attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_r,
                     TcAttnParams p) {
-  using Cfg = TcaCfg<DK, DV, BN, KC>;
+  using Cfg = TcaCfg<DK, DV, BN, KC, QR>;
   static_assert(KC == DK || (MIX && !LAT), "keys in parts: only layers with sizes of their own");
   constexpr int KS = Cfg::K_STAGES, VS = Cfg::V_STAGES;
   extern __shared__ __align__(128) uint8_t smem_dyn[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~uintptr_t(1023));
-  uint8_t* sQ = smem;                                  // [HALVES][128 rows][128 B]
+  uint8_t* sQ = smem;                                  // [HALVES][QR rows][128 B]
   uint8_t* sK = sQ + Cfg::Q_BYTES;                     // [KS][HALVES][BN keys][128 B]
   uint8_t* sV = sK + KS * Cfg::K_TILE;                 // [VS][HALVES][BN keys][128 B]
   __shared__ uint64_t k_full[KS], k_empty[KS], v_full[VS], v_empty[VS], s_full[Cfg::S_BUFS], p_full[Cfg::S_BUFS], o_done[Cfg::S_BUFS], q_full;
@@ -175,13 +177,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   const int rows = q_len * G;
   // CTAs are dispatched in block-index order: the last row tiles of a causal prompt see the most keys, so they go first and
   // the tail of the grid is made of short CTAs
-  const int row0 = int(gridDim.x - 1 - blockIdx.x) * TCA_BM;
+  const int row0 = int(gridDim.x - 1 - blockIdx.x) * QR;
   if (rows * (MIX ? p.maps : 1) < p.min_rows || row0 >= rows) return;      // before anything is allocated
   if (LAT && p.lat.row_base[b] < 0) return;
   const int past = p.past_lens[b];
   const bool full = p.window < 0;
   const int32_t* table = p.block_table + size_t(b) * p.table_cols;
-  const int last_tq = min(q_len - 1, (row0 + TCA_BM - 1) / G);
+  const int last_tq = min(q_len - 1, (row0 + QR - 1) / G);
   const int kv_hi = full ? past : past + last_tq + 1;
   int kv_lo = 0;
   if (p.window > 0) kv_lo = max(0, past + row0 / G - p.window + 1);
@@ -292,10 +294,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
         if (!mbar_wait_bounded(&k_full[st], (n / KS) & 1, abort_p)) return false;
         tc_fence_after();
         if (lane == 0) {
-          const uint32_t k_addr = k_ring + st * Cfg::K_TILE, q_part = q_addr + part * (KC / 64) * (TCA_BM * 128);
+          const uint32_t k_addr = k_ring + st * Cfg::K_TILE, q_part = q_addr + part * (KC / 64) * Cfg::Q_HALF;
 #pragma unroll
           for (int ks = 0; ks < KC / 16; ++ks) {
-            const uint64_t da = umma_desc_sw128(q_part + (ks >> 2) * (TCA_BM * 128) + (ks & 3) * 32);
+            const uint64_t da = umma_desc_sw128(q_part + (ks >> 2) * Cfg::Q_HALF + (ks & 3) * 32);
             const uint64_t db = umma_desc_sw128(k_addr + (ks >> 2) * (BN * 128) + (ks & 3) * 32);
             umma_f16(tmem_base + (it % Cfg::S_BUFS) * Cfg::S_COLS, da, db, idesc_qk, part > 0 || ks > 0);
           }
@@ -339,7 +341,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     const int quarter = warp & 3, half = warp >> 2;
     const int r = quarter * 32 + lane;
     const int gr = row0 + r;
-    const bool valid = gr < rows;
+    const bool valid = gr < rows && (QR == TCA_BM || r < QR);
     const int tq = valid ? gr / G : q_len - 1;
     const int hq = MIX ? tca_query(kvh, valid ? gr % G : 0, G, p.maps) : kvh * G + (valid ? gr % G : 0);
     const int qpos = past + tq;
@@ -359,7 +361,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           const int col = c * 8 < NOPE ? c * 8 : c * 8 - NOPE, width = c * 8 < NOPE ? p.lat.dim : p.lat.rot;
           if (valid && col < width) v = *reinterpret_cast<const uint4*>(src + (c * 8 < NOPE ? col : p.lat.dim + col));
         } else if (valid && (!MIX || c * 8 < p.dk)) v = *reinterpret_cast<const uint4*>(src + c * 8);
-        *reinterpret_cast<uint4*>(sQ + (c >> 3) * (TCA_BM * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+        if (QR == TCA_BM || r < QR) *reinterpret_cast<uint4*>(sQ + (c >> 3) * Cfg::Q_HALF + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
       }
       fence_proxy_async_smem();
       mbar_arrive(&q_full);
@@ -369,7 +371,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     const float inv_cap = CAP ? p.scale / p.softcap : 0.f, capl = p.softcap * TCA_LOG2E;
     // a tile every key of which every row of this lane quarter sees needs no masks
     const int wq_lo = past + min(q_len - 1, (row0 + quarter * 32) / G), wq_hi = past + min(q_len - 1, (row0 + quarter * 32 + 31) / G);
-    const bool rows_full = row0 + quarter * 32 + 31 < rows;
+    const bool rows_full = row0 + quarter * 32 + 31 < rows && quarter * 32 < QR;
     auto tile_interior = [&](int it) {
       const int j0 = (tile_begin + it) * BN;
       return j0 >= kv_lo && j0 + BN <= kv_hi && (full || j0 + BN - 1 <= wq_lo) && (p.window <= 0 || j0 > wq_hi - p.window) &&
@@ -571,10 +573,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   if (warp == TCA_K_WARP) tmem_dealloc(tmem_base, Cfg::TMEM_COLS);
 }
 
-template <int DK, int DV, int BN, bool MIX, bool CAP, int KC = DK>
+template <int DK, int DV, int BN, bool MIX, bool CAP, int KC = DK, int QR = TCA_BM>
 static int LaunchTcForm(const TcAttnParams& p, const void* k_cache, const void* v_cache, int max_q_len, int cache_slots, cudaStream_t stream) {
-  using Cfg = TcaCfg<DK, DV, BN, KC>;
-  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP, KC>;
+  using Cfg = TcaCfg<DK, DV, BN, KC, QR>;
+  auto kern = attention_tc_kernel<DK, DV, BN, false, DK, MIX, CAP, KC, QR>;
   const int kw = MIX && p.joint ? p.dk : p.Hkv * (MIX ? p.dk : DK), vw = MIX ? p.Hkv / p.maps * p.dv : p.Hkv * DV;      // row widths of the caches
   static bool configured[OGB_MAX_DEVICES] = {};
   if (!set_max_dyn_smem(kern, Cfg::SMEM, configured)) return -3;
@@ -584,7 +586,7 @@ static int LaunchTcForm(const TcAttnParams& p, const void* k_cache, const void* 
   if (!MakeMapBf16(&mk, k_cache, cache_slots, kw, kw, 16)) return -2;
   if (!MakeMapBf16(&mv, v_cache, cache_slots, vw, vw, 16)) return -2;
   const int G = p.Hq / p.Hkv;
-  dim3 grid((max_q_len * G + TCA_BM - 1) / TCA_BM, p.Hkv, p.B);
+  dim3 grid((max_q_len * G + QR - 1) / QR, p.Hkv, p.B);
   launch_pdl(kern, grid, dim3(TCA_THREADS), Cfg::SMEM, stream, mk, mv, mv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -1,6 +1,6 @@
 // Prefill attention on the tensor cores (attention_tc.cuh) for layers whose heads have sizes of their own: queries and keys of dk columns
-// staged as 64, 128, 192 or 256, values of dv columns staged as 64, 128 or 256.  Joint layers (a query meets the keys of all key heads) also with keys of up to 512
-// columns, which arrive in parts of 128.
+// staged as 64, 128, 192 or 256, values of dv columns staged as 64, 128 or 256.  Joint layers (a query meets the keys of all key heads) also with keys of up to 1024
+// columns, which arrive in parts of 128 (beyond 512 columns to tiles of 64 query rows).
 #include "attention_tc.cuh"
 
 namespace ogb {
@@ -22,8 +22,9 @@ static int LaunchTcMixedKeys(const TcAttnParams& p, const void* k, const void* v
 
 template <int DK, int DV>
 static int LaunchTcWide(const TcAttnParams& p, const void* k, const void* v, int max_q_len, int cache_slots, cudaStream_t s) {
-  return p.softcap > 0.f ? LaunchTcForm<DK, DV, 64, true, true, 128>(p, k, v, max_q_len, cache_slots, s)
-                         : LaunchTcForm<DK, DV, 64, true, false, 128>(p, k, v, max_q_len, cache_slots, s);
+  constexpr int QR = DK <= 512 ? TCA_BM : 64;
+  return p.softcap > 0.f ? LaunchTcForm<DK, DV, 64, true, true, 128, QR>(p, k, v, max_q_len, cache_slots, s)
+                         : LaunchTcForm<DK, DV, 64, true, false, 128, QR>(p, k, v, max_q_len, cache_slots, s);
 }
 template <int DK>
 static int LaunchTcWideKeys(const TcAttnParams& p, const void* k, const void* v, int max_q_len, int cache_slots, cudaStream_t s) {
@@ -37,7 +38,7 @@ static int LaunchTcWideKeys(const TcAttnParams& p, const void* k, const void* v,
 using namespace ogb;
 
 OGB_API int ogb_attention_tc_joint_supported(int dk, int dv, int block_size, int cache_slots) {
-  return dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && dk <= 512 && dv <= 256 && block_size % 16 == 0 && cache_slots >= 16;
+  return dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && dk <= 1024 && dv <= 256 && block_size % 16 == 0 && cache_slots >= 16;
 }
 
 OGB_API int ogb_attention_tc_mixed_supported(int dk, int dv, int block_size, int cache_slots) {
@@ -81,5 +82,7 @@ OGB_API int ogb_attention_tc_mixed(const OgbAttnLayer* a, const void* q, int q_s
   if (p.dk <= 192) return LaunchTcMixedKeys<192>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 256) return LaunchTcMixedKeys<256>(p, k_cache, v_cache, max_q_len, cache_slots, s);
   if (p.dk <= 384) return LaunchTcWideKeys<384>(p, k_cache, v_cache, max_q_len, cache_slots, s);
-  return LaunchTcWideKeys<512>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  if (p.dk <= 512) return LaunchTcWideKeys<512>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  if (p.dk <= 768) return LaunchTcWideKeys<768>(p, k_cache, v_cache, max_q_len, cache_slots, s);
+  return LaunchTcWideKeys<1024>(p, k_cache, v_cache, max_q_len, cache_slots, s);
 }

@@ -571,7 +571,8 @@ __global__ void __launch_bounds__(256) qkv_prep_mixed_kernel(const T* __restrict
 }
 
 // The same where every part is whole pieces of 8 columns (dim = key_row, rot / 2, value_row) and a head at most 32 pieces: LPH lanes per head (a power of two),
-// one piece each, norms and the partners of a rotation by shuffles; then a thread mixes a piece of a key head's queries into four heads at a time.
+// one piece each, norms and the partners of a rotation by shuffles; then a thread mixes a piece of a key head's queries into four heads at a time.  Steps of few
+// tokens: the CTAs (t, y) of a token have `per_cta` key heads each, with their queries and values.
 template <typename T> __device__ __forceinline__ void store8(T* dst, const float (&v)[8]) {
   if constexpr (sizeof(T) == 4) {
     reinterpret_cast<float4*>(dst)[0] = make_float4(v[0], v[1], v[2], v[3]);
@@ -583,23 +584,28 @@ template <typename T> __device__ __forceinline__ void store8(T* dst, const float
 
 template <typename T>
 __global__ void __launch_bounds__(256) qkv_prep_mixed_pieces_kernel(const T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, QkvPrep p,
-                                                                    const float* __restrict__ talk, T* __restrict__ mixed, int LPH) {
+                                                                    const float* __restrict__ talk, T* __restrict__ mixed, int LPH,
+                                                                    int per_cta) {
   extern __shared__ __align__(16) float sm[];
-  float* sq = sm;                            // [Hq][dim]
-  float* st = sm + p.Hq * p.dim;             // [Hq][Hq]
+  const int G = p.Hq / p.Hkv, c0 = blockIdx.y * per_cta, nc = min(per_cta, p.Hkv - c0), q0 = c0 * G, nq = nc * G;      // key heads and queries of this CTA
+  float* sq = sm;                            // [nq][dim]
+  float* st = sm + nq * p.dim;               // [Hq][nq]
   pdl_launch_dependents();
-  for (int i = threadIdx.x; i < p.Hq * p.Hq; i += blockDim.x) st[i] = talk[i];
+  if (nq == p.Hq)
+    for (int i = threadIdx.x; i < p.Hq * nq; i += blockDim.x) st[i] = talk[i];
+  else
+    for (int i = threadIdx.x; i < p.Hq * nq; i += blockDim.x) st[i] = talk[i / nq * p.Hq + q0 + i % nq];
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, dim = p.dim, half = p.rot >> 1, turn = half / 8;
   const T* row = proj + size_t(t) * p.ldp;
-  const int slot = p.slots[t], heads = p.Hq + p.Hkv;
+  const int slot = p.slots[t], heads = nq + nc;
   const size_t at = size_t(min(max(p.positions[t], 0), p.max_pos - 1)) * half;
   const int l = tid % LPH, per = blockDim.x / LPH;
   for (int h0 = 0; h0 < heads; h0 += per) {
     const int head = h0 + tid / LPH;
-    const bool is_q = head < p.Hq, live = head < heads && l * 8 < dim;
+    const bool is_q = head < nq, live = head < heads && l * 8 < dim;
     float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (live) load8(row + size_t(head) * dim + l * 8, f);
+    if (live) load8(row + size_t(is_q ? q0 + head : p.Hq + c0 + head - nq) * dim + l * 8, f);
     const float* w = is_q ? p.q_norm : p.k_norm;
     if (p.q_norm || p.k_norm) {
       float ss = 0.f;
@@ -630,17 +636,17 @@ __global__ void __launch_bounds__(256) qkv_prep_mixed_pieces_kernel(const T* __r
     }
     if (live) {
       if (is_q) store8(sq + head * dim + l * 8, f);
-      else if (slot >= 0) store8(k_cache + (size_t(slot) * p.Hkv + (head - p.Hq)) * dim + l * 8, f);
+      else if (slot >= 0) store8(k_cache + (size_t(slot) * p.Hkv + c0 + head - nq) * dim + l * 8, f);
     }
   }
   if (slot >= 0)
-    for (int i = tid; i < p.Hv * p.value_row / 8; i += blockDim.x) {
+    for (int i = blockIdx.y * blockDim.x + tid; i < p.Hv * p.value_row / 8; i += gridDim.y * blockDim.x) {
       float f[8];
-      load8(row + size_t(heads) * dim + i * 8, f);
+      load8(row + size_t(p.Hq + p.Hkv) * dim + i * 8, f);
       store8(v_cache + size_t(slot) * p.Hv * p.value_row + i * 8, f);
     }
   __syncthreads();
-  const int G = p.Hq / p.Hkv, dp = dim / 8, items = p.Hkv * dp;      // item: (key head, piece)
+  const int dp = dim / 8, items = nc * dp;      // item: (key head, piece)
   T* out = mixed + size_t(t) * p.Hq * p.Hkv * dim;
   for (int i = tid; i < (p.Hq + 3) / 4 * items; i += blockDim.x) {
     const int hb = i / items * 4, item = i % items, c = item / dp, d = (item - c * dp) * 8;
@@ -650,14 +656,14 @@ __global__ void __launch_bounds__(256) qkv_prep_mixed_pieces_kernel(const T* __r
       load8<float>(sq + (c * G + g) * dim + d, q);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float m = hb + j < p.Hq ? st[(hb + j) * p.Hq + c * G + g] : 0.f;
+        const float m = hb + j < p.Hq ? st[(hb + j) * nq + c * G + g] : 0.f;
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[j][e] = fmaf(m, q[e], acc[j][e]);
       }
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (hb + j < p.Hq) store8(out + (size_t(hb + j) * p.Hkv + c) * dim + d, acc[j]);
+      if (hb + j < p.Hq) store8(out + (size_t(hb + j) * p.Hkv + c0 + c) * dim + d, acc[j]);
   }
 }
 
@@ -868,10 +874,12 @@ OGB_API int ogb_qkv_prep(void* proj, int ldp, int Hq, int Hkv, int Hv, int dim, 
       static bool p32[OGB_MAX_DEVICES] = {}, p16[OGB_MAX_DEVICES] = {};
       using B = __nv_bfloat16;
       if (fp32 ? !set_max_dyn_smem(qkv_prep_mixed_pieces_kernel<float>, 200 * 1024, p32) : !set_max_dyn_smem(qkv_prep_mixed_pieces_kernel<B>, 200 * 1024, p16)) return -3;
-      return (fp32 ? launch_pdl(qkv_prep_mixed_pieces_kernel<float>, dim3(T), block, smem, s, static_cast<const float*>(proj), static_cast<float*>(k_cache),
-                                static_cast<float*>(v_cache), p, talk, static_cast<float*>(mixed), lph)
-                   : launch_pdl(qkv_prep_mixed_pieces_kernel<B>, dim3(T), block, smem, s, static_cast<const B*>(proj), static_cast<B*>(k_cache),
-                                static_cast<B*>(v_cache), p, talk, static_cast<B*>(mixed), lph)) ? 0 : -4;
+      const int parts = T >= 1200 ? 1 : (1200 / T < Hkv ? 1200 / T : Hkv), per = (Hkv + parts - 1) / parts;      // (256 tokens: 9.2 us; in one part 14)
+      const dim3 g2(T, (Hkv + per - 1) / per);
+      return (fp32 ? launch_pdl(qkv_prep_mixed_pieces_kernel<float>, g2, block, smem, s, static_cast<const float*>(proj), static_cast<float*>(k_cache),
+                                static_cast<float*>(v_cache), p, talk, static_cast<float*>(mixed), lph, per)
+                   : launch_pdl(qkv_prep_mixed_pieces_kernel<B>, g2, block, smem, s, static_cast<const B*>(proj), static_cast<B*>(k_cache),
+                                static_cast<B*>(v_cache), p, talk, static_cast<B*>(mixed), lph, per)) ? 0 : -4;
     }
     static bool done32[OGB_MAX_DEVICES] = {}, done16[OGB_MAX_DEVICES] = {};
     if (fp32) {

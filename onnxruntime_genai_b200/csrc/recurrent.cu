@@ -3,7 +3,7 @@
 // the recurrences are plain fp32.
 //
 // Gated average, every column on its own:   z = sigmoid(z'),  c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0),  S <- (1 - z) S + z c,  out = S * silu(g) * scale.
-//   min_gru_step_kernel   decode-shaped steps: a thread walks the tokens of its columns.
+//   min_gru_step_kernel   decode-shaped steps: a thread walks the tokens of one column, or of four.
 //   min_gru_chunk_kernel  prompts, in two passes over chunks of tokens: what a chunk does to a state is an affine function per column; the second pass
 //                         applies the functions of the chunks before its own to the first state and walks its tokens.
 //
@@ -57,22 +57,52 @@ struct MinGruParams {
 
 template <typename T> __device__ __forceinline__ float mg_candidate(float u) { return u >= 0.f ? u + 0.5f : rec_gate<T>(u); }
 
-template <typename T>
+template <int N> __device__ __forceinline__ void rec_load(const float* p, float (&v)[N]) {
+  if constexpr (N == 4) { const float4 f = *reinterpret_cast<const float4*>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+  else v[0] = *p;
+}
+template <int N> __device__ __forceinline__ void rec_load(const __nv_bfloat16* p, float (&v)[N]) {
+  if constexpr (N == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  } else v[0] = bf2f(*p);
+}
+template <int N> __device__ __forceinline__ void rec_store(float* p, const float (&v)[N]) {
+  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+template <int N> __device__ __forceinline__ void rec_store(__nv_bfloat16* p, const float (&v)[N]) {
+  if constexpr (N == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  else *p = f2bf(v[0]);
+}
+
+// A thread has N neighbouring columns (N = 4: everything on boundaries of four).
+template <typename T, int N>
 __global__ void __launch_bounds__(128) min_gru_step_kernel(MinGruParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int b = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int b = blockIdx.y, c = (blockIdx.x * blockDim.x + threadIdx.x) * N;
   const int t0 = p.cu_seqlens[b], t1 = p.cu_seqlens[b + 1];
   if (c >= p.W || t0 >= t1) return;
   float* st = p.state + size_t(p.slots[b]) * p.slot_stride + c;
   const T *z = static_cast<const T*>(p.z) + c, *x = static_cast<const T*>(p.x) + c, *g = static_cast<const T*>(p.g) + c;
-  float S = p.past_lens[b] == 0 ? 0.f : *st;
+  float S[N] = {};
+  if (p.past_lens[b] != 0) rec_load(st, S);
   for (int t = t0; t < t1; ++t) {
-    const float zz = rec_gate<T>(rec_f32(z[size_t(t) * p.ld])), gg = rec_f32(g[size_t(t) * p.ld]);
-    S = fmaf(zz, mg_candidate<T>(rec_f32(x[size_t(t) * p.ld])), (1.f - zz) * S);
-    static_cast<T*>(p.out)[size_t(t) * p.ldo + c] = rec_from<T>(S * gg * rec_gate<T>(gg) * p.scale);
+    float zz[N], u[N], gg[N], o[N];
+    rec_load(z + size_t(t) * p.ld, zz);
+    rec_load(x + size_t(t) * p.ld, u);
+    rec_load(g + size_t(t) * p.ld, gg);
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      const float a = rec_gate<T>(zz[e]);
+      S[e] = fmaf(a, mg_candidate<T>(u[e]), (1.f - a) * S[e]);
+      o[e] = S[e] * gg[e] * rec_gate<T>(gg[e]) * p.scale;
+    }
+    rec_store(static_cast<T*>(p.out) + size_t(t) * p.ldo + c, o);
   }
-  *st = S;
+  rec_store(st, S);
 }
 
 // Prompts, in chunks of MG_L tokens.  Pass 1: what a chunk does to a state, S -> A S + D, per column; the state before the request's first token is kept beside
@@ -757,8 +787,11 @@ OGB_API int ogb_min_gru(const void* z, const void* x, const void* g, int ld, flo
   const bool even = W % 2 == 0 && ld % 2 == 0 && ldo % 2 == 0 && ((addr(z) | addr(x) | addr(g) | addr(out)) & (fp32 ? 7 : 3)) == 0;
   using H = __nv_bfloat16;
   if (!scratch || !even) {
-    const dim3 grid((W + 127) / 128, B), block(128);
-    return (fp32 ? launch_pdl(min_gru_step_kernel<float>, grid, block, 0, s, p) : launch_pdl(min_gru_step_kernel<H>, grid, block, 0, s, p)) ? 0 : -4;
+    const bool four = W % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && slot_stride % 4 == 0 && (addr(state) & 15) == 0 &&
+                      ((addr(z) | addr(x) | addr(g) | addr(out)) & (fp32 ? 15 : 7)) == 0;
+    const dim3 grid(four ? (W / 4 + 127) / 128 : (W + 127) / 128, B), block(128);
+    if (four) return (fp32 ? launch_pdl(min_gru_step_kernel<float, 4>, grid, block, 0, s, p) : launch_pdl(min_gru_step_kernel<H, 4>, grid, block, 0, s, p)) ? 0 : -4;
+    return (fp32 ? launch_pdl(min_gru_step_kernel<float, 1>, grid, block, 0, s, p) : launch_pdl(min_gru_step_kernel<H, 1>, grid, block, 0, s, p)) ? 0 : -4;
   }
   if (scratch_bytes < ogb_min_gru_scratch_bytes(T, B, W) || (addr(scratch) & 15)) return -2;
   auto* maps = static_cast<float4*>(scratch);

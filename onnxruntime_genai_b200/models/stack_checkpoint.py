@@ -84,8 +84,8 @@ def load_stack_decoder(model_dir: str, filename: str, context_length: int, devic
 def build_stack_decoder(arch: ArchConfig, get: Callable[[str], torch.Tensor], device, dtype) -> DecoderModel:
     """DecoderModel from a tensor source: input projections stacked per layer, the key map transposed per head, the output projections
     of both sub-layers of a parallel block joined side by side, the factors on a sub-layer's normed output multiplied into one vector,
-    experts stacked, two mixers' input projections joined where they stand side by side, heads and feed-forwards filled up with zeros where a kernel wants whole tiles, small vectors and recurrence constants
-    in fp32."""
+    experts stacked, two mixers' input projections joined where they stand side by side, heads and feed-forwards filled up with zeros where a
+    kernel wants whole tiles, small vectors and recurrence constants in fp32."""
     shapes = stack_weight_shapes(arch)
     model = DecoderModel(arch, device, dtype)
     cuda = torch.device(device).type == "cuda"

@@ -933,11 +933,13 @@ def choose_kv_splits(batch: int, Hkv: int, max_q_len: int, max_kv_len: int, sm_c
     return int(splits), int(chunk)
 
 
-def choose_joint_splits(batch: int, Hq: int, max_q_len: int, span: int) -> int:
-    """Key splits of a launch for heads whose scores are mixed (one CTA per token and 32 heads).  Measured on B200 with requests of 192..2112 keys, 4 key heads
-    of 128: 1 request 16 splits 18.4 us, 16 requests 12 splits 26.1 us, 64 requests 6 splits 46.5 us (4: 50), 256 requests 2 splits 116 us (1: 137)."""
+def choose_joint_splits(batch: int, Hq: int, max_q_len: int, span: int, cols: int) -> int:
+    """Key splits of a launch for heads whose scores are mixed (one CTA per token and 32 heads; rows of `cols` columns).  Measured on B200 with requests of
+    192..2112 keys, 4 key heads of 128: 1 request 16 splits 18.4 us, 16 requests 12 splits 26.1 us, 64 requests 6 splits 46.5 us (4: 50), 256 requests
+    2 splits 116 us (1: 137).  8 key heads of 128 (one CTA per SM): 16 requests 12 splits 48 us, 64 requests 4 splits 102 us (6: 117), 256 in one 311 us
+    (2: 335)."""
     ctas = max(1, batch * max_q_len * ((Hq + 31) // 32))
-    return max(1, min(int(round((200 if ctas <= 32 else 400) / ctas)), span // 32, 16))
+    return max(1, min(int(round((200 if ctas <= 32 else (400 if cols <= 512 else 256)) / ctas)), span // 32, 16))
 
 
 TC_ATTENTION_MIN_ROWS = 128      # query rows (tokens x heads of a GQA group) from which a request takes the tcgen05 prefill kernel
@@ -1071,7 +1073,7 @@ def _paged_attention_mixed(q, k_cache, v_cache, cu_seqlens, past_lens, block_tab
             if chunk > 0 or window > 0:
                 span = min(span, (chunk or window) + 63)
             if joint:
-                splits = choose_joint_splits(B, Hq, max_q_len, span)
+                splits = choose_joint_splits(B, Hq, max_q_len, span, max(dk, Hkv * dv))
             else:
                 splits = choose_kv_splits(B, Hkv, max_q_len, span, group=G, ordered=order is not None)
         sp, ch = splits if isinstance(splits, tuple) else (splits, 0)
@@ -1122,7 +1124,8 @@ MLSTM_LONG_TOKENS = 24      # requests that feed at least this many tokens run i
 
 def mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out, max_q_len=0, min_q_len=0):
     """Matrix memories over packed sequences (see csrc/recurrent.cu): proj [T, queries | keys | values | output gate], gates fp32 [T, input | forget logits],
-    their biases gate_b and the heads' norm weight fp32; state [slots, heads * (dim * vdim + dim + 1)] fp32, updated in place; out [T, heads * vdim].  max_q_len, min_q_len: most and fewest tokens a request feeds (0: unknown)."""
+    their biases gate_b and the heads' norm weight fp32; state [slots, heads * (dim * vdim + dim + 1)] fp32, updated in place; out [T, heads * vdim].
+    max_q_len, min_q_len: most and fewest tokens a request feeds (0: unknown)."""
     if not proj.is_cuda:
         return ref.mlstm(proj, gates, gate_b, heads, dim, vdim, cap, norm_w, eps, state, slots, cu_seqlens, past_lens, out)
     import ctypes

@@ -205,7 +205,7 @@ def test_mixed_queries_have_the_scores_of_mixed_heads(runtime, shape):
 
 # (heads, key heads, key and value columns): keys of all heads together from one 16-byte piece to more than any tensor-core form takes
 SHAPES = [(4, 2, 24, 16), (3, 3, 16, 8), (6, 2, 128, 72), (8, 1, 64, 128), (4, 2, 128, 128), (8, 4, 128, 128), (4, 4, 64, 64), (16, 4, 128, 64), (10, 5, 8, 40), (20, 1, 40, 40),
-          (32, 4, 64, 64), (12, 3, 136, 24), (16, 8, 128, 32), (2, 2, 32, 264)]
+          (32, 4, 64, 64), (12, 3, 136, 24), (16, 8, 128, 32), (2, 2, 32, 264), (32, 8, 80, 64), (18, 6, 128, 136)]
 
 
 def _attention_case(shape, lens, window, seed, dt, needles=(), loud=1.0):
